@@ -437,7 +437,8 @@ void paged_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
                   int64_t max_splits, int64_t window, double scale,
                   const c10::optional<Tensor>& status, const c10::optional<Tensor>& page_ml,
                   const c10::optional<Tensor>& block_mass, const c10::optional<Tensor>& q8,
-                  const c10::optional<Tensor>& q8_d, const c10::optional<Tensor>& q8_s) {
+                  const c10::optional<Tensor>& q8_d, const c10::optional<Tensor>& q8_s, int64_t keep_first, int64_t out_d,
+                  bool exact_p) {
   TORCH_CHECK(q.dim() == 3 && k_cache.dim() == 4, "paged_decode: q [B,Hq,D], cache [blk,Hkv,16,D]");
   TORCH_CHECK(k_cache.size(2) == 16, "paged_decode: 16-token pages");
   oxb::DecodeAttnParams p{};
@@ -463,6 +464,11 @@ void paged_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
   TORCH_CHECK(part_o.numel() >= batch * p.Hq * max_splits * D, "paged_decode: part_o too small");
   TORCH_CHECK(part_ml.numel() >= batch * p.Hq * max_splits * 2, "paged_decode: part_ml too small");
   p.window = static_cast<int>(window);
+  p.keep_first = window > 0 ? static_cast<int>(keep_first) : 0;
+  p.out_d = static_cast<int>(out_d);
+  p.exact_p = exact_p ? 1 : 0;
+  TORCH_CHECK(out_d >= 0 && out_d <= D, "paged_decode: out_d");
+  TORCH_CHECK(!(page_ml.has_value() && (keep_first > 0 || exact_p)), "paged_decode: block mass goes with the plain window");
   p.scale_log2 = static_cast<float>(scale * 1.4426950408889634);
   p.status = opt_ptr<int>(status);  // given only when bounds checking is on
   p.num_blocks = p.status != nullptr ? static_cast<int>(k_cache.size(0)) : 0;
@@ -495,7 +501,7 @@ void paged_prefill_tc(const Tensor& q, const Tensor& k_cache, const Tensor& v_ca
                       const Tensor& block_tables, const Tensor& tile_seq, const Tensor& tile_q0,
                       const Tensor& q_start, const Tensor& q_lens, const Tensor& ctx_lens,
                       const Tensor& out, int64_t n_tiles, int64_t window, double scale,
-                      const Tensor& status) {
+                      const Tensor& status, int64_t keep_first, int64_t out_d, bool exact_p) {
   TORCH_CHECK(q.dim() == 3 && k_cache.dim() == 4, "paged_prefill_tc: q [T,Hq,D], cache [blk,Hkv,16,D]");
   TORCH_CHECK(k_cache.is_contiguous() && v_cache.is_contiguous(), "paged_prefill_tc: contiguous caches");
   oxb::PrefillAttnParams p{};
@@ -518,6 +524,10 @@ void paged_prefill_tc(const Tensor& q, const Tensor& k_cache, const Tensor& v_ca
   p.Hq = static_cast<int>(q.size(1));
   p.Hkv = static_cast<int>(k_cache.size(1));
   p.window = static_cast<int>(window);
+  p.keep_first = window > 0 ? static_cast<int>(keep_first) : 0;
+  p.out_d = static_cast<int>(out_d);
+  p.exact_p = exact_p ? 1 : 0;
+  TORCH_CHECK(out_d >= 0 && out_d <= D, "paged_prefill_tc: out_d");
   p.scale_log2 = static_cast<float>(scale * 1.4426950408889634);
   const uint64_t T = q.size(0);
   const uint64_t kv_rows = static_cast<uint64_t>(k_cache.size(0)) * p.Hkv * 16;
@@ -745,7 +755,7 @@ std::tuple<Tensor, int64_t> alloc_mapped_host(int64_t n_words) {
 void advance_decode_step(const Tensor& token_ids, const Tensor& positions, const Tensor& slot_mapping,
                          const Tensor& seq_lens, const Tensor& block_tables, const Tensor& sampled,
                          int64_t mailbox_dev, const Tensor& step_counter, int64_t rows, int64_t ring,
-                         const c10::optional<Tensor>& status) {
+                         const c10::optional<Tensor>& status, const c10::optional<Tensor>& prev_ids) {
   TORCH_CHECK(token_ids.is_cuda() && token_ids.scalar_type() == at::kInt && positions.scalar_type() == at::kInt &&
                   slot_mapping.scalar_type() == at::kLong && seq_lens.scalar_type() == at::kInt &&
                   block_tables.scalar_type() == at::kInt && sampled.scalar_type() == at::kInt &&
@@ -759,6 +769,10 @@ void advance_decode_step(const Tensor& token_ids, const Tensor& positions, const
   TORCH_CHECK(mailbox_dev != 0 && ring > 0, "advance_decode_step: mailbox");
   oxb::AdvanceStepParams p{};
   p.token_ids = token_ids.data_ptr<int>();
+  if (prev_ids.has_value() && prev_ids->defined()) {
+    TORCH_CHECK(prev_ids->scalar_type() == at::kInt && prev_ids->numel() >= rows, "advance_decode_step: prev_ids");
+    p.prev_ids = prev_ids->data_ptr<int>();
+  }
   p.positions = positions.data_ptr<int>();
   p.slot_mapping = reinterpret_cast<long long*>(slot_mapping.data_ptr<int64_t>());
   p.seq_lens = seq_lens.data_ptr<int>();

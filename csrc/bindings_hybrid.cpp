@@ -1,0 +1,325 @@
+// Python bindings of the layer-list kernels (torch extension `oxb_hybrid`). Every function launches on
+// torch's current CUDA stream and allocates nothing. The argument checks cover what the kernels index with.
+#include <ATen/cuda/CUDAContext.h>
+#include <cuda_runtime.h>
+#include <torch/extension.h>
+
+#include "common/device_info.h"
+#include "kernels/hybrid.cuh"
+
+namespace py = pybind11;
+using torch::Tensor;
+using OptTensor = c10::optional<Tensor>;
+
+namespace {
+
+cudaStream_t cur_stream() { return at::cuda::getCurrentCUDAStream().stream(); }
+
+void check_launch(cudaError_t e, const char* what) {
+  const cudaError_t last = cudaGetLastError();
+  if (e == cudaSuccess) e = last;
+  TORCH_CHECK(e == cudaSuccess, "oxb: launch of ", what, " failed: ", cudaGetErrorString(e));
+}
+
+int dtype_code(const Tensor& t, const char* what) {
+  TORCH_CHECK(t.is_cuda() && (t.scalar_type() == torch::kBFloat16 || t.scalar_type() == torch::kFloat32), what,
+              ": CUDA bf16 or fp32 expected");
+  return t.scalar_type() == torch::kBFloat16 ? 0 : 1;
+}
+bool given(const OptTensor& t) { return t.has_value() && t->defined(); }
+
+const float* f32(const Tensor& t, int64_t need, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.scalar_type() == torch::kFloat32 && t.numel() >= need && t.is_contiguous(), what,
+              ": contiguous CUDA fp32 of at least ", need, " values expected");
+  return t.data_ptr<float>();
+}
+const float* f32(const OptTensor& t, int64_t need, const char* what) { return given(t) ? f32(*t, need, what) : nullptr; }
+const int* i32(const Tensor& t, int64_t need, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.scalar_type() == torch::kInt32 && t.numel() >= need && t.is_contiguous(), what,
+              ": contiguous CUDA int32 of at least ", need, " values expected");
+  return t.data_ptr<int>();
+}
+int* status_ptr(const Tensor& t) { return const_cast<int*>(i32(t, 1, "status")); }
+// rows x cols view with unit column stride; returns the row pitch
+int64_t pitch(const Tensor& t, int64_t rows, int64_t cols, const char* what) {
+  TORCH_CHECK(t.dim() == 2 && t.stride(1) == 1 && t.size(0) >= rows && t.size(1) >= cols, what, ": [", rows, ", ", cols,
+              "] rows expected");
+  return t.stride(0);
+}
+oxb::RotaryParams rotary(const OptTensor& hi, const OptTensor& lo, bool interleaved, int64_t D) {
+  oxb::RotaryParams r{};
+  if (given(hi)) {
+    r.dims = static_cast<int>(2 * hi->numel());
+    TORCH_CHECK(r.dims <= D, "rotary: more dimensions than a head has");
+    r.freq_hi = f32(*hi, 1, "rotary");
+    TORCH_CHECK(given(lo), "rotary: frequencies are given as two terms");
+    r.freq_lo = f32(*lo, hi->numel(), "rotary");
+    r.interleaved = interleaved ? 1 : 0;
+  }
+  return r;
+}
+
+void stream_norm(const Tensor& x, int64_t rows, const OptTensor& tokens, const OptTensor& prev, const OptTensor& embed,
+                 const OptTensor& bigram, int64_t mul_prev, int64_t mul_cur, const OptTensor& y, bool zero_y, const OptTensor& mix,
+                 const OptTensor& out_w, const OptTensor& in_w, bool store_x, const Tensor& norm_w, double eps, double w_offset,
+                 const Tensor& h, const OptTensor& row_map, const OptTensor& clear, const Tensor& status) {
+  TORCH_CHECK(x.dim() == 3, "stream_norm: x [rows, streams, N]");
+  oxb::StreamNormParams p{};
+  p.rows = static_cast<int>(rows);
+  p.S = static_cast<int>(x.size(1));
+  p.N = static_cast<int>(x.size(2));
+  TORCH_CHECK(p.S >= 1 && p.S <= oxb::kMaxStreams, "stream_norm: 1..16 streams");
+  TORCH_CHECK(p.N <= 32768, "stream_norm: rows of at most 32768 values");
+  TORCH_CHECK(x.size(0) >= rows, "stream_norm: rows");
+  p.x = const_cast<float*>(f32(x, rows * p.S * p.N, "stream_norm x"));
+  const int dt = dtype_code(h, "stream_norm h");
+  TORCH_CHECK(given(tokens) != given(y), "stream_norm: either tokens or the sublayer's output");
+  if (given(tokens)) {
+    TORCH_CHECK(given(embed) && embed->scalar_type() == h.scalar_type() && embed->is_contiguous() && embed->dim() == 2 &&
+                    embed->size(1) == p.N,
+                "stream_norm: embed [vocab, N] of h's type");
+    p.tokens = i32(*tokens, rows, "stream_norm tokens");
+    p.embed = embed->data_ptr();
+    p.vocab = static_cast<int>(embed->size(0));
+    if (given(bigram)) {
+      TORCH_CHECK(given(prev) && bigram->scalar_type() == h.scalar_type() && bigram->is_contiguous() && bigram->dim() == 2 &&
+                      bigram->size(1) == p.N && bigram->size(0) >= 2 && mul_prev >= 0 && mul_cur >= 0,
+                  "stream_norm: bigram [buckets + 1, N], prev, multipliers >= 0");
+      p.prev = i32(*prev, rows, "stream_norm prev");
+      p.bigram = bigram->data_ptr();
+      p.buckets = static_cast<int>(bigram->size(0)) - 1;
+      p.mul_prev = mul_prev;
+      p.mul_cur = mul_cur;
+    }
+  } else {
+    p.ldy = pitch(*y, rows, p.N, "stream_norm y");
+    TORCH_CHECK(y->is_cuda() && y->scalar_type() == torch::kFloat32, "stream_norm: fp32 y");
+    p.y = y->data_ptr<float>();
+    p.zero_y = zero_y ? 1 : 0;
+    TORCH_CHECK(given(mix) && given(out_w), "stream_norm: mix and out belong to y");
+    p.mix = f32(*mix, p.S * p.S, "stream_norm mix");
+    p.out = f32(*out_w, p.S, "stream_norm out");
+  }
+  p.in = f32(in_w, p.S, "stream_norm in");
+  p.store_x = store_x ? 1 : 0;
+  p.norm_w = f32(norm_w, p.N, "stream_norm norm_w");
+  p.eps = static_cast<float>(eps);
+  p.w_offset = static_cast<float>(w_offset);
+  p.ldh = pitch(h, given(row_map) ? 1 : rows, p.N, "stream_norm h");
+  p.h = h.data_ptr();
+  if (given(row_map)) p.row_map = i32(*row_map, rows, "stream_norm row_map");
+  if (given(clear)) {
+    p.clear_ld = pitch(*clear, rows, 1, "stream_norm clear");
+    TORCH_CHECK(clear->scalar_type() == torch::kFloat32 && clear->is_cuda() && p.clear_ld % 4 == 0 && clear->size(1) % 4 == 0,
+                "stream_norm: clear is fp32 in whole 16-byte pieces");
+    p.clear = clear->data_ptr<float>();
+    p.clear_n = static_cast<int>(clear->size(1));
+  }
+  p.status = status_ptr(status);
+  check_launch(oxb::launch_stream_norm(p, dt, cur_stream()), "stream_norm");
+}
+
+void heads(const Tensor& proj, int64_t M, int64_t H, int64_t G, int64_t D, int64_t E, const OptTensor& q_norm,
+           const OptTensor& k_norm, double eps, const OptTensor& freq_hi, const OptTensor& freq_lo, bool interleaved,
+           const Tensor& positions, double k_scale, const Tensor& q_out, int64_t q_hd, const OptTensor& k_out,
+           const OptTensor& k_cache, const OptTensor& v_cache, const OptTensor& slots, const Tensor& status) {
+  oxb::HeadsParams p{};
+  // storage type: that of the caches; dense q and k are fp32 whatever the projection is
+  const int proj_dt = dtype_code(proj, "heads proj");
+  const int dt = given(k_cache) ? dtype_code(*k_cache, "heads k_cache") : proj_dt;
+  p.proj_f32 = proj_dt;
+  TORCH_CHECK(dt == 0 || proj_dt == 1, "heads: fp32 caches take fp32 projections");
+  TORCH_CHECK(H >= 1 && G >= 1 && D >= 1 && q_hd >= D, "heads: sizes");
+  p.proj = proj.data_ptr();
+  p.M = static_cast<int>(M);
+  p.H = static_cast<int>(H);
+  p.G = static_cast<int>(G);
+  p.D = static_cast<int>(D);
+  p.E = static_cast<int>(E);
+  p.q_norm = f32(q_norm, H * D, "heads q_norm");
+  p.k_norm = f32(k_norm, G * D, "heads k_norm");
+  TORCH_CHECK((p.q_norm == nullptr) == (p.k_norm == nullptr), "heads: q and k norm go together");
+  p.eps = static_cast<float>(eps);
+  p.rot = rotary(freq_hi, freq_lo, interleaved, D);
+  p.positions = i32(positions, M, "heads positions");
+  p.k_scale = static_cast<float>(k_scale);
+  p.q_ld = pitch(q_out, M, H * q_hd, "heads q_out");
+  p.q_out = q_out.data_ptr();
+  p.q_hd = static_cast<int>(q_hd);
+  if (given(k_out)) {
+    TORCH_CHECK(q_out.scalar_type() == torch::kFloat32 && k_out->scalar_type() == torch::kFloat32, "heads: dense q and k are fp32");
+    p.ld = pitch(proj, M, (H + G) * D, "heads proj");
+    p.k_ld = pitch(*k_out, M, G * D, "heads k_out");
+    p.k_out = k_out->data_ptr<float>();
+    p.k_hd = static_cast<int>(D);
+  } else {
+    TORCH_CHECK(given(k_cache) && given(v_cache) && given(slots), "heads: caches and slots, or k_out");
+    TORCH_CHECK(q_out.scalar_type() == k_cache->scalar_type() && v_cache->scalar_type() == k_cache->scalar_type(),
+                "heads: one storage type");
+    TORCH_CHECK(k_cache->dim() == 4 && v_cache->dim() == 4 && k_cache->is_contiguous() && v_cache->is_contiguous() &&
+                    k_cache->size(1) == G && v_cache->size(1) == G && k_cache->size(2) == 16 && v_cache->size(2) == 16 &&
+                    k_cache->size(0) == v_cache->size(0) && k_cache->size(3) >= D && v_cache->size(3) >= E,
+                "heads: caches [blocks, G, 16, >= head size]");
+    p.ld = pitch(proj, M, (H + G) * D + G * E, "heads proj");
+    p.k_cache = k_cache->data_ptr();
+    p.v_cache = v_cache->data_ptr();
+    p.DP = static_cast<int>(k_cache->size(3));
+    p.EP = static_cast<int>(v_cache->size(3));
+    TORCH_CHECK(slots->is_cuda() && slots->scalar_type() == torch::kInt64 && slots->numel() >= M, "heads: slots int64");
+    p.slots = reinterpret_cast<const long long*>(slots->data_ptr<int64_t>());
+    p.num_slots = k_cache->size(0) * 16;
+  }
+  p.status = status_ptr(status);
+  check_launch(oxb::launch_heads(p, dt, cur_stream()), "heads");
+}
+
+void row_attention(const Tensor& q, int64_t q_hd, const Tensor& k_cache, const Tensor& v_cache, const Tensor& block_tables,
+                   const OptTensor& seq_lens, const OptTensor& tile_seq, const OptTensor& tile_q0, const OptTensor& q_start,
+                   const OptTensor& q_lens, const OptTensor& ctx_lens, int64_t n, int64_t H, int64_t D, int64_t E, int64_t window,
+                   int64_t keep_first, double scale, const Tensor& out, const Tensor& status) {
+  oxb::RowAttnParams p{};
+  const int dt = dtype_code(q, "row_attention q");
+  TORCH_CHECK(k_cache.dim() == 4 && v_cache.dim() == 4 && k_cache.is_contiguous() && v_cache.is_contiguous() &&
+                  k_cache.size(2) == 16 && v_cache.size(2) == 16 && k_cache.size(1) == v_cache.size(1) &&
+                  k_cache.size(0) == v_cache.size(0),
+              "row_attention: caches [blocks, G, 16, head size]");
+  TORCH_CHECK(k_cache.scalar_type() == q.scalar_type() && v_cache.scalar_type() == q.scalar_type() &&
+                  out.scalar_type() == q.scalar_type(),
+              "row_attention: one storage type");
+  p.G = static_cast<int>(k_cache.size(1));
+  p.H = static_cast<int>(H);
+  p.D = static_cast<int>(D);
+  p.E = static_cast<int>(E);
+  p.DP = static_cast<int>(k_cache.size(3));
+  p.EP = static_cast<int>(v_cache.size(3));
+  TORCH_CHECK(H % p.G == 0 && D <= p.DP && E <= p.EP && E <= 1024 && D <= 4096 && q_hd >= D, "row_attention: head sizes");
+  p.q = q.data_ptr();
+  p.q_ld = pitch(q, 1, H * q_hd, "row_attention q");
+  p.q_hd = static_cast<int>(q_hd);
+  p.k_cache = k_cache.data_ptr();
+  p.v_cache = v_cache.data_ptr();
+  TORCH_CHECK(block_tables.dim() == 2 && block_tables.is_contiguous(), "row_attention: block_tables");
+  p.block_tables = i32(block_tables, 1, "row_attention block_tables");
+  p.max_blocks = static_cast<int>(block_tables.size(1));
+  p.num_blocks = static_cast<int>(k_cache.size(0));
+  p.n_rows = static_cast<int>(n);
+  if (given(tile_seq)) {
+    p.tile_seq = i32(*tile_seq, n, "row_attention tile_seq");
+    p.tile_q0 = i32(*tile_q0, n, "row_attention tile_q0");
+    p.q_start = i32(*q_start, 1, "row_attention q_start");
+    p.q_lens = i32(*q_lens, 1, "row_attention q_lens");
+    p.ctx_lens = i32(*ctx_lens, 1, "row_attention ctx_lens");
+  } else {
+    TORCH_CHECK(given(seq_lens) && block_tables.size(0) >= n, "row_attention: seq_lens");
+    p.seq_lens = i32(*seq_lens, n, "row_attention seq_lens");
+  }
+  p.window = static_cast<int>(window);
+  p.keep_first = static_cast<int>(keep_first);
+  p.scale = static_cast<float>(scale);
+  p.ldo = pitch(out, 1, H * E, "row_attention out");
+  p.out = out.data_ptr();
+  p.status = status_ptr(status);
+  check_launch(oxb::launch_row_attention(p, dt, cur_stream()), "row_attention");
+}
+
+oxb::RetentionParams retention_common(const Tensor& proj, int64_t M, int64_t H, int64_t D, int64_t E, const Tensor& decay_pow,
+                                      const Tensor& state, double eps, const Tensor& out, const Tensor& status) {
+  oxb::RetentionParams p{};
+  p.proj = proj.data_ptr();
+  p.ld = pitch(proj, M, 2 * H * (D + E), "retention proj");
+  p.H = static_cast<int>(H);
+  p.D = static_cast<int>(D);
+  p.E = static_cast<int>(E);
+  p.decay_pow = f32(decay_pow, H * (oxb::kRetChunk + 1), "retention decay_pow");
+  TORCH_CHECK(state.dim() == 4 && state.size(1) == H && state.size(2) == D && state.size(3) == E,
+              "retention: state [slots, H, D, E]");
+  p.state = const_cast<float*>(f32(state, 1, "retention state"));
+  p.num_slots = static_cast<int>(state.size(0));
+  p.eps = static_cast<float>(eps);
+  p.proj_f32 = dtype_code(proj, "retention proj");
+  TORCH_CHECK(dtype_code(out, "retention out") == 0 || p.proj_f32 == 1, "retention: fp32 rows take fp32 projections");
+  p.ldo = pitch(out, M, H * E, "retention out");
+  p.out = out.data_ptr();
+  p.status = status_ptr(status);
+  return p;
+}
+
+void retention_decode(const Tensor& proj, int64_t rows, int64_t H, int64_t D, int64_t E, const Tensor& decay_pow,
+                      const OptTensor& freq_hi, const OptTensor& freq_lo, bool interleaved, double k_scale, double eps,
+                      const Tensor& state, const Tensor& row_slots, const Tensor& positions, const Tensor& out,
+                      const Tensor& status) {
+  const int dt = dtype_code(out, "retention_decode out");
+  oxb::RetentionParams p = retention_common(proj, rows, H, D, E, decay_pow, state, eps, out, status);
+  TORCH_CHECK(D <= 4096 && E <= 4096, "retention_decode: head sizes");
+  p.rot = rotary(freq_hi, freq_lo, interleaved, D);
+  p.k_scale = static_cast<float>(k_scale);
+  p.row_slots = i32(row_slots, rows, "retention_decode row_slots");
+  p.positions = i32(positions, rows, "retention_decode positions");
+  p.rows = static_cast<int>(rows);
+  check_launch(oxb::launch_retention_decode(p, dt, cur_stream()), "retention_decode");
+}
+
+void retention_prefill(const Tensor& proj, int64_t M, int64_t H, int64_t D, int64_t E, const Tensor& decay_pow, double eps,
+                       const Tensor& state, const Tensor& seq_slots, const Tensor& tile_seq, const Tensor& tile_q0,
+                       const Tensor& q_start, const Tensor& q_lens, const Tensor& ctx_lens, int64_t n_tiles, int64_t n_seqs,
+                       const Tensor& q_rot, const Tensor& k_rot, const OptTensor& ws, const OptTensor& o_buf, const Tensor& out,
+                       const Tensor& status) {
+  const int dt = dtype_code(out, "retention_prefill out");
+  oxb::RetentionParams p = retention_common(proj, M, H, D, E, decay_pow, state, eps, out, status);
+  p.seq_slots = i32(seq_slots, n_seqs, "retention_prefill seq_slots");
+  p.tile_seq = i32(tile_seq, n_tiles, "retention_prefill tile_seq");
+  p.tile_q0 = i32(tile_q0, n_tiles, "retention_prefill tile_q0");
+  p.q_start = i32(q_start, n_seqs, "retention_prefill q_start");
+  p.q_lens = i32(q_lens, n_seqs, "retention_prefill q_lens");
+  p.ctx_lens = i32(ctx_lens, n_seqs, "retention_prefill ctx_lens");
+  p.n_tiles = static_cast<int>(n_tiles);
+  p.n_seqs = static_cast<int>(n_seqs);
+  p.q_rot = f32(q_rot, M * H * D, "retention_prefill q_rot");
+  p.k_rot = f32(k_rot, M * H * D, "retention_prefill k_rot");
+  if (given(ws)) {
+    TORCH_CHECK(dt == 0 && oxb::retention_chunks_ok(static_cast<int>(D), static_cast<int>(E)), "retention_prefill: chunked form");
+    p.ws = const_cast<float*>(f32(*ws, 2 * n_tiles * H * D * E, "retention_prefill ws"));
+    check_launch(oxb::launch_retention_chunks(p, cur_stream()), "retention_prefill");
+  } else {
+    TORCH_CHECK(given(o_buf) && D <= 1600, "retention_prefill: o_buf for the token-by-token form");
+    p.o_buf = const_cast<float*>(f32(*o_buf, M * H * E, "retention_prefill o_buf"));
+    check_launch(oxb::launch_retention_scan(p, dt, cur_stream()), "retention_prefill");
+  }
+}
+
+void gemm_f32(const Tensor& a, const Tensor& w, const Tensor& out) {
+  TORCH_CHECK(a.is_cuda() && w.is_cuda() && out.is_cuda() && a.scalar_type() == torch::kFloat32 &&
+                  w.scalar_type() == torch::kFloat32 && out.scalar_type() == torch::kFloat32 && a.dim() == 2 && w.dim() == 2 &&
+                  a.stride(1) == 1 && w.stride(1) == 1 && a.size(1) == w.size(1),
+              "gemm_f32: fp32 a [M, K], w [N, K]");
+  const int64_t M = a.size(0), N = w.size(0), K = a.size(1);
+  const int64_t ldo = pitch(out, M, N, "gemm_f32 out");
+  check_launch(oxb::launch_gemm_f32(a.data_ptr<float>(), a.stride(0), w.data_ptr<float>(), w.stride(0), out.data_ptr<float>(), ldo,
+                                    static_cast<int>(M), static_cast<int>(N), static_cast<int>(K), cur_stream()),
+               "gemm_f32");
+}
+
+void glu_f32(const Tensor& gu, const Tensor& out, int64_t M, int64_t I, int64_t act) {
+  TORCH_CHECK(gu.is_cuda() && gu.scalar_type() == torch::kFloat32 && out.scalar_type() == torch::kFloat32, "glu_f32: fp32");
+  const int64_t ldg = pitch(gu, M, 2 * I, "glu_f32 gu"), ldo = pitch(out, M, I, "glu_f32 out");
+  check_launch(oxb::launch_glu_f32(gu.data_ptr<float>(), ldg, out.data_ptr<float>(), ldo, static_cast<int>(M),
+                                   static_cast<int>(I), static_cast<int>(act), cur_stream()),
+               "glu_f32");
+}
+
+}  // namespace
+
+PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
+  m.doc() = "sm_100a kernels of layer-list decoders";
+  m.attr("RETENTION_CHUNK") = oxb::kRetChunk;
+  m.attr("MAX_STREAMS") = oxb::kMaxStreams;
+  m.def("set_pdl", [](bool on) { oxb::pdl_enabled() = on; });
+  m.def("stream_norm", &stream_norm);
+  m.def("heads", &heads);
+  m.def("row_attention", &row_attention);
+  m.def("retention_decode", &retention_decode);
+  m.def("retention_prefill", &retention_prefill);
+  m.def("retention_chunks_ok", [](int64_t D, int64_t E) { return oxb::retention_chunks_ok((int)D, (int)E); });
+  m.def("gemm_f32", &gemm_f32);
+  m.def("glu_f32", &glu_f32);
+}

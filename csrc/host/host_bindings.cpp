@@ -126,7 +126,8 @@ PYBIND11_MODULE(oxb_host, m) {
       .def_readwrite("sla_budget", &SchedulerConfig::sla_budget)
       .def_readwrite("context_shift", &SchedulerConfig::context_shift)
       .def_readwrite("shift_keep_tokens", &SchedulerConfig::shift_keep_tokens)
-      .def_readwrite("shift_step_tokens", &SchedulerConfig::shift_step_tokens);
+      .def_readwrite("shift_step_tokens", &SchedulerConfig::shift_step_tokens)
+      .def_readwrite("state_slots", &SchedulerConfig::state_slots);
 
   py::class_<TokenEvent>(m, "TokenEvent")
       .def_readonly("req_id", &TokenEvent::req_id)
@@ -146,6 +147,9 @@ PYBIND11_MODULE(oxb_host, m) {
       .def_readonly("max_blocks", &StepPlan::max_blocks)
       .def_readonly("prefill_tokens", &StepPlan::prefill_tokens)
       .def_property_readonly("token_ids", [](const StepPlan& p) { return to_array(p.token_ids); })
+      .def_property_readonly("prev_ids", [](const StepPlan& p) { return to_array(p.prev_ids); })
+      .def_property_readonly("decode_slots", [](const StepPlan& p) { return to_array(p.decode_slots); })
+      .def_property_readonly("prefill_slots", [](const StepPlan& p) { return to_array(p.prefill_slots); })
       .def_property_readonly("positions", [](const StepPlan& p) { return to_array(p.positions); })
       .def_property_readonly("slot_mapping", [](const StepPlan& p) { return to_array(p.slot_mapping); })
       .def_property_readonly("decode_ids", [](const StepPlan& p) { return to_array(p.decode_ids); })
@@ -199,6 +203,14 @@ PYBIND11_MODULE(oxb_host, m) {
              return out;
            })
       .def("take_events", &Scheduler::take_events)
+      .def("feed",
+           [](Scheduler& s, const std::vector<std::tuple<int64_t, std::vector<int32_t>, std::vector<int32_t>>>& entries) {
+             std::vector<FeedEntry> es;
+             for (auto& e : entries) es.push_back({std::get<0>(e), std::get<1>(e), std::get<2>(e)});
+             return s.feed(es);
+           })
+      .def("feed_done", &Scheduler::feed_done)
+      .def("num_free_slots", &Scheduler::num_free_slots)
       .def("schedule", &Scheduler::schedule)
       .def("update",
            [](Scheduler& s, const StepPlan& plan,
@@ -230,6 +242,7 @@ PYBIND11_MODULE(oxb_host, m) {
              d["generated"] = r->generated();
              d["prefix_hit"] = r->prefix_hit;
              d["phase"] = static_cast<int>(r->phase);
+             d["slot"] = r->slot;
              d["preemptions"] = r->preemptions;
              d["blocks"] = r->table->blocks();
              return d;

@@ -10,11 +10,33 @@ namespace {
 constexpr int kTileQ = 128;  // query rows per prefill-attention tile (one tcgen05 M tile)
 }
 
-Scheduler::Scheduler(const SchedulerConfig& cfg) : cfg_(cfg), pool_(cfg.num_blocks), radix_(&pool_) {}
+Scheduler::Scheduler(const SchedulerConfig& cfg) : cfg_(cfg), pool_(cfg.num_blocks), radix_(&pool_) {
+  if (cfg_.state_slots > 0) {
+    cfg_.enable_radix = false;
+    cfg_.context_shift = false;
+  }
+  for (int i = cfg_.state_slots - 1; i >= 0; --i) free_slots_.push_back(i);
+}
+
+bool Scheduler::take_slot(Request* r) {
+  if (cfg_.state_slots <= 0 || r->slot >= 0) return true;
+  if (free_slots_.empty()) return false;
+  r->slot = free_slots_.back();
+  free_slots_.pop_back();
+  return true;
+}
+
+void Scheduler::release(Request* r) {
+  r->table->release_all();
+  if (r->slot >= 0) free_slots_.push_back(r->slot);
+  r->slot = -1;
+}
 
 void Scheduler::add_request(int64_t id, const std::vector<int32_t>& prompt, int max_new_tokens,
                             const std::vector<int32_t>& stop_ids, bool ignore_eos) {
   if (prompt.empty()) throw std::invalid_argument("empty prompt");
+  for (auto& r : running_)
+    if (r->phase == Phase::Fed) throw std::invalid_argument("fed requests are live: end them before queueing a prompt");
   if (static_cast<int>(prompt.size()) + 1 > cfg_.max_blocks_per_seq * kTokensPerBlock)
     throw std::invalid_argument("prompt longer than the per-sequence KV capacity");
   std::unique_ptr<Request> r(new Request());
@@ -54,7 +76,7 @@ bool Scheduler::cancel(int64_t id, std::vector<TokenEvent>* events) {
   for (auto it = running_.begin(); it != running_.end(); ++it) {
     if ((*it)->id == id) {
       if (events) events->push_back({id, -1, true, "cancelled"});
-      (*it)->table->release_all();
+      release(it->get());
       running_.erase(it);
       return true;
     }
@@ -63,13 +85,16 @@ bool Scheduler::cancel(int64_t id, std::vector<TokenEvent>* events) {
 }
 
 void Scheduler::set_drafts(int64_t id, const std::vector<int32_t>& drafts) {
-  // a pruned sequence decodes one token at a time (its KV is no longer a contiguous prefix)
+  // a pruned sequence decodes one token at a time (its KV is no longer a contiguous prefix), and so
+  // does one with a recurrent state (rejected drafts could not be taken out of it)
+  if (cfg_.state_slots > 0) return;
   for (auto& r : running_)
     if (r->id == id && r->phase == Phase::Decode && r->dropped == 0) r->drafts = drafts;
 }
 
 std::vector<int> Scheduler::prune_request(int64_t id, const std::vector<float>& block_scores,
                                           int sink_blocks, int rolling_blocks, int budget_blocks) {
+  if (cfg_.state_slots > 0) return {};
   for (auto& r : running_) {
     if (r->id != id || r->phase != Phase::Decode) continue;
     const int before = static_cast<int>(r->table->blocks().size());
@@ -153,7 +178,7 @@ void Scheduler::preempt(Request* r) {
   // recompute-style preemption: drop the KV, keep the tokens, go back to the head of the queue
   ++preemptions_;
   ++r->preemptions;
-  r->table->release_all();
+  release(r);
   r->computed = 0;
   r->dropped = 0;
   r->cached_blocks = 0;
@@ -171,7 +196,7 @@ void Scheduler::preempt(Request* r) {
 
 void Scheduler::abort(Request* r, const std::string& reason) {
   deferred_.push_back({r->id, -1, true, reason});
-  r->table->release_all();
+  release(r);
   r->phase = Phase::Finished;
   for (auto it = running_.begin(); it != running_.end(); ++it) {
     if (it->get() == r) {
@@ -274,7 +299,7 @@ void Scheduler::offer_to_radix(Request* r) {
 
 void Scheduler::finish(Request* r) {
   offer_to_radix(r);
-  r->table->release_all();
+  release(r);
   r->phase = Phase::Finished;
   for (auto it = running_.begin(); it != running_.end(); ++it) {
     if (it->get() == r) {
@@ -294,11 +319,6 @@ StepPlan Scheduler::schedule() {
               return a->arrival < b->arrival;
             });
 
-  struct Item {
-    Request* r;
-    int len;
-    int kind;  // 0 decode, 1 prefill chunk, 2 verify chunk
-  };
   std::vector<Item> decodes, chunks;
   // A preempted request may already sit in this step's lists (it was given blocks earlier in the
   // pass): take it out again.
@@ -409,8 +429,9 @@ StepPlan Scheduler::schedule() {
     }
     const int remaining = static_cast<int>(r->tokens.size()) - r->computed;
     const int c = std::min(remaining, budget);
+    if (!take_slot(r)) break;  // every state slot is held by a running request
     if (!ensure_blocks(r, c, &plan)) {
-      r->table->release_all();
+      release(r);
       r->computed = 0;
       r->cached_blocks = 0;
       if (running_.empty()) {
@@ -430,7 +451,14 @@ StepPlan Scheduler::schedule() {
     budget -= c;
   }
 
-  // ---- build the flat arrays: decode rows first, then chunk rows ----
+  build_rows(decodes, chunks, /*want_logits=*/true, &plan);
+  return plan;
+}
+
+// The flat arrays of a step: decode rows first, then chunk rows.
+void Scheduler::build_rows(const std::vector<Item>& decodes, const std::vector<Item>& chunks, bool want_logits,
+                           StepPlan* out) {
+  StepPlan& plan = *out;
   int max_blocks = 1;
   for (auto& d : decodes) max_blocks = std::max<int>(max_blocks, d.r->table->blocks().size());
   for (auto& c : chunks) max_blocks = std::max<int>(max_blocks, c.r->table->blocks().size());
@@ -453,20 +481,26 @@ StepPlan Scheduler::schedule() {
   for (auto& d : decodes) {
     Request* r = d.r;
     const int pos = r->computed;
+    const size_t n_tok = r->tokens.size();
     plan.token_ids.push_back(r->tokens.back());
+    plan.prev_ids.push_back(n_tok >= 2 ? r->tokens[n_tok - 2] : -1);
+    plan.decode_slots.push_back(r->slot);
     plan.positions.push_back(pos);
     plan.slot_mapping.push_back(slot_of(r, pos));
     plan.decode_ids.push_back(r->id);
     plan.decode_seq_lens.push_back(pos + 1 - r->dropped);
     push_table(&plan.decode_block_tables, r);
-    plan.logit_rows.push_back(static_cast<int32_t>(plan.token_ids.size()) - 1);
-    plan.logit_req.push_back(r->id);
+    if (want_logits) {
+      plan.logit_rows.push_back(static_cast<int32_t>(plan.token_ids.size()) - 1);
+      plan.logit_req.push_back(r->id);
+    }
   }
   int s = 0;
   for (auto& c : chunks) {
     Request* r = c.r;
     const int start = static_cast<int>(plan.token_ids.size());
     plan.prefill_ids.push_back(r->id);
+    plan.prefill_slots.push_back(r->slot);
     plan.q_start.push_back(start);
     plan.q_lens.push_back(c.len);
     plan.ctx_lens.push_back(r->computed - r->dropped + c.len);
@@ -482,13 +516,21 @@ StepPlan Scheduler::schedule() {
         tok = j == 0 ? r->tokens.back() : r->drafts[j - 1];
       else
         tok = r->tokens[pos];
+      int32_t prev;  // the row before it in this chunk, or the last token of what is already computed
+      if (j > 0)
+        prev = plan.token_ids.back();
+      else if (c.kind == 2)
+        prev = r->tokens.size() >= 2 ? r->tokens[r->tokens.size() - 2] : -1;
+      else
+        prev = pos > 0 ? r->tokens[pos - 1] : -1;
       plan.token_ids.push_back(tok);
+      plan.prev_ids.push_back(prev);
       plan.positions.push_back(pos);
       plan.slot_mapping.push_back(slot_of(r, pos));
       const bool last = j == c.len - 1;
-      const bool wants_logits =
+      const bool row_logits =
           c.kind == 2 || (last && r->computed + c.len == static_cast<int>(r->tokens.size()));
-      if (wants_logits) {
+      if (want_logits && row_logits) {
         plan.logit_rows.push_back(static_cast<int32_t>(plan.token_ids.size()) - 1);
         plan.logit_req.push_back(r->id);
       }
@@ -497,7 +539,74 @@ StepPlan Scheduler::schedule() {
     ++s;
   }
   plan.n_tokens = static_cast<int>(plan.token_ids.size());
+}
+
+StepPlan Scheduler::feed(const std::vector<FeedEntry>& entries) {
+  StepPlan plan;
+  cow_owner_.clear();
+  feed_lens_.clear();
+  if (!waiting_.empty()) throw std::invalid_argument("feed: requests are queued for generation");
+  std::vector<Item> decodes, chunks;
+  for (auto& e : entries) {
+    if (e.tokens.empty()) throw std::invalid_argument("feed: an entry without tokens");
+    Request* r = nullptr;
+    for (auto& up : running_) {
+      if (up->phase != Phase::Fed) throw std::invalid_argument("feed: requests are being generated");
+      if (up->id == e.id) r = up.get();
+    }
+    for (auto& seen : {&decodes, &chunks})
+      for (auto& it : *seen)
+        if (it.r->id == e.id) throw std::invalid_argument("feed: a request appears twice in one step");
+    for (int32_t w : e.want)
+      if (w < 0 || w >= static_cast<int32_t>(e.tokens.size())) throw std::invalid_argument("feed: want is out of range");
+    const int n = static_cast<int>(e.tokens.size());
+    if (r == nullptr) {
+      if (static_cast<int>(running_.size()) >= cfg_.max_num_seqs) throw std::runtime_error("feed: too many live requests");
+      std::unique_ptr<Request> owned(new Request());
+      r = owned.get();
+      r->id = e.id;
+      r->phase = Phase::Fed;
+      r->arrival = arrivals_++;
+      r->table.reset(new SequenceBlockTable(&pool_));
+      running_.push_back(std::move(owned));
+    }
+    if (static_cast<int>(r->tokens.size()) + n > cfg_.max_blocks_per_seq * kTokensPerBlock)
+      throw std::runtime_error("feed: a request outgrows the per-sequence KV capacity");
+    if (!take_slot(r)) throw std::runtime_error("feed: no free state slot");
+    if (!ensure_blocks(r, n, &plan)) throw std::runtime_error("feed: the KV pool is exhausted");
+    r->tokens.insert(r->tokens.end(), e.tokens.begin(), e.tokens.end());
+    r->prompt_len = static_cast<int>(r->tokens.size());
+    if (n == 1 && r->computed > 0)
+      decodes.push_back({r, 1, 0});
+    else
+      chunks.push_back({r, n, 1});
+  }
+  build_rows(decodes, chunks, /*want_logits=*/false, &plan);
+  // first row of every request of the step, then the wanted rows in the caller's order
+  std::unordered_map<int64_t, int> first;
+  for (size_t i = 0; i < decodes.size(); ++i) first[decodes[i].r->id] = static_cast<int>(i);
+  for (size_t i = 0; i < chunks.size(); ++i) first[chunks[i].r->id] = plan.q_start[i];
+  for (auto& e : entries)
+    for (int32_t w : e.want) {
+      plan.logit_rows.push_back(first[e.id] + w);
+      plan.logit_req.push_back(e.id);
+    }
+  for (auto& d : decodes) feed_lens_.push_back(d.len);
+  for (auto& c : chunks) feed_lens_.push_back(c.len);
   return plan;
+}
+
+void Scheduler::feed_done(const StepPlan& plan) {
+  auto book = [&](int64_t id, int n) {
+    for (auto& r : running_)
+      if (r->id == id && r->phase == Phase::Fed) {
+        r->computed += n;
+        r->table->commit();
+      }
+  };
+  size_t k = 0;
+  for (int64_t id : plan.decode_ids) book(id, feed_lens_[k++]);
+  for (int64_t id : plan.prefill_ids) book(id, feed_lens_[k++]);
 }
 
 std::vector<TokenEvent> Scheduler::update(const StepPlan& plan, const std::vector<int32_t>& sampled) {
@@ -553,7 +662,7 @@ std::vector<TokenEvent> Scheduler::update(const StepPlan& plan, const std::vecto
     if (fault != prefill_faults_.end() && r->phase == Phase::Prefill) {
       events.push_back({id, -1, true, "prefill_error: " + fault->second});
       prefill_faults_.erase(fault);
-      r->table->release_all();
+      release(r);
       for (auto it = running_.begin(); it != running_.end(); ++it)
         if (it->get() == r) {
           running_.erase(it);

@@ -48,9 +48,15 @@ struct SchedulerConfig {
   bool context_shift = false;
   int shift_keep_tokens = 4;
   int shift_step_tokens = 256;
+  // Models with recurrent layers keep a fixed-size state per live sequence beside the paged KV: every
+  // running request holds one of `state_slots` slots from its admission until it ends or is preempted
+  // (0: the model has no such state). A state cannot be cut back or shared, so such a model runs without
+  // the prefix cache, speculative drafts, pruning and context shift.
+  int state_slots = 0;
 };
 
-enum class Phase : int { Waiting = 0, Prefill = 1, Decode = 2, Finished = 3 };
+// Fed: a request whose tokens the caller supplies step by step (Scheduler::feed); schedule() leaves it alone.
+enum class Phase : int { Waiting = 0, Prefill = 1, Decode = 2, Finished = 3, Fed = 4 };
 
 struct Request {
   int64_t id = 0;
@@ -68,6 +74,7 @@ struct Request {
   uint64_t arrival = 0;
   int preemptions = 0;
   std::unique_ptr<SequenceBlockTable> table;
+  int slot = -1;                // recurrent-state slot while running (SchedulerConfig::state_slots)
   int generated() const { return static_cast<int>(tokens.size()) - prompt_len; }
 };
 
@@ -84,7 +91,9 @@ struct StepPlan {
   int n_prefill = 0;
   int max_blocks = 0;  // columns of the block-table arrays
   std::vector<int32_t> token_ids, positions;
+  std::vector<int32_t> prev_ids;  // the token before each row's token in its sequence, -1 for a first token
   std::vector<int64_t> slot_mapping;
+  std::vector<int32_t> decode_slots, prefill_slots;  // state slot of every decode row / chunk (-1 without state)
   std::vector<int64_t> decode_ids;
   std::vector<int32_t> decode_seq_lens, decode_block_tables;
   std::vector<int64_t> prefill_ids;
@@ -93,6 +102,13 @@ struct StepPlan {
   std::vector<int64_t> logit_req;
   std::vector<int32_t> cow_src, cow_dst;
   int prefill_tokens = 0;
+};
+
+// One request's share of a fed step: its next tokens and the places among them whose logits are wanted.
+struct FeedEntry {
+  int64_t id = 0;
+  std::vector<int32_t> tokens;
+  std::vector<int32_t> want;
 };
 
 class Scheduler {
@@ -133,6 +149,15 @@ class Scheduler {
   // `sampled[i]` is the token drawn from logits row i of the plan that was just executed.
   std::vector<TokenEvent> update(const StepPlan& plan, const std::vector<int32_t>& sampled);
 
+  // Replay of given tokens: one step made of `entries`, which run together as one batch (single tokens
+  // of requests with a past as decode rows, the rest as chunks). A request is admitted at its first
+  // entry and lives until cancel(). logit_rows / logit_req follow the order of the entries and of their
+  // `want`. Nothing is sampled: feed_done() books the step's tokens as computed. Throws when a request
+  // has been queued the ordinary way, or when the pool or the state slots are short.
+  StepPlan feed(const std::vector<FeedEntry>& entries);
+  void feed_done(const StepPlan& plan);
+
+  int num_free_slots() const { return static_cast<int>(free_slots_.size()); }
   int prefill_budget(int active_decodes) const;
   int num_waiting() const { return static_cast<int>(waiting_.size()); }
   int num_running() const { return static_cast<int>(running_.size()); }
@@ -147,6 +172,15 @@ class Scheduler {
   std::vector<int64_t> running_ids() const;
 
  private:
+  // One sequence's rows of the step being planned. kind: 0 decode row, 1 prompt chunk, 2 verify chunk.
+  struct Item {
+    Request* r;
+    int len;
+    int kind;
+  };
+  void build_rows(const std::vector<Item>& decodes, const std::vector<Item>& chunks, bool want_logits, StepPlan* plan);
+  bool take_slot(Request* r);
+  void release(Request* r);  // KV blocks and state slot
   bool ensure_blocks(Request* r, int n_tokens, StepPlan* plan);
   void shift_context(Request* r, int incoming);
   void preempt(Request* r);
@@ -162,6 +196,8 @@ class Scheduler {
   std::vector<std::unique_ptr<Request>> running_;
   std::unordered_map<int64_t, std::string> prefill_faults_;
   std::vector<TokenEvent> deferred_;
+  std::vector<int> free_slots_;     // recurrent-state slots that no request holds
+  std::vector<int> feed_lens_;      // tokens of every sequence of the fed step in flight (plan order)
   std::vector<int64_t> cow_owner_;  // request id of each copy-on-write pair of the plan being built
   uint64_t arrivals_ = 0;
   uint64_t preemptions_ = 0;

@@ -21,6 +21,9 @@ struct DecodeAttnParams {
   __nv_bfloat16* out;          // [B, Hq*D], row stride out_stride
   long long out_stride;
   int max_blocks, Hq, Hkv, max_splits, window;
+  int keep_first;    // with a window: the first positions stay visible too (0: none); they keep their true positions
+  int out_d;         // values stored per head in `out` (<= D; 0: D). The caches and q are padded to D
+  int exact_p;       // 1: softmax weights enter the value product as two bf16 terms (about 16 bits) instead of one
   float scale_log2;  // softmax scale * log2(e)
   // Bounds check of block-table entries: an id outside [0, num_blocks) is recorded in *status
   // (kStatusBadIndex) and page 0 is read instead. num_blocks <= 0 or status == nullptr: no check.
@@ -60,6 +63,7 @@ struct PrefillAttnParams {
   __nv_bfloat16* out;       // [T, Hq*D], row stride out_stride
   long long out_stride;
   int max_blocks, Hq, Hkv, window;
+  int keep_first, out_d, exact_p;  // as in DecodeAttnParams
   float scale_log2;
   int num_blocks;  // bound for block-table entries (<= 0: unchecked), violations go to *status
   int* status;

@@ -83,7 +83,8 @@ __device__ __forceinline__ float ex2(float x) {
 
 // D = head dim (64 or 128); NT = number of 8-head column tiles (group size <= 8*NT).
 // MASS: also record the per-page softmax statistics of every head (see DecodeAttnParams::page_ml).
-template <int D, int NT, bool MASS>
+// EXACT: the softmax weights enter the value product as hi + lo bf16 terms (DecodeAttnParams::exact_p).
+template <int D, int NT, bool MASS, bool EXACT>
 __global__ void __launch_bounds__(kWarps * 32)
 paged_decode_kernel(const DecodeAttnParams p) {
   constexpr int KS = D / 16;   // k-steps of QK^T
@@ -109,11 +110,25 @@ paged_decode_kernel(const DecodeAttnParams p) {
     if (p.status != nullptr && threadIdx.x == 0) atomicCAS(p.status, 0, 5 /* kStatusBadIndex */);
     n_pages = p.max_blocks;
   }
-  const int pps = *p.pages_per_split;
+  int pps = *p.pages_per_split;
   const int first_page = win_start / kPage;
-  const int pg_lo = first_page + split * pps;
+  // The walk is over a list of pages: the ones that hold kept first positions and lie before the window,
+  // then the window's. List entry l is page l + (l < n_first ? 0 : skip).
+  int n_first = 0;
+  if (p.keep_first > 0 && first_page > 0) {
+    n_first = (p.keep_first + kPage - 1) / kPage;
+    if (n_first > first_page) n_first = first_page;
+  }
+  const int skip = first_page - n_first;
+  const int n_list = n_pages - skip;
+  if (p.window > 0 && skip > 0) {
+    // the host sized the splits for the whole context: spread the visible pages over as many splits
+    const int used = (n_pages + pps - 1) / pps;
+    pps = ((n_list + used - 1) / used + kWarps - 1) / kWarps * kWarps;
+  }
+  const int pg_lo = split * pps;
   int pg_hi = pg_lo + pps;
-  if (pg_hi > n_pages) pg_hi = n_pages;
+  if (pg_hi > n_list) pg_hi = n_list;
 
   const long long part_idx0 = (static_cast<long long>(seq) * p.Hq + kvh * G) * p.max_splits;
   if (pg_lo >= pg_hi || seq_len <= 0) {
@@ -194,22 +209,24 @@ paged_decode_kernel(const DecodeAttnParams p) {
     }
   };
   // block ids run one page ahead of the copies, the copies kRing - 1 pages ahead of the math
-  int page = pg_lo + warp;
-  int issue_page = page;
-  int blk_next = issue_page < pg_hi ? checked(bt[issue_page]) : 0;
+  auto page_of = [&](int l) -> int { return l < n_first ? l : l + skip; };
+  int item = pg_lo + warp;
+  int issue_page = item;
+  int blk_next = issue_page < pg_hi ? checked(bt[page_of(issue_page)]) : 0;
 #pragma unroll
   for (int i = 0; i < kRing - 1; ++i) {
     if (issue_page < pg_hi) {
       const int b = blk_next;
       const int np = issue_page + kWarps;
-      blk_next = np < pg_hi ? checked(bt[np]) : 0;
+      blk_next = np < pg_hi ? checked(bt[page_of(np)]) : 0;
       issue(i, b);
     }
     cp_async_commit();
     issue_page += kWarps;
   }
   int slot = 0;
-  for (; page < pg_hi; page += kWarps) {
+  for (; item < pg_hi; item += kWarps) {
+    const int page = page_of(item);
     // top up the ring, then wait until the oldest page has landed
     {
       int s_new = slot + kRing - 1;
@@ -217,7 +234,7 @@ paged_decode_kernel(const DecodeAttnParams p) {
       if (issue_page < pg_hi) {
         const int b = blk_next;
         const int np = issue_page + kWarps;
-        blk_next = np < pg_hi ? checked(bt[np]) : 0;
+        blk_next = np < pg_hi ? checked(bt[page_of(np)]) : 0;
         issue(s_new, b);
       }
       cp_async_commit();
@@ -262,9 +279,10 @@ paged_decode_kernel(const DecodeAttnParams p) {
 
     // ---- online softmax over the page's 16 tokens (rows of S^T) ----
     const int tok0 = page * kPage + g;
-    const bool v0 = tok0 < seq_len && tok0 >= win_start;
-    const bool v1 = tok0 + 8 < seq_len && tok0 + 8 >= win_start;
+    const bool v0 = tok0 < seq_len && (tok0 >= win_start || tok0 < p.keep_first);
+    const bool v1 = tok0 + 8 < seq_len && (tok0 + 8 >= win_start || tok0 + 8 < p.keep_first);
     uint32_t pb[NT][2];
+    uint32_t pl[EXACT ? NT : 1][2];  // low terms of the weights
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt) {
       float x00 = v0 ? s[nt][0] * p.scale_log2 : -INFINITY;  // tok g,   head 2t
@@ -311,6 +329,11 @@ paged_decode_kernel(const DecodeAttnParams p) {
       // P^T fragments: (tok 2t,2t+1 | head g) and (tok 2t+8,2t+9 | head g)
       pb[nt][0] = movmatrix_trans(pack2(p00, p01));
       pb[nt][1] = movmatrix_trans(pack2(p10, p11));
+      if constexpr (EXACT) {
+        auto rest = [](float x) { return x - __bfloat162float(__float2bfloat16(x)); };
+        pl[nt][0] = movmatrix_trans(pack2(rest(p00), rest(p01)));
+        pl[nt][1] = movmatrix_trans(pack2(rest(p10), rest(p11)));
+      }
     }
 
     // ---- O^T += V^T * P^T ----
@@ -327,8 +350,10 @@ paged_decode_kernel(const DecodeAttnParams p) {
         const uint32_t a2 = __byte_perm(vc[e], vd[e], 0x5410);  // dim 2e   | tok 2t+8, 2t+9
         const uint32_t a3 = __byte_perm(vc[e], vd[e], 0x7632);  // dim 2e+1 | tok 2t+8, 2t+9
 #pragma unroll
-        for (int nt = 0; nt < NT; ++nt)
+        for (int nt = 0; nt < NT; ++nt) {
           mma_bf16_16816(o_acc[nt][4 * c + e], a0, a1, a2, a3, pb[nt][0], pb[nt][1]);
+          if constexpr (EXACT) mma_bf16_16816(o_acc[nt][4 * c + e], a0, a1, a2, a3, pl[nt][0], pl[nt][1]);
+        }
       }
     }
     __syncwarp();  // every lane is done with this slot before it is refilled
@@ -410,7 +435,8 @@ __global__ void __launch_bounds__(D) decode_merge_kernel(const DecodeAttnParams 
   }
   const float r = L > 0.f ? acc / L : 0.f;
   const __nv_bfloat16 rb = __float2bfloat16(r);
-  p.out[static_cast<long long>(seq) * p.out_stride + head * D + d] = rb;
+  const int od = p.out_d > 0 ? p.out_d : D;
+  if (d < od) p.out[static_cast<long long>(seq) * p.out_stride + head * od + d] = rb;
   if (p.q8 != nullptr) {
     // a warp holds one block of 32 values: scale = amax / 127, codes, scale * sum
     const float v = __bfloat162float(rb);
@@ -442,7 +468,8 @@ __global__ void __launch_bounds__(128) block_mass_kernel(const DecodeAttnParams 
   if (n_pages > p.max_blocks) n_pages = p.max_blocks;
   const int win_start = (p.window > 0 && seq_len > p.window) ? seq_len - p.window : 0;
   const int first_page = win_start / kPage;
-  int last_page = first_page + *p.pages_per_split * p.max_splits;  // pages past the last split were not walked
+  // (with a window the splits are respread inside the kernel and cover all of it)
+  int last_page = p.window > 0 ? n_pages : first_page + *p.pages_per_split * p.max_splits;  // pages past the last split were not walked
   if (last_page > n_pages) last_page = n_pages;
   for (int h = threadIdx.x; h < p.Hq; h += blockDim.x) {
     const long long base = (static_cast<long long>(seq) * p.Hq + h) * p.max_splits;
@@ -480,11 +507,15 @@ void launch_split(const DecodeAttnParams& p, dim3 grid, cudaStream_t stream) {
   constexpr size_t merge = sizeof(float) * kWarps * 8 * NT * (D + 2);
   constexpr size_t smem = ring > merge ? ring : merge;
   if (p.page_ml != nullptr) {
-    auto kern = paged_decode_kernel<D, NT, true>;
+    auto kern = paged_decode_kernel<D, NT, true, false>;
+    ensure_dynamic_smem(kern, smem);
+    launch_kernel(kern, grid, dim3(kWarps * 32), smem, stream, /*pdl=*/true, false, p);
+  } else if (p.exact_p != 0) {
+    auto kern = paged_decode_kernel<D, NT, false, true>;
     ensure_dynamic_smem(kern, smem);
     launch_kernel(kern, grid, dim3(kWarps * 32), smem, stream, /*pdl=*/true, false, p);
   } else {
-    auto kern = paged_decode_kernel<D, NT, false>;
+    auto kern = paged_decode_kernel<D, NT, false, false>;
     ensure_dynamic_smem(kern, smem);
     launch_kernel(kern, grid, dim3(kWarps * 32), smem, stream, /*pdl=*/true, false, p);
   }

@@ -40,22 +40,23 @@ __device__ __forceinline__ float ex2a(float x) {
   return y;
 }
 
-template <int D>
+template <int D, bool EXACT>
 struct Smem {
   static constexpr int DH = D / 64;
   static constexpr int kQ = 0;
   static constexpr int kK = kQ + DH * kHalfBytes;           // 2 stages
   static constexpr int kV = kK + 2 * DH * kHalfBytes;       // 2 stages
   static constexpr int kP = kV + 2 * DH * kHalfBytes;       // [128 x 128] as two halves
-  static constexpr int kBar = kP + 2 * kHalfBytes;
+  static constexpr int kBar = kP + (EXACT ? 4 : 2) * kHalfBytes;   // EXACT: a second [128 x 128] of low terms
   static constexpr int kTotal = kBar + 256 + 1024;
 };
 
-template <int D>
+// EXACT: the softmax weights enter the value product as hi + lo bf16 terms (PrefillAttnParams::exact_p).
+template <int D, bool EXACT>
 __global__ void __launch_bounds__(kThreads, 1)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                   const __grid_constant__ CUtensorMap tmV, const PrefillAttnParams p, int* status) {
-  using L = Smem<D>;
+  using L = Smem<D, EXACT>;
   constexpr int DH = D / 64;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem =
@@ -96,7 +97,15 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     const int lo = pos_off + q0 - p.window + 1;
     if (lo > 0) first_tile = lo / BKV;
   }
-  const int n_tiles = max_pos / BKV + 1 - first_tile;
+  // KV tiles that hold kept first positions and lie before the window come first, then the window's:
+  // list entry j is tile j + (j < n_first ? 0 : skip)
+  int n_first = 0;
+  if (p.keep_first > 0 && first_tile > 0) {
+    n_first = (p.keep_first + BKV - 1) / BKV;
+    if (n_first > first_tile) n_first = first_tile;
+  }
+  const int skip = first_tile - n_first;
+  const int n_tiles = max_pos / BKV + 1 - skip;
 
   if (threadIdx.x == 0) {
     tma_prefetch_desc(&tmQ);
@@ -156,7 +165,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         }
         __syncwarp();
         if (issuer) {
-          const int pi = (first_tile + j) * (BKV / 16) + pg;
+          const int pi = (j < n_first ? j : j + skip) * (BKV / 16) + pg;
           int blk = pi < p.max_blocks ? bt[pi] : 0;
           if (p.num_blocks > 0 && static_cast<unsigned>(blk) >= static_cast<unsigned>(p.num_blocks)) {
             set_status_once(status, kStatusBadIndex);
@@ -212,6 +221,14 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                      make_desc_mnmajor_sw128(vb + kk * 2048, kHalfBytes, 1024), idesc_o,
                      (j | kk) != 0 ? 1u : 0u);
         }
+        if constexpr (EXACT) {
+#pragma unroll
+          for (int kk = 0; kk < BKV / 16; ++kk) {
+            const uint32_t aoff = (2 + (kk >> 2)) * kHalfBytes + (kk & 3) * 32;
+            tc_mma_f16(tmem_o, make_desc_kmajor_sw128(pa + aoff),
+                       make_desc_mnmajor_sw128(vb + kk * 2048, kHalfBytes, 1024), idesc_o, 1u);
+          }
+        }
         tc_commit(&kv_empty[s]);
         tc_commit(pv_done);
       }
@@ -234,7 +251,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       if (!ok) break;
       tc_fence_after_sync();
       const uint32_t s_addr = tmem_s0 + b * BKV + lane_sel;
-      const int t0 = (first_tile + j) * BKV;
+      const int t0 = (j < n_first ? j : j + skip) * BKV;
       // ---- pass 1: row maximum over the unmasked scores ----
       float mx = -INFINITY;
 #pragma unroll 1
@@ -245,7 +262,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           const int t = t0 + c * 32 + i;
-          const bool keep = t <= pos && (p.window <= 0 || t > pos - p.window);
+          const bool keep = t <= pos && (p.window <= 0 || t > pos - p.window || t < p.keep_first);
           if (keep) mx = fmaxf(mx, __uint_as_float(v[i]));
         }
       }
@@ -289,7 +306,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           const int t = t0 + c * 32 + i;
-          const bool keep = t <= pos && (p.window <= 0 || t > pos - p.window);
+          const bool keep = t <= pos && (p.window <= 0 || t > pos - p.window || t < p.keep_first);
           pv[i] = keep ? ex2a(__uint_as_float(v[i]) * p.scale_log2 - m_sub) : 0.f;
           l_sum += pv[i];
         }
@@ -303,6 +320,16 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
           o4.z = pack_bf16x2(pv[i * 8 + 4], pv[i * 8 + 5]);
           o4.w = pack_bf16x2(pv[i * 8 + 6], pv[i * 8 + 7]);
           *reinterpret_cast<uint4*>(base + ((ch ^ (r & 7)) * 16)) = o4;
+          if constexpr (EXACT) {
+            float lo[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) lo[e] = pv[i * 8 + e] - __bfloat162float(__float2bfloat16(pv[i * 8 + e]));
+            o4.x = pack_bf16x2(lo[0], lo[1]);
+            o4.y = pack_bf16x2(lo[2], lo[3]);
+            o4.z = pack_bf16x2(lo[4], lo[5]);
+            o4.w = pack_bf16x2(lo[6], lo[7]);
+            *reinterpret_cast<uint4*>(base + 2 * kHalfBytes + ((ch ^ (r & 7)) * 16)) = o4;
+          }
         }
       }
       // S buffer may be overwritten; P is ready for the tensor core
@@ -323,7 +350,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     if (ok && n_tiles > 0) {
       tc_fence_after_sync();
       const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
-      __nv_bfloat16* orow = p.out + static_cast<long long>(row_base + qi) * p.out_stride + head * D;
+      const int od = p.out_d > 0 ? p.out_d : D;  // values stored per head
+      const bool out_vec = (od & 7) == 0 && (p.out_stride & 7) == 0;
+      __nv_bfloat16* orow = p.out + static_cast<long long>(row_base + qi) * p.out_stride + head * od;
 #pragma unroll 1
       for (int c = 0; c < D / 32; ++c) {
         uint32_t v[32];
@@ -337,7 +366,13 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             o4.y = pack_bf16x2(__uint_as_float(v[i + 2]) * inv, __uint_as_float(v[i + 3]) * inv);
             o4.z = pack_bf16x2(__uint_as_float(v[i + 4]) * inv, __uint_as_float(v[i + 5]) * inv);
             o4.w = pack_bf16x2(__uint_as_float(v[i + 6]) * inv, __uint_as_float(v[i + 7]) * inv);
-            *reinterpret_cast<uint4*>(orow + c * 32 + i) = o4;
+            if (out_vec) {
+              if (c * 32 + i < od) *reinterpret_cast<uint4*>(orow + c * 32 + i) = o4;
+            } else {
+#pragma unroll
+              for (int e = 0; e < 8; ++e)
+                if (c * 32 + i + e < od) orow[c * 32 + i + e] = __float2bfloat16(__uint_as_float(v[i + e]) * inv);
+            }
           }
         }
       }
@@ -352,11 +387,11 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
   }
 }
 
-template <int D>
+template <int D, bool EXACT>
 void launch_tc(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV,
                const PrefillAttnParams& p, int n_tiles, int* status, cudaStream_t stream) {
-  using L = Smem<D>;
-  auto kern = prefill_tc_kernel<D>;
+  using L = Smem<D, EXACT>;
+  auto kern = prefill_tc_kernel<D, EXACT>;
   ensure_dynamic_smem(kern, L::kTotal);
   dim3 grid(n_tiles, p.Hq);
   kern<<<grid, kThreads, L::kTotal, stream>>>(tmQ, tmK, tmV, p, status);
@@ -368,10 +403,13 @@ void launch_paged_prefill_tc(const CUtensorMap& tmQ, const CUtensorMap& tmK, con
                              const PrefillAttnParams& p, int n_tiles, int head_dim, int* status,
                              cudaStream_t stream) {
   if (n_tiles <= 0) return;
-  if (head_dim == 128)
-    launch_tc<128>(tmQ, tmK, tmV, p, n_tiles, status, stream);
-  else
-    launch_tc<64>(tmQ, tmK, tmV, p, n_tiles, status, stream);
+  if (head_dim == 128) {
+    if (p.exact_p != 0) launch_tc<128, true>(tmQ, tmK, tmV, p, n_tiles, status, stream);
+    else launch_tc<128, false>(tmQ, tmK, tmV, p, n_tiles, status, stream);
+  } else {
+    if (p.exact_p != 0) launch_tc<64, true>(tmQ, tmK, tmV, p, n_tiles, status, stream);
+    else launch_tc<64, false>(tmQ, tmK, tmV, p, n_tiles, status, stream);
+  }
 }
 
 }  // namespace oxb

@@ -622,6 +622,7 @@ __global__ void advance_decode_step_kernel(const AdvanceStepParams p) {
       if (blk >= p.max_blocks) {
         if (p.status != nullptr) atomicCAS(p.status, 0, kStatusBadIndex);
       } else {
+        if (p.prev_ids != nullptr) p.prev_ids[r] = p.token_ids[r];
         p.token_ids[r] = tok;
         p.positions[r] = pos;
         p.seq_lens[r] += 1;

@@ -110,6 +110,7 @@ void launch_softcap(float* logits, long long n, float cap, cudaStream_t stream);
 // the device and counts from 1.
 struct AdvanceStepParams {
   int* token_ids;            // [rows]
+  int* prev_ids;             // [rows] the token before it in the sequence, or nullptr
   int* positions;            // [rows]
   long long* slot_mapping;   // [rows]
   int* seq_lens;             // [rows]

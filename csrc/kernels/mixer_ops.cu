@@ -1,0 +1,224 @@
+// Projections -> heads (sm_100a): RMS norm over the whole q / k projection, rotation in either pair layout
+// on the first dimensions of every head, write of k and v into the paged cache (or of q and k to dense
+// fp32 buffers for a recurrence); plus plain fp32 pieces of the 32-bit path (GEMM, gated unit).
+#include "../common/device_info.h"
+#include "hybrid_dev.cuh"
+
+namespace oxb {
+
+namespace {
+
+// grid (rows, head ranges): a range of the H + G (+ G value) heads per CTA. The norm spans heads of other
+// CTAs: each CTA re-reads the row's q / k (a few KB from L2) for the sum of squares it needs.
+// T: storage type (cache, dense q of the attention), TQ: type of q_out, P: type of the projection rows.
+template <typename T, typename TQ, typename P>
+__global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
+  extern __shared__ float s_mem[];
+  __shared__ float s_red[32];
+  pdl_launch_dependents();
+  const int rot2 = p.rot.dims >> 1;
+  float* s_sin = s_mem;
+  float* s_cos = s_mem + rot2;
+  pdl_wait();  // the projection comes from the kernel before this one
+  const int row = blockIdx.x;
+  const int H = p.H, G = p.G, D = p.D, E = p.E;
+  const int n_heads = H + G + (p.v_cache != nullptr ? G : 0);
+  const int hpc = (n_heads + gridDim.y - 1) / gridDim.y;
+  const int h_lo = blockIdx.y * hpc;
+  const int h_hi = min(h_lo + hpc, n_heads);
+  if (h_lo >= h_hi) return;
+  const P* pr = static_cast<const P*>(p.proj) + static_cast<long long>(row) * p.ld;
+  const int pos = p.positions[row];
+  if (h_lo < H + G)
+    for (int i = threadIdx.x; i < rot2; i += blockDim.x) rotary_sincos(p.rot, i, pos, &s_sin[i], &s_cos[i]);
+  float rq = 1.f, rk = 1.f;
+  if (p.q_norm != nullptr) {
+    if (h_lo < H) {
+      float ss = 0.f;
+      for (int c = threadIdx.x; c < H * D; c += blockDim.x) {
+        const float v = to_f(pr[c]);
+        ss = fmaf(v, v, ss);
+      }
+      rq = 1.f / sqrtf(block_sum_all(ss, s_red) / static_cast<float>(H * D) + p.eps);
+    }
+    if (h_lo < H + G && h_hi > H) {
+      float ss = 0.f;
+      for (int c = threadIdx.x; c < G * D; c += blockDim.x) {
+        const float v = to_f(pr[H * D + c]);
+        ss = fmaf(v, v, ss);
+      }
+      rk = 1.f / sqrtf(block_sum_all(ss, s_red) / static_cast<float>(G * D) + p.eps);
+    }
+  }
+  __syncthreads();
+  const long long slot = p.slots != nullptr ? p.slots[row] : -1;
+  const bool store_kv = slot >= 0 && slot < p.num_slots;
+  if (p.slots != nullptr && slot >= p.num_slots && threadIdx.x == 0) set_status_once(p.status, kStatusBadIndex);
+  const long long blk = slot >> 4;
+  const int off = static_cast<int>(slot & 15);
+
+  // q and k heads: one item per rotation pair, one per dimension that passes
+  const int r_hi = min(h_hi, H + G);
+  const int items = D - rot2;
+  for (int i = threadIdx.x; i < (r_hi - h_lo) * items; i += blockDim.x) {
+    const int h = h_lo + i / items, it = i % items;
+    const bool is_q = h < H;
+    const int base = h * D;  // k follows q in the projection row
+    const float r = is_q ? rq : rk;
+    const float* w = is_q ? p.q_norm : p.k_norm;
+    const int wo = is_q ? base : base - H * D;
+    int d0, d1 = -1;
+    float y0, y1 = 0.f;
+    if (it < rot2) {
+      rotary_pair(p.rot, it, &d0, &d1);
+      float u = to_f(pr[base + d0]) * r, v = to_f(pr[base + d1]) * r;
+      if (w != nullptr) {
+        u *= w[wo + d0];
+        v *= w[wo + d1];
+      }
+      y0 = u * s_cos[it] - v * s_sin[it];
+      y1 = v * s_cos[it] + u * s_sin[it];
+    } else {
+      d0 = rot2 + it;
+      y0 = to_f(pr[base + d0]) * r;
+      if (w != nullptr) y0 *= w[wo + d0];
+    }
+    if (is_q) {
+      TQ* q = static_cast<TQ*>(p.q_out) + static_cast<long long>(row) * p.q_ld + h * p.q_hd;
+      q[d0] = from_f<TQ>(y0);
+      if (d1 >= 0) q[d1] = from_f<TQ>(y1);
+    } else if (p.k_out != nullptr) {
+      float* k = p.k_out + static_cast<long long>(row) * p.k_ld + (h - H) * p.k_hd;
+      k[d0] = y0 * p.k_scale;
+      if (d1 >= 0) k[d1] = y1 * p.k_scale;
+    } else if (store_kv) {
+      T* k = static_cast<T*>(p.k_cache) + ((blk * G + (h - H)) * 16 + off) * p.DP;
+      k[d0] = from_f<T>(y0 * p.k_scale);
+      if (d1 >= 0) k[d1] = from_f<T>(y1 * p.k_scale);
+    }
+  }
+  if (store_kv && h_hi > H + G) {
+    const int v_lo = max(h_lo, H + G);
+    const P* vr = pr + (H + G) * D;
+    for (int i = threadIdx.x; i < (h_hi - v_lo) * E; i += blockDim.x) {
+      const int g = v_lo - H - G + i / E, e = i % E;
+      static_cast<T*>(p.v_cache)[((blk * G + g) * 16 + off) * p.EP + e] = from_f<T>(to_f(vr[g * E + e]));
+    }
+  }
+}
+
+constexpr int kFT = 64, kFK = 16;
+
+// 64 x 64 tiles, 256 threads of 4 x 4 outputs, K in steps of 16.
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* a, long long lda, const float* w, long long ldw,
+                                                       float* out, long long ldo, int M, int N, int K) {
+  __shared__ float sa[kFK][kFT + 4], sw[kFK][kFT + 4];
+  pdl_wait();
+  const int m0 = blockIdx.y * kFT, n0 = blockIdx.x * kFT;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += kFK) {
+    for (int i = threadIdx.x; i < kFT * kFK; i += 256) {
+      const int r = i / kFK, c = i % kFK;
+      const bool kin = k0 + c < K;
+      sa[c][r] = (kin && m0 + r < M) ? a[static_cast<long long>(m0 + r) * lda + k0 + c] : 0.f;
+      sw[c][r] = (kin && n0 + r < N) ? w[static_cast<long long>(n0 + r) * ldw + k0 + c] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kFK; ++k) {
+      float x[4], y[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        x[i] = sa[k][ty * 4 + i];
+        y[i] = sw[k][tx * 4 + i];
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(x[i], y[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (m0 + ty * 4 + i < M && n0 + tx * 4 + j < N)
+        out[static_cast<long long>(m0 + ty * 4 + i) * ldo + n0 + tx * 4 + j] = acc[i][j];
+}
+
+// Few rows: one warp per output column, the row values re-read from cache.
+constexpr int kFewRows = 8;
+__global__ void __launch_bounds__(256) gemv_f32_kernel(const float* a, long long lda, const float* w, long long ldw,
+                                                       float* out, long long ldo, int M, int N, int K) {
+  pdl_wait();
+  const int n = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (n >= N) return;
+  float acc[kFewRows] = {};
+  for (int k = lane; k < K; k += 32) {
+    const float wv = w[static_cast<long long>(n) * ldw + k];
+#pragma unroll
+    for (int m = 0; m < kFewRows; ++m)
+      if (m < M) acc[m] = fmaf(a[static_cast<long long>(m) * lda + k], wv, acc[m]);
+  }
+#pragma unroll
+  for (int m = 0; m < kFewRows; ++m) {
+    const float v = warp_sum(acc[m]);
+    if (lane == 0 && m < M) out[static_cast<long long>(m) * ldo + n] = v;
+  }
+}
+
+__global__ void __launch_bounds__(256) glu_f32_kernel(const float* gu, long long ldg, float* out, long long ldo, int M,
+                                                      int I, int act) {
+  pdl_wait();
+  const long long total = static_cast<long long>(M) * I;
+  for (long long i = blockIdx.x * 256ll + threadIdx.x; i < total; i += gridDim.x * 256ll) {
+    const long long m = i / I;
+    const int c = static_cast<int>(i - m * I);
+    const float g = gu[m * ldg + c], u = gu[m * ldg + I + c];
+    const float a = act == 0 ? silu_f(g)
+                             : 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+    out[m * ldo + c] = a * u;
+  }
+}
+
+}  // namespace
+
+cudaError_t launch_heads(const HeadsParams& p, int dtype, cudaStream_t stream) {
+  if (p.M <= 0) return cudaSuccess;
+  const int n_heads = p.H + p.G + (p.v_cache != nullptr ? p.G : 0);
+  // ranges of at least 4 heads until about two CTAs per SM exist
+  int chunks = (2 * sm_count() + p.M - 1) / p.M;
+  chunks = chunks > n_heads / 4 ? n_heads / 4 : chunks;
+  if (chunks < 1) chunks = 1;
+  const size_t smem = static_cast<size_t>(p.rot.dims) * sizeof(float);
+  const dim3 grid(p.M, chunks), block(256);
+  using bf16 = __nv_bfloat16;
+  auto kern = dtype == 1          ? heads_kernel<float, float, float>
+              : p.k_out != nullptr ? (p.proj_f32 ? heads_kernel<bf16, float, float> : heads_kernel<bf16, float, bf16>)
+                                   : (p.proj_f32 ? heads_kernel<bf16, bf16, float> : heads_kernel<bf16, bf16, bf16>);
+  return launch_kernel(kern, grid, block, smem, stream, true, false, p);
+}
+
+cudaError_t launch_gemm_f32(const float* a, long long lda, const float* w, long long ldw, float* out, long long ldo,
+                            int M, int N, int K, cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return cudaSuccess;
+  if (M <= kFewRows)
+    return launch_kernel(gemv_f32_kernel, dim3((N + 7) / 8), dim3(256), 0, stream, true, false, a, lda, w, ldw, out,
+                         ldo, M, N, K);
+  return launch_kernel(gemm_f32_kernel, dim3((N + kFT - 1) / kFT, (M + kFT - 1) / kFT), dim3(256), 0, stream, true,
+                       false, a, lda, w, ldw, out, ldo, M, N, K);
+}
+
+cudaError_t launch_glu_f32(const float* gu, long long ldg, float* out, long long ldo, int M, int I, int act,
+                           cudaStream_t stream) {
+  const long long total = static_cast<long long>(M) * I;
+  if (total <= 0) return cudaSuccess;
+  long long blocks = (total + 255) / 256;
+  if (blocks > sm_count() * 16) blocks = sm_count() * 16;
+  return launch_kernel(glu_f32_kernel, dim3(static_cast<unsigned>(blocks)), dim3(256), 0, stream, true, false, gu, ldg,
+                       out, ldo, M, I, act);
+}
+
+}  // namespace oxb

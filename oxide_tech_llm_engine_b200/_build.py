@@ -1,9 +1,11 @@
 """In-tree build and loading of the native extensions.
 
-Two extensions live beside this file after a build:
+These extensions live beside this file after a build:
 
 * ``oxb_cuda``  - the sm_100a kernels (``csrc/kernels/*.cu`` + ``csrc/bindings.cpp``), compiled with
   ``-gencode arch=compute_100a,code=sm_100a``; nvcc cross-compiles them on a machine without a GPU.
+* ``oxb_hybrid`` - the kernels that only layer-list decoders use (``HYBRID_KERNELS`` +
+  ``csrc/bindings_hybrid.cpp``); built when such a model is first loaded.
 * ``oxb_host``  - the C++ host runtime (block manager, radix prefix cache, scheduler core, GGUF
   block codecs); no CUDA dependency, so CPU-only tests can import it.
 
@@ -40,9 +42,16 @@ CUDA_FLAGS = [
 ]
 
 
+# kernels of the extension that only layer-list decoders load
+HYBRID_KERNELS = ("stream_ops.cu", "mixer_ops.cu", "attn_rows.cu", "retention.cu")
+HYBRID_HEADERS = ("hybrid.cuh", "hybrid_dev.cuh")
+
+
 def _sources(name: str) -> list[Path]:
     if name == "oxb_cuda":
-        return sorted((_CSRC / "kernels").glob("*.cu")) + [_CSRC / "bindings.cpp"]
+        return sorted(p for p in (_CSRC / "kernels").glob("*.cu") if p.name not in HYBRID_KERNELS) + [_CSRC / "bindings.cpp"]
+    if name == "oxb_hybrid":
+        return [_CSRC / "kernels" / k for k in HYBRID_KERNELS] + [_CSRC / "bindings_hybrid.cpp"]
     if name == "oxb_host":
         return sorted((_CSRC / "host").glob("*.cpp"))
     raise KeyError(name)
@@ -53,7 +62,10 @@ def _headers(name: str) -> list[Path]:
     not make this one stale)."""
     if name == "oxb_host":
         return sorted((_CSRC / "host").glob("*.h"))
-    return sorted(list((_CSRC / "common").glob("*")) + list((_CSRC / "kernels").glob("*.cuh")))
+    common = list((_CSRC / "common").glob("*"))
+    if name == "oxb_hybrid":
+        return sorted(common + [_CSRC / "kernels" / h for h in HYBRID_HEADERS])
+    return sorted(common + [p for p in (_CSRC / "kernels").glob("*.cuh") if p.name not in HYBRID_HEADERS])
 
 
 def source_hash(name: str) -> str:
@@ -94,7 +106,7 @@ def build(name: str, verbose: bool = False) -> Path:
         verbose=verbose,
         is_python_module=True,
     )
-    if name == "oxb_cuda":
+    if name != "oxb_host":
         kwargs["extra_cuda_cflags"] = CUDA_FLAGS
         kwargs["with_cuda"] = True
     os.environ.setdefault("MAX_JOBS", str(os.cpu_count() or 8))
@@ -159,7 +171,7 @@ def _load_locked(name: str):
         import shutil
 
         have_compiler = shutil.which("g++") is not None and (
-            name != "oxb_cuda" or shutil.which("nvcc") is not None
+            name == "oxb_host" or shutil.which("nvcc") is not None
         )
         if have_compiler and os.environ.get("OXB_NO_BUILD", "0") != "1":
             build(name)
@@ -218,6 +230,10 @@ def noalloc_lib_path() -> Path:
 
 def cuda_ext():
     return load("oxb_cuda")
+
+
+def hybrid_ext():
+    return load("oxb_hybrid")
 
 
 def host_ext():

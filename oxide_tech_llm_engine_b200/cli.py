@@ -55,6 +55,8 @@ def add_common(p: argparse.ArgumentParser) -> None:
     p.add_argument("--n-gpu-layers", type=int, default=-1)
     p.add_argument("-b", "--backend", default="auto")
     p.add_argument("--weights", default="auto", choices=["auto", "bf16", "quant", "fp8"])
+    p.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
+                   help="float32: weights, activations and KV in 32-bit (layer-list models)")
     p.add_argument("--max-slots", type=int, default=64)
     p.add_argument("--gpu", type=int, default=0)
     p.add_argument("-p", "--prompt")
@@ -147,7 +149,7 @@ def engine_config_from_args(args) -> EngineConfig:
         max_num_seqs=args.max_slots, num_kv_blocks=args.kv_device_blocks, seed=args.seed, backend=be,
         weight_mode=args.weights, speculative=spec, draft_tokens=args.draft_tokens, tp=args.tp, dp=args.dp,
         max_num_batched_tokens=args.max_batched_tokens, cuda_graph=not args.no_cuda_graph,
-        enable_radix=not args.no_radix, kv_host_blocks=args.kv_host_blocks, kv_storage_blocks=args.kv_storage_blocks,
+        enable_radix=not args.no_radix, dtype=args.dtype, kv_host_blocks=args.kv_host_blocks, kv_storage_blocks=args.kv_storage_blocks,
         kv_storage_dir=args.kv_storage_dir, kv_host_quant=args.kv_host_quant, decode_burst=args.decode_burst)
 
 

@@ -20,6 +20,7 @@ class EngineConfig:
     alias: Optional[str] = None
     models_dir: Optional[str] = None
     weight_mode: str = "auto"           # auto | bf16 | quant | fp8  (quant: GGUF blocks packed in HBM; fp8: 128x128 block-scaled e4m3)
+    dtype: str = "bfloat16"             # bfloat16 | float32 (weights, activations and KV in 32-bit: layer-list models)
     tp: int = 1
     pp: int = 1
     dp: int = 1

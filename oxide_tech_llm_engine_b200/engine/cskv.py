@@ -138,11 +138,18 @@ def read_dense(path: str) -> tuple[CskvHeader, list[np.ndarray], list[np.ndarray
     return h, ks, vs
 
 
+def _needs_uniform_kv(engine) -> None:
+    if engine.model_cfg.layers:
+        raise EngineError(f"{engine.model_cfg.name}: a state file holds K and V of one shape per layer; layer-list "
+                          "models (several cache shapes, recurrent states) are not stored")
+
+
 def save_sequence(engine, req_id: int, path: str, f16: bool = True) -> CskvHeader:
     """Gathers the pages of a running or just-finished request into a CSKV file (per rank: this
     rank's KV-head shard; rank 0 also writes `<path>.manifest.json`)."""
     import torch
 
+    _needs_uniform_kv(engine)
     info = engine.sched.request_info(req_id)
     if info is None:
         raise EngineError(f"request {req_id} is not resident")
@@ -174,6 +181,7 @@ def load_prefix(engine, path: str) -> int:
     resumes without recomputation. Returns the number of tokens restored (whole blocks)."""
     import torch
 
+    _needs_uniform_kv(engine)
     man = json.load(open(path + ".manifest.json"))
     rank, world = getattr(engine, "rank", 0), getattr(engine, "world", 1)
     if man["world"] != world:

@@ -26,7 +26,8 @@ from .._build import host_ext
 from ..config import EngineConfig
 from ..errors import ConfigError, EngineError, OutOfMemory
 from ..models.config import ModelConfig, preset
-from ..models.llama import DeviceModel, StepInputs
+from ..models.llama import StepInputs
+from ..models.registry import architecture
 from ..sampling_params import SamplingParams
 
 
@@ -107,12 +108,18 @@ class LLMEngine:
             return
         self.device = device or torch.device("cuda", torch.cuda.current_device())
         if model_cfg is None:
+            if weights is None and not random_init and os.path.exists(cfg.model):
+                from ..models.weights import open_weights
+
+                weights = open_weights(cfg.model)
             if weights is not None:
                 model_cfg = weights.cfg
             else:
                 model_cfg = preset(cfg.model)
         self.model_cfg = model_cfg
         mc = model_cfg
+        model_cls = architecture(mc).device_model()
+        self._check_features(cfg, mc)
         H = host_ext()
         self.block = H.TOKENS_PER_BLOCK
         max_blocks_per_seq = (min(cfg.ctx_size, mc.max_ctx) + self.block - 1) // self.block
@@ -139,13 +146,16 @@ class LLMEngine:
         num_blocks = cfg.num_kv_blocks
         if num_blocks <= 0:
             num_blocks = self._auto_blocks(mc, weight_mode, random_init or weights is not None)
-        self.model = DeviceModel(mc, rank=rank, world=world, group=group, device=self.device,
+        # one recurrent-state slot per sequence that may run (0 for models without such state)
+        state_slots = cfg.max_num_seqs if mc.is_recurrent else 0
+        self.model = model_cls(mc, rank=rank, world=world, group=group, device=self.device,
                                  max_tokens=self.max_tokens, max_seqs=cfg.max_num_seqs,
                                  num_blocks=num_blocks, max_blocks_per_seq=max_blocks_per_seq,
                                  max_logits=max(cfg.max_num_seqs * (1 + (cfg.draft_tokens if cfg.speculative != "off" else 0)), 64),
                                  max_splits=cfg.max_splits, weight_mode=weight_mode,
                                  tile_weights=False if (cfg.comm == "nccl" or cfg.gemm == "library") else None,
-                                 layer_range=pp.layers(mc.n_layers) if pp is not None else None)
+                                 layer_range=pp.layers(mc.n_layers) if pp is not None else None,
+                                 dtype=cfg.dtype, state_slots=state_slots)
         if cfg.h2o_pruning:
             self.model.enable_block_mass()
         if pp is not None:
@@ -173,6 +183,7 @@ class LLMEngine:
         sc.sla_budget = cfg.sla_budget
         sc.context_shift, sc.shift_keep_tokens, sc.shift_step_tokens = (cfg.context_shift, cfg.shift_keep_tokens,
                                                                         cfg.shift_step_tokens)
+        sc.state_slots = state_slots
         self.sched = H.Scheduler(sc)
         self._init_kv_tiers()
         self.max_blocks_per_seq = max_blocks_per_seq
@@ -181,8 +192,9 @@ class LLMEngine:
         i32, i64 = np.int32, np.int64
         self.st = _Staging({
             "token_ids": (M, i32), "positions": (M, i32), "logit_map": (M, i32), "slot_mapping": (M, i64),
-            "pages_per_split": (4, i32), "seq_lens": (S, i32), "block_tables": (S * max_blocks_per_seq, i32),
-            "q_start": (S, i32), "q_lens": (S, i32), "ctx_lens": (S, i32), "tile_seq": (n_tiles_max, i32),
+            "prev_ids": (M, i32), "decode_slots": (S, i32), "pages_per_split": (4, i32), "seq_lens": (S, i32), "block_tables": (S * max_blocks_per_seq, i32),
+            "q_start": (S, i32), "q_lens": (S, i32), "ctx_lens": (S, i32), "prefill_slots": (S, i32),
+            "tile_seq": (n_tiles_max, i32),
             "tile_q0": (n_tiles_max, i32), "prefill_block_tables": (S * max_blocks_per_seq, i32),
             "cow_src": (S, i32), "cow_dst": (S, i32),
             "temperature": (self.model.max_logits, np.float32), "top_k": (self.model.max_logits, i32),
@@ -217,14 +229,25 @@ class LLMEngine:
                       "h2d_bytes": 0, "d2h_bytes": 0, "degraded": False}
         self.stop_ids_default = [mc.eos_id]
         self._drafter = None
-        if cfg.speculative in ("ngram", "auto"):
+        # a recurrent state cannot be cut back to the accepted drafts, so such models decode without them
+        if cfg.speculative in ("ngram", "auto") and not mc.is_recurrent:
             from .spec_decode import NgramDrafter
 
             self._drafter = NgramDrafter(cfg.draft_tokens)
 
+    @staticmethod
+    def _check_features(cfg: EngineConfig, mc: ModelConfig) -> None:
+        """Options that address the KV cache as the whole past of a sequence do not fit layer-list models
+        (fixed windows by true position, recurrent states); they are refused rather than ignored."""
+        if not mc.layers:
+            return
+        for on, what in ((cfg.h2o_pruning, "h2o_pruning"), (cfg.context_shift, "context_shift"),
+                         (cfg.comm == "nccl", "comm='nccl'"), (cfg.gemm == "library", "gemm='library'")):
+            if on:
+                raise ConfigError(f"{mc.name}: {what} is not available for layer-list models")
+
     def _init_cpu(self, cfg: EngineConfig, model_cfg, weights) -> None:
         """fp32 torch backend over the same scheduler / block manager (no GPU needed)."""
-        from ..models.cpu_model import CpuPagedModel
         from ..models.weights import SyntheticSource
 
         self.device = torch.device("cpu")
@@ -233,12 +256,14 @@ class LLMEngine:
         if weights is None:
             weights = SyntheticSource(model_cfg, seed=cfg.seed)
         self.model_cfg = mc = model_cfg
+        self._check_features(cfg, mc)
+        state_slots = cfg.max_num_seqs if mc.is_recurrent else 0
         H = host_ext()
         self.block = H.TOKENS_PER_BLOCK
         self.max_blocks_per_seq = (min(cfg.ctx_size, mc.max_ctx) + self.block - 1) // self.block
         num_blocks = cfg.num_kv_blocks if cfg.num_kv_blocks > 0 else min(
             4096, cfg.max_num_seqs * self.max_blocks_per_seq + 16)
-        self.model = CpuPagedModel(mc, weights, num_blocks)
+        self.model = architecture(mc).cpu_model()(mc, weights, num_blocks, state_slots=state_slots)
         sc = H.SchedulerConfig()
         sc.num_blocks = num_blocks
         sc.max_num_seqs = cfg.max_num_seqs
@@ -250,6 +275,7 @@ class LLMEngine:
         sc.sla_budget = cfg.sla_budget
         sc.context_shift, sc.shift_keep_tokens, sc.shift_step_tokens = (cfg.context_shift, cfg.shift_keep_tokens,
                                                                         cfg.shift_step_tokens)
+        sc.state_slots = state_slots
         self.sched = H.Scheduler(sc)
         self._init_kv_tiers()
         self.requests = {}
@@ -259,7 +285,8 @@ class LLMEngine:
                       "h2d_bytes": 0, "d2h_bytes": 0, "degraded": False}
         self.stop_ids_default = [mc.eos_id]
         self._drafter = None
-        if cfg.speculative in ("ngram", "auto"):
+        # a recurrent state cannot be cut back to the accepted drafts, so such models decode without them
+        if cfg.speculative in ("ngram", "auto") and not mc.is_recurrent:
             from .spec_decode import NgramDrafter
 
             self._drafter = NgramDrafter(cfg.draft_tokens)
@@ -296,12 +323,20 @@ class LLMEngine:
             per = {"bf16": 2.0, "fp8": 1.02, "nvfp4": 0.7}.get(weight_mode, 0.6)
             n = mc.n_params()
             w_bytes = int((n - mc.vocab_size * mc.d_model) / tp * per + mc.vocab_size * mc.d_model * 2)
+        model_cls = architecture(mc).device_model()
         act = self.max_tokens * (mc.d_model * 16 + (mc.q_dim + 2 * mc.kv_dim) // tp * 8 + mc.ffn_dim // tp * 4)
         act += self.cfg.max_num_seqs * (mc.vocab_size // tp) * 4 * 2
         if mc.is_moe:
             act += (mc.n_experts // tp) * self.max_tokens * (mc.d_model + mc.ffn_dim) * 2
         budget = int(free * self.cfg.gpu_memory_utilization) - w_bytes - act - (2 << 30) - getattr(self, "_dense_bytes", 0)
-        per_block = 2 * mc.n_layers * (mc.n_kv_heads // tp) * 16 * mc.head_dim * 2
+        budget -= self.cfg.max_num_seqs * model_cls.state_bytes_per_seq(mc)
+        if mc.layers:
+            # streams, fp32 projections, rotated q / k and the chunk states of one prompt step
+            wide = max((L.mixer.heads * (L.mixer.dim + L.mixer.vdim) for L in mc.layers))
+            chunk = max((L.mixer.state_elems for L in mc.layers if L.mixer.kind == "retention"), default=0)
+            budget -= self.max_tokens * 4 * (max(1, mc.streams) * mc.d_model + 6 * wide)
+            budget -= 8 * (self.max_tokens // 128 + self.cfg.max_num_seqs) * chunk
+        per_block = max(1, model_cls.kv_block_bytes(mc, tp, self.cfg.dtype))
         n = budget // per_block
         if n < 16:
             raise OutOfMemory(f"not enough device memory for the KV pool ({budget} bytes left for blocks)")
@@ -379,6 +414,9 @@ class LLMEngine:
         tok[n:m] = 0
         pos[n:m] = 0
         slot[n:m] = -1
+        prev = h("prev_ids")
+        prev[:n] = plan.prev_ids
+        prev[n:m] = -1
         rows = plan.logit_rows
         if bucket is not None:
             lmap[:m] = np.arange(m, dtype=np.int32)  # graph buckets compute logits for every row
@@ -392,6 +430,9 @@ class LLMEngine:
             sl = h("seq_lens")
             sl[:nd] = plan.decode_seq_lens
             sl[nd:nd_pad] = 0
+            ds = h("decode_slots")
+            ds[:nd] = plan.decode_slots
+            ds[nd:nd_pad] = -1
             bt = h("block_tables").reshape(-1, W)
             bt[:nd, :w] = plan.decode_block_tables.reshape(nd, w)
             max_len = int(plan.decode_seq_lens.max()) + extra_len
@@ -410,6 +451,7 @@ class LLMEngine:
             h("q_start")[:npf] = plan.q_start
             h("q_lens")[:npf] = plan.q_lens
             h("ctx_lens")[:npf] = plan.ctx_lens
+            h("prefill_slots")[:npf] = plan.prefill_slots
             n_tiles = plan.tile_seq.size
             h("tile_seq")[:n_tiles] = plan.tile_seq
             h("tile_q0")[:n_tiles] = plan.tile_q0
@@ -428,11 +470,10 @@ class LLMEngine:
                        seq_lens=d("seq_lens"), block_tables=d("block_tables").view(-1, W),
                        pages_per_split=d("pages_per_split"), tile_seq=d("tile_seq"), tile_q0=d("tile_q0"),
                        q_start=d("q_start"), q_lens=d("q_lens"), ctx_lens=d("ctx_lens"),
-                       prefill_block_tables=d("prefill_block_tables").view(-1, W), logit_map=d("logit_map"))
+                       prefill_block_tables=d("prefill_block_tables").view(-1, W), logit_map=d("logit_map"),
+                       prev_ids=d("prev_ids"), decode_slots=d("decode_slots"), prefill_slots=d("prefill_slots"))
         if n_cow:
-            for li in range(self.model_cfg.n_layers):
-                ops.kv_block_copy(self.model.k_cache[li], self.model.v_cache[li], d("cow_src")[:n_cow],
-                                  d("cow_dst")[:n_cow])
+            self.model.copy_blocks(d("cow_src")[:n_cow], d("cow_dst")[:n_cow])
         return s, bucket
 
     def _forward(self, s: StepInputs, bucket: Optional[int]) -> torch.Tensor:
@@ -453,7 +494,8 @@ class LLMEngine:
                 fwd(s)
             self.graph_launches[bucket] = ops.launch_count - c0
             self.graphs[bucket] = g
-            # the capture did not execute; the warm-up run already produced this step's state
+            # the capture did not execute; the warm-up run already produced this step's state (kernels
+            # that update a state in place run once)
             return self.model.logits[:s.n_logits]
         g.replay()
         ops.launch_count += self.graph_launches[bucket]  # kernels inside the replayed graph
@@ -526,7 +568,8 @@ class LLMEngine:
         the library-GEMM + NCCL all-reduce path, and compares the sampled tokens and the logits.
         The fused result is the one the scheduler advances with. Used by bench.py as evidence that
         the fused multi-rank path computes what the plain one does."""
-        if self.cpu or self.model.weight_mode != "bf16" or self.model_cfg.is_moe or self.pp is not None:
+        if (self.cpu or self.model.weight_mode != "bf16" or self.model_cfg.is_moe or self.pp is not None
+                or not hasattr(self.model, "forward_baseline")):
             return {"steps": 0}
         same = total = 0
         worst = 0.0
@@ -654,7 +697,8 @@ class LLMEngine:
         (oxide-alloc/src/hierarchical_kv.rs:27-310: demotion T1->T2->T3 :135-173, promote on hit :207-242)."""
         self.kv_tier = None
         cfg = self.cfg
-        if cfg.kv_host_blocks > 0 and cfg.enable_radix and self.pp is None:
+        if (cfg.kv_host_blocks > 0 and cfg.enable_radix and self.pp is None
+                and getattr(self.model, "supports_kv_tiers", True)):
             from .kv_tiers import HierarchicalKvCache
 
             # every rank keeps its own shard of the KV heads: its files must not meet another rank's
@@ -1060,6 +1104,32 @@ class LLMEngine:
             self.stats["spec_proposed"] = self.stats.get("spec_proposed", 0) + r.n_drafted
             self.stats["spec_accepted"] = self.stats.get("spec_accepted", 0) + acc
             r.n_drafted = 0
+
+    # ------------------------------------------------------------------ replay of given tokens
+    def feed(self, entries: list) -> np.ndarray:
+        """One step of given tokens instead of sampled ones: `entries` = [(request id, tokens, want), ...]
+        run together as one batch through the same plan, step function, cache and kernels as generation,
+        from the KV and state that earlier steps left. A request is admitted at its first entry and lives
+        until `cancel`. Returns the fp32 logits [wanted places, vocab] in the order of the entries and
+        of their `want`."""
+        plan = self.sched.feed([(int(i), [int(t) for t in toks], [int(w) for w in want]) for i, toks, want in entries])
+        if self.cpu:
+            if plan.cow_src.size:
+                self.model.copy_blocks(plan.cow_src, plan.cow_dst)
+            out = self.model.forward_plan(plan).numpy().copy()
+        else:
+            s, bucket = self._fill(plan)
+            logits = self._forward(s, bucket)
+            # a decode bucket has a logits row for every token row, other steps one per wanted place
+            if bucket is not None:
+                logits = logits[torch.as_tensor(plan.logit_rows.astype(np.int64), device=self.device)]
+            out = logits[:plan.logit_rows.size].float().cpu().numpy()
+            self.check_device_status()
+        self.sched.feed_done(plan)
+        self.stats["steps"] += 1
+        self.stats["decode_tokens"] += plan.n_decode
+        self.stats["prefill_tokens"] += plan.prefill_tokens
+        return out
 
     # ------------------------------------------------------------------ convenience
     def generate(self, prompts: list, params: Optional[SamplingParams] = None, max_steps: int = 1 << 30):

@@ -13,7 +13,7 @@ from dataclasses import dataclass
 from typing import Callable, Optional
 
 from ..errors import ModelLoadError
-from ..models.config import PRESETS
+from ..models.config import preset_names
 
 
 @dataclass
@@ -77,7 +77,7 @@ class ModelManager:
             if key in self.models:
                 return self.models[key]
         path = self.resolve_path(name)
-        if path is None and name not in PRESETS:
+        if path is None and name not in preset_names():
             raise ModelLoadError(f"model {name!r} not found (searched {self.models_dir or '.'}, ./models, catalog)")
         m = self.loader(name, path)
         self.register(m, alias)

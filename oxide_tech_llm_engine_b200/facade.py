@@ -3,6 +3,7 @@ crate (`OxideEngine::builder()`, src/lib.rs of the workspace root), mapped onto 
 `LLMEngine` and `EngineHandle`."""
 from __future__ import annotations
 
+import os
 from typing import Optional
 
 from .config import EngineConfig
@@ -78,7 +79,7 @@ class EngineBuilder:
 
         cfg = self.config()
         weights, mc = self._weights, self._model_cfg
-        if weights is None and not self._random_init and (cfg.model.endswith(".gguf") or cfg.model.endswith(".safetensors")):
+        if weights is None and not self._random_init and (cfg.model.endswith((".gguf", ".safetensors")) or os.path.isdir(cfg.model)):
             from .models.weights import open_weights
 
             weights = open_weights(cfg.model)

@@ -104,6 +104,9 @@ class SafeTensorsRepo:
     def f32(self, name):
         return self.files[self.where[name]].f32(name)
 
+    def dtype(self, name):
+        return self.files[self.where[name]].info(name)["dtype"]
+
     def model_config(self):
         from ..models.config import ModelConfig
 
@@ -111,6 +114,11 @@ class SafeTensorsRepo:
         if not os.path.exists(cfg_path):
             raise UnsupportedFormat(f"{cfg_path} is needed to size a SafeTensors model")
         c = json.load(open(cfg_path))
+        from ..models.registry import config_from_json
+
+        native = config_from_json(c)
+        if native is not None:
+            return native
         n_heads = c["num_attention_heads"]
         arch = "mixtral" if c.get("num_local_experts", 0) else "llama"
         rs = c.get("rope_scaling") or {}

@@ -46,6 +46,13 @@ class ModelConfig:
     routed_scale: float = 1.0
     bos_id: int = 1
     eos_id: int = 2
+    # layer-list designs (models.layer_spec): one LayerSpec per layer, the range of layers that runs
+    # several times, the number of hyper-connected residual streams (0: one plain residual), and the
+    # second embedding. Empty for the Llama family.
+    layers: tuple = ()
+    loop: Any = None           # (start, stop, times)
+    streams: int = 0
+    bigram: Any = None         # layer_spec.BigramSpec
 
     @property
     def q_dim(self) -> int:
@@ -59,7 +66,25 @@ class ModelConfig:
     def is_moe(self) -> bool:
         return self.n_experts > 0
 
+    @property
+    def layer_runs(self) -> list:
+        """Layer index of every layer run, in order (a looped layer counts each time)."""
+        from .layer_spec import layer_runs
+
+        return layer_runs(self.n_layers, self.loop)
+
+    @property
+    def is_recurrent(self) -> bool:
+        """Some layer carries a per-sequence state besides the paged KV."""
+        return any(L.mixer.kind == "retention" for L in self.layers)
+
     def n_params(self) -> int:
+        if self.layers:
+            from math import prod
+
+            from .layer_spec import layer_list_tensors
+
+            return sum(prod(s) for _, s in layer_list_tensors(self))
         per_layer = self.d_model * (self.q_dim + 2 * self.kv_dim) + self.q_dim * self.d_model
         ffn = 3 * self.d_model * self.ffn_dim
         per_layer += ffn * max(1, self.n_experts) + (self.n_experts * self.d_model if self.is_moe else 0)
@@ -75,6 +100,9 @@ class ModelConfig:
         return self.n_layers * per_layer + 2 * self.vocab_size * self.d_model
 
     def kv_bytes_per_token(self, dtype_bytes: int = 2) -> int:
+        if self.layers:
+            att = [self.layers[i].mixer for i in self.layer_runs if self.layers[i].mixer.kind == "attention"]
+            return sum(a.kv_heads * (a.dim + a.vdim) for a in att) * dtype_bytes
         return 2 * self.n_layers * self.kv_dim * dtype_bytes
 
     def to_dict(self) -> dict[str, Any]:
@@ -105,9 +133,43 @@ PRESETS: dict[str, ModelConfig] = {
 }
 
 
+def _kipolix_preset(name: str, *, width: int, vocab: int, ff: int, pattern: str, heads: int, kv_heads: int, dim: int,
+                    window: int, keep_first: int, r_heads: int, r_dim: int, r_vdim: int, streams: int = 2,
+                    loop=None, buckets: int = 0) -> ModelConfig:
+    """A Kipolix-shaped configuration: one letter per layer, 'a' attention or 'r' retention. Decays are
+    1 - 2^(-5 - i), the usual multi-scale choice of retention heads."""
+    from .layer_spec import AttentionSpec, BigramSpec, DenseMlpSpec, LayerSpec, RetentionSpec, RotarySpec
+
+    att = AttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, RotarySpec(dim // 2, 10000.0, True), window,
+                        keep_first, "projection")
+    ret = RetentionSpec(r_heads, r_dim, r_vdim, tuple(1.0 - 2.0 ** (-5 - 8.0 * i / max(1, r_heads)) for i in range(r_heads)),
+                        RotarySpec(r_dim, 500000.0, False))
+    mlp = DenseMlpSpec(ff)
+    layers = tuple(LayerSpec(att if ch == "a" else ret, mlp) for ch in pattern)
+    return ModelConfig(name=name, arch="kipolix", n_layers=len(layers), d_model=width, n_heads=heads, n_kv_heads=kv_heads,
+                       head_dim=dim, ffn_dim=ff, vocab_size=vocab, max_ctx=1 << 20, rms_eps=1e-5, norm_weight_offset=1.0,
+                       bos_id=-1, eos_id=-1, layers=layers, loop=loop, streams=streams,
+                       bigram=BigramSpec(buckets, 40503, 10007) if buckets else None)
+
+
+LAYER_LIST_PRESETS = {
+    "kipolix-tiny": dict(width=128, vocab=1024, ff=256, pattern="arar", heads=4, kv_heads=2, dim=64, window=56,
+                         keep_first=3, r_heads=2, r_dim=64, r_vdim=64, streams=2, loop=(1, 3, 2), buckets=1000),
+    # the shapes of llama3-8b's layers (width, FFN, heads), alternating attention and retention
+    "kipolix-8b": dict(width=4096, vocab=128256, ff=14336, pattern="ar" * 16, heads=32, kv_heads=8, dim=128, window=4096,
+                       keep_first=16, r_heads=32, r_dim=128, r_vdim=128, streams=2, buckets=65521),
+}
+
+
+def preset_names() -> list:
+    return [*PRESETS, *LAYER_LIST_PRESETS]
+
+
 def preset(name: str, **overrides) -> ModelConfig:
+    if name in LAYER_LIST_PRESETS:
+        return replace(_kipolix_preset(name, **LAYER_LIST_PRESETS[name]), **overrides)
     if name not in PRESETS:
-        raise KeyError(f"unknown model preset {name!r}; known: {sorted(PRESETS)}")
+        raise KeyError(f"unknown model preset {name!r}; known: {sorted(preset_names())}")
     return replace(PRESETS[name], **overrides)
 
 
@@ -169,6 +231,8 @@ def config_from_gguf(g) -> ModelConfig:
 
 def gguf_metadata(cfg: ModelConfig) -> dict[str, Any]:
     """Metadata block of a GGUF checkpoint for this config (inverse of config_from_gguf)."""
+    if cfg.layers:
+        raise ValueError(f"{cfg.name}: layer-list models have no GGUF form (SafeTensors with config.json)")
     a = cfg.arch
     md: dict[str, Any] = {
         "general.architecture": a,

@@ -16,7 +16,7 @@ from .weights import WeightSource
 
 
 class CpuPagedModel(ReferenceModel):
-    def __init__(self, cfg: ModelConfig, src: WeightSource, num_blocks: int):
+    def __init__(self, cfg: ModelConfig, src: WeightSource, num_blocks: int, state_slots: int = 0):
         super().__init__(cfg, src)
         self.num_blocks = num_blocks
         shape = (num_blocks, cfg.n_kv_heads, 16, cfg.head_dim)

@@ -32,6 +32,7 @@ from ..errors import ConfigError
 from ..formats import quants
 from ..parallel.comm import SymmetricWorkspace
 from .config import ModelConfig
+from .gemm_shapes import GemmShapes
 from .rope import inv_freq_table
 from .weights import WeightSource
 
@@ -69,6 +70,9 @@ class StepInputs:
     ctx_lens: Optional[torch.Tensor] = None
     prefill_block_tables: Optional[torch.Tensor] = None
     logit_map: Optional[torch.Tensor] = None  # [M] int32: logits row of each token row or -1
+    prev_ids: Optional[torch.Tensor] = None      # [M] int32: the token before it in its sequence or -1
+    decode_slots: Optional[torch.Tensor] = None  # [n_decode] int32: recurrent-state slot of each decode row (-1 = padding)
+    prefill_slots: Optional[torch.Tensor] = None  # [n_prefill] int32
 
 
 class QuantLinear:
@@ -135,12 +139,14 @@ def fuse_quant_rows(parts: list) -> Optional[QuantLinear]:
     return lin
 
 
-class DeviceModel:
+class DeviceModel(GemmShapes):
     def __init__(self, cfg: ModelConfig, *, rank: int = 0, world: int = 1, group=None,
                  device: Optional[torch.device] = None, max_tokens: int = 2048, max_seqs: int = 256,
                  num_blocks: int = 1024, max_blocks_per_seq: int = 512, max_logits: Optional[int] = None,
                  max_splits: int = 16, weight_mode: str = "bf16", tile_weights: Optional[bool] = None,
-                 layer_range: Optional[tuple] = None):
+                 layer_range: Optional[tuple] = None, dtype: str = "bfloat16", state_slots: int = 0):
+        if dtype != "bfloat16":
+            raise ConfigError(f"{cfg.name}: the Llama-family kernels run with bf16 activations, not {dtype}")
         self.cfg = cfg
         self.rank, self.tp, self.group = rank, world, group
         self.device = device or torch.device("cuda", torch.cuda.current_device())
@@ -263,6 +269,20 @@ class DeviceModel:
         self.lm_head = None
         self.out_norm = None
         self._act_code = 1 if cfg.act == "gelu_tanh" else 0
+
+    @staticmethod
+    def kv_block_bytes(cfg: ModelConfig, tp: int = 1, dtype: str = "bfloat16") -> int:
+        """Device bytes of one 16-token KV block over all layers of a rank."""
+        return 2 * cfg.n_layers * (cfg.n_kv_heads // tp) * 16 * cfg.head_dim * 2
+
+    @staticmethod
+    def state_bytes_per_seq(cfg: ModelConfig) -> int:
+        return 0
+
+    def copy_blocks(self, src: torch.Tensor, dst: torch.Tensor) -> None:
+        """Copies KV blocks src[i] -> dst[i] in every layer (copy on write)."""
+        for k, v in zip(self.k_cache, self.v_cache):
+            ops.kv_block_copy(k, v, src, dst)
 
     # ------------------------------------------------------------------ weights
     def kv_bytes(self) -> int:
@@ -511,40 +531,6 @@ class DeviceModel:
             return {}
         return dict(ag_flags=self.ws.local("flags")[flag_base:flag_base + self.tp], ag_expected=expected,
                     ag_rows_per_src=rows_per_src, ag_ticket=self.tickets[ticket:ticket + 1])
-
-    def _gemm_shape(self, m: int, n: int, k: int, *, swiglu: bool = False, routed: bool = False,
-                    store: bool = False) -> dict:
-        """Tile width, rows per tile, split-K factor and split-K mode of one projection. Steps of
-        129 to 256 rows (large decode batches) keep every row with the CTA that streams a weight
-        tile and split K to fill the SMs, combined inside the kernel; a routed projection on one GPU
-        adds its splits straight into the fp32 accumulator instead. Other steps use 128-row tiles."""
-        key = (m, n, k, swiglu, routed, store)
-        c = self._gemm_cfg.get(key)
-        if c is not None:
-            return c
-        # the in-kernel split-K costs about 10 us of partial-tile traffic and barrier: it pays for the
-        # large weight streams (gate/up, down), not for the small ones (QKV, O), measured in situ
-        big = n * k * 2 >= (48 << 20)
-        if 128 < m <= 256 and big and os.environ.get("OXB_DECODE_GEMM", "1") != "0":
-            bn, mt, sp = ops.pick_decode_cfg(m, n, k, swiglu=swiglu, sms=self._sms)
-            fixup = sp > 1 and not (routed and self.tp == 1)
-        else:
-            m_tiles = (m + 127) // 128
-            bn = ops.pick_bn(n, m_tiles, can_split=not swiglu)
-            mt = 1
-            sp = 1 if swiglu else ops.pick_splits(m, n, k, bn, self._sms)
-            fixup = False
-            if sp > 1 and (store or (routed and self.tp > 1)):
-                # these epilogues cannot add into an fp32 accumulator: combine the splits in the kernel
-                # when the launch is one wave, else do not split
-                fits = (((n + bn - 1) // bn) * m_tiles * sp <= self._sms
-                        and sp <= ops.max_fixup_splits(bn, 1, False))
-                fixup = fits
-                if not fits:
-                    sp = 1
-        c = dict(bn=bn, mt=mt, splits=sp, fixup=fixup)
-        self._gemm_cfg[key] = c
-        return c
 
     def _ag_kwargs_quant(self, flag_base: int, ticket: int, expected: int) -> dict:
         if self.tp == 1:

@@ -54,6 +54,10 @@ def hf_name_to_gguf(name: str) -> Optional[str]:
 
 def tensor_names(cfg: ModelConfig) -> list[tuple[str, tuple[int, ...]]]:
     """(name, row-major shape) of every tensor of the architecture."""
+    if cfg.layers:
+        from .layer_spec import layer_list_tensors
+
+        return layer_list_tensors(cfg)
     out = [("token_embd.weight", (cfg.vocab_size, cfg.d_model))]
     for i in range(cfg.n_layers):
         p = f"blk.{i}."
@@ -140,6 +144,15 @@ class SyntheticSource(WeightSource):
         shape = self._shapes[name]
         if name.endswith("norm.weight"):
             return np.full(shape, 1.0 - self.cfg.norm_weight_offset, dtype=np.float32)
+        if self.cfg.layers and len(shape) == 1 and ".hc" not in name:
+            # norms: q / k norms are plain weights, the others are stored as the distance from one
+            one = name.endswith((".q.norm", ".k.norm"))
+            return np.full(shape, 1.0 if one else 1.0 - self.cfg.norm_weight_offset, dtype=np.float32)
+        if ".hc" in name:
+            # hyper-connections start as an ordinary residual: read the mean of the streams, write to all
+            s = self.cfg.streams
+            return (np.eye(s, dtype=np.float32) if name.endswith(".mix")
+                    else np.full(shape, 1.0 / s if name.endswith(".in") else 1.0, dtype=np.float32))
         h = np.frombuffer(name.encode(), dtype=np.uint8).astype(np.uint64)
         key = int((h * np.arange(1, h.size + 1, dtype=np.uint64)).sum() % (2 ** 31))
         rng = np.random.default_rng([self.seed, key])
@@ -178,18 +191,28 @@ class GgufSource(WeightSource):
 
 
 class SafeTensorsSource(WeightSource):
-    """Hugging Face layout (sharded or single file) mapped onto the GGUF tensor names."""
+    """SafeTensors checkpoint (sharded or single file): the Hugging Face layout mapped onto the GGUF
+    tensor names, or the native names of a design whose registry entry says so."""
 
     def __init__(self, path: str, cfg: Optional[ModelConfig] = None):
         from ..formats.safetensors import SafeTensorsRepo
 
+        from .registry import architecture
+
         self.repo = SafeTensorsRepo(path)
+        self.cfg = cfg or self.repo.model_config()
         self._map: dict[str, str] = {}
+        native = not architecture(self.cfg).hf_names
         for hf in self.repo.names():
-            g = hf_name_to_gguf(hf)
+            g = hf if native else hf_name_to_gguf(hf)
             if g is not None:
                 self._map[g] = hf
-        self.cfg = cfg or self.repo.model_config()
+        if native:
+            for name, shape in tensor_names(self.cfg):
+                if name not in self._map:
+                    raise ModelLoadError(f"tensor {name} not found in {path}")
+                if tuple(self.repo.shape(name)) != tuple(shape):
+                    raise ModelLoadError(f"tensor {name} is {tuple(self.repo.shape(name))}, the configuration says {shape}")
         self._experts: dict[str, list[str]] = {}
         if self.cfg.is_moe:
             for i in range(self.cfg.n_layers):

@@ -423,16 +423,18 @@ def untile_weight(w: torch.Tensor) -> torch.Tensor:
 def paged_decode(q, k_cache, v_cache, block_tables, seq_lens, pages_per_split, part_o, part_ml, out,
                  *, batch: int, max_splits: int, window: int = 0, scale: float,
                  page_ml: Optional[torch.Tensor] = None, block_mass: Optional[torch.Tensor] = None,
-                 q8=None) -> None:
+                 q8=None, keep_first: int = 0, out_d: int = 0, exact_p: bool = False) -> None:
     """Paged split-KV decode attention + merge. With `page_ml` [B, max_blocks, Hq, 2] and `block_mass`
     [B, max_blocks] (fp32) the kernels also produce the softmax probability mass per KV block, summed
     over heads: the heavy-hitter score of H2O pruning (the reference accumulates it in its decode
     kernel too, oxide-backend-cuda/src/kernels/megakernel_ops.cu:577-617). `q8` = (int8 [B, Hq*D],
-    scales, sums): the merge also writes the int8 view of `out` (see `finalize_norm`)."""
+    scales, sums): the merge also writes the int8 view of `out` (see `finalize_norm`). `keep_first`: with a
+    window, the first positions of the sequence stay visible. `out_d`: values stored per head when the
+    heads are padded to D. `exact_p`: softmax weights enter the value product with 16 instead of 8 bits."""
     q8t, q8d, q8s = q8 if q8 is not None else (None, None, None)
     _ext().paged_decode(q, k_cache, v_cache, block_tables, seq_lens, pages_per_split, part_o, part_ml,
                         out, batch, max_splits, window, scale, status_word(q.device) if CHECK_BOUNDS else None,
-                        page_ml, block_mass, q8t, q8d, q8s)
+                        page_ml, block_mass, q8t, q8d, q8s, keep_first, out_d, exact_p)
     _bump(3 if page_ml is not None else 2)
 
 
@@ -442,11 +444,12 @@ CHECK_BOUNDS = os.environ.get("OXB_CHECKS", "0") != "0"
 
 
 def paged_prefill(q, k_cache, v_cache, block_tables, tile_seq, tile_q0, q_start, q_lens, ctx_lens, out,
-                  *, n_tiles: int, window: int = 0, scale: float) -> None:
+                  *, n_tiles: int, window: int = 0, scale: float, keep_first: int = 0, out_d: int = 0,
+                  exact_p: bool = False) -> None:
     """Causal paged attention over ragged prefill chunks on 128-row query tiles (tcgen05 / TMEM,
-    attn_prefill_tc.cu); `tile_q0` entries are multiples of 128."""
+    attn_prefill_tc.cu); `tile_q0` entries are multiples of 128. Options as in `paged_decode`."""
     _ext().paged_prefill_tc(q, k_cache, v_cache, block_tables, tile_seq, tile_q0, q_start, q_lens,
-                            ctx_lens, out, n_tiles, window, scale, status_word(q.device))
+                            ctx_lens, out, n_tiles, window, scale, status_word(q.device), keep_first, out_d, exact_p)
     _bump()
 
 
@@ -550,7 +553,8 @@ def advance_decode_step(s, sampled, mailbox_dev: int, step_counter, *, rows: int
     `rows` rows of the step descriptor `s` for the next decode step from the sampled ids and posts
     the ids to the mapped-host ring at `mailbox_dev`."""
     _ext().advance_decode_step(s.token_ids, s.positions, s.slot_mapping, s.seq_lens, s.block_tables, sampled,
-                               int(mailbox_dev), step_counter, rows, ring, status_word(sampled.device))
+                               int(mailbox_dev), step_counter, rows, ring, status_word(sampled.device),
+                               getattr(s, "prev_ids", None))
     _bump()
 
 

@@ -1,0 +1,108 @@
+"""Python front-ends of the layer-list kernels (``csrc/kernels/{stream_ops,mixer_ops,attn_rows,retention}.cu``).
+
+Activations, weights and caches are bf16, or fp32 throughout; residual streams, states, norms, scores
+and angles are fp32 in both cases. As in `ops`, nothing here falls back to PyTorch.
+"""
+from __future__ import annotations
+
+from typing import Optional
+
+import torch
+
+from .. import ops
+from .._build import hybrid_ext
+
+
+class Rotary:
+    """Device frequencies of a layer_spec.RotarySpec, each as the sum of two fp32 numbers."""
+
+    def __init__(self, spec, device):
+        self.interleaved = bool(spec is not None and spec.interleaved)
+        self.hi = self.lo = None
+        if spec is not None and spec.dims > 0:
+            i = torch.arange(spec.dims // 2, dtype=torch.float64)
+            f = torch.pow(torch.tensor(float(spec.base), dtype=torch.float64), -2.0 * i / spec.dims)
+            hi = f.to(torch.float32)
+            self.hi = hi.to(device)
+            self.lo = (f - hi.to(torch.float64)).to(torch.float32).to(device)
+
+
+def retention_chunk() -> int:
+    return int(hybrid_ext().RETENTION_CHUNK)
+
+
+def max_streams() -> int:
+    return int(hybrid_ext().MAX_STREAMS)
+
+
+def retention_chunks_ok(d: int, e: int) -> bool:
+    return bool(hybrid_ext().retention_chunks_ok(d, e))
+
+
+def set_pdl(on: bool) -> None:
+    hybrid_ext().set_pdl(bool(on))
+
+
+def decay_powers(decay, device) -> torch.Tensor:
+    """[heads, chunk + 1] fp32: decay^0 .. decay^chunk, each rounded once."""
+    d = torch.tensor([float(x) for x in decay], dtype=torch.float64)
+    n = torch.arange(retention_chunk() + 1, dtype=torch.float64)
+    return torch.pow(d[:, None], n[None, :]).to(torch.float32).to(device).contiguous()
+
+
+def stream_norm(x: torch.Tensor, rows: int, *, norm_w: torch.Tensor, eps: float, h: torch.Tensor, w_offset: float = 1.0,
+                tokens=None, prev=None, embed=None, bigram=None, mul_prev: int = 0, mul_cur: int = 0,
+                y: Optional[torch.Tensor] = None, zero_y: bool = True, mix=None, out_w=None, in_w=None,
+                store_x: bool = True, row_map=None, clear=None) -> None:
+    """Embedding or hyper-connection update of the residual streams x [M, S, N], read-out for the next
+    sublayer and its RMS norm (StreamNormParams in csrc/kernels/hybrid.cuh). `clear`: fp32 rows zeroed on
+    the way, the accumulator of the split-K GEMM that follows."""
+    hybrid_ext().stream_norm(x, rows, tokens, prev, embed, bigram, mul_prev, mul_cur, y, zero_y, mix, out_w, in_w, store_x,
+                             norm_w, eps, w_offset, h, row_map, clear, ops.status_word(x.device))
+    ops._bump()
+
+
+def heads(proj: torch.Tensor, m: int, *, h: int, g: int, d: int, e: int, rot: Rotary, positions, q_out, q_hd: int,
+          q_norm=None, k_norm=None, eps: float = 1e-5, k_scale: float = 1.0, k_out=None, k_cache=None, v_cache=None,
+          slots=None) -> None:
+    """Projection rows q | k | v -> normed and rotated heads; k and v into the paged cache, or q and k to
+    dense fp32 buffers (HeadsParams)."""
+    hybrid_ext().heads(proj, m, h, g, d, e, q_norm, k_norm, eps, rot.hi, rot.lo, rot.interleaved, positions, k_scale, q_out,
+                       q_hd, k_out, k_cache, v_cache, slots, ops.status_word(proj.device))
+    ops._bump()
+
+
+def row_attention(q, q_hd: int, k_cache, v_cache, block_tables, *, n: int, h: int, d: int, e: int, window: int,
+                  keep_first: int, scale: float, out, seq_lens=None, tile_seq=None, tile_q0=None, q_start=None, q_lens=None,
+                  ctx_lens=None) -> None:
+    """Softmax attention of any head size in fp32 FMAs: decode rows (seq_lens) or prompt tiles."""
+    hybrid_ext().row_attention(q, q_hd, k_cache, v_cache, block_tables, seq_lens, tile_seq, tile_q0, q_start, q_lens,
+                               ctx_lens, n, h, d, e, window, keep_first, scale, out, ops.status_word(q.device))
+    ops._bump()
+
+
+def retention_decode(proj, rows: int, *, h: int, d: int, e: int, decay_pow, rot: Rotary, k_scale: float, eps: float, state,
+                     row_slots, positions, out) -> None:
+    """One token per row: rotation, state update, read-out, head norm and gate in one launch."""
+    hybrid_ext().retention_decode(proj, rows, h, d, e, decay_pow, rot.hi, rot.lo, rot.interleaved, k_scale, eps, state,
+                                  row_slots, positions, out, ops.status_word(proj.device))
+    ops._bump()
+
+
+def retention_prefill(proj, m: int, *, h: int, d: int, e: int, decay_pow, eps: float, state, seq_slots, tile_seq, tile_q0,
+                      q_start, q_lens, ctx_lens, n_tiles: int, n_seqs: int, q_rot, k_rot, out, ws=None, o_buf=None) -> None:
+    """Prompt chunks: the chunked tensor-core form with a workspace `ws`, else token by token."""
+    hybrid_ext().retention_prefill(proj, m, h, d, e, decay_pow, eps, state, seq_slots, tile_seq, tile_q0, q_start, q_lens,
+                                   ctx_lens, n_tiles, n_seqs, q_rot, k_rot, ws, o_buf, out, ops.status_word(proj.device))
+    ops._bump(3 if ws is not None else 2)
+
+
+def gemm_f32(a, w, out) -> None:
+    """out = a @ w^T in fp32 FMAs."""
+    hybrid_ext().gemm_f32(a, w, out)
+    ops._bump()
+
+
+def glu_f32(gu, out, m: int, i: int, act: int) -> None:
+    hybrid_ext().glu_f32(gu, out, m, i, act)
+    ops._bump()
