@@ -117,7 +117,16 @@ def main() -> None:
                     help="nccl: comparison path with library GEMMs and NCCL all-reduces")
     ap.add_argument("--open-loop", type=int, default=12, help="requests of the open-loop TTFT phase (0 = skip)")
     ap.add_argument("--check-steps", type=int, default=2, help="decode steps compared against the baseline path (0 = skip)")
+    ap.add_argument("--kipolix", action="store_true",
+                    help="instead of the headline workload: layer-list decoders (attention + retention) beside the Llama model of "
+                         "equal size, engine throughput and kernels against their rooflines")
+    ap.add_argument("--kipolix-size", default="", help="only this size of --kipolix")
     args = ap.parse_args()
+    if args.kipolix and args.impl != "reference":
+        from oxide_tech_llm_engine_b200.bench_hybrid import run
+
+        run(args)
+        return
     if args.impl == "reference":
         reference_arm()
         return
