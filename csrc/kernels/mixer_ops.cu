@@ -10,6 +10,25 @@ namespace {
 
 // grid (rows, head ranges): a range of the H + G (+ G value) heads per CTA. The norm spans heads of other
 // CTAs: each CTA re-reads the row's q / k (a few KB from L2) for the sum of squares it needs.
+// This thread's share of the sum of squares of n values
+template <typename P>
+__device__ __forceinline__ float row_ssq(const P* v, int n, long long ld) {
+  float ss = 0.f;
+  if ((n & 3) == 0 && (ld & 3) == 0 && (reinterpret_cast<uintptr_t>(v) & 15) == 0) {
+    for (int c = threadIdx.x * 4; c < n; c += blockDim.x * 4) {
+      float x[4];
+      load4<P>(v + c, x);
+      ss = fmaf(x[0], x[0], fmaf(x[1], x[1], fmaf(x[2], x[2], fmaf(x[3], x[3], ss))));
+    }
+  } else {
+    for (int c = threadIdx.x; c < n; c += blockDim.x) {
+      const float x = to_f(v[c]);
+      ss = fmaf(x, x, ss);
+    }
+  }
+  return ss;
+}
+
 // T: storage type (cache, dense q of the attention), TQ: type of q_out, P: type of the projection rows.
 template <typename T, typename TQ, typename P>
 __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
@@ -33,22 +52,9 @@ __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
     for (int i = threadIdx.x; i < rot2; i += blockDim.x) rotary_sincos(p.rot, i, pos, &s_sin[i], &s_cos[i]);
   float rq = 1.f, rk = 1.f;
   if (p.q_norm != nullptr) {
-    if (h_lo < H) {
-      float ss = 0.f;
-      for (int c = threadIdx.x; c < H * D; c += blockDim.x) {
-        const float v = to_f(pr[c]);
-        ss = fmaf(v, v, ss);
-      }
-      rq = 1.f / sqrtf(block_sum_all(ss, s_red) / static_cast<float>(H * D) + p.eps);
-    }
-    if (h_lo < H + G && h_hi > H) {
-      float ss = 0.f;
-      for (int c = threadIdx.x; c < G * D; c += blockDim.x) {
-        const float v = to_f(pr[H * D + c]);
-        ss = fmaf(v, v, ss);
-      }
-      rk = 1.f / sqrtf(block_sum_all(ss, s_red) / static_cast<float>(G * D) + p.eps);
-    }
+    if (h_lo < H) rq = 1.f / sqrtf(block_sum_all(row_ssq(pr, H * D, p.ld), s_red) / static_cast<float>(H * D) + p.eps);
+    if (h_lo < H + G && h_hi > H)
+      rk = 1.f / sqrtf(block_sum_all(row_ssq(pr + H * D, G * D, p.ld), s_red) / static_cast<float>(G * D) + p.eps);
   }
   __syncthreads();
   const long long slot = p.slots != nullptr ? p.slots[row] : -1;
@@ -57,52 +63,47 @@ __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
   const long long blk = slot >> 4;
   const int off = static_cast<int>(slot & 15);
 
-  // q and k heads: one item per rotation pair, one per dimension that passes
+  // q and k heads, one warp per head: a lane takes rotation pairs, then dimensions that pass
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int r_hi = min(h_hi, H + G);
-  const int items = D - rot2;
-  for (int i = threadIdx.x; i < (r_hi - h_lo) * items; i += blockDim.x) {
-    const int h = h_lo + i / items, it = i % items;
+  for (int h = h_lo + warp; h < r_hi; h += nw) {
     const bool is_q = h < H;
-    const int base = h * D;  // k follows q in the projection row
+    if (!is_q && p.k_out == nullptr && !store_kv) continue;
+    const P* src = pr + h * D;  // k follows q in the projection row
     const float r = is_q ? rq : rk;
     const float* w = is_q ? p.q_norm : p.k_norm;
-    const int wo = is_q ? base : base - H * D;
-    int d0, d1 = -1;
-    float y0, y1 = 0.f;
-    if (it < rot2) {
+    if (w != nullptr) w += (is_q ? h : h - H) * D;
+    const float ks = is_q ? 1.f : p.k_scale;
+    TQ* qd = nullptr;
+    float* kd = nullptr;
+    T* kc = nullptr;
+    if (is_q) qd = static_cast<TQ*>(p.q_out) + static_cast<long long>(row) * p.q_ld + h * p.q_hd;
+    else if (p.k_out != nullptr) kd = p.k_out + static_cast<long long>(row) * p.k_ld + (h - H) * p.k_hd;
+    else kc = static_cast<T*>(p.k_cache) + ((blk * G + (h - H)) * 16 + off) * p.DP;
+    auto put = [&](int d, float y) {
+      if (qd != nullptr) qd[d] = from_f<TQ>(y);
+      else if (kd != nullptr) kd[d] = y * ks;
+      else kc[d] = from_f<T>(y * ks);
+    };
+    for (int it = lane; it < rot2; it += 32) {
+      int d0, d1;
       rotary_pair(p.rot, it, &d0, &d1);
-      float u = to_f(pr[base + d0]) * r, v = to_f(pr[base + d1]) * r;
+      float u = to_f(src[d0]) * r, v = to_f(src[d1]) * r;
       if (w != nullptr) {
-        u *= w[wo + d0];
-        v *= w[wo + d1];
+        u *= w[d0];
+        v *= w[d1];
       }
-      y0 = u * s_cos[it] - v * s_sin[it];
-      y1 = v * s_cos[it] + u * s_sin[it];
-    } else {
-      d0 = rot2 + it;
-      y0 = to_f(pr[base + d0]) * r;
-      if (w != nullptr) y0 *= w[wo + d0];
+      put(d0, u * s_cos[it] - v * s_sin[it]);
+      put(d1, v * s_cos[it] + u * s_sin[it]);
     }
-    if (is_q) {
-      TQ* q = static_cast<TQ*>(p.q_out) + static_cast<long long>(row) * p.q_ld + h * p.q_hd;
-      q[d0] = from_f<TQ>(y0);
-      if (d1 >= 0) q[d1] = from_f<TQ>(y1);
-    } else if (p.k_out != nullptr) {
-      float* k = p.k_out + static_cast<long long>(row) * p.k_ld + (h - H) * p.k_hd;
-      k[d0] = y0 * p.k_scale;
-      if (d1 >= 0) k[d1] = y1 * p.k_scale;
-    } else if (store_kv) {
-      T* k = static_cast<T*>(p.k_cache) + ((blk * G + (h - H)) * 16 + off) * p.DP;
-      k[d0] = from_f<T>(y0 * p.k_scale);
-      if (d1 >= 0) k[d1] = from_f<T>(y1 * p.k_scale);
-    }
+    for (int d = 2 * rot2 + lane; d < D; d += 32) put(d, to_f(src[d]) * r * (w != nullptr ? w[d] : 1.f));
   }
   if (store_kv && h_hi > H + G) {
-    const int v_lo = max(h_lo, H + G);
     const P* vr = pr + (H + G) * D;
-    for (int i = threadIdx.x; i < (h_hi - v_lo) * E; i += blockDim.x) {
-      const int g = v_lo - H - G + i / E, e = i % E;
-      static_cast<T*>(p.v_cache)[((blk * G + g) * 16 + off) * p.EP + e] = from_f<T>(to_f(vr[g * E + e]));
+    for (int h = max(h_lo, H + G) + warp; h < h_hi; h += nw) {
+      const int g = h - H - G;
+      T* vc = static_cast<T*>(p.v_cache) + ((blk * G + g) * 16 + off) * p.EP;
+      for (int e = lane; e < E; e += 32) vc[e] = from_f<T>(to_f(vr[g * E + e]));
     }
   }
 }

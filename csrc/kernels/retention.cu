@@ -156,15 +156,13 @@ constexpr int kLdP = C + 4;
 struct Tf {
   uint32_t hi, lo;
 };
-__device__ __forceinline__ uint32_t to_tf32(float x) {
-  uint32_t y;
-  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(y) : "f"(x));
-  return y;
-}
+// x = hi + lo with both parts representable in TF32 (10 stored bits; the rest is cut off, so lo keeps the
+// bits that hi lost and the pair carries about 21)
+constexpr uint32_t kTf32Mask = 0xffffe000u;
 __device__ __forceinline__ Tf split_tf32(float x) {
   Tf t;
-  t.hi = to_tf32(x);
-  t.lo = to_tf32(x - __uint_as_float(t.hi));
+  t.hi = __float_as_uint(x) & kTf32Mask;
+  t.lo = __float_as_uint(x - __uint_as_float(t.hi)) & kTf32Mask;
   return t;
 }
 __device__ __forceinline__ void mma_tf32(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
@@ -251,64 +249,82 @@ __device__ __forceinline__ ChunkPos chunk_pos(const RetentionParams& p, int chun
   return {p.q_start[seq] + q0, left < C ? left : C};
 }
 
-// 1. grid (chunks, H, D / 64): U_c[d, e] of 64 head dimensions x all value dimensions.
+// 1. grid (chunks, H): U_c[d, e], 64 head dimensions at a time, the next keys on their way meanwhile.
+template <int ET>
+struct SumSmem {
+  static constexpr int kLdK = 64 + 8, kLdV = ET + 8;
+  static constexpr int kFloats = 2 * C * kLdK + C * kLdV;
+};
 template <int ET, typename P>
 __global__ void __launch_bounds__(kChThreads) retention_chunk_sum_kernel(const RetentionParams p) {
-  constexpr int kLdK = 64 + 8, kLdV = ET + 8;
+  using L = SumSmem<ET>;
   extern __shared__ __align__(16) float s_mem[];
-  float* sK = s_mem;              // [C][64] keys times their decay
-  float* sV = sK + C * kLdK;      // [C][ET]
+  __shared__ float s_w[C];                    // decay of every row of the chunk up to its end
+  float* sV = s_mem + 2 * C * L::kLdK;        // [C][ET]
   pdl_launch_dependents();
   pdl_wait();
-  const int chunk = blockIdx.x, head = blockIdx.y, d0 = blockIdx.z * 64;
+  const int chunk = blockIdx.x, head = blockIdx.y;
   const ChunkPos cp = chunk_pos(p, chunk);
   if (cp.n <= 0) return;
   const int D = p.D, E = p.E;
   const long long ldk = static_cast<long long>(p.H) * D;
-  const float* pw = p.decay_pow + head * (C + 1);
+  const float* ksrc = p.k_rot + cp.row0 * ldk + head * D;
+  const int n_it = (D + 63) / 64;
+  auto load_k = [&](int it) {
+    tile_f32<C, 64>(s_mem + (it & 1) * C * L::kLdK, L::kLdK, ksrc + it * 64, ldk, cp.n, D - it * 64, D % 4 == 0);
+    cp_commit();
+  };
+  load_k(0);
   const P* vsrc = static_cast<const P*>(p.proj) + cp.row0 * p.ld + 2 * p.H * D + head * E;
   const bool vec_v = (E % 4 == 0) && (p.ld % 4 == 0) && ((2 * p.H * D) % 4 == 0);
-  tile_values<ET, P>(sV, kLdV, vsrc, p.ld, cp.n, E, vec_v);
-  const float* ksrc = p.k_rot + cp.row0 * ldk + head * D + d0;
-  for (int i = threadIdx.x; i < C * 64; i += kChThreads) {
-    const int r = i >> 6, c = i & 63;
-    sK[r * kLdK + c] = (r < cp.n && d0 + c < D) ? ksrc[r * ldk + c] * pw[cp.n - 1 - r] : 0.f;
-  }
-  __syncthreads();
+  tile_values<ET, P>(sV, L::kLdV, vsrc, p.ld, cp.n, E, vec_v);
+  for (int r = threadIdx.x; r < C; r += kChThreads) s_w[r] = r < cp.n ? p.decay_pow[head * (C + 1) + cp.n - 1 - r] : 0.f;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   const int m0 = (warp & 3) * 16;
   constexpr int NT = ET / 16;     // 8-column tiles of this warp's half
   const int n0 = (warp >> 2) * (ET / 2);
-  float acc[NT][4] = {};
-#pragma unroll 2
-  for (int kk = 0; kk < C; kk += 8) {
-    FragA a;
-    a.v[0] = split_tf32(sK[(kk + t) * kLdK + m0 + g]);
-    a.v[1] = split_tf32(sK[(kk + t) * kLdK + m0 + g + 8]);
-    a.v[2] = split_tf32(sK[(kk + t + 4) * kLdK + m0 + g]);
-    a.v[3] = split_tf32(sK[(kk + t + 4) * kLdK + m0 + g + 8]);
-#pragma unroll
-    for (int n = 0; n < NT; ++n) {
-      const uint32_t b0 = __float_as_uint(sV[(kk + t) * kLdV + n0 + n * 8 + g]);
-      const uint32_t b1 = __float_as_uint(sV[(kk + t + 4) * kLdV + n0 + n * 8 + g]);
-      mma_2x(acc[n], a, b0, b1);
-    }
-  }
   float* w = p.ws + (static_cast<long long>(chunk) * p.H + head) * D * E;
+  for (int it = 0; it < n_it; ++it) {
+    if (it + 1 < n_it) {
+      load_k(it + 1);
+      cp_wait<1>();
+    } else {
+      cp_wait<0>();
+    }
+    __syncthreads();
+    const float* sK = s_mem + (it & 1) * C * L::kLdK;
+    float acc[NT][4] = {};
+#pragma unroll 2
+    for (int kk = 0; kk < C; kk += 8) {
+      const float w0 = s_w[kk + t], w1 = s_w[kk + t + 4];
+      FragA a;
+      a.v[0] = split_tf32(sK[(kk + t) * L::kLdK + m0 + g] * w0);
+      a.v[1] = split_tf32(sK[(kk + t) * L::kLdK + m0 + g + 8] * w0);
+      a.v[2] = split_tf32(sK[(kk + t + 4) * L::kLdK + m0 + g] * w1);
+      a.v[3] = split_tf32(sK[(kk + t + 4) * L::kLdK + m0 + g + 8] * w1);
 #pragma unroll
-  for (int n = 0; n < NT; ++n)
-#pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      const int d = d0 + m0 + g + 8 * h, e = n0 + n * 8 + 2 * t;
-      if (d < D) {
-        if (e + 1 < E && (E & 1) == 0) {
-          *reinterpret_cast<float2*>(w + static_cast<long long>(d) * E + e) = make_float2(acc[n][2 * h], acc[n][2 * h + 1]);
-        } else {
-          if (e < E) w[static_cast<long long>(d) * E + e] = acc[n][2 * h];
-          if (e + 1 < E) w[static_cast<long long>(d) * E + e + 1] = acc[n][2 * h + 1];
-        }
+      for (int n = 0; n < NT; ++n) {
+        const uint32_t b0 = __float_as_uint(sV[(kk + t) * L::kLdV + n0 + n * 8 + g]);
+        const uint32_t b1 = __float_as_uint(sV[(kk + t + 4) * L::kLdV + n0 + n * 8 + g]);
+        mma_2x(acc[n], a, b0, b1);
       }
     }
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int d = it * 64 + m0 + g + 8 * h, e = n0 + n * 8 + 2 * t;
+        if (d < D) {
+          if (e + 1 < E && (E & 1) == 0) {
+            *reinterpret_cast<float2*>(w + static_cast<long long>(d) * E + e) = make_float2(acc[n][2 * h], acc[n][2 * h + 1]);
+          } else {
+            if (e < E) w[static_cast<long long>(d) * E + e] = acc[n][2 * h];
+            if (e + 1 < E) w[static_cast<long long>(d) * E + e + 1] = acc[n][2 * h + 1];
+          }
+        }
+      }
+    __syncthreads();  // the stage may be refilled
+  }
 }
 
 // 2. grid (D E / (256 V), H, sequences): walks the chunks of a sequence, eight loads ahead.
@@ -615,11 +631,11 @@ cudaError_t launch_decode(const RetentionParams& p, int slices, cudaStream_t str
 template <int ET, typename P>
 cudaError_t launch_chunks(const RetentionParams& p, cudaStream_t stream) {
   const int chunks = 2 * p.n_tiles;
-  const size_t smem1 = (C * (64 + 8) + C * (ET + 8)) * sizeof(float);
+  const size_t smem1 = SumSmem<ET>::kFloats * sizeof(float);
   const size_t smem3 = OutSmem<ET>::kFloats * sizeof(float);
   ensure_dynamic_smem(retention_chunk_sum_kernel<ET, P>, smem1);
   ensure_dynamic_smem(retention_chunk_out_kernel<ET, P>, smem3);
-  cudaError_t e = launch_kernel(retention_chunk_sum_kernel<ET, P>, dim3(chunks, p.H, (p.D + 63) / 64), dim3(kChThreads), smem1,
+  cudaError_t e = launch_kernel(retention_chunk_sum_kernel<ET, P>, dim3(chunks, p.H), dim3(kChThreads), smem1,
                                 stream, true, false, p);
   if (e != cudaSuccess) return e;
   const long long de = static_cast<long long>(p.D) * p.E;

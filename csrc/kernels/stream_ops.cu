@@ -10,9 +10,10 @@ namespace oxb {
 namespace {
 
 // One CTA per row (looping). V = 4: rows of whole 16-byte pieces, V = 1: any width. S: largest stream count
-// of this instantiation.
-template <typename T, int S, int V>
-__global__ void __launch_bounds__(1024) stream_norm_kernel(const StreamNormParams p) {
+// of this instantiation. CH: pieces per thread whose loads are issued together (the kernel is a stream of
+// fp32 rows; the bytes in flight set its rate).
+template <typename T, int S, int V, int CH>
+__global__ void __launch_bounds__(CH == 1 ? 1024 : (CH == 2 ? 512 : 256)) stream_norm_kernel(const StreamNormParams p) {
   extern __shared__ float s_u[];  // N read-out values
   __shared__ float s_red[32];
   __shared__ float s_mix[S * S], s_out[S], s_in[S];
@@ -27,6 +28,7 @@ __global__ void __launch_bounds__(1024) stream_norm_kernel(const StreamNormParam
   pdl_wait();  // streams, the sublayer's output and the step's tokens come from earlier kernels
   for (int row = blockIdx.x; row < p.rows; row += gridDim.x) {
     float* xr = p.x + static_cast<long long>(row) * n_s * N;
+    float* yr = p.y != nullptr ? p.y + static_cast<long long>(row) * p.ldy : nullptr;
     const T* er = nullptr;
     const T* br = nullptr;
     if (p.tokens != nullptr) {
@@ -46,59 +48,63 @@ __global__ void __launch_bounds__(1024) stream_norm_kernel(const StreamNormParam
     }
     const int dst = p.row_map != nullptr ? p.row_map[row] : row;
     float ssq = 0.f;
-    for (int c = threadIdx.x * V; c < N; c += blockDim.x * V) {
-      float x[S][V];
-      if (er != nullptr) {
-        float e[V];
-        if constexpr (V == 4) {
-          load4<T>(er + c, e);
-          if (br != nullptr) {
-            float b[4];
-            load4<T>(br + c, b);
+    for (int base = 0; base < N; base += blockDim.x * V * CH) {
+      float x[CH][S][V], y[CH][V];
 #pragma unroll
-            for (int j = 0; j < 4; ++j) e[j] += b[j];
+      for (int k = 0; k < CH; ++k) {
+        const int c = base + (k * blockDim.x + threadIdx.x) * V;
+        if (c >= N) continue;
+        if (er != nullptr) {
+          float e[V];
+          if constexpr (V == 4) {
+            load4<T>(er + c, e);
+            if (br != nullptr) {
+              float b[4];
+              load4<T>(br + c, b);
+#pragma unroll
+              for (int j = 0; j < 4; ++j) e[j] += b[j];
+            }
+          } else {
+            e[0] = to_f(er[c]) + (br != nullptr ? to_f(br[c]) : 0.f);
           }
+#pragma unroll
+          for (int s = 0; s < S; ++s)
+#pragma unroll
+            for (int j = 0; j < V; ++j) x[k][s][j] = e[j];
         } else {
-          e[0] = to_f(er[c]) + (br != nullptr ? to_f(br[c]) : 0.f);
-        }
 #pragma unroll
-        for (int s = 0; s < S; ++s)
-#pragma unroll
-          for (int j = 0; j < V; ++j) x[s][j] = e[j];
-      } else {
-#pragma unroll
-        for (int s = 0; s < S; ++s) {
-          if (s < n_s) {
-            if constexpr (V == 4) load4<float>(xr + static_cast<long long>(s) * N + c, x[s]);
-            else x[s][0] = xr[static_cast<long long>(s) * N + c];
-          }
+          for (int s = 0; s < S; ++s)
+            if (s < n_s) {
+              if constexpr (V == 4) load4<float>(xr + static_cast<long long>(s) * N + c, x[k][s]);
+              else x[k][s][0] = xr[static_cast<long long>(s) * N + c];
+            }
+          if constexpr (V == 4) load4<float>(yr + c, y[k]);
+          else y[k][0] = yr[c];
         }
       }
-      float u[V];
 #pragma unroll
-      for (int j = 0; j < V; ++j) u[j] = 0.f;
-      if (p.y != nullptr) {
-        float y[V];
-        float* yp = p.y + static_cast<long long>(row) * p.ldy + c;
-        if constexpr (V == 4) {
-          load4<float>(yp, y);
-          if (p.zero_y) *reinterpret_cast<float4*>(yp) = make_float4(0.f, 0.f, 0.f, 0.f);
-        } else {
-          y[0] = *yp;
-          if (p.zero_y) *yp = 0.f;
-        }
+      for (int k = 0; k < CH; ++k) {
+        const int c = base + (k * blockDim.x + threadIdx.x) * V;
+        if (c >= N) continue;
+        float u[V];
+#pragma unroll
+        for (int j = 0; j < V; ++j) u[j] = 0.f;
 #pragma unroll
         for (int t = 0; t < S; ++t) {
           if (t < n_s) {
             float z[V];
+            if (yr != nullptr) {
 #pragma unroll
-            for (int j = 0; j < V; ++j) z[j] = s_out[t] * y[j];
+              for (int j = 0; j < V; ++j) z[j] = s_out[t] * y[k][j];
 #pragma unroll
-            for (int s = 0; s < S; ++s) {
-              if (s < n_s) {
+              for (int s = 0; s < S; ++s)
+                if (s < n_s) {
 #pragma unroll
-                for (int j = 0; j < V; ++j) z[j] = fmaf(s_mix[s * S + t], x[s][j], z[j]);
-              }
+                  for (int j = 0; j < V; ++j) z[j] = fmaf(s_mix[s * S + t], x[k][s][j], z[j]);
+                }
+            } else {
+#pragma unroll
+              for (int j = 0; j < V; ++j) z[j] = x[k][t][j];
             }
 #pragma unroll
             for (int j = 0; j < V; ++j) u[j] = fmaf(s_in[t], z[j], u[j]);
@@ -108,23 +114,14 @@ __global__ void __launch_bounds__(1024) stream_norm_kernel(const StreamNormParam
             }
           }
         }
-      } else {
-#pragma unroll
-        for (int t = 0; t < S; ++t) {
-          if (t < n_s) {
-#pragma unroll
-            for (int j = 0; j < V; ++j) u[j] = fmaf(s_in[t], x[t][j], u[j]);
-            if (p.store_x) {
-              if constexpr (V == 4) store4<float>(xr + static_cast<long long>(t) * N + c, x[t]);
-              else xr[static_cast<long long>(t) * N + c] = x[t][0];
-            }
-          }
+        if (yr != nullptr && p.zero_y) {
+          if constexpr (V == 4) *reinterpret_cast<float4*>(yr + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+          else yr[c] = 0.f;
         }
-      }
+        if constexpr (V == 4) *reinterpret_cast<float4*>(s_u + c) = make_float4(u[0], u[1], u[2], u[3]);
+        else s_u[c] = u[0];
 #pragma unroll
-      for (int j = 0; j < V; ++j) {
-        s_u[c + j] = u[j];
-        ssq = fmaf(u[j], u[j], ssq);
+        for (int j = 0; j < V; ++j) ssq = fmaf(u[j], u[j], ssq);
       }
     }
     if (dst < 0) continue;  // a row without a logits row; the same for every thread of the CTA
@@ -135,8 +132,11 @@ __global__ void __launch_bounds__(1024) stream_norm_kernel(const StreamNormParam
       if constexpr (V == 4) {
         float w[4], o[4];
         load4<float>(p.norm_w + c, w);
-#pragma unroll
-        for (int j = 0; j < 4; ++j) o[j] = s_u[c + j] * r * (w[j] + p.w_offset);
+        const float4 u = *reinterpret_cast<const float4*>(s_u + c);
+        o[0] = u.x * r * (w[0] + p.w_offset);
+        o[1] = u.y * r * (w[1] + p.w_offset);
+        o[2] = u.z * r * (w[2] + p.w_offset);
+        o[3] = u.w * r * (w[3] + p.w_offset);
         store4<T>(hr + c, o);
       } else {
         hr[c] = from_f<T>(s_u[c] * r * (p.norm_w[c] + p.w_offset));
@@ -145,22 +145,30 @@ __global__ void __launch_bounds__(1024) stream_norm_kernel(const StreamNormParam
   }
 }
 
+template <typename T, int S, int V, int CH>
+cudaError_t launch_ch(const StreamNormParams& p, int threads, cudaStream_t stream) {
+  auto kern = stream_norm_kernel<T, S, V, CH>;
+  const size_t smem = static_cast<size_t>(p.N) * sizeof(float);
+  ensure_dynamic_smem(kern, smem);
+  const int cap = 8 * sm_count();
+  return launch_kernel(kern, dim3(p.rows < cap ? p.rows : cap), dim3(threads), smem, stream, /*pdl=*/true, false, p);
+}
+
 template <typename T, int S>
 cudaError_t launch_s(const StreamNormParams& p, cudaStream_t stream) {
   constexpr int VW = S <= 8 ? 4 : 1;  // 16 streams x 4 values would spill
   const bool vec = VW == 4 && p.N % 4 == 0 && p.ldy % 4 == 0 && p.ldh % 4 == 0;
   const int v = vec ? 4 : 1;
   int threads = (p.N / v + 31) / 32 * 32;
-  threads = threads < 32 ? 32 : (threads > 1024 ? 1024 : threads);
-  // many rows: smaller CTAs, so that several rows per SM are in flight
-  if (p.rows > 2 * sm_count() && threads > 256) threads = 256;
-  const int per_sm = 2048 / threads;
-  const int cap = sm_count() * per_sm;
-  const int grid = p.rows < cap ? p.rows : cap;
-  const size_t smem = static_cast<size_t>(p.N) * sizeof(float);
-  auto kern = vec ? stream_norm_kernel<T, S, VW> : stream_norm_kernel<T, S, 1>;
-  ensure_dynamic_smem(kern, smem);
-  return launch_kernel(kern, dim3(grid), dim3(threads), smem, stream, /*pdl=*/true, false, p);
+  if (threads < 32) threads = 32;
+  constexpr int CHM = S <= 2 ? 4 : (S <= 4 ? 2 : 1);  // pieces in flight that the registers hold
+  if (vec && CHM > 1 && p.rows > 2 * sm_count() && threads > 256) {
+    // many rows: several CTAs per SM, each with a whole row (or most of it) in flight
+    if (CHM == 4 && threads > 512) return launch_ch<T, S, VW, CHM>(p, 256, stream);
+    return launch_ch<T, S, VW, 2>(p, 256, stream);
+  }
+  if (threads > 1024) threads = 1024;
+  return vec ? launch_ch<T, S, VW, 1>(p, threads, stream) : launch_ch<T, S, 1, 1>(p, threads, stream);
 }
 
 template <typename T>

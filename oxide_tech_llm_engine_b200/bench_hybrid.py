@@ -66,9 +66,10 @@ def engine_numbers(mc, *, batch: int, prompt: int, warmup: int, steps: int) -> d
     from .sampling_params import SamplingParams
 
     chunk = 8192
-    eng = _engine(mc, batch, prompt, warmup + steps + 8, chunk)
+    budget = warmup + steps + 16 + batch * prompt // chunk      # early requests decode while others prefill
+    eng = _engine(mc, batch, prompt, budget, chunk)
     rng = np.random.default_rng(0)
-    sp = SamplingParams(greedy=True, max_tokens=warmup + steps + 8, ignore_eos=True)
+    sp = SamplingParams(greedy=True, max_tokens=budget, ignore_eos=True)
 
     def submit():
         for _ in range(batch):
@@ -84,8 +85,11 @@ def engine_numbers(mc, *, batch: int, prompt: int, warmup: int, steps: int) -> d
     full = batch * prompt // chunk          # steps made of whole chunks of prompt tokens
     n_pre = max(1, min(full, 8))
     t_pre = _time_steps(eng, n_pre)
-    while eng.stats["decode_tokens"] == 0:
+    while True:                             # until every request decodes
+        before = eng.stats["prefill_tokens"]
         eng.step()
+        if eng.stats["prefill_tokens"] == before:
+            break
     for _ in range(warmup):
         eng.step()
     t_dec = _time_steps(eng, steps)
