@@ -30,7 +30,8 @@ __device__ __forceinline__ float row_ssq(const P* v, int n, long long ld) {
 }
 
 // T: storage type (cache, dense q of the attention), TQ: type of q_out, P: type of the projection rows.
-template <typename T, typename TQ, typename P>
+// VEC: every size and pitch is a multiple of 4, values move four at a time.
+template <typename T, typename TQ, typename P, bool VEC>
 __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
   extern __shared__ float s_mem[];
   __shared__ float s_red[32];
@@ -52,9 +53,11 @@ __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
     for (int i = threadIdx.x; i < rot2; i += blockDim.x) rotary_sincos(p.rot, i, pos, &s_sin[i], &s_cos[i]);
   float rq = 1.f, rk = 1.f;
   if (p.q_norm != nullptr) {
-    if (h_lo < H) rq = 1.f / sqrtf(block_sum_all(row_ssq(pr, H * D, p.ld), s_red) / static_cast<float>(H * D) + p.eps);
-    if (h_lo < H + G && h_hi > H)
-      rk = 1.f / sqrtf(block_sum_all(row_ssq(pr + H * D, G * D, p.ld), s_red) / static_cast<float>(G * D) + p.eps);
+    const bool need_k = h_lo < H + G && h_hi > H;
+    const float sq = h_lo < H ? row_ssq(pr, H * D, p.ld) : 0.f;
+    const float sk = need_k ? row_ssq(pr + H * D, G * D, p.ld) : 0.f;
+    if (h_lo < H) rq = 1.f / sqrtf(block_sum_all(sq, s_red) / static_cast<float>(H * D) + p.eps);
+    if (need_k) rk = 1.f / sqrtf(block_sum_all(sk, s_red) / static_cast<float>(G * D) + p.eps);
   }
   __syncthreads();
   const long long slot = p.slots != nullptr ? p.slots[row] : -1;
@@ -63,7 +66,77 @@ __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
   const long long blk = slot >> 4;
   const int off = static_cast<int>(slot & 15);
 
-  // q and k heads, one warp per head: a lane takes rotation pairs, then dimensions that pass
+  if constexpr (VEC) {
+    // four values (two pairs of the interleaved layout) or two times four (the other) per item, items of all
+    // heads of this CTA dealt out over its threads
+    const int r_end = min(h_hi, H + G);
+    const int rq4 = p.rot.interleaved ? (2 * rot2) >> 2 : rot2 >> 2;   // rotated items of a head
+    const int per = rq4 + ((D - 2 * rot2) >> 2);
+    for (int i = threadIdx.x; i < (r_end - h_lo) * per; i += blockDim.x) {
+      const int lh = i / per, it = i - lh * per, h = h_lo + lh;
+      const bool is_q = h < H;
+      if (!is_q && p.k_out == nullptr && !store_kv) continue;
+      const P* src = pr + h * D;
+      const float r = is_q ? rq : rk, ks = is_q ? 1.f : p.k_scale;
+      const float* w = is_q ? p.q_norm : p.k_norm;
+      if (w != nullptr) w += (is_q ? h : h - H) * D;
+      auto get = [&](int d, float (&v)[4]) {
+        load4<P>(src + d, v);
+        if (w != nullptr) {
+          float g4[4];
+          load4<float>(w + d, g4);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) v[j] *= r * g4[j];
+        }
+      };
+      auto put = [&](int d, float (&v)[4]) {
+        if (is_q) {
+          store4<TQ>(static_cast<TQ*>(p.q_out) + static_cast<long long>(row) * p.q_ld + h * p.q_hd + d, v);
+          return;
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[j] *= ks;
+        if (p.k_out != nullptr) store4<float>(p.k_out + static_cast<long long>(row) * p.k_ld + (h - H) * p.k_hd + d, v);
+        else store4<T>(static_cast<T*>(p.k_cache) + ((blk * G + (h - H)) * 16 + off) * p.DP + d, v);
+      };
+      float x[4];
+      if (it >= rq4) {
+        const int d = 2 * rot2 + (it - rq4) * 4;
+        get(d, x);
+        put(d, x);
+      } else if (p.rot.interleaved) {
+        const int f = it * 2;
+        get(it * 4, x);
+        float y[4] = {x[0] * s_cos[f] - x[1] * s_sin[f], x[1] * s_cos[f] + x[0] * s_sin[f],
+                      x[2] * s_cos[f + 1] - x[3] * s_sin[f + 1], x[3] * s_cos[f + 1] + x[2] * s_sin[f + 1]};
+        put(it * 4, y);
+      } else {
+        const int f = it * 4;
+        float z[4], y0[4], y1[4];
+        get(f, x);
+        get(f + rot2, z);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          y0[j] = x[j] * s_cos[f + j] - z[j] * s_sin[f + j];
+          y1[j] = z[j] * s_cos[f + j] + x[j] * s_sin[f + j];
+        }
+        put(f, y0);
+        put(f + rot2, y1);
+      }
+    }
+    if (store_kv && h_hi > H + G) {
+      const int v_lo = max(h_lo, H + G), e4 = E >> 2;
+      const P* vr = pr + (H + G) * D;
+      for (int i = threadIdx.x; i < (h_hi - v_lo) * e4; i += blockDim.x) {
+        const int lh = i / e4, e = (i - lh * e4) * 4, g = v_lo + lh - H - G;
+        float x[4];
+        load4<P>(vr + g * E + e, x);
+        store4<T>(static_cast<T*>(p.v_cache) + ((blk * G + g) * 16 + off) * p.EP + e, x);
+      }
+    }
+    return;
+  }
+  // any sizes: one warp per head, a lane takes rotation pairs, then dimensions that pass
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int r_hi = min(h_hi, H + G);
   for (int h = h_lo + warp; h < r_hi; h += nw) {
@@ -186,6 +259,15 @@ __global__ void __launch_bounds__(256) glu_f32_kernel(const float* gu, long long
 
 }  // namespace
 
+template <bool VEC>
+static cudaError_t launch_heads_v(const HeadsParams& p, int dtype, dim3 grid, dim3 block, size_t smem, cudaStream_t stream) {
+  using bf16 = __nv_bfloat16;
+  auto kern = dtype == 1          ? heads_kernel<float, float, float, VEC>
+              : p.k_out != nullptr ? (p.proj_f32 ? heads_kernel<bf16, float, float, VEC> : heads_kernel<bf16, float, bf16, VEC>)
+                                   : (p.proj_f32 ? heads_kernel<bf16, bf16, float, VEC> : heads_kernel<bf16, bf16, bf16, VEC>);
+  return launch_kernel(kern, grid, block, smem, stream, true, false, p);
+}
+
 cudaError_t launch_heads(const HeadsParams& p, int dtype, cudaStream_t stream) {
   if (p.M <= 0) return cudaSuccess;
   const int n_heads = p.H + p.G + (p.v_cache != nullptr ? p.G : 0);
@@ -195,11 +277,11 @@ cudaError_t launch_heads(const HeadsParams& p, int dtype, cudaStream_t stream) {
   if (chunks < 1) chunks = 1;
   const size_t smem = static_cast<size_t>(p.rot.dims) * sizeof(float);
   const dim3 grid(p.M, chunks), block(256);
-  using bf16 = __nv_bfloat16;
-  auto kern = dtype == 1          ? heads_kernel<float, float, float>
-              : p.k_out != nullptr ? (p.proj_f32 ? heads_kernel<bf16, float, float> : heads_kernel<bf16, float, bf16>)
-                                   : (p.proj_f32 ? heads_kernel<bf16, bf16, float> : heads_kernel<bf16, bf16, bf16>);
-  return launch_kernel(kern, grid, block, smem, stream, true, false, p);
+  auto al = [](const void* x) { return reinterpret_cast<uintptr_t>(x) % 16 == 0; };
+  const bool vec = p.D % 4 == 0 && p.E % 4 == 0 && p.rot.dims % (p.rot.interleaved ? 4 : 8) == 0 && p.ld % 4 == 0 && p.q_ld % 4 == 0 &&
+                   p.q_hd % 4 == 0 && p.k_ld % 4 == 0 && p.k_hd % 4 == 0 && p.DP % 4 == 0 && p.EP % 4 == 0 && al(p.proj) &&
+                   al(p.q_out) && al(p.k_out) && al(p.q_norm) && al(p.k_norm);
+  return vec ? launch_heads_v<true>(p, dtype, grid, block, smem, stream) : launch_heads_v<false>(p, dtype, grid, block, smem, stream);
 }
 
 cudaError_t launch_gemm_f32(const float* a, long long lda, const float* w, long long ldw, float* out, long long ldo,

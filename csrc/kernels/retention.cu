@@ -388,17 +388,18 @@ struct OutSmem {
   static constexpr int kS = KT * kLdS;                       // one stage of the state
   static constexpr int kStage = 2 * kQK + kS;
   static constexpr int kV = C * kLdS;
-  static constexpr int kFloats = 2 * kStage + kV;
+  static constexpr bool kShareV = kV <= kStage;             // the values reuse the second stage after the loop
+  static constexpr int kFloats = 2 * kStage + (kShareV ? 0 : kV);
   static_assert(C * kLdP <= kStage, "the weights reuse the first stage");
 };
 
 template <int ET, typename P>
-__global__ void __launch_bounds__(kChThreads) retention_chunk_out_kernel(const RetentionParams p) {
+__global__ void __launch_bounds__(kChThreads, ET <= 128 ? 3 : 1) retention_chunk_out_kernel(const RetentionParams p) {
   using L = OutSmem<ET>;
   extern __shared__ __align__(16) float s_mem[];
   __shared__ float s_pw[C + 1];
   __shared__ float s_ssq[2][C];
-  float* sV = s_mem + 2 * L::kStage;
+  float* sV = s_mem + (L::kShareV ? L::kStage : 2 * L::kStage);
   pdl_launch_dependents();
   pdl_wait();
   const int chunk = blockIdx.x, head = blockIdx.y;
@@ -424,7 +425,7 @@ __global__ void __launch_bounds__(kChThreads) retention_chunk_out_kernel(const R
   };
   const int n_it = (D + KT - 1) / KT;
   load_stage(0);
-  tile_values<ET, P>(sV, L::kLdS, prow, p.ld, cp.n, E, vec_v);
+  if constexpr (!L::kShareV) tile_values<ET, P>(sV, L::kLdS, prow, p.ld, cp.n, E, vec_v);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   const int m0 = (warp & 3) * 16, half = warp >> 2;
@@ -466,6 +467,7 @@ __global__ void __launch_bounds__(kChThreads) retention_chunk_out_kernel(const R
     }
     __syncthreads();  // the stage may be refilled
   }
+  if constexpr (L::kShareV) tile_values<ET, P>(sV, L::kLdS, prow, p.ld, cp.n, E, vec_v);
   // weights of the chunk's own rows, and decay of what came before it
   float* sP = s_mem;
   const int i0 = m0 + g, i1 = m0 + g + 8;
