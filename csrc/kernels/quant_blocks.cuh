@@ -9,27 +9,9 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
-namespace oxb {
+#include "quant_types.cuh"
 
-// GGUF tensor type codes (subset with device decoders)
-enum QuantType : int {
-  kQ_F32 = 0,
-  kQ_F16 = 1,
-  kQ_Q4_0 = 2,
-  kQ_Q4_1 = 3,
-  kQ_Q5_0 = 6,
-  kQ_Q5_1 = 7,
-  kQ_Q8_0 = 8,
-  kQ_Q2_K = 10,
-  kQ_Q3_K = 11,
-  kQ_Q4_K = 12,
-  kQ_Q5_K = 13,
-  kQ_Q6_K = 14,
-  kQ_IQ4_NL = 20,
-  kQ_BF16 = 30,
-  kQ_TQ2_0 = 35,
-  kQ_NVFP4 = 144,
-};
+namespace oxb {
 
 template <int T> struct QInfo;
 template <> struct QInfo<kQ_Q4_0> { static constexpr int qk = 32, bytes = 18; };

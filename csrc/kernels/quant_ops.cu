@@ -630,15 +630,6 @@ bool launch_mmvq(int qtype, const MmvqParams& p, cudaStream_t stream) {
   return true;
 }
 
-bool mmvq_has_int8_path(int qtype) {
-  switch (qtype) {
-    case kQ_Q4_0: case kQ_Q4_1: case kQ_Q5_0: case kQ_Q5_1: case kQ_Q8_0: case kQ_Q4_K: case kQ_Q5_K: case kQ_Q6_K:
-      return true;
-    default:
-      return false;
-  }
-}
-
 bool launch_mmvq_mixed(const MmvqParams& p, cudaStream_t stream) {
   if (p.M <= 0 || p.N <= 0) return true;
   if (p.n_seg < 1 || p.n_seg > 4 || p.xq == nullptr) return false;
@@ -661,26 +652,6 @@ bool launch_dequant_rows(int qtype, const uint8_t* w, long long row_bytes, const
   OXB_QDISPATCH(qtype, CALL)
 #undef CALL
   return true;
-}
-
-long long quant_row_bytes(int qtype, long long K) {
-  switch (qtype) {
-    case kQ_F32: return K * 4;
-    case kQ_F16: case kQ_BF16: return K * 2;
-    case kQ_Q4_0: case kQ_IQ4_NL: return K / 32 * 18;
-    case kQ_Q4_1: return K / 32 * 20;
-    case kQ_Q5_0: return K / 32 * 22;
-    case kQ_Q5_1: return K / 32 * 24;
-    case kQ_Q8_0: return K / 32 * 34;
-    case kQ_Q2_K: return K / 256 * 84;
-    case kQ_Q3_K: return K / 256 * 110;
-    case kQ_Q4_K: return K / 256 * 144;
-    case kQ_Q5_K: return K / 256 * 176;
-    case kQ_Q6_K: return K / 256 * 210;
-    case kQ_TQ2_0: return K / 256 * 66;
-    case kQ_NVFP4: return K / 16 * 16;
-    default: return -1;
-  }
 }
 
 }  // namespace oxb

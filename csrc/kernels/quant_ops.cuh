@@ -3,6 +3,8 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#include "quant_types.cuh"
+
 namespace oxb {
 
 struct MmvqParams {
@@ -40,10 +42,8 @@ bool launch_mmvq(int qtype, const MmvqParams& p, cudaStream_t stream);
 // Q | K | V or gate | up projections of a mixed-precision GGUF file). Needs the int8 activations
 // (xq / xd / xs). Returns false when a segment's type has no integer path or an operand is misaligned.
 bool launch_mmvq_mixed(const MmvqParams& p, cudaStream_t stream);
-bool mmvq_has_int8_path(int qtype);
 bool launch_dequant_rows(int qtype, const uint8_t* w, long long row_bytes, const int* row_ids,
                          int n_rows, int K, __nv_bfloat16* out, long long ldo, float scale,
                          int n_src_rows, cudaStream_t stream);
-long long quant_row_bytes(int qtype, long long K);
 
 }  // namespace oxb

@@ -4,6 +4,8 @@ These extensions live beside this file after a build:
 
 * ``oxb_cuda``  - the sm_100a kernels (``csrc/kernels/*.cu`` + ``csrc/bindings.cpp``), compiled with
   ``-gencode arch=compute_100a,code=sm_100a``; nvcc cross-compiles them on a machine without a GPU.
+* ``oxb_quant`` - the kernels of quantised weights (``QUANT_KERNELS`` + ``csrc/bindings_quant.cpp``); built
+  when such weights are first used.
 * ``oxb_hybrid`` - the kernels that only layer-list decoders use (``HYBRID_KERNELS`` +
   ``csrc/bindings_hybrid.cpp``); built when such a model is first loaded.
 * ``oxb_host``  - the C++ host runtime (block manager, radix prefix cache, scheduler core, GGUF
@@ -45,11 +47,16 @@ CUDA_FLAGS = [
 # kernels of the extension that only layer-list decoders load
 HYBRID_KERNELS = ("stream_ops.cu", "mixer_ops.cu", "attn_rows.cu", "retention.cu")
 HYBRID_HEADERS = ("hybrid.cuh", "hybrid_dev.cuh")
+# kernels of the extension that only quantised weights load
+QUANT_KERNELS = ("quant_ops.cu", "gemm_fp8_block.cu", "nvfp4_quant.cu")
 
 
 def _sources(name: str) -> list[Path]:
     if name == "oxb_cuda":
-        return sorted(p for p in (_CSRC / "kernels").glob("*.cu") if p.name not in HYBRID_KERNELS) + [_CSRC / "bindings.cpp"]
+        return sorted(p for p in (_CSRC / "kernels").glob("*.cu") if p.name not in HYBRID_KERNELS + QUANT_KERNELS) + [
+            _CSRC / "bindings.cpp"]
+    if name == "oxb_quant":
+        return [_CSRC / "kernels" / k for k in QUANT_KERNELS] + [_CSRC / "bindings_quant.cpp"]
     if name == "oxb_hybrid":
         return [_CSRC / "kernels" / k for k in HYBRID_KERNELS] + [_CSRC / "bindings_hybrid.cpp"]
     if name == "oxb_host":
@@ -230,6 +237,10 @@ def noalloc_lib_path() -> Path:
 
 def cuda_ext():
     return load("oxb_cuda")
+
+
+def quant_ext():
+    return load("oxb_quant")
 
 
 def hybrid_ext():

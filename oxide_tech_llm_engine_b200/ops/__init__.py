@@ -11,7 +11,7 @@ from typing import Optional, Sequence
 
 import torch
 
-from .._build import cuda_ext
+from .._build import cuda_ext, quant_ext
 
 EPI_STORE_BF16 = 0
 EPI_RED_F32 = 1
@@ -35,6 +35,19 @@ launch_count = 0
 
 def _ext():
     return cuda_ext()
+
+
+def _quant_ext():
+    """The extension of the quantised-weight kernels, built and loaded with the first model that needs it."""
+    global _quant_pdl
+    m = quant_ext()
+    if _quant_pdl != _pdl:
+        m.set_pdl(_pdl)
+        _quant_pdl = _pdl
+    return m
+
+
+_pdl = _quant_pdl = False   # programmatic dependent launch: wanted, and as the quantised-weight extension has it
 
 
 def _bump(n: int = 1) -> None:
@@ -79,7 +92,9 @@ def set_pdl(on: bool) -> None:
     prologue (and, in the GEMM, requests the first weight tiles of its operand ring) and then waits
     for the earlier kernel to complete before it touches anything that kernel produced. Also holds
     inside CUDA graphs captured afterwards."""
-    _ext().set_pdl(bool(on))
+    global _pdl
+    _pdl = bool(on)
+    _ext().set_pdl(_pdl)
 
 
 def pdl_enabled() -> bool:
@@ -346,7 +361,7 @@ def quant_act_nvfp4(x: torch.Tensor, bufs=None, group_counts: Optional[torch.Ten
         q = bufs[0][:rows * K // 2].view(*x.shape[:-1], K // 2)
         sf = bufs[1][:tiles * (K // 64) * 512]
         gs = bufs[2][:rows]
-    _ext().quant_act_nvfp4(x, q, sf, gs, group_counts, ag_flags, ag_expected, ag_ticket, status_word(x.device),
+    _quant_ext().quant_act_nvfp4(x, q, sf, gs, group_counts, ag_flags, ag_expected, ag_ticket, status_word(x.device),
                            SPIN_LIMIT)
     _bump()
     return q, sf, gs
@@ -382,7 +397,7 @@ def quant_act_fp8(x: torch.Tensor, q: Optional[torch.Tensor] = None, sa_t: Optio
         q = torch.empty(M, K, dtype=torch.float8_e4m3fn, device=x.device)
     if sa_t is None:
         sa_t = torch.empty((K + 127) // 128, M, dtype=torch.float32, device=x.device)
-    _ext().quant_act_fp8(x, q, sa_t, ag_flags, ag_expected, ag_rows_per_src, ag_ticket, status_word(x.device))
+    _quant_ext().quant_act_fp8(x, q, sa_t, ag_flags, ag_expected, ag_rows_per_src, ag_ticket, status_word(x.device))
     _bump()
     return q, sa_t
 
@@ -397,7 +412,7 @@ def gemm_fp8_block(a8: torch.Tensor, sa_t: torch.Tensor, w8: torch.Tensor, sw: t
     to the row owner's receive slab, the last CTA signals the owners)."""
     if out is None and not slab_ptrs:
         out = torch.empty(a8.shape[0], w8.shape[0], dtype=torch.bfloat16, device=a8.device)
-    _ext().gemm_fp8_block(a8, sa_t, w8, sw, out, bias, status_word(a8.device), list(slab_ptrs), list(arrive_ptrs),
+    _quant_ext().gemm_fp8_block(a8, sa_t, w8, sw, out, bias, status_word(a8.device), list(slab_ptrs), list(arrive_ptrs),
                           done_ticket, rows_per_owner, my_rank, slab_ld)
     _bump()
     return out
@@ -563,7 +578,7 @@ def mmvq(qtype: int, w, x, out, *, n: int, k: int, bias=None, add: bool = False,
     `quant_q8_1(x)`: the block types of `INT8_MMVQ_CODES` then take the integer dot-product (dp4a)
     path, the others expand their weights to fp32."""
     q8, xd, xs = xq if xq is not None else (None, None, None)
-    _ext().mmvq(qtype, w, x, bias, out, n, k, add, q8, xd, xs)
+    _quant_ext().mmvq(qtype, w, x, bias, out, n, k, add, q8, xd, xs)
     _bump()
 
 
@@ -577,7 +592,7 @@ def mmvq_mixed(parts: Sequence, x, out, *, k: int, xq) -> None:
     the Q|K|V and gate|up projections of a mixed-precision GGUF file (Q4_K_M keeps attn_v in Q6_K)
     stay on one launch (reference: gemv_qkv_mixed_*, quant_gemv_kquants.cu:399-917)."""
     q8, xd, xs = xq
-    _ext().mmvq_mixed([int(c) for c, _, _ in parts], [w for _, w, _ in parts], [int(n) for _, _, n in parts],
+    _quant_ext().mmvq_mixed([int(c) for c, _, _ in parts], [w for _, w, _ in parts], [int(n) for _, _, n in parts],
                       x, out, k, q8, xd, xs)
     _bump()
 
@@ -601,13 +616,13 @@ def quant_q8_1(x: torch.Tensor, bufs=None):
         q8 = bufs[0][:M * K].view(M, K)
         xd = bufs[1][:M * (K // 32)].view(M, K // 32)
         xs = bufs[2][:M * (K // 32)].view(M, K // 32)
-    _ext().quant_q8_1(x, q8, xd, xs)
+    _quant_ext().quant_q8_1(x, q8, xd, xs)
     _bump()
     return q8, xd, xs
 
 
 def dequant_rows(qtype: int, w, out, *, n_src_rows: int, k: int, row_ids=None, scale: float = 1.0) -> None:
-    _ext().dequant_rows(qtype, w, row_ids, out, n_src_rows, k, scale)
+    _quant_ext().dequant_rows(qtype, w, row_ids, out, n_src_rows, k, scale)
     _bump()
 
 
