@@ -125,7 +125,7 @@ def main() -> None:
     if args.kipolix and args.impl != "reference":
         from oxide_tech_llm_engine_b200.bench_hybrid import run
 
-        run(args)
+        run(args, ClockSampler(0))
         return
     if args.impl == "reference":
         reference_arm()

@@ -143,16 +143,23 @@ void heads(const Tensor& proj, int64_t M, int64_t H, int64_t G, int64_t D, int64
   p.rot = rotary(freq_hi, freq_lo, interleaved, D);
   p.positions = i32(positions, M, "heads positions");
   p.k_scale = static_cast<float>(k_scale);
-  p.q_ld = pitch(q_out, M, H * q_hd, "heads q_out");
   p.q_out = q_out.data_ptr();
-  p.q_hd = static_cast<int>(q_hd);
   if (given(k_out)) {
-    TORCH_CHECK(q_out.scalar_type() == torch::kFloat32 && k_out->scalar_type() == torch::kFloat32, "heads: dense q and k are fp32");
+    // dense fp32 q [H, >= M, D] and k [G, >= M, D], rows of a head together
+    auto dense = [&](const Tensor& t, int64_t n) {
+      TORCH_CHECK(t.is_cuda() && t.scalar_type() == torch::kFloat32 && t.dim() == 3 && t.size(0) == n && t.size(1) >= M &&
+                      t.size(2) == D && t.stride(2) == 1 && t.stride(1) == D,
+                  "heads: dense q and k are fp32 [heads, rows, D]");
+      return t.stride(0);
+    };
     p.ld = pitch(proj, M, (H + G) * D, "heads proj");
-    p.k_ld = pitch(*k_out, M, G * D, "heads k_out");
+    p.q_hd = dense(q_out, H);
+    p.k_hd = dense(*k_out, G);
+    p.q_ld = p.k_ld = D;
     p.k_out = k_out->data_ptr<float>();
-    p.k_hd = static_cast<int>(D);
   } else {
+    p.q_ld = pitch(q_out, M, H * q_hd, "heads q_out");
+    p.q_hd = q_hd;
     TORCH_CHECK(given(k_cache) && given(v_cache) && given(slots), "heads: caches and slots, or k_out");
     TORCH_CHECK(q_out.scalar_type() == k_cache->scalar_type() && v_cache->scalar_type() == k_cache->scalar_type(),
                 "heads: one storage type");
@@ -274,8 +281,11 @@ void retention_prefill(const Tensor& proj, int64_t M, int64_t H, int64_t D, int6
   p.ctx_lens = i32(ctx_lens, n_seqs, "retention_prefill ctx_lens");
   p.n_tiles = static_cast<int>(n_tiles);
   p.n_seqs = static_cast<int>(n_seqs);
+  TORCH_CHECK(q_rot.dim() == 3 && q_rot.size(0) == H && q_rot.size(1) >= M && q_rot.size(2) == D && q_rot.sizes() == k_rot.sizes(),
+              "retention_prefill: q_rot and k_rot [H, rows, D]");
   p.q_rot = f32(q_rot, M * H * D, "retention_prefill q_rot");
   p.k_rot = f32(k_rot, M * H * D, "retention_prefill k_rot");
+  p.rot_hd = q_rot.stride(0);
   if (given(ws)) {
     TORCH_CHECK(dt == 0 && oxb::retention_chunks_ok(static_cast<int>(D), static_cast<int>(E)), "retention_prefill: chunked form");
     p.ws = const_cast<float*>(f32(*ws, 2 * n_tiles * H * D * E, "retention_prefill ws"));

@@ -68,12 +68,10 @@ struct HeadsParams {
   RotaryParams rot;
   const int* positions;     // [M]
   float k_scale;
-  void* q_out;
-  long long q_ld;
-  int q_hd;
+  void* q_out;              // element (row, head, d) at row * q_ld + head * q_hd + d
+  long long q_ld, q_hd;
   float* k_out;             // dense fp32 (then q_out is fp32 too) or nullptr
-  long long k_ld;
-  int k_hd;
+  long long k_ld, k_hd;
   void* k_cache;
   void* v_cache;
   const long long* slots;   // [M] cache slot of each row, < 0: not stored
@@ -133,8 +131,9 @@ struct RetentionParams {
   const int* q_lens;
   const int* ctx_lens;
   int n_tiles, n_seqs;
-  const float* q_rot;       // [M, H*D] fp32, rotated
-  const float* k_rot;       // [M, H*D] fp32, rotated and scaled
+  const float* q_rot;       // fp32, rotated: [H][M][D], heads rot_hd apart (a chunk of a head is one contiguous run)
+  const float* k_rot;       // the same layout, rotated and scaled
+  long long rot_hd;
   float* ws;                // [2 * n_tiles, H, D, E]: what each chunk adds to the state, then the state before it
   float* o_buf;             // [M, H*E] fp32 (token-by-token form only)
   void* out;                // [M, ldo]: norm(o) * silu(gate)

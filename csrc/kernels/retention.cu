@@ -267,8 +267,8 @@ __global__ void __launch_bounds__(kChThreads) retention_chunk_sum_kernel(const R
   const ChunkPos cp = chunk_pos(p, chunk);
   if (cp.n <= 0) return;
   const int D = p.D, E = p.E;
-  const long long ldk = static_cast<long long>(p.H) * D;
-  const float* ksrc = p.k_rot + cp.row0 * ldk + head * D;
+  const long long ldk = D;
+  const float* ksrc = p.k_rot + head * p.rot_hd + cp.row0 * ldk;
   const int n_it = (D + 63) / 64;
   auto load_k = [&](int it) {
     tile_f32<C, 64>(s_mem + (it & 1) * C * L::kLdK, L::kLdK, ksrc + it * 64, ldk, cp.n, D - it * 64, D % 4 == 0);
@@ -327,57 +327,70 @@ __global__ void __launch_bounds__(kChThreads) retention_chunk_sum_kernel(const R
   }
 }
 
-// 2. grid (D E / (256 V), H, sequences): walks the chunks of a sequence, eight loads ahead.
-template <int V>
+// 2. grid (D E / (256 V CH), H, sequences): walks the chunks of a sequence, U chunks of CH pieces per thread in
+// flight (a CTA covers CH x 4 KB of a state in one run).
+template <int V, int CH, int U>
 __global__ void __launch_bounds__(256) retention_scan_chunks_kernel(const RetentionParams p) {
   pdl_launch_dependents();
   pdl_wait();
   const int seq = blockIdx.z, head = blockIdx.y;
   const long long DE = static_cast<long long>(p.D) * p.E;
-  const long long i = (blockIdx.x * 256ll + threadIdx.x) * V;
+  const long long i0 = (static_cast<long long>(blockIdx.x) * 256 * CH + threadIdx.x) * V;
   const int slot = p.seq_slots[seq];
   if (slot < 0 || slot >= p.num_slots) {
-    if (i == 0) set_status_once(p.status, kStatusBadIndex);
+    if (i0 == 0) set_status_once(p.status, kStatusBadIndex);
     return;
   }
-  if (i >= DE) return;
   int tile0 = 0;
   for (int s = 0; s < seq; ++s) tile0 += (p.q_lens[s] + 127) >> 7;
   const int len = p.q_lens[seq];
   const int n_chunks = (len + C - 1) / C;
   const float* pw = p.decay_pow + head * (C + 1);
   const float g_full = pw[C], g_last = pw[len - (n_chunks - 1) * C];
-  float* st = p.state + (static_cast<long long>(slot) * p.H + head) * DE + i;
-  float* w = p.ws + (static_cast<long long>(2 * tile0) * p.H + head) * DE + i;
+  float* st = p.state + (static_cast<long long>(slot) * p.H + head) * DE + i0;
+  float* w = p.ws + (static_cast<long long>(2 * tile0) * p.H + head) * DE + i0;
   const long long step = static_cast<long long>(p.H) * DE;
-  float S[V];
+  const bool past = p.ctx_lens[seq] != len;
+  float S[CH][V];
+  bool in[CH];
 #pragma unroll
-  for (int j = 0; j < V; ++j) S[j] = 0.f;
-  if (p.ctx_lens[seq] != len) {  // the sequence has a past
-    if constexpr (V == 4) load4<float>(st, S);
-    else S[0] = *st;
+  for (int h = 0; h < CH; ++h) {
+    in[h] = i0 + h * 256 * V < DE;
+#pragma unroll
+    for (int j = 0; j < V; ++j) S[h][j] = 0.f;
+    if (past && in[h]) {
+      if constexpr (V == 4) load4<float>(st + h * 256 * V, S[h]);
+      else S[h][0] = st[h * 256 * V];
+    }
   }
-  constexpr int U = 8;
   for (int c0 = 0; c0 < n_chunks; c0 += U) {
-    float u[U][V];
+    float u[U][CH][V];
 #pragma unroll
     for (int k = 0; k < U; ++k)
-      if (c0 + k < n_chunks) {
-        if constexpr (V == 4) load4<float>(w + (c0 + k) * step, u[k]);
-        else u[k][0] = w[(c0 + k) * step];
-      }
+#pragma unroll
+      for (int h = 0; h < CH; ++h)
+        if (c0 + k < n_chunks && in[h]) {
+          if constexpr (V == 4) load4<float>(w + (c0 + k) * step + h * 256 * V, u[k][h]);
+          else u[k][h][0] = w[(c0 + k) * step + h * 256 * V];
+        }
 #pragma unroll
     for (int k = 0; k < U; ++k)
-      if (c0 + k < n_chunks) {
-        if constexpr (V == 4) store4<float>(w + (c0 + k) * step, S);
-        else w[(c0 + k) * step] = S[0];
-        const float g = c0 + k == n_chunks - 1 ? g_last : g_full;
 #pragma unroll
-        for (int j = 0; j < V; ++j) S[j] = fmaf(g, S[j], u[k][j]);
-      }
+      for (int h = 0; h < CH; ++h)
+        if (c0 + k < n_chunks && in[h]) {
+          if constexpr (V == 4) store4<float>(w + (c0 + k) * step + h * 256 * V, S[h]);
+          else w[(c0 + k) * step + h * 256 * V] = S[h][0];
+          const float g = c0 + k == n_chunks - 1 ? g_last : g_full;
+#pragma unroll
+          for (int j = 0; j < V; ++j) S[h][j] = fmaf(g, S[h][j], u[k][h][j]);
+        }
   }
-  if constexpr (V == 4) store4<float>(st, S);
-  else *st = S[0];
+#pragma unroll
+  for (int h = 0; h < CH; ++h)
+    if (in[h]) {
+      if constexpr (V == 4) store4<float>(st + h * 256 * V, S[h]);
+      else st[h * 256 * V] = S[h][0];
+    }
 }
 
 // 3. grid (chunks, H): the chunk's outputs over all value dimensions.
@@ -406,9 +419,9 @@ __global__ void __launch_bounds__(kChThreads, ET <= 128 ? 3 : 1) retention_chunk
   const ChunkPos cp = chunk_pos(p, chunk);
   if (cp.n <= 0) return;
   const int D = p.D, E = p.E;
-  const long long ldq = static_cast<long long>(p.H) * D;
-  const float* qsrc = p.q_rot + cp.row0 * ldq + head * D;
-  const float* ksrc = p.k_rot + cp.row0 * ldq + head * D;
+  const long long ldq = D;
+  const float* qsrc = p.q_rot + head * p.rot_hd + cp.row0 * ldq;
+  const float* ksrc = p.k_rot + head * p.rot_hd + cp.row0 * ldq;
   const float* ssrc = p.ws + (static_cast<long long>(chunk) * p.H + head) * D * E;
   const P* prow = static_cast<const P*>(p.proj) + cp.row0 * p.ld + 2 * p.H * D + head * E;
   const bool vec_d = D % 4 == 0, vec_e = E % 4 == 0;
@@ -562,8 +575,8 @@ __global__ void __launch_bounds__(256) retention_scan_kernel(const RetentionPara
   const float gamma = p.decay_pow[head * (kRetChunk + 1) + 1];
   for (int i = 0; i < len; ++i) {
     const long long row = p.q_start[seq] + i;
-    const float* q = p.q_rot + (row * p.H + head) * D;
-    const float* k = p.k_rot + (row * p.H + head) * D;
+    const float* q = p.q_rot + head * p.rot_hd + row * D;
+    const float* k = p.k_rot + head * p.rot_hd + row * D;
     const float v = e < E ? to_f(from_f<T>(to_f(static_cast<const P*>(p.proj)[row * p.ld + 2 * p.H * D + head * E + e]))) : 0.f;
     float acc = 0.f;
     for (int d = w; d < D; d += 8) {
@@ -642,9 +655,12 @@ cudaError_t launch_chunks(const RetentionParams& p, cudaStream_t stream) {
   if (e != cudaSuccess) return e;
   const long long de = static_cast<long long>(p.D) * p.E;
   const int v = p.E % 4 == 0 ? 4 : 1;
-  const dim3 grid2(static_cast<unsigned>((de + 256 * v - 1) / (256 * v)), p.H, p.n_seqs);
-  e = launch_kernel(v == 4 ? retention_scan_chunks_kernel<4> : retention_scan_chunks_kernel<1>, grid2, dim3(256), 0, stream,
-                    true, false, p);
+  // whole runs of 16 KB per CTA where that still leaves enough CTAs
+  const bool wide = v == 4 && de >= 4096 && (de / 4096) * p.H * p.n_seqs >= 2 * sm_count();
+  const long long per = 256ll * v * (wide ? 4 : 1);
+  const dim3 grid2(static_cast<unsigned>((de + per - 1) / per), p.H, p.n_seqs);
+  auto scan = wide ? retention_scan_chunks_kernel<4, 4, 2> : (v == 4 ? retention_scan_chunks_kernel<4, 1, 8> : retention_scan_chunks_kernel<1, 1, 8>);
+  e = launch_kernel(scan, grid2, dim3(256), 0, stream, true, false, p);
   if (e != cudaSuccess) return e;
   return launch_kernel(retention_chunk_out_kernel<ET, P>, dim3(chunks, p.H), dim3(kChThreads), smem3, stream, true, false, p);
 }

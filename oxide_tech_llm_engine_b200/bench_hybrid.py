@@ -245,7 +245,7 @@ def kernel_numbers(kip, lla, peaks: dict, timer: Timer, batch: int, ctx: int, m:
                                              row_slots=sl, positions=ps, out=out)
     add(f"retention_decode [{batch} x {h} states of {D} x {E}]", rd, batch * (h * D * E * 8 + 2 * (WR + h * E)))
     C = hops.retention_chunk()
-    qr_, kr_ = torch.randn(m, h * D, device=dev), torch.randn(m, h * D, device=dev)
+    qr_, kr_ = torch.randn(h, m, D, device=dev), torch.randn(h, m, D, device=dev)
     ws = torch.empty(2 * len(tiles) * h * D * E, device=dev)
     sl = torch.arange(ns, dtype=torch.int32, device=dev)
     proj = torch.randn(m, WR, **bf)
@@ -268,7 +268,8 @@ def kernel_numbers(kip, lla, peaks: dict, timer: Timer, batch: int, ctx: int, m:
     return rows
 
 
-def run(args) -> None:
+def run(args, clocks) -> None:
+    """`clocks`: bench.py's nvidia-smi sampler."""
     from .utils.roofline import load_measured_peaks
 
     torch.cuda.set_device(0)
@@ -279,6 +280,7 @@ def run(args) -> None:
     timer = Timer(max(3, args.warmup), max(20, args.steps))
     out = {"bench": "kipolix beside llama", "layers": args.layers or 8, "data": "random tokens, random weights", "peaks": {
         k: peaks.get(k) for k in ("hbm_gbs", "bf16_tflops")}, "sizes": {}}
+    clocks.start()
     names = [args.kipolix_size] if args.kipolix_size else list(SIZES)
     for name in names:
         kip, lla = _configs(name, out["layers"])
@@ -292,4 +294,5 @@ def run(args) -> None:
         res["kernels"] = kernel_numbers(kip, lla, peaks, timer, batch=64, ctx=4096, m=8192)
         out["sizes"][name] = res
         torch.cuda.empty_cache()
+    out["clocks"] = clocks.stop()
     print(json.dumps(out), flush=True)

@@ -116,9 +116,9 @@ class RetentionRun:
                                   positions=s.positions, **kw)
         if s.n_prefill > 0:
             hd = r.heads * r.dim
-            q_rot, k_rot = m.scratch("q_rot", M * hd).view(M, hd), m.scratch("k_rot", M * hd).view(M, hd)
+            q_rot, k_rot = (m.scratch(n, M * hd).view(r.heads, M, r.dim) for n in ("q_rot", "k_rot"))
             hops.heads(proj[nd:M], M - nd, h=r.heads, g=r.heads, d=r.dim, e=r.vdim, rot=w["rot"], positions=s.positions[nd:],
-                       q_out=q_rot[nd:], q_hd=r.dim, k_out=k_rot[nd:], k_scale=self.k_scale)
+                       q_out=q_rot[:, nd:], q_hd=r.dim, k_out=k_rot[:, nd:], k_scale=self.k_scale)
             if self.chunked:
                 kw["ws"] = m.scratch("chunk_states", 2 * s.n_tiles * r.state_elems)
             else:

@@ -65,8 +65,8 @@ def stream_norm(x: torch.Tensor, rows: int, *, norm_w: torch.Tensor, eps: float,
 def heads(proj: torch.Tensor, m: int, *, h: int, g: int, d: int, e: int, rot: Rotary, positions, q_out, q_hd: int,
           q_norm=None, k_norm=None, eps: float = 1e-5, k_scale: float = 1.0, k_out=None, k_cache=None, v_cache=None,
           slots=None) -> None:
-    """Projection rows q | k | v -> normed and rotated heads; k and v into the paged cache, or q and k to
-    dense fp32 buffers (HeadsParams)."""
+    """Projection rows q | k | v -> normed and rotated heads; k and v into the paged cache with q [M, h * q_hd], or
+    q and k to dense fp32 buffers [heads, M, d] (HeadsParams)."""
     hybrid_ext().heads(proj, m, h, g, d, e, q_norm, k_norm, eps, rot.hi, rot.lo, rot.interleaved, positions, k_scale, q_out,
                        q_hd, k_out, k_cache, v_cache, slots, ops.status_word(proj.device))
     ops._bump()

@@ -44,7 +44,7 @@ CONFIGS = {
     "retention": model(96, 90, [mlp(ret(2, 32, 48, 32, [1.0, 0.25]), 64), ret(4, 24, 20, 12, [0.99, 0.97, 0.9, 0.5])],
                        streams=4, loop=(0, 2, 2), mul=(13, 5)),
     # head sizes beyond the tensor-core attention, more streams than four, no bigram, window of one
-    "wide": model(128, 200, [mlp(att(2, 1, 144, 72, 40, 40, 3, gain=1.5), 64), mlp(att(3, 3, 16, 144, 16, 1, 2), 64),
+    "wide": model(128, 200, [mlp(att(2, 1, 144, 72, 40, 41, 3, gain=1.5), 64), mlp(att(3, 3, 16, 144, 16, 1, 2), 64),
                              mlp(ret(1, 136, 264, 8, [0.995]), 96)], streams=5, buckets=0),
 }
 

@@ -181,7 +181,7 @@ def run_attention(H, path, q, k, v, scale, size, keep, mode, splits=4):
 
 
 @pytest.mark.parametrize("path", ["tc", "bf16", "f32"])
-@pytest.mark.parametrize("heads,G,D,E,T,size,keep", [(4, 2, 64, 64, 300, 40, 4), (3, 1, 48, 96, 420, 129, 17), (2, 2, 96, 32, 200, 16, 0),
+@pytest.mark.parametrize("heads,G,D,E,T,size,keep", [(4, 2, 64, 64, 300, 44, 6), (3, 1, 48, 96, 420, 129, 17), (2, 2, 96, 32, 200, 16, 0),
                                                      (8, 1, 128, 128, 530, 257, 130), (2, 1, 80, 72, 150, 1, 3), (4, 4, 32, 40, 270, 1000, 5)])
 def test_attention_sees_the_window_and_the_kept_first_positions_and_nothing_else(H, path, heads, G, D, E, T, size, keep):
     g = gen(T + D)
@@ -244,7 +244,7 @@ def run_retention(H, q, k, v, gate, decay, cuts, dtype, slots, proj_f32, chunked
             H.retention_decode(pr, 1, rot=rot, k_scale=k_scale, row_slots=i32([slots]), positions=pos, **kw)
         else:
             tiles = -(-n // 128)
-            qr, kr = torch.empty(n, h * D, device=DEV), torch.empty(n, h * D, device=DEV)
+            qr, kr = torch.empty(h, n, D, device=DEV), torch.empty(h, n, D, device=DEV)
             H.heads(pr, n, h=h, g=h, d=D, e=E, rot=rot, positions=pos, q_out=qr, q_hd=D, k_out=kr, k_scale=k_scale)
             if chunked:
                 kw["ws"] = torch.full((2 * tiles * h * D * E,), float("nan"), device=DEV)
@@ -316,7 +316,7 @@ def test_ragged_batch_of_chunks_and_decode_rows_keeps_states_apart(H):
     i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=DEV)
     start = np.cumsum([0] + lens[:-1]).tolist()
     tiles = [(s, t * 128) for s, n in enumerate(lens) for t in range(-(-n // 128))]
-    qr, kr = torch.empty(M, h * D, device=DEV), torch.empty(M, h * D, device=DEV)
+    qr, kr = torch.empty(h, M, D, device=DEV), torch.empty(h, M, D, device=DEV)
     H.heads(proj, M, h=h, g=h, d=D, e=E, rot=H.Rotary(None, DEV), positions=i32([0] * M), q_out=qr, q_hd=D, k_out=kr)
     out = torch.zeros(M, h * E, dtype=torch.bfloat16, device=DEV)
     H.retention_prefill(proj, M, h=h, d=D, e=E, decay_pow=H.decay_powers(decay, DEV), eps=1e-3, state=state, seq_slots=i32(slots),
