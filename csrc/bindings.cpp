@@ -7,8 +7,9 @@
 #include <pybind11/stl.h>
 #include <torch/extension.h>
 
-#include <string>
+#include <cmath>
 #include <cstring>
+#include <string>
 #include <vector>
 
 #include "common/device_info.h"
@@ -74,41 +75,45 @@ void gemm_bf16(const Tensor& a, const Tensor& w, int64_t epi, const c10::optiona
   TORCH_CHECK(a.stride(-1) == 1 && w.stride(-1) == 1, "gemm_bf16: K must be contiguous");
   TORCH_CHECK(b_tiled == 0 || !(group_counts.has_value() && group_counts->defined()),
               "gemm_bf16: grouped GEMMs take row-major weights");
+  // packed rows of all groups in one [rows, K] operand (see GemmParams::packed_rows)
+  const bool packed_rows = a.dim() == 2 && w.dim() == 3;
   const bool grouped3d = a.dim() == 3;
   const bool tiled = b_tiled != 0;
+  TORCH_CHECK(!packed_rows || (group_counts.has_value() && group_counts->defined() && !fp4 && out.has_value() && out->dim() == 2),
+              "gemm_bf16: packed rows need group_counts, bf16 operands and a 2-D out");
   if (tiled) {
     TORCH_CHECK(a.dim() == 2 && w.dim() == 4 && w.size(2) == 128 && w.size(3) == 64 && w.is_contiguous(),
                 "gemm_bf16: tile-major weights are [N/128, K/64, 128, 64] contiguous, 2-D activations");
   } else {
-    TORCH_CHECK(w.dim() == a.dim(), "gemm_bf16: a and w must have the same rank");
+    TORCH_CHECK(w.dim() == a.dim() || packed_rows, "gemm_bf16: a and w must have the same rank");
   }
-  const int64_t G = grouped3d ? a.size(0) : 1;
+  const int64_t G = grouped3d || packed_rows ? w.size(0) : 1;
   const int64_t M = grouped3d ? a.size(1) : a.size(0);
   // K in operand elements of 2 bytes for the tile arithmetic below: a row of the packed fp4 operands
   // has K / 2 bytes = K / 4 such units, and one 128-byte k block covers 256 fp4 values
   const int64_t K = fp4 ? a.size(-1) / 2 : a.size(-1);
-  const int64_t N = tiled ? w.size(0) * 128 : (grouped3d ? w.size(1) : w.size(0));
+  const int64_t N = tiled ? w.size(0) * 128 : (w.dim() == 3 ? w.size(1) : w.size(0));
   TORCH_CHECK(tiled ? w.size(1) * 64 == K : w.size(-1) == a.size(-1), "gemm_bf16: K mismatch");
   TORCH_CHECK(K % 8 == 0, "gemm_bf16: K must be a multiple of 8 (16-byte TMA rows)");
   if (fp4) {
     TORCH_CHECK(!tiled && a.size(-1) % 128 == 0, "gemm (nvfp4): K must be a multiple of 256, row-major weights");
   }
   if (grouped3d) {
-    TORCH_CHECK(w.size(0) == G, "gemm_bf16: group mismatch");
+    TORCH_CHECK(a.size(0) == G, "gemm_bf16: group mismatch");
   }
 
   const uint64_t eb = fp4 ? 1 : 2;  // bytes per tensor element
   const uint64_t a_row = static_cast<uint64_t>(a.stride(-2)) * eb;
   const uint64_t w_row = tiled ? 128 : static_cast<uint64_t>(w.stride(-2)) * eb;
   const uint64_t a_grp = grouped3d ? static_cast<uint64_t>(a.stride(0)) * eb : a_row * M;
-  const uint64_t w_grp = tiled ? 16384 : (grouped3d ? static_cast<uint64_t>(w.stride(0)) * eb : w_row * N);
+  const uint64_t w_grp = tiled ? 16384 : (w.dim() == 3 ? static_cast<uint64_t>(w.stride(0)) * eb : w_row * N);
   const int bn_i = bn == 64 ? 64 : (bn == 256 ? 256 : 128);
   // decode tiles (mt = 2): one copy per operand and stage instead of two 16 KB boxes each
   const bool wide = mt == 2 && !grouped3d && wide_boxes != 0;
   const CUtensorMapDataType dt = fp4 ? CU_TENSOR_MAP_DATA_TYPE_UINT8 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   const uint64_t k_inner = fp4 ? static_cast<uint64_t>(a.size(-1)) : static_cast<uint64_t>(K);  // elements of the map's type
   const uint32_t box_inner = fp4 ? 128 : 64;
-  CUtensorMap tmA = oxb::make_tma_map(a.data_ptr(), dt, static_cast<int>(eb), 3, k_inner, M, G,
+  CUtensorMap tmA = oxb::make_tma_map(a.data_ptr(), dt, static_cast<int>(eb), 3, k_inner, M, packed_rows ? 1 : G,
                                       a_row, a_grp, box_inner, wide ? 256 : 128, 1, CU_TENSOR_MAP_SWIZZLE_128B);
   const uint64_t total_kb_u = static_cast<uint64_t>((K + 63) / 64);
   CUtensorMap tmB =
@@ -203,8 +208,12 @@ void gemm_bf16(const Tensor& a, const Tensor& w, int64_t epi, const c10::optiona
     TORCH_CHECK(mt_i == 1 && !fixup, "gemm_bf16: grouped GEMMs use 128-row tiles without the split-K fix-up");
     p.group_counts = reinterpret_cast<const uint32_t*>(group_counts->data_ptr());
     p.n_groups = static_cast<int>(G);
+    p.packed_rows = packed_rows ? 1 : 0;
+    TORCH_CHECK(group_counts->numel() >= G && G <= 1024, "gemm_bf16: one row count per group, at most 1024 groups");
     TORCH_CHECK(m_tiles_override > 0, "gemm_bf16: grouped mode needs the m-tile bound");
     m_tiles = static_cast<int>(m_tiles_override);
+    TORCH_CHECK(!packed_rows || (static_cast<int64_t>(m_tiles) * 128 <= M && out->size(0) >= M),
+                "gemm_bf16: packed rows in whole 128-row tiles");
     if (row_meta.has_value() && row_meta->defined()) {
       p.row_meta = reinterpret_cast<const oxb::RowMeta*>(row_meta->data_ptr());
       p.meta_group_stride = M;
@@ -314,7 +323,7 @@ void paged_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
                   const c10::optional<Tensor>& status, const c10::optional<Tensor>& page_ml,
                   const c10::optional<Tensor>& block_mass, const c10::optional<Tensor>& q8,
                   const c10::optional<Tensor>& q8_d, const c10::optional<Tensor>& q8_s, int64_t keep_first, int64_t out_d,
-                  bool exact_p) {
+                  bool exact_p, int64_t chunk, double sink) {
   TORCH_CHECK(q.dim() == 3 && k_cache.dim() == 4, "paged_decode: q [B,Hq,D], cache [blk,Hkv,16,D]");
   TORCH_CHECK(k_cache.size(2) == 16, "paged_decode: 16-token pages");
   oxb::DecodeAttnParams p{};
@@ -344,7 +353,11 @@ void paged_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
   p.out_d = static_cast<int>(out_d);
   p.exact_p = exact_p ? 1 : 0;
   TORCH_CHECK(out_d >= 0 && out_d <= D, "paged_decode: out_d");
-  TORCH_CHECK(!(page_ml.has_value() && (keep_first > 0 || exact_p)), "paged_decode: block mass goes with the plain window");
+  TORCH_CHECK(chunk >= 0 && (chunk == 0 || (window == 0 && keep_first == 0)), "paged_decode: a window or a chunk");
+  p.chunk = static_cast<int>(chunk);
+  p.sink_log2 = static_cast<float>(sink * 1.4426950408889634);
+  TORCH_CHECK(!(page_ml.has_value() && (keep_first > 0 || exact_p || std::isfinite(sink))),
+              "paged_decode: block mass goes with the plain window");
   p.scale_log2 = static_cast<float>(scale * 1.4426950408889634);
   p.status = opt_ptr<int>(status);  // given only when bounds checking is on
   p.num_blocks = p.status != nullptr ? static_cast<int>(k_cache.size(0)) : 0;
@@ -377,7 +390,7 @@ void paged_prefill_tc(const Tensor& q, const Tensor& k_cache, const Tensor& v_ca
                       const Tensor& block_tables, const Tensor& tile_seq, const Tensor& tile_q0,
                       const Tensor& q_start, const Tensor& q_lens, const Tensor& ctx_lens,
                       const Tensor& out, int64_t n_tiles, int64_t window, double scale,
-                      const Tensor& status, int64_t keep_first, int64_t out_d, bool exact_p) {
+                      const Tensor& status, int64_t keep_first, int64_t out_d, bool exact_p, int64_t chunk, double sink) {
   TORCH_CHECK(q.dim() == 3 && k_cache.dim() == 4, "paged_prefill_tc: q [T,Hq,D], cache [blk,Hkv,16,D]");
   TORCH_CHECK(k_cache.is_contiguous() && v_cache.is_contiguous(), "paged_prefill_tc: contiguous caches");
   oxb::PrefillAttnParams p{};
@@ -404,6 +417,9 @@ void paged_prefill_tc(const Tensor& q, const Tensor& k_cache, const Tensor& v_ca
   p.out_d = static_cast<int>(out_d);
   p.exact_p = exact_p ? 1 : 0;
   TORCH_CHECK(out_d >= 0 && out_d <= D, "paged_prefill_tc: out_d");
+  TORCH_CHECK(chunk >= 0 && (chunk == 0 || (window == 0 && keep_first == 0)), "paged_prefill_tc: a window or a chunk");
+  p.chunk = static_cast<int>(chunk);
+  p.sink_log2 = static_cast<float>(sink * 1.4426950408889634);
   p.scale_log2 = static_cast<float>(scale * 1.4426950408889634);
   const uint64_t T = q.size(0);
   const uint64_t kv_rows = static_cast<uint64_t>(k_cache.size(0)) * p.Hkv * 16;

@@ -4,6 +4,8 @@
 #include <cuda_runtime.h>
 #include <torch/extension.h>
 
+#include <vector>
+
 #include "common/device_info.h"
 #include "kernels/hybrid.cuh"
 
@@ -46,8 +48,9 @@ int64_t pitch(const Tensor& t, int64_t rows, int64_t cols, const char* what) {
               "] rows expected");
   return t.stride(0);
 }
-oxb::RotaryParams rotary(const OptTensor& hi, const OptTensor& lo, bool interleaved, int64_t D) {
+oxb::RotaryParams rotary(const OptTensor& hi, const OptTensor& lo, bool interleaved, double gain, int64_t D) {
   oxb::RotaryParams r{};
+  r.gain = static_cast<float>(gain);
   if (given(hi)) {
     r.dims = static_cast<int>(2 * hi->numel());
     TORCH_CHECK(r.dims <= D, "rotary: more dimensions than a head has");
@@ -121,7 +124,7 @@ void stream_norm(const Tensor& x, int64_t rows, const OptTensor& tokens, const O
 
 void heads(const Tensor& proj, int64_t M, int64_t H, int64_t G, int64_t D, int64_t E, const OptTensor& q_norm,
            const OptTensor& k_norm, double eps, const OptTensor& freq_hi, const OptTensor& freq_lo, bool interleaved,
-           const Tensor& positions, double k_scale, const Tensor& q_out, int64_t q_hd, const OptTensor& k_out,
+           double gain, const Tensor& positions, double k_scale, const Tensor& q_out, int64_t q_hd, const OptTensor& k_out,
            const OptTensor& k_cache, const OptTensor& v_cache, const OptTensor& slots, const Tensor& status) {
   oxb::HeadsParams p{};
   // storage type: that of the caches; dense q and k are fp32 whatever the projection is
@@ -140,7 +143,7 @@ void heads(const Tensor& proj, int64_t M, int64_t H, int64_t G, int64_t D, int64
   p.k_norm = f32(k_norm, G * D, "heads k_norm");
   TORCH_CHECK((p.q_norm == nullptr) == (p.k_norm == nullptr), "heads: q and k norm go together");
   p.eps = static_cast<float>(eps);
-  p.rot = rotary(freq_hi, freq_lo, interleaved, D);
+  p.rot = rotary(freq_hi, freq_lo, interleaved, gain, D);
   p.positions = i32(positions, M, "heads positions");
   p.k_scale = static_cast<float>(k_scale);
   p.q_out = q_out.data_ptr();
@@ -183,7 +186,7 @@ void heads(const Tensor& proj, int64_t M, int64_t H, int64_t G, int64_t D, int64
 void row_attention(const Tensor& q, int64_t q_hd, const Tensor& k_cache, const Tensor& v_cache, const Tensor& block_tables,
                    const OptTensor& seq_lens, const OptTensor& tile_seq, const OptTensor& tile_q0, const OptTensor& q_start,
                    const OptTensor& q_lens, const OptTensor& ctx_lens, int64_t n, int64_t H, int64_t D, int64_t E, int64_t window,
-                   int64_t keep_first, double scale, const Tensor& out, const Tensor& status) {
+                   int64_t keep_first, int64_t chunk, double scale, double sink, const Tensor& out, const Tensor& status) {
   oxb::RowAttnParams p{};
   const int dt = dtype_code(q, "row_attention q");
   TORCH_CHECK(k_cache.dim() == 4 && v_cache.dim() == 4 && k_cache.is_contiguous() && v_cache.is_contiguous() &&
@@ -222,7 +225,10 @@ void row_attention(const Tensor& q, int64_t q_hd, const Tensor& k_cache, const T
   }
   p.window = static_cast<int>(window);
   p.keep_first = static_cast<int>(keep_first);
+  TORCH_CHECK(chunk >= 0 && (chunk == 0 || (window == 0 && keep_first == 0)), "row_attention: a window or a chunk");
+  p.chunk = static_cast<int>(chunk);
   p.scale = static_cast<float>(scale);
+  p.sink = static_cast<float>(sink);
   p.ldo = pitch(out, 1, H * E, "row_attention out");
   p.out = out.data_ptr();
   p.status = status_ptr(status);
@@ -252,13 +258,13 @@ oxb::RetentionParams retention_common(const Tensor& proj, int64_t M, int64_t H, 
 }
 
 void retention_decode(const Tensor& proj, int64_t rows, int64_t H, int64_t D, int64_t E, const Tensor& decay_pow,
-                      const OptTensor& freq_hi, const OptTensor& freq_lo, bool interleaved, double k_scale, double eps,
+                      const OptTensor& freq_hi, const OptTensor& freq_lo, bool interleaved, double gain, double k_scale, double eps,
                       const Tensor& state, const Tensor& row_slots, const Tensor& positions, const Tensor& out,
                       const Tensor& status) {
   const int dt = dtype_code(out, "retention_decode out");
   oxb::RetentionParams p = retention_common(proj, rows, H, D, E, decay_pow, state, eps, out, status);
   TORCH_CHECK(D <= 4096 && E <= 4096, "retention_decode: head sizes");
-  p.rot = rotary(freq_hi, freq_lo, interleaved, D);
+  p.rot = rotary(freq_hi, freq_lo, interleaved, gain, D);
   p.k_scale = static_cast<float>(k_scale);
   p.row_slots = i32(row_slots, rows, "retention_decode row_slots");
   p.positions = i32(positions, rows, "retention_decode positions");
@@ -297,6 +303,263 @@ void retention_prefill(const Tensor& proj, int64_t M, int64_t H, int64_t D, int6
   }
 }
 
+void branch_norm(const Tensor& x, int64_t rows, const OptTensor& tokens, const OptTensor& embed, double embed_scale,
+                 const std::vector<Tensor>& ys, const std::vector<OptTensor>& ws, const std::vector<double>& gains,
+                 const std::vector<bool>& clears, const OptTensor& e_rows, const OptTensor& e_slot, const OptTensor& e_weight,
+                 int64_t top, bool store_x, const std::vector<Tensor>& norm_ws, const std::vector<Tensor>& hs, double eps,
+                 double w_offset, const OptTensor& row_map, const OptTensor& clear, const Tensor& status) {
+  TORCH_CHECK(x.dim() == 2, "branch_norm: x [rows, N]");
+  oxb::BranchNormParams p{};
+  p.rows = static_cast<int>(rows);
+  p.N = static_cast<int>(x.size(1));
+  TORCH_CHECK(x.size(0) >= rows && p.N <= 32768, "branch_norm: rows of at most 32768 values");
+  p.x = const_cast<float*>(f32(x, rows * p.N, "branch_norm x"));
+  TORCH_CHECK(!hs.empty() && hs.size() <= 2 && hs.size() == norm_ws.size(), "branch_norm: one or two outputs");
+  const int dt = dtype_code(hs[0], "branch_norm h");
+  p.n_out = static_cast<int>(hs.size());
+  for (size_t o = 0; o < hs.size(); ++o) {
+    TORCH_CHECK(hs[o].scalar_type() == hs[0].scalar_type(), "branch_norm: one storage type");
+    p.ldh = pitch(hs[o], given(row_map) ? 1 : rows, p.N, "branch_norm h");
+    TORCH_CHECK(p.ldh == hs[0].stride(0), "branch_norm: one row pitch of h");
+    p.h[o] = hs[o].data_ptr();
+    p.norm_w[o] = f32(norm_ws[o], p.N, "branch_norm norm_w");
+  }
+  TORCH_CHECK(ys.size() <= oxb::kMaxBranches && ws.size() == ys.size() && gains.size() == ys.size() && clears.size() == ys.size(),
+              "branch_norm: at most ", oxb::kMaxBranches, " branches");
+  p.n_branches = static_cast<int>(ys.size());
+  for (size_t b = 0; b < ys.size(); ++b) {
+    TORCH_CHECK(ys[b].is_cuda() && ys[b].scalar_type() == torch::kFloat32, "branch_norm: fp32 branches");
+    p.ldy = pitch(ys[b], rows, p.N, "branch_norm y");
+    TORCH_CHECK(p.ldy == ys[0].stride(0), "branch_norm: one row pitch of the branches");
+    p.y[b] = ys[b].data_ptr<float>();
+    p.w[b] = f32(ws[b], p.N, "branch_norm branch weight");
+    p.gain[b] = static_cast<float>(gains[b]);
+    p.clear_y[b] = clears[b] ? 1 : 0;
+  }
+  if (given(tokens)) {
+    TORCH_CHECK(given(embed) && embed->scalar_type() == hs[0].scalar_type() && embed->is_contiguous() && embed->dim() == 2 &&
+                    embed->size(1) == p.N && !given(e_rows),
+                "branch_norm: embed [vocab, N] of h's type");
+    p.tokens = i32(*tokens, rows, "branch_norm tokens");
+    p.embed = embed->data_ptr();
+    p.vocab = static_cast<int>(embed->size(0));
+    p.embed_scale = static_cast<float>(embed_scale);
+  } else {
+    TORCH_CHECK(!ys.empty(), "branch_norm: tokens or branches");
+  }
+  if (given(e_rows)) {
+    TORCH_CHECK(given(e_slot) && given(e_weight) && top >= 1 && e_rows->scalar_type() == hs[0].scalar_type() && e_rows->is_cuda(),
+                "branch_norm: expert rows of h's type, with slots and weights");
+    p.lde = pitch(*e_rows, 1, p.N, "branch_norm expert rows");
+    p.n_e_rows = e_rows->size(0);
+    p.e_rows = e_rows->data_ptr();
+    p.e_slot = i32(*e_slot, rows * top, "branch_norm slots");
+    p.e_weight = f32(*e_weight, rows * top, "branch_norm weights");
+    p.top = static_cast<int>(top);
+  }
+  p.store_x = store_x ? 1 : 0;
+  p.eps = static_cast<float>(eps);
+  p.w_offset = static_cast<float>(w_offset);
+  if (given(row_map)) p.row_map = i32(*row_map, rows, "branch_norm row_map");
+  if (given(clear)) {
+    p.clear_ld = pitch(*clear, rows, 1, "branch_norm clear");
+    TORCH_CHECK(clear->scalar_type() == torch::kFloat32 && clear->is_cuda() && p.clear_ld % 4 == 0 && clear->size(1) % 4 == 0,
+                "branch_norm: clear is fp32 in whole 16-byte pieces");
+    p.clear = clear->data_ptr<float>();
+    p.clear_n = static_cast<int>(clear->size(1));
+  }
+  p.status = status_ptr(status);
+  check_launch(oxb::launch_branch_norm(p, dt, cur_stream()), "branch_norm");
+}
+
+// Sizes, weights and state of a state-space layer. proj: rows z | x | B | C | dt, heads of EP, states of NP.
+oxb::SsdParams ssd_common(const Tensor& proj, int64_t M, int64_t H, int64_t G, const std::vector<Tensor>& w, const Tensor& state,
+                          const Tensor& conv_state, const Tensor& y, const Tensor& status) {
+  oxb::SsdParams p{};
+  TORCH_CHECK(state.dim() == 4 && state.size(1) == H && state.size(2) % 16 == 0 && state.size(3) % 16 == 0,
+              "ssd: state [slots, H, N, E], N and E multiples of 16");
+  p.state = const_cast<float*>(f32(state, 1, "ssd state"));
+  p.num_slots = static_cast<int>(state.size(0));
+  TORCH_CHECK(G >= 1 && H % G == 0, "ssd: groups divide the heads");
+  p.H = static_cast<int>(H);
+  p.G = static_cast<int>(G);
+  p.NP = static_cast<int>(state.size(2));
+  p.EP = static_cast<int>(state.size(3));
+  TORCH_CHECK(p.NP <= 1600 && p.EP <= 4096, "ssd: state and head sizes");
+  const int64_t inner = H * p.EP, ch = inner + 2 * G * p.NP;
+  TORCH_CHECK(w.size() == 5 && w[0].dim() == 2 && w[0].size(0) == ch, "ssd: weights conv [channels, taps], bias, dt_bias, A_log, D");
+  p.taps = static_cast<int>(w[0].size(1));
+  TORCH_CHECK(p.taps >= 1 && p.taps <= 32, "ssd: 1..32 taps");
+  p.conv_w = f32(w[0], ch * p.taps, "ssd conv");
+  p.conv_b = f32(w[1], ch, "ssd conv bias");
+  p.dt_bias = f32(w[2], H, "ssd dt_bias");
+  p.A_log = f32(w[3], H, "ssd A_log");
+  p.D = f32(w[4], H, "ssd D");
+  p.conv_state = const_cast<float*>(f32(conv_state, static_cast<int64_t>(p.num_slots) * p.taps * ch, "ssd conv_state"));
+  p.ld = pitch(proj, M, 2 * inner + 2 * G * p.NP + H, "ssd proj");
+  p.proj = proj.data_ptr();
+  p.proj_f32 = dtype_code(proj, "ssd proj");
+  TORCH_CHECK(p.ld % 4 == 0 && reinterpret_cast<uintptr_t>(p.proj) % 16 == 0, "ssd: projection rows in whole 16-byte pieces");
+  TORCH_CHECK(dtype_code(y, "ssd y") == 0 || p.proj_f32 == 1, "ssd: fp32 rows take fp32 projections");
+  p.ldy = pitch(y, M, inner, "ssd y");
+  TORCH_CHECK(p.ldy % 4 == 0, "ssd: row pitch of y");
+  p.y = y.data_ptr();
+  p.status = status_ptr(status);
+  return p;
+}
+
+void ssd_decode(const Tensor& proj, int64_t rows, int64_t H, int64_t G, const std::vector<Tensor>& w, const Tensor& state,
+                const Tensor& conv_state, const Tensor& row_slots, const Tensor& positions, const Tensor& y, const Tensor& status) {
+  oxb::SsdParams p = ssd_common(proj, rows, H, G, w, state, conv_state, y, status);
+  p.row_slots = i32(row_slots, rows, "ssd_decode row_slots");
+  p.positions = i32(positions, rows, "ssd_decode positions");
+  p.rows = static_cast<int>(rows);
+  check_launch(oxb::launch_ssd_decode(p, dtype_code(y, "ssd y"), cur_stream()), "ssd_decode");
+}
+
+void ssd_prefill(const Tensor& proj, int64_t M, int64_t H, int64_t G, const std::vector<Tensor>& w, const Tensor& state,
+                 const Tensor& conv_state, const Tensor& seq_slots, const Tensor& tile_seq, const Tensor& tile_q0, const Tensor& q_start,
+                 const Tensor& q_lens, const Tensor& ctx_lens, int64_t n_tiles, int64_t n_seqs, const Tensor& u, const Tensor& y,
+                 bool runs, const Tensor& status) {
+  oxb::SsdParams p = ssd_common(proj, M, H, G, w, state, conv_state, y, status);
+  const int dt = dtype_code(y, "ssd y");
+  p.seq_slots = i32(seq_slots, n_seqs, "ssd_prefill seq_slots");
+  p.tile_seq = i32(tile_seq, n_tiles, "ssd_prefill tile_seq");
+  p.tile_q0 = i32(tile_q0, n_tiles, "ssd_prefill tile_q0");
+  p.q_start = i32(q_start, n_seqs, "ssd_prefill q_start");
+  p.q_lens = i32(q_lens, n_seqs, "ssd_prefill q_lens");
+  p.ctx_lens = i32(ctx_lens, n_seqs, "ssd_prefill ctx_lens");
+  p.n_tiles = static_cast<int>(n_tiles);
+  p.n_seqs = static_cast<int>(n_seqs);
+  TORCH_CHECK(u.scalar_type() == y.scalar_type() && u.is_cuda(), "ssd_prefill: u of y's type");
+  p.ldu = pitch(u, M, H * p.EP + 2 * G * p.NP, "ssd_prefill u");
+  TORCH_CHECK(p.ldu % 8 == 0 && reinterpret_cast<uintptr_t>(u.data_ptr()) % 16 == 0, "ssd_prefill: u in whole 16-byte pieces");
+  p.u = u.data_ptr();
+  check_launch(oxb::launch_ssd_conv(p, dt, cur_stream()), "ssd_conv");
+  if (runs) {
+    TORCH_CHECK(dt == 0 && oxb::ssd_chunks_ok(p.NP), "ssd_prefill: runs on tensor cores");
+    check_launch(oxb::launch_ssd_chunks(p, cur_stream()), "ssd_prefill");
+  } else {
+    check_launch(oxb::launch_ssd_scan(p, dt, cur_stream()), "ssd_prefill");
+  }
+}
+
+void gated_norm(const Tensor& y, const Tensor& z, int64_t M, int64_t H, int64_t E, int64_t EP, int64_t groups, const Tensor& w, double eps,
+                const Tensor& out) {
+  oxb::GatedNormParams p{};
+  const int dt = dtype_code(y, "gated_norm y");
+  TORCH_CHECK(H >= 1 && E >= 1 && EP >= E && groups >= 1 && (H * E) % groups == 0 && H * E / groups <= 49152, "gated_norm: sizes");
+  TORCH_CHECK(out.scalar_type() == y.scalar_type() && out.is_cuda(), "gated_norm: out of y's type");
+  p.z_f32 = dtype_code(z, "gated_norm z");
+  TORCH_CHECK(dt == 0 || p.z_f32 == 1, "gated_norm: fp32 rows take an fp32 gate");
+  p.ldy = pitch(y, M, H * EP, "gated_norm y");
+  p.ldz = pitch(z, M, H * EP, "gated_norm z");
+  p.ldo = pitch(out, M, H * E, "gated_norm out");
+  auto al = [](const void* x) { return reinterpret_cast<uintptr_t>(x) % 16 == 0; };
+  TORCH_CHECK(al(y.data_ptr()) && al(z.data_ptr()) && al(out.data_ptr()), "gated_norm: rows start on 16 bytes");
+  p.y = y.data_ptr();
+  p.z = z.data_ptr();
+  p.M = static_cast<int>(M);
+  p.H = static_cast<int>(H);
+  p.E = static_cast<int>(E);
+  p.EP = static_cast<int>(EP);
+  p.groups = static_cast<int>(groups);
+  p.w = f32(w, H * E, "gated_norm w");
+  p.eps = static_cast<float>(eps);
+  p.out = out.data_ptr();
+  check_launch(oxb::launch_gated_norm(p, dt, cur_stream()), "gated_norm");
+}
+
+// mode: see MoeRouteParams
+void moe_route(const Tensor& h, const Tensor& router, const OptTensor& logits, int64_t M, int64_t E, int64_t top, const Tensor& weight,
+               const Tensor& expert, const Tensor& slot, int64_t mode, const OptTensor& counts, const OptTensor& xs, const Tensor& status) {
+  oxb::MoeRouteParams p{};
+  const int dt = dtype_code(h, "moe_route h");
+  TORCH_CHECK(E >= 1 && E <= oxb::kMaxExperts && top >= 1 && top <= oxb::kMaxTop && top <= E, "moe_route: at most ", oxb::kMaxExperts,
+              " experts, ", oxb::kMaxTop, " of them chosen");
+  p.N = static_cast<int>(h.size(1));
+  TORCH_CHECK(router.dim() == 2 && router.size(0) >= E && router.size(1) == p.N && router.stride(1) == 1 &&
+                  router.scalar_type() == h.scalar_type() && router.is_cuda() && p.N % 8 == 0 && p.N <= 32768,
+              "moe_route: router [E, N] of h's type");
+  auto al = [](const Tensor& t) { return reinterpret_cast<uintptr_t>(t.data_ptr()) % 16 == 0 && t.stride(0) % 8 == 0; };
+  p.ldh = pitch(h, M, p.N, "moe_route h");
+  p.ldr = router.stride(0);
+  TORCH_CHECK(al(h) && al(router), "moe_route: rows in whole 16-byte pieces");
+  p.h = h.data_ptr();
+  p.router = router.data_ptr();
+  p.M = static_cast<int>(M);
+  p.E = static_cast<int>(E);
+  p.top = static_cast<int>(top);
+  p.mode = static_cast<int>(mode);
+  if (given(logits)) {
+    TORCH_CHECK(logits->is_cuda() && logits->scalar_type() == torch::kFloat32, "moe_route: fp32 logits");
+    p.ldl = pitch(*logits, M, E, "moe_route logits");
+    p.logits = logits->data_ptr<float>();
+  }
+  p.weight = const_cast<float*>(f32(weight, M * top, "moe_route weight"));
+  p.expert = const_cast<int*>(i32(expert, M * top, "moe_route expert"));
+  p.slot = const_cast<int*>(i32(slot, M * top, "moe_route slot"));
+  TORCH_CHECK(mode >= 0 && mode <= 2, "moe_route: mode");
+  if (mode != 0) {
+    TORCH_CHECK(given(counts), "moe_route: counts");
+    p.counts = reinterpret_cast<uint32_t*>(const_cast<int*>(i32(*counts, E, "moe_route counts")));
+  }
+  if (mode == 1) {
+    TORCH_CHECK(M <= 128 && given(xs) && xs->scalar_type() == h.scalar_type() && al(*xs), "moe_route: slabs of 128 rows");
+    p.ldx = pitch(*xs, E * 128, p.N, "moe_route xs");
+    p.xs = xs->data_ptr();
+  }
+  TORCH_CHECK(mode != 2 || given(logits), "moe_route: ranks take given logits");
+  p.status = status_ptr(status);
+  check_launch(oxb::launch_moe_route(p, dt, cur_stream()), "moe_route");
+}
+
+void moe_scatter(const Tensor& h, int64_t M, int64_t E, int64_t top, const Tensor& expert, const Tensor& slot, const Tensor& counts,
+                 const Tensor& xs, const Tensor& status) {
+  oxb::MoeScatterParams p{};
+  TORCH_CHECK(dtype_code(h, "moe_scatter h") == 0 && xs.scalar_type() == h.scalar_type(), "moe_scatter: bf16");
+  TORCH_CHECK(E >= 1 && E <= oxb::kMaxExperts && top >= 1 && top <= oxb::kMaxTop, "moe_scatter: sizes");
+  p.N = static_cast<int>(h.size(1));
+  p.ldh = pitch(h, M, p.N, "moe_scatter h");
+  p.ldx = pitch(xs, 1, p.N, "moe_scatter xs");
+  TORCH_CHECK(p.N % 8 == 0 && p.ldh % 8 == 0 && p.ldx % 8 == 0, "moe_scatter: rows in whole 16-byte pieces");
+  p.h = h.data_ptr();
+  p.M = static_cast<int>(M);
+  p.E = static_cast<int>(E);
+  p.top = static_cast<int>(top);
+  p.expert = i32(expert, M * top, "moe_scatter expert");
+  p.slot = const_cast<int*>(i32(slot, M * top, "moe_scatter slot"));
+  p.counts = reinterpret_cast<const uint32_t*>(i32(counts, E, "moe_scatter counts"));
+  p.xs = xs.data_ptr();
+  p.max_rows = xs.size(0);
+  p.status = status_ptr(status);
+  check_launch(oxb::launch_moe_scatter(p, cur_stream()), "moe_scatter");
+}
+
+void moe_rows(const Tensor& x, const Tensor& w, const Tensor& expert, int64_t pairs, int64_t top, bool per_pair, int64_t act,
+              const Tensor& y) {
+  oxb::MoeRowsParams p{};
+  const int dt = dtype_code(x, "moe_rows x");
+  TORCH_CHECK(w.dim() == 3 && w.is_contiguous() && w.scalar_type() == x.scalar_type() && y.scalar_type() == x.scalar_type() && top >= 1,
+              "moe_rows: w [E, N, K] of x's type");
+  p.E = static_cast<int>(w.size(0));
+  p.N = static_cast<int>(w.size(1));
+  p.K = static_cast<int>(w.size(2));
+  p.ldx = pitch(x, per_pair ? pairs : (pairs + top - 1) / top, p.K, "moe_rows x");
+  TORCH_CHECK(p.K % 8 == 0 && p.ldx % 8 == 0 && reinterpret_cast<uintptr_t>(x.data_ptr()) % 16 == 0, "moe_rows: whole 16-byte pieces");
+  p.ldy = pitch(y, pairs, p.N, "moe_rows y");
+  p.x = x.data_ptr();
+  p.w = w.data_ptr();
+  p.y = y.data_ptr();
+  p.pairs = static_cast<int>(pairs);
+  p.top = static_cast<int>(top);
+  p.per_pair = per_pair ? 1 : 0;
+  p.expert = i32(expert, pairs, "moe_rows expert");
+  TORCH_CHECK(act == 0 || act == 2, "moe_rows: act 0 or 2");
+  p.act = static_cast<int>(act);
+  check_launch(oxb::launch_moe_rows(p, dt, cur_stream()), "moe_rows");
+}
+
 void gemm_f32(const Tensor& a, const Tensor& w, const Tensor& out) {
   TORCH_CHECK(a.is_cuda() && w.is_cuda() && out.is_cuda() && a.scalar_type() == torch::kFloat32 &&
                   w.scalar_type() == torch::kFloat32 && out.scalar_type() == torch::kFloat32 && a.dim() == 2 && w.dim() == 2 &&
@@ -330,6 +593,16 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("retention_decode", &retention_decode);
   m.def("retention_prefill", &retention_prefill);
   m.def("retention_chunks_ok", [](int64_t D, int64_t E) { return oxb::retention_chunks_ok((int)D, (int)E); });
+  m.attr("MAX_EXPERTS") = oxb::kMaxExperts;
+  m.attr("MAX_TOP") = oxb::kMaxTop;
+  m.def("branch_norm", &branch_norm);
+  m.def("ssd_decode", &ssd_decode);
+  m.def("ssd_prefill", &ssd_prefill);
+  m.def("ssd_chunks_ok", [](int64_t NP) { return oxb::ssd_chunks_ok(static_cast<int>(NP)); });
+  m.def("gated_norm", &gated_norm);
+  m.def("moe_route", &moe_route);
+  m.def("moe_scatter", &moe_scatter);
+  m.def("moe_rows", &moe_rows);
   m.def("gemm_f32", &gemm_f32);
   m.def("glu_f32", &glu_f32);
 }

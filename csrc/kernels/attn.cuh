@@ -4,6 +4,7 @@
 #include <cuda.h>
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
+#include <math.h>
 #include <stdint.h>
 
 namespace oxb {
@@ -24,7 +25,10 @@ struct DecodeAttnParams {
   int keep_first;    // with a window: the first positions stay visible too (0: none); they keep their true positions
   int out_d;         // values stored per head in `out` (<= D; 0: D). The caches and q are padded to D
   int exact_p;       // 1: softmax weights enter the value product as two bf16 terms (about 16 bits) instead of one
+  int chunk;         // > 0: only positions of the query's own chunk are visible (chunks count from position 0)
   float scale_log2;  // softmax scale * log2(e)
+  // score (times log2(e)) of a sink: one more term of the softmax denominator, without a value
+  float sink_log2 = -INFINITY;
   // Bounds check of block-table entries: an id outside [0, num_blocks) is recorded in *status
   // (kStatusBadIndex) and page 0 is read instead. num_blocks <= 0 or status == nullptr: no check.
   int num_blocks;
@@ -63,8 +67,9 @@ struct PrefillAttnParams {
   __nv_bfloat16* out;       // [T, Hq*D], row stride out_stride
   long long out_stride;
   int max_blocks, Hq, Hkv, window;
-  int keep_first, out_d, exact_p;  // as in DecodeAttnParams
+  int keep_first, out_d, exact_p, chunk;  // as in DecodeAttnParams
   float scale_log2;
+  float sink_log2 = -INFINITY;
   int num_blocks;  // bound for block-table entries (<= 0: unchecked), violations go to *status
   int* status;
 };

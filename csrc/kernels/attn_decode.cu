@@ -81,6 +81,12 @@ __device__ __forceinline__ float ex2(float x) {
   return y;
 }
 
+// First visible position of the last of `seq_len` tokens (kept first positions aside): its window's or its chunk's.
+__device__ __forceinline__ int visible_from(const DecodeAttnParams& p, int seq_len) {
+  if (p.chunk > 0) return seq_len > 0 ? (seq_len - 1) / p.chunk * p.chunk : 0;
+  return (p.window > 0 && seq_len > p.window) ? seq_len - p.window : 0;
+}
+
 // D = head dim (64 or 128); NT = number of 8-head column tiles (group size <= 8*NT).
 // MASS: also record the per-page softmax statistics of every head (see DecodeAttnParams::page_ml).
 // EXACT: the softmax weights enter the value product as hi + lo bf16 terms (DecodeAttnParams::exact_p).
@@ -103,7 +109,7 @@ paged_decode_kernel(const DecodeAttnParams p) {
   const int G = p.Hq / p.Hkv;
 
   const int seq_len = p.seq_lens[seq];
-  const int win_start = (p.window > 0 && seq_len > p.window) ? seq_len - p.window : 0;
+  const int win_start = visible_from(p, seq_len);
   int n_pages = (seq_len + kPage - 1) / kPage;
   if (n_pages > p.max_blocks) {
     // a length beyond the block-table row: recorded, and the walk stops at the end of the row
@@ -121,7 +127,7 @@ paged_decode_kernel(const DecodeAttnParams p) {
   }
   const int skip = first_page - n_first;
   const int n_list = n_pages - skip;
-  if (p.window > 0 && skip > 0) {
+  if (skip > 0) {
     // the host sized the splits for the whole context: spread the visible pages over as many splits
     const int used = (n_pages + pps - 1) / pps;
     pps = ((n_list + used - 1) / used + kWarps - 1) / kWarps * kWarps;
@@ -414,7 +420,8 @@ paged_decode_kernel(const DecodeAttnParams p) {
   }
 }
 
-// out[seq, head, :] = sum_s w_s O_s / sum_s w_s l_s  with  w_s = 2^(m_s - max m)
+// out[seq, head, :] = sum_s w_s O_s / (sum_s w_s l_s + sink)  with  w_s = 2^(m_s - max m); the sink is one more term of
+// the denominator and of the maximum
 template <int D>
 __global__ void __launch_bounds__(D) decode_merge_kernel(const DecodeAttnParams p) {
   pdl_launch_dependents();
@@ -423,9 +430,9 @@ __global__ void __launch_bounds__(D) decode_merge_kernel(const DecodeAttnParams 
   const int head = blockIdx.y;
   const int d = threadIdx.x;
   const long long base = (static_cast<long long>(seq) * p.Hq + head) * p.max_splits;
-  float M = -INFINITY;
+  float M = p.sink_log2;
   for (int s = 0; s < p.max_splits; ++s) M = fmaxf(M, p.part_ml[(base + s) * 2]);
-  float acc = 0.f, L = 0.f;
+  float acc = 0.f, L = p.sink_log2 == -INFINITY ? 0.f : ex2(p.sink_log2 - M);
   for (int s = 0; s < p.max_splits; ++s) {
     const float ms = p.part_ml[(base + s) * 2];
     if (ms == -INFINITY) continue;
@@ -466,10 +473,10 @@ __global__ void __launch_bounds__(128) block_mass_kernel(const DecodeAttnParams 
   const int seq_len = p.seq_lens[seq];
   int n_pages = (seq_len + kPage - 1) / kPage;
   if (n_pages > p.max_blocks) n_pages = p.max_blocks;
-  const int win_start = (p.window > 0 && seq_len > p.window) ? seq_len - p.window : 0;
+  const int win_start = visible_from(p, seq_len);
   const int first_page = win_start / kPage;
   // (with a window the splits are respread inside the kernel and cover all of it)
-  int last_page = p.window > 0 ? n_pages : first_page + *p.pages_per_split * p.max_splits;  // pages past the last split were not walked
+  int last_page = p.window > 0 || p.chunk > 0 ? n_pages : first_page + *p.pages_per_split * p.max_splits;  // pages past the last split were not walked
   if (last_page > n_pages) last_page = n_pages;
   for (int h = threadIdx.x; h < p.Hq; h += blockDim.x) {
     const long long base = (static_cast<long long>(seq) * p.Hq + h) * p.max_splits;

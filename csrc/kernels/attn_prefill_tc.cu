@@ -9,8 +9,8 @@
 //                         memory in the swizzled K-major layout the next MMA expects
 //     O += P V            tcgen05.mma with V as an MN-major operand, accumulator in TMEM
 // The running maximum is updated lazily (O is rescaled in TMEM only when a row's maximum grows by
-// more than 2^8), causal / sliding-window masks are applied from absolute positions, and the
-// tiles above the diagonal are skipped. Warp roles: warp 0 = TMA producer, warp 1 = MMA issuer,
+// more than 2^8), causal / sliding-window / chunk masks are applied from absolute positions, and the
+// tiles above the diagonal or before the window are skipped. Warp roles: warp 0 = TMA producer, warp 1 = MMA issuer,
 // warps 2..5 = softmax + epilogue. Every wait is bounded.
 //
 // Replaces flash_causal_batched_prefill_kernel
@@ -92,11 +92,13 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
   int last_row = q0 + BQ - 1;
   if (last_row > q_len - 1) last_row = q_len - 1;
   const int max_pos = pos_off + last_row;
-  int first_tile = 0;
-  if (p.window > 0) {
-    const int lo = pos_off + q0 - p.window + 1;
-    if (lo > 0) first_tile = lo / BKV;
-  }
+  // first position that a query at `pos` sees (kept first positions aside): its window's or its chunk's
+  auto visible_from = [&](int pos) -> int {
+    if (p.chunk > 0) return pos / p.chunk * p.chunk;
+    return p.window > 0 ? pos - p.window + 1 : 0;
+  };
+  int first_tile = visible_from(pos_off + q0) / BKV;
+  if (first_tile < 0) first_tile = 0;
   // KV tiles that hold kept first positions and lie before the window come first, then the window's:
   // list entry j is tile j + (j < n_first ? 0 : skip)
   int n_first = 0;
@@ -241,6 +243,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     const int qi = q0 + r;
     const bool row_valid = qi < q_len;
     const int pos = pos_off + (row_valid ? qi : q_len - 1);
+    const int lo = visible_from(pos);
     const uint32_t lane_sel = static_cast<uint32_t>(q * 32) << 16;
     float m_used = -INFINITY, l_sum = 0.f;
     bool ok = true;
@@ -262,7 +265,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           const int t = t0 + c * 32 + i;
-          const bool keep = t <= pos && (p.window <= 0 || t > pos - p.window || t < p.keep_first);
+          const bool keep = t <= pos && (t >= lo || t < p.keep_first);
           if (keep) mx = fmaxf(mx, __uint_as_float(v[i]));
         }
       }
@@ -306,7 +309,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           const int t = t0 + c * 32 + i;
-          const bool keep = t <= pos && (p.window <= 0 || t > pos - p.window || t < p.keep_first);
+          const bool keep = t <= pos && (t >= lo || t < p.keep_first);
           pv[i] = keep ? ex2a(__uint_as_float(v[i]) * p.scale_log2 - m_sub) : 0.f;
           l_sum += pv[i];
         }
@@ -349,6 +352,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     if (!ok && lane == 0) set_status_once(status, kStatusMbarTimeoutEpilogue);
     if (ok && n_tiles > 0) {
       tc_fence_after_sync();
+      if (p.sink_log2 != -INFINITY) l_sum += ex2a(p.sink_log2 - m_used);
       const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
       const int od = p.out_d > 0 ? p.out_d : D;  // values stored per head
       const bool out_vec = (od & 7) == 0 && (p.out_stride & 7) == 0;

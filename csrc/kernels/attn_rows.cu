@@ -1,5 +1,5 @@
 // Softmax attention of single query rows over the paged cache, in fp32 FMAs: any head sizes, fp32 or bf16
-// storage, sliding window with kept first positions. One CTA per (row, query head) walks the visible keys
+// storage, sliding window with kept first positions or chunks, optional sink. One CTA per (row, query head) walks the visible keys
 // 128 at a time: thread = key for the scores, thread = value dimension for the sums. The 32-bit path and
 // head sizes beyond the tensor-core kernels use it; it is not tuned for throughput.
 #include "../common/device_info.h"
@@ -37,10 +37,10 @@ __global__ void __launch_bounds__(kKeys) row_attention_kernel(const RowAttnParam
   for (int d = threadIdx.x; d < p.D; d += kKeys) s_q[d] = to_f(qp[d]);
   const int kvh = head / (p.H / p.G);
   // visible keys: [0, n_first) and [lo, pos]
-  const int lo = (p.window > 0 && pos + 1 > p.window) ? pos + 1 - p.window : 0;
+  const int lo = p.chunk > 0 ? pos / p.chunk * p.chunk : ((p.window > 0 && pos + 1 > p.window) ? pos + 1 - p.window : 0);
   const int n_first = min(p.keep_first, lo);
   const int n_vis = n_first + (pos + 1 - lo);
-  float m_run = -INFINITY, l_run = 0.f, acc[kMaxV];
+  float m_run = p.sink, l_run = p.sink == -INFINITY ? 0.f : 1.f, acc[kMaxV];
 #pragma unroll
   for (int i = 0; i < kMaxV; ++i) acc[i] = 0.f;
   __syncthreads();

@@ -33,7 +33,8 @@
 //  * Dense weights may be stored tile-major ([N/128][K/64][128][64]) so that each TMA box of the
 //    weight stream is one contiguous 16 KB run of HBM instead of 128 row segments 2K bytes apart.
 //  * Grouped mode walks a device-side table of per-expert row counts, so the grid is static
-//    (CUDA-graph friendly) while the work is data dependent.
+//    (CUDA-graph friendly) while the work is data dependent. Expert rows lie in slabs of one height, or
+//    packed one expert after the other in whole 128-row tiles.
 //
 // Replaces the reference's cuBLAS prefill path (cublas_ops.cu:242-260), the `*_fused_add`
 // output projections (launch_wrappers.cu:202-247) and the host-loop grouped expert GEMM
@@ -256,7 +257,9 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
   uint64_t* fix_bar = tmem_empty + 2;    // landing of the partial slabs in the split-K fix-up
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(fix_bar + 1);
   int* s_misc = reinterpret_cast<int*>(tmem_slot + 2);  // [0] start-up ok, [1] tile barrier ok
-  int* s_counts = s_misc + 2;                           // first m tile per group, grouped mode
+  // grouped mode: first m tile of every group (and the end of the last), then rows of every group
+  int* s_counts = reinterpret_cast<int*>(smem + L::kBarOffset + 512);
+  int* s_rows = s_counts + p.n_groups + 1;
 
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
@@ -294,20 +297,36 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
     mbar_init(&tmem_empty[1], 4);
     mbar_init(fix_bar, 1);
     fence_mbar_init();
-    int ok = 1;
-    if (grouped) {
-      pdl_wait();
-      // The per-group row counts are final only once every source has finished dispatching.
-      if (p.ag_flags != nullptr) ok = wait_sources(p, 0, p.ag_n_src - 1, gridDim.x) ? 1 : 0;
-      int acc = 0;
-      for (int e = 0; e < p.n_groups; ++e) {
-        s_counts[e] = acc;  // first m tile of group e
-        acc += (static_cast<int>(__ldcg(p.group_counts + e)) + BM - 1) / BM;
-      }
-      s_counts[p.n_groups] = acc;
-    }
-    s_misc[0] = ok;
+    if (!grouped) s_misc[0] = 1;
     s_misc[1] = 1;
+  }
+  if (grouped && warp == 1) {
+    pdl_wait();
+    // The per-group row counts are final only once every source has finished dispatching.
+    int ok = 1;
+    if (p.ag_flags != nullptr && lane == 0) ok = wait_sources(p, 0, p.ag_n_src - 1, gridDim.x) ? 1 : 0;
+    ok = __shfl_sync(0xffffffffu, ok, 0);
+    int acc = 0;
+    for (int e0 = 0; e0 < p.n_groups; e0 += 32) {
+      const int e = e0 + lane;
+      const int rows = e < p.n_groups ? static_cast<int>(__ldcg(p.group_counts + e)) : 0;
+      const int tiles = (rows + BM - 1) / BM;
+      int incl = tiles;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int up = __shfl_up_sync(0xffffffffu, incl, o);
+        if (lane >= o) incl += up;
+      }
+      if (e < p.n_groups) {
+        s_counts[e] = acc + incl - tiles;
+        s_rows[e] = rows;
+      }
+      acc += __shfl_sync(0xffffffffu, incl, 31);
+    }
+    if (lane == 0) {
+      s_counts[p.n_groups] = acc;
+      s_misc[0] = ok;
+    }
   }
   __syncthreads();  // barriers, start-up state
   // The producer warp goes ahead (its first weight tiles depend on no earlier kernel). The other
@@ -345,14 +364,21 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
     it.valid = all_ok && it.nkb > 0;
     if (grouped) {
       it.valid = false;
-      for (int e = 0; e < p.n_groups; ++e) {
-        if (mt >= s_counts[e] && mt < s_counts[e + 1]) {
-          it.group = e;
-          it.m0 = (mt - s_counts[e]) * BM;
-          it.rows = static_cast<int>(__ldcg(p.group_counts + e));
-          it.valid = all_ok && it.nkb > 0;
-          break;
+      if (mt < s_counts[p.n_groups]) {
+        int lo = 0, hi = p.n_groups;  // the last group that starts at or before this tile (empty groups are passed over)
+        while (hi - lo > 1) {
+          const int mid = (lo + hi) >> 1;
+          if (s_counts[mid] <= mt) lo = mid;
+          else hi = mid;
         }
+        it.group = lo;
+        it.m0 = (mt - s_counts[lo]) * BM;
+        it.rows = s_rows[lo];
+        if (p.packed_rows) {  // rows and the bound count from the start of the packed buffer
+          it.m0 += s_counts[lo] * BM;
+          it.rows += s_counts[lo] * BM;
+        }
+        it.valid = all_ok && it.nkb > 0;
       }
     }
     return it;
@@ -383,10 +409,10 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
                   L::kSFABytes, &full[s]);
       // rows past M read as zeros (the box is filled in full either way)
       if (p.wide_boxes && MT == 2) {
-        if (op == 2) tma_load_3d(sA + s * L::kABytes, &tmA, &full[s], (it.kb0 + kb) * kXStep, it.m0, it.group);
+        if (op == 2) tma_load_3d(sA + s * L::kABytes, &tmA, &full[s], (it.kb0 + kb) * kXStep, it.m0, 0);
       } else if (op >= 2 && op < 2 + MT)
         tma_load_3d(sA + s * L::kABytes + (op - 2) * (BM * BK * 2), &tmA, &full[s], (it.kb0 + kb) * kXStep,
-                    it.m0 + (op - 2) * BM, it.group);
+                    it.m0 + (op - 2) * BM, p.packed_rows ? 0 : it.group);
     };
     for (int w = blockIdx.x; w < n_work && ok; w += gridDim.x) {
       const WorkItem it = decode(w);
@@ -832,6 +858,13 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
               for (int j = 0; j < 64; ++j)
                 if (col0 + j < p.N) a[j] += __bfloat162float(bias[col0 + j]);
             }
+            if (p.act == 2 && p.epi == kEpiStoreBf16) {
+#pragma unroll
+              for (int j = 0; j < 64; ++j) {
+                const float r = fmaxf(a[j], 0.f);
+                a[j] = r * r;
+              }
+            }
 #pragma unroll
             for (int j = 0; j < 64; j += 8) {
               uint4 o4;
@@ -933,13 +966,14 @@ void launch_impl(const CUtensorMap& tmA, const CUtensorMap& tmB, const GemmParam
                  cudaStream_t stream) {
   using L = SmemLayout<BN, STAGES, MT, KIND>;
   auto kern = gemm_bf16_kernel<BN, STAGES, MT, KIND>;
-  ensure_dynamic_smem(kern, L::kTotal);
+  const size_t smem = L::kTotal + (p.group_counts != nullptr ? (2 * static_cast<size_t>(p.n_groups) + 1) * sizeof(int) : 0);
+  ensure_dynamic_smem(kern, smem);
   const int sms = sm_count();
   const int n_work = ((p.N + BN - 1) / BN) * p.m_tiles * p.splits;
   const int grid = n_work < sms ? n_work : sms;
   // the splits of a tile wait for each other: ask for a launch that is resident as a whole
   const bool cooperative = p.ws != nullptr && p.splits > 1;
-  launch_kernel(kern, dim3(grid), dim3(KIND == 2 ? kThreads + 32 * kDequantWarps : kThreads), L::kTotal, stream,
+  launch_kernel(kern, dim3(grid), dim3(KIND == 2 ? kThreads + 32 * kDequantWarps : kThreads), smem, stream,
                 /*pdl=*/true, cooperative, tmA, tmB, p);
 }
 

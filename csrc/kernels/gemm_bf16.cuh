@@ -33,7 +33,7 @@ struct GemmParams {
   int splits;         // number of K slices
   int m_tiles;        // M tiles of 128 * mt rows (grouped mode: upper bound over all groups, mt = 1)
   int epi;
-  int act;            // kEpiSwigluBf16: 0 = SiLU, 1 = tanh-GELU
+  int act;            // kEpiSwigluBf16: 0 = SiLU, 1 = tanh-GELU; kEpiStoreBf16: 2 = squared ReLU, else none
   int wide_boxes;     // 1: one TMA copy per operand and stage (A box of 256 rows; tile-major B through a
                       //    4-D map that spans both 128-row weight tiles of a 256-wide tile)
   int b_tiled;        // 1: B is stored tile-major [N/128][K/64][128][64]: every TMA box is one contiguous 16 KB
@@ -44,6 +44,8 @@ struct GemmParams {
   // --- grouped (MoE) mode ---
   const uint32_t* group_counts;  // [n_groups] rows used in each group (device); nullptr = dense
   int n_groups;
+  int packed_rows;    // 1: A and C are [rows, ..] with the groups one after the other, each from a multiple of 128 on
+                      // (instead of one slab of the same height per group)
   const RowMeta* row_meta;       // [n_groups, meta_group_stride] routing of each slab row
   long long meta_group_stride;
   // --- routed fp32 reduction (split-K on one GPU; reduce-scatter / combine across GPUs) ---

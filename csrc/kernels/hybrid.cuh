@@ -45,6 +45,47 @@ struct StreamNormParams {
 };
 cudaError_t launch_stream_norm(const StreamNormParams& p, int dtype, cudaStream_t stream);
 
+// What stands between two layers whose mixer and feed-forward run side by side on one residual stream x. With N
+// values per row:
+//   tokens given : x = embed[token] * embed_scale
+//   else         : x += sum_b gain[b] * (w[b] ? y_b / sqrt(mean(y_b^2) + eps) * w[b] : y_b)   (dense branches)
+//                     + sum_c weight[c] * expert_rows[slot[c]]                                (chosen experts)
+//   then         : h_o = x / sqrt(mean(x^2) + eps) * (w_offset + norm_w[o])                   for every output o
+// x is written back when store_x is set. Where clear_y is set for a branch, its rows are zeroed on the way (the
+// split-K GEMM of the layer that follows adds into them).
+constexpr int kMaxBranches = 2;
+struct BranchNormParams {
+  float* x;                 // [rows, N]
+  int rows, N;
+  const int* tokens;        // [rows] or nullptr
+  const void* embed;        // [vocab, N]
+  int vocab;
+  float embed_scale;
+  int n_branches;
+  float* y[kMaxBranches];   // [rows, ldy]
+  const float* w[kMaxBranches];
+  float gain[kMaxBranches];
+  int clear_y[kMaxBranches];
+  long long ldy;
+  const void* e_rows;       // expert outputs [n_e_rows, lde] or nullptr
+  long long lde, n_e_rows;
+  const int* e_slot;        // [rows, top], < 0: nothing
+  const float* e_weight;    // [rows, top]
+  int top;
+  int store_x;
+  int n_out;
+  const float* norm_w[2];
+  void* h[2];
+  float eps, w_offset;
+  long long ldh;
+  const int* row_map;       // destination row of h, < 0: skipped
+  float* clear;             // [rows, clear_ld] or nullptr, zeroed as in StreamNormParams
+  long long clear_ld;
+  int clear_n;
+  int* status;
+};
+cudaError_t launch_branch_norm(const BranchNormParams& p, int dtype, cudaStream_t stream);
+
 // Rotary positions: pair i turns by position * (freq_hi[i] + freq_lo[i]) (the frequency as an unevaluated
 // sum of two floats, so the angle is good to the last bits of a 32-bit float at any position).
 struct RotaryParams {
@@ -52,6 +93,7 @@ struct RotaryParams {
   const float* freq_lo;
   int dims;                 // 0: no rotation
   int interleaved;          // pairs (2i, 2i+1), else (i, i + dims/2)
+  float gain;               // factor on sin and cos
 };
 
 // Projection rows q | k | v -> per-head vectors: optional RMS norm over the whole q (k) projection with
@@ -100,7 +142,9 @@ struct RowAttnParams {
   int max_blocks, num_blocks;
   int H, G, D, E, DP, EP;
   int window, keep_first;
+  int chunk;                // > 0: only positions of the query's own chunk (counted from position 0) are visible
   float scale;
+  float sink;               // score of one more term of the softmax denominator, without a value (-inf: none)
   void* out;                // [rows, ldo], head stride E
   long long ldo;
   int* status;
@@ -147,6 +191,119 @@ cudaError_t launch_retention_chunks(const RetentionParams& p, cudaStream_t strea
 // Prompt chunks token by token in plain fp32 (the fp32 path, and head sizes above the chunked form's).
 cudaError_t launch_retention_scan(const RetentionParams& p, int dtype, cudaStream_t stream);
 bool retention_chunks_ok(int D, int E);
+
+// State-space layer with a scalar decay per head and step (Mamba-2). Head h uses group g = h / (H / G):
+//   u    = silu(conv(xbc) + bias)              per channel, causal, `taps` taps (the last one: the current token)
+//   dt   = softplus(dt_in + dt_bias[h])
+//   S_t  = exp(-exp(A_log[h]) dt_t) S_{t-1} + dt_t B_t x_t^T,   y_t = S_t^T C_t + D[h] x_t     (S: [NP, EP])
+// A projection row holds z (H * EP) | x (H * EP) | B (G * NP) | C (G * NP) | dt (H); head sizes E and state sizes N
+// are padded with zero channels to EP and NP, multiples of 16. conv_state keeps the inputs of the last `taps` tokens
+// of a sequence by position modulo taps, so a decode step never overwrites an input that the step still reads.
+struct SsdParams {
+  const void* proj;         // [M, ld], first column z
+  int proj_f32;
+  long long ld;
+  int H, G, EP, NP, taps;
+  const float* conv_w;      // [channels, taps], channels = H * EP + 2 * G * NP
+  const float* conv_b;      // [channels]
+  const float* dt_bias;     // [H]
+  const float* A_log;       // [H]
+  const float* D;           // [H]
+  float* state;             // [slots, H, NP, EP]
+  float* conv_state;        // [slots, taps, channels]
+  int num_slots;
+  // decode rows
+  const int* row_slots;     // [rows], < 0: padding row
+  const int* positions;     // [rows]; a row at position 0 starts from the zero state
+  int rows;
+  // prompt chunks
+  const int* seq_slots;     // [sequences]
+  const int* tile_seq;      // 128-row tiles
+  const int* tile_q0;
+  const int* q_start;
+  const int* q_lens;
+  const int* ctx_lens;
+  int n_tiles, n_seqs;
+  void* u;                  // [M, ldu] convolved channels (x | B | C)
+  long long ldu;
+  void* y;                  // [M, ldy]: H * EP
+  long long ldy;
+  int* status;
+};
+// One token per row: convolution, state update and read-out in one launch.
+cudaError_t launch_ssd_decode(const SsdParams& p, int dtype, cudaStream_t stream);
+// Prompt chunks: convolution of all rows (and the convolution's state).
+cudaError_t launch_ssd_conv(const SsdParams& p, int dtype, cudaStream_t stream);
+// Prompt chunks, bf16: runs of 64 tokens on tensor cores, fp32 operands split into three bf16 terms.
+cudaError_t launch_ssd_chunks(const SsdParams& p, cudaStream_t stream);
+// Prompt chunks token by token in fp32 FMAs.
+cudaError_t launch_ssd_scan(const SsdParams& p, int dtype, cudaStream_t stream);
+bool ssd_chunks_ok(int NP);
+
+// out[row] = rms_groups(y * silu(z)) * w: `groups` equal parts of H * E values, each by its own root mean square.
+// y and z hold heads of E values EP apart.
+struct GatedNormParams {
+  const void* y;            // [M, ldy], storage type
+  long long ldy;
+  const void* z;            // [M, ldz], storage type or fp32 when z_f32 is set
+  int z_f32;
+  long long ldz;
+  int M, H, E, EP, groups;
+  const float* w;           // [H * E]
+  float eps;
+  void* out;                // [M, ldo]
+  long long ldo;
+};
+cudaError_t launch_gated_norm(const GatedNormParams& p, int dtype, cudaStream_t stream);
+
+// Router of a mixture of experts: softmax over all experts, the `top` largest scores divided by their sum (+ 1e-20).
+constexpr int kMaxExperts = 512;
+constexpr int kMaxTop = 32;
+struct MoeRouteParams {
+  const float* logits;      // [M, ldl], or nullptr: computed here from h and router
+  long long ldl;
+  const void* h;            // [M, ldh]
+  long long ldh;
+  const void* router;       // [E, ldr]
+  long long ldr;
+  int M, N, E, top;
+  float* weight;            // [M, top]
+  int* expert;              // [M, top]
+  int* slot;                // [M, top]: row of the expert buffers that belongs to the choice
+  int mode;                 // 0: slot = its own index; 1: rows of 128-row slabs per expert, h copied there (M <= 128);
+                            // 2: slot = rank inside the expert (launch_moe_scatter turns it into a packed row)
+  uint32_t* counts;         // [E] rows per expert, zero before the launch (modes 1 and 2)
+  void* xs;                 // [E * 128, ldx] (mode 1)
+  long long ldx;
+  int* status;
+};
+cudaError_t launch_moe_route(const MoeRouteParams& p, int dtype, cudaStream_t stream);
+// slot[i] += first packed row of the expert (whole 128-row tiles per expert); h rows are copied there.
+struct MoeScatterParams {
+  const void* h;
+  long long ldh;
+  int M, N, E, top;
+  const int* expert;
+  int* slot;
+  const uint32_t* counts;
+  void* xs;                 // [max_rows, ldx]
+  long long ldx, max_rows;
+  int* status;
+};
+cudaError_t launch_moe_scatter(const MoeScatterParams& p, cudaStream_t stream);   // bf16
+// y[p] = act(W[expert[p]] x[per_pair ? p : p / top]) for every (row, choice) pair p. act 0: none, 2: squared ReLU.
+struct MoeRowsParams {
+  const void* x;
+  long long ldx;
+  int per_pair;
+  const void* w;            // [E, N, K]
+  int pairs, top, E, N, K;
+  const int* expert;        // [pairs]
+  int act;
+  void* y;                  // [pairs, ldy]
+  long long ldy;
+};
+cudaError_t launch_moe_rows(const MoeRowsParams& p, int dtype, cudaStream_t stream);
 
 // out[M, N] = a[M, K] w[N, K]^T in fp32 FMAs.
 cudaError_t launch_gemm_f32(const float* a, long long lda, const float* w, long long ldw, float* out, long long ldo,

@@ -70,8 +70,8 @@ __device__ __forceinline__ void rotary_sincos(const RotaryParams& r, int i, int 
   const float e = fmaf(x, r.freq_hi[i], -a) + x * r.freq_lo[i];
   float s, c;
   sincosf(a, &s, &c);
-  *sn = fmaf(e, fmaf(-0.5f * e, s, c), s);   // second-order turn: e reaches 1/100 at angles of 2^18
-  *cs = fmaf(-e, fmaf(0.5f * e, c, s), c);
+  *sn = r.gain * fmaf(e, fmaf(-0.5f * e, s, c), s);   // second-order turn: e reaches 1/100 at angles of 2^18
+  *cs = r.gain * fmaf(-e, fmaf(0.5f * e, c, s), c);
 }
 __device__ __forceinline__ void rotary_pair(const RotaryParams& r, int i, int* u, int* v) {
   *u = r.interleaved ? 2 * i : i;

@@ -1,7 +1,9 @@
 // Residual streams between the sublayers of a layer-list decoder (sm_100a): the hyper-connection update of
 // the sublayer that just ran, the read-out for the next one and its RMS norm in one pass over the row,
 // with the embedding gather (and its hashed bigram row) folded into the first of them. Streams stay fp32.
-// With one stream, mix = in = out = 1 it is residual-add + RMSNorm.
+// With one stream, mix = in = out = 1 it is residual-add + RMSNorm. `branch_norm` is its counterpart for layers whose
+// mixer and feed-forward run side by side: the branches of the layer that just ran, each by its own norm, the weighted
+// rows of the chosen experts, and the norms of the next layer's mixer and feed-forward in one pass.
 #include "../common/device_info.h"
 #include "hybrid_dev.cuh"
 
@@ -180,7 +182,252 @@ cudaError_t launch_t(const StreamNormParams& p, cudaStream_t stream) {
   return launch_s<T, kMaxStreams>(p, stream);
 }
 
+// Layers whose mixer and feed-forward run side by side: V values per piece, CH pieces per thread that stay in
+// registers (CH = 0: any row length, the row goes through shared memory).
+template <typename T>
+__device__ __forceinline__ float4 expert_sum4(const BranchNormParams& p, int row, int c) {
+  float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int k = 0; k < p.top; ++k) {
+    const int s = p.e_slot[row * p.top + k];
+    if (s < 0 || s >= p.n_e_rows) continue;
+    const float wk = p.e_weight[row * p.top + k];
+    float v[4];
+    load4<T>(static_cast<const T*>(p.e_rows) + static_cast<long long>(s) * p.lde + c, v);
+    a.x = fmaf(wk, v[0], a.x);
+    a.y = fmaf(wk, v[1], a.y);
+    a.z = fmaf(wk, v[2], a.z);
+    a.w = fmaf(wk, v[3], a.w);
+  }
+  return a;
+}
+template <typename T>
+__device__ __forceinline__ float expert_sum(const BranchNormParams& p, int row, int c) {
+  float a = 0.f;
+  for (int k = 0; k < p.top; ++k) {
+    const int s = p.e_slot[row * p.top + k];
+    if (s < 0 || s >= p.n_e_rows) continue;
+    a = fmaf(p.e_weight[row * p.top + k], to_f(static_cast<const T*>(p.e_rows)[static_cast<long long>(s) * p.lde + c]), a);
+  }
+  return a;
+}
+// sums of both branches at once over the block
+__device__ __forceinline__ float2 block_sum2(float2 v, float2* scratch) {
+  v.x = warp_sum(v.x);
+  v.y = warp_sum(v.y);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  __syncthreads();
+  if (lane == 0) scratch[warp] = v;
+  __syncthreads();
+  const int nw = (blockDim.x + 31) >> 5;
+  const float2 s = lane < nw ? scratch[lane] : make_float2(0.f, 0.f);
+  return make_float2(warp_sum(s.x), warp_sum(s.y));
+}
+
+template <typename T, int CH>
+__global__ void __launch_bounds__(CH == 4 ? 512 : 1024) branch_norm_kernel(const BranchNormParams p) {
+  __shared__ float s_red[32];
+  __shared__ float2 s_red2[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int N = p.N;
+  const float inv_n = 1.f / static_cast<float>(N);
+  for (int row = blockIdx.x; row < p.rows; row += gridDim.x) {
+    float* xr = p.x + static_cast<long long>(row) * N;
+    if (p.clear != nullptr) {
+      float* z = p.clear + static_cast<long long>(row) * p.clear_ld;
+      for (int c = threadIdx.x * 4; c < p.clear_n; c += blockDim.x * 4)
+        *reinterpret_cast<float4*>(z + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    const int dst = p.row_map != nullptr ? p.row_map[row] : row;
+    float x[CH][4];
+    if (p.tokens != nullptr) {
+      const int tok = p.tokens[row];
+      const bool ok = tok >= 0 && tok < p.vocab;
+      if (!ok && threadIdx.x == 0) set_status_once(p.status, kStatusBadIndex);
+      const T* er = static_cast<const T*>(p.embed) + static_cast<long long>(ok ? tok : 0) * N;
+#pragma unroll
+      for (int k = 0; k < CH; ++k) {
+        const int c = (k * blockDim.x + threadIdx.x) * 4;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) x[k][j] = 0.f;
+        if (c < N) {
+          load4<T>(er + c, x[k]);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) x[k][j] *= p.embed_scale;
+        }
+      }
+      for (int b = 0; b < kMaxBranches; ++b)
+        if (b < p.n_branches && p.clear_y[b])
+          for (int c = threadIdx.x * 4; c < N; c += blockDim.x * 4)
+            *reinterpret_cast<float4*>(p.y[b] + static_cast<long long>(row) * p.ldy + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+    } else {
+      float y[kMaxBranches][CH][4];
+      float ss[kMaxBranches] = {};
+#pragma unroll
+      for (int k = 0; k < CH; ++k) {
+        const int c = (k * blockDim.x + threadIdx.x) * 4;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) x[k][j] = 0.f;
+        if (c < N) load4<float>(xr + c, x[k]);
+#pragma unroll
+        for (int b = 0; b < kMaxBranches; ++b) {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) y[b][k][j] = 0.f;
+          if (b < p.n_branches && c < N) {
+            load4<float>(p.y[b] + static_cast<long long>(row) * p.ldy + c, y[b][k]);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) ss[b] = fmaf(y[b][k][j], y[b][k][j], ss[b]);
+          }
+        }
+      }
+      const float2 tot = block_sum2(make_float2(ss[0], ss[1]), s_red2);
+      const float r[kMaxBranches] = {1.f / sqrtf(tot.x * inv_n + p.eps), 1.f / sqrtf(tot.y * inv_n + p.eps)};
+#pragma unroll
+      for (int k = 0; k < CH; ++k) {
+        const int c = (k * blockDim.x + threadIdx.x) * 4;
+        if (c >= N) continue;
+        float a[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int b = 0; b < kMaxBranches; ++b)
+          if (b < p.n_branches) {
+            float w[4] = {1.f, 1.f, 1.f, 1.f};
+            if (p.w[b] != nullptr) load4<float>(p.w[b] + c, w);
+            const float g = p.gain[b] * (p.w[b] != nullptr ? r[b] : 1.f);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) a[j] = fmaf(g * w[j], y[b][k][j], a[j]);
+            if (p.clear_y[b])
+              *reinterpret_cast<float4*>(p.y[b] + static_cast<long long>(row) * p.ldy + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+          }
+        if (p.e_rows != nullptr) {
+          const float4 e = expert_sum4<T>(p, row, c);
+          a[0] += e.x;
+          a[1] += e.y;
+          a[2] += e.z;
+          a[3] += e.w;
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) x[k][j] += a[j];
+      }
+    }
+    float ssq = 0.f;
+#pragma unroll
+    for (int k = 0; k < CH; ++k) {
+      const int c = (k * blockDim.x + threadIdx.x) * 4;
+      if (c >= N) continue;
+      if (p.store_x) store4<float>(xr + c, x[k]);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) ssq = fmaf(x[k][j], x[k][j], ssq);
+    }
+    if (dst < 0) continue;  // a row without outputs; the same for every thread of the CTA
+    const float r = 1.f / sqrtf(block_sum_all(ssq, s_red) * inv_n + p.eps);
+#pragma unroll
+    for (int o = 0; o < 2; ++o) {
+      if (o >= p.n_out) break;
+      T* hr = static_cast<T*>(p.h[o]) + static_cast<long long>(dst) * p.ldh;
+#pragma unroll
+      for (int k = 0; k < CH; ++k) {
+        const int c = (k * blockDim.x + threadIdx.x) * 4;
+        if (c >= N) continue;
+        float w[4], v[4];
+        load4<float>(p.norm_w[o] + c, w);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[j] = x[k][j] * r * (w[j] + p.w_offset);
+        store4<T>(hr + c, v);
+      }
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) branch_norm_any_kernel(const BranchNormParams p) {
+  extern __shared__ float s_u[];  // N values of the row
+  __shared__ float s_red[32];
+  __shared__ float2 s_red2[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int N = p.N;
+  const float inv_n = 1.f / static_cast<float>(N);
+  for (int row = blockIdx.x; row < p.rows; row += gridDim.x) {
+    float* xr = p.x + static_cast<long long>(row) * N;
+    if (p.clear != nullptr)
+      for (int c = threadIdx.x; c < p.clear_n; c += blockDim.x) p.clear[static_cast<long long>(row) * p.clear_ld + c] = 0.f;
+    const int dst = p.row_map != nullptr ? p.row_map[row] : row;
+    const T* er = nullptr;
+    float r[kMaxBranches] = {};
+    if (p.tokens != nullptr) {
+      const int tok = p.tokens[row];
+      const bool ok = tok >= 0 && tok < p.vocab;
+      if (!ok && threadIdx.x == 0) set_status_once(p.status, kStatusBadIndex);
+      er = static_cast<const T*>(p.embed) + static_cast<long long>(ok ? tok : 0) * N;
+    } else {
+      float ss[kMaxBranches] = {};
+      for (int c = threadIdx.x; c < N; c += blockDim.x)
+#pragma unroll
+        for (int b = 0; b < kMaxBranches; ++b)
+          if (b < p.n_branches) {
+            const float y = p.y[b][static_cast<long long>(row) * p.ldy + c];
+            ss[b] = fmaf(y, y, ss[b]);
+          }
+      const float2 tot = block_sum2(make_float2(ss[0], ss[1]), s_red2);
+      r[0] = 1.f / sqrtf(tot.x * inv_n + p.eps);
+      r[1] = 1.f / sqrtf(tot.y * inv_n + p.eps);
+    }
+    float ssq = 0.f;
+    for (int c = threadIdx.x; c < N; c += blockDim.x) {
+      float x;
+      if (er != nullptr) {
+        x = to_f(er[c]) * p.embed_scale;
+      } else {
+        x = p.e_rows != nullptr ? expert_sum<T>(p, row, c) : 0.f;
+#pragma unroll
+        for (int b = 0; b < kMaxBranches; ++b)
+          if (b < p.n_branches) {
+            const float y = p.y[b][static_cast<long long>(row) * p.ldy + c];
+            x = fmaf(p.gain[b] * (p.w[b] != nullptr ? r[b] * p.w[b][c] : 1.f), y, x);
+          }
+        x += xr[c];
+      }
+#pragma unroll
+      for (int b = 0; b < kMaxBranches; ++b)
+        if (b < p.n_branches && p.clear_y[b]) p.y[b][static_cast<long long>(row) * p.ldy + c] = 0.f;
+      if (p.store_x) xr[c] = x;
+      s_u[c] = x;
+      ssq = fmaf(x, x, ssq);
+    }
+    if (dst < 0) continue;
+    const float rr = 1.f / sqrtf(block_sum_all(ssq, s_red) * inv_n + p.eps);
+    for (int o = 0; o < p.n_out; ++o) {
+      T* hr = static_cast<T*>(p.h[o]) + static_cast<long long>(dst) * p.ldh;
+      for (int c = threadIdx.x; c < N; c += blockDim.x) hr[c] = from_f<T>(s_u[c] * rr * (p.norm_w[o][c] + p.w_offset));
+    }
+  }
+}
+
+template <typename T>
+cudaError_t launch_branch(const BranchNormParams& p, cudaStream_t stream) {
+  const int cap = 8 * sm_count();
+  const dim3 grid(p.rows < cap ? p.rows : cap);
+  const bool vec = p.N % 4 == 0 && p.ldy % 4 == 0 && p.ldh % 4 == 0 && p.lde % 4 == 0;
+  const int quads = (p.N + 3) / 4;
+  auto threads = [&](int ch) { return dim3(((quads + ch - 1) / ch + 31) / 32 * 32); };
+  // few rows: one piece per thread; many rows: more bytes in flight per thread, several CTAs per SM
+  const bool many = p.rows > 2 * sm_count() && quads > 256;
+  if (vec && quads <= 2048) {
+    if (many && quads > 512) return launch_kernel(branch_norm_kernel<T, 4>, grid, threads(4), 0, stream, true, false, p);
+    if (many || quads > 1024) return launch_kernel(branch_norm_kernel<T, 2>, grid, threads(2), 0, stream, true, false, p);
+    return launch_kernel(branch_norm_kernel<T, 1>, grid, threads(1), 0, stream, true, false, p);
+  }
+  const size_t smem = static_cast<size_t>(p.N) * sizeof(float);
+  ensure_dynamic_smem(branch_norm_any_kernel<T>, smem);
+  return launch_kernel(branch_norm_any_kernel<T>, grid, dim3(256), smem, stream, true, false, p);
+}
+
 }  // namespace
+
+cudaError_t launch_branch_norm(const BranchNormParams& p, int dtype, cudaStream_t stream) {
+  if (p.rows <= 0) return cudaSuccess;
+  return dtype == 0 ? launch_branch<__nv_bfloat16>(p, stream) : launch_branch<float>(p, stream);
+}
 
 cudaError_t launch_stream_norm(const StreamNormParams& p, int dtype, cudaStream_t stream) {
   if (p.rows <= 0) return cudaSuccess;

@@ -45,7 +45,7 @@ CUDA_FLAGS = [
 
 
 # kernels of the extension that only layer-list decoders load
-HYBRID_KERNELS = ("stream_ops.cu", "mixer_ops.cu", "attn_rows.cu", "retention.cu")
+HYBRID_KERNELS = ("stream_ops.cu", "mixer_ops.cu", "attn_rows.cu", "retention.cu", "ssd.cu", "moe_ops.cu")
 HYBRID_HEADERS = ("hybrid.cuh", "hybrid_dev.cuh")
 # kernels of the extension that only quantised weights load
 QUANT_KERNELS = ("quant_ops.cu", "gemm_fp8_block.cu", "nvfp4_quant.cu")

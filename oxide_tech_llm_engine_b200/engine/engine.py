@@ -331,11 +331,7 @@ class LLMEngine:
         budget = int(free * self.cfg.gpu_memory_utilization) - w_bytes - act - (2 << 30) - getattr(self, "_dense_bytes", 0)
         budget -= self.cfg.max_num_seqs * model_cls.state_bytes_per_seq(mc)
         if mc.layers:
-            # streams, fp32 projections, rotated q / k and the chunk states of one prompt step
-            wide = max((L.mixer.heads * (L.mixer.dim + L.mixer.vdim) for L in mc.layers))
-            chunk = max((L.mixer.state_elems for L in mc.layers if L.mixer.kind == "retention"), default=0)
-            budget -= self.max_tokens * 4 * (max(1, mc.streams) * mc.d_model + 6 * wide)
-            budget -= 8 * (self.max_tokens // 128 + self.cfg.max_num_seqs) * chunk
+            budget -= model_cls.step_bytes(mc, self.max_tokens, self.cfg.max_num_seqs)
         per_block = max(1, model_cls.kv_block_bytes(mc, tp, self.cfg.dtype))
         n = budget // per_block
         if n < 16:

@@ -76,7 +76,7 @@ class ModelConfig:
     @property
     def is_recurrent(self) -> bool:
         """Some layer carries a per-sequence state besides the paged KV."""
-        return any(L.mixer.kind == "retention" for L in self.layers)
+        return any(hasattr(part, "state_elems") for L in self.layers for part in L.mixer.parts)
 
     def n_params(self) -> int:
         if self.layers:
@@ -93,6 +93,10 @@ class ModelConfig:
         return self.n_layers * per_layer + emb + self.d_model
 
     def active_params(self) -> int:
+        if self.layers:
+            idle = sum(2 * (L.mlp.experts - L.mlp.top) * L.mlp.ff * self.d_model for L in self.layers
+                       if L.mlp is not None and L.mlp.kind == "moe")
+            return self.n_params() - idle
         if not self.is_moe:
             return self.n_params()
         per_layer = self.d_model * (self.q_dim + 2 * self.kv_dim) + self.q_dim * self.d_model
@@ -101,7 +105,7 @@ class ModelConfig:
 
     def kv_bytes_per_token(self, dtype_bytes: int = 2) -> int:
         if self.layers:
-            att = [self.layers[i].mixer for i in self.layer_runs if self.layers[i].mixer.kind == "attention"]
+            att = [m for i in self.layer_runs for m in self.layers[i].mixer.parts if m.kind == "attention"]
             return sum(a.kv_heads * (a.dim + a.vdim) for a in att) * dtype_bytes
         return 2 * self.n_layers * self.kv_dim * dtype_bytes
 
@@ -152,6 +156,17 @@ def _kipolix_preset(name: str, *, width: int, vocab: int, ff: int, pattern: str,
                        bigram=BigramSpec(buckets, 40503, 10007) if buckets else None)
 
 
+def _povatar_preset(name: str, *, width: int, vocab: int, n_layers: int, heads: int, kv_heads: int, dim: int, chunk: int,
+                    s_heads: int, s_vdim: int, state: int, groups: int, ff: int, experts: int, top: int) -> ModelConfig:
+    """A Povatar-shaped configuration of equal layers: a quarter of every head rotates, four taps."""
+    from .layer_spec import AttentionSpec, LayerSpec, MoeSpec, ParallelSpec, RotarySpec, SsdSpec, YarnSpec, povatar_model
+
+    left = AttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, RotarySpec(dim // 4, 500000.0, False, YarnSpec(8.0, 8192, 32.0, 1.0)),
+                         chunk=chunk, sink=0.0)
+    layer = LayerSpec(ParallelSpec(left, SsdSpec(s_heads, s_vdim, state, groups, 4, groups)), MoeSpec(ff, experts, top), parallel=True)
+    return povatar_model((layer,) * n_layers, width=width, vocab=vocab, eps=1e-5, emb_scale=width ** 0.5, name=name)
+
+
 LAYER_LIST_PRESETS = {
     "kipolix-tiny": dict(width=128, vocab=1024, ff=256, pattern="arar", heads=4, kv_heads=2, dim=64, window=56,
                          keep_first=3, r_heads=2, r_dim=64, r_vdim=64, streams=2, loop=(1, 3, 2), buckets=1000),
@@ -161,13 +176,24 @@ LAYER_LIST_PRESETS = {
 }
 
 
+POVATAR_PRESETS = {
+    "povatar-tiny": dict(width=128, vocab=1024, n_layers=3, heads=4, kv_heads=2, dim=64, chunk=80, s_heads=4, s_vdim=48, state=40,
+                         groups=2, ff=80, experts=12, top=3),
+    # layers of a mid-size mixture: heads of 128 over 8192-token chunks, a state of 128 x 64 per head, 8 of 64 experts
+    "povatar-16b": dict(width=2048, vocab=128256, n_layers=32, heads=16, kv_heads=4, dim=128, chunk=8192, s_heads=64, s_vdim=64,
+                        state=128, groups=8, ff=1408, experts=64, top=8),
+}
+
+
 def preset_names() -> list:
-    return [*PRESETS, *LAYER_LIST_PRESETS]
+    return [*PRESETS, *LAYER_LIST_PRESETS, *POVATAR_PRESETS]
 
 
 def preset(name: str, **overrides) -> ModelConfig:
     if name in LAYER_LIST_PRESETS:
         return replace(_kipolix_preset(name, **LAYER_LIST_PRESETS[name]), **overrides)
+    if name in POVATAR_PRESETS:
+        return replace(_povatar_preset(name, **POVATAR_PRESETS[name]), **overrides)
     if name not in PRESETS:
         raise KeyError(f"unknown model preset {name!r}; known: {sorted(preset_names())}")
     return replace(PRESETS[name], **overrides)

@@ -1,6 +1,7 @@
 """Device model of layer-list decoders: layers of different kinds (softmax attention over the paged KV
-cache, retention with a per-sequence state), hyper-connected residual streams, looped layers, a
-hashed bigram embedding. One GPU; bf16 kernels, or fp32 throughout (`dtype="float32"`).
+cache, retention or a state-space layer with a per-sequence state, two mixers side by side), dense or
+mixture-of-experts feed-forwards behind or beside the mixer, hyper-connected residual streams, looped
+layers, a hashed bigram embedding. One GPU; bf16 kernels, or fp32 throughout (`dtype="float32"`).
 
 Launch sequence of a step (every row is a token, decode rows first, then prompt chunks):
 
@@ -12,6 +13,16 @@ Launch sequence of a step (every row is a token, decode rows first, then prompt 
       MLP:        gemm(gate|up, SwiGLU epilogue) -> gemm(down, fp32 accumulator)
       stream_norm stream update with the accumulator, read-out and norm of the next sublayer
     final stream_norm over the logit rows -> gemm(head)
+
+and with mixer and feed-forward side by side:
+
+    branch_norm   embedding -> residual, norms of the first layer's mixer and feed-forward
+    per layer:
+      gemm(q|k|v | z|x|B|C|dt) -> heads, paged attention -> gemm(O, fp32)
+                               -> convolution, state-space layer, gated_norm -> gemm(O, fp32)
+      moe_route (-> moe_scatter) -> grouped gemm(up, squared ReLU) -> grouped gemm(down)
+      branch_norm   norms of both mixer outputs, weighted expert rows, residual, norms of the next layer
+    final branch_norm over the logit rows -> gemm(head)
 
 KV blocks come from the scheduler's paged pool like any model's (one cache per attention run, so a
 looped layer has one per pass); recurrent states live in slots that the scheduler hands to running
@@ -48,8 +59,16 @@ class _Sublayer:
         self.last_of = last_of       # index of the layer run that this sublayer ends, or -1
 
 
+class _ParallelLayer:
+    """Norm weights of the layer's inputs (mixer, feed-forward), of its two mixer outputs, and the function that runs it."""
+
+    def __init__(self, norms: list, out: tuple, run):
+        self.norms, self.out, self.run = norms, out, run
+
+
 class AttentionRun:
-    """One run of an attention layer: weights shared by all passes, a KV cache of its own."""
+    """One run of an attention layer: weights shared by all passes, a KV cache of its own. Its projection rows
+    may be the first columns of wider ones (a layer with two mixers)."""
 
     def __init__(self, m: "HybridModel", spec, w: dict):
         self.m, self.spec, self.w = m, spec, w
@@ -66,15 +85,18 @@ class AttentionRun:
         m.v_cache.append(self.v)
 
     def __call__(self, s: StepInputs, h: torch.Tensor) -> None:
+        self.m.into_acc(self.attend(s, self.m.project(h, self.w["w_in"], self.width)), self.w["w_o"])
+
+    def attend(self, s: StepInputs, proj: torch.Tensor) -> torch.Tensor:
         m, a, w, M = self.m, self.spec, self.w, s.m
-        proj = m.project(h, w["w_in"], self.width)
         q = m.buffer(("q", a.heads * self.dp, a.dim), a.heads * self.dp)
         hops.heads(proj, M, h=a.heads, g=a.kv_heads, d=a.dim, e=a.vdim, rot=w["rot"], positions=s.positions, q_out=q,
                    q_hd=self.dp, q_norm=w["q_norm"], k_norm=w["k_norm"], eps=m.cfg.rms_eps, k_cache=self.k,
                    v_cache=self.v, slots=s.slot_mapping)
         out = m.buffer(("o", a.out_dim), round_up(a.out_dim, 64))
         nd = s.n_decode
-        kw = dict(window=a.window, keep_first=a.keep_first if a.window else 0, scale=a.scale)
+        kw = dict(window=a.window, keep_first=a.keep_first if a.window else 0, scale=a.scale, chunk=a.chunk,
+                  sink=-math.inf if a.sink is None else a.sink)
         if self.tc:
             kw.update(out_d=a.vdim, exact_p=True)
             if nd > 0:
@@ -90,7 +112,7 @@ class AttentionRun:
             if s.n_prefill > 0:
                 hops.row_attention(q, self.dp, self.k, self.v, s.prefill_block_tables, n=s.n_tiles, tile_seq=s.tile_seq,
                                    tile_q0=s.tile_q0, q_start=s.q_start, q_lens=s.q_lens, ctx_lens=s.ctx_lens, **kw)
-        m.into_acc(out[:M], w["w_o"])
+        return out[:M]
 
 
 class RetentionRun:
@@ -127,6 +149,98 @@ class RetentionRun:
                                    q_start=s.q_start, q_lens=s.q_lens, ctx_lens=s.ctx_lens, n_tiles=s.n_tiles,
                                    n_seqs=s.n_prefill, q_rot=q_rot, k_rot=k_rot, **kw)
         m.into_acc(out[:M], w["w_o"])
+
+
+class SsdRun:
+    """One run of a state-space layer: a recurrent and a convolution state per slot."""
+
+    def __init__(self, m: "HybridModel", spec, w: dict):
+        self.m, self.spec, self.w = m, spec, w
+        r = spec
+        f32 = dict(dtype=torch.float32, device=m.device)
+        self.state = torch.zeros(m.state_slots, r.heads, r.state_p, r.vdim_p, **f32)
+        self.conv_state = torch.zeros(m.state_slots, r.taps, r.channels_p, **f32)
+        m.states += [self.state, self.conv_state]
+        self.runs = m.dtype == torch.bfloat16 and hops.ssd_chunks_ok(r.state_p)
+
+    def mix(self, s: StepInputs, proj: torch.Tensor) -> torch.Tensor:
+        """Projection rows z | x | B | C | dt -> gated and normed rows [M, heads * vdim]."""
+        m, r, w, M, nd = self.m, self.spec, self.w, s.m, s.n_decode
+        y = m.buffer(("ssd_y", r.heads * r.vdim_p), r.heads * r.vdim_p)
+        kw = dict(h=r.heads, g=r.groups, w=w["ssd"], state=self.state, conv_state=self.conv_state, y=y)
+        if nd > 0:
+            hops.ssd_decode(proj, nd, row_slots=s.decode_slots, positions=s.positions, **kw)
+        if s.n_prefill > 0:
+            hops.ssd_prefill(proj, M, seq_slots=s.prefill_slots, tile_seq=s.tile_seq, tile_q0=s.tile_q0, q_start=s.q_start,
+                             q_lens=s.q_lens, ctx_lens=s.ctx_lens, n_tiles=s.n_tiles, n_seqs=s.n_prefill,
+                             u=m.buffer(("ssd_u", r.channels_p), r.channels_p), runs=self.runs, **kw)
+        out = m.buffer(("ssd_o", r.inner), round_up(r.inner, 64))
+        hops.gated_norm(y, proj, M, h=r.heads, e=r.vdim, ep=r.vdim_p, groups=r.norm_groups, w=w["norm"], eps=m.cfg.rms_eps, out=out)
+        return out[:M]
+
+
+class MoeRun:
+    """Mixture of experts. Its result stays where the experts leave it: `experts` = (rows, slots, weights, top)
+    for the kernel that adds the weighted rows to the residual."""
+
+    def __init__(self, m: "HybridModel", spec, w: dict):
+        self.m, self.spec, self.w = m, spec, w
+        self.fp = round_up(spec.ff, 64)
+        self.b = m.moe_buffers(spec.experts, spec.top, self.fp)
+
+    def __call__(self, s: StepInputs, h: torch.Tensor) -> tuple:
+        m, e, w, b, M = self.m, self.spec, self.w, self.b, s.m
+        E, top = e.experts, e.top
+        route = dict(e=E, top=top, weight=b["weight"], expert=b["expert"], slot=b["slot"])
+        if m.dtype == torch.float32 or m.few_rows(M):
+            hops.moe_route(h, w["router"], M, **route)
+            pairs = M * top
+            rows, act = b["out"][:pairs], b["act"][:pairs]
+            hops.moe_rows(h, w["up"], b["expert"], pairs, top=top, per_pair=False, y=act, act=2)
+            hops.moe_rows(act, w["down"], b["expert"], pairs, top=top, per_pair=True, y=rows)
+            return rows, b["slot"], b["weight"], top
+        if M <= 128:
+            # one slab of 128 rows per expert: a single launch routes and places
+            xs, act, rows = (b[k][:E * 128] for k in ("xs", "act", "out"))
+            hops.moe_route(h, w["router"], M, mode=1, counts=b["counts"], xs=xs, **route)
+            m_tiles = min(E, M * top)
+            gx, ga, gr = xs.view(E, 128, -1), act.view(E, 128, -1), rows.view(E, 128, -1)
+        else:
+            m_tiles = (M * top + 127 * min(E, M * top)) // 128
+            n = m_tiles * 128
+            gx, ga, gr = b["xs"][:n], b["act"][:n], b["out"][:n]
+            rows = gr
+            logits = b["logits"][:M]
+            ops.gemm(h, w["router_p"], out=logits, epi=ops.EPI_STORE_F32, **m._gemm_shape(M, logits.shape[1], m.dp, store=True))
+            hops.moe_route(h, w["router"], M, mode=2, logits=logits, counts=b["counts"], **route)
+            hops.moe_scatter(h, M, e=E, top=top, expert=b["expert"], slot=b["slot"], counts=b["counts"], xs=gx)
+        ops.gemm(gx, w["up"], out=ga, group_counts=b["counts"], m_tiles=m_tiles, act=2, bn=m.group_bn(m_tiles, self.fp))
+        ops.gemm(ga, w["down"], out=gr, group_counts=b["counts"], m_tiles=m_tiles, bn=m.group_bn(m_tiles, m.dp),
+                 done_ticket=b["ticket"], reset_on_done=b["counts"])
+        return rows, b["slot"], b["weight"], top
+
+
+class ParallelRun:
+    """Two mixers on the same rows, each into an accumulator of its own, beside a feed-forward."""
+
+    def __init__(self, m: "HybridModel", spec, w: dict, mlp):
+        self.m, self.w, self.mlp = m, w, mlp
+        self.left = AttentionRun(m, spec.left, w["left"])
+        self.right = SsdRun(m, spec.right, w["right"])
+        self.split = round_up(self.left.width, 64)        # first column of the right mixer's projection
+        self.width = self.split + spec.right.width_p
+        self.k = (round_up(spec.left.out_dim, 64), round_up(spec.right.out_dim, 64))
+
+    def clears(self, M: int) -> tuple:
+        """Which accumulators have to be zero when the layer starts."""
+        return tuple(self.m.adds_up(M, k) for k in self.k)
+
+    def __call__(self, s: StepInputs, h: torch.Tensor, h2: Optional[torch.Tensor]) -> Optional[tuple]:
+        m, w = self.m, self.w
+        proj = m.project(h, w["w_in"], self.width)
+        m.into_branch(0, self.left.attend(s, proj), w["left"]["w_o"])
+        m.into_branch(1, self.right.mix(s, proj[:, self.split:]), w["right"]["w_o"])
+        return self.mlp(s, h2) if self.mlp is not None else None
 
 
 class MlpRun:
@@ -193,11 +307,21 @@ class HybridModel(GemmShapes):
         d = cfg.d_model
         self.dp = round_up(d, 64)
         dev = self.device
-        att = [L.mixer for L in cfg.layers if L.mixer.kind == "attention"]
+        self.parallel = any(L.parallel for L in cfg.layers)
+        if self.parallel and (cfg.streams or cfg.loop or cfg.bigram or not all(L.parallel for L in cfg.layers)):
+            raise ConfigError(f"{cfg.name}: layers with mixer and feed-forward side by side come without hyper-connected streams, "
+                              "loops and a bigram embedding, and without other layers")
+        moe = [L.mlp for L in cfg.layers if L.mlp is not None and L.mlp.kind == "moe"]
+        if any(e.experts > hops.max_experts()[0] or e.top > hops.max_experts()[1] for e in moe):
+            raise ConfigError(f"{cfg.name}: at most {hops.max_experts()[0]} experts, {hops.max_experts()[1]} of them chosen")
+        att = [p for L in cfg.layers for p in L.mixer.parts if p.kind == "attention"]
         self.hkv = min((a.kv_heads for a in att), default=1)
         self.x = torch.zeros(max_tokens, self.streams, d, dtype=torch.float32, device=dev)
         self.h = torch.zeros(max_tokens, self.dp, dtype=self.dtype, device=dev)
-        self.acc = torch.zeros(max_tokens, self.dp, dtype=torch.float32, device=dev)
+        n_acc = 2 if self.parallel else 1
+        self.branches = torch.zeros(n_acc, max_tokens, self.dp, dtype=torch.float32, device=dev)
+        self.acc = self.branches[0]
+        self.h2 = torch.zeros_like(self.h) if self.parallel else None
         self.vp = round_up(cfg.vocab_size, 64)
         self.v_l = cfg.vocab_size
         self.lm_h = torch.zeros(self.max_logits, self.dp, dtype=self.dtype, device=dev)
@@ -212,16 +336,20 @@ class HybridModel(GemmShapes):
                          if self.dtype == torch.bfloat16 else None)
         self._buffers: dict = {}
         self._scratch: dict = {}
+        self._moe: dict = {}
         self.k_cache: list = []
         self.v_cache: list = []
         self.states: list = []
         self.embed = self.bigram = self.head = self.out_norm = None
         self.sublayers: list = []
+        self._rots: dict = {}         # device frequencies by RotarySpec
         self.layer_hook = None        # called with (layer run, summed streams [rows, width]) after every layer run
 
     # ------------------------------------------------------------------ sizes
     @staticmethod
     def _in_width(mix) -> int:
+        if mix.kind == "parallel":
+            return round_up(HybridModel._in_width(mix.left) + mix.right.width_p, 64)
         w = (mix.heads * mix.dim + mix.kv_heads * (mix.dim + mix.vdim) if mix.kind == "attention"
              else 2 * mix.heads * (mix.dim + mix.vdim))
         return round_up(w, 64)
@@ -230,10 +358,7 @@ class HybridModel(GemmShapes):
     def kv_block_bytes(cfg: ModelConfig, tp: int = 1, dtype: str = "bfloat16") -> int:
         """Device bytes of one 16-token KV block over all attention runs (0: no attention layers)."""
         total = 0
-        for i in cfg.layer_runs:
-            a = cfg.layers[i].mixer
-            if a.kind != "attention":
-                continue
+        for a in (p for i in cfg.layer_runs for p in cfg.layers[i].mixer.parts if p.kind == "attention"):
             big = max(a.dim, a.vdim)
             if dtype == "bfloat16" and big <= 128 and a.heads // a.kv_heads <= 16:
                 total += a.kv_heads * 16 * 2 * (64 if big <= 64 else 128) * 2
@@ -243,7 +368,42 @@ class HybridModel(GemmShapes):
 
     @staticmethod
     def state_bytes_per_seq(cfg: ModelConfig) -> int:
-        return sum(4 * cfg.layers[i].mixer.state_elems for i in cfg.layer_runs if cfg.layers[i].mixer.kind == "retention")
+        return sum(4 * getattr(p, "state_elems", 0) for i in cfg.layer_runs for p in cfg.layers[i].mixer.parts)
+
+    @staticmethod
+    def step_bytes(cfg: ModelConfig, max_tokens: int, max_seqs: int) -> int:
+        """Device bytes of a step's work space: streams, fp32 projections, rotated q / k, chunk states of
+        retention, rows of the experts."""
+        parts = [p for L in cfg.layers for p in L.mixer.parts]
+        wide = max(p.width_p if p.kind == "ssd" else p.heads * (p.dim + p.vdim) for p in parts)
+        chunk = max((p.state_elems for p in parts if p.kind == "retention"), default=0)
+        n = max_tokens * 4 * (max(1, cfg.streams) * cfg.d_model + 6 * wide) + 8 * (max_tokens // 128 + max_seqs) * chunk
+        return n + max((HybridModel._moe_rows(L.mlp.experts, L.mlp.top, max_tokens) * 4 * (2 * cfg.d_model + L.mlp.ff)
+                        for L in cfg.layers if L.mlp is not None and L.mlp.kind == "moe"), default=0)
+
+    @staticmethod
+    def _moe_rows(experts: int, top: int, max_tokens: int) -> int:
+        """Rows of the expert buffers: 128-row slabs of every expert, or packed rows in whole 128-row tiles."""
+        return max(experts * 128, (max_tokens * top + 127 * experts + 127) // 128 * 128)
+
+    def moe_buffers(self, experts: int, top: int, fp: int) -> dict:
+        """Work space of a mixture of experts, shared by the layers of one shape."""
+        b = self._moe.get((experts, top, fp))
+        if b is None:
+            dev, n, T = self.device, self._moe_rows(experts, top, self.max_tokens), self.max_tokens
+            i32 = dict(dtype=torch.int32, device=dev)
+            b = {"weight": torch.zeros(T * top, device=dev), "expert": torch.zeros(T * top, **i32), "slot": torch.zeros(T * top, **i32),
+                 "counts": torch.zeros(experts, **i32), "ticket": torch.zeros(1, **i32),
+                 "act": torch.zeros(n, fp, dtype=self.dtype, device=dev), "out": torch.zeros(n, self.dp, dtype=self.dtype, device=dev)}
+            if self.dtype == torch.bfloat16:
+                b["xs"] = torch.zeros(n, self.dp, dtype=self.dtype, device=dev)
+                b["logits"] = torch.zeros(T, round_up(experts, 64), device=dev)
+            self._moe[experts, top, fp] = b
+        return b
+
+    def group_bn(self, m_tiles: int, n: int) -> int:
+        """Tile width of an expert GEMM: narrow while the tiles would not fill the SMs."""
+        return 64 if m_tiles * ((n + 127) // 128) < self._sms else 128
 
     def buffer(self, key: tuple, width: int) -> torch.Tensor:
         """[max_tokens, width] activation rows of one layout. Columns that no kernel of that layout writes
@@ -270,8 +430,66 @@ class HybridModel(GemmShapes):
             w = out
         return ops.tile_weight(w) if self.tile_weights and self.dtype == torch.bfloat16 else w.contiguous()
 
+    def _ssd_weights(self, r, p: str, mat, vec) -> dict:
+        """Tensors of a state-space layer in the padded channel layout (z | x | B | C | dt; zero rows as padding)."""
+        def blocks(t: torch.Tensor, n: int, k: int, kp: int) -> torch.Tensor:
+            """n blocks of k rows -> n blocks of kp."""
+            out = t.new_zeros(n, kp, *t.shape[1:])
+            out[:, :k] = t.view(n, k, *t.shape[1:])
+            return out.flatten(0, 1)
+
+        inner, gn = r.inner, r.groups * r.state
+
+        def channels(t: torch.Tensor) -> torch.Tensor:
+            x, b, c = t.split([inner, gn, gn])
+            return torch.cat([blocks(x, r.heads, r.vdim, r.vdim_p), blocks(b, r.groups, r.state, r.state_p),
+                              blocks(c, r.groups, r.state, r.state_p)])
+
+        w = mat(p + "in")
+        z, xbc, dt = w.split([inner, inner + 2 * gn, r.heads])
+        return {"in": torch.cat([blocks(z, r.heads, r.vdim, r.vdim_p), channels(xbc), dt]),
+                "ssd": tuple(t.contiguous() for t in (channels(vec(p + "conv")), channels(vec(p + "conv.b")), vec(p + "dt_bias"),
+                                                      vec(p + "A_log"), vec(p + "D"))),
+                "norm": vec(p + "norm"), "w_o": self._pad(mat(p + "o"))}
+
+    def _moe_weights(self, e, p: str, mat) -> dict:
+        fp = round_up(e.ff, 64)
+        kw = dict(dtype=self.dtype, device=self.device)
+        up, down = torch.zeros(e.experts, fp, self.dp, **kw), torch.zeros(e.experts, self.dp, fp, **kw)
+        router = torch.zeros(round_up(e.experts, 64), self.dp, **kw)
+        d = self.cfg.d_model
+        for i in range(e.experts):
+            up[i, :e.ff, :d] = mat(f"{p}e{i}.up")
+            down[i, :d, :e.ff] = mat(f"{p}e{i}.down")
+        router[:e.experts, :d] = mat(p + "router")
+        return {"up": up, "down": down, "router": router[:e.experts], "router_p": router}
+
+    def _build_parallel(self, get) -> None:
+        """Layers whose mixer and feed-forward run side by side."""
+        mat = lambda name: get(name, False)
+        vec = lambda name: get(name, True).contiguous()
+        self.embed, self.head, self.out_norm = mat("embed").contiguous(), self._pad(mat("head")), vec("final.norm")
+        self.k_cache, self.v_cache, self.states, self.sublayers = [], [], [], []
+        for i, L in enumerate(self.cfg.layers):
+            p, mx = f"l{i}.", L.mixer
+            a = mx.left
+            if a.rot not in self._rots:
+                self._rots[a.rot] = hops.Rotary(a.rot, self.device)
+            q = torch.cat([mat(f"{p}mix.left.{n}") for n in ("q", "k", "v")])
+            ssd = self._ssd_weights(mx.right, p + "mix.right.", mat, vec)
+            w_in = torch.cat([q, q.new_zeros(round_up(q.shape[0], 64) - q.shape[0], q.shape[1]), ssd.pop("in")])
+            w = {"w_in": self._pad(w_in), "right": ssd,
+                 "left": {"rot": self._rots[a.rot], "q_norm": None, "k_norm": None, "w_o": self._pad(mat(p + "mix.left.o"))}}
+            mlp = MoeRun(self, L.mlp, self._moe_weights(L.mlp, p + "mlp.", mat)) if L.mlp is not None else None
+            norms = [vec(p + "norm1")] + ([vec(p + "norm2")] if mlp is not None else [])
+            out = (vec(p + "mix.left.out"), vec(p + "mix.right.out"))
+            self.sublayers.append(_ParallelLayer(norms, out, ParallelRun(self, mx, w, mlp)))
+        torch.cuda.empty_cache()
+
     def _build(self, get) -> None:
         """`get(name, fp32)` returns a named tensor on the device, in fp32 or in the model's dtype."""
+        if self.parallel:
+            return self._build_parallel(get)
         cfg = self.cfg
         mat = lambda name: get(name, False)
         vec = lambda name: get(name, True).contiguous()
@@ -280,7 +498,7 @@ class HybridModel(GemmShapes):
         self.head = self._pad(mat("head"))
         self.out_norm = vec("final.norm")
         one = torch.ones(1, dtype=torch.float32, device=self.device)
-        rots: dict = {}
+        rots = self._rots
 
         def hc(p: str, q: int) -> dict:
             if not cfg.streams:
@@ -328,7 +546,7 @@ class HybridModel(GemmShapes):
     def init_random(self, seed: int = 0, std: float = 0.02) -> None:
         """Random weights generated on the device (benchmarks): N(0, std) matrices, unit norms, and
         hyper-connections that act as a plain residual."""
-        from .layer_spec import layer_list_tensors
+        from .layer_spec import initial_vector, layer_list_tensors
 
         g = torch.Generator(device=self.device)
         g.manual_seed(seed)
@@ -341,9 +559,9 @@ class HybridModel(GemmShapes):
                 t = torch.eye(s) if name.endswith(".mix") else torch.full(shape, 1.0 / s if name.endswith(".in") else 1.0)
                 return t.to(self.device)
             if len(shape) == 1:
-                return torch.full(shape, 1.0 if name.endswith((".q.norm", ".k.norm")) else 0.0, device=self.device)
-            t = torch.empty(*shape, dtype=self.dtype, device=self.device)
-            return t.normal_(0.0, std, generator=g)
+                return torch.from_numpy(initial_vector(self.cfg, name, shape)).to(self.device)
+            t = torch.empty(*shape, dtype=torch.float32 if f32 else self.dtype, device=self.device)
+            return t.normal_(0.0, self.cfg.d_model ** -0.5 if name.endswith(".router") else std, generator=g)
 
         self._build(get)
 
@@ -379,10 +597,24 @@ class HybridModel(GemmShapes):
                 ops.gemm(h, w, out=out, **gc)
         return out
 
-    def into_acc(self, x: torch.Tensor, w: torch.Tensor) -> None:
+    def adds_up(self, M: int, k: int) -> bool:
+        """Whether an output projection of K = k splits K and adds its parts into the accumulator (which then has
+        to be zero); otherwise it stores."""
+        return (self.dtype == torch.bfloat16 and not self.few_rows(M)
+                and self._gemm_shape(M, self.dp, k, routed=True)["splits"] > 1)
+
+    def into_branch(self, b: int, x: torch.Tensor, w: torch.Tensor) -> None:
+        """branches[b] = x @ w^T (fp32)."""
+        M, k = x.shape
+        if not self.adds_up(M, k) and self.dtype == torch.bfloat16 and not self.few_rows(M):
+            ops.gemm(x, w, out=self.branches[b, :M], epi=ops.EPI_STORE_F32, **self._gemm_shape(M, self.dp, k, routed=True))
+        else:
+            self.into_acc(x, w, self.branches[b])
+
+    def into_acc(self, x: torch.Tensor, w: torch.Tensor, acc: Optional[torch.Tensor] = None) -> None:
         """acc = x @ w^T (fp32). The accumulator is zero here: stream_norm clears what it has read."""
         M, k = x.shape
-        acc = self.acc[:M]
+        acc = (self.acc if acc is None else acc)[:M]
         if self.dtype == torch.float32:
             hops.gemm_f32(x, w, acc)
         elif self.few_rows(M):
@@ -395,6 +627,8 @@ class HybridModel(GemmShapes):
     def forward(self, s: StepInputs, hidden_in: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Runs one step; returns fp32 logits [n_logits, vocab] (a view of a static buffer; steps with more
         logit rows than the buffer holds get one of their own)."""
+        if self.parallel:
+            return self._forward_parallel(s)
         cfg, M = self.cfg, s.m
         h = self.h[:M]
         subs = self.sublayers
@@ -404,10 +638,7 @@ class HybridModel(GemmShapes):
                          in_w=subs[0].hc["in"], norm_w=subs[0].norm, eps=cfg.rms_eps, h=h,
                          clear=self._proj_splits(M, subs[0]))
         n_log = max(s.n_logits, 1)
-        lm_h, logits = self.lm_h, self.logits_buf
-        if n_log > self.max_logits:
-            lm_h = torch.zeros(n_log, self.dp, dtype=self.dtype, device=self.device)
-            logits = torch.empty(n_log, self.vp, dtype=torch.float32, device=self.device)
+        lm_h, logits = self._logit_rows(n_log)
         for i, sub in enumerate(subs):
             sub.run(s, h)
             kw = dict(y=self.acc, mix=sub.hc["mix"], out_w=sub.hc["out"], eps=cfg.rms_eps)
@@ -419,6 +650,47 @@ class HybridModel(GemmShapes):
                                  store_x=self.layer_hook is not None, **kw)
             if self.layer_hook is not None and sub.last_of >= 0:
                 self.layer_hook(sub.last_of, self.x[:M].sum(1))
+        return self._head(lm_h, logits, n_log)
+
+    def _forward_parallel(self, s: StepInputs) -> torch.Tensor:
+        cfg, M, layers = self.cfg, s.m, self.sublayers
+        h, h2 = self.h[:M], self.h2[:M]
+        x = self.x.view(self.max_tokens, -1)
+        n_log = max(s.n_logits, 1)
+        lm_h, logits = self._logit_rows(n_log)
+        experts = None
+        for i in range(len(layers) + 1):
+            # what the layer before left, into the residual; then the norms of this one (or of the head)
+            last = i == len(layers)
+            clears = (False, False) if last else layers[i].run.clears(M)
+            kw = dict(eps=cfg.rms_eps, w_offset=cfg.norm_weight_offset)
+            if i == 0:
+                kw.update(tokens=s.token_ids, embed=self.embed, embed_scale=cfg.emb_scale)
+                out = (None, None)
+            else:
+                kw.update(experts=experts)
+                out = layers[i - 1].out
+            kw["branches"] = [(self.branches[b], out[b], 0.5, clears[b]) for b in range(2)]
+            if last:
+                kw.update(norm_w=[self.out_norm], h=[lm_h], row_map=s.logit_map, store_x=self.layer_hook is not None)
+            else:
+                norms = layers[i].norms
+                kw.update(norm_w=norms, h=[h, h2][:len(norms)], clear=self._proj_splits(M, layers[i]))
+            hops.branch_norm(x, M, **kw)
+            if self.layer_hook is not None and i > 0:
+                self.layer_hook(i - 1, x[:M])
+            if not last:
+                experts = layers[i].run(s, h, h2)
+        return self._head(lm_h, logits, n_log)
+
+    def _logit_rows(self, n_log: int) -> tuple:
+        """Static buffers of the normed logit rows and the logits; larger ones for a step that has more of them."""
+        if n_log <= self.max_logits:
+            return self.lm_h, self.logits_buf
+        return (torch.zeros(n_log, self.dp, dtype=self.dtype, device=self.device),
+                torch.empty(n_log, self.vp, dtype=torch.float32, device=self.device))
+
+    def _head(self, lm_h: torch.Tensor, logits: torch.Tensor, n_log: int) -> torch.Tensor:
         lm_h, logits = lm_h[:n_log], logits[:n_log]
         if self.dtype == torch.float32:
             hops.gemm_f32(lm_h, self.head, logits)
@@ -426,7 +698,7 @@ class HybridModel(GemmShapes):
             ops.gemv(lm_h, self.head, logits)
         else:
             ops.gemm(lm_h, self.head, out=logits, epi=ops.EPI_STORE_F32, **self._gemm_shape(n_log, self.vp, self.dp, store=True))
-        return logits[:, :cfg.vocab_size]
+        return logits[:, :self.cfg.vocab_size]
 
     # ------------------------------------------------------------------ state
     def copy_blocks(self, src: torch.Tensor, dst: torch.Tensor) -> None:
@@ -441,7 +713,10 @@ class HybridModel(GemmShapes):
     def reset_sync_state(self) -> None:
         """Clears what kernels accumulate into, after a step that a device error cut short."""
         torch.cuda.synchronize(self.device)
-        self.acc.zero_()
+        self.branches.zero_()
+        for b in self._moe.values():
+            b["counts"].zero_()
+            b["ticket"].zero_()
         if self.proj_acc is not None:
             self.proj_acc.zero_()
         ops.gemm_workspace(self.device)[1].zero_()
@@ -449,4 +724,5 @@ class HybridModel(GemmShapes):
 
     def close(self) -> None:
         self._buffers.clear()
+        self._moe.clear()
         self._scratch.clear()

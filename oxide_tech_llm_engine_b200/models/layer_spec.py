@@ -1,7 +1,7 @@
 """Descriptions of decoders that are given as a list of layers rather than as one repeated block.
 
-A `LayerSpec` names a token mixer (attention, retention, ...) and a feed-forward, each with its own
-sizes and constants, so layers of one model may differ in kind, in head layout and in window. The
+A `LayerSpec` names a token mixer (attention, retention, several side by side, ...) and a feed-forward
+(dense, mixture of experts), each with its own sizes and constants, so layers of one model may differ in kind, in head layout and in window. The
 specs are plain data: `models.hybrid` builds the device layers from them, `models.cpu_hybrid` the
 CPU ones, `models.weights` the tensor list. A further design adds its mixer here as one more
 dataclass with the constants as fields, and registers its configuration reader in
@@ -9,6 +9,7 @@ dataclass with the constants as fields, and registers its configuration reader i
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 from typing import Any, Optional, Union
 
@@ -16,19 +17,49 @@ from ..errors import ConfigError
 
 
 @dataclass(frozen=True)
+class YarnSpec:
+    """YaRN scaling of rotation frequencies: pairs that turn fewer than `slow` times within `original`
+    positions are slowed down by `factor`, pairs that turn more than `fast` times stay, a ramp over the
+    pair index lies between; sin and cos carry the factor 0.1 ln(factor) + 1."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+    def frequencies(self, dims: int, base: float, freqs: list) -> tuple[list, float]:
+        def pair_that_turns(n: float) -> float:
+            return dims * math.log(self.original / (2.0 * math.pi * n)) / (2.0 * math.log(base))
+
+        lo = max(math.floor(pair_that_turns(self.fast)), 0)
+        hi = min(math.ceil(pair_that_turns(self.slow)), dims - 1)
+        out = []
+        for i, f in enumerate(freqs):
+            r = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+            out.append(f / self.factor * r + f * (1.0 - r))
+        return out, 0.1 * math.log(self.factor) + 1.0
+
+
+@dataclass(frozen=True)
 class RotarySpec:
     """Rotation of the first `dims` dimensions of every head: pairs (2i, 2i+1) when `interleaved`,
-    else (i, i + dims/2), by the angle position * base^(-2i/dims)."""
+    else (i, i + dims/2), by the angle position * base^(-2i/dims), its frequency scaled by `scaling`."""
     dims: int
     base: float
     interleaved: bool = False
+    scaling: Optional[YarnSpec] = None
+
+    def frequencies(self) -> tuple[list, float]:
+        """Frequency of every pair, and the factor on sin and cos."""
+        f = [float(self.base) ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        return (f, 1.0) if self.scaling is None else self.scaling.frequencies(self.dims, float(self.base), f)
 
 
 @dataclass(frozen=True)
 class AttentionSpec:
     """Softmax attention with grouped key/value heads. `window` 0: every earlier position is visible;
     else the last `window` positions and the first `keep_first` ones of the sequence (which keep their
-    true positions). `qk_norm` "projection": RMS norm over all heads of q (of k) at once, before the
+    true positions). `chunk` (instead of a window): only positions of the same chunk, counted from position
+    0. `sink`: score of one more term of the softmax denominator that has no value. `qk_norm` "projection": RMS norm over all heads of q (of k) at once, before the
     rotation."""
     heads: int
     kv_heads: int
@@ -39,8 +70,14 @@ class AttentionSpec:
     window: int = 0
     keep_first: int = 0
     qk_norm: str = "none"      # none | projection
+    chunk: int = 0
+    sink: Optional[float] = None
 
     kind = "attention"
+
+    @property
+    def parts(self) -> tuple:
+        return (self,)
 
     @property
     def out_dim(self) -> int:
@@ -67,6 +104,10 @@ class RetentionSpec:
     kind = "retention"
 
     @property
+    def parts(self) -> tuple:
+        return (self,)
+
+    @property
     def out_dim(self) -> int:
         return self.heads * self.vdim
 
@@ -80,20 +121,125 @@ class RetentionSpec:
         return [("q", (hd, d)), ("k", (hd, d)), ("v", (hv, d)), ("g", (hv, d)), ("o", (d, hv))]
 
 
+def _pad16(n: int) -> int:
+    return (n + 15) // 16 * 16
+
+
+@dataclass(frozen=True)
+class SsdSpec:
+    """State-space layer with one decay per head and step (Mamba-2). The input projection gives z | x | B | C |
+    step sizes; x, B and C pass a causal convolution of `taps` taps and silu; with dt = softplus(dt + dt_bias),
+    S <- exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x (S: state x vdim per head, head h uses B and C of group
+    h / (heads / groups)); y * silu(z) is normalised in `norm_groups` equal parts and projected."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    taps: int
+    norm_groups: int
+
+    kind = "ssd"
+
+    @property
+    def parts(self) -> tuple:
+        return (self,)
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def out_dim(self) -> int:
+        return self.inner
+
+    # device layout: heads and states padded to whole 16-value pieces with zero channels
+    @property
+    def vdim_p(self) -> int:
+        return _pad16(self.vdim)
+
+    @property
+    def state_p(self) -> int:
+        return _pad16(self.state)
+
+    @property
+    def channels_p(self) -> int:
+        """Channels of the convolution."""
+        return self.heads * self.vdim_p + 2 * self.groups * self.state_p
+
+    @property
+    def width_p(self) -> int:
+        """Columns of the projection."""
+        return self.heads * self.vdim_p + self.channels_p + self.heads
+
+    @property
+    def state_elems(self) -> int:
+        """fp32 values of one sequence's state: the recurrence's and the convolution's."""
+        return self.heads * self.state_p * self.vdim_p + self.taps * self.channels_p
+
+    def tensors(self, d: int) -> list[tuple[str, tuple[int, ...]]]:
+        gn, h = self.groups * self.state, self.heads
+        return [("in", (2 * self.inner + 2 * gn + h, d)), ("conv", (self.inner + 2 * gn, self.taps)),
+                ("conv.b", (self.inner + 2 * gn,)), ("dt_bias", (h,)), ("A_log", (h,)), ("D", (h,)), ("norm", (self.inner,)),
+                ("o", (d, self.inner))]
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Two mixers side by side on the same input; the result is half the sum of the two outputs, each by its
+    own RMS norm over the model width."""
+    left: AttentionSpec
+    right: SsdSpec
+
+    kind = "parallel"
+
+    @property
+    def parts(self) -> tuple:
+        return (*self.left.parts, *self.right.parts)
+
+    def tensors(self, d: int) -> list[tuple[str, tuple[int, ...]]]:
+        out = []
+        for side in ("left", "right"):
+            out += [(f"{side}.{n}", s) for n, s in getattr(self, side).tensors(d)]
+        return out + [("left.out", (d,)), ("right.out", (d,))]
+
+
 @dataclass(frozen=True)
 class DenseMlpSpec:
     """W_down (act(W_gate h) * (W_up h))."""
     ff: int
     act: str = "silu"          # silu | gelu_tanh
 
+    kind = "dense"
+
     def tensors(self, d: int) -> list[tuple[str, tuple[int, ...]]]:
         return [("gate", (self.ff, d)), ("up", (self.ff, d)), ("down", (d, self.ff))]
 
 
 @dataclass(frozen=True)
+class MoeSpec:
+    """Mixture of `experts` feed-forwards W_down act(W_up h); a token uses the `top` ones with the largest scores
+    of a softmax over all experts, weighted by their scores divided by the scores' sum."""
+    ff: int
+    experts: int
+    top: int
+    act: str = "relu2"         # square of relu
+
+    kind = "moe"
+
+    def tensors(self, d: int) -> list[tuple[str, tuple[int, ...]]]:
+        out = []
+        for e in range(self.experts):
+            out += [(f"e{e}.up", (self.ff, d)), (f"e{e}.down", (d, self.ff))]
+        return out + [("router", (self.experts, d))]
+
+
+@dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[AttentionSpec, RetentionSpec]
-    mlp: Optional[DenseMlpSpec]
+    """`parallel`: mixer and feed-forward read the same residual stream, each through its own norm, and both are
+    added to it; else the feed-forward follows the mixer."""
+    mixer: Union[AttentionSpec, RetentionSpec, SsdSpec, ParallelSpec]
+    mlp: Union[DenseMlpSpec, MoeSpec, None]
+    parallel: bool = False
 
     @property
     def sublayers(self) -> int:
@@ -126,7 +272,9 @@ def rotary_from_json(c: Optional[dict], interleaved: bool, dim: int) -> Optional
     dims = int(c["dims"])
     if dims % 2 or dims > dim or dims < 0:
         raise ConfigError(f"rotary dims {dims} do not fit a head of {dim}")
-    return RotarySpec(dims, float(c["base"]), interleaved) if dims else None
+    sc = c.get("scaling")
+    yarn = YarnSpec(*(float(sc[k]) for k in ("factor", "original", "fast", "slow"))) if sc else None
+    return RotarySpec(dims, float(c["base"]), interleaved, yarn) if dims else None
 
 
 def mlp_from_json(c: Optional[dict]) -> Optional[DenseMlpSpec]:
@@ -208,6 +356,102 @@ def kipolix_json(cfg) -> dict[str, Any]:
     if cfg.loop is not None:
         out["loop"] = dict(zip(("start", "stop", "times"), cfg.loop))
     return out
+
+
+def chunked_attention_from_json(c: dict) -> AttentionSpec:
+    """Left mixer of a Povatar layer: rotation of the half layout, chunks, and a sink of score 0."""
+    a = AttentionSpec(heads=int(c["heads"]), kv_heads=int(c["kv_heads"]), dim=int(c["dim"]), vdim=int(c["vdim"]),
+                      scale=float(c["scale"]), rot=rotary_from_json(c.get("rot"), False, int(c["dim"])),
+                      chunk=int((c.get("mask") or {}).get("size", 0)), sink=0.0)
+    if a.heads % a.kv_heads:
+        raise ConfigError(f"{a.heads} query heads do not divide over {a.kv_heads} key/value heads")
+    return a
+
+
+def ssd_from_json(c: dict) -> SsdSpec:
+    s = SsdSpec(heads=int(c["heads"]), vdim=int(c["vdim"]), state=int(c["state"]), groups=int(c["groups"]), taps=int(c["conv"]),
+                norm_groups=int(c["norm_groups"]))
+    if s.heads % s.groups:
+        raise ConfigError(f"{s.heads} heads do not divide over {s.groups} groups")
+    if s.inner % s.norm_groups:
+        raise ConfigError(f"{s.inner} values do not divide into {s.norm_groups} norm groups")
+    return s
+
+
+def moe_from_json(c: Optional[dict]) -> Optional[MoeSpec]:
+    if c is None:
+        return None
+    if c.get("kind") != "moe":
+        raise ConfigError(f"feed-forward kind {c.get('kind')!r} is not part of this design")
+    m = MoeSpec(int(c["expert"]["ff"]), int(c["router"]["experts"]), int(c["router"]["top"]))
+    if not 1 <= m.top <= m.experts:
+        raise ConfigError(f"{m.top} of {m.experts} experts")
+    return m
+
+
+def povatar_layer(c: dict) -> LayerSpec:
+    if c["type"] != "parallel":
+        raise ConfigError(f"layer type {c['type']!r} is not part of this design")
+    mx = c["mixer"]
+    return LayerSpec(ParallelSpec(chunked_attention_from_json(mx["left"]), ssd_from_json(mx["right"])), moe_from_json(c.get("mlp")),
+                     parallel=True)
+
+
+def povatar_model(layers: tuple, *, width: int, vocab: int, eps: float, emb_scale: float, name: str = "povatar"):
+    """ModelConfig of Povatar layers. No tokenizer comes with the design, so there is no end-of-text id."""
+    from .config import ModelConfig
+
+    left = layers[0].mixer.left
+    return ModelConfig(name=name, arch="povatar", n_layers=len(layers), d_model=width, n_heads=left.heads,
+                       n_kv_heads=left.kv_heads, head_dim=left.dim, ffn_dim=max((L.mlp.ff for L in layers if L.mlp), default=0),
+                       vocab_size=vocab, max_ctx=1 << 20, rms_eps=eps, emb_scale=emb_scale, bos_id=-1, eos_id=-1, layers=layers)
+
+
+def povatar_config(c: dict[str, Any]):
+    """ModelConfig of a Povatar checkpoint from its config.json."""
+    return povatar_model(tuple(povatar_layer(x) for x in c["layers"]), width=int(c["width"]), vocab=int(c["vocab"]),
+                         eps=float(c["norm"]["eps"]), emb_scale=float((c.get("embedding") or {}).get("scale", 1.0)))
+
+
+def povatar_json(cfg) -> dict[str, Any]:
+    """config.json of a Povatar ModelConfig (inverse of povatar_config)."""
+    layers = []
+    for L in cfg.layers:
+        a, r = L.mixer.left, L.mixer.right
+        left: dict[str, Any] = {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim, "scale": a.scale}
+        if a.chunk:
+            left["mask"] = {"size": a.chunk}
+        if a.rot is not None:
+            left["rot"] = {"base": a.rot.base, "dims": a.rot.dims}
+            if a.rot.scaling is not None:
+                y = a.rot.scaling
+                left["rot"]["scaling"] = {"factor": y.factor, "original": y.original, "fast": y.fast, "slow": y.slow}
+        right = {"heads": r.heads, "vdim": r.vdim, "state": r.state, "groups": r.groups, "conv": r.taps, "norm_groups": r.norm_groups}
+        mlp = None if L.mlp is None else {"kind": "moe", "expert": {"ff": L.mlp.ff},
+                                          "router": {"experts": L.mlp.experts, "top": L.mlp.top}}
+        layers.append({"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": mlp})
+    return {"architecture": "Povatar", "vocab": cfg.vocab_size, "width": cfg.d_model, "norm": {"eps": cfg.rms_eps},
+            "embedding": {"scale": cfg.emb_scale}, "layers": layers}
+
+
+def initial_vector(cfg, name: str, shape: tuple):
+    """Starting values of a vector (synthetic weights): unit norms (stored as the distance from one where the design
+    does so), step sizes of 0.001 to 0.1, decay rates of 1 to 16."""
+    import numpy as np
+
+    n = shape[0]
+    ramp = np.arange(n, dtype=np.float64) / max(1, n - 1)
+    if name.endswith(".dt_bias"):
+        v = np.log(np.expm1(10.0 ** (-3.0 + 2.0 * ramp)))
+    elif name.endswith(".A_log"):
+        v = np.log(1.0 + 15.0 * ramp)
+    elif name.endswith(".conv.b"):
+        v = np.zeros(n)
+    elif name.endswith((".q.norm", ".k.norm", ".D")):
+        v = np.ones(n)
+    else:
+        v = np.full(n, 1.0 - cfg.norm_weight_offset)
+    return v.astype(np.float32)
 
 
 def layer_list_tensors(cfg) -> list[tuple[str, tuple[int, ...]]]:

@@ -52,6 +52,12 @@ def _kipolix_json(c: dict):
     return kipolix_config(c)
 
 
+def _povatar_json(c: dict):
+    from .layer_spec import povatar_config
+
+    return povatar_config(c)
+
+
 ARCHITECTURES: dict[str, Architecture] = {}
 
 
@@ -62,6 +68,7 @@ def register(a: Architecture) -> None:
 register(Architecture("llama", _llama, _llama_cpu))
 register(Architecture("mixtral", _llama, _llama_cpu))
 register(Architecture("kipolix", _hybrid, _hybrid_cpu, from_json=_kipolix_json, hf_names=False))
+register(Architecture("povatar", _hybrid, _hybrid_cpu, from_json=_povatar_json, hf_names=False))
 
 
 def architecture(cfg) -> Architecture:

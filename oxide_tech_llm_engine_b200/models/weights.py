@@ -145,9 +145,9 @@ class SyntheticSource(WeightSource):
         if name.endswith("norm.weight"):
             return np.full(shape, 1.0 - self.cfg.norm_weight_offset, dtype=np.float32)
         if self.cfg.layers and len(shape) == 1 and ".hc" not in name:
-            # norms: q / k norms are plain weights, the others are stored as the distance from one
-            one = name.endswith((".q.norm", ".k.norm"))
-            return np.full(shape, 1.0 if one else 1.0 - self.cfg.norm_weight_offset, dtype=np.float32)
+            from .layer_spec import initial_vector
+
+            return initial_vector(self.cfg, name, shape)
         if ".hc" in name:
             # hyper-connections start as an ordinary residual: read the mean of the streams, write to all
             s = self.cfg.streams
@@ -157,7 +157,7 @@ class SyntheticSource(WeightSource):
         key = int((h * np.arange(1, h.size + 1, dtype=np.uint64)).sum() % (2 ** 31))
         rng = np.random.default_rng([self.seed, key])
         std = self.std
-        if name.endswith("ffn_gate_inp.weight"):
+        if name.endswith(("ffn_gate_inp.weight", ".router")):
             # router logits of O(1): hidden states after RMSNorm have unit RMS
             std = 1.0 / np.sqrt(self.cfg.d_model)
         if name.endswith(".bias"):

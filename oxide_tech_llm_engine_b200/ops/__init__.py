@@ -438,18 +438,21 @@ def untile_weight(w: torch.Tensor) -> torch.Tensor:
 def paged_decode(q, k_cache, v_cache, block_tables, seq_lens, pages_per_split, part_o, part_ml, out,
                  *, batch: int, max_splits: int, window: int = 0, scale: float,
                  page_ml: Optional[torch.Tensor] = None, block_mass: Optional[torch.Tensor] = None,
-                 q8=None, keep_first: int = 0, out_d: int = 0, exact_p: bool = False) -> None:
+                 q8=None, keep_first: int = 0, out_d: int = 0, exact_p: bool = False, chunk: int = 0,
+                 sink: float = float("-inf")) -> None:
     """Paged split-KV decode attention + merge. With `page_ml` [B, max_blocks, Hq, 2] and `block_mass`
     [B, max_blocks] (fp32) the kernels also produce the softmax probability mass per KV block, summed
     over heads: the heavy-hitter score of H2O pruning (the reference accumulates it in its decode
     kernel too, oxide-backend-cuda/src/kernels/megakernel_ops.cu:577-617). `q8` = (int8 [B, Hq*D],
     scales, sums): the merge also writes the int8 view of `out` (see `finalize_norm`). `keep_first`: with a
     window, the first positions of the sequence stay visible. `out_d`: values stored per head when the
-    heads are padded to D. `exact_p`: softmax weights enter the value product with 16 instead of 8 bits."""
+    heads are padded to D. `exact_p`: softmax weights enter the value product with 16 instead of 8 bits.
+    `chunk`: instead of a window, only positions of the query's own chunk (counted from position 0) are
+    visible. `sink`: score of one more term of the softmax denominator, which has no value."""
     q8t, q8d, q8s = q8 if q8 is not None else (None, None, None)
     _ext().paged_decode(q, k_cache, v_cache, block_tables, seq_lens, pages_per_split, part_o, part_ml,
                         out, batch, max_splits, window, scale, status_word(q.device) if CHECK_BOUNDS else None,
-                        page_ml, block_mass, q8t, q8d, q8s, keep_first, out_d, exact_p)
+                        page_ml, block_mass, q8t, q8d, q8s, keep_first, out_d, exact_p, chunk, sink)
     _bump(3 if page_ml is not None else 2)
 
 
@@ -460,11 +463,12 @@ CHECK_BOUNDS = os.environ.get("OXB_CHECKS", "0") != "0"
 
 def paged_prefill(q, k_cache, v_cache, block_tables, tile_seq, tile_q0, q_start, q_lens, ctx_lens, out,
                   *, n_tiles: int, window: int = 0, scale: float, keep_first: int = 0, out_d: int = 0,
-                  exact_p: bool = False) -> None:
+                  exact_p: bool = False, chunk: int = 0, sink: float = float("-inf")) -> None:
     """Causal paged attention over ragged prefill chunks on 128-row query tiles (tcgen05 / TMEM,
     attn_prefill_tc.cu); `tile_q0` entries are multiples of 128. Options as in `paged_decode`."""
     _ext().paged_prefill_tc(q, k_cache, v_cache, block_tables, tile_seq, tile_q0, q_start, q_lens,
-                            ctx_lens, out, n_tiles, window, scale, status_word(q.device), keep_first, out_d, exact_p)
+                            ctx_lens, out, n_tiles, window, scale, status_word(q.device), keep_first, out_d, exact_p,
+                            chunk, sink)
     _bump()
 
 

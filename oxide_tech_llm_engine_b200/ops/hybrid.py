@@ -1,4 +1,4 @@
-"""Python front-ends of the layer-list kernels (``csrc/kernels/{stream_ops,mixer_ops,attn_rows,retention}.cu``).
+"""Python front-ends of the layer-list kernels (``csrc/kernels/{stream_ops,mixer_ops,attn_rows,retention,ssd,moe_ops}.cu``).
 
 Activations, weights and caches are bf16, or fp32 throughout; residual streams, states, norms, scores
 and angles are fp32 in both cases. As in `ops`, nothing here falls back to PyTorch.
@@ -14,14 +14,15 @@ from .._build import hybrid_ext
 
 
 class Rotary:
-    """Device frequencies of a layer_spec.RotarySpec, each as the sum of two fp32 numbers."""
+    """Device frequencies of a layer_spec.RotarySpec, each as the sum of two fp32 numbers, and the factor on sin and cos."""
 
     def __init__(self, spec, device):
         self.interleaved = bool(spec is not None and spec.interleaved)
         self.hi = self.lo = None
+        self.gain = 1.0
         if spec is not None and spec.dims > 0:
-            i = torch.arange(spec.dims // 2, dtype=torch.float64)
-            f = torch.pow(torch.tensor(float(spec.base), dtype=torch.float64), -2.0 * i / spec.dims)
+            freqs, self.gain = spec.frequencies()
+            f = torch.tensor(freqs, dtype=torch.float64)
             hi = f.to(torch.float32)
             self.hi = hi.to(device)
             self.lo = (f - hi.to(torch.float64)).to(torch.float32).to(device)
@@ -67,25 +68,25 @@ def heads(proj: torch.Tensor, m: int, *, h: int, g: int, d: int, e: int, rot: Ro
           slots=None) -> None:
     """Projection rows q | k | v -> normed and rotated heads; k and v into the paged cache with q [M, h * q_hd], or
     q and k to dense fp32 buffers [heads, M, d] (HeadsParams)."""
-    hybrid_ext().heads(proj, m, h, g, d, e, q_norm, k_norm, eps, rot.hi, rot.lo, rot.interleaved, positions, k_scale, q_out,
-                       q_hd, k_out, k_cache, v_cache, slots, ops.status_word(proj.device))
+    hybrid_ext().heads(proj, m, h, g, d, e, q_norm, k_norm, eps, rot.hi, rot.lo, rot.interleaved, rot.gain, positions,
+                       k_scale, q_out, q_hd, k_out, k_cache, v_cache, slots, ops.status_word(proj.device))
     ops._bump()
 
 
 def row_attention(q, q_hd: int, k_cache, v_cache, block_tables, *, n: int, h: int, d: int, e: int, window: int,
-                  keep_first: int, scale: float, out, seq_lens=None, tile_seq=None, tile_q0=None, q_start=None, q_lens=None,
-                  ctx_lens=None) -> None:
+                  keep_first: int, scale: float, out, chunk: int = 0, sink: float = float("-inf"), seq_lens=None,
+                  tile_seq=None, tile_q0=None, q_start=None, q_lens=None, ctx_lens=None) -> None:
     """Softmax attention of any head size in fp32 FMAs: decode rows (seq_lens) or prompt tiles."""
     hybrid_ext().row_attention(q, q_hd, k_cache, v_cache, block_tables, seq_lens, tile_seq, tile_q0, q_start, q_lens,
-                               ctx_lens, n, h, d, e, window, keep_first, scale, out, ops.status_word(q.device))
+                               ctx_lens, n, h, d, e, window, keep_first, chunk, scale, sink, out, ops.status_word(q.device))
     ops._bump()
 
 
 def retention_decode(proj, rows: int, *, h: int, d: int, e: int, decay_pow, rot: Rotary, k_scale: float, eps: float, state,
                      row_slots, positions, out) -> None:
     """One token per row: rotation, state update, read-out, head norm and gate in one launch."""
-    hybrid_ext().retention_decode(proj, rows, h, d, e, decay_pow, rot.hi, rot.lo, rot.interleaved, k_scale, eps, state,
-                                  row_slots, positions, out, ops.status_word(proj.device))
+    hybrid_ext().retention_decode(proj, rows, h, d, e, decay_pow, rot.hi, rot.lo, rot.interleaved, rot.gain, k_scale, eps,
+                                  state, row_slots, positions, out, ops.status_word(proj.device))
     ops._bump()
 
 
@@ -95,6 +96,67 @@ def retention_prefill(proj, m: int, *, h: int, d: int, e: int, decay_pow, eps: f
     hybrid_ext().retention_prefill(proj, m, h, d, e, decay_pow, eps, state, seq_slots, tile_seq, tile_q0, q_start, q_lens,
                                    ctx_lens, n_tiles, n_seqs, q_rot, k_rot, ws, o_buf, out, ops.status_word(proj.device))
     ops._bump(3 if ws is not None else 2)
+
+
+def ssd_chunks_ok(n: int) -> bool:
+    return bool(hybrid_ext().ssd_chunks_ok(n))
+
+
+def max_experts() -> tuple[int, int]:
+    """Largest number of experts, and of chosen ones."""
+    ext = hybrid_ext()
+    return int(ext.MAX_EXPERTS), int(ext.MAX_TOP)
+
+
+def branch_norm(x: torch.Tensor, rows: int, *, norm_w, h, eps: float, w_offset: float = 0.0, tokens=None, embed=None,
+                embed_scale: float = 1.0, branches=(), experts=None, store_x: bool = True, row_map=None, clear=None) -> None:
+    """Embedding or the sum of a layer's branches into the residual stream x [M, N], and its RMS norm with one weight per
+    output (BranchNormParams in csrc/kernels/hybrid.cuh). `branches`: (fp32 rows, norm weight or None, gain, clear);
+    `experts`: (rows, slots, weights, chosen per row)."""
+    rows_e, slot, weight, top = experts if experts is not None else (None, None, None, 0)
+    hybrid_ext().branch_norm(x, rows, tokens, embed, embed_scale, [b[0] for b in branches], [b[1] for b in branches],
+                             [b[2] for b in branches], [bool(b[3]) for b in branches], rows_e, slot, weight, top, store_x,
+                             list(norm_w), list(h), eps, w_offset, row_map, clear, ops.status_word(x.device))
+    ops._bump()
+
+
+def ssd_decode(proj, rows: int, *, h: int, g: int, w, state, conv_state, row_slots, positions, y) -> None:
+    """State-space layer, one token per row: convolution, step size, state update and read-out in one launch. `w`:
+    (conv, conv bias, dt_bias, A_log, D) in fp32."""
+    hybrid_ext().ssd_decode(proj, rows, h, g, list(w), state, conv_state, row_slots, positions, y, ops.status_word(proj.device))
+    ops._bump()
+
+
+def ssd_prefill(proj, m: int, *, h: int, g: int, w, state, conv_state, seq_slots, tile_seq, tile_q0, q_start, q_lens, ctx_lens,
+                n_tiles: int, n_seqs: int, u, y, runs: bool) -> None:
+    """Prompt chunks: convolution into `u`, then runs of 64 tokens on tensor cores (`runs`) or token by token."""
+    hybrid_ext().ssd_prefill(proj, m, h, g, list(w), state, conv_state, seq_slots, tile_seq, tile_q0, q_start, q_lens, ctx_lens,
+                             n_tiles, n_seqs, u, y, runs, ops.status_word(proj.device))
+    ops._bump(2)
+
+
+def gated_norm(y, z, m: int, *, h: int, e: int, ep: int, groups: int, w, eps: float, out) -> None:
+    """out = (y * silu(z)) normalised in `groups` equal parts, times w; heads of e values lie ep apart in y and z."""
+    hybrid_ext().gated_norm(y, z, m, h, e, ep, groups, w, eps, out)
+    ops._bump()
+
+
+def moe_route(h, router, m: int, *, e: int, top: int, weight, expert, slot, mode: int = 0, logits=None, counts=None, xs=None) -> None:
+    """Chosen experts, their weights and row slots (MoeRouteParams); logits from h and router unless given."""
+    hybrid_ext().moe_route(h, router, logits, m, e, top, weight, expert, slot, mode, counts, xs, ops.status_word(h.device))
+    ops._bump()
+
+
+def moe_scatter(h, m: int, *, e: int, top: int, expert, slot, counts, xs) -> None:
+    """Ranks -> packed rows, and the rows' copies there."""
+    hybrid_ext().moe_scatter(h, m, e, top, expert, slot, counts, xs, ops.status_word(h.device))
+    ops._bump()
+
+
+def moe_rows(x, w, expert, pairs: int, *, top: int, per_pair: bool, y, act: int = 0) -> None:
+    """Expert products of single (row, choice) pairs."""
+    hybrid_ext().moe_rows(x, w, expert, pairs, top, per_pair, act, y)
+    ops._bump()
 
 
 def gemm_f32(a, w, out) -> None:
