@@ -121,9 +121,18 @@ def main() -> None:
                     help="instead of the headline workload: layer-list decoders (attention + retention) beside the Llama model of "
                          "equal size, engine throughput and kernels against their rooflines")
     ap.add_argument("--kipolix-size", default="", help="only this size of --kipolix")
+    ap.add_argument("--povatar", action="store_true",
+                    help="instead of the headline workload: layers with attention and a state-space mixer side by side and a mixture "
+                         "of experts, beside the Mixtral-shaped model of equal size")
+    ap.add_argument("--povatar-size", default="", help="only this size of --povatar")
     args = ap.parse_args()
     if args.kipolix and args.impl != "reference":
         from oxide_tech_llm_engine_b200.bench_hybrid import run
+
+        run(args, ClockSampler(0))
+        return
+    if args.povatar and args.impl != "reference":
+        from oxide_tech_llm_engine_b200.bench_povatar import run
 
         run(args, ClockSampler(0))
         return

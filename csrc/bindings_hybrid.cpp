@@ -348,7 +348,7 @@ void branch_norm(const Tensor& x, int64_t rows, const OptTensor& tokens, const O
     TORCH_CHECK(!ys.empty(), "branch_norm: tokens or branches");
   }
   if (given(e_rows)) {
-    TORCH_CHECK(given(e_slot) && given(e_weight) && top >= 1 && e_rows->scalar_type() == hs[0].scalar_type() && e_rows->is_cuda(),
+    TORCH_CHECK(given(e_slot) && given(e_weight) && top >= 1 && top <= oxb::kMaxTop && e_rows->scalar_type() == hs[0].scalar_type() && e_rows->is_cuda(),
                 "branch_norm: expert rows of h's type, with slots and weights");
     p.lde = pitch(*e_rows, 1, p.N, "branch_norm expert rows");
     p.n_e_rows = e_rows->size(0);
@@ -420,7 +420,7 @@ void ssd_decode(const Tensor& proj, int64_t rows, int64_t H, int64_t G, const st
 void ssd_prefill(const Tensor& proj, int64_t M, int64_t H, int64_t G, const std::vector<Tensor>& w, const Tensor& state,
                  const Tensor& conv_state, const Tensor& seq_slots, const Tensor& tile_seq, const Tensor& tile_q0, const Tensor& q_start,
                  const Tensor& q_lens, const Tensor& ctx_lens, int64_t n_tiles, int64_t n_seqs, const Tensor& u, const Tensor& y,
-                 bool runs, const Tensor& status) {
+                 bool runs, int64_t segment, const OptTensor& ws, const Tensor& status) {
   oxb::SsdParams p = ssd_common(proj, M, H, G, w, state, conv_state, y, status);
   const int dt = dtype_code(y, "ssd y");
   p.seq_slots = i32(seq_slots, n_seqs, "ssd_prefill seq_slots");
@@ -438,6 +438,13 @@ void ssd_prefill(const Tensor& proj, int64_t M, int64_t H, int64_t G, const std:
   check_launch(oxb::launch_ssd_conv(p, dt, cur_stream()), "ssd_conv");
   if (runs) {
     TORCH_CHECK(dt == 0 && oxb::ssd_chunks_ok(p.NP), "ssd_prefill: runs on tensor cores");
+    TORCH_CHECK(segment >= 0 && segment % 128 == 0 && (segment == 0 || given(ws)), "ssd_prefill: segments of whole tiles, with ws");
+    if (segment > 0) {
+      const int64_t states = n_tiles * H * p.NP * p.EP;
+      p.segment = static_cast<int>(segment);
+      p.ws = const_cast<float*>(f32(*ws, states + n_tiles * H, "ssd_prefill ws"));
+      p.ws_decay = p.ws + states;
+    }
     check_launch(oxb::launch_ssd_chunks(p, cur_stream()), "ssd_prefill");
   } else {
     check_launch(oxb::launch_ssd_scan(p, dt, cur_stream()), "ssd_prefill");
@@ -599,6 +606,9 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("ssd_decode", &ssd_decode);
   m.def("ssd_prefill", &ssd_prefill);
   m.def("ssd_chunks_ok", [](int64_t NP) { return oxb::ssd_chunks_ok(static_cast<int>(NP)); });
+  m.def("ssd_segment", [](int64_t H, int64_t EP, int64_t n_tiles, int64_t n_seqs) {
+    return oxb::ssd_segment(static_cast<int>(H), static_cast<int>(EP), static_cast<int>(n_tiles), static_cast<int>(n_seqs));
+  });
   m.def("gated_norm", &gated_norm);
   m.def("moe_route", &moe_route);
   m.def("moe_scatter", &moe_scatter);

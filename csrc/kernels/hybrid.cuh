@@ -54,6 +54,7 @@ cudaError_t launch_stream_norm(const StreamNormParams& p, int dtype, cudaStream_
 // x is written back when store_x is set. Where clear_y is set for a branch, its rows are zeroed on the way (the
 // split-K GEMM of the layer that follows adds into them).
 constexpr int kMaxBranches = 2;
+constexpr int kMaxTop = 32;   // most experts that a token may use
 struct BranchNormParams {
   float* x;                 // [rows, N]
   int rows, N;
@@ -228,6 +229,9 @@ struct SsdParams {
   long long ldu;
   void* y;                  // [M, ldy]: H * EP
   long long ldy;
+  int segment;              // > 0: sequences are walked in segments of this many rows (a multiple of 128) at once
+  float* ws;                // [n_tiles, H, NP, EP] states of the segments, by their first tile
+  float* ws_decay;          // [n_tiles, H]
   int* status;
 };
 // One token per row: convolution, state update and read-out in one launch.
@@ -239,6 +243,7 @@ cudaError_t launch_ssd_chunks(const SsdParams& p, cudaStream_t stream);
 // Prompt chunks token by token in fp32 FMAs.
 cudaError_t launch_ssd_scan(const SsdParams& p, int dtype, cudaStream_t stream);
 bool ssd_chunks_ok(int NP);
+int ssd_segment(int H, int EP, int n_tiles, int n_seqs);   // rows per segment that suit the device, 0: whole sequences
 
 // out[row] = rms_groups(y * silu(z)) * w: `groups` equal parts of H * E values, each by its own root mean square.
 // y and z hold heads of E values EP apart.
@@ -258,7 +263,6 @@ cudaError_t launch_gated_norm(const GatedNormParams& p, int dtype, cudaStream_t 
 
 // Router of a mixture of experts: softmax over all experts, the `top` largest scores divided by their sum (+ 1e-20).
 constexpr int kMaxExperts = 512;
-constexpr int kMaxTop = 32;
 struct MoeRouteParams {
   const float* logits;      // [M, ldl], or nullptr: computed here from h and router
   long long ldl;

@@ -79,5 +79,12 @@ __device__ __forceinline__ void rotary_pair(const RotaryParams& r, int i, int* u
 }
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+// silu of a value that is stored as T: a bf16 result does not need the full-precision exponential and division
+template <typename T>
+__device__ __forceinline__ float silu_as(float z);
+template <>
+__device__ __forceinline__ float silu_as<float>(float z) { return silu_f(z); }
+template <>
+__device__ __forceinline__ float silu_as<__nv_bfloat16>(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 
 }  // namespace oxb

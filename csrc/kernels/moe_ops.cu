@@ -86,10 +86,12 @@ struct Pack<float> {
 };
 
 // One CTA per row: logits (unless given), choice, slot, and the row's copies (mode 1).
+constexpr int kRouteThreads = 1024, kRouteWarps = kRouteThreads / 32;
 template <typename T, int R>
-__global__ void __launch_bounds__(256) moe_route_row_kernel(const MoeRouteParams p) {
+__global__ void __launch_bounds__(kRouteThreads) moe_route_row_kernel(const MoeRouteParams p) {
   extern __shared__ float s_h[];   // N values of the row
   __shared__ float s_l[R * 32];
+  __shared__ float s_part[kRouteWarps][2];
   __shared__ int s_slot[kMaxTop];
   pdl_launch_dependents();
   pdl_wait();
@@ -97,37 +99,56 @@ __global__ void __launch_bounds__(256) moe_route_row_kernel(const MoeRouteParams
   const T* hr = static_cast<const T*>(p.h) + static_cast<long long>(row) * p.ldh;
   constexpr int W = Pack<T>::n;
   if (p.logits == nullptr) {
-    for (int c = threadIdx.x * W; c < p.N; c += 256 * W) {
+    for (int c = threadIdx.x * W; c < p.N; c += kRouteThreads * W) {
       float v[W];
       Pack<T>::get(hr + c, v);
 #pragma unroll
       for (int j = 0; j < W; ++j) s_h[c + j] = v[j];
     }
     __syncthreads();
-    constexpr int U = 4;   // experts per warp at a time
-    for (int e0 = warp * U; e0 < p.E; e0 += 8 * U) {
-      float acc[U] = {};
-      const T* w[U];
+    // two experts per warp; where warps are left over, several share the two experts and split the row
+    const int pairs = (p.E + 1) / 2;
+    const int ks = pairs >= kRouteWarps ? 1 : kRouteWarps / pairs;
+    for (int q0 = 0; q0 < pairs; q0 += kRouteWarps) {
+      const int q = ks == 1 ? q0 + warp : warp / ks, part = ks == 1 ? 0 : warp % ks;
+      float a0 = 0.f, a1 = 0.f;
+      if (q < pairs) {
+        const T* w0 = static_cast<const T*>(p.router) + static_cast<long long>(2 * q) * p.ldr;
+        const T* w1 = 2 * q + 1 < p.E ? w0 + p.ldr : w0;
+#pragma unroll 4
+        for (int c = (part * 32 + lane) * W; c < p.N; c += ks * 32 * W) {
+          float u[W], v[W];
+          Pack<T>::get(w0 + c, u);
+          Pack<T>::get(w1 + c, v);
 #pragma unroll
-      for (int u = 0; u < U; ++u)
-        w[u] = static_cast<const T*>(p.router) + static_cast<long long>(e0 + u < p.E ? e0 + u : p.E - 1) * p.ldr;
-      for (int c = lane * W; c < p.N; c += 32 * W) {
-        float v[U][W];
-#pragma unroll
-        for (int u = 0; u < U; ++u) Pack<T>::get(w[u] + c, v[u]);
-#pragma unroll
-        for (int u = 0; u < U; ++u)
-#pragma unroll
-          for (int j = 0; j < W; ++j) acc[u] = fmaf(v[u][j], s_h[c + j], acc[u]);
+          for (int j = 0; j < W; ++j) {
+            a0 = fmaf(u[j], s_h[c + j], a0);
+            a1 = fmaf(v[j], s_h[c + j], a1);
+          }
+        }
       }
-#pragma unroll
-      for (int u = 0; u < U; ++u) {
-        const float t = warp_sum(acc[u]);
-        if (lane == 0 && e0 + u < p.E) s_l[e0 + u] = t;
+      a0 = warp_sum(a0);
+      a1 = warp_sum(a1);
+      if (ks == 1) {
+        if (lane == 0 && q < pairs) {
+          s_l[2 * q] = a0;
+          if (2 * q + 1 < p.E) s_l[2 * q + 1] = a1;
+        }
+      } else {
+        if (lane == 0) {
+          s_part[warp][0] = a0;
+          s_part[warp][1] = a1;
+        }
+        __syncthreads();
+        for (int e = threadIdx.x; e < p.E; e += kRouteThreads) {
+          float t = 0.f;
+          for (int k = 0; k < ks; ++k) t += s_part[(e >> 1) * ks + k][e & 1];
+          s_l[e] = t;
+        }
       }
     }
   } else {
-    for (int e = threadIdx.x; e < p.E; e += 256) s_l[e] = p.logits[static_cast<long long>(row) * p.ldl + e];
+    for (int e = threadIdx.x; e < p.E; e += kRouteThreads) s_l[e] = p.logits[static_cast<long long>(row) * p.ldl + e];
   }
   __syncthreads();
   if (warp == 0) {
@@ -157,7 +178,7 @@ __global__ void __launch_bounds__(256) moe_route_row_kernel(const MoeRouteParams
     const int slot = s_slot[c];
     if (slot < 0) continue;
     T* dst = static_cast<T*>(p.xs) + static_cast<long long>(slot) * p.ldx;
-    for (int k = threadIdx.x * W; k < p.N; k += 256 * W)
+    for (int k = threadIdx.x * W; k < p.N; k += kRouteThreads * W)
       *reinterpret_cast<uint4*>(dst + k) = *reinterpret_cast<const uint4*>(hr + k);
   }
 }
@@ -302,7 +323,7 @@ cudaError_t launch_route(const MoeRouteParams& p, cudaStream_t stream) {
     return launch_kernel(moe_route_rank_kernel<R>, dim3((p.M + kRouteRows - 1) / kRouteRows), dim3(256), 0, stream, true, false, p);
   const size_t smem = p.logits == nullptr ? static_cast<size_t>(p.N) * sizeof(float) : 0;
   ensure_dynamic_smem(moe_route_row_kernel<T, R>, smem);
-  return launch_kernel(moe_route_row_kernel<T, R>, dim3(p.M), dim3(256), smem, stream, true, false, p);
+  return launch_kernel(moe_route_row_kernel<T, R>, dim3(p.M), dim3(kRouteThreads), smem, stream, true, false, p);
 }
 
 template <typename T>

@@ -11,6 +11,9 @@
 //   l_i = sum_{k <= i} log a_k inside the run:
 //       P_ij = (C_i . B_j) exp(l_i - l_j) dt_j  (j <= i)
 //       Y    = P x + exp(l_i) C S,         S <- exp(l_end) S + sum_j exp(l_end - l_j) dt_j B_j x_j^T
+//   Where sequences and heads are too few for the SMs, sequences are cut into segments: a first launch leaves every
+//   segment's own contribution to the state, a scan turns these into the states before the segments, and the walk then
+//   runs over all segments at once.
 //   x, B and C are bf16, so C B^T is exact products summed in fp32. P, S and the weighted x are fp32: each enters its
 //   product as three bf16 terms, which carry all 24 bits. An accumulator of S^T is at the same time the B-operand
 //   fragment of C S, so the state never leaves the registers between runs.
@@ -32,9 +35,37 @@ __device__ __forceinline__ int ssd_channels(const SsdParams& p) { return p.H * p
 constexpr int kDecThreads = 256;
 constexpr int kDecUnroll = 8;
 
+// Convolution of one channel at the newest token: history from the ring, `cur` goes there. TAPS 0: any number.
+template <int TAPS>
+__device__ __forceinline__ float conv_step(const SsdParams& p, const float* ring, int c, int ch, int r0, int pos, float cur) {
+  const int taps = TAPS > 0 ? TAPS : p.taps;
+  const float* w = p.conv_w + static_cast<long long>(c) * taps;
+  float acc = p.conv_b[c];
+  if constexpr (TAPS > 0) {
+    float h[TAPS], wv[TAPS];   // all loads before the first use
+#pragma unroll
+    for (int k = 1; k < TAPS; ++k) {
+      const int r = r0 >= k ? r0 - k : r0 - k + TAPS;
+      h[k] = k <= pos ? ring[static_cast<long long>(r) * ch + c] : 0.f;
+    }
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k) wv[k] = w[TAPS - 1 - k];
+    acc = fmaf(wv[0], cur, acc);
+#pragma unroll
+    for (int k = 1; k < TAPS; ++k) acc = fmaf(wv[k], h[k], acc);
+  } else {
+    acc = fmaf(w[taps - 1], cur, acc);
+    for (int k = 1; k < taps && k <= pos; ++k) {
+      const int r = r0 >= k ? r0 - k : r0 - k + taps;
+      acc = fmaf(w[taps - 1 - k], ring[static_cast<long long>(r) * ch + c], acc);
+    }
+  }
+  return silu_f(acc);
+}
+
 // grid (slices, H, rows). T: storage type, P: type of the projection rows.
-template <typename T, typename P>
-__global__ void __launch_bounds__(kDecThreads) ssd_decode_kernel(const SsdParams p) {
+template <typename T, typename P, int TAPS>
+__global__ void __launch_bounds__(kDecThreads, 3) ssd_decode_kernel(const SsdParams p) {
   extern __shared__ float s_mem[];
   const int EP = p.EP, NP = p.NP;
   const int Es = EP / static_cast<int>(gridDim.x);
@@ -77,19 +108,14 @@ __global__ void __launch_bounds__(kDecThreads) ssd_decode_kernel(const SsdParams
   float* ring = p.conv_state + static_cast<long long>(slot) * taps * ch;
   const int r0 = pos % taps;
   const bool shared_owner = head % (p.H / p.G) == 0 && blockIdx.x == 0;   // writes the inputs of B and C
+#pragma unroll 2
   for (int i = threadIdx.x; i < Es + 2 * NP; i += kDecThreads) {
     int c;                                           // channel
     if (i < Es) c = head * EP + e0 + i;
     else if (i < Es + NP) c = inner + group * NP + i - Es;
     else c = inner + p.G * NP + group * NP + i - Es - NP;
     const float cur = to_f(pr[inner + c]);
-    const float* w = p.conv_w + static_cast<long long>(c) * taps;
-    float acc = fmaf(w[taps - 1], cur, p.conv_b[c]);
-    for (int k = 1; k < taps && k <= pos; ++k) {
-      const int r = r0 >= k ? r0 - k : r0 - k + taps;
-      acc = fmaf(w[taps - 1 - k], ring[static_cast<long long>(r) * ch + c], acc);
-    }
-    s_x[i] = silu_f(acc);                            // s_x, s_b and s_c follow one another
+    s_x[i] = conv_step<TAPS>(p, ring, c, ch, r0, pos, cur);   // s_x, s_b and s_c follow one another
     if (i < Es || shared_owner) ring[static_cast<long long>(r0) * ch + c] = cur;
   }
   const float dt = softplus_f(to_f(pr[2 * inner + 2 * p.G * NP + head]) + p.dt_bias[head]);
@@ -135,13 +161,12 @@ __global__ void __launch_bounds__(kDecThreads) ssd_decode_kernel(const SsdParams
 // convolution of prompt chunks
 // ------------------------------------------------------------------------------------------------
 constexpr int kConvRows = 32;   // rows per CTA, four pieces per 128-row tile
-constexpr int kConvBatch = 8;   // rows whose loads are issued together
 
 // grid (tiles * 4, channels / 1024): four channels per thread. Only the first piece of a sequence's portion reads
 // inputs from before it (taps <= kConvRows), and the same thread writes the channel's new state after that.
 // TAPS 0: any number of taps, inputs re-read.
 template <typename T, typename P, int TAPS>
-__global__ void __launch_bounds__(256) ssd_conv_kernel(const SsdParams p) {
+__global__ void __launch_bounds__(256, 3) ssd_conv_kernel(const SsdParams p) {
   pdl_launch_dependents();
   pdl_wait();
   const int tile = blockIdx.x >> 2, piece = blockIdx.x & 3;
@@ -176,38 +201,37 @@ __global__ void __launch_bounds__(256) ssd_conv_kernel(const SsdParams p) {
   load4<float>(p.conv_b + c, b);
   const int q1 = min(q0 + kConvRows, len);
   if constexpr (TAPS > 0) {
-    float w[4][TAPS], h[TAPS][4];              // h[k]: input k + 1 rows back
+    constexpr int kConvBatch = sizeof(P) == 2 ? 8 : 4;   // rows whose loads are issued together
+    constexpr int H = TAPS - 1;                // rows of history before a batch
+    float w[4][TAPS], v[H + kConvBatch][4];
 #pragma unroll
     for (int j = 0; j < 4; ++j)
 #pragma unroll
       for (int k = 0; k < TAPS; ++k) w[j][k] = p.conv_w[static_cast<long long>(c + j) * TAPS + k];
 #pragma unroll
-    for (int k = 0; k < TAPS - 1; ++k) input(q0 - 1 - k, h[k]);
+    for (int k = 0; k < H; ++k) input(q0 - H + k, v[k]);
     for (int q = q0; q < q1; q += kConvBatch) {
-      float v[kConvBatch][4];
-#pragma unroll
-      for (int i = 0; i < kConvBatch; ++i)
-        if (q + i < q1) load4<P>(src + (q + i) * p.ld, v[i]);
 #pragma unroll
       for (int i = 0; i < kConvBatch; ++i) {
-        if (q + i < q1) {
-          float o[4];
-#pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            float acc = fmaf(w[j][TAPS - 1], v[i][j], b[j]);
-#pragma unroll
-            for (int k = 0; k < TAPS - 1; ++k) acc = fmaf(w[j][TAPS - 2 - k], h[k][j], acc);
-            o[j] = silu_f(acc);
-          }
-          store4<T>(dst + (q + i) * p.ldu, o);
-#pragma unroll
-          for (int k = TAPS - 1; k > 0; --k)
-#pragma unroll
-            for (int j = 0; j < 4; ++j) h[k][j] = h[k - 1][j];
-#pragma unroll
-          for (int j = 0; j < 4; ++j) h[0][j] = v[i][j];
-        }
+        const int qi = q + i < q1 ? q + i : q1 - 1;   // rows past the end are not stored
+        load4<P>(src + qi * p.ld, v[H + i]);
       }
+#pragma unroll
+      for (int i = 0; i < kConvBatch; ++i) {
+        float o[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          float acc = b[j];
+#pragma unroll
+          for (int k = 0; k < TAPS; ++k) acc = fmaf(w[j][k], v[i + k][j], acc);
+          o[j] = silu_as<T>(acc);
+        }
+        if (q + i < q1) store4<T>(dst + (q + i) * p.ldu, o);
+      }
+#pragma unroll
+      for (int k = 0; k < H; ++k)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[k][j] = v[kConvBatch + k][j];
     }
   } else {
     for (int q = q0; q < q1; ++q) {
@@ -219,7 +243,7 @@ __global__ void __launch_bounds__(256) ssd_conv_kernel(const SsdParams p) {
         for (int j = 0; j < 4; ++j) acc[j] = fmaf(p.conv_w[static_cast<long long>(c + j) * taps + taps - 1 - k], v[j], acc[j]);
       }
 #pragma unroll
-      for (int j = 0; j < 4; ++j) acc[j] = silu_f(acc[j]);
+      for (int j = 0; j < 4; ++j) acc[j] = silu_as<T>(acc[j]);
       store4<T>(dst + q * p.ldu, acc);
     }
   }
@@ -237,8 +261,7 @@ __global__ void __launch_bounds__(256) ssd_conv_kernel(const SsdParams p) {
 constexpr int C = 64;
 
 __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 "
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 "
       "{%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
@@ -281,12 +304,13 @@ struct RunSmem {
   static constexpr int kP = C * C * 2;                        // one term, rows of 128 bytes, 16-byte chunks swizzled
   __host__ __device__ static constexpr int x_pitch(int W) { return W * 32 + 16; }
   __host__ __device__ static constexpr int stage(int W) { return 2 * kCB + C * x_pitch(W); }
-  __host__ __device__ static constexpr int total(int W) { return 2 * stage(W) + 3 * kP + 4 * C * 4; }
+  __host__ __device__ static constexpr int total(int W) { return 2 * stage(W) + 3 * kP + 7 * C * 4; }
 };
 
-// grid (column slices, H, sequences), W warps.
-template <int NT, typename P>
-__global__ void __launch_bounds__(256) ssd_run_kernel(const SsdParams p) {
+// grid (column slices, H, sequences or tiles), W warps. PART 0: whole sequences; 1: what every segment (but a
+// sequence's last) adds to the state; 2: outputs of every segment. A segment is named by its first tile.
+template <int NT, typename P, int PART>
+__global__ void __launch_bounds__(128) ssd_run_kernel(const SsdParams p) {
   using L = RunSmem<NT>;
   extern __shared__ __align__(16) uint8_t s_raw[];
   const int W = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
@@ -297,6 +321,12 @@ __global__ void __launch_bounds__(256) ssd_run_kernel(const SsdParams p) {
   float* s_dt = s_la + C;
   float* s_ea = s_dt + C;                                                       // exp(l_i)
   float* s_w = s_ea + C;                                                        // exp(l_end - l_j) dt_j
+  // exp(l_i - l_j) dt_j of a 16 x 16 block left of the diagonal, with r the block's first row:
+  // exp(l_i - l_r) times exp(l_r - l_j) dt_j, both factors at most 1 (times dt_j)
+  float* s_row = s_w + C;                                                       // exp(l_i - l_(first row of i's block))
+  auto col_factor = [&](int mi, int j) -> float& {                              // mi 1..3, j < 16 mi: 96 values
+    return s_row[C + (mi == 1 ? 0 : (mi == 2 ? 16 : 48)) + j];
+  };
   // columns of C and B beyond the state size stay zero
   const int NP = p.NP, EP = p.EP, H = p.H;
   if (NP < L::kN)
@@ -306,16 +336,22 @@ __global__ void __launch_bounds__(256) ssd_run_kernel(const SsdParams p) {
     }
   pdl_launch_dependents();
   pdl_wait();
-  const int head = blockIdx.y, seq = blockIdx.z, e_cta = blockIdx.x * W * 16;
+  const int head = blockIdx.y, e_cta = blockIdx.x * W * 16;
+  const int tile = PART == 0 ? 0 : blockIdx.z;
+  const int seq = PART == 0 ? blockIdx.z : p.tile_seq[tile];
   const int group = head / (H / p.G);
   const int slot = p.seq_slots[seq];
   if (slot < 0 || slot >= p.num_slots) {
     if (threadIdx.x == 0) set_status_once(p.status, kStatusBadIndex);
     return;
   }
-  const int len = p.q_lens[seq];
-  if (len <= 0) return;
-  const long long row0 = p.q_start[seq];
+  const int q_first = PART == 0 ? 0 : p.tile_q0[tile];
+  if (PART != 0 && q_first % p.segment != 0) return;
+  int len = p.q_lens[seq] - q_first;           // rows of this CTA
+  const bool last = PART == 0 || len <= p.segment;
+  if (!last) len = p.segment;
+  if (len <= 0 || (PART == 1 && last)) return;
+  const long long row0 = p.q_start[seq] + q_first;
   const int inner = H * EP;
   const __nv_bfloat16* u = static_cast<const __nv_bfloat16*>(p.u) + row0 * p.ldu;
   const __nv_bfloat16* xsrc = u + head * EP + e_cta;
@@ -329,23 +365,36 @@ __global__ void __launch_bounds__(256) ssd_run_kernel(const SsdParams p) {
   auto load_stage = [&](int c) {
     const int q0 = c * C;
     const uint32_t st = smem + (c & 1) * stage_bytes;
-    const int cpr = NP >> 3;   // 16-byte chunks per row
-    for (int i = threadIdx.x; i < C * cpr; i += blockDim.x) {
-      const int r = i / cpr, k = i - r * cpr;
-      const bool in = q0 + r < len;
-      const long long off = static_cast<long long>(in ? q0 + r : 0) * p.ldu + k * 8;
-      cp_async16(st + r * L::kPitch + k * 16, csrc + off, in);
-      cp_async16(st + L::kCB + r * L::kPitch + k * 16, bsrc + off, in);
+    // thread -> 16-byte piece of a row, rows apart by the same step every time
+    {
+      const int k = threadIdx.x % NT, dr = blockDim.x / NT;
+      int r = threadIdx.x / NT;
+      if (k * 8 < NP) {
+        const long long step = dr * p.ldu;
+        long long off = (q0 + r) * p.ldu + k * 8;
+        uint32_t dst = st + r * L::kPitch + k * 16;
+        for (; r < C; r += dr, off += step, dst += dr * L::kPitch) {
+          const bool in = q0 + r < len;
+          if constexpr (PART != 1) cp_async16(dst, in ? csrc + off : csrc, in);
+          cp_async16(dst + L::kCB, in ? bsrc + off : bsrc, in);
+        }
+      }
     }
-    const int xpr = W * 2;
-    for (int i = threadIdx.x; i < C * xpr; i += blockDim.x) {
-      const int r = i / xpr, k = i - r * xpr;
-      const bool in = q0 + r < len && k * 8 < x_cols;
-      cp_async16(st + 2 * L::kCB + r * xp + k * 16, in ? xsrc + static_cast<long long>(q0 + r) * p.ldu + k * 8 : xsrc, in);
+    {
+      const int k = threadIdx.x % (2 * W), dr = 16;   // 2 W pieces per row, 32 W threads
+      int r = threadIdx.x / (2 * W);
+      const bool cols = k * 8 < x_cols;
+      long long off = (q0 + r) * p.ldu + k * 8;
+      uint32_t dst = st + 2 * L::kCB + r * xp + k * 16;
+#pragma unroll
+      for (int i = 0; i < C / 16; ++i, r += dr, off += dr * p.ldu, dst += dr * xp) {
+        const bool in = cols && q0 + r < len;
+        cp_async16(dst, in ? xsrc + off : xsrc, in);
+      }
     }
     cp_commit();
   };
-  float dt_next[2];            // warp 0: raw step sizes of rows 2 lane, 2 lane + 1 of the next run
+  float dt_next[2];            // last warp: raw step sizes of rows 2 lane, 2 lane + 1 of the next run
   auto load_dt = [&](int c) {
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
@@ -354,19 +403,22 @@ __global__ void __launch_bounds__(256) ssd_run_kernel(const SsdParams p) {
     }
   };
   load_stage(0);
-  if (warp == 0) load_dt(0);
+  if (warp == W - 1) load_dt(0);
 
   const int e_w = e_cta + warp * 16;   // this warp's columns
   const bool active = e_w < EP;
   float S[NT][4];                      // S^T: rows e_w + g (+ 8), columns 8 i + 2 t (+ 1)
   float* st_g = p.state + (static_cast<long long>(slot) * H + head) * NP * EP + e_w + g;
-  const bool past = p.ctx_lens[seq] != len;
+  float* ws_g = PART == 0 ? nullptr : p.ws + (static_cast<long long>(tile) * H + head) * NP * EP + e_w + g;
+  const float* from = PART == 2 ? ws_g : st_g;
+  const bool past = PART == 2 || (PART == 0 && p.ctx_lens[seq] != len);
+  float decay_all = 1.f;               // over the rows of this CTA
 #pragma unroll
   for (int i = 0; i < NT; ++i) {
 #pragma unroll
     for (int x = 0; x < 4; ++x) {
       const int n = i * 8 + 2 * t + (x & 1);
-      S[i][x] = (past && active && n < NP) ? st_g[static_cast<long long>(n) * EP + (x >> 1) * 8] : 0.f;
+      S[i][x] = (past && active && n < NP) ? from[static_cast<long long>(n) * EP + (x >> 1) * 8] : 0.f;
     }
   }
   // fragment addresses: 8x8 matrices of an x4 load, rows lane & 7 of matrix lane / 8
@@ -376,17 +428,17 @@ __global__ void __launch_bounds__(256) ssd_run_kernel(const SsdParams p) {
 
   __nv_bfloat16* yrow = static_cast<__nv_bfloat16*>(p.y) + row0 * p.ldy + head * EP + e_w;
   for (int c = 0; c < n_runs; ++c) {
-    const int n = min(C, len - c * C);
+    const int n = min(C, len - c * C);   // rows past the end are zero and have step 0: they change nothing
     cp_wait<0>();
     __syncthreads();   // this run's stage has landed, the other stage and P have been read
     const float raw0 = dt_next[0], raw1 = dt_next[1];
     if (c + 1 < n_runs) {
       load_stage(c + 1);
-      if (warp == 0) load_dt(c + 1);
+      if (warp == W - 1) load_dt(c + 1);
     }
     const uint32_t sC = smem + (c & 1) * stage_bytes, sB = sC + L::kCB, sX = sB + L::kCB;
-    if (warp == 0) {
-      // step sizes and running log decays; rows past the end have step 0 and change nothing
+    if (warp == W - 1) {
+      // step sizes and running log decays
       const float d0 = 2 * lane < n ? softplus_f(raw0 + dt_bias) : 0.f;
       const float d1 = 2 * lane + 1 < n ? softplus_f(raw1 + dt_bias) : 0.f;
       const float l0 = -A * d0, pair = l0 - A * d1;
@@ -407,36 +459,67 @@ __global__ void __launch_bounds__(256) ssd_run_kernel(const SsdParams p) {
       s_ea[2 * lane + 1] = expf(la1);
       s_w[2 * lane] = expf(end - la0) * d0;
       s_w[2 * lane + 1] = expf(end - la1) * d1;
-    }
-    // ---- C B^T of this warp's 16 x 16 blocks on and below the diagonal ----
-    constexpr int kItems = 10;
-    for (int it0 = warp; it0 < kItems || it0 == warp; it0 += W) {
-      float cb[2][4] = {};
-      int mi = 0, nj = it0;
-      while (nj > mi) {
-        nj -= mi + 1;
-        ++mi;
-      }
-      if (it0 < kItems) {
+      if constexpr (PART != 1) {
+        const float ref = __shfl_sync(0xffffffffu, la0, lane & 24);   // first row of this row's block
+        s_row[2 * lane] = expf(la0 - ref);
+        s_row[2 * lane + 1] = expf(la1 - ref);
 #pragma unroll
-        for (int k = 0; k < NT / 2; ++k) {
-          uint32_t a[4], b[4];
-          ldsm4(sC + (mi * 16 + row_a) * L::kPitch + k * 32 + col_a, a);
-          ldsm4(sB + (nj * 16 + row_b) * L::kPitch + k * 32 + col_b, b);
-          mma_bf16(cb[0], a[0], a[1], a[2], a[3], b[0], b[1]);
-          mma_bf16(cb[1], a[0], a[1], a[2], a[3], b[2], b[3]);
+        for (int mi = 1; mi < 4; ++mi) {
+          const float lr = __shfl_sync(0xffffffffu, la0, mi * 8);
+          if (lane < mi * 8) {
+            col_factor(mi, 2 * lane) = expf(lr - la0) * d0;
+            col_factor(mi, 2 * lane + 1) = expf(lr - la1) * d1;
+          }
         }
       }
+    }
+    // ---- C B^T of this warp's 16 x 16 blocks on and below the diagonal, kPar of them at a time ----
+    constexpr int kItems = 10, kPar = 3;
+    if constexpr (PART == 1) __syncthreads();   // step sizes are there
+    for (int it0 = PART == 1 ? kItems : warp; it0 < kItems; it0 += kPar * W) {
+      float cb[kPar][2][4] = {};
+      int mis[kPar], njs[kPar];
+#pragma unroll
+      for (int y = 0; y < kPar; ++y) {
+        const int it = it0 + y * W;
+        mis[y] = 0;
+        njs[y] = it < kItems ? it : 0;
+        while (njs[y] > mis[y]) {
+          njs[y] -= mis[y] + 1;
+          ++mis[y];
+        }
+      }
+#pragma unroll
+      for (int k = 0; k < NT / 2; ++k)
+#pragma unroll
+        for (int y = 0; y < kPar; ++y)
+        {   // (a block past the last one repeats the first and is not used)
+          uint32_t a[4], b[4];
+          ldsm4(sC + (mis[y] * 16 + row_a) * L::kPitch + k * 32 + col_a, a);
+          ldsm4(sB + (njs[y] * 16 + row_b) * L::kPitch + k * 32 + col_b, b);
+          mma_bf16(cb[y][0], a[0], a[1], a[2], a[3], b[0], b[1]);
+          mma_bf16(cb[y][1], a[0], a[1], a[2], a[3], b[2], b[3]);
+        }
       if (it0 == warp) __syncthreads();   // step sizes are there (every warp passes here once)
-      if (it0 < kItems) {
+#pragma unroll
+      for (int y = 0; y < kPar; ++y) {
+        const int mi = mis[y], nj = njs[y];
+        if (it0 + y * W >= kItems) continue;
 #pragma unroll
         for (int h = 0; h < 2; ++h)
 #pragma unroll
           for (int r = 0; r < 2; ++r) {
             const int i = mi * 16 + g + r * 8, j = nj * 16 + h * 8 + 2 * t;
-            const float li = s_la[i];
-            const float v0 = j <= i ? cb[h][2 * r] * expf(li - s_la[j]) * s_dt[j] : 0.f;
-            const float v1 = j + 1 <= i ? cb[h][2 * r + 1] * expf(li - s_la[j + 1]) * s_dt[j + 1] : 0.f;
+            float v0, v1;
+            if (nj < mi) {
+              const float f = s_row[i];
+              v0 = cb[y][h][2 * r] * (f * col_factor(mi, j));
+              v1 = cb[y][h][2 * r + 1] * (f * col_factor(mi, j + 1));
+            } else {
+              const float li = s_la[i];
+              v0 = j <= i ? cb[y][h][2 * r] * (expf(li - s_la[j]) * s_dt[j]) : 0.f;
+              v1 = j + 1 <= i ? cb[y][h][2 * r + 1] * (expf(li - s_la[j + 1]) * s_dt[j + 1]) : 0.f;
+            }
             uint32_t tm[3];
             split3(v0, v1, tm);
             const uint32_t off = i * 128 + (((j >> 3) ^ (i & 7)) << 4) + (j & 7) * 2;
@@ -448,7 +531,7 @@ __global__ void __launch_bounds__(256) ssd_run_kernel(const SsdParams p) {
     }
     // ---- exp(l_i) C S ----
     float Y[4][2][4] = {};
-    if (active) {
+    if (PART != 1 && active) {
 #pragma unroll
       for (int k = 0; k < NT / 2; ++k) {
         uint32_t b[2][2][3];   // [column tile][k half][term]
@@ -456,16 +539,17 @@ __global__ void __launch_bounds__(256) ssd_run_kernel(const SsdParams p) {
         for (int h = 0; h < 2; ++h)
 #pragma unroll
           for (int q = 0; q < 2; ++q) split3(S[2 * k + q][2 * h], S[2 * k + q][2 * h + 1], b[h][q]);
+        uint32_t a[4][4];
 #pragma unroll
-        for (int mi = 0; mi < 4; ++mi) {
-          if (mi * 16 >= n) continue;
-          uint32_t a[4];
-          ldsm4(sC + (mi * 16 + row_a) * L::kPitch + k * 32 + col_a, a);
+        for (int mi = 0; mi < 4; ++mi)
+          ldsm4(sC + (mi * 16 + row_a) * L::kPitch + k * 32 + col_a, a[mi]);
+        // eight independent products between two of one accumulator
 #pragma unroll
-          for (int h = 0; h < 2; ++h)
+        for (int x = 2; x >= 0; --x)
 #pragma unroll
-            for (int x = 2; x >= 0; --x) mma_bf16(Y[mi][h], a[0], a[1], a[2], a[3], b[h][0][x], b[h][1][x]);
-        }
+          for (int mi = 0; mi < 4; ++mi)
+#pragma unroll
+            for (int h = 0; h < 2; ++h) mma_bf16(Y[mi][h], a[mi][0], a[mi][1], a[mi][2], a[mi][3], b[h][0][x], b[h][1][x]);
       }
 #pragma unroll
       for (int mi = 0; mi < 4; ++mi) {
@@ -479,7 +563,8 @@ __global__ void __launch_bounds__(256) ssd_run_kernel(const SsdParams p) {
         }
       }
     }
-    __syncthreads();   // P is there
+    if constexpr (PART != 1) __syncthreads();   // P is there
+    if constexpr (PART == 1) decay_all *= s_ea[C - 1];
     if (active) {
       const float a_end = s_ea[C - 1];
 #pragma unroll
@@ -488,24 +573,21 @@ __global__ void __launch_bounds__(256) ssd_run_kernel(const SsdParams p) {
         for (int x = 0; x < 4; ++x) S[i][x] *= a_end;
 #pragma unroll
       for (int kj = 0; kj < 4; ++kj) {
-        if (kj * 16 >= n) continue;
         // x rows of this block as B operand [k = j][n = e] and, transposed, as A operand [m = e][k = j]
         uint32_t xb[4];
         ldsm4t(sX + (kj * 16 + row_a) * xp + warp * 32 + col_a, xb);   // (j lo, e lo) (j hi, e lo) (j lo, e hi) (j hi, e hi)
         // ---- Y += P x ----
 #pragma unroll
-        for (int mi = kj; mi < 4; ++mi) {
-          if (mi * 16 >= n) continue;
-          const int pr = mi * 16 + row_a;
-          const uint32_t pa = sP + pr * 128 + (((kj * 2 + (col_a >> 4)) ^ (pr & 7)) << 4);
+        for (int x = 2; x >= 0; --x)
 #pragma unroll
-          for (int x = 2; x >= 0; --x) {
-            uint32_t a[4];
-            ldsm4(pa + x * L::kP, a);
-            mma_bf16(Y[mi][0], a[0], a[1], a[2], a[3], xb[0], xb[1]);
-            mma_bf16(Y[mi][1], a[0], a[1], a[2], a[3], xb[2], xb[3]);
-          }
-        }
+          for (int mi = kj; mi < 4; ++mi)
+            if (PART != 1) {
+              const int pr = mi * 16 + row_a;
+              uint32_t a[4];
+              ldsm4(sP + x * L::kP + pr * 128 + (((kj * 2 + (col_a >> 4)) ^ (pr & 7)) << 4), a);
+              mma_bf16(Y[mi][0], a[0], a[1], a[2], a[3], xb[0], xb[1]);
+              mma_bf16(Y[mi][1], a[0], a[1], a[2], a[3], xb[2], xb[3]);
+            }
         // ---- S^T += (w_j x_j)^T B_j ----
         uint32_t av[4][3];   // A fragments: (e lo, j lo) (e hi, j lo) (e lo, j hi) (e hi, j hi)
         const int j0 = kj * 16 + 2 * t;
@@ -517,15 +599,19 @@ __global__ void __launch_bounds__(256) ssd_run_kernel(const SsdParams p) {
         weigh(xb[2], w0, w1, av[1]);
         weigh(xb[1], w2, w3, av[2]);
         weigh(xb[3], w2, w3, av[3]);
+        constexpr int kPairs = NT >= 8 ? 4 : NT / 2;   // pairs of column tiles at a time
 #pragma unroll
-        for (int i = 0; i < NT; i += 2) {
-          uint32_t b[4];
-          ldsm4t(sB + (kj * 16 + row_a) * L::kPitch + i * 16 + col_a, b);   // (j lo, n lo) (j hi, n lo) (j lo, n hi) (j hi, n hi)
+        for (int i = 0; i < NT; i += 2 * kPairs) {
+          uint32_t b[kPairs][4];   // (j lo, n lo) (j hi, n lo) (j lo, n hi) (j hi, n hi)
 #pragma unroll
-          for (int x = 2; x >= 0; --x) {
-            mma_bf16(S[i], av[0][x], av[1][x], av[2][x], av[3][x], b[0], b[1]);
-            mma_bf16(S[i + 1], av[0][x], av[1][x], av[2][x], av[3][x], b[2], b[3]);
-          }
+          for (int q = 0; q < kPairs; ++q) ldsm4t(sB + (kj * 16 + row_a) * L::kPitch + (i + 2 * q) * 16 + col_a, b[q]);
+#pragma unroll
+          for (int x = 2; x >= 0; --x)
+#pragma unroll
+            for (int q = 0; q < kPairs; ++q) {
+              mma_bf16(S[i + 2 * q], av[0][x], av[1][x], av[2][x], av[3][x], b[q][0], b[q][1]);
+              mma_bf16(S[i + 2 * q + 1], av[0][x], av[1][x], av[2][x], av[3][x], b[q][2], b[q][3]);
+            }
         }
       }
       // ---- Y + D x ----
@@ -534,7 +620,7 @@ __global__ void __launch_bounds__(256) ssd_run_kernel(const SsdParams p) {
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
           const int i = mi * 16 + g + r * 8;
-          if (i >= n) continue;
+          if (PART == 1 || i >= n) continue;
 #pragma unroll
           for (int h = 0; h < 2; ++h) {
             const int e = h * 8 + 2 * t;
@@ -547,13 +633,52 @@ __global__ void __launch_bounds__(256) ssd_run_kernel(const SsdParams p) {
         }
     }
   }
-  if (active) {
+  if (active && (PART == 1 || last)) {
+    float* to = PART == 1 ? ws_g : st_g;
 #pragma unroll
     for (int i = 0; i < NT; ++i)
 #pragma unroll
       for (int x = 0; x < 4; ++x) {
         const int nn = i * 8 + 2 * t + (x & 1);
-        if (nn < NP) st_g[static_cast<long long>(nn) * EP + (x >> 1) * 8] = S[i][x];
+        if (nn < NP) to[static_cast<long long>(nn) * EP + (x >> 1) * 8] = S[i][x];
+      }
+  }
+  if (PART == 1 && threadIdx.x == 0 && blockIdx.x == 0) p.ws_decay[static_cast<long long>(tile) * H + head] = decay_all;
+}
+
+// Contributions of the segments -> states before the segments. grid (NP EP / 1024, H, sequences).
+__global__ void __launch_bounds__(256) ssd_segment_scan_kernel(const SsdParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int seq = blockIdx.z, head = blockIdx.y;
+  const long long ne = static_cast<long long>(p.NP) * p.EP;
+  const long long i0 = (static_cast<long long>(blockIdx.x) * 256 + threadIdx.x) * 4;
+  if (i0 >= ne) return;
+  const int slot = p.seq_slots[seq], len = p.q_lens[seq];
+  if (slot < 0 || slot >= p.num_slots) return;
+  int tile0 = 0;
+  for (int s = 0; s < seq; ++s) tile0 += (p.q_lens[s] + 127) >> 7;
+  const int n_seg = (len + p.segment - 1) / p.segment, per = p.segment >> 7;
+  float S[4] = {0.f, 0.f, 0.f, 0.f};
+  if (p.ctx_lens[seq] != len) load4<float>(p.state + (static_cast<long long>(slot) * p.H + head) * ne + i0, S);
+  constexpr int U = 4;   // segments whose loads are issued together
+  for (int s0 = 0; s0 < n_seg; s0 += U) {
+    float u[U][4], a[U];
+#pragma unroll
+    for (int k = 0; k < U; ++k)
+      if (s0 + k < n_seg - 1) {
+        const long long at = static_cast<long long>(tile0 + (s0 + k) * per) * p.H + head;
+        load4<float>(p.ws + at * ne + i0, u[k]);
+        a[k] = p.ws_decay[at];
+      }
+#pragma unroll
+    for (int k = 0; k < U; ++k)
+      if (s0 + k < n_seg) {
+        store4<float>(p.ws + (static_cast<long long>(tile0 + (s0 + k) * per) * p.H + head) * ne + i0, S);
+        if (s0 + k < n_seg - 1) {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) S[j] = fmaf(a[k], S[j], u[k][j]);
+        }
       }
   }
 }
@@ -616,16 +741,18 @@ __global__ void __launch_bounds__(256) ssd_scan_kernel(const SsdParams p) {
 // ------------------------------------------------------------------------------------------------
 // gate and norm
 // ------------------------------------------------------------------------------------------------
-// TPG threads per (row, part); the gated values of a part wait in shared memory for its root mean square.
-template <typename T, typename P, int TPG>
+// One (row, part) per CTA, or per warp (WARPS) where a part is small; the gated values of a part wait in shared
+// memory for its root mean square.
+template <typename T, typename P, bool WARPS>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const GatedNormParams p) {
   extern __shared__ __align__(16) float s_mem[];
   __shared__ float s_red[32];
   pdl_launch_dependents();
   pdl_wait();
   const int inner = p.H * p.E, part = inner / p.groups;
-  const int sub = threadIdx.x / TPG, tid = threadIdx.x % TPG;
-  const long long item = static_cast<long long>(blockIdx.x) * (256 / TPG) + sub;
+  const int TPG = WARPS ? 32 : blockDim.x;
+  const int sub = WARPS ? threadIdx.x >> 5 : 0, tid = WARPS ? threadIdx.x & 31 : threadIdx.x;
+  const long long item = WARPS ? static_cast<long long>(blockIdx.x) * 8 + sub : blockIdx.x;
   const bool on = item < static_cast<long long>(p.M) * p.groups;
   const long long row = on ? item / p.groups : 0;
   const int c0 = on ? static_cast<int>(item - row * p.groups) * part : 0;
@@ -637,13 +764,14 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const GatedNormParams p
   float ss = 0.f;
   if (on) {
     if (vec) {
+#pragma unroll 4
       for (int c = tid * 4; c < part; c += TPG * 4) {
         float a[4], b[4];
         load4<T>(y + c0 + c, a);
         load4<P>(z + c0 + c, b);
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-          a[j] *= silu_f(b[j]);
+          a[j] *= silu_as<T>(b[j]);
           ss = fmaf(a[j], a[j], ss);
         }
         store4<float>(s_g + c, a);
@@ -651,13 +779,13 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const GatedNormParams p
     } else {
       for (int c = tid; c < part; c += TPG) {
         const int h = (c0 + c) / p.E, k = h * p.EP + (c0 + c) - h * p.E;
-        const float a = to_f(y[k]) * silu_f(to_f(z[k]));
+        const float a = to_f(y[k]) * silu_as<T>(to_f(z[k]));
         ss = fmaf(a, a, ss);
         s_g[c] = a;
       }
     }
   }
-  const float total = TPG == 32 ? warp_sum(ss) : block_sum_all(ss, s_red);
+  const float total = WARPS ? warp_sum(ss) : block_sum_all(ss, s_red);
   if (!on) return;
   const float r = 1.f / sqrtf(total / static_cast<float>(part) + p.eps);
   if (vec) {
@@ -679,8 +807,9 @@ cudaError_t launch_decode(const SsdParams& p, int slices, cudaStream_t stream) {
   const int Es = p.EP / slices, groups = Es >> 2;
   const int gt = groups < kDecThreads ? groups : kDecThreads, lanes = kDecThreads / gt;
   const size_t smem = (Es + 2 * static_cast<size_t>(p.NP) + static_cast<size_t>(lanes) * Es) * sizeof(float);
-  ensure_dynamic_smem(ssd_decode_kernel<T, P>, smem);
-  return launch_kernel(ssd_decode_kernel<T, P>, dim3(slices, p.H, p.rows), dim3(kDecThreads), smem, stream, true, false, p);
+  auto kern = p.taps == 4 ? ssd_decode_kernel<T, P, 4> : ssd_decode_kernel<T, P, 0>;
+  ensure_dynamic_smem(kern, smem);
+  return launch_kernel(kern, dim3(slices, p.H, p.rows), dim3(kDecThreads), smem, stream, true, false, p);
 }
 
 template <typename T, typename P>
@@ -691,16 +820,26 @@ cudaError_t launch_conv(const SsdParams& p, cudaStream_t stream) {
   return launch_kernel(ssd_conv_kernel<T, P, 0>, grid, dim3(256), 0, stream, true, false, p);
 }
 
+int run_warps(int EP) { return EP / 16 < 2 ? 1 : (EP / 16 < 4 ? 2 : 4); }   // of 16 columns each
+
 template <int NT, typename P>
 cudaError_t launch_run(const SsdParams& p, cudaStream_t stream) {
-  // four warps (64 columns) per CTA; two where that would leave SMs idle
-  int W = p.EP / 16 < 4 ? p.EP / 16 : 4;
-  const int slices4 = (p.EP + W * 16 - 1) / (W * 16);
-  if (W == 4 && slices4 * p.H * p.n_seqs < sm_count()) W = 2;
+  const int W = run_warps(p.EP);
   const size_t smem = RunSmem<NT>::total(W);
-  ensure_dynamic_smem(ssd_run_kernel<NT, P>, smem);
-  const dim3 grid((p.EP + W * 16 - 1) / (W * 16), p.H, p.n_seqs);
-  return launch_kernel(ssd_run_kernel<NT, P>, grid, dim3(W * 32), smem, stream, true, false, p);
+  const int slices = (p.EP + W * 16 - 1) / (W * 16);
+  if (p.segment <= 0) {
+    ensure_dynamic_smem(ssd_run_kernel<NT, P, 0>, smem);
+    return launch_kernel(ssd_run_kernel<NT, P, 0>, dim3(slices, p.H, p.n_seqs), dim3(W * 32), smem, stream, true, false, p);
+  }
+  ensure_dynamic_smem(ssd_run_kernel<NT, P, 1>, smem);
+  ensure_dynamic_smem(ssd_run_kernel<NT, P, 2>, smem);
+  const dim3 grid(slices, p.H, p.n_tiles);
+  cudaError_t e = launch_kernel(ssd_run_kernel<NT, P, 1>, grid, dim3(W * 32), smem, stream, true, false, p);
+  if (e != cudaSuccess) return e;
+  const dim3 sgrid((p.NP * p.EP + 1023) / 1024, p.H, p.n_seqs);
+  e = launch_kernel(ssd_segment_scan_kernel, sgrid, dim3(256), 0, stream, true, false, p);
+  if (e != cudaSuccess) return e;
+  return launch_kernel(ssd_run_kernel<NT, P, 2>, grid, dim3(W * 32), smem, stream, true, false, p);
 }
 template <typename P>
 cudaError_t run_of(const SsdParams& p, cudaStream_t stream) {
@@ -723,19 +862,29 @@ template <typename T, typename P>
 cudaError_t launch_gated(const GatedNormParams& p, cudaStream_t stream) {
   const int part = p.H * p.E / p.groups;
   const long long items = static_cast<long long>(p.M) * p.groups;
-  if (part <= 512) {
+  if (part <= 128 || (part <= 1024 && items >= 32ll * sm_count())) {
     const size_t smem = 8 * static_cast<size_t>(part) * sizeof(float);
-    return launch_kernel(gated_norm_kernel<T, P, 32>, dim3(static_cast<unsigned>((items + 7) / 8)), dim3(256), smem, stream, true,
+    return launch_kernel(gated_norm_kernel<T, P, true>, dim3(static_cast<unsigned>((items + 7) / 8)), dim3(256), smem, stream, true,
                          false, p);
   }
   const size_t smem = static_cast<size_t>(part) * sizeof(float);
-  ensure_dynamic_smem(gated_norm_kernel<T, P, 256>, smem);
-  return launch_kernel(gated_norm_kernel<T, P, 256>, dim3(static_cast<unsigned>(items)), dim3(256), smem, stream, true, false, p);
+  ensure_dynamic_smem(gated_norm_kernel<T, P, false>, smem);
+  const int threads = part >= 1024 ? 256 : (part / 4 + 31) / 32 * 32;
+  return launch_kernel(gated_norm_kernel<T, P, false>, dim3(static_cast<unsigned>(items)), dim3(threads), smem, stream, true, false, p);
 }
 
 }  // namespace
 
 bool ssd_chunks_ok(int NP) { return NP <= 256; }
+
+int ssd_segment(int H, int EP, int n_tiles, int n_seqs) {
+  const int W = run_warps(EP), slices = (EP + W * 16 - 1) / (W * 16);
+  const int slots = 2 * sm_count();   // CTAs that run at a time
+  if (static_cast<long long>(slices) * H * n_seqs * 4 >= 3ll * slots || n_tiles < 3 * n_seqs) return 0;
+  int seg = 256;
+  while (seg < 2048 && static_cast<long long>(n_tiles) * 128 / seg * slices * H > 4ll * slots) seg *= 2;
+  return seg;
+}
 
 cudaError_t launch_ssd_decode(const SsdParams& p, int dtype, cudaStream_t stream) {
   if (p.rows <= 0) return cudaSuccess;

@@ -184,30 +184,35 @@ cudaError_t launch_t(const StreamNormParams& p, cudaStream_t stream) {
 
 // Layers whose mixer and feed-forward run side by side: V values per piece, CH pieces per thread that stay in
 // registers (CH = 0: any row length, the row goes through shared memory).
-template <typename T>
-__device__ __forceinline__ float4 expert_sum4(const BranchNormParams& p, int row, int c) {
-  float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-  for (int k = 0; k < p.top; ++k) {
+// The chosen experts' rows of a token wait in shared memory as (row, weight): a row outside the buffer weighs nothing.
+struct ChosenRow {
+  int row;
+  float weight;
+};
+__device__ __forceinline__ void chosen_rows(const BranchNormParams& p, int row, ChosenRow* s_e) {
+  for (int k = threadIdx.x; k < p.top; k += blockDim.x) {
     const int s = p.e_slot[row * p.top + k];
-    if (s < 0 || s >= p.n_e_rows) continue;
-    const float wk = p.e_weight[row * p.top + k];
-    float v[4];
-    load4<T>(static_cast<const T*>(p.e_rows) + static_cast<long long>(s) * p.lde + c, v);
-    a.x = fmaf(wk, v[0], a.x);
-    a.y = fmaf(wk, v[1], a.y);
-    a.z = fmaf(wk, v[2], a.z);
-    a.w = fmaf(wk, v[3], a.w);
+    const bool ok = s >= 0 && s < p.n_e_rows;
+    s_e[k] = {ok ? s : 0, ok ? p.e_weight[row * p.top + k] : 0.f};
   }
-  return a;
 }
 template <typename T>
-__device__ __forceinline__ float expert_sum(const BranchNormParams& p, int row, int c) {
-  float a = 0.f;
+__device__ __forceinline__ void expert_sum4(const BranchNormParams& p, const ChosenRow* s_e, int c, float (&a)[4]) {
+  const T* rows = static_cast<const T*>(p.e_rows) + c;
+#pragma unroll 8
   for (int k = 0; k < p.top; ++k) {
-    const int s = p.e_slot[row * p.top + k];
-    if (s < 0 || s >= p.n_e_rows) continue;
-    a = fmaf(p.e_weight[row * p.top + k], to_f(static_cast<const T*>(p.e_rows)[static_cast<long long>(s) * p.lde + c]), a);
+    const ChosenRow e = s_e[k];
+    float v[4];
+    load4<T>(rows + static_cast<long long>(e.row) * p.lde, v);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) a[j] = fmaf(e.weight, v[j], a[j]);
   }
+}
+template <typename T>
+__device__ __forceinline__ float expert_sum(const BranchNormParams& p, const ChosenRow* s_e, int c) {
+  float a = 0.f;
+  for (int k = 0; k < p.top; ++k)
+    a = fmaf(s_e[k].weight, to_f(static_cast<const T*>(p.e_rows)[static_cast<long long>(s_e[k].row) * p.lde + c]), a);
   return a;
 }
 // sums of both branches at once over the block
@@ -227,12 +232,17 @@ template <typename T, int CH>
 __global__ void __launch_bounds__(CH == 4 ? 512 : 1024) branch_norm_kernel(const BranchNormParams p) {
   __shared__ float s_red[32];
   __shared__ float2 s_red2[32];
+  __shared__ ChosenRow s_e[kMaxTop];
   pdl_launch_dependents();
   pdl_wait();
   const int N = p.N;
   const float inv_n = 1.f / static_cast<float>(N);
   for (int row = blockIdx.x; row < p.rows; row += gridDim.x) {
     float* xr = p.x + static_cast<long long>(row) * N;
+    if (p.e_rows != nullptr) {
+      __syncthreads();               // the row before has been read out
+      chosen_rows(p, row, s_e);      // published by the barriers of the branches' sums
+    }
     if (p.clear != nullptr) {
       float* z = p.clear + static_cast<long long>(row) * p.clear_ld;
       for (int c = threadIdx.x * 4; c < p.clear_n; c += blockDim.x * 4)
@@ -298,13 +308,7 @@ __global__ void __launch_bounds__(CH == 4 ? 512 : 1024) branch_norm_kernel(const
             if (p.clear_y[b])
               *reinterpret_cast<float4*>(p.y[b] + static_cast<long long>(row) * p.ldy + c) = make_float4(0.f, 0.f, 0.f, 0.f);
           }
-        if (p.e_rows != nullptr) {
-          const float4 e = expert_sum4<T>(p, row, c);
-          a[0] += e.x;
-          a[1] += e.y;
-          a[2] += e.z;
-          a[3] += e.w;
-        }
+        if (p.e_rows != nullptr) expert_sum4<T>(p, s_e, c, a);
 #pragma unroll
         for (int j = 0; j < 4; ++j) x[k][j] += a[j];
       }
@@ -343,12 +347,17 @@ __global__ void __launch_bounds__(256) branch_norm_any_kernel(const BranchNormPa
   extern __shared__ float s_u[];  // N values of the row
   __shared__ float s_red[32];
   __shared__ float2 s_red2[32];
+  __shared__ ChosenRow s_e[kMaxTop];
   pdl_launch_dependents();
   pdl_wait();
   const int N = p.N;
   const float inv_n = 1.f / static_cast<float>(N);
   for (int row = blockIdx.x; row < p.rows; row += gridDim.x) {
     float* xr = p.x + static_cast<long long>(row) * N;
+    if (p.e_rows != nullptr) {
+      __syncthreads();
+      chosen_rows(p, row, s_e);
+    }
     if (p.clear != nullptr)
       for (int c = threadIdx.x; c < p.clear_n; c += blockDim.x) p.clear[static_cast<long long>(row) * p.clear_ld + c] = 0.f;
     const int dst = p.row_map != nullptr ? p.row_map[row] : row;
@@ -378,7 +387,7 @@ __global__ void __launch_bounds__(256) branch_norm_any_kernel(const BranchNormPa
       if (er != nullptr) {
         x = to_f(er[c]) * p.embed_scale;
       } else {
-        x = p.e_rows != nullptr ? expert_sum<T>(p, row, c) : 0.f;
+        x = p.e_rows != nullptr ? expert_sum<T>(p, s_e, c) : 0.f;
 #pragma unroll
         for (int b = 0; b < kMaxBranches; ++b)
           if (b < p.n_branches) {

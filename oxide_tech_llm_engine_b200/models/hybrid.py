@@ -171,6 +171,9 @@ class SsdRun:
         if nd > 0:
             hops.ssd_decode(proj, nd, row_slots=s.decode_slots, positions=s.positions, **kw)
         if s.n_prefill > 0:
+            seg = hops.ssd_segment(r.heads, r.vdim_p, s.n_tiles, s.n_prefill) if self.runs else 0
+            if seg:
+                kw.update(segment=seg, ws=m.scratch("ssd_ws", hops.ssd_ws_elems(r.heads, r.vdim_p, r.state_p, s.n_tiles)))
             hops.ssd_prefill(proj, M, seq_slots=s.prefill_slots, tile_seq=s.tile_seq, tile_q0=s.tile_q0, q_start=s.q_start,
                              q_lens=s.q_lens, ctx_lens=s.ctx_lens, n_tiles=s.n_tiles, n_seqs=s.n_prefill,
                              u=m.buffer(("ssd_u", r.channels_p), r.channels_p), runs=self.runs, **kw)
@@ -403,7 +406,10 @@ class HybridModel(GemmShapes):
 
     def group_bn(self, m_tiles: int, n: int) -> int:
         """Tile width of an expert GEMM: narrow while the tiles would not fill the SMs."""
-        return 64 if m_tiles * ((n + 127) // 128) < self._sms else 128
+        for bn in (256, 128):
+            if m_tiles * ((n + bn - 1) // bn) >= self._sms:
+                return bn
+        return 64
 
     def buffer(self, key: tuple, width: int) -> torch.Tensor:
         """[max_tokens, width] activation rows of one layout. Columns that no kernel of that layout writes

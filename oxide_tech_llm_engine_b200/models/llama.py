@@ -221,7 +221,7 @@ class DeviceModel(GemmShapes):
             self.cap = (M + 127) // 128 * 128 if weight_mode == "nvfp4" else M
             specs["slab"] = ((self.e_l, self.cap, d), "bf16")
             specs["meta"] = ((self.e_l, self.cap, 4), "i32")
-            specs["cnt"] = ((16,), "i32")
+            specs["cnt"] = ((max(16, self.e_l),), "i32")
         self.ws = SymmetricWorkspace(specs, rank=rank, world=world, group=group, device=dev)
         self.tickets = torch.zeros(16, dtype=torch.int32, device=dev)
         bf = dict(dtype=torch.bfloat16, device=dev)

@@ -102,6 +102,15 @@ def ssd_chunks_ok(n: int) -> bool:
     return bool(hybrid_ext().ssd_chunks_ok(n))
 
 
+def ssd_segment(h: int, ep: int, n_tiles: int, n_seqs: int) -> int:
+    """Rows per segment for a step of so many tiles and sequences; 0: sequences are walked whole."""
+    return int(hybrid_ext().ssd_segment(h, ep, n_tiles, n_seqs))
+
+
+def ssd_ws_elems(h: int, ep: int, np_: int, n_tiles: int) -> int:
+    return n_tiles * h * (np_ * ep + 1)
+
+
 def max_experts() -> tuple[int, int]:
     """Largest number of experts, and of chosen ones."""
     ext = hybrid_ext()
@@ -128,11 +137,12 @@ def ssd_decode(proj, rows: int, *, h: int, g: int, w, state, conv_state, row_slo
 
 
 def ssd_prefill(proj, m: int, *, h: int, g: int, w, state, conv_state, seq_slots, tile_seq, tile_q0, q_start, q_lens, ctx_lens,
-                n_tiles: int, n_seqs: int, u, y, runs: bool) -> None:
-    """Prompt chunks: convolution into `u`, then runs of 64 tokens on tensor cores (`runs`) or token by token."""
+                n_tiles: int, n_seqs: int, u, y, runs: bool, segment: int = 0, ws=None) -> None:
+    """Prompt chunks: convolution into `u`, then runs of 64 tokens on tensor cores (`runs`) or token by token. `segment` (see
+    ssd_segment): rows of a sequence that are walked in one piece, with `ws` for the states between the pieces."""
     hybrid_ext().ssd_prefill(proj, m, h, g, list(w), state, conv_state, seq_slots, tile_seq, tile_q0, q_start, q_lens, ctx_lens,
-                             n_tiles, n_seqs, u, y, runs, ops.status_word(proj.device))
-    ops._bump(2)
+                             n_tiles, n_seqs, u, y, runs, segment, ws, ops.status_word(proj.device))
+    ops._bump(4 if segment else 2)
 
 
 def gated_norm(y, z, m: int, *, h: int, e: int, ep: int, groups: int, w, eps: float, out) -> None:
