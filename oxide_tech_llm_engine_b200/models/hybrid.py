@@ -24,6 +24,9 @@ and with mixer and feed-forward side by side:
       branch_norm   norms of both mixer outputs, weighted expert rows, residual, norms of the next layer
     final branch_norm over the logit rows -> gemm(head)
 
+In a captured decode step the three lines between two branch_norms run on streams of their own: the
+experts beside the projection and the mixers, the state-space mixer beside the attention.
+
 KV blocks come from the scheduler's paged pool like any model's (one cache per attention run, so a
 looped layer has one per pass); recurrent states live in slots that the scheduler hands to running
 sequences. All sizes and constants come from the LayerSpec list; matrices are zero-padded to the
@@ -33,6 +36,7 @@ from __future__ import annotations
 
 import math
 import os
+from contextlib import contextmanager, nullcontext
 from typing import Optional
 
 import numpy as np
@@ -163,13 +167,14 @@ class SsdRun:
         m.states += [self.state, self.conv_state]
         self.runs = m.dtype == torch.bfloat16 and hops.ssd_chunks_ok(r.state_p)
 
-    def mix(self, s: StepInputs, proj: torch.Tensor) -> torch.Tensor:
-        """Projection rows z | x | B | C | dt -> gated and normed rows [M, heads * vdim]."""
+    def mix(self, s: StepInputs, proj: torch.Tensor, start=nullcontext()) -> torch.Tensor:
+        """Projection rows z | x | B | C | dt -> gated and normed rows [M, heads * vdim]. `start`: context of the first launch."""
         m, r, w, M, nd = self.m, self.spec, self.w, s.m, s.n_decode
         y = m.buffer(("ssd_y", r.heads * r.vdim_p), r.heads * r.vdim_p)
         kw = dict(h=r.heads, g=r.groups, w=w["ssd"], state=self.state, conv_state=self.conv_state, y=y)
         if nd > 0:
-            hops.ssd_decode(proj, nd, row_slots=s.decode_slots, positions=s.positions, **kw)
+            with start:
+                hops.ssd_decode(proj, nd, row_slots=s.decode_slots, positions=s.positions, **kw)
         if s.n_prefill > 0:
             seg = hops.ssd_segment(r.heads, r.vdim_p, s.n_tiles, s.n_prefill) if self.runs else 0
             if seg:
@@ -191,12 +196,13 @@ class MoeRun:
         self.fp = round_up(spec.ff, 64)
         self.b = m.moe_buffers(spec.experts, spec.top, self.fp)
 
-    def __call__(self, s: StepInputs, h: torch.Tensor) -> tuple:
+    def __call__(self, s: StepInputs, h: torch.Tensor, start=nullcontext()) -> tuple:
         m, e, w, b, M = self.m, self.spec, self.w, self.b, s.m
         E, top = e.experts, e.top
         route = dict(e=E, top=top, weight=b["weight"], expert=b["expert"], slot=b["slot"])
         if m.dtype == torch.float32 or m.few_rows(M):
-            hops.moe_route(h, w["router"], M, **route)
+            with start:
+                hops.moe_route(h, w["router"], M, **route)
             pairs = M * top
             rows, act = b["out"][:pairs], b["act"][:pairs]
             hops.moe_rows(h, w["up"], b["expert"], pairs, top=top, per_pair=False, y=act, act=2)
@@ -205,7 +211,8 @@ class MoeRun:
         if M <= 128:
             # one slab of 128 rows per expert: a single launch routes and places
             xs, act, rows = (b[k][:E * 128] for k in ("xs", "act", "out"))
-            hops.moe_route(h, w["router"], M, mode=1, counts=b["counts"], xs=xs, **route)
+            with start:
+                hops.moe_route(h, w["router"], M, mode=1, counts=b["counts"], xs=xs, **route)
             m_tiles = min(E, M * top)
             gx, ga, gr = xs.view(E, 128, -1), act.view(E, 128, -1), rows.view(E, 128, -1)
         else:
@@ -231,7 +238,7 @@ class ParallelRun:
         self.left = AttentionRun(m, spec.left, w["left"])
         self.right = SsdRun(m, spec.right, w["right"])
         self.split = round_up(self.left.width, 64)        # first column of the right mixer's projection
-        self.width = self.split + spec.right.width_p
+        self.width = m._in_width(spec)
         self.k = (round_up(spec.left.out_dim, 64), round_up(spec.right.out_dim, 64))
 
     def clears(self, M: int) -> tuple:
@@ -240,10 +247,32 @@ class ParallelRun:
 
     def __call__(self, s: StepInputs, h: torch.Tensor, h2: Optional[torch.Tensor]) -> Optional[tuple]:
         m, w = self.m, self.w
+        if m.side_streams(s):
+            return self._on_streams(s, h, h2)
         proj = m.project(h, w["w_in"], self.width)
         m.into_branch(0, self.left.attend(s, proj), w["left"]["w_o"])
         m.into_branch(1, self.right.mix(s, proj[:, self.split:]), w["right"]["w_o"])
         return self.mlp(s, h2) if self.mlp is not None else None
+
+    def _on_streams(self, s: StepInputs, h: torch.Tensor, h2: Optional[torch.Tensor]) -> Optional[tuple]:
+        """The same, forked and joined. A launch that waits for another stream takes a full dependency, not a
+        programmatic one."""
+        m, w = self.m, self.w
+        main, experts = torch.cuda.current_stream(m.device), None
+        s_right, s_moe = m.streams2
+        if self.mlp is not None:
+            s_moe.wait_stream(main)
+            with torch.cuda.stream(s_moe):
+                experts = self.mlp(s, h2, start=m.full_dependency())
+        proj = m.project(h, w["w_in"], self.width)
+        s_right.wait_stream(main)
+        with torch.cuda.stream(s_right):
+            m.into_branch(1, self.right.mix(s, proj[:, self.split:], start=m.full_dependency()), w["right"]["w_o"])
+        m.into_branch(0, self.left.attend(s, proj), w["left"]["w_o"])
+        main.wait_stream(s_right)
+        if self.mlp is not None:
+            main.wait_stream(s_moe)
+        return experts
 
 
 class MlpRun:
@@ -294,6 +323,7 @@ class HybridModel(GemmShapes):
         self.device = device or torch.device("cuda", torch.cuda.current_device())
         self.weight_mode = weight_mode
         pdl = os.environ.get("OXB_PDL", "1") != "0"
+        self._pdl = pdl
         ops.set_pdl(pdl)
         hops.set_pdl(pdl)
         self._sms = torch.cuda.get_device_properties(self.device).multi_processor_count
@@ -325,6 +355,8 @@ class HybridModel(GemmShapes):
         self.branches = torch.zeros(n_acc, max_tokens, self.dp, dtype=torch.float32, device=dev)
         self.acc = self.branches[0]
         self.h2 = torch.zeros_like(self.h) if self.parallel else None
+        on = self.parallel and os.environ.get("OXB_STREAMS", "1") != "0"
+        self.streams2 = tuple(torch.cuda.Stream(dev) for _ in range(2)) if on else None
         self.vp = round_up(cfg.vocab_size, 64)
         self.v_l = cfg.vocab_size
         self.lm_h = torch.zeros(self.max_logits, self.dp, dtype=self.dtype, device=dev)
@@ -352,7 +384,8 @@ class HybridModel(GemmShapes):
     @staticmethod
     def _in_width(mix) -> int:
         if mix.kind == "parallel":
-            return round_up(HybridModel._in_width(mix.left) + mix.right.width_p, 64)
+            n = HybridModel._in_width(mix.left) + mix.right.width_p
+            return round_up(n, 256 if n >= 2048 else 64)      # wide projections in whole tiles of the widest kind
         w = (mix.heads * mix.dim + mix.kv_heads * (mix.dim + mix.vdim) if mix.kind == "attention"
              else 2 * mix.heads * (mix.dim + mix.vdim))
         return round_up(w, 64)
@@ -483,7 +516,11 @@ class HybridModel(GemmShapes):
                 self._rots[a.rot] = hops.Rotary(a.rot, self.device)
             q = torch.cat([mat(f"{p}mix.left.{n}") for n in ("q", "k", "v")])
             ssd = self._ssd_weights(mx.right, p + "mix.right.", mat, vec)
-            w_in = torch.cat([q, q.new_zeros(round_up(q.shape[0], 64) - q.shape[0], q.shape[1]), ssd.pop("in")])
+            right = ssd.pop("in")
+            w_in = q.new_zeros(self._in_width(mx), q.shape[1])
+            w_in[:q.shape[0]] = q
+            at = round_up(q.shape[0], 64)
+            w_in[at:at + right.shape[0]] = right
             w = {"w_in": self._pad(w_in), "right": ssd,
                  "left": {"rot": self._rots[a.rot], "q_norm": None, "k_norm": None, "w_o": self._pad(mat(p + "mix.left.o"))}}
             mlp = MoeRun(self, L.mlp, self._moe_weights(L.mlp, p + "mlp.", mat)) if L.mlp is not None else None
@@ -570,6 +607,21 @@ class HybridModel(GemmShapes):
             return t.normal_(0.0, self.cfg.d_model ** -0.5 if name.endswith(".router") else std, generator=g)
 
         self._build(get)
+
+    # ------------------------------------------------------------------ streams
+    def side_streams(self, s: StepInputs) -> bool:
+        """Whether the parts of a layer run on streams of their own: small decode steps that are being captured."""
+        return (self.streams2 is not None and s.n_prefill == 0 and s.m <= 128 and self.dtype == torch.bfloat16
+                and torch.cuda.is_current_stream_capturing())
+
+    @contextmanager
+    def full_dependency(self):
+        """Launches inside take no programmatic dependency (the ones of this module's kernels)."""
+        hops.set_pdl(False)
+        try:
+            yield
+        finally:
+            hops.set_pdl(self._pdl)
 
     # ------------------------------------------------------------------ projections
     def few_rows(self, M: int) -> bool:
@@ -682,7 +734,9 @@ class HybridModel(GemmShapes):
             else:
                 norms = layers[i].norms
                 kw.update(norm_w=norms, h=[h, h2][:len(norms)], clear=self._proj_splits(M, layers[i]))
-            hops.branch_norm(x, M, **kw)
+            joins = i > 0 and self.side_streams(s)
+            with self.full_dependency() if joins else nullcontext():
+                hops.branch_norm(x, M, **kw)
             if self.layer_hook is not None and i > 0:
                 self.layer_hook(i - 1, x[:M])
             if not last:
