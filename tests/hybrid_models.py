@@ -73,18 +73,23 @@ def weights(cfg, seed=0):
             x = x * 0.7
         else:
             x = x * ((0.7 if name.endswith((".o", ".down")) else 1.0) / np.sqrt(shape[1]))
-        u = np.ascontiguousarray(x, dtype=np.float32).view(np.uint32)
-        out[name] = ((u + 0x8000) & 0xFFFF0000).astype(np.uint32).view(np.float32).reshape(shape).copy()
+        out[name] = bf16_exact(x)
     return out
+
+
+def bf16_exact(x):
+    """The values rounded to what bf16 holds."""
+    u = np.ascontiguousarray(x, dtype=np.float32).view(np.uint32)
+    return ((u + 0x8000) & 0xFFFF0000).astype(np.uint32).view(np.float32).reshape(np.shape(x)).copy()
 
 
 class DictSource:
     """A checkpoint in memory, with the interface of models.weights.WeightSource."""
 
     def __init__(self, cfg, w):
-        from oxide_tech_llm_engine_b200.models.layer_spec import kipolix_config
+        from oxide_tech_llm_engine_b200.models.registry import config_from_json
 
-        self.cfg, self.w = kipolix_config(cfg), w
+        self.cfg, self.w = config_from_json(cfg), w
 
     def names(self):
         return self.w.keys()

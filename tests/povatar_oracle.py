@@ -145,8 +145,17 @@ def relu_squared(z):
     return torch.clamp(z, min=0.0) ** 2
 
 
-def experts(c, w, p, h):
-    ids, wt = choose(h @ w[p + "router"].T, c["router"]["top"])
+def margin(logits, top):
+    """How clear the choice of a token is: gap between the last chosen and the next logit, in their standard deviation."""
+    s = torch.sort(logits, -1, descending=True).values
+    return (s[:, top - 1] - s[:, top]) / logits.std() if s.shape[1] > top else torch.full((len(s),), math.inf, dtype=s.dtype)
+
+
+def experts(c, w, p, h, margins=None):
+    lg, top = h @ w[p + "router"].T, c["router"]["top"]
+    if margins is not None:
+        margins.append(margin(lg, top))
+    ids, wt = choose(lg, top)
     out = torch.zeros_like(h)
     for t in range(h.shape[0]):
         for e, a in zip(ids[t].tolist(), wt[t]):
@@ -155,8 +164,9 @@ def experts(c, w, p, h):
 
 
 # ---------------------------------------------------------------- model
-def forward(cfg, w, tokens, want_layers=False):
-    """Logits [T, vocab] of one whole sequence (and the residual stream after every layer)."""
+def forward(cfg, w, tokens, want_layers=False, margins=None):
+    """Logits [T, vocab] of one whole sequence (and the residual stream after every layer). `margins`: a list that takes
+    the tokens' margins of every router."""
     w = {k: torch.as_tensor(v).to(F64) for k, v in w.items()}
     eps = cfg["norm"]["eps"]
     pos = torch.arange(len(tokens))
@@ -169,7 +179,7 @@ def forward(cfg, w, tokens, want_layers=False):
         b = right_mixer(L["mixer"]["right"], w, p + "mix.right.", h, eps)
         y = 0.5 * (rms(a, eps) * w[p + "mix.left.out"] + rms(b, eps) * w[p + "mix.right.out"])
         if L["mlp"] is not None:
-            y = y + experts(L["mlp"], w, p + "mlp.", rms(x, eps) * w[p + "norm2"])
+            y = y + experts(L["mlp"], w, p + "mlp.", rms(x, eps) * w[p + "norm2"], margins)
         x = x + y
         seen.append(x)
     logits = rms(x, eps) * w["final.norm"] @ w["head"].T

@@ -138,8 +138,9 @@ def paged(k, v, DP, EP, dt, seed):
     return kc.to(dt).to(DEV), vc.to(dt).to(DEV), perm[:nb].to(torch.int32)
 
 
-def run_attention(H, path, q, k, v, scale, size, keep, mode, splits=4):
-    """Rows of the last `n` positions through the prompt kernel, or every row through the decode kernel."""
+def run_attention(H, path, q, k, v, scale, size, keep, mode, splits=4, **extra):
+    """Rows of the last `n` positions through the prompt kernel, or every row through the decode kernel. `extra`: further
+    options of the kernels (chunk, sink)."""
     from oxide_tech_llm_engine_b200 import ops
 
     T, heads, D = q.shape
@@ -153,7 +154,7 @@ def run_attention(H, path, q, k, v, scale, size, keep, mode, splits=4):
     qp = torch.zeros(T, heads, DP, dtype=dt, device=DEV)
     qp[..., :D] = q.to(DEV)
     i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=DEV)
-    kw = dict(window=size, keep_first=keep, scale=scale)
+    kw = dict(window=size, keep_first=keep, scale=scale, **extra)
     if mode == "decode":
         tables = bt[None].repeat(T, 1).contiguous().to(DEV)
         lens = i32(list(range(1, T + 1)))
