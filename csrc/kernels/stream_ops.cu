@@ -232,17 +232,18 @@ template <typename T, int CH>
 __global__ void __launch_bounds__(CH == 4 ? 512 : 1024) branch_norm_kernel(const BranchNormParams p) {
   __shared__ float s_red[32];
   __shared__ float2 s_red2[32];
-  __shared__ ChosenRow s_e[kMaxTop];
+  __shared__ ChosenRow s_chosen[2][kMaxTop];   // of this row and of the CTA's next one
   pdl_launch_dependents();
   pdl_wait();
   const int N = p.N;
   const float inv_n = 1.f / static_cast<float>(N);
-  for (int row = blockIdx.x; row < p.rows; row += gridDim.x) {
+  if (p.e_rows != nullptr) {
+    chosen_rows(p, blockIdx.x, s_chosen[0]);
+    __syncthreads();
+  }
+  int parity = 0;
+  for (int row = blockIdx.x; row < p.rows; row += gridDim.x, parity ^= 1) {
     float* xr = p.x + static_cast<long long>(row) * N;
-    if (p.e_rows != nullptr) {
-      __syncthreads();               // the row before has been read out
-      chosen_rows(p, row, s_e);      // published by the barriers of the branches' sums
-    }
     if (p.clear != nullptr) {
       float* z = p.clear + static_cast<long long>(row) * p.clear_ld;
       for (int c = threadIdx.x * 4; c < p.clear_n; c += blockDim.x * 4)
@@ -278,7 +279,10 @@ __global__ void __launch_bounds__(CH == 4 ? 512 : 1024) branch_norm_kernel(const
         const int c = (k * blockDim.x + threadIdx.x) * 4;
 #pragma unroll
         for (int j = 0; j < 4; ++j) x[k][j] = 0.f;
-        if (c < N) load4<float>(xr + c, x[k]);
+        if (c < N) {
+          load4<float>(xr + c, x[k]);
+          if (p.e_rows != nullptr) expert_sum4<T>(p, s_chosen[parity], c, x[k]);
+        }
 #pragma unroll
         for (int b = 0; b < kMaxBranches; ++b) {
 #pragma unroll
@@ -290,6 +294,8 @@ __global__ void __launch_bounds__(CH == 4 ? 512 : 1024) branch_norm_kernel(const
           }
         }
       }
+      // (the barriers of the sums and of the norm below publish the next row's table)
+      if (p.e_rows != nullptr && row + gridDim.x < p.rows) chosen_rows(p, row + gridDim.x, s_chosen[parity ^ 1]);
       const float2 tot = block_sum2(make_float2(ss[0], ss[1]), s_red2);
       const float r[kMaxBranches] = {1.f / sqrtf(tot.x * inv_n + p.eps), 1.f / sqrtf(tot.y * inv_n + p.eps)};
 #pragma unroll
@@ -308,7 +314,6 @@ __global__ void __launch_bounds__(CH == 4 ? 512 : 1024) branch_norm_kernel(const
             if (p.clear_y[b])
               *reinterpret_cast<float4*>(p.y[b] + static_cast<long long>(row) * p.ldy + c) = make_float4(0.f, 0.f, 0.f, 0.f);
           }
-        if (p.e_rows != nullptr) expert_sum4<T>(p, s_e, c, a);
 #pragma unroll
         for (int j = 0; j < 4; ++j) x[k][j] += a[j];
       }

@@ -260,7 +260,8 @@ def kernel_numbers(pov, mix, peaks: dict, timer: Timer, batch: int, ctx: int, m:
                                             q_start=qs, q_lens=ql, ctx_lens=ql, n_tiles=len(tl), n_seqs=nseq, u=u, y=y, runs=True,
                                             segment=seg, ws=sws)
         C = 64
-        # the projection in, the convolved channels out and in again, y out, the states; the run form's arithmetic
+        # the projection in, the convolved channels out and in again, y out, the states of the sequences; the run form's
+        # arithmetic (for retention its inputs, output and states; neither counts the states between chunks or segments)
         add(f"ssd convolution and runs [{mm} tokens of {L}, {h} heads {N} x {V}]", sp, mm * 2 * (3 * ch + h * V) + nseq * h * N * V * 8,
             mm * (h * (4.0 * N * V + (C + 1) * V) + G * (C + 1) * N))
         qr_, kr_ = torch.randn(h, mm, N, device=dev), torch.randn(h, mm, N, device=dev)
@@ -272,8 +273,7 @@ def kernel_numbers(pov, mix, peaks: dict, timer: Timer, batch: int, ctx: int, m:
             return lambda: hops.retention_prefill(proj, mm, h=h, d=N, e=V, decay_pow=pw, eps=1e-5, state=st, seq_slots=sq, tile_seq=ts,
                                                   tile_q0=tq, q_start=qs, q_lens=ql, ctx_lens=ql, n_tiles=len(tl), n_seqs=nseq,
                                                   q_rot=qr_, k_rot=kr_, ws=ws, out=out)
-        n_ch = mm // C
-        add(f"retention_prefill [{mm} tokens of {L}, {h} heads {N} x {V}]", rp, mm * h * (2 * N * 4 + 3 * V * 2) + 4.0 * n_ch * h * N * V * 4,
+        add(f"retention_prefill [{mm} tokens of {L}, {h} heads {N} x {V}]", rp, mm * h * (2 * N * 4 + 3 * V * 2) + nseq * h * N * V * 8,
             mm * h * (4.0 * N * V + (C + 1) * (N + V)))
     return rows
 
