@@ -28,6 +28,17 @@ __device__ __forceinline__ void load4<__nv_bfloat16>(const __nv_bfloat16* p, flo
   const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.y));
   v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
 }
+// The same past L1: rows that are read once, next to vectors that every row reads again
+__device__ __forceinline__ void load4_stream(const float* p, float (&v)[4]) {
+  const float4 x = __ldcg(reinterpret_cast<const float4*>(p));
+  v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+}
+__device__ __forceinline__ void load4_stream(const __nv_bfloat16* p, float (&v)[4]) {
+  const uint2 x = __ldcg(reinterpret_cast<const uint2*>(p));
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.y));
+  v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+}
 template <typename T>
 __device__ __forceinline__ void store4(T* p, const float (&v)[4]);
 template <>

@@ -182,8 +182,8 @@ cudaError_t launch_t(const StreamNormParams& p, cudaStream_t stream) {
   return launch_s<T, kMaxStreams>(p, stream);
 }
 
-// Layers whose mixer and feed-forward run side by side: V values per piece, CH pieces per thread that stay in
-// registers (CH = 0: any row length, the row goes through shared memory).
+// Layers whose mixer and feed-forward run side by side: four values per piece, CH pieces per thread, which stay
+// in registers.
 // The chosen experts' rows of a token wait in shared memory as (row, weight): a row outside the buffer weighs nothing.
 struct ChosenRow {
   int row;
@@ -203,7 +203,7 @@ __device__ __forceinline__ void expert_sum4(const BranchNormParams& p, const Cho
   for (int k = 0; k < p.top; ++k) {
     const ChosenRow e = s_e[k];
     float v[4];
-    load4<T>(rows + static_cast<long long>(e.row) * p.lde, v);
+    load4_stream(rows + static_cast<long long>(e.row) * p.lde, v);
 #pragma unroll
     for (int j = 0; j < 4; ++j) a[j] = fmaf(e.weight, v[j], a[j]);
   }
@@ -229,7 +229,7 @@ __device__ __forceinline__ float2 block_sum2(float2 v, float2* scratch) {
 }
 
 template <typename T, int CH>
-__global__ void __launch_bounds__(CH == 4 ? 512 : 1024) branch_norm_kernel(const BranchNormParams p) {
+__global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchNormParams p) {
   __shared__ float s_red[32];
   __shared__ float2 s_red2[32];
   __shared__ ChosenRow s_chosen[2][kMaxTop];   // of this row and of the CTA's next one
@@ -280,7 +280,7 @@ __global__ void __launch_bounds__(CH == 4 ? 512 : 1024) branch_norm_kernel(const
 #pragma unroll
         for (int j = 0; j < 4; ++j) x[k][j] = 0.f;
         if (c < N) {
-          load4<float>(xr + c, x[k]);
+          load4_stream(xr + c, x[k]);
           if (p.e_rows != nullptr) expert_sum4<T>(p, s_chosen[parity], c, x[k]);
         }
 #pragma unroll
@@ -288,7 +288,7 @@ __global__ void __launch_bounds__(CH == 4 ? 512 : 1024) branch_norm_kernel(const
 #pragma unroll
           for (int j = 0; j < 4; ++j) y[b][k][j] = 0.f;
           if (b < p.n_branches && c < N) {
-            load4<float>(p.y[b] + static_cast<long long>(row) * p.ldy + c, y[b][k]);
+            load4_stream(p.y[b] + static_cast<long long>(row) * p.ldy + c, y[b][k]);
 #pragma unroll
             for (int j = 0; j < 4; ++j) ss[b] = fmaf(y[b][k][j], y[b][k][j], ss[b]);
           }
@@ -347,6 +347,7 @@ __global__ void __launch_bounds__(CH == 4 ? 512 : 1024) branch_norm_kernel(const
   }
 }
 
+// Any row length; the row waits in shared memory.
 template <typename T>
 __global__ void __launch_bounds__(256) branch_norm_any_kernel(const BranchNormParams p) {
   extern __shared__ float s_u[];  // N values of the row
@@ -424,13 +425,9 @@ cudaError_t launch_branch(const BranchNormParams& p, cudaStream_t stream) {
   const bool vec = p.N % 4 == 0 && p.ldy % 4 == 0 && p.ldh % 4 == 0 && p.lde % 4 == 0;
   const int quads = (p.N + 3) / 4;
   auto threads = [&](int ch) { return dim3(((quads + ch - 1) / ch + 31) / 32 * 32); };
-  // few rows: one piece per thread; many rows: more bytes in flight per thread, several CTAs per SM
-  const bool many = p.rows > 2 * sm_count() && quads > 256;
-  if (vec && quads <= 2048) {
-    if (many && quads > 512) return launch_kernel(branch_norm_kernel<T, 4>, grid, threads(4), 0, stream, true, false, p);
-    if (many || quads > 1024) return launch_kernel(branch_norm_kernel<T, 2>, grid, threads(2), 0, stream, true, false, p);
-    return launch_kernel(branch_norm_kernel<T, 1>, grid, threads(1), 0, stream, true, false, p);
-  }
+  // one piece per thread: whole rows in flight, as many warps as the row has (measured against two and four pieces)
+  if (vec && quads <= 1024) return launch_kernel(branch_norm_kernel<T, 1>, grid, threads(1), 0, stream, true, false, p);
+  if (vec && quads <= 2048) return launch_kernel(branch_norm_kernel<T, 2>, grid, threads(2), 0, stream, true, false, p);
   const size_t smem = static_cast<size_t>(p.N) * sizeof(float);
   ensure_dynamic_smem(branch_norm_any_kernel<T>, smem);
   return launch_kernel(branch_norm_any_kernel<T>, grid, dim3(256), smem, stream, true, false, p);
