@@ -177,7 +177,7 @@ def kernel_numbers(pov, mix, peaks: dict, timer: Timer, batch: int, ctx: int, m:
         # where each slab row goes back to
         meta = torch.zeros(E, cap, 4, dtype=torch.int32, device=dev)
         meta[..., 1] = torch.randint(0, M, (E, cap), device=dev)
-        add(f"expert gate|up, SwiGLU (Mixtral) [{M} rows x {top}]", lambda i: (lambda: ops.gemm(
+        add(f"expert gate and up, SwiGLU (Mixtral) [{M} rows x {top}]", lambda i: (lambda: ops.gemm(
             slab, gus[i % reps], out=acts, epi=ops.EPI_SWIGLU_BF16, group_counts=counts, m_tiles=(M * top + 127) // 128 + E, bn=128)),
             active * 2 * d * fm_ * 2 + pairs * (d + fm_) * 2, 4.0 * pairs * d * fm_)
         add(f"expert down, combine (Mixtral) [{M} rows x {top}]", lambda i: (lambda: ops.gemm(
