@@ -218,8 +218,11 @@ void gemm_bf16(const Tensor& a, const Tensor& w, int64_t epi, const c10::optiona
       p.row_meta = reinterpret_cast<const oxb::RowMeta*>(row_meta->data_ptr());
       p.meta_group_stride = M;
     }
-  } else {
-    TORCH_CHECK(G == 1, "gemm_bf16: 3-D operands need group_counts");
+  } else if (grouped3d && G > 1) {
+    // equal groups: M rows each
+    TORCH_CHECK(mt_i == 1 && !fixup && G <= 1024 && !routed && out->dim() == 3, "gemm_bf16: equal groups store [G, M, N]");
+    p.n_groups = static_cast<int>(G);
+    m_tiles *= static_cast<int>(G);
   }
   if (ag_flags.has_value() && ag_flags->defined()) {
     TORCH_CHECK(ag_ticket.has_value(), "gemm_bf16: ag_ticket required with ag_flags");
@@ -323,12 +326,13 @@ void paged_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
                   const c10::optional<Tensor>& status, const c10::optional<Tensor>& page_ml,
                   const c10::optional<Tensor>& block_mass, const c10::optional<Tensor>& q8,
                   const c10::optional<Tensor>& q8_d, const c10::optional<Tensor>& q8_s, int64_t keep_first, int64_t out_d,
-                  bool exact_p, int64_t chunk, double sink) {
+                  bool exact_p, int64_t chunk, double sink, const std::vector<double>& diff) {
   TORCH_CHECK(q.dim() == 3 && k_cache.dim() == 4, "paged_decode: q [B,Hq,D], cache [blk,Hkv,16,D]");
   TORCH_CHECK(k_cache.size(2) == 16, "paged_decode: 16-token pages");
   oxb::DecodeAttnParams p{};
   const int D = static_cast<int>(q.size(2));
-  TORCH_CHECK(D == 64 || D == 128, "paged_decode: head_dim 64 or 128");
+  TORCH_CHECK(D == 64 || D == 128 || D == 256, "paged_decode: head_dim 64, 128 or 256");
+  TORCH_CHECK(D != 256 || !page_ml.has_value(), "paged_decode: no block mass for heads of 256");
   p.q = reinterpret_cast<const __nv_bfloat16*>(q.data_ptr());
   p.q_stride = q.stride(0);
   TORCH_CHECK(q.stride(1) == D && q.stride(2) == 1, "paged_decode: q heads must be packed");
@@ -356,6 +360,14 @@ void paged_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
   TORCH_CHECK(chunk >= 0 && (chunk == 0 || (window == 0 && keep_first == 0)), "paged_decode: a window or a chunk");
   p.chunk = static_cast<int>(chunk);
   p.sink_log2 = static_cast<float>(sink * 1.4426950408889634);
+  if (!diff.empty()) {
+    TORCH_CHECK(diff.size() == 3 && p.Hq % 2 == 0 && !page_ml.has_value() && !q8.has_value() && !std::isfinite(sink),
+                "paged_decode: diff is (lambda, gain, eps) over pairs of query heads");
+    p.diff = 1;
+    p.diff_lambda = static_cast<float>(diff[0]);
+    p.diff_gain = static_cast<float>(diff[1]);
+    p.diff_eps = static_cast<float>(diff[2]);
+  }
   TORCH_CHECK(!(page_ml.has_value() && (keep_first > 0 || exact_p || std::isfinite(sink))),
               "paged_decode: block mass goes with the plain window");
   p.scale_log2 = static_cast<float>(scale * 1.4426950408889634);
@@ -407,7 +419,8 @@ void paged_prefill_tc(const Tensor& q, const Tensor& k_cache, const Tensor& v_ca
   p.q_start = q_start.data_ptr<int>();
   p.q_lens = q_lens.data_ptr<int>();
   p.ctx_lens = ctx_lens.data_ptr<int>();
-  p.out = reinterpret_cast<__nv_bfloat16*>(out.data_ptr());
+  if (out.scalar_type() == torch::kFloat32) p.out_f32 = out.data_ptr<float>();
+  else p.out = reinterpret_cast<__nv_bfloat16*>(out.data_ptr());
   p.out_stride = out.stride(0);
   p.max_blocks = static_cast<int>(block_tables.size(1));
   p.Hq = static_cast<int>(q.size(1));

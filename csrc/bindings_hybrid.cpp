@@ -4,9 +4,12 @@
 #include <cuda_runtime.h>
 #include <torch/extension.h>
 
+#include <cmath>
 #include <vector>
 
 #include "common/device_info.h"
+#include "common/tma_host.h"
+#include "kernels/attn.cuh"
 #include "kernels/hybrid.cuh"
 
 namespace py = pybind11;
@@ -22,6 +25,8 @@ void check_launch(cudaError_t e, const char* what) {
   if (e == cudaSuccess) e = last;
   TORCH_CHECK(e == cudaSuccess, "oxb: launch of ", what, " failed: ", cudaGetErrorString(e));
 }
+
+void check_launch(const char* what) { check_launch(cudaSuccess, what); }
 
 int dtype_code(const Tensor& t, const char* what) {
   TORCH_CHECK(t.is_cuda() && (t.scalar_type() == torch::kBFloat16 || t.scalar_type() == torch::kFloat32), what,
@@ -125,14 +130,18 @@ void stream_norm(const Tensor& x, int64_t rows, const OptTensor& tokens, const O
 void heads(const Tensor& proj, int64_t M, int64_t H, int64_t G, int64_t D, int64_t E, const OptTensor& q_norm,
            const OptTensor& k_norm, double eps, const OptTensor& freq_hi, const OptTensor& freq_lo, bool interleaved,
            double gain, const Tensor& positions, double k_scale, const Tensor& q_out, int64_t q_hd, const OptTensor& k_out,
-           const OptTensor& k_cache, const OptTensor& v_cache, const OptTensor& slots, const Tensor& status) {
+           const OptTensor& k_cache, const OptTensor& v_cache, const OptTensor& slots, int64_t q_pd, int64_t maps, const OptTensor& bias,
+           double t_coef, double t_every, const Tensor& status) {
   oxb::HeadsParams p{};
   // storage type: that of the caches; dense q and k are fp32 whatever the projection is
   const int proj_dt = dtype_code(proj, "heads proj");
-  const int dt = given(k_cache) ? dtype_code(*k_cache, "heads k_cache") : proj_dt;
+  const int dt = given(k_cache) ? dtype_code(*k_cache, "heads k_cache") : (given(k_out) ? proj_dt : dtype_code(q_out, "heads q_out"));
   p.proj_f32 = proj_dt;
   TORCH_CHECK(dt == 0 || proj_dt == 1, "heads: fp32 caches take fp32 projections");
-  TORCH_CHECK(H >= 1 && G >= 1 && D >= 1 && q_hd >= D, "heads: sizes");
+  if (q_pd == 0) q_pd = D;
+  TORCH_CHECK(H >= 1 && G >= 0 && D >= 1 && maps >= 1 && G % maps == 0 && q_hd >= (maps - 1) * D + D && q_pd >= D, "heads: sizes");
+  p.maps = static_cast<int>(maps);
+  p.q_pd = q_pd;
   p.proj = proj.data_ptr();
   p.M = static_cast<int>(M);
   p.H = static_cast<int>(H);
@@ -143,6 +152,11 @@ void heads(const Tensor& proj, int64_t M, int64_t H, int64_t G, int64_t D, int64
   p.k_norm = f32(k_norm, G * D, "heads k_norm");
   TORCH_CHECK((p.q_norm == nullptr) == (p.k_norm == nullptr), "heads: q and k norm go together");
   p.eps = static_cast<float>(eps);
+  TORCH_CHECK(p.q_norm == nullptr || (q_pd == D && !given(bias)), "heads: the norm spans packed heads without bias");
+  p.bias = f32(bias, H * q_pd + G * D + G / maps * E, "heads bias");
+  TORCH_CHECK(t_coef == 0.0 || t_every > 0.0, "heads: temperature");
+  p.t_coef = static_cast<float>(t_coef);
+  p.t_every = static_cast<float>(t_every);
   p.rot = rotary(freq_hi, freq_lo, interleaved, gain, D);
   p.positions = i32(positions, M, "heads positions");
   p.k_scale = static_cast<float>(k_scale);
@@ -155,22 +169,30 @@ void heads(const Tensor& proj, int64_t M, int64_t H, int64_t G, int64_t D, int64
                   "heads: dense q and k are fp32 [heads, rows, D]");
       return t.stride(0);
     };
-    p.ld = pitch(proj, M, (H + G) * D, "heads proj");
+    TORCH_CHECK(maps == 1, "heads: dense keys have one map");
+    p.ld = pitch(proj, M, H * q_pd + G * D, "heads proj");
     p.q_hd = dense(q_out, H);
     p.k_hd = dense(*k_out, G);
     p.q_ld = p.k_ld = D;
     p.k_out = k_out->data_ptr<float>();
   } else {
-    p.q_ld = pitch(q_out, M, H * q_hd, "heads q_out");
+    p.q_ld = pitch(q_out, M, (H - 1) * q_hd + maps * D, "heads q_out");
     p.q_hd = q_hd;
+    if (G == 0) {
+      TORCH_CHECK(!given(k_cache) && !given(v_cache), "heads: queries only");
+      p.ld = pitch(proj, M, (H - 1) * q_pd + D, "heads proj");
+      p.status = status_ptr(status);
+      check_launch(oxb::launch_heads(p, dt, cur_stream()), "heads");
+      return;
+    }
     TORCH_CHECK(given(k_cache) && given(v_cache) && given(slots), "heads: caches and slots, or k_out");
     TORCH_CHECK(q_out.scalar_type() == k_cache->scalar_type() && v_cache->scalar_type() == k_cache->scalar_type(),
                 "heads: one storage type");
     TORCH_CHECK(k_cache->dim() == 4 && v_cache->dim() == 4 && k_cache->is_contiguous() && v_cache->is_contiguous() &&
-                    k_cache->size(1) == G && v_cache->size(1) == G && k_cache->size(2) == 16 && v_cache->size(2) == 16 &&
-                    k_cache->size(0) == v_cache->size(0) && k_cache->size(3) >= D && v_cache->size(3) >= E,
+                    k_cache->size(1) == G / maps && v_cache->size(1) == G / maps && k_cache->size(2) == 16 && v_cache->size(2) == 16 &&
+                    k_cache->size(0) == v_cache->size(0) && k_cache->size(3) >= maps * D && v_cache->size(3) >= E,
                 "heads: caches [blocks, G, 16, >= head size]");
-    p.ld = pitch(proj, M, (H + G) * D + G * E, "heads proj");
+    p.ld = pitch(proj, M, H * q_pd + G * D + G / maps * E, "heads proj");
     p.k_cache = k_cache->data_ptr();
     p.v_cache = v_cache->data_ptr();
     p.DP = static_cast<int>(k_cache->size(3));
@@ -186,7 +208,7 @@ void heads(const Tensor& proj, int64_t M, int64_t H, int64_t G, int64_t D, int64
 void row_attention(const Tensor& q, int64_t q_hd, const Tensor& k_cache, const Tensor& v_cache, const Tensor& block_tables,
                    const OptTensor& seq_lens, const OptTensor& tile_seq, const OptTensor& tile_q0, const OptTensor& q_start,
                    const OptTensor& q_lens, const OptTensor& ctx_lens, int64_t n, int64_t H, int64_t D, int64_t E, int64_t window,
-                   int64_t keep_first, int64_t chunk, double scale, double sink, const Tensor& out, const Tensor& status) {
+                   int64_t keep_first, int64_t chunk, double scale, double sink, const Tensor& out, int64_t o_hd, const Tensor& status) {
   oxb::RowAttnParams p{};
   const int dt = dtype_code(q, "row_attention q");
   TORCH_CHECK(k_cache.dim() == 4 && v_cache.dim() == 4 && k_cache.is_contiguous() && v_cache.is_contiguous() &&
@@ -194,8 +216,9 @@ void row_attention(const Tensor& q, int64_t q_hd, const Tensor& k_cache, const T
                   k_cache.size(0) == v_cache.size(0),
               "row_attention: caches [blocks, G, 16, head size]");
   TORCH_CHECK(k_cache.scalar_type() == q.scalar_type() && v_cache.scalar_type() == q.scalar_type() &&
-                  out.scalar_type() == q.scalar_type(),
-              "row_attention: one storage type");
+                  (out.scalar_type() == q.scalar_type() || out.scalar_type() == torch::kFloat32),
+              "row_attention: one storage type (or fp32 out)");
+  p.out_f32 = out.scalar_type() == torch::kFloat32 ? 1 : 0;
   p.G = static_cast<int>(k_cache.size(1));
   p.H = static_cast<int>(H);
   p.D = static_cast<int>(D);
@@ -229,7 +252,10 @@ void row_attention(const Tensor& q, int64_t q_hd, const Tensor& k_cache, const T
   p.chunk = static_cast<int>(chunk);
   p.scale = static_cast<float>(scale);
   p.sink = static_cast<float>(sink);
-  p.ldo = pitch(out, 1, H * E, "row_attention out");
+  if (o_hd == 0) o_hd = E;
+  TORCH_CHECK(o_hd >= E, "row_attention: o_hd");
+  p.o_hd = static_cast<int>(o_hd);
+  p.ldo = pitch(out, 1, (H - 1) * o_hd + E, "row_attention out");
   p.out = out.data_ptr();
   p.status = status_ptr(status);
   check_launch(oxb::launch_row_attention(p, dt, cur_stream()), "row_attention");
@@ -304,7 +330,7 @@ void retention_prefill(const Tensor& proj, int64_t M, int64_t H, int64_t D, int6
 }
 
 void branch_norm(const Tensor& x, int64_t rows, const OptTensor& tokens, const OptTensor& embed, double embed_scale,
-                 const std::vector<Tensor>& ys, const std::vector<OptTensor>& ws, const std::vector<double>& gains,
+                 const std::vector<OptTensor>& ys, const std::vector<OptTensor>& ws, const std::vector<double>& gains,
                  const std::vector<bool>& clears, const OptTensor& e_rows, const OptTensor& e_slot, const OptTensor& e_weight,
                  int64_t top, bool store_x, const std::vector<Tensor>& norm_ws, const std::vector<Tensor>& hs, double eps,
                  double w_offset, const OptTensor& row_map, const OptTensor& clear, const Tensor& status) {
@@ -327,11 +353,18 @@ void branch_norm(const Tensor& x, int64_t rows, const OptTensor& tokens, const O
   TORCH_CHECK(ys.size() <= oxb::kMaxBranches && ws.size() == ys.size() && gains.size() == ys.size() && clears.size() == ys.size(),
               "branch_norm: at most ", oxb::kMaxBranches, " branches");
   p.n_branches = static_cast<int>(ys.size());
+  int from_experts = 0;
   for (size_t b = 0; b < ys.size(); ++b) {
-    TORCH_CHECK(ys[b].is_cuda() && ys[b].scalar_type() == torch::kFloat32, "branch_norm: fp32 branches");
-    p.ldy = pitch(ys[b], rows, p.N, "branch_norm y");
-    TORCH_CHECK(p.ldy == ys[0].stride(0), "branch_norm: one row pitch of the branches");
-    p.y[b] = ys[b].data_ptr<float>();
+    if (given(ys[b])) {
+      TORCH_CHECK(ys[b]->is_cuda() && ys[b]->scalar_type() == torch::kFloat32, "branch_norm: fp32 branches");
+      const long long ld = pitch(*ys[b], rows, p.N, "branch_norm y");
+      TORCH_CHECK(p.ldy == 0 || p.ldy == ld, "branch_norm: one row pitch of the branches");
+      p.ldy = ld;
+      p.y[b] = ys[b]->data_ptr<float>();
+    } else {
+      ++from_experts;
+      TORCH_CHECK(given(e_rows) && !clears[b] && from_experts == 1, "branch_norm: one branch may be the expert rows");
+    }
     p.w[b] = f32(ws[b], p.N, "branch_norm branch weight");
     p.gain[b] = static_cast<float>(gains[b]);
     p.clear_y[b] = clears[b] ? 1 : 0;
@@ -479,11 +512,17 @@ void gated_norm(const Tensor& y, const Tensor& z, int64_t M, int64_t H, int64_t 
 
 // mode: see MoeRouteParams
 void moe_route(const Tensor& h, const Tensor& router, const OptTensor& logits, int64_t M, int64_t E, int64_t top, const Tensor& weight,
-               const Tensor& expert, const Tensor& slot, int64_t mode, const OptTensor& counts, const OptTensor& xs, const Tensor& status) {
+               const Tensor& expert, const Tensor& slot, int64_t mode, const OptTensor& counts, const OptTensor& xs, bool softmax,
+               int64_t groups, int64_t keep, const Tensor& status) {
   oxb::MoeRouteParams p{};
   const int dt = dtype_code(h, "moe_route h");
   TORCH_CHECK(E >= 1 && E <= oxb::kMaxExperts && top >= 1 && top <= oxb::kMaxTop && top <= E, "moe_route: at most ", oxb::kMaxExperts,
               " experts, ", oxb::kMaxTop, " of them chosen");
+  TORCH_CHECK(groups == 0 || (groups <= oxb::kMaxGroups && E % groups == 0 && keep >= 1 && keep <= groups && keep * (E / groups) >= top),
+              "moe_route: at most ", oxb::kMaxGroups, " equal groups that leave enough experts");
+  p.softmax = softmax ? 1 : 0;
+  p.groups = static_cast<int>(groups);
+  p.keep = static_cast<int>(keep);
   p.N = static_cast<int>(h.size(1));
   TORCH_CHECK(router.dim() == 2 && router.size(0) >= E && router.size(1) == p.N && router.stride(1) == 1 &&
                   router.scalar_type() == h.scalar_type() && router.is_cuda() && p.N % 8 == 0 && p.N <= 32768,
@@ -554,7 +593,8 @@ void moe_rows(const Tensor& x, const Tensor& w, const Tensor& expert, int64_t pa
   p.K = static_cast<int>(w.size(2));
   p.ldx = pitch(x, per_pair ? pairs : (pairs + top - 1) / top, p.K, "moe_rows x");
   TORCH_CHECK(p.K % 8 == 0 && p.ldx % 8 == 0 && reinterpret_cast<uintptr_t>(x.data_ptr()) % 16 == 0, "moe_rows: whole 16-byte pieces");
-  p.ldy = pitch(y, pairs, p.N, "moe_rows y");
+  TORCH_CHECK(act != 3 || p.N % 64 == 0, "moe_rows: gate and up rows in units of 32");
+  p.ldy = pitch(y, pairs, act == 3 ? p.N / 2 : p.N, "moe_rows y");
   p.x = x.data_ptr();
   p.w = w.data_ptr();
   p.y = y.data_ptr();
@@ -562,9 +602,297 @@ void moe_rows(const Tensor& x, const Tensor& w, const Tensor& expert, int64_t pa
   p.top = static_cast<int>(top);
   p.per_pair = per_pair ? 1 : 0;
   p.expert = i32(expert, pairs, "moe_rows expert");
-  TORCH_CHECK(act == 0 || act == 2, "moe_rows: act 0 or 2");
+  TORCH_CHECK(act == 0 || act == 2 || act == 3, "moe_rows: act 0, 2 or 3");
   p.act = static_cast<int>(act);
   check_launch(oxb::launch_moe_rows(p, dt, cur_stream()), "moe_rows");
+}
+
+// Two maps per head -> their difference, normed (DiffNormParams)
+void diff_norm(const Tensor& a, int64_t M, int64_t H, int64_t E, double lambda, double gain, double eps, const Tensor& out) {
+  oxb::DiffNormParams p{};
+  TORCH_CHECK(a.is_cuda() && a.scalar_type() == torch::kFloat32, "diff_norm: fp32 maps");
+  p.lda = pitch(a, M, 2 * H * E, "diff_norm a");
+  p.a = a.data_ptr<float>();
+  p.M = static_cast<int>(M);
+  p.H = static_cast<int>(H);
+  p.E = static_cast<int>(E);
+  p.lambda = static_cast<float>(lambda);
+  p.gain = static_cast<float>(gain);
+  p.eps = static_cast<float>(eps);
+  p.ldo = pitch(out, M, H * E, "diff_norm out");
+  p.out = out.data_ptr();
+  check_launch(oxb::launch_diff_norm(p, dtype_code(out, "diff_norm out"), cur_stream()), "diff_norm");
+}
+
+// kv: columns of the latent, its norm weight and the cache; none for a layer that reads another one's cache
+void latent_rows(const Tensor& proj, int64_t M, int64_t Q, const Tensor& q_norm, const Tensor& q_out, int64_t kv_col, int64_t R,
+                 const OptTensor& kv_norm, const OptTensor& cache, const OptTensor& slots, const OptTensor& freq_hi,
+                 const OptTensor& freq_lo, bool interleaved, double gain, const Tensor& positions, double eps, const Tensor& status) {
+  oxb::LatentRowsParams p{};
+  const int dt = dtype_code(q_out, "latent_rows q_out");
+  p.proj_f32 = dtype_code(proj, "latent_rows proj");
+  TORCH_CHECK(dt == 0 || p.proj_f32 == 1, "latent_rows: fp32 rows take fp32 projections");
+  TORCH_CHECK(Q >= 1 && R >= 0 && Q + R <= 49152, "latent_rows: sizes");
+  p.proj = proj.data_ptr();
+  p.M = static_cast<int>(M);
+  p.Q = static_cast<int>(Q);
+  p.R = static_cast<int>(R);
+  p.kv_col = static_cast<int>(kv_col);
+  p.q_norm = f32(q_norm, Q, "latent_rows q_norm");
+  p.ldq = pitch(q_out, M, Q, "latent_rows q_out");
+  p.q_out = q_out.data_ptr();
+  p.eps = static_cast<float>(eps);
+  p.positions = i32(positions, M, "latent_rows positions");
+  p.ld = pitch(proj, M, Q, "latent_rows proj");
+  if (R > 0) {
+    TORCH_CHECK(given(kv_norm) && given(cache) && given(slots), "latent_rows: norm weight, cache and slots of the latent");
+    TORCH_CHECK(cache->scalar_type() == q_out.scalar_type() && cache->is_contiguous() && cache->dim() == 4 && cache->size(1) == 1 &&
+                    cache->size(2) == 16,
+                "latent_rows: cache [blocks, 1, 16, values]");
+    p.CP = static_cast<int>(cache->size(3));
+    p.rot = rotary(freq_hi, freq_lo, interleaved, gain, p.CP - R);
+    TORCH_CHECK(R + p.rot.dims <= p.CP && kv_col >= Q && p.ld >= kv_col + R + p.rot.dims && proj.size(1) >= kv_col + R + p.rot.dims,
+                "latent_rows: columns");
+    p.kv_norm = f32(*kv_norm, R, "latent_rows kv_norm");
+    p.cache = cache->data_ptr();
+    TORCH_CHECK(slots->is_cuda() && slots->scalar_type() == torch::kInt64 && slots->numel() >= M, "latent_rows: slots int64");
+    p.slots = reinterpret_cast<const long long*>(slots->data_ptr<int64_t>());
+    p.num_slots = cache->size(0) * 16;
+  }
+  p.status = status_ptr(status);
+  check_launch(oxb::launch_latent_rows(p, dt, cur_stream()), "latent_rows");
+}
+
+void latent_gather(const Tensor& cache, const Tensor& block_tables, const Tensor& ctx_lens, const Tensor& row0, int64_t seq0, int64_t n_seqs,
+                   int64_t max_pages, const Tensor& out, const Tensor& status) {
+  oxb::LatentGatherParams p{};
+  TORCH_CHECK(dtype_code(cache, "latent_gather cache") == 0 && dtype_code(out, "latent_gather out") == 0 && cache.dim() == 4 &&
+                  cache.is_contiguous() && cache.size(1) == 1 && cache.size(2) == 16 && cache.size(3) % 8 == 0,
+              "latent_gather: bf16 cache [blocks, 1, 16, values]");
+  p.CP = static_cast<int>(cache.size(3));
+  TORCH_CHECK(out.dim() == 2 && out.is_contiguous() && out.size(1) == p.CP, "latent_gather: out [rows, values]");
+  TORCH_CHECK(block_tables.dim() == 2 && block_tables.is_contiguous() && block_tables.size(0) >= seq0 + n_seqs, "latent_gather: block_tables");
+  p.cache = cache.data_ptr();
+  p.num_blocks = static_cast<int>(cache.size(0));
+  p.block_tables = i32(block_tables, 1, "latent_gather block_tables");
+  p.max_blocks = static_cast<int>(block_tables.size(1));
+  p.ctx_lens = i32(ctx_lens, seq0 + n_seqs, "latent_gather ctx_lens");
+  p.row0 = i32(row0, seq0 + n_seqs, "latent_gather row0");
+  p.seq0 = static_cast<int>(seq0);
+  p.n_seqs = static_cast<int>(n_seqs);
+  p.max_pages = static_cast<int>(max_pages);
+  p.out = out.data_ptr();
+  p.rows = out.size(0);
+  p.status = status_ptr(status);
+  check_launch(oxb::launch_latent_gather(p, cur_stream()), "latent_gather");
+}
+
+void latent_decode(const Tensor& q, const Tensor& cache, const Tensor& block_tables, const Tensor& seq_lens, const Tensor& pages_per_split,
+                   int64_t rows, int64_t R, int64_t max_splits, double scale, const Tensor& part_o, const Tensor& part_ml, const Tensor& out,
+                   int64_t o_hd, const Tensor& status) {
+  oxb::LatentDecodeParams p{};
+  TORCH_CHECK(dtype_code(q, "latent_decode q") == 0 && dtype_code(cache, "latent_decode cache") == 0 && dtype_code(out, "latent_decode out") == 0,
+              "latent_decode: bf16");
+  TORCH_CHECK(cache.dim() == 4 && cache.is_contiguous() && cache.size(1) == 1 && cache.size(2) == 16, "latent_decode: cache [blocks, 1, 16, values]");
+  p.CP = static_cast<int>(cache.size(3));
+  TORCH_CHECK(q.dim() == 3 && q.size(0) >= rows && q.size(2) == p.CP && q.is_contiguous(), "latent_decode: q [rows, heads, values]");
+  p.H = static_cast<int>(q.size(1));
+  p.R = static_cast<int>(R);
+  p.rows = static_cast<int>(rows);
+  TORCH_CHECK(R >= 1 && R <= p.CP && oxb::latent_decode_ok(p.R, p.CP) && max_splits >= 1 && max_splits <= 64, "latent_decode: sizes");
+  TORCH_CHECK(reinterpret_cast<uintptr_t>(q.data_ptr()) % 16 == 0 && reinterpret_cast<uintptr_t>(cache.data_ptr()) % 16 == 0, "latent_decode: alignment");
+  p.q = reinterpret_cast<const __nv_bfloat16*>(q.data_ptr());
+  p.cache = reinterpret_cast<const __nv_bfloat16*>(cache.data_ptr());
+  p.num_blocks = static_cast<int>(cache.size(0));
+  TORCH_CHECK(block_tables.dim() == 2 && block_tables.is_contiguous() && block_tables.size(0) >= rows, "latent_decode: block_tables");
+  p.block_tables = i32(block_tables, 1, "latent_decode block_tables");
+  p.max_blocks = static_cast<int>(block_tables.size(1));
+  p.seq_lens = i32(seq_lens, rows, "latent_decode seq_lens");
+  p.pages_per_split = i32(pages_per_split, 1, "latent_decode pages_per_split");
+  p.max_splits = static_cast<int>(max_splits);
+  p.scale_log2 = static_cast<float>(scale * 1.4426950408889634);
+  p.part_o = const_cast<float*>(f32(part_o, rows * p.H * max_splits * R, "latent_decode part_o"));
+  p.part_ml = const_cast<float*>(f32(part_ml, rows * p.H * max_splits * 2, "latent_decode part_ml"));
+  TORCH_CHECK(o_hd >= R, "latent_decode: o_hd");
+  p.o_hd = static_cast<int>(o_hd);
+  p.ldo = pitch(out, rows, (p.H - 1) * o_hd + R, "latent_decode out");
+  p.out = reinterpret_cast<__nv_bfloat16*>(out.data_ptr());
+  p.status = status_ptr(status);
+  check_launch(oxb::launch_latent_decode(p, cur_stream()), "latent_decode");
+}
+
+// Causal attention of prompt tiles over plain rows of keys and values: kv [rows, columns], head g's keys from column
+// g * dk on, its values from v_col0 + g * dv on; position t of sequence s is row row0[s] + t.
+void prefill_rows(const Tensor& q, const Tensor& kv, int64_t dk, int64_t dv, int64_t v_col0, int64_t G, const Tensor& row0,
+                  const Tensor& tile_seq, const Tensor& tile_q0, const Tensor& q_start, const Tensor& q_lens, const Tensor& ctx_lens,
+                  const Tensor& out, int64_t n_tiles, double scale, int64_t out_d, const Tensor& status) {
+  const int bkv = oxb::prefill_wide_tile(static_cast<int>(dk), static_cast<int>(dv));
+  TORCH_CHECK(bkv > 0, "prefill_rows: head sizes ", dk, ", ", dv);
+  TORCH_CHECK(dtype_code(q, "prefill_rows q") == 0 && dtype_code(kv, "prefill_rows kv") == 0, "prefill_rows: bf16");
+  TORCH_CHECK(q.dim() == 3 && q.size(2) == dk && q.stride(2) == 1 && q.stride(1) == dk, "prefill_rows: q [rows, heads, dk]");
+  TORCH_CHECK(kv.dim() == 2 && kv.stride(1) == 1 && kv.size(1) >= v_col0 + G * dv && v_col0 >= G * dk && v_col0 % 8 == 0 && kv.stride(0) % 8 == 0,
+              "prefill_rows: kv columns");
+  oxb::PrefillAttnParams p{};
+  p.Hq = static_cast<int>(q.size(1));
+  p.Hkv = static_cast<int>(G);
+  TORCH_CHECK(G >= 1 && p.Hq % p.Hkv == 0 && out_d >= 1 && out_d <= dv, "prefill_rows: heads");
+  p.q = reinterpret_cast<const __nv_bfloat16*>(q.data_ptr());
+  p.q_stride = q.stride(0);
+  TORCH_CHECK(tile_seq.is_cuda() && tile_seq.numel() >= n_tiles && tile_q0.numel() >= n_tiles, "prefill_rows: tiles");
+  p.tile_seq = tile_seq.data_ptr<int>();
+  p.tile_q0 = tile_q0.data_ptr<int>();
+  p.q_start = i32(q_start, 1, "prefill_rows q_start");
+  p.q_lens = i32(q_lens, 1, "prefill_rows q_lens");
+  p.ctx_lens = i32(ctx_lens, 1, "prefill_rows ctx_lens");
+  p.kv_row0 = i32(row0, 1, "prefill_rows row0");
+  p.block_tables = p.kv_row0;   // not read in this form
+  p.k_hd = static_cast<int>(dk);
+  p.v_col0 = static_cast<int>(v_col0);
+  p.v_hd = static_cast<int>(dv);
+  p.out_stride = pitch(out, 1, p.Hq * out_d, "prefill_rows out");
+  if (out.scalar_type() == torch::kFloat32) p.out_f32 = out.data_ptr<float>();
+  else p.out = reinterpret_cast<__nv_bfloat16*>(out.data_ptr());
+  p.out_d = static_cast<int>(out_d);
+  p.exact_p = 1;
+  p.scale_log2 = static_cast<float>(scale * 1.4426950408889634);
+  const auto bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+  const auto sw = CU_TENSOR_MAP_SWIZZLE_128B;
+  CUtensorMap tmQ = oxb::make_tma_map(q.data_ptr(), bf, 2, 2, static_cast<uint64_t>(p.Hq) * dk, q.size(0), 1, static_cast<uint64_t>(q.stride(0)) * 2,
+                                      0, 64, 128, 1, sw);
+  CUtensorMap tmKV = oxb::make_tma_map(kv.data_ptr(), bf, 2, 2, static_cast<uint64_t>(v_col0 + G * dv), kv.size(0), 1,
+                                       static_cast<uint64_t>(kv.stride(0)) * 2, 0, 64, bkv, 1, sw);
+  oxb::launch_prefill_wide(tmQ, tmKV, tmKV, p, static_cast<int>(n_tiles), static_cast<int>(dk), static_cast<int>(dv), status_ptr(status), cur_stream());
+  check_launch("prefill_rows");
+}
+
+// The paged form of the same for heads of up to 256 values: q [rows, H, D], caches [blocks, G, 16, D].
+void prefill_pages(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& block_tables, const Tensor& tile_seq,
+                   const Tensor& tile_q0, const Tensor& q_start, const Tensor& q_lens, const Tensor& ctx_lens, const Tensor& out,
+                   int64_t n_tiles, double scale, int64_t out_d, const Tensor& status) {
+  const int dk = static_cast<int>(q.size(2)), dv = static_cast<int>(v_cache.size(3));
+  const int bkv = oxb::prefill_wide_tile(dk, dv);
+  TORCH_CHECK(bkv > 0, "prefill_pages: head sizes ", dk, ", ", dv);
+  TORCH_CHECK(dtype_code(q, "prefill_pages q") == 0 && dtype_code(k_cache, "prefill_pages k") == 0 && dtype_code(v_cache, "prefill_pages v") == 0,
+              "prefill_pages: bf16");
+  TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && q.stride(1) == dk && k_cache.dim() == 4 && k_cache.is_contiguous() && v_cache.is_contiguous() &&
+                  k_cache.size(2) == 16 && v_cache.size(2) == 16 && k_cache.size(3) == dk && k_cache.size(0) == v_cache.size(0) &&
+                  k_cache.size(1) == v_cache.size(1),
+              "prefill_pages: q [rows, heads, D], caches [blocks, G, 16, D]");
+  oxb::PrefillAttnParams p{};
+  p.Hq = static_cast<int>(q.size(1));
+  p.Hkv = static_cast<int>(k_cache.size(1));
+  TORCH_CHECK(p.Hq % p.Hkv == 0 && out_d >= 1 && out_d <= dv, "prefill_pages: heads");
+  p.q = reinterpret_cast<const __nv_bfloat16*>(q.data_ptr());
+  p.q_stride = q.stride(0);
+  TORCH_CHECK(block_tables.dim() == 2 && block_tables.is_contiguous(), "prefill_pages: block_tables");
+  p.block_tables = i32(block_tables, 1, "prefill_pages block_tables");
+  p.max_blocks = static_cast<int>(block_tables.size(1));
+  p.num_blocks = static_cast<int>(k_cache.size(0));
+  p.tile_seq = i32(tile_seq, n_tiles, "prefill_pages tile_seq");
+  p.tile_q0 = i32(tile_q0, n_tiles, "prefill_pages tile_q0");
+  p.q_start = i32(q_start, 1, "prefill_pages q_start");
+  p.q_lens = i32(q_lens, 1, "prefill_pages q_lens");
+  p.ctx_lens = i32(ctx_lens, 1, "prefill_pages ctx_lens");
+  p.out_stride = pitch(out, 1, p.Hq * out_d, "prefill_pages out");
+  if (out.scalar_type() == torch::kFloat32) p.out_f32 = out.data_ptr<float>();
+  else p.out = reinterpret_cast<__nv_bfloat16*>(out.data_ptr());
+  p.out_d = static_cast<int>(out_d);
+  p.exact_p = 1;
+  p.scale_log2 = static_cast<float>(scale * 1.4426950408889634);
+  const auto bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+  const auto sw = CU_TENSOR_MAP_SWIZZLE_128B;
+  const uint64_t kv_rows = static_cast<uint64_t>(p.num_blocks) * p.Hkv * 16;
+  CUtensorMap tmQ = oxb::make_tma_map(q.data_ptr(), bf, 2, 2, static_cast<uint64_t>(p.Hq) * dk, q.size(0), 1, static_cast<uint64_t>(q.stride(0)) * 2,
+                                      0, 64, 128, 1, sw);
+  CUtensorMap tmK = oxb::make_tma_map(k_cache.data_ptr(), bf, 2, 2, dk, kv_rows, 1, static_cast<uint64_t>(dk) * 2, 0, 64, 16, 1, sw);
+  CUtensorMap tmV = oxb::make_tma_map(v_cache.data_ptr(), bf, 2, 2, dv, kv_rows, 1, static_cast<uint64_t>(dv) * 2, 0, 64, 16, 1, sw);
+  oxb::launch_prefill_wide(tmQ, tmK, tmV, p, static_cast<int>(n_tiles), dk, dv, status_ptr(status), cur_stream());
+  check_launch("prefill_pages");
+}
+
+// Sizes, gates and state of a matrix memory. proj: rows q | k | v | gate.
+oxb::MemoryParams memory_common(const Tensor& proj, int64_t M, int64_t H, int64_t D, int64_t E, const OptTensor& z, const Tensor& z_bias,
+                                double cap, double eps, const Tensor& norm_w, const Tensor& state, const Tensor& state_m, const Tensor& out,
+                                const Tensor& status) {
+  oxb::MemoryParams p{};
+  TORCH_CHECK(H >= 1 && D >= 1 && E >= 1 && D <= 4096 && E <= 4096 && cap > 0, "memory: sizes");
+  p.proj = proj.data_ptr();
+  p.proj_f32 = dtype_code(proj, "memory proj");
+  TORCH_CHECK(dtype_code(out, "memory out") == 0 || p.proj_f32 == 1, "memory: fp32 rows take fp32 projections");
+  p.ld = pitch(proj, M, 2 * H * (D + E), "memory proj");
+  p.H = static_cast<int>(H);
+  p.D = static_cast<int>(D);
+  p.E = static_cast<int>(E);
+  if (given(z)) {
+    TORCH_CHECK(z->is_cuda() && z->scalar_type() == torch::kFloat32, "memory: fp32 gate pre-activations");
+    p.ldz = pitch(*z, M, 2 * H, "memory z");
+    p.z = z->data_ptr<float>();
+  }
+  p.z_bias = f32(z_bias, 2 * H, "memory z_bias");
+  p.cap = static_cast<float>(cap);
+  p.scale = static_cast<float>(1.0 / std::sqrt(static_cast<double>(D)));
+  p.eps = static_cast<float>(eps);
+  p.norm_w = f32(norm_w, H * E, "memory norm_w");
+  TORCH_CHECK(state.dim() == 3 && state.size(1) == H && state.size(2) == D * E + D && state_m.dim() == 2 && state_m.size(1) == H &&
+                  state_m.size(0) == state.size(0),
+              "memory: state [slots, H, D * E + D], maxima [slots, H]");
+  p.state = const_cast<float*>(f32(state, 1, "memory state"));
+  p.state_m = const_cast<float*>(f32(state_m, 1, "memory state_m"));
+  p.num_slots = static_cast<int>(state.size(0));
+  p.ldo = pitch(out, M, H * E, "memory out");
+  p.out = out.data_ptr();
+  p.status = status_ptr(status);
+  return p;
+}
+
+void memory_decode(const Tensor& proj, int64_t rows, int64_t H, int64_t D, int64_t E, const OptTensor& z, const OptTensor& h, const OptTensor& z_w,
+                   const Tensor& z_bias, double cap, double eps, const Tensor& norm_w, const Tensor& state, const Tensor& state_m,
+                   const Tensor& row_slots, const Tensor& positions, const Tensor& out, const Tensor& status) {
+  oxb::MemoryParams p = memory_common(proj, rows, H, D, E, z, z_bias, cap, eps, norm_w, state, state_m, out, status);
+  if (!given(z)) {
+    TORCH_CHECK(given(h) && given(z_w) && dtype_code(*h, "memory h") == 0 && dtype_code(*z_w, "memory z_w") == 0 && z_w->dim() == 2 &&
+                    z_w->size(0) >= 2 * H && z_w->stride(1) == 1 && h->size(1) == z_w->size(1) && h->size(1) % 4 == 0,
+                "memory_decode: bf16 rows and gate weights");
+    p.ldh = pitch(*h, rows, h->size(1), "memory h");
+    p.h = h->data_ptr();
+    p.z_w = z_w->data_ptr();
+    p.ldw = z_w->stride(0);
+    p.N = static_cast<int>(h->size(1));
+    TORCH_CHECK(p.ldh % 4 == 0 && p.ldw % 4 == 0 && reinterpret_cast<uintptr_t>(p.h) % 8 == 0 && reinterpret_cast<uintptr_t>(p.z_w) % 8 == 0,
+                "memory_decode: alignment");
+  }
+  p.row_slots = i32(row_slots, rows, "memory_decode row_slots");
+  p.positions = i32(positions, rows, "memory_decode positions");
+  p.rows = static_cast<int>(rows);
+  check_launch(oxb::launch_memory_decode(p, dtype_code(out, "memory out"), cur_stream()), "memory_decode");
+}
+
+void memory_prefill(const Tensor& proj, int64_t M, int64_t H, int64_t D, int64_t E, const Tensor& z, const Tensor& z_bias, double cap, double eps,
+                    const Tensor& norm_w, const Tensor& state, const Tensor& state_m, const Tensor& seq_slots, const Tensor& tile_seq,
+                    const Tensor& tile_q0, const Tensor& q_start, const Tensor& q_lens, const Tensor& ctx_lens, int64_t n_tiles, int64_t n_seqs,
+                    const Tensor& ws, bool chunks, const Tensor& out, const Tensor& status) {
+  oxb::MemoryParams p = memory_common(proj, M, H, D, E, z, z_bias, cap, eps, norm_w, state, state_m, out, status);
+  const int dt = dtype_code(out, "memory out");
+  p.seq_slots = i32(seq_slots, n_seqs, "memory_prefill seq_slots");
+  p.tile_seq = i32(tile_seq, n_tiles, "memory_prefill tile_seq");
+  p.tile_q0 = i32(tile_q0, n_tiles, "memory_prefill tile_q0");
+  p.q_start = i32(q_start, n_seqs, "memory_prefill q_start");
+  p.q_lens = i32(q_lens, n_seqs, "memory_prefill q_lens");
+  p.ctx_lens = i32(ctx_lens, n_seqs, "memory_prefill ctx_lens");
+  p.n_tiles = static_cast<int>(n_tiles);
+  p.n_seqs = static_cast<int>(n_seqs);
+  if (chunks) {
+    TORCH_CHECK(dt == 0 && oxb::memory_chunks_ok(p.D, p.E), "memory_prefill: chunked form");
+    const int64_t n = 2 * n_tiles * H;
+    p.ws = const_cast<float*>(f32(ws, n * (D * E + D + 3), "memory_prefill ws"));
+    p.ws_m = p.ws + n * (D * E + D);
+    check_launch(oxb::launch_memory_chunks(p, cur_stream()), "memory_prefill");
+  } else {
+    TORCH_CHECK(D <= 1600, "memory_prefill: head size");
+    p.o_buf = const_cast<float*>(f32(ws, M * H * E + n_seqs * H * (D + 1), "memory_prefill ws"));
+    p.n_buf = p.o_buf + M * H * E;
+    check_launch(oxb::launch_memory_scan(p, dt, cur_stream()), "memory_prefill");
+  }
 }
 
 void gemm_f32(const Tensor& a, const Tensor& w, const Tensor& out) {
@@ -613,6 +941,19 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("moe_route", &moe_route);
   m.def("moe_scatter", &moe_scatter);
   m.def("moe_rows", &moe_rows);
+  m.def("diff_norm", &diff_norm);
+  m.def("latent_rows", &latent_rows);
+  m.def("latent_gather", &latent_gather);
+  m.def("latent_decode", &latent_decode);
+  m.def("latent_decode_ok", [](int64_t R, int64_t CP) { return oxb::latent_decode_ok(static_cast<int>(R), static_cast<int>(CP)); });
+  m.def("prefill_rows", &prefill_rows);
+  m.def("prefill_pages", &prefill_pages);
+  m.def("prefill_wide_tile", [](int64_t dk, int64_t dv) { return oxb::prefill_wide_tile(static_cast<int>(dk), static_cast<int>(dv)); });
+  m.def("memory_decode", &memory_decode);
+  m.def("memory_prefill", &memory_prefill);
+  m.def("memory_chunks_ok", [](int64_t D, int64_t E) { return oxb::memory_chunks_ok(static_cast<int>(D), static_cast<int>(E)); });
+  m.attr("MEMORY_CHUNK") = oxb::kMemChunk;
+  m.attr("MAX_GROUPS") = oxb::kMaxGroups;
   m.def("gemm_f32", &gemm_f32);
   m.def("glu_f32", &glu_f32);
 }

@@ -29,6 +29,10 @@ struct DecodeAttnParams {
   float scale_log2;  // softmax scale * log2(e)
   // score (times log2(e)) of a sink: one more term of the softmax denominator, without a value
   float sink_log2 = -INFINITY;
+  // Differential attention (diff != 0): query heads 2 h and 2 h + 1 are the two maps of head h. The merge writes
+  // o = a1 - diff_lambda a2, o / sqrt(mean(o^2) + diff_eps) * diff_gain, one row of out_d values per pair.
+  int diff;
+  float diff_lambda, diff_gain, diff_eps;
   // Bounds check of block-table entries: an id outside [0, num_blocks) is recorded in *status
   // (kStatusBadIndex) and page 0 is read instead. num_blocks <= 0 or status == nullptr: no check.
   int num_blocks;
@@ -72,7 +76,17 @@ struct PrefillAttnParams {
   float sink_log2 = -INFINITY;
   int num_blocks;  // bound for block-table entries (<= 0: unchecked), violations go to *status
   int* status;
+  float* out_f32;  // fp32 rows instead of `out` (the same pitch), or nullptr
+  // Keys and values in plain rows instead of pages (kv_row0 != nullptr): position t of sequence s is row kv_row0[s] + t,
+  // head g's keys start at column g * k_hd, its values at column v_col0 + g * v_hd
+  const int* kv_row0;
+  int k_hd, v_col0, v_hd;
 };
+
+// Head sizes (keys, values) of the plain-row form and of unequal or larger sizes than 128.
+void launch_prefill_wide(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV,
+                         const PrefillAttnParams& p, int n_tiles, int dk, int dv, int* status, cudaStream_t stream);
+int prefill_wide_tile(int dk, int dv);   // KV positions per tile, 0: sizes that are not built
 
 void launch_paged_prefill_tc(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV,
                              const PrefillAttnParams& p, int n_tiles, int head_dim, int* status,

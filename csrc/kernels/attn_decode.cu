@@ -87,7 +87,7 @@ __device__ __forceinline__ int visible_from(const DecodeAttnParams& p, int seq_l
   return (p.window > 0 && seq_len > p.window) ? seq_len - p.window : 0;
 }
 
-// D = head dim (64 or 128); NT = number of 8-head column tiles (group size <= 8*NT).
+// D = head dim (64, 128 or 256); NT = number of 8-head column tiles (group size <= 8*NT).
 // MASS: also record the per-page softmax statistics of every head (see DecodeAttnParams::page_ml).
 // EXACT: the softmax weights enter the value product as hi + lo bf16 terms (DecodeAttnParams::exact_p).
 template <int D, int NT, bool MASS, bool EXACT>
@@ -465,6 +465,43 @@ __global__ void __launch_bounds__(D) decode_merge_kernel(const DecodeAttnParams 
   }
 }
 
+// The same for the two maps of one head of differential attention, then their difference and its norm. grid (seq, head).
+template <int D>
+__global__ void __launch_bounds__(D) decode_merge_diff_kernel(const DecodeAttnParams p) {
+  __shared__ float s_red[D / 32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int seq = blockIdx.x, head = blockIdx.y, d = threadIdx.x;
+  float a[2];
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    const long long base = (static_cast<long long>(seq) * p.Hq + 2 * head + m) * p.max_splits;
+    float M = -INFINITY;
+    for (int s = 0; s < p.max_splits; ++s) M = fmaxf(M, p.part_ml[(base + s) * 2]);
+    float acc = 0.f, L = 0.f;
+    for (int s = 0; s < p.max_splits; ++s) {
+      const float ms = p.part_ml[(base + s) * 2];
+      if (ms == -INFINITY) continue;
+      const float f = ex2(ms - M);
+      acc += f * p.part_o[(base + s) * D + d];
+      L += f * p.part_ml[(base + s) * 2 + 1];
+    }
+    a[m] = L > 0.f ? acc / L : 0.f;
+  }
+  const int od = p.out_d > 0 ? p.out_d : D;
+  const float o = d < od ? a[0] - p.diff_lambda * a[1] : 0.f;
+  float ss = o * o;
+#pragma unroll
+  for (int x = 16; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+  if ((d & 31) == 0) s_red[d >> 5] = ss;
+  __syncthreads();
+  ss = 0.f;
+#pragma unroll
+  for (int x = 0; x < D / 32; ++x) ss += s_red[x];
+  const float r = p.diff_gain / sqrtf(ss / static_cast<float>(od) + p.diff_eps);
+  if (d < od) p.out[static_cast<long long>(seq) * p.out_stride + head * od + d] = __float2bfloat16(o * r);
+}
+
 // block_mass[seq, page] = sum_h page_sum[h] * 2^(page_max[h] - M_h) / L_h, with (M_h, L_h) the merged
 // statistics of head h over all splits: the softmax probability mass the step's query put on the page.
 __global__ void __launch_bounds__(128) block_mass_kernel(const DecodeAttnParams p) {
@@ -513,7 +550,11 @@ void launch_split(const DecodeAttnParams& p, dim3 grid, cudaStream_t stream) {
   constexpr size_t ring = static_cast<size_t>(kWarps) * kRing * 2 * kPage * D * 2;
   constexpr size_t merge = sizeof(float) * kWarps * 8 * NT * (D + 2);
   constexpr size_t smem = ring > merge ? ring : merge;
-  if (p.page_ml != nullptr) {
+  if constexpr (D == 256) {  // softmax weights always in two terms, no block mass
+    auto kern = paged_decode_kernel<D, NT, false, true>;
+    ensure_dynamic_smem(kern, smem);
+    launch_kernel(kern, grid, dim3(kWarps * 32), smem, stream, /*pdl=*/true, false, p);
+  } else if (p.page_ml != nullptr) {
     auto kern = paged_decode_kernel<D, NT, true, false>;
     ensure_dynamic_smem(kern, smem);
     launch_kernel(kern, grid, dim3(kWarps * 32), smem, stream, /*pdl=*/true, false, p);
@@ -532,7 +573,12 @@ cudaError_t launch_paged_decode(const DecodeAttnParams& p, int batch, int head_d
   const int G = p.Hq / p.Hkv;
   dim3 grid(batch, p.Hkv, p.max_splits);
   dim3 mgrid(batch, p.Hq);
-  if (head_dim == 128) {
+  if (head_dim == 256) {
+    if (G <= 8)
+      launch_split<256, 1>(p, grid, stream);
+    else
+      launch_split<256, 2>(p, grid, stream);
+  } else if (head_dim == 128) {
     if (G <= 8)
       launch_split<128, 1>(p, grid, stream);
     else
@@ -546,7 +592,16 @@ cudaError_t launch_paged_decode(const DecodeAttnParams& p, int batch, int head_d
   // a failed first launch leaves the partials stale: do not merge them into `out`
   const cudaError_t e = cudaPeekAtLastError();
   if (e != cudaSuccess) return e;
-  if (head_dim == 128)
+  if (p.diff) {
+    const dim3 dgrid(batch, p.Hq / 2);
+    if (head_dim == 256) launch_kernel(decode_merge_diff_kernel<256>, dgrid, dim3(256), 0, stream, /*pdl=*/true, false, p);
+    else if (head_dim == 128) launch_kernel(decode_merge_diff_kernel<128>, dgrid, dim3(128), 0, stream, /*pdl=*/true, false, p);
+    else launch_kernel(decode_merge_diff_kernel<64>, dgrid, dim3(64), 0, stream, /*pdl=*/true, false, p);
+    return cudaPeekAtLastError();
+  }
+  if (head_dim == 256)
+    launch_kernel(decode_merge_kernel<256>, mgrid, dim3(256), 0, stream, /*pdl=*/true, false, p);
+  else if (head_dim == 128)
     launch_kernel(decode_merge_kernel<128>, mgrid, dim3(128), 0, stream, /*pdl=*/true, false, p);
   else
     launch_kernel(decode_merge_kernel<64>, mgrid, dim3(64), 0, stream, /*pdl=*/true, false, p);

@@ -81,11 +81,13 @@ __global__ void __launch_bounds__(kKeys) row_attention_kernel(const RowAttnParam
     }
     __syncthreads();
   }
-  T* o = static_cast<T*>(p.out) + static_cast<long long>(row) * p.ldo + head * p.E;
+  const long long at = static_cast<long long>(row) * p.ldo + head * p.o_hd;
 #pragma unroll
   for (int i = 0; i < kMaxV; ++i) {
     const int c = threadIdx.x + i * kKeys;
-    if (c < p.E) o[c] = from_f<T>(acc[i] / l_run);
+    if (c >= p.E) continue;
+    if (p.out_f32) static_cast<float*>(p.out)[at + c] = acc[i] / l_run;
+    else static_cast<T*>(p.out)[at + c] = from_f<T>(acc[i] / l_run);
   }
 }
 

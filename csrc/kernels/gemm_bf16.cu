@@ -264,7 +264,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
   const int total_kb = FP4 ? p.kb_total : (p.K + BK - 1) / BK;
-  const bool grouped = p.group_counts != nullptr;
+  const bool grouped = p.n_groups > 0;
   const int n_tiles = (p.N + BN - 1) / BN;
   const int m_tiles = p.m_tiles;
   const int n_work = n_tiles * m_tiles * p.splits;
@@ -309,7 +309,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
     int acc = 0;
     for (int e0 = 0; e0 < p.n_groups; e0 += 32) {
       const int e = e0 + lane;
-      const int rows = e < p.n_groups ? static_cast<int>(__ldcg(p.group_counts + e)) : 0;
+      const int rows = e >= p.n_groups ? 0 : (p.group_counts != nullptr ? static_cast<int>(__ldcg(p.group_counts + e)) : p.M);
       const int tiles = (rows + BM - 1) / BM;
       int incl = tiles;
 #pragma unroll
@@ -966,7 +966,7 @@ void launch_impl(const CUtensorMap& tmA, const CUtensorMap& tmB, const GemmParam
                  cudaStream_t stream) {
   using L = SmemLayout<BN, STAGES, MT, KIND>;
   auto kern = gemm_bf16_kernel<BN, STAGES, MT, KIND>;
-  const size_t smem = L::kTotal + (p.group_counts != nullptr ? (2 * static_cast<size_t>(p.n_groups) + 1) * sizeof(int) : 0);
+  const size_t smem = L::kTotal + (p.n_groups > 0 ? (2 * static_cast<size_t>(p.n_groups) + 1) * sizeof(int) : 0);
   ensure_dynamic_smem(kern, smem);
   const int sms = sm_count();
   const int n_work = ((p.N + BN - 1) / BN) * p.m_tiles * p.splits;

@@ -42,8 +42,8 @@ struct GemmParams {
   long long c_group_stride;   // elements between groups of C
   const __nv_bfloat16* bias;  // optional, length N (per group: bias + g * N)
   // --- grouped (MoE) mode ---
-  const uint32_t* group_counts;  // [n_groups] rows used in each group (device); nullptr = dense
-  int n_groups;
+  const uint32_t* group_counts;  // [n_groups] rows used in each group (device); nullptr = M rows in every group
+  int n_groups;                  // 0 = dense
   int packed_rows;    // 1: A and C are [rows, ..] with the groups one after the other, each from a multiple of 128 on
                       // (instead of one slab of the same height per group)
   const RowMeta* row_meta;       // [n_groups, meta_group_stride] routing of each slab row

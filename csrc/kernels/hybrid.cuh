@@ -45,11 +45,12 @@ struct StreamNormParams {
 };
 cudaError_t launch_stream_norm(const StreamNormParams& p, int dtype, cudaStream_t stream);
 
-// What stands between two layers whose mixer and feed-forward run side by side on one residual stream x. With N
-// values per row:
+// What stands between two layers whose mixer and feed-forward run side by side on one residual stream x, or between
+// two sublayers with a norm on either side. With N values per row:
 //   tokens given : x = embed[token] * embed_scale
 //   else         : x += sum_b gain[b] * (w[b] ? y_b / sqrt(mean(y_b^2) + eps) * w[b] : y_b)   (dense branches)
-//                     + sum_c weight[c] * expert_rows[slot[c]]                                (chosen experts)
+//                     + e,   e = sum_c weight[c] * expert_rows[slot[c]]                       (chosen experts)
+//                  where y_b of a branch without rows is e, which is then not added a second time
 //   then         : h_o = x / sqrt(mean(x^2) + eps) * (w_offset + norm_w[o])                   for every output o
 // x is written back when store_x is set. Where clear_y is set for a branch, its rows are zeroed on the way (the
 // split-K GEMM of the layer that follows adds into them).
@@ -63,7 +64,7 @@ struct BranchNormParams {
   int vocab;
   float embed_scale;
   int n_branches;
-  float* y[kMaxBranches];   // [rows, ldy]
+  float* y[kMaxBranches];   // [rows, ldy], or nullptr: the weighted expert rows
   const float* w[kMaxBranches];
   float gain[kMaxBranches];
   int clear_y[kMaxBranches];
@@ -97,14 +98,21 @@ struct RotaryParams {
   float gain;               // factor on sin and cos
 };
 
-// Projection rows q | k | v -> per-head vectors: optional RMS norm over the whole q (k) projection with
-// plain weights, rotation of q and k, k times k_scale. q goes to a dense buffer (head stride q_hd); k goes
-// to a dense buffer (k_out) or, with v, into the paged cache [blocks, G, 16, DP] / [blocks, G, 16, EP].
+// Projection rows q | k | v -> per-head vectors: optional bias, optional RMS norm over the whole q (k) projection
+// with plain weights, rotation of q and k, k times k_scale, q times a temperature that grows with the position
+// (1 + t_coef ln(floor((p + 1) / t_every) + 1)). q goes to a dense buffer (head stride q_hd); k goes to a dense buffer
+// (k_out) or, with v, into the paged cache [blocks, G / maps, 16, DP] / [blocks, G / maps, 16, EP].
+// maps > 1: that many key heads share a value head and lie side by side in one cache row; query head h belongs to
+// the map h % maps and goes to the columns of that map, so its product with the whole row is the one with its own key.
 struct HeadsParams {
   const void* proj;         // [M, ld], of the storage type, or fp32 when proj_f32 is set (split-K accumulator)
   int proj_f32;
   long long ld;
-  int M, H, G, D, E;
+  int M, H, G, D, E;        // G 0: queries only
+  int maps;
+  long long q_pd;           // columns between query heads of the projection (D where they are packed); k starts at H * q_pd
+  const float* bias;        // [columns of q | k | v] or nullptr
+  float t_coef, t_every;    // t_coef 0: no temperature
   const float* q_norm;      // [H * D] or nullptr
   const float* k_norm;      // [G * D]
   float eps;
@@ -146,7 +154,8 @@ struct RowAttnParams {
   int chunk;                // > 0: only positions of the query's own chunk (counted from position 0) are visible
   float scale;
   float sink;               // score of one more term of the softmax denominator, without a value (-inf: none)
-  void* out;                // [rows, ldo], head stride E
+  void* out;                // [rows, ldo], heads o_hd apart; fp32 when out_f32 is set
+  int out_f32, o_hd;
   long long ldo;
   int* status;
 };
@@ -261,8 +270,128 @@ struct GatedNormParams {
 };
 cudaError_t launch_gated_norm(const GatedNormParams& p, int dtype, cudaStream_t stream);
 
-// Router of a mixture of experts: softmax over all experts, the `top` largest scores divided by their sum (+ 1e-20).
+// Differential attention: o = a1 - lambda a2 of the two maps of every head, o / sqrt(mean(o^2) + eps) * gain.
+struct DiffNormParams {
+  const float* a;           // [M, lda]: heads of [map 1: E | map 2: E]
+  long long lda;
+  int M, H, E;
+  float lambda, gain, eps;
+  void* out;                // [M, ldo], heads of E
+  long long ldo;
+};
+cudaError_t launch_diff_norm(const DiffNormParams& p, int dtype, cudaStream_t stream);
+
+// Latent attention. What a token keeps is one row of R latent values (normed) and T rotated key values that all
+// heads share: cache [blocks, 16, CP]. Projection rows hold the query latent (Q values, kv_col columns wide) and, from
+// column kv_col on, the R + T raw values.
+struct LatentRowsParams {
+  const void* proj;         // [M, ld], storage type or fp32 when proj_f32 is set
+  int proj_f32;
+  long long ld;
+  int M, Q, R, kv_col;      // R 0: the layer reads another one's cache
+  const float* q_norm;      // [Q]
+  const float* kv_norm;     // [R]
+  float eps;
+  RotaryParams rot;         // of the last rot.dims values
+  const int* positions;
+  void* q_out;              // [M, ldq] normed query latent
+  long long ldq;
+  void* cache;
+  int CP;
+  const long long* slots;   // [M], < 0: not stored
+  long long num_slots;
+  int* status;
+};
+cudaError_t launch_latent_rows(const LatentRowsParams& p, int dtype, cudaStream_t stream);
+// Cache rows of a step's prompts -> consecutive rows: position t of sequence s at row row0[s] + t.
+struct LatentGatherParams {
+  const void* cache;        // [blocks, 16, CP], bf16
+  int CP, num_blocks, max_blocks;
+  const int* block_tables;  // [sequences, max_blocks]
+  const int* ctx_lens;
+  const int* row0;
+  int seq0, n_seqs, max_pages;
+  void* out;                // [rows, CP]
+  long long rows;
+  int* status;
+};
+cudaError_t launch_latent_gather(const LatentGatherParams& p, cudaStream_t stream);
+// Decoding: all heads of a row against the latents themselves. q rows [H, CP]: the query's product with the key
+// expansion (R values), then its rotated part; the output is the weighted sum of latents, per head R values.
+struct LatentDecodeParams {
+  const __nv_bfloat16* q;   // [rows, H, CP]
+  const __nv_bfloat16* cache;
+  const int* block_tables;  // [rows, max_blocks]
+  const int* seq_lens;
+  const int* pages_per_split;
+  int rows, H, R, CP, max_blocks, max_splits, num_blocks;
+  float scale_log2;
+  float* part_o;            // [rows, H, max_splits, R]
+  float* part_ml;           // [rows, H, max_splits, 2]
+  __nv_bfloat16* out;       // [rows, ldo], heads o_hd apart
+  long long ldo;
+  int o_hd;
+  int* status;
+};
+cudaError_t launch_latent_decode(const LatentDecodeParams& p, cudaStream_t stream);
+bool latent_decode_ok(int R, int CP);
+
+// Matrix memory with a running maximum (mLSTM). Log gates per head: i = cap tanh(zi / cap), f = logsigmoid(cap tanh(zf / cap));
+//   m' = max(f + m, i), S' = exp(f + m - m') S + exp(i - m') k v^T, n' likewise with k alone, m starts at 0
+//   o = scale S'^T q / (max(|scale n' q|, exp(-m')) + 1e-6), then o / rms(o) * norm_w * sigmoid(gate)
+// state [slots, H, D * E + D]: S row by row, then n; state_m [slots, H].
+constexpr int kMemChunk = 64;
+struct MemoryParams {
+  const void* proj;         // [M, ld]: q (H * D) | k (H * D) | v (H * E) | gate (H * E); type as in HeadsParams
+  int proj_f32;
+  long long ld;
+  int H, D, E;
+  const float* z;           // [M, ldz] pre-activations zi (H) | zf (H) without bias (prompt chunks, fp32 path)
+  long long ldz;
+  const float* z_bias;      // [2 H]
+  const void* h;            // decode: normed rows and gate weights instead of z
+  long long ldh;
+  const void* z_w;          // [2 H, ldw] bf16
+  long long ldw;
+  int N;
+  float cap, scale, eps;
+  const float* norm_w;      // [H * E]
+  float* state;
+  float* state_m;
+  int num_slots;
+  // decode rows
+  const int* row_slots;     // [rows], < 0: padding row
+  const int* positions;     // [rows]; a row at position 0 starts from the zero state
+  int rows;
+  // prompt chunks
+  const int* seq_slots;
+  const int* tile_seq;
+  const int* tile_q0;
+  const int* q_start;
+  const int* q_lens;
+  const int* ctx_lens;
+  int n_tiles, n_seqs;
+  float* ws;                // [2 n_tiles, H, D * E + D]: what each chunk adds, then the state before it
+  float* ws_m;              // [2 n_tiles, H]: maximum before each chunk
+  float* o_buf;             // [M, H * E] fp32 (token-by-token form only)
+  float* n_buf;             // [n_seqs, H, D + 1] (token-by-token form only)
+  void* out;                // [M, ldo]
+  long long ldo;
+  int* status;
+};
+cudaError_t launch_memory_decode(const MemoryParams& p, int dtype, cudaStream_t stream);
+// Prompt chunks, bf16: chunk sums, scan over the chunks, outputs (fp32 operands in three bf16 terms).
+cudaError_t launch_memory_chunks(const MemoryParams& p, cudaStream_t stream);
+// Prompt chunks token by token in fp32 FMAs.
+cudaError_t launch_memory_scan(const MemoryParams& p, int dtype, cudaStream_t stream);
+bool memory_chunks_ok(int D, int E);
+
+// Router of a mixture of experts. softmax 1: scores are a softmax over all experts, the weights the `top` largest ones
+// divided by their sum (+ 1e-20). softmax 0: scores are sigmoids, the weights the chosen scores themselves. With
+// `groups` > 0 the experts form that many equal groups of neighbours; only experts of the `keep` groups whose two
+// largest scores have the largest sum can be chosen.
 constexpr int kMaxExperts = 512;
+constexpr int kMaxGroups = 32;
 struct MoeRouteParams {
   const float* logits;      // [M, ldl], or nullptr: computed here from h and router
   long long ldl;
@@ -271,6 +400,7 @@ struct MoeRouteParams {
   const void* router;       // [E, ldr]
   long long ldr;
   int M, N, E, top;
+  int softmax, groups, keep;
   float* weight;            // [M, top]
   int* expert;              // [M, top]
   int* slot;                // [M, top]: row of the expert buffers that belongs to the choice
@@ -295,7 +425,8 @@ struct MoeScatterParams {
   int* status;
 };
 cudaError_t launch_moe_scatter(const MoeScatterParams& p, cudaStream_t stream);   // bf16
-// y[p] = act(W[expert[p]] x[per_pair ? p : p / top]) for every (row, choice) pair p. act 0: none, 2: squared ReLU.
+// y[p] = act(W[expert[p]] x[per_pair ? p : p / top]) for every (row, choice) pair p. act 0: none, 2: squared ReLU,
+// 3: W holds gate and up rows in units of 32 | 32, y = silu(gate) * up with N / 2 values.
 struct MoeRowsParams {
   const void* x;
   long long ldx;

@@ -1,6 +1,7 @@
-// Projections -> heads (sm_100a): RMS norm over the whole q / k projection, rotation in either pair layout
+// Projections -> heads (sm_100a): bias, RMS norm over the whole q / k projection, rotation in either pair layout
 // on the first dimensions of every head, write of k and v into the paged cache (or of q and k to dense
-// fp32 buffers for a recurrence); plus plain fp32 pieces of the 32-bit path (GEMM, gated unit).
+// fp32 buffers for a recurrence); the difference of the two maps of differential attention with its norm; plus plain
+// fp32 pieces of the 32-bit path (GEMM, gated unit).
 #include "../common/device_info.h"
 #include "hybrid_dev.cuh"
 
@@ -42,7 +43,8 @@ __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
   pdl_wait();  // the projection comes from the kernel before this one
   const int row = blockIdx.x;
   const int H = p.H, G = p.G, D = p.D, E = p.E;
-  const int n_heads = H + G + (p.v_cache != nullptr ? G : 0);
+  const int GV = G / p.maps;   // value heads = rows of a cache block
+  const int n_heads = H + G + (p.v_cache != nullptr ? GV : 0);
   const int hpc = (n_heads + gridDim.y - 1) / gridDim.y;
   const int h_lo = blockIdx.y * hpc;
   const int h_hi = min(h_lo + hpc, n_heads);
@@ -59,6 +61,8 @@ __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
     if (h_lo < H) rq = 1.f / sqrtf(block_sum_all(sq, s_red) / static_cast<float>(H * D) + p.eps);
     if (need_k) rk = 1.f / sqrtf(block_sum_all(sk, s_red) / static_cast<float>(G * D) + p.eps);
   }
+  const float qt = p.t_coef != 0.f ? 1.f + p.t_coef * logf(floorf(static_cast<float>(pos + 1) / p.t_every) + 1.f) : 1.f;
+  const long long k_col = p.q_pd * H;   // k follows q in the projection row
   __syncthreads();
   const long long slot = p.slots != nullptr ? p.slots[row] : -1;
   const bool store_kv = slot >= 0 && slot < p.num_slots;
@@ -76,12 +80,19 @@ __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
       const int lh = i / per, it = i - lh * per, h = h_lo + lh;
       const bool is_q = h < H;
       if (!is_q && p.k_out == nullptr && !store_kv) continue;
-      const P* src = pr + h * D;
-      const float r = is_q ? rq : rk, ks = is_q ? 1.f : p.k_scale;
+      const long long col = is_q ? h * p.q_pd : k_col + (h - H) * D;
+      const P* src = pr + col;
+      const float r = is_q ? rq : rk, ks = is_q ? qt : p.k_scale;
       const float* w = is_q ? p.q_norm : p.k_norm;
       if (w != nullptr) w += (is_q ? h : h - H) * D;
       auto get = [&](int d, float (&v)[4]) {
         load4<P>(src + d, v);
+        if (p.bias != nullptr) {
+          float b4[4];
+          load4<float>(p.bias + col + d, b4);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) v[j] += b4[j];
+        }
         if (w != nullptr) {
           float g4[4];
           load4<float>(w + d, g4);
@@ -90,14 +101,15 @@ __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
         }
       };
       auto put = [&](int d, float (&v)[4]) {
-        if (is_q) {
-          store4<TQ>(static_cast<TQ*>(p.q_out) + static_cast<long long>(row) * p.q_ld + h * p.q_hd + d, v);
-          return;
-        }
 #pragma unroll
         for (int j = 0; j < 4; ++j) v[j] *= ks;
-        if (p.k_out != nullptr) store4<float>(p.k_out + static_cast<long long>(row) * p.k_ld + (h - H) * p.k_hd + d, v);
-        else store4<T>(static_cast<T*>(p.k_cache) + ((blk * G + (h - H)) * 16 + off) * p.DP + d, v);
+        if (is_q) {
+          store4<TQ>(static_cast<TQ*>(p.q_out) + static_cast<long long>(row) * p.q_ld + h * p.q_hd + (h % p.maps) * D + d, v);
+          return;
+        }
+        const int g = h - H;
+        if (p.k_out != nullptr) store4<float>(p.k_out + static_cast<long long>(row) * p.k_ld + g * p.k_hd + d, v);
+        else store4<T>(static_cast<T*>(p.k_cache) + ((blk * GV + g / p.maps) * 16 + off) * p.DP + (g % p.maps) * D + d, v);
       };
       float x[4];
       if (it >= rq4) {
@@ -126,12 +138,18 @@ __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
     }
     if (store_kv && h_hi > H + G) {
       const int v_lo = max(h_lo, H + G), e4 = E >> 2;
-      const P* vr = pr + (H + G) * D;
+      const long long v_col = k_col + G * D;
       for (int i = threadIdx.x; i < (h_hi - v_lo) * e4; i += blockDim.x) {
         const int lh = i / e4, e = (i - lh * e4) * 4, g = v_lo + lh - H - G;
         float x[4];
-        load4<P>(vr + g * E + e, x);
-        store4<T>(static_cast<T*>(p.v_cache) + ((blk * G + g) * 16 + off) * p.EP + e, x);
+        load4<P>(pr + v_col + g * E + e, x);
+        if (p.bias != nullptr) {
+          float b4[4];
+          load4<float>(p.bias + v_col + g * E + e, b4);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) x[j] += b4[j];
+        }
+        store4<T>(static_cast<T*>(p.v_cache) + ((blk * GV + g) * 16 + off) * p.EP + e, x);
       }
     }
     return;
@@ -142,26 +160,34 @@ __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
   for (int h = h_lo + warp; h < r_hi; h += nw) {
     const bool is_q = h < H;
     if (!is_q && p.k_out == nullptr && !store_kv) continue;
-    const P* src = pr + h * D;  // k follows q in the projection row
+    const long long col = is_q ? h * p.q_pd : k_col + (h - H) * D;
+    const P* src = pr + col;
+    const float* bias = p.bias != nullptr ? p.bias + col : nullptr;
     const float r = is_q ? rq : rk;
     const float* w = is_q ? p.q_norm : p.k_norm;
     if (w != nullptr) w += (is_q ? h : h - H) * D;
-    const float ks = is_q ? 1.f : p.k_scale;
+    const float ks = is_q ? qt : p.k_scale;
     TQ* qd = nullptr;
     float* kd = nullptr;
     T* kc = nullptr;
-    if (is_q) qd = static_cast<TQ*>(p.q_out) + static_cast<long long>(row) * p.q_ld + h * p.q_hd;
+    if (is_q) qd = static_cast<TQ*>(p.q_out) + static_cast<long long>(row) * p.q_ld + h * p.q_hd + (h % p.maps) * D;
     else if (p.k_out != nullptr) kd = p.k_out + static_cast<long long>(row) * p.k_ld + (h - H) * p.k_hd;
-    else kc = static_cast<T*>(p.k_cache) + ((blk * G + (h - H)) * 16 + off) * p.DP;
+    else kc = static_cast<T*>(p.k_cache) + ((blk * GV + (h - H) / p.maps) * 16 + off) * p.DP + ((h - H) % p.maps) * D;
     auto put = [&](int d, float y) {
-      if (qd != nullptr) qd[d] = from_f<TQ>(y);
+      if (qd != nullptr) qd[d] = from_f<TQ>(y * ks);
       else if (kd != nullptr) kd[d] = y * ks;
       else kc[d] = from_f<T>(y * ks);
     };
     for (int it = lane; it < rot2; it += 32) {
       int d0, d1;
       rotary_pair(p.rot, it, &d0, &d1);
-      float u = to_f(src[d0]) * r, v = to_f(src[d1]) * r;
+      float u = to_f(src[d0]), v = to_f(src[d1]);
+      if (bias != nullptr) {
+        u += bias[d0];
+        v += bias[d1];
+      }
+      u *= r;
+      v *= r;
       if (w != nullptr) {
         u *= w[d0];
         v *= w[d1];
@@ -169,16 +195,63 @@ __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
       put(d0, u * s_cos[it] - v * s_sin[it]);
       put(d1, v * s_cos[it] + u * s_sin[it]);
     }
-    for (int d = 2 * rot2 + lane; d < D; d += 32) put(d, to_f(src[d]) * r * (w != nullptr ? w[d] : 1.f));
+    for (int d = 2 * rot2 + lane; d < D; d += 32) put(d, (to_f(src[d]) + (bias != nullptr ? bias[d] : 0.f)) * r * (w != nullptr ? w[d] : 1.f));
   }
   if (store_kv && h_hi > H + G) {
-    const P* vr = pr + (H + G) * D;
     for (int h = max(h_lo, H + G) + warp; h < h_hi; h += nw) {
       const int g = h - H - G;
-      T* vc = static_cast<T*>(p.v_cache) + ((blk * G + g) * 16 + off) * p.EP;
-      for (int e = lane; e < E; e += 32) vc[e] = from_f<T>(to_f(vr[g * E + e]));
+      const long long col = k_col + G * D + g * E;
+      T* vc = static_cast<T*>(p.v_cache) + ((blk * GV + g) * 16 + off) * p.EP;
+      for (int e = lane; e < E; e += 32) vc[e] = from_f<T>(to_f(pr[col + e]) + (p.bias != nullptr ? p.bias[col + e] : 0.f));
     }
   }
+}
+
+// One warp per (row, head).
+template <typename T>
+__global__ void __launch_bounds__(256) diff_norm_kernel(const DiffNormParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const long long item = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  if (item >= static_cast<long long>(p.M) * p.H) return;
+  const long long row = item / p.H;
+  const int head = static_cast<int>(item - row * p.H), E = p.E;
+  const float* a = p.a + row * p.lda + 2ll * head * E;
+  T* out = static_cast<T*>(p.out) + row * p.ldo + static_cast<long long>(head) * E;
+  float ss = 0.f;
+  if (E % 4 == 0 && p.lda % 4 == 0 && p.ldo % 4 == 0 && E <= 1024) {
+    float o[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int e = (i * 32 + lane) * 4;
+      if (e >= E) break;
+      float x[4], y[4];
+      load4_stream(a + e, x);
+      load4_stream(a + E + e, y);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        o[i][j] = fmaf(-p.lambda, y[j], x[j]);
+        ss = fmaf(o[i][j], o[i][j], ss);
+      }
+    }
+    const float r = p.gain / sqrtf(warp_sum(ss) / static_cast<float>(E) + p.eps);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int e = (i * 32 + lane) * 4;
+      if (e >= E) break;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) o[i][j] *= r;
+      store4<T>(out + e, o[i]);
+    }
+    return;
+  }
+  for (int e = lane; e < E; e += 32) {
+    const float o = fmaf(-p.lambda, a[E + e], a[e]);
+    ss = fmaf(o, o, ss);
+  }
+  const float r = p.gain / sqrtf(warp_sum(ss) / static_cast<float>(E) + p.eps);
+  for (int e = lane; e < E; e += 32) out[e] = from_f<T>(fmaf(-p.lambda, a[E + e], a[e]) * r);
 }
 
 constexpr int kFT = 64, kFK = 16;
@@ -270,7 +343,7 @@ static cudaError_t launch_heads_v(const HeadsParams& p, int dtype, dim3 grid, di
 
 cudaError_t launch_heads(const HeadsParams& p, int dtype, cudaStream_t stream) {
   if (p.M <= 0) return cudaSuccess;
-  const int n_heads = p.H + p.G + (p.v_cache != nullptr ? p.G : 0);
+  const int n_heads = p.H + p.G + (p.v_cache != nullptr ? p.G / p.maps : 0);
   // ranges of at least 4 heads until about two CTAs per SM exist
   int chunks = (2 * sm_count() + p.M - 1) / p.M;
   chunks = chunks > n_heads / 4 ? n_heads / 4 : chunks;
@@ -279,9 +352,17 @@ cudaError_t launch_heads(const HeadsParams& p, int dtype, cudaStream_t stream) {
   const dim3 grid(p.M, chunks), block(256);
   auto al = [](const void* x) { return reinterpret_cast<uintptr_t>(x) % 16 == 0; };
   const bool vec = p.D % 4 == 0 && p.E % 4 == 0 && p.rot.dims % (p.rot.interleaved ? 4 : 8) == 0 && p.ld % 4 == 0 && p.q_ld % 4 == 0 &&
-                   p.q_hd % 4 == 0 && p.k_ld % 4 == 0 && p.k_hd % 4 == 0 && p.DP % 4 == 0 && p.EP % 4 == 0 && al(p.proj) &&
+                   p.q_hd % 4 == 0 && p.q_pd % 4 == 0 && al(p.bias) && p.k_ld % 4 == 0 && p.k_hd % 4 == 0 && p.DP % 4 == 0 && p.EP % 4 == 0 && al(p.proj) &&
                    al(p.q_out) && al(p.k_out) && al(p.q_norm) && al(p.k_norm);
   return vec ? launch_heads_v<true>(p, dtype, grid, block, smem, stream) : launch_heads_v<false>(p, dtype, grid, block, smem, stream);
+}
+
+cudaError_t launch_diff_norm(const DiffNormParams& p, int dtype, cudaStream_t stream) {
+  const long long items = static_cast<long long>(p.M) * p.H;
+  if (items <= 0) return cudaSuccess;
+  const dim3 grid(static_cast<unsigned>((items + 7) / 8));
+  return dtype == 0 ? launch_kernel(diff_norm_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, true, false, p)
+                    : launch_kernel(diff_norm_kernel<float>, grid, dim3(256), 0, stream, true, false, p);
 }
 
 cudaError_t launch_gemm_f32(const float* a, long long lda, const float* w, long long ldw, float* out, long long ldo,

@@ -1,5 +1,5 @@
-// Mixture of experts around the grouped GEMM (sm_100a): router (softmax over all experts, largest scores, weights
-// divided by their sum), placement of the chosen rows, and expert products of a handful of rows.
+// Mixture of experts around the grouped GEMM (sm_100a): router (softmax over all experts with weights divided by their
+// sum, or sigmoid scores; best groups of experts first where experts form groups), placement of the chosen rows, and expert products of a handful of rows.
 //
 // Three ways from the normed rows to expert rows:
 //   a step of a few rows (and the 32-bit path): every (row, choice) pair is a row of its own, `moe_rows` streams the
@@ -17,9 +17,59 @@ namespace {
 
 constexpr int kSlab = 128;   // rows of a slab = rows of a GEMM tile
 
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+
+// Takes the experts of all but the best groups out of the choice (logit -inf).
+template <int R>
+__device__ __forceinline__ void keep_groups(float (&l)[R], int E, int groups, int keep, int lane) {
+  const int size = E / groups;
+  float mine = -INFINITY;   // lane g: score of group g
+  for (int g = 0; g < groups; ++g) {
+    float a = -INFINITY, b = -INFINITY;   // largest and second largest logit of the group
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      const int e = lane + 32 * i;
+      if (e >= g * size && e < (g + 1) * size) {
+        b = fmaxf(b, fminf(a, l[i]));
+        a = fmaxf(a, l[i]);
+      }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float oa = __shfl_xor_sync(0xffffffffu, a, o), ob = __shfl_xor_sync(0xffffffffu, b, o);
+      b = fmaxf(fmaxf(b, ob), fminf(a, oa));
+      a = fmaxf(a, oa);
+    }
+    if (lane == g) mine = sigmoid_f(a) + (size > 1 ? sigmoid_f(b) : 0.f);
+  }
+  unsigned kept = 0;
+  for (int c = 0; c < keep; ++c) {
+    float best = mine;
+    int at = lane;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+      if (ob > best || (ob == best && oa < at)) {
+        best = ob;
+        at = oa;
+      }
+    }
+    kept |= 1u << at;
+    if (lane == at) mine = -INFINITY;
+  }
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int e = lane + 32 * i;
+    if (e < E && ((kept >> (e / size)) & 1u) == 0) l[i] = -INFINITY;
+  }
+}
+
 // Chosen experts of one row: logits of expert e in l[e / 32] of lane e % 32. Lane c < top gets choice c and its weight.
 template <int R>
-__device__ __forceinline__ void choose(float (&l)[R], int E, int top, int lane, int* expert, float* weight) {
+__device__ __forceinline__ void choose(float (&l)[R], const MoeRouteParams& p, int lane, int* expert, float* weight) {
+  const int E = p.E, top = p.top;
+  if (p.groups > 0) keep_groups<R>(l, E, p.groups, p.keep, lane);
   float m = -INFINITY;
 #pragma unroll
   for (int i = 0; i < R; ++i) m = fmaxf(m, l[i]);
@@ -55,8 +105,13 @@ __device__ __forceinline__ void choose(float (&l)[R], int E, int top, int lane, 
       if (lane + 32 * i == at) l[i] = -INFINITY;
     if (lane == c) {
       my_e = at;
-      my_s = expf(best - m) / z;
+      my_s = p.softmax ? expf(best - m) / z : sigmoid_f(best);
     }
+  }
+  if (!p.softmax) {
+    *expert = my_e;
+    *weight = my_s;
+    return;
   }
   const float sum = warp_sum(my_s);
   *expert = my_e;
@@ -157,7 +212,7 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_row_kernel(const MoeR
     for (int i = 0; i < R; ++i) l[i] = lane + 32 * i < p.E ? s_l[lane + 32 * i] : -INFINITY;
     int e;
     float w;
-    choose<R>(l, p.E, p.top, lane, &e, &w);
+    choose<R>(l, p, lane, &e, &w);
     if (lane < p.top) {
       const int i = row * p.top + lane;
       int slot = i;
@@ -205,7 +260,7 @@ __global__ void __launch_bounds__(256) moe_route_rank_kernel(const MoeRouteParam
     for (int k = 0; k < R; ++k) l[k] = lane + 32 * k < p.E ? p.logits[static_cast<long long>(row) * p.ldl + lane + 32 * k] : -INFINITY;
     float w;
     int ex;
-    choose<R>(l, p.E, p.top, lane, &ex, &w);
+    choose<R>(l, p, lane, &ex, &w);
     if (lane < p.top) {
       e[i] = ex;
       rank[i] = atomicAdd(&s_cnt[ex], 1u);
@@ -276,17 +331,19 @@ __global__ void __launch_bounds__(256) moe_scatter_kernel(const MoeScatterParams
   }
 }
 
-// grid (pairs, N / 16): 8 warps of two output values each.
+// grid (pairs, N / 16): 8 warps of two rows of W each, which are two outputs or the gate and up row of one.
 template <typename T>
 __global__ void __launch_bounds__(256) moe_rows_kernel(const MoeRowsParams p) {
   pdl_wait();
   const int pair = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int n0 = (blockIdx.y * 8 + warp) * 2;
-  if (n0 >= p.N) return;
+  const int n2 = (blockIdx.y * 8 + warp) * 2;
+  if (n2 >= p.N) return;
+  const bool glu = p.act == 3;
+  const int n0 = glu ? (n2 >> 6) * 64 + ((n2 >> 1) & 31) : n2;
   const int e = p.expert[pair];
   if (static_cast<unsigned>(e) >= static_cast<unsigned>(p.E)) return;
   const T* x = static_cast<const T*>(p.x) + static_cast<long long>(p.per_pair ? pair : pair / p.top) * p.ldx;
-  const int n1 = n0 + 1 < p.N ? n0 + 1 : n0;
+  const int n1 = glu ? n0 + 32 : (n0 + 1 < p.N ? n0 + 1 : n0);
   const T* w0 = static_cast<const T*>(p.w) + (static_cast<long long>(e) * p.N + n0) * p.K;
   const T* w1 = static_cast<const T*>(p.w) + (static_cast<long long>(e) * p.N + n1) * p.K;
   constexpr int W = Pack<T>::n;
@@ -311,7 +368,11 @@ __global__ void __launch_bounds__(256) moe_rows_kernel(const MoeRowsParams p) {
     a1 = fmaxf(a1, 0.f) * fmaxf(a1, 0.f);
   }
   if (lane == 0) {
-    T* y = static_cast<T*>(p.y) + static_cast<long long>(pair) * p.ldy + n0;
+    T* y = static_cast<T*>(p.y) + static_cast<long long>(pair) * p.ldy + (glu ? n2 >> 1 : n0);
+    if (glu) {
+      y[0] = from_f<T>(silu_f(a0) * a1);
+      return;
+    }
     y[0] = from_f<T>(a0);
     if (n1 != n0) y[1] = from_f<T>(a1);
   }
@@ -339,6 +400,7 @@ cudaError_t route_of(const MoeRouteParams& p, cudaStream_t stream) {
 cudaError_t launch_moe_route(const MoeRouteParams& p, int dtype, cudaStream_t stream) {
   if (p.M <= 0) return cudaSuccess;
   if (p.E > kMaxExperts || p.top > kMaxTop || p.top > p.E) return cudaErrorInvalidValue;
+  if (p.groups > kMaxGroups || (p.groups > 0 && (p.E % p.groups != 0 || p.keep < 1 || p.keep > p.groups))) return cudaErrorInvalidValue;
   return dtype == 0 ? route_of<__nv_bfloat16>(p, stream) : route_of<float>(p, stream);
 }
 

@@ -215,6 +215,9 @@ __device__ __forceinline__ float expert_sum(const BranchNormParams& p, const Cho
     a = fmaf(s_e[k].weight, to_f(static_cast<const T*>(p.e_rows)[static_cast<long long>(s_e[k].row) * p.lde + c]), a);
   return a;
 }
+__device__ __forceinline__ bool experts_are_branch(const BranchNormParams& p) {
+  return (p.n_branches > 0 && p.y[0] == nullptr) || (p.n_branches > 1 && p.y[1] == nullptr);
+}
 // sums of both branches at once over the block
 __device__ __forceinline__ float2 block_sum2(float2 v, float2* scratch) {
   v.x = warp_sum(v.x);
@@ -237,6 +240,7 @@ __global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchNormParam
   pdl_wait();
   const int N = p.N;
   const float inv_n = 1.f / static_cast<float>(N);
+  const bool e_plain = p.e_rows != nullptr && !experts_are_branch(p);
   if (p.e_rows != nullptr) {
     chosen_rows(p, blockIdx.x, s_chosen[0]);
     __syncthreads();
@@ -281,14 +285,15 @@ __global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchNormParam
         for (int j = 0; j < 4; ++j) x[k][j] = 0.f;
         if (c < N) {
           load4_stream(xr + c, x[k]);
-          if (p.e_rows != nullptr) expert_sum4<T>(p, s_chosen[parity], c, x[k]);
+          if (e_plain) expert_sum4<T>(p, s_chosen[parity], c, x[k]);
         }
 #pragma unroll
         for (int b = 0; b < kMaxBranches; ++b) {
 #pragma unroll
           for (int j = 0; j < 4; ++j) y[b][k][j] = 0.f;
           if (b < p.n_branches && c < N) {
-            load4_stream(p.y[b] + static_cast<long long>(row) * p.ldy + c, y[b][k]);
+            if (p.y[b] != nullptr) load4_stream(p.y[b] + static_cast<long long>(row) * p.ldy + c, y[b][k]);
+            else expert_sum4<T>(p, s_chosen[parity], c, y[b][k]);
 #pragma unroll
             for (int j = 0; j < 4; ++j) ss[b] = fmaf(y[b][k][j], y[b][k][j], ss[b]);
           }
@@ -367,6 +372,11 @@ __global__ void __launch_bounds__(256) branch_norm_any_kernel(const BranchNormPa
     if (p.clear != nullptr)
       for (int c = threadIdx.x; c < p.clear_n; c += blockDim.x) p.clear[static_cast<long long>(row) * p.clear_ld + c] = 0.f;
     const int dst = p.row_map != nullptr ? p.row_map[row] : row;
+    if (p.e_rows != nullptr) __syncthreads();
+    const bool e_plain = p.e_rows != nullptr && !experts_are_branch(p);
+    auto branch = [&](int b, int c) {
+      return p.y[b] != nullptr ? p.y[b][static_cast<long long>(row) * p.ldy + c] : expert_sum<T>(p, s_e, c);
+    };
     const T* er = nullptr;
     float r[kMaxBranches] = {};
     if (p.tokens != nullptr) {
@@ -380,7 +390,7 @@ __global__ void __launch_bounds__(256) branch_norm_any_kernel(const BranchNormPa
 #pragma unroll
         for (int b = 0; b < kMaxBranches; ++b)
           if (b < p.n_branches) {
-            const float y = p.y[b][static_cast<long long>(row) * p.ldy + c];
+            const float y = branch(b, c);
             ss[b] = fmaf(y, y, ss[b]);
           }
       const float2 tot = block_sum2(make_float2(ss[0], ss[1]), s_red2);
@@ -393,11 +403,11 @@ __global__ void __launch_bounds__(256) branch_norm_any_kernel(const BranchNormPa
       if (er != nullptr) {
         x = to_f(er[c]) * p.embed_scale;
       } else {
-        x = p.e_rows != nullptr ? expert_sum<T>(p, s_e, c) : 0.f;
+        x = e_plain ? expert_sum<T>(p, s_e, c) : 0.f;
 #pragma unroll
         for (int b = 0; b < kMaxBranches; ++b)
           if (b < p.n_branches) {
-            const float y = p.y[b][static_cast<long long>(row) * p.ldy + c];
+            const float y = branch(b, c);
             x = fmaf(p.gain[b] * (p.w[b] != nullptr ? r[b] * p.w[b][c] : 1.f), y, x);
           }
         x += xr[c];

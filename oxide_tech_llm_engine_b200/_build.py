@@ -45,8 +45,10 @@ CUDA_FLAGS = [
 
 
 # kernels of the extension that only layer-list decoders load
-HYBRID_KERNELS = ("stream_ops.cu", "mixer_ops.cu", "attn_rows.cu", "retention.cu", "ssd.cu", "moe_ops.cu")
-HYBRID_HEADERS = ("hybrid.cuh", "hybrid_dev.cuh")
+HYBRID_KERNELS = ("stream_ops.cu", "mixer_ops.cu", "attn_rows.cu", "retention.cu", "ssd.cu", "moe_ops.cu", "latent.cu", "memory.cu",
+                  "attn_prefill_wide.cu")
+HYBRID_HEADERS = ("hybrid.cuh", "hybrid_dev.cuh", "hybrid_mma.cuh")
+SHARED_HEADERS = ("attn.cuh", "attn_prefill_tc.cuh")   # of both kernel extensions
 # kernels of the extension that only quantised weights load
 QUANT_KERNELS = ("quant_ops.cu", "gemm_fp8_block.cu", "nvfp4_quant.cu")
 
@@ -71,7 +73,7 @@ def _headers(name: str) -> list[Path]:
         return sorted((_CSRC / "host").glob("*.h"))
     common = list((_CSRC / "common").glob("*"))
     if name == "oxb_hybrid":
-        return sorted(common + [_CSRC / "kernels" / h for h in HYBRID_HEADERS])
+        return sorted(common + [_CSRC / "kernels" / h for h in HYBRID_HEADERS + SHARED_HEADERS])
     return sorted(common + [p for p in (_CSRC / "kernels").glob("*.cuh") if p.name not in HYBRID_HEADERS])
 
 

@@ -193,7 +193,7 @@ class LLMEngine:
         self.st = _Staging({
             "token_ids": (M, i32), "positions": (M, i32), "logit_map": (M, i32), "slot_mapping": (M, i64),
             "prev_ids": (M, i32), "decode_slots": (S, i32), "pages_per_split": (4, i32), "seq_lens": (S, i32), "block_tables": (S * max_blocks_per_seq, i32),
-            "q_start": (S, i32), "q_lens": (S, i32), "ctx_lens": (S, i32), "prefill_slots": (S, i32),
+            "q_start": (S, i32), "q_lens": (S, i32), "ctx_lens": (S, i32), "prefill_slots": (S, i32), "kv_start": (S, i32),
             "tile_seq": (n_tiles_max, i32),
             "tile_q0": (n_tiles_max, i32), "prefill_block_tables": (S * max_blocks_per_seq, i32),
             "cow_src": (S, i32), "cow_dst": (S, i32),
@@ -442,7 +442,7 @@ class LLMEngine:
             pps = max(4, -(-pages // splits))
             pps = (pps + 3) // 4 * 4
             h("pages_per_split")[0] = pps
-        n_tiles = 0
+        n_tiles, passes = 0, ()
         if npf > 0:
             h("q_start")[:npf] = plan.q_start
             h("q_lens")[:npf] = plan.q_lens
@@ -453,6 +453,8 @@ class LLMEngine:
             h("tile_q0")[:n_tiles] = plan.tile_q0
             pbt = h("prefill_block_tables").reshape(-1, W)
             pbt[:npf, :w] = plan.prefill_block_tables.reshape(npf, w)
+            if getattr(self.model, "latents", None):
+                passes = self._kv_passes(plan, h("kv_start"))
         n_cow = plan.cow_src.size
         if n_cow:
             h("cow_src")[:n_cow] = plan.cow_src
@@ -467,10 +469,31 @@ class LLMEngine:
                        pages_per_split=d("pages_per_split"), tile_seq=d("tile_seq"), tile_q0=d("tile_q0"),
                        q_start=d("q_start"), q_lens=d("q_lens"), ctx_lens=d("ctx_lens"),
                        prefill_block_tables=d("prefill_block_tables").view(-1, W), logit_map=d("logit_map"),
-                       prev_ids=d("prev_ids"), decode_slots=d("decode_slots"), prefill_slots=d("prefill_slots"))
+                       prev_ids=d("prev_ids"), decode_slots=d("decode_slots"), prefill_slots=d("prefill_slots"),
+                       kv_start=d("kv_start"), kv_passes=passes)
         if n_cow:
             self.model.copy_blocks(d("cow_src")[:n_cow], d("cow_dst")[:n_cow])
         return s, bucket
+
+    @staticmethod
+    def _kv_passes(plan, kv_start: np.ndarray) -> tuple:
+        """First rows of the prompts' contexts when they lie one after the other, in passes of a bounded number of rows
+        (StepInputs.kv_passes)."""
+        from ..models.hybrid import KV_PASS_ROWS
+
+        pages = (np.asarray(plan.ctx_lens, dtype=np.int64) + 15) // 16
+        tiles = (np.asarray(plan.q_lens, dtype=np.int64) + 127) // 128
+        out, s0, t0, rows = [], 0, 0, 0
+        for i in range(plan.n_prefill + 1):
+            last = i == plan.n_prefill
+            if i > s0 and (last or rows + 16 * pages[i] > KV_PASS_ROWS):
+                t1 = t0 + int(tiles[s0:i].sum())
+                out.append((s0, i, t0, t1, rows, int(pages[s0:i].max())))
+                s0, t0, rows = i, t1, 0
+            if not last:
+                kv_start[i] = rows
+                rows += 16 * int(pages[i])
+        return tuple(out)
 
     def _forward(self, s: StepInputs, bucket: Optional[int]) -> torch.Tensor:
         baseline = self.cfg.comm == "nccl" or self.cfg.gemm == "library"

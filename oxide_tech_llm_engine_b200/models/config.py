@@ -94,7 +94,7 @@ class ModelConfig:
 
     def active_params(self) -> int:
         if self.layers:
-            idle = sum(2 * (L.mlp.experts - L.mlp.top) * L.mlp.ff * self.d_model for L in self.layers
+            idle = sum((3 if L.mlp.glu else 2) * (L.mlp.experts - L.mlp.top) * L.mlp.ff * self.d_model for L in self.layers
                        if L.mlp is not None and L.mlp.kind == "moe")
             return self.n_params() - idle
         if not self.is_moe:
@@ -105,8 +105,7 @@ class ModelConfig:
 
     def kv_bytes_per_token(self, dtype_bytes: int = 2) -> int:
         if self.layers:
-            att = [m for i in self.layer_runs for m in self.layers[i].mixer.parts if m.kind == "attention"]
-            return sum(a.kv_heads * (a.dim + a.vdim) for a in att) * dtype_bytes
+            return sum(getattr(m, "cache_values", 0) for i in self.layer_runs for m in self.layers[i].mixer.parts) * dtype_bytes
         return 2 * self.n_layers * self.kv_dim * dtype_bytes
 
     def to_dict(self) -> dict[str, Any]:
@@ -167,6 +166,28 @@ def _povatar_preset(name: str, *, width: int, vocab: int, n_layers: int, heads: 
     return povatar_model((layer,) * n_layers, width=width, vocab=vocab, eps=1e-5, emb_scale=width ** 0.5, name=name)
 
 
+def _zagolix_preset(name: str, *, width: int, vocab: int, pattern: str, ff: int, heads: int, kv_heads: int, dim: int, l_heads: int,
+                    l_dim: int, rot: int, l_vdim: int, q_rank: int, kv_rank: int, m_heads: int, m_dim: int, m_vdim: int, e_ff: int,
+                    experts: int, top: int, groups: int, keep: int) -> ModelConfig:
+    """A Zagolix-shaped configuration: one letter per layer, 'a' differential attention, 'l' latent attention, 's' latent
+    attention that reads what the last 'l' keeps, 'm' matrix memory. The first layer's feed-forward is dense."""
+    from .layer_spec import AttentionSpec, DenseMlpSpec, LatentSpec, LayerSpec, MemorySpec, MoeSpec, RotarySpec, zagolix_model
+
+    moe = MoeSpec(e_ff, experts, top, act="silu_glu", scores="sigmoid", groups=groups, keep=keep)
+    layers, owner = [], None
+    for i, ch in enumerate(pattern):
+        if ch == "a":
+            mx = AttentionSpec(heads, kv_heads, dim, 2 * dim, dim ** -0.5, bias=True, diff=0.5, temp_coef=0.1, temp_every=8192.0)
+        elif ch == "m":
+            mx = MemorySpec(m_heads, m_dim, m_vdim, 15.0)
+        else:
+            owner = i if ch == "l" else owner
+            mx = LatentSpec(l_heads, l_dim, l_vdim, q_rank, kv_rank, (l_dim + rot) ** -0.5, RotarySpec(rot, 10000.0, True),
+                            owner if ch == "s" else None)
+        layers.append(LayerSpec(mx, DenseMlpSpec(ff, act="gelu_tanh") if i == 0 else moe, post_norm=True))
+    return zagolix_model(tuple(layers), width=width, vocab=vocab, eps=1e-5, emb_scale=width ** 0.5, name=name)
+
+
 LAYER_LIST_PRESETS = {
     "kipolix-tiny": dict(width=128, vocab=1024, ff=256, pattern="arar", heads=4, kv_heads=2, dim=64, window=56,
                          keep_first=3, r_heads=2, r_dim=64, r_vdim=64, streams=2, loop=(1, 3, 2), buckets=1000),
@@ -185,8 +206,18 @@ POVATAR_PRESETS = {
 }
 
 
+ZAGOLIX_PRESETS = {
+    "zagolix-tiny": dict(width=128, vocab=1024, pattern="alsm", ff=256, heads=2, kv_heads=1, dim=32, l_heads=3, l_dim=32, rot=16,
+                         l_vdim=48, q_rank=56, kv_rank=64, m_heads=2, m_dim=32, m_vdim=64, e_ff=80, experts=9, top=3, groups=3, keep=2),
+    # layers of a mid-size mixture: latents of 512 + 64 values, two layers per latent, memories of 256 x 512, 8 of 64 experts
+    "zagolix-16b": dict(width=2048, vocab=128256, pattern="alsm" * 8, ff=10944, heads=16, kv_heads=4, dim=64, l_heads=16, l_dim=128,
+                        rot=64, l_vdim=128, q_rank=1536, kv_rank=512, m_heads=4, m_dim=256, m_vdim=512, e_ff=1408, experts=64,
+                        top=6, groups=8, keep=4),
+}
+
+
 def preset_names() -> list:
-    return [*PRESETS, *LAYER_LIST_PRESETS, *POVATAR_PRESETS]
+    return [*PRESETS, *LAYER_LIST_PRESETS, *POVATAR_PRESETS, *ZAGOLIX_PRESETS]
 
 
 def preset(name: str, **overrides) -> ModelConfig:
@@ -194,6 +225,8 @@ def preset(name: str, **overrides) -> ModelConfig:
         return replace(_kipolix_preset(name, **LAYER_LIST_PRESETS[name]), **overrides)
     if name in POVATAR_PRESETS:
         return replace(_povatar_preset(name, **POVATAR_PRESETS[name]), **overrides)
+    if name in ZAGOLIX_PRESETS:
+        return replace(_zagolix_preset(name, **ZAGOLIX_PRESETS[name]), **overrides)
     if name not in PRESETS:
         raise KeyError(f"unknown model preset {name!r}; known: {sorted(preset_names())}")
     return replace(PRESETS[name], **overrides)

@@ -20,6 +20,7 @@ class CpuHybridModel:
         self.cfg, self.num_blocks = cfg, num_blocks
         self.w = {n: torch.from_numpy(np.ascontiguousarray(src.f32(n), dtype=np.float32)) for n, _ in tensor_names(cfg)}
         self.embed = self.w["embed"]
+        self.head = self.w["embed" if cfg.tie_embeddings else "head"]
         self.runs = []
         self.pk, self.pv, self.states = [], [], []
         for li in cfg.layer_runs:
@@ -27,8 +28,19 @@ class CpuHybridModel:
             for mx in cfg.layers[li].mixer.parts:
                 if mx.kind == "attention":
                     at.append(len(self.pk))
-                    self.pk.append(torch.zeros(num_blocks, mx.kv_heads, 16, mx.dim))
+                    self.pk.append(torch.zeros(num_blocks, mx.kv_heads, 16, mx.maps * mx.dim))
                     self.pv.append(torch.zeros(num_blocks, mx.kv_heads, 16, mx.vdim))
+                elif mx.kind == "latent_attention":   # the latents, and the rotated key parts of all heads
+                    if mx.kv_from is not None:
+                        at.append(self.runs[mx.kv_from][1][0])
+                        continue
+                    at.append(len(self.pk))
+                    self.pk.append(torch.zeros(num_blocks, 1, 16, mx.rot_dim))
+                    self.pv.append(torch.zeros(num_blocks, 1, 16, mx.kv_rank))
+                elif mx.kind == "mlstm":   # memory, normaliser, running maximum
+                    at.append(len(self.states))
+                    self.states.append((torch.zeros(state_slots, mx.heads, mx.dim, mx.vdim), torch.zeros(state_slots, mx.heads, mx.dim),
+                                        torch.zeros(state_slots, mx.heads)))
                 elif mx.kind == "ssd":   # state, and the last inputs of the convolution, the newest last
                     at.append(len(self.states))
                     self.states.append((torch.zeros(state_slots, mx.heads, mx.state, mx.vdim),
@@ -66,18 +78,21 @@ class CpuHybridModel:
         return torch.cat([out, rest], -1)
 
     def _attention(self, a, p: str, ci: int, h, pos, seqs, blk, off):
-        T, w = h.shape[0], self.w
-        q, k = h @ w[p + "q"].T, h @ w[p + "k"].T
+        T, w, n2 = h.shape[0], self.w, a.maps
+        q, k, v = (h @ w[p + n].T + (w[f"{p}{n}.b"] if a.bias else 0.0) for n in ("q", "k", "v"))
         if a.qk_norm == "projection":
             q, k = self._unit(q) * w[p + "q.norm"], self._unit(k) * w[p + "k.norm"]
-        q = self._rotate(q.view(T, a.heads, a.dim), pos, a.rot)
-        self.pk[ci][blk, :, off] = self._rotate(k.view(T, a.kv_heads, a.dim), pos, a.rot)
-        self.pv[ci][blk, :, off] = (h @ w[p + "v"].T).view(T, a.kv_heads, a.vdim)
-        out = torch.zeros(T, a.heads, a.vdim)
-        g = a.heads // a.kv_heads
+        q = self._rotate(q.view(T, a.heads * n2, a.dim), pos, a.rot)
+        if a.temp_coef:
+            q = q * (1.0 + a.temp_coef * torch.log(torch.floor((pos + 1) / a.temp_every) + 1.0))[:, None, None]
+        self.pk[ci][blk, :, off] = self._rotate(k.view(T, a.kv_heads * n2, a.dim), pos, a.rot).reshape(T, a.kv_heads, n2 * a.dim)
+        self.pv[ci][blk, :, off] = v.view(T, a.kv_heads, a.vdim)
+        out = torch.zeros(T, a.heads * n2, a.vdim)
         for r0, n, ctx, table, _ in seqs:
-            pages = torch.as_tensor(table[:(ctx + 15) // 16].astype(np.int64))
-            take = lambda c: c[pages].permute(0, 2, 1, 3).reshape(-1, c.shape[1], c.shape[3])[:ctx].repeat_interleave(g, 1)
+            keys = self._pages(self.pk[ci], table, ctx).reshape(ctx, a.kv_heads, n2, a.dim)
+            values = self._pages(self.pv[ci], table, ctx)
+            g = a.heads // a.kv_heads
+            keys = keys.repeat_interleave(g, 1).reshape(ctx, a.heads * n2, a.dim)
             i = torch.arange(ctx - n, ctx)[:, None]
             j = torch.arange(ctx)[None]
             see = j <= i
@@ -85,12 +100,60 @@ class CpuHybridModel:
                 see = see & ((i - j < a.window) | (j < a.keep_first))
             if a.chunk:
                 see = see & (i // a.chunk == j // a.chunk)
-            s = torch.einsum("ihd,jhd->hij", q[r0:r0 + n], take(self.pk[ci])) * a.scale
+            s = torch.einsum("ihd,jhd->hij", q[r0:r0 + n], keys) * a.scale
             s = s.masked_fill(~see[None], float("-inf"))
             if a.sink is not None:
                 s = torch.cat([s, torch.full_like(s[..., :1], a.sink)], -1)
-            out[r0:r0 + n] = torch.einsum("hij,jhe->ihe", torch.softmax(s, -1)[..., :ctx], take(self.pv[ci]))
+            out[r0:r0 + n] = torch.einsum("hij,jhe->ihe", torch.softmax(s, -1)[..., :ctx], values.repeat_interleave(g * n2, 1))
+        if a.diff is not None:
+            lam = torch.exp((w[p + "lq1"] * w[p + "lk1"]).sum()) - torch.exp((w[p + "lq2"] * w[p + "lk2"]).sum()) + a.diff
+            two = out.view(T, a.heads, 2, a.vdim)
+            out = self._unit(two[:, :, 0] - lam * two[:, :, 1]) * (1.0 - a.diff)
         return out.reshape(T, -1) @ w[p + "o"].T
+
+    @staticmethod
+    def _pages(c: torch.Tensor, table, ctx: int) -> torch.Tensor:
+        """Cached rows of a sequence in order: [ctx, heads, values]."""
+        pages = torch.as_tensor(table[:(ctx + 15) // 16].astype(np.int64))
+        return c[pages].permute(0, 2, 1, 3).reshape(-1, c.shape[1], c.shape[3])[:ctx]
+
+    def _latent(self, a, p: str, ci: int, h, pos, seqs, blk, off):
+        T, w, H = h.shape[0], self.w, a.heads
+        q = ((self._unit(h @ w[p + "dq"].T) * w[p + "dq.norm"]) @ w[p + "uq"].T).view(T, H, a.dim + a.rot_dim)
+        qn, qr = q[..., :a.dim], self._rotate(q[..., a.dim:], pos, a.rot)
+        if a.kv_from is None:
+            kv = h @ w[p + "dkv"].T
+            self.pv[ci][blk, :, off] = (self._unit(kv[:, :a.kv_rank]) * w[p + "dkv.norm"])[:, None]
+            self.pk[ci][blk, :, off] = self._rotate(kv[:, None, a.kv_rank:], pos, a.rot)
+        out = torch.zeros(T, H, a.vdim)
+        uk, uv = w[p + "uk"].view(H, a.dim, -1), w[p + "uv"].view(H, a.vdim, -1)
+        for r0, n, ctx, table, _ in seqs:
+            c, kr = self._pages(self.pv[ci], table, ctx)[:, 0], self._pages(self.pk[ci], table, ctx)[:, 0]
+            s = torch.einsum("ihd,hdr,jr->hij", qn[r0:r0 + n], uk, c) + torch.einsum("ihd,jd->hij", qr[r0:r0 + n], kr)
+            see = torch.arange(ctx)[None] <= torch.arange(ctx - n, ctx)[:, None]
+            pr = torch.softmax((s * a.scale).masked_fill(~see[None], float("-inf")), -1)
+            out[r0:r0 + n] = torch.einsum("hij,jr,her->ihe", pr, c, uv)
+        return out.reshape(T, -1) @ w[p + "o"].T
+
+    def _memory(self, r, p: str, ci: int, h, seqs):
+        T, w, F = h.shape[0], self.w, torch.nn.functional
+        q = (h @ w[p + "q"].T).view(T, r.heads, r.dim) * r.dim ** -0.5
+        k, v = (h @ w[p + "k"].T).view(T, r.heads, r.dim), (h @ w[p + "v"].T).view(T, r.heads, r.vdim)
+        cap = lambda n: r.gate_cap * torch.tanh((h @ w[p + n].T + w[f"{p}{n}.b"]) / r.gate_cap)
+        gi, gf = cap("i"), F.logsigmoid(cap("f"))
+        out = torch.zeros(T, r.heads, r.vdim)
+        for r0, n, ctx, _, slot in seqs:
+            S, N, m = (torch.zeros_like(x[slot]) if ctx == n else x[slot] for x in self.states[ci])
+            for t in range(r0, r0 + n):
+                m2 = torch.maximum(gf[t] + m, gi[t])
+                keep, add, m = torch.exp(gf[t] + m - m2), torch.exp(gi[t] - m2), m2
+                S = keep[:, None, None] * S + (add[:, None] * k[t])[:, :, None] * v[t][:, None, :]
+                N = keep[:, None] * N + add[:, None] * k[t]
+                den = torch.maximum((N * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+                out[t] = torch.einsum("hde,hd->he", S, q[t]) / den[:, None]
+            for x, y in zip(self.states[ci], (S, N, m)):
+                x[slot] = y
+        return (self._unit(out).reshape(T, -1) * w[p + "norm"] * torch.sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T
 
     def _retention(self, r, p: str, ci: int, h, pos, seqs):
         T, w = h.shape[0], self.w
@@ -135,17 +198,55 @@ class CpuHybridModel:
         return (self._unit(u).reshape(T, -1) * w[p + "norm"]) @ w[p + "o"].T
 
     def _moe(self, e, p: str, h):
-        w = self.w
-        s = torch.softmax(h @ w[p + "router"].T, -1)
-        v, ids = torch.topk(s, e.top, -1)
-        v = v / (v.sum(-1, keepdim=True) + 1e-20)
+        w, F = self.w, torch.nn.functional
+        z = h @ w[p + "router"].T
+        s = torch.softmax(z, -1) if e.scores == "softmax" else torch.sigmoid(z)
+        open_ = s
+        if e.groups:
+            best = torch.topk(s.view(len(s), e.groups, -1), min(2, e.experts // e.groups), -1).values.sum(-1)
+            kept = torch.zeros_like(best).scatter_(1, torch.topk(best, e.keep, -1).indices, 1.0)
+            open_ = torch.where(kept.repeat_interleave(e.experts // e.groups, 1) > 0, s, torch.full_like(s, -1.0))
+        v, ids = torch.topk(open_, e.top, -1)
+        if e.scores == "softmax":
+            v = v / (v.sum(-1, keepdim=True) + 1e-20)
         out = torch.zeros_like(h)
         for i in range(e.experts):
             t, k = torch.nonzero(ids == i, as_tuple=True)
             if t.numel():
-                y = torch.relu(h[t] @ w[f"{p}e{i}.up"].T).square() @ w[f"{p}e{i}.down"].T
-                out.index_add_(0, t, v[t, k][:, None] * y)
+                q, x = f"{p}e{i}.", h[t]
+                u = x @ w[q + "up"].T
+                u = F.silu(x @ w[q + "gate"].T) * u if e.glu else torch.relu(u).square()
+                out.index_add_(0, t, v[t, k][:, None] * (u @ w[q + "down"].T))
         return out
+
+    def _dense(self, f, p: str, h):
+        w, F = self.w, torch.nn.functional
+        act = (lambda z: F.gelu(z, approximate="tanh")) if f.act == "gelu_tanh" else F.silu
+        return (act(h @ w[p + "gate"].T) * (h @ w[p + "up"].T)) @ w[p + "down"].T
+
+    def _mix(self, mx, p: str, ci: int, h, pos, seqs, blk, off):
+        if mx.kind == "attention":
+            return self._attention(mx, p, ci, h, pos, seqs, blk, off)
+        if mx.kind == "latent_attention":
+            return self._latent(mx, p, ci, h, pos, seqs, blk, off)
+        if mx.kind == "mlstm":
+            return self._memory(mx, p, ci, h, seqs)
+        return self._retention(mx, p, ci, h, pos, seqs)
+
+    def _feed(self, f, p: str, h):
+        return self._moe(f, p, h) if f.kind == "moe" else self._dense(f, p, h)
+
+    def _sandwich_layers(self, x, pos, seqs, blk, off):
+        """Layers with a norm on either side of every sublayer; returns the stream."""
+        w, one = self.w, self.cfg.norm_weight_offset
+        for li, (ci,) in self.runs:
+            L, p = self.cfg.layers[li], f"l{li}."
+            y = self._mix(L.mixer, p + "mix.", ci, self._unit(x) * (w[p + "norm1"] + one), pos, seqs, blk, off)
+            x = x + self._unit(y) * w[p + "norm1b"] * w[p + "ls1"]
+            if L.mlp is not None:
+                y = self._feed(L.mlp, p + "mlp.", self._unit(x) * (w[p + "norm2"] + one))
+                x = x + self._unit(y) * w[p + "norm2b"] * w[p + "ls2"]
+        return x
 
     def _parallel_layers(self, x, pos, seqs, blk, off):
         """Layers whose mixer and feed-forward read one residual stream side by side; returns the stream."""
@@ -183,6 +284,8 @@ class CpuHybridModel:
             x = x + w["bigram"][row]
         if any(L.parallel for L in cfg.layers):
             return self._head(self._parallel_layers(x * cfg.emb_scale, pos, seqs, blk, off), plan)
+        if any(L.post_norm for L in cfg.layers):
+            return self._head(self._sandwich_layers(x * cfg.emb_scale, pos, seqs, blk, off), plan)
         xs = x[None].repeat(max(1, cfg.streams), 1, 1)
         one = torch.ones(1)
 
@@ -194,17 +297,13 @@ class CpuHybridModel:
 
         for li, (ci,) in self.runs:
             L, p = cfg.layers[li], f"l{li}."
-            if L.mixer.kind == "attention":
-                sub(p, 1, lambda h: self._attention(L.mixer, p + "mix.", ci, h, pos, seqs, blk, off))
-            else:
-                sub(p, 1, lambda h: self._retention(L.mixer, p + "mix.", ci, h, pos, seqs))
+            sub(p, 1, lambda h: self._mix(L.mixer, p + "mix.", ci, h, pos, seqs, blk, off))
             if L.mlp is not None:
-                act = (lambda z: torch.nn.functional.gelu(z, approximate="tanh")) if L.mlp.act == "gelu_tanh" else torch.nn.functional.silu
-                sub(p, 2, lambda h: (act(h @ w[p + "mlp.gate"].T) * (h @ w[p + "mlp.up"].T)) @ w[p + "mlp.down"].T)
+                sub(p, 2, lambda h: self._feed(L.mlp, p + "mlp.", h))
         return self._head(xs.sum(0), plan)
 
     def _head(self, x: torch.Tensor, plan) -> torch.Tensor:
         rows = torch.as_tensor(plan.logit_rows.astype(np.int64))
         hl = self._unit(x[rows]) * (self.w["final.norm"] + self.cfg.norm_weight_offset)
-        self.logits = hl @ self.w["head"].T
+        self.logits = hl @ self.head.T
         return self.logits

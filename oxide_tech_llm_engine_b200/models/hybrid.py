@@ -24,6 +24,21 @@ and with mixer and feed-forward side by side:
       branch_norm   norms of both mixer outputs, weighted expert rows, residual, norms of the next layer
     final branch_norm over the logit rows -> gemm(head)
 
+and with a norm on either side of every sublayer:
+
+    branch_norm   embedding -> residual, norm of the first sublayer
+    per sublayer:
+      differential attention: as attention, two maps per head; their difference and its norm in the merge (decoding)
+                              or in diff_norm
+      latent attention:       gemm(query latent | latent) -> latent_rows -> gemm(q)
+        decoding:  heads (rotation), grouped gemm(q W_uk) -> latent_decode -> grouped gemm(W_uv)
+        prompts:   heads (rotation), latent_gather -> gemm(keys | values of all heads) -> prefill_rows
+      matrix memory:          gemm(q|k|v|gate) -> memory_decode / gemm(gates, fp32), chunked memory
+                  -> gemm(O, fp32 accumulator)
+      MLP:        as above;  experts: moe_route (-> moe_scatter) -> grouped gemm(gate|up, SwiGLU) -> grouped gemm(down)
+      branch_norm  norm of the sublayer's result (of the weighted expert rows), residual, norm of the next sublayer
+    final branch_norm over the logit rows -> gemm(head)
+
 In a captured decode step the three lines between two branch_norms run on streams of their own: the
 experts beside the projection and the mixers, the state-space mixer beside the attention.
 
@@ -55,12 +70,40 @@ def round_up(n: int, k: int) -> int:
     return (n + k - 1) // k * k
 
 
+def tc_head(a) -> int:
+    """Padded head size of the tensor-core attention kernels for a spec, 0 when they do not take it."""
+    big = max(a.maps * a.dim, a.vdim)
+    if a.heads * a.maps // a.kv_heads > 16 or big > 256:
+        return 0
+    if big > 128:      # plain causal attention only
+        return 256 if not (a.window or a.chunk or a.sink is not None) else 0
+    return 64 if big <= 64 else 128
+
+
+def latent_layout(a) -> tuple:
+    """(key columns, value columns, first unrotated column) of a latent-attention head; no value columns: the prompt
+    kernel does not take heads of these sizes."""
+    at = round_up(a.rot_dim, 8)
+    z = hops.prefill_size(at + round_up(a.dim, 8), round_up(a.vdim, 8))
+    return (*z, at) if z is not None else (at + round_up(a.dim, 8), 0, at)
+
+
+KV_PASS_ROWS = 65536      # positions whose keys and values are expanded at a time
+
+
 class _Sublayer:
     """What stream_norm needs around a sublayer, and the function that runs it."""
 
     def __init__(self, norm, hc, run, last_of: int):
         self.norm, self.hc, self.run = norm, hc, run
         self.last_of = last_of       # index of the layer run that this sublayer ends, or -1
+
+
+class _NormedSublayer:
+    """Norm weights of a sublayer's input and result (the latter times the layer scale), and the function that runs it."""
+
+    def __init__(self, norm, out, run, last_of: int):
+        self.norm, self.out, self.run, self.last_of = norm, out, run, last_of
 
 
 class _ParallelLayer:
@@ -72,17 +115,18 @@ class _ParallelLayer:
 
 class AttentionRun:
     """One run of an attention layer: weights shared by all passes, a KV cache of its own. Its projection rows
-    may be the first columns of wider ones (a layer with two mixers)."""
+    may be the first columns of wider ones (a layer with two mixers). With two maps per head both keys of a value head
+    lie in one cache row, and a query has zeros where the other map's key is."""
 
     def __init__(self, m: "HybridModel", spec, w: dict):
         self.m, self.spec, self.w = m, spec, w
         a = spec
-        self.group = a.heads // a.kv_heads
-        self.width = a.heads * a.dim + a.kv_heads * (a.dim + a.vdim)
-        big = max(a.dim, a.vdim)
-        # head sizes of the tensor-core kernels: q, k and v padded to 64 or 128 with zeros
-        self.tc = m.dtype == torch.bfloat16 and big <= 128 and self.group <= 16
-        self.dp, self.ep = (64 if big <= 64 else 128,) * 2 if self.tc else (a.dim, a.vdim)
+        self.nq, self.dk = a.heads * a.maps, a.maps * a.dim     # query heads, values of a key row
+        self.width = a.in_width
+        self.acc_k = round_up(a.out_dim, 64)
+        # head sizes of the tensor-core kernels: q, k and v padded with zeros
+        self.tc = m.dtype == torch.bfloat16 and tc_head(a) > 0
+        self.dp, self.ep = (tc_head(a),) * 2 if self.tc else (self.dk, a.vdim)
         self.k = torch.zeros(m.num_blocks, a.kv_heads, 16, self.dp, dtype=m.dtype, device=m.device)
         self.v = torch.zeros(m.num_blocks, a.kv_heads, 16, self.ep, dtype=m.dtype, device=m.device)
         m.k_cache.append(self.k)
@@ -93,30 +137,156 @@ class AttentionRun:
 
     def attend(self, s: StepInputs, proj: torch.Tensor) -> torch.Tensor:
         m, a, w, M = self.m, self.spec, self.w, s.m
-        q = m.buffer(("q", a.heads * self.dp, a.dim), a.heads * self.dp)
-        hops.heads(proj, M, h=a.heads, g=a.kv_heads, d=a.dim, e=a.vdim, rot=w["rot"], positions=s.positions, q_out=q,
+        q = m.buffer(("q", self.nq * self.dp, a.dim, a.maps), self.nq * self.dp)
+        hops.heads(proj, M, h=self.nq, g=a.kv_heads * a.maps, d=a.dim, e=a.vdim, rot=w["rot"], positions=s.positions, q_out=q,
                    q_hd=self.dp, q_norm=w["q_norm"], k_norm=w["k_norm"], eps=m.cfg.rms_eps, k_cache=self.k,
-                   v_cache=self.v, slots=s.slot_mapping)
-        out = m.buffer(("o", a.out_dim), round_up(a.out_dim, 64))
+                   v_cache=self.v, slots=s.slot_mapping, maps=a.maps, bias=w.get("bias"), temp_coef=a.temp_coef,
+                   temp_every=a.temp_every)
+        out = m.buffer(("o", a.out_dim), self.acc_k)
+        # both maps' results in fp32, where the difference is not taken in the merge
+        both = m.maps_buffer(self.nq * a.vdim) if a.diff is not None else out
+        lam = (w["lam"], 1.0 - a.diff, m.cfg.rms_eps) if a.diff is not None else ()
         nd = s.n_decode
         kw = dict(window=a.window, keep_first=a.keep_first if a.window else 0, scale=a.scale, chunk=a.chunk,
                   sink=-math.inf if a.sink is None else a.sink)
+        done = 0       # rows whose difference has been taken
         if self.tc:
-            kw.update(out_d=a.vdim, exact_p=True)
             if nd > 0:
-                ops.paged_decode(q[:nd].view(nd, a.heads, self.dp), self.k, self.v, s.block_tables, s.seq_lens,
-                                 s.pages_per_split, m.part_o, m.part_ml, out[:nd], batch=nd, max_splits=m.max_splits, **kw)
+                ops.paged_decode(q[:nd].view(nd, self.nq, self.dp), self.k, self.v, s.block_tables, s.seq_lens,
+                                 s.pages_per_split, m.part_o, m.part_ml, out[:nd], batch=nd, max_splits=m.max_splits, out_d=a.vdim,
+                                 exact_p=True, diff=lam, **kw)
+                done = nd
             if s.n_prefill > 0:
-                ops.paged_prefill(q.view(-1, a.heads, self.dp), self.k, self.v, s.prefill_block_tables, s.tile_seq, s.tile_q0,
-                                  s.q_start, s.q_lens, s.ctx_lens, out, n_tiles=s.n_tiles, **kw)
+                args = (q.view(-1, self.nq, self.dp), self.k, self.v, s.prefill_block_tables, s.tile_seq, s.tile_q0,
+                        s.q_start, s.q_lens, s.ctx_lens, both)
+                if self.dp > 128:
+                    hops.prefill_pages(*args, n_tiles=s.n_tiles, scale=a.scale, out_d=a.vdim)
+                else:
+                    ops.paged_prefill(*args, n_tiles=s.n_tiles, out_d=a.vdim, exact_p=True, **kw)
         else:
-            kw.update(h=a.heads, d=a.dim, e=a.vdim, out=out)
+            kw.update(h=self.nq, d=self.dk, e=a.vdim, out=both)
             if nd > 0:
                 hops.row_attention(q, self.dp, self.k, self.v, s.block_tables, n=nd, seq_lens=s.seq_lens, **kw)
             if s.n_prefill > 0:
                 hops.row_attention(q, self.dp, self.k, self.v, s.prefill_block_tables, n=s.n_tiles, tile_seq=s.tile_seq,
                                    tile_q0=s.tile_q0, q_start=s.q_start, q_lens=s.q_lens, ctx_lens=s.ctx_lens, **kw)
+        if lam and done < M:
+            hops.diff_norm(both[done:], M - done, h=a.heads, e=a.vdim, lam=lam[0], gain=lam[1], eps=lam[2], out=out[done:])
         return out[:M]
+
+
+class LatentRun:
+    """One run of a latent-attention layer; the cache is its own or that of the layer it reads. Heads lie in padded
+    layouts: queries and expanded keys [rotated | unrotated | zeros], so both parts start on 16 bytes."""
+
+    def __init__(self, m: "HybridModel", spec, w: dict):
+        self.m, self.spec, self.w = m, spec, w
+        a = spec
+        self.width, self.cp = a.in_width, a.cache_row
+        self.dk, self.dv, self.at = latent_layout(a)
+        self.d8, self.r8, self.ep = round_up(a.dim, 8), round_up(a.kv_rank, 8), round_up(a.vdim, 8)
+        self.acc_k = round_up(a.heads * self.ep, 64)
+        bf16 = m.dtype == torch.bfloat16
+        self.expand = bf16 and self.dv > 0                                    # prompts over expanded keys and values
+        self.tc = bf16 and hops.latent_decode_ok(a.kv_rank, self.cp)
+        if a.kv_from is None:
+            self.cache = torch.zeros(m.num_blocks, 1, 16, self.cp, dtype=m.dtype, device=m.device)
+            m.k_cache.append(self.cache)
+        else:
+            self.cache = m.latents[a.kv_from].cache
+
+    def __call__(self, s: StepInputs, h: torch.Tensor) -> None:
+        m, a, w, M = self.m, self.spec, self.w, s.m
+        proj = m.project(h, w["w_in"], self.width)
+        cq = m.buffer(("cq", a.q_rank), round_up(a.q_rank, 64))
+        kw = dict(kv_col=a.kv_col, kv_rank=a.kv_rank, kv_norm=w["kv_norm"], cache=self.cache, slots=s.slot_mapping,
+                  rot=w["rot"]) if a.kv_from is None else {}
+        hops.latent_rows(proj, M, q_rank=a.q_rank, q_norm=w["q_norm"], q_out=cq, positions=s.positions, eps=m.cfg.rms_eps, **kw)
+        q = m.buffer(("q_up", a.heads, self.dk), round_up(a.heads * self.dk, 64))
+        m.product(cq[:M], w["w_uq"], q)
+        o = m.buffer(("o_lat", a.heads, self.ep), self.acc_k)
+        na = s.n_decode if self.expand else M
+        if na > 0:
+            self._absorbed(s, q, o, na)
+        if self.expand and s.n_prefill > 0:
+            self._expanded(s, q, o)
+        m.into_acc(o[:M], w["w_o"])
+
+    def _absorbed(self, s: StepInputs, q: torch.Tensor, o: torch.Tensor, n: int) -> None:
+        """Rows against the latents: queries times W_uk, sums of latents times W_uv."""
+        m, a, w, H, nd = self.m, self.spec, self.w, self.spec.heads, s.n_decode
+        qa = m.buffer(("q_lat", H, self.cp, a.kv_rank), H * self.cp)
+        ctx = m.buffer(("ctx", H, self.r8, a.kv_rank), H * self.r8)
+        if a.rot is not None:
+            hops.heads(q, n, h=H, g=0, d=a.rot_dim, e=4, rot=w["rot"], positions=s.positions, q_out=qa[:, a.kv_rank:], q_hd=self.cp,
+                       q_pd=self.dk)
+        heads = lambda t, width, lo, hi: t[:n, :H * width].view(n, H, width)[:, :, lo:hi].transpose(0, 1)
+        m.per_head(heads(q, self.dk, self.at, self.at + self.d8), w["w_uk"], heads(qa, self.cp, 0, a.kv_rank))
+        if self.tc:
+            hops.latent_decode(qa[:n].view(n, H, self.cp), self.cache, s.block_tables, s.seq_lens, s.pages_per_split, m.part_o,
+                               m.part_ml, ctx, rows=n, kv_rank=a.kv_rank, max_splits=m.max_splits, scale=a.scale, o_hd=self.r8)
+        else:
+            kw = dict(h=H, d=a.kv_rank + a.rot_dim, e=a.kv_rank, window=0, keep_first=0, scale=a.scale, out=ctx, o_hd=self.r8)
+            if nd > 0:
+                hops.row_attention(qa, self.cp, self.cache, self.cache, s.block_tables, n=nd, seq_lens=s.seq_lens, **kw)
+            if s.n_prefill > 0:
+                hops.row_attention(qa, self.cp, self.cache, self.cache, s.prefill_block_tables, n=s.n_tiles, tile_seq=s.tile_seq,
+                                   tile_q0=s.tile_q0, q_start=s.q_start, q_lens=s.q_lens, ctx_lens=s.ctx_lens, **kw)
+        m.per_head(heads(ctx, self.r8, 0, self.r8), w["w_uv"], heads(o, self.ep, 0, self.ep))
+
+    def _expanded(self, s: StepInputs, q: torch.Tensor, o: torch.Tensor) -> None:
+        m, a, w, H, nd = self.m, self.spec, self.w, self.spec.heads, s.n_decode
+        if a.rot is not None:      # in place: a row's heads are read and written by one CTA, value by value
+            hops.heads(q[nd:], s.m - nd, h=H, g=0, d=a.rot_dim, e=4, rot=w["rot"], positions=s.positions[nd:], q_out=q[nd:],
+                       q_hd=self.dk, q_pd=self.dk)
+        for i, (s0, s1, t0, t1, rows, pages) in enumerate(s.kv_passes):
+            lat = m.rows("latents", rows, self.cp)
+            kv = m.rows("kv", rows, H * (self.dk + self.dv))
+            if m.gathered != (i, id(self.cache)):
+                hops.latent_gather(self.cache, s.prefill_block_tables, s.ctx_lens, s.kv_start, seq0=s0, n_seqs=s1 - s0, max_pages=pages,
+                                   out=lat)
+                m.gathered = (i, id(self.cache))
+            m.product(lat, w["w_kv"], kv)
+            hops.prefill_rows(q[:, :H * self.dk].view(-1, H, self.dk), kv, s.tile_seq[t0:], s.tile_q0[t0:], s.q_start, s.q_lens,
+                              s.ctx_lens, s.kv_start, o, dk=self.dk, dv=self.dv, g=H, n_tiles=t1 - t0, scale=a.scale, out_d=self.ep)
+
+
+class MemoryRun:
+    """One run of a matrix-memory layer: a memory with its normaliser and a running maximum per slot."""
+
+    def __init__(self, m: "HybridModel", spec, w: dict):
+        self.m, self.spec, self.w = m, spec, w
+        r = spec
+        self.width, self.acc_k = r.in_width, round_up(r.out_dim, 64)
+        f32 = dict(dtype=torch.float32, device=m.device)
+        self.state = torch.zeros(m.state_slots, r.heads, r.dim * r.vdim + r.dim, **f32)
+        self.state_m = torch.zeros(m.state_slots, r.heads, **f32)
+        m.states += [self.state, self.state_m]
+        self.chunks = m.dtype == torch.bfloat16 and hops.memory_chunks_ok(r.dim, r.vdim)
+        self.zp = round_up(2 * r.heads, 64)
+
+    def __call__(self, s: StepInputs, h: torch.Tensor) -> None:
+        m, r, w, M, nd = self.m, self.spec, self.w, s.m, s.n_decode
+        proj = m.project(h, w["w_in"], self.width)
+        out = m.buffer(("o", r.out_dim), self.acc_k)
+        kw = dict(h=r.heads, d=r.dim, e=r.vdim, z_bias=w["z_bias"], cap=r.gate_cap, eps=m.cfg.rms_eps, norm_w=w["norm"],
+                  state=self.state, state_m=self.state_m)
+        z = None
+        if m.dtype == torch.float32 or s.n_prefill > 0:
+            # pre-activations of the gates in fp32; bf16 decode rows take theirs from the rows themselves
+            lo = 0 if m.dtype == torch.float32 else nd
+            z = m.gates_buffer(self.zp)
+            m.product_f32(h[lo:], w["w_z"], z[lo:M])
+        if nd > 0:
+            own = dict(z=z) if m.dtype == torch.float32 else dict(hidden=h, z_w=w["w_z"])
+            hops.memory_decode(proj, nd, row_slots=s.decode_slots, positions=s.positions, out=out, **own, **kw)
+        if s.n_prefill > 0:
+            n = (hops.memory_ws_elems(r.heads, r.dim, r.vdim, s.n_tiles) if self.chunks
+                 else M * r.out_dim + s.n_prefill * r.heads * (r.dim + 1))
+            hops.memory_prefill(proj, M, z=z, seq_slots=s.prefill_slots, tile_seq=s.tile_seq, tile_q0=s.tile_q0, q_start=s.q_start,
+                                q_lens=s.q_lens, ctx_lens=s.ctx_lens, n_tiles=s.n_tiles, n_seqs=s.n_prefill,
+                                ws=m.scratch("chunk_states", n), chunks=self.chunks, out=out, **kw)
+        m.into_acc(out[:M], w["w_o"])
 
 
 class RetentionRun:
@@ -194,18 +364,20 @@ class MoeRun:
     def __init__(self, m: "HybridModel", spec, w: dict):
         self.m, self.spec, self.w = m, spec, w
         self.fp = round_up(spec.ff, 64)
+        self.acc_k = 0             # no fp32 accumulator
         self.b = m.moe_buffers(spec.experts, spec.top, self.fp)
 
     def __call__(self, s: StepInputs, h: torch.Tensor, start=nullcontext()) -> tuple:
         m, e, w, b, M = self.m, self.spec, self.w, self.b, s.m
         E, top = e.experts, e.top
-        route = dict(e=E, top=top, weight=b["weight"], expert=b["expert"], slot=b["slot"])
+        route = dict(e=E, top=top, weight=b["weight"], expert=b["expert"], slot=b["slot"], softmax=e.scores == "softmax",
+                     groups=e.groups, keep=e.keep)
         if m.dtype == torch.float32 or m.few_rows(M):
             with start:
                 hops.moe_route(h, w["router"], M, **route)
             pairs = M * top
             rows, act = b["out"][:pairs], b["act"][:pairs]
-            hops.moe_rows(h, w["up"], b["expert"], pairs, top=top, per_pair=False, y=act, act=2)
+            hops.moe_rows(h, w["up"], b["expert"], pairs, top=top, per_pair=False, y=act, act=3 if e.glu else 2)
             hops.moe_rows(act, w["down"], b["expert"], pairs, top=top, per_pair=True, y=rows)
             return rows, b["slot"], b["weight"], top
         if M <= 128:
@@ -224,7 +396,11 @@ class MoeRun:
             ops.gemm(h, w["router_p"], out=logits, epi=ops.EPI_STORE_F32, **m._gemm_shape(M, logits.shape[1], m.dp, store=True))
             hops.moe_route(h, w["router"], M, mode=2, logits=logits, counts=b["counts"], **route)
             hops.moe_scatter(h, M, e=E, top=top, expert=b["expert"], slot=b["slot"], counts=b["counts"], xs=gx)
-        ops.gemm(gx, w["up"], out=ga, group_counts=b["counts"], m_tiles=m_tiles, act=2, bn=m.group_bn(m_tiles, self.fp))
+        if e.glu:
+            ops.gemm(gx, w["up"], out=ga, epi=ops.EPI_SWIGLU_BF16, group_counts=b["counts"], m_tiles=m_tiles,
+                     bn=m.group_bn(m_tiles, 2 * self.fp, whole=True))
+        else:
+            ops.gemm(gx, w["up"], out=ga, group_counts=b["counts"], m_tiles=m_tiles, act=2, bn=m.group_bn(m_tiles, self.fp))
         ops.gemm(ga, w["down"], out=gr, group_counts=b["counts"], m_tiles=m_tiles, bn=m.group_bn(m_tiles, m.dp),
                  done_ticket=b["ticket"], reset_on_done=b["counts"])
         return rows, b["slot"], b["weight"], top
@@ -278,7 +454,7 @@ class ParallelRun:
 class MlpRun:
     def __init__(self, m: "HybridModel", spec, w: dict):
         self.m, self.spec, self.w = m, spec, w
-        self.ip = round_up(spec.ff, 64)
+        self.ip = self.acc_k = round_up(spec.ff, 64)
         self.act = 1 if spec.act == "gelu_tanh" else 0
 
     def __call__(self, s: StepInputs, h: torch.Tensor) -> None:
@@ -297,7 +473,8 @@ class MlpRun:
         m.into_acc(act[:M], self.w["w_down"])
 
 
-RUNS = {"attention": AttentionRun, "retention": RetentionRun}
+RUNS = {"attention": AttentionRun, "retention": RetentionRun, "latent_attention": LatentRun, "mlstm": MemoryRun}
+MLP_RUNS = {"dense": MlpRun, "moe": MoeRun}
 
 
 class HybridModel(GemmShapes):
@@ -344,11 +521,19 @@ class HybridModel(GemmShapes):
         if self.parallel and (cfg.streams or cfg.loop or cfg.bigram or not all(L.parallel for L in cfg.layers)):
             raise ConfigError(f"{cfg.name}: layers with mixer and feed-forward side by side come without hyper-connected streams, "
                               "loops and a bigram embedding, and without other layers")
+        self.sandwich = any(L.post_norm for L in cfg.layers)
+        if self.sandwich and (self.parallel or cfg.streams or cfg.loop or cfg.bigram or not all(L.post_norm for L in cfg.layers)):
+            raise ConfigError(f"{cfg.name}: layers with a norm behind every sublayer come without hyper-connected streams, loops and "
+                              "a bigram embedding, and without other layers")
         moe = [L.mlp for L in cfg.layers if L.mlp is not None and L.mlp.kind == "moe"]
         if any(e.experts > hops.max_experts()[0] or e.top > hops.max_experts()[1] for e in moe):
             raise ConfigError(f"{cfg.name}: at most {hops.max_experts()[0]} experts, {hops.max_experts()[1]} of them chosen")
+        if any(e.groups > hops.max_groups() for e in moe):
+            raise ConfigError(f"{cfg.name}: at most {hops.max_groups()} groups of experts")
         att = [p for L in cfg.layers for p in L.mixer.parts if p.kind == "attention"]
-        self.hkv = min((a.kv_heads for a in att), default=1)
+        lat = [p for L in cfg.layers for p in L.mixer.parts if p.kind == "latent_attention"]
+        # CTAs per sequence and split of the decode attention
+        self.hkv = min([a.kv_heads for a in att] + [(a.heads + 31) // 32 for a in lat], default=1)
         self.x = torch.zeros(max_tokens, self.streams, d, dtype=torch.float32, device=dev)
         self.h = torch.zeros(max_tokens, self.dp, dtype=self.dtype, device=dev)
         n_acc = 2 if self.parallel else 1
@@ -362,8 +547,9 @@ class HybridModel(GemmShapes):
         self.lm_h = torch.zeros(self.max_logits, self.dp, dtype=self.dtype, device=dev)
         self.logits_buf = torch.zeros(self.max_logits, self.vp, dtype=torch.float32, device=dev)
         self.logits = self.logits_buf[:, :cfg.vocab_size]
-        heads = max((a.heads for a in att), default=1)
-        self.part_o = torch.zeros(max_seqs * heads * max_splits * 128, dtype=torch.float32, device=dev)
+        heads = max([a.heads * a.maps for a in att] + [a.heads for a in lat], default=1)
+        part = max([a.heads * a.maps * max(128, tc_head(a)) for a in att] + [a.heads * a.kv_rank for a in lat], default=128)
+        self.part_o = torch.zeros(max_seqs * max_splits * part, dtype=torch.float32, device=dev)
         self.part_ml = torch.zeros(max_seqs * heads * max_splits * 2, dtype=torch.float32, device=dev)
         widths = [self._in_width(L.mixer) for L in cfg.layers]
         self.proj = torch.zeros(max_tokens * max(widths), dtype=self.dtype, device=dev)
@@ -372,6 +558,9 @@ class HybridModel(GemmShapes):
         self._buffers: dict = {}
         self._scratch: dict = {}
         self._moe: dict = {}
+        self._rows: dict = {}
+        self.latents: dict = {}       # runs of latent attention by layer
+        self.gathered = None          # (pass, cache) of this step whose latents lie in the gather buffer
         self.k_cache: list = []
         self.v_cache: list = []
         self.states: list = []
@@ -386,20 +575,19 @@ class HybridModel(GemmShapes):
         if mix.kind == "parallel":
             n = HybridModel._in_width(mix.left) + mix.right.width_p
             return round_up(n, 256 if n >= 2048 else 64)      # wide projections in whole tiles of the widest kind
-        w = (mix.heads * mix.dim + mix.kv_heads * (mix.dim + mix.vdim) if mix.kind == "attention"
-             else 2 * mix.heads * (mix.dim + mix.vdim))
-        return round_up(w, 64)
+        return round_up(mix.in_width, 64)
 
     @staticmethod
     def kv_block_bytes(cfg: ModelConfig, tp: int = 1, dtype: str = "bfloat16") -> int:
         """Device bytes of one 16-token KV block over all attention runs (0: no attention layers)."""
-        total = 0
-        for a in (p for i in cfg.layer_runs for p in cfg.layers[i].mixer.parts if p.kind == "attention"):
-            big = max(a.dim, a.vdim)
-            if dtype == "bfloat16" and big <= 128 and a.heads // a.kv_heads <= 16:
-                total += a.kv_heads * 16 * 2 * (64 if big <= 64 else 128) * 2
-            else:
-                total += a.kv_heads * 16 * (a.dim + a.vdim) * (2 if dtype == "bfloat16" else 4)
+        total, size = 0, 2 if dtype == "bfloat16" else 4
+        for a in (p for i in cfg.layer_runs for p in cfg.layers[i].mixer.parts):
+            if a.kind == "latent_attention":
+                total += 16 * a.cache_row * size if a.kv_from is None else 0
+            elif a.kind == "attention" and dtype == "bfloat16" and tc_head(a):
+                total += a.kv_heads * 16 * 2 * tc_head(a) * 2
+            elif a.kind == "attention":
+                total += 16 * a.cache_values * size
         return total
 
     @staticmethod
@@ -411,9 +599,11 @@ class HybridModel(GemmShapes):
         """Device bytes of a step's work space: streams, fp32 projections, rotated q / k, chunk states of
         retention, rows of the experts."""
         parts = [p for L in cfg.layers for p in L.mixer.parts]
-        wide = max(p.width_p if p.kind == "ssd" else p.heads * (p.dim + p.vdim) for p in parts)
-        chunk = max((p.state_elems for p in parts if p.kind == "retention"), default=0)
-        n = max_tokens * 4 * (max(1, cfg.streams) * cfg.d_model + 6 * wide) + 8 * (max_tokens // 128 + max_seqs) * chunk
+        wide = max(p.width_p if p.kind == "ssd" else p.heads * getattr(p, "maps", 1) * (p.dim + p.vdim) for p in parts)
+        chunk = max((p.state_elems for p in parts if p.kind in ("retention", "mlstm")), default=0)
+        # gathered latents, keys and values of all heads in the largest pass
+        lat = max((p.cache_row + p.heads * sum(latent_layout(p)[:2]) for p in parts if p.kind == "latent_attention"), default=0)
+        n = 2 * lat * max(KV_PASS_ROWS, max_tokens) + max_tokens * 4 * (max(1, cfg.streams) * cfg.d_model + 6 * wide) + 8 * (max_tokens // 128 + max_seqs) * chunk
         return n + max((HybridModel._moe_rows(L.mlp.experts, L.mlp.top, max_tokens) * 4 * (2 * cfg.d_model + L.mlp.ff)
                         for L in cfg.layers if L.mlp is not None and L.mlp.kind == "moe"), default=0)
 
@@ -437,9 +627,11 @@ class HybridModel(GemmShapes):
             self._moe[experts, top, fp] = b
         return b
 
-    def group_bn(self, m_tiles: int, n: int) -> int:
-        """Tile width of an expert GEMM: narrow while the tiles would not fill the SMs."""
+    def group_bn(self, m_tiles: int, n: int, whole: bool = False) -> int:
+        """Tile width of an expert GEMM: narrow while the tiles would not fill the SMs; `whole`: a divisor of n."""
         for bn in (256, 128):
+            if whole and n % bn:
+                continue
             if m_tiles * ((n + bn - 1) // bn) >= self._sms:
                 return bn
         return 64
@@ -451,6 +643,26 @@ class HybridModel(GemmShapes):
         if b is None:
             b = self._buffers[key] = torch.zeros(self.max_tokens, width, dtype=self.dtype, device=self.device)
         return b
+
+    def maps_buffer(self, width: int) -> torch.Tensor:
+        """fp32 rows of both maps of differential attention, shared by the layers of one width."""
+        return self._f32_rows("maps", width)
+
+    def gates_buffer(self, width: int) -> torch.Tensor:
+        return self._f32_rows("gates", width)
+
+    def _f32_rows(self, name: str, width: int) -> torch.Tensor:
+        b = self._buffers.get((name, width))
+        if b is None:
+            b = self._buffers[name, width] = torch.zeros(self.max_tokens, width, dtype=torch.float32, device=self.device)
+        return b
+
+    def rows(self, name: str, n: int, width: int) -> torch.Tensor:
+        """[n, width] rows of prompt steps in the model's dtype, grown on demand; never uninitialised memory."""
+        b = self._rows.get(name)
+        if b is None or b.numel() < n * width:
+            self._rows[name] = b = torch.zeros(n * width, dtype=self.dtype, device=self.device)
+        return b[:n * width].view(n, width)
 
     def scratch(self, name: str, n: int) -> torch.Tensor:
         """fp32 work space of prompt chunks (steps that are never captured in a graph), grown on demand."""
@@ -494,14 +706,100 @@ class HybridModel(GemmShapes):
     def _moe_weights(self, e, p: str, mat) -> dict:
         fp = round_up(e.ff, 64)
         kw = dict(dtype=self.dtype, device=self.device)
-        up, down = torch.zeros(e.experts, fp, self.dp, **kw), torch.zeros(e.experts, self.dp, fp, **kw)
+        up, down = torch.zeros(e.experts, (2 if e.glu else 1) * fp, self.dp, **kw), torch.zeros(e.experts, self.dp, fp, **kw)
         router = torch.zeros(round_up(e.experts, 64), self.dp, **kw)
         d = self.cfg.d_model
         for i in range(e.experts):
-            up[i, :e.ff, :d] = mat(f"{p}e{i}.up")
+            if e.glu:
+                g, u = (torch.cat([t, t.new_zeros(fp - e.ff, d)]) for t in (mat(f"{p}e{i}.gate"), mat(f"{p}e{i}.up")))
+                up[i, :, :d] = interleave32(g, u)
+            else:
+                up[i, :e.ff, :d] = mat(f"{p}e{i}.up")
             down[i, :d, :e.ff] = mat(f"{p}e{i}.down")
         router[:e.experts, :d] = mat(p + "router")
         return {"up": up, "down": down, "router": router[:e.experts], "router_p": router}
+
+    def _rotary(self, spec) -> hops.Rotary:
+        if spec not in self._rots:
+            self._rots[spec] = hops.Rotary(spec, self.device)
+        return self._rots[spec]
+
+    def _mixer_weights(self, mx, p: str, mat, vec) -> dict:
+        if mx.kind == "latent_attention":
+            return self._latent_weights(mx, p, mat, vec)
+        names = ("q", "k", "v") if mx.kind == "attention" else ("q", "k", "v", "g")
+        w = {"w_in": self._pad(torch.cat([mat(p + n) for n in names])), "w_o": self._pad(mat(p + "o")),
+             "rot": self._rotary(getattr(mx, "rot", None)), "q_norm": None, "k_norm": None}
+        if mx.kind == "attention":
+            if mx.qk_norm == "projection":
+                w["q_norm"], w["k_norm"] = vec(p + "q.norm"), vec(p + "k.norm")
+            if mx.bias:
+                w["bias"] = torch.cat([vec(f"{p}{n}.b") for n in names])
+            if mx.diff is not None:
+                a, b, c, d = (vec(p + n).double().cpu() for n in ("lq1", "lk1", "lq2", "lk2"))
+                w["lam"] = float(torch.exp((a * b).sum()) - torch.exp((c * d).sum())) + mx.diff
+        elif mx.kind == "retention":
+            w["decay_pow"] = hops.decay_powers(mx.decay, self.device)
+        elif mx.kind == "mlstm":
+            z = torch.cat([mat(p + "i"), mat(p + "f")])
+            wz = z.new_zeros(round_up(z.shape[0], 64), self.dp)
+            wz[:z.shape[0], :z.shape[1]] = z
+            w.update(w_z=wz, z_bias=torch.cat([vec(p + "i.b"), vec(p + "f.b")]), norm=vec(p + "norm"))
+        return w
+
+    def _latent_weights(self, a, p: str, mat, vec) -> dict:
+        """Tensors of latent attention in the head layouts of LatentRun. The expansion of a step's latents to keys takes the
+        rotated part through a unit matrix, so one product makes whole keys and values."""
+        H, R, D, T, E = a.heads, a.kv_rank, a.dim, a.rot_dim, a.vdim
+        dk, dv, at = latent_layout(a)
+        d8, r8, ep = round_up(D, 8), round_up(R, 8), round_up(E, 8)
+        uq, uk, uv = mat(p + "uq").view(H, D + T, a.q_rank), mat(p + "uk").view(H, D, R), mat(p + "uv").view(H, E, R)
+        q = uq.new_zeros(H, dk, a.q_rank)
+        q[:, :T], q[:, at:at + D] = uq[:, D:], uq[:, :D]
+        k = uk.new_zeros(H, R, d8)
+        k[:, :, :D] = uk.transpose(1, 2)
+        v = uv.new_zeros(H, ep, r8)
+        v[:, :E, :R] = uv
+        o = mat(p + "o").view(-1, H, E)
+        wo = o.new_zeros(o.shape[0], H, ep)
+        wo[:, :, :E] = o
+        dq = mat(p + "dq")
+        rows = [dq, dq.new_zeros(a.kv_col - a.q_rank, dq.shape[1])] + ([mat(p + "dkv")] if a.kv_from is None else [])
+        w = {"w_in": self._pad(torch.cat(rows)), "w_uq": self._pad(q.flatten(0, 1)), "w_uk": k, "w_uv": v,
+             "w_o": self._pad(wo.flatten(1)), "rot": self._rotary(a.rot), "q_norm": vec(p + "dq.norm"),
+             "kv_norm": vec(p + "dkv.norm") if a.kv_from is None else None}
+        if dv and self.dtype == torch.bfloat16:
+            kv = uk.new_zeros(H * (dk + dv), a.cache_row)
+            keys, values = kv[:H * dk].view(H, dk, -1), kv[H * dk:].view(H, dv, -1)
+            keys[:, at:at + D, :R], values[:, :E, :R] = uk, uv
+            for t in range(T):
+                keys[:, t, R + t] = 1.0
+            w["w_kv"] = ops.tile_weight(kv) if self.tile_weights else kv
+        return w
+
+    def _mlp_weights(self, f, p: str, mat) -> dict:
+        if f.kind == "moe":
+            return self._moe_weights(f, p, mat)
+        ip = round_up(f.ff, 64)
+        g, u = mat(p + "gate"), mat(p + "up")
+        if ip != f.ff:   # whole units of the interleaved layout; act(0) * 0 adds nothing
+            g, u = (torch.cat([t, t.new_zeros(ip - f.ff, t.shape[1])]) for t in (g, u))
+        gu = interleave32(g, u) if self.dtype == torch.bfloat16 else torch.cat([g, u])
+        return {"w_gu": self._pad(gu), "w_down": self._pad(mat(p + "down"))}
+
+    def _build_sandwich(self, mat, vec) -> None:
+        """Layers with a norm on either side of every sublayer; the layer scale is part of the second one's weight."""
+        self.k_cache, self.v_cache, self.states, self.sublayers, self.latents = [], [], [], [], {}
+        for i, L in enumerate(self.cfg.layers):
+            p = f"l{i}."
+            norms = [(vec(f"{p}norm{q}"), vec(f"{p}norm{q}b") * vec(f"{p}ls{q}")) for q in range(1, L.sublayers + 1)]
+            mixer = RUNS[L.mixer.kind](self, L.mixer, self._mixer_weights(L.mixer, p + "mix.", mat, vec))
+            if L.mixer.kind == "latent_attention":
+                self.latents[i] = mixer
+            self.sublayers.append(_NormedSublayer(*norms[0], mixer, i if L.mlp is None else -1))
+            if L.mlp is not None:
+                self.sublayers.append(_NormedSublayer(*norms[1], MLP_RUNS[L.mlp.kind](self, L.mlp, self._mlp_weights(L.mlp, p + "mlp.", mat)), i))
+        torch.cuda.empty_cache()
 
     def _build_parallel(self, get) -> None:
         """Layers whose mixer and feed-forward run side by side."""
@@ -512,8 +810,6 @@ class HybridModel(GemmShapes):
         for i, L in enumerate(self.cfg.layers):
             p, mx = f"l{i}.", L.mixer
             a = mx.left
-            if a.rot not in self._rots:
-                self._rots[a.rot] = hops.Rotary(a.rot, self.device)
             q = torch.cat([mat(f"{p}mix.left.{n}") for n in ("q", "k", "v")])
             ssd = self._ssd_weights(mx.right, p + "mix.right.", mat, vec)
             right = ssd.pop("in")
@@ -522,7 +818,7 @@ class HybridModel(GemmShapes):
             at = round_up(q.shape[0], 64)
             w_in[at:at + right.shape[0]] = right
             w = {"w_in": self._pad(w_in), "right": ssd,
-                 "left": {"rot": self._rots[a.rot], "q_norm": None, "k_norm": None, "w_o": self._pad(mat(p + "mix.left.o"))}}
+                 "left": {"rot": self._rotary(a.rot), "q_norm": None, "k_norm": None, "w_o": self._pad(mat(p + "mix.left.o"))}}
             mlp = MoeRun(self, L.mlp, self._moe_weights(L.mlp, p + "mlp.", mat)) if L.mlp is not None else None
             norms = [vec(p + "norm1")] + ([vec(p + "norm2")] if mlp is not None else [])
             out = (vec(p + "mix.left.out"), vec(p + "mix.right.out"))
@@ -538,10 +834,11 @@ class HybridModel(GemmShapes):
         vec = lambda name: get(name, True).contiguous()
         self.embed = mat("embed").contiguous()
         self.bigram = mat("bigram").contiguous() if cfg.bigram is not None else None
-        self.head = self._pad(mat("head"))
+        self.head = self._pad(mat("embed" if cfg.tie_embeddings else "head"))
         self.out_norm = vec("final.norm")
+        if self.sandwich:
+            return self._build_sandwich(mat, vec)
         one = torch.ones(1, dtype=torch.float32, device=self.device)
-        rots = self._rots
 
         def hc(p: str, q: int) -> dict:
             if not cfg.streams:
@@ -550,25 +847,12 @@ class HybridModel(GemmShapes):
 
         layers = []
         for i, L in enumerate(cfg.layers):
-            p, mx = f"l{i}.", L.mixer
-            names = ("q", "k", "v") if mx.kind == "attention" else ("q", "k", "v", "g")
-            if mx.rot not in rots:
-                rots[mx.rot] = hops.Rotary(mx.rot, self.device)
-            w = {"w_in": self._pad(torch.cat([mat(f"{p}mix.{n}") for n in names])), "w_o": self._pad(mat(p + "mix.o")),
-                 "rot": rots[mx.rot], "q_norm": None, "k_norm": None}
-            if mx.kind == "attention" and mx.qk_norm == "projection":
-                w["q_norm"], w["k_norm"] = vec(p + "mix.q.norm"), vec(p + "mix.k.norm")
-            if mx.kind == "retention":
-                w["decay_pow"] = hops.decay_powers(mx.decay, self.device)
+            p = f"l{i}."
+            w = self._mixer_weights(L.mixer, p + "mix.", mat, vec)
             subs = [(vec(p + "norm1"), hc(p, 1))]
             mw = None
             if L.mlp is not None:
-                ip = round_up(L.mlp.ff, 64)
-                g, u = mat(p + "mlp.gate"), mat(p + "mlp.up")
-                if ip != L.mlp.ff:   # whole units of the interleaved layout; act(0) * 0 adds nothing
-                    g, u = (torch.cat([t, t.new_zeros(ip - L.mlp.ff, t.shape[1])]) for t in (g, u))
-                gu = interleave32(g, u) if self.dtype == torch.bfloat16 else torch.cat([g, u])
-                mw = {"w_gu": self._pad(gu), "w_down": self._pad(mat(p + "mlp.down"))}
+                mw = self._mlp_weights(L.mlp, p + "mlp.", mat)
                 subs.append((vec(p + "norm2"), hc(p, 2)))
             layers.append((L, w, mw, subs))
         self.k_cache, self.v_cache, self.states, self.sublayers = [], [], [], []
@@ -655,6 +939,36 @@ class HybridModel(GemmShapes):
                 ops.gemm(h, w, out=out, **gc)
         return out
 
+    def product(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+        """out[:M] = x @ w^T in the model's dtype."""
+        M, k = x.shape
+        n = w.shape[0] * 128 if w.dim() == 4 else w.shape[0]
+        out = out[:M, :n]
+        if self.dtype == torch.float32:
+            hops.gemm_f32(x, w, out)
+        elif self.few_rows(M):
+            ops.gemv(x, w, out)
+        else:
+            ops.gemm(x, w, out=out, **self._gemm_shape(M, n, k, store=True))
+
+    def product_f32(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+        """out = x @ w^T in fp32, w row-major."""
+        M, k = x.shape
+        if self.dtype == torch.float32:
+            hops.gemm_f32(x, w, out)
+        elif self.few_rows(M):
+            ops.gemv(x, w, out)
+        else:
+            ops.gemm(x, w, out=out, epi=ops.EPI_STORE_F32, **self._gemm_shape(M, w.shape[0], k, store=True))
+
+    def per_head(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+        """out[h] = x[h] @ w[h]^T: x [heads, M, K] and out [heads, M, N] views of rows, w [heads, N, K]."""
+        if self.dtype == torch.float32:
+            for h in range(w.shape[0]):
+                hops.gemm_f32(x[h], w[h], out[h])
+        else:
+            ops.gemm(x, w, out=out, bn=128 if w.shape[0] * w.shape[1] >= 128 * self._sms else 64)
+
     def adds_up(self, M: int, k: int) -> bool:
         """Whether an output projection of K = k splits K and adds its parts into the accumulator (which then has
         to be zero); otherwise it stores."""
@@ -670,8 +984,11 @@ class HybridModel(GemmShapes):
             self.into_acc(x, w, self.branches[b])
 
     def into_acc(self, x: torch.Tensor, w: torch.Tensor, acc: Optional[torch.Tensor] = None) -> None:
-        """acc = x @ w^T (fp32). The accumulator is zero here: stream_norm clears what it has read."""
+        """acc = x @ w^T (fp32). The accumulator is zero here: stream_norm clears what it has read, branch_norm where
+        the next product adds its splits up."""
         M, k = x.shape
+        if acc is None and self.sandwich:
+            return self.into_branch(0, x, w)
         acc = (self.acc if acc is None else acc)[:M]
         if self.dtype == torch.float32:
             hops.gemm_f32(x, w, acc)
@@ -687,6 +1004,8 @@ class HybridModel(GemmShapes):
         logit rows than the buffer holds get one of their own)."""
         if self.parallel:
             return self._forward_parallel(s)
+        if self.sandwich:
+            return self._forward_sandwich(s)
         cfg, M = self.cfg, s.m
         h = self.h[:M]
         subs = self.sublayers
@@ -743,6 +1062,37 @@ class HybridModel(GemmShapes):
                 experts = layers[i].run(s, h, h2)
         return self._head(lm_h, logits, n_log)
 
+    def _forward_sandwich(self, s: StepInputs) -> torch.Tensor:
+        cfg, M, subs = self.cfg, s.m, self.sublayers
+        h = self.h[:M]
+        x = self.x.view(self.max_tokens, -1)
+        n_log = max(s.n_logits, 1)
+        lm_h, logits = self._logit_rows(n_log)
+        experts = self.gathered = None
+        for i in range(len(subs) + 1):
+            # what the sublayer before left, normed, into the residual; then the norm of this one (or of the head)
+            last = i == len(subs)
+            # the accumulator has to be zero when the next sublayer that adds its splits up in it starts
+            user = next((t.run.acc_k for t in subs[i:] if t.run.acc_k), 0)
+            clear = bool(user) and self.adds_up(M, user)
+            kw = dict(eps=cfg.rms_eps, w_offset=cfg.norm_weight_offset)
+            if i == 0:
+                kw.update(tokens=s.token_ids, embed=self.embed, embed_scale=cfg.emb_scale, branches=[(self.acc, None, 1.0, clear)])
+            elif subs[i - 1].run.acc_k:
+                kw["branches"] = [(self.acc, subs[i - 1].out, 1.0, clear)]
+            else:
+                kw.update(branches=[(None, subs[i - 1].out, 1.0, False)], experts=experts)
+            if last:
+                kw.update(norm_w=[self.out_norm], h=[lm_h], row_map=s.logit_map, store_x=self.layer_hook is not None)
+            else:
+                kw.update(norm_w=[subs[i].norm], h=[h], clear=self._proj_splits(M, subs[i]))
+            hops.branch_norm(x, M, **kw)
+            if self.layer_hook is not None and i > 0 and subs[i - 1].last_of >= 0:
+                self.layer_hook(subs[i - 1].last_of, x[:M])
+            if not last:
+                experts = subs[i].run(s, h)
+        return self._head(lm_h, logits, n_log)
+
     def _logit_rows(self, n_log: int) -> tuple:
         """Static buffers of the normed logit rows and the logits; larger ones for a step that has more of them."""
         if n_log <= self.max_logits:
@@ -786,3 +1136,4 @@ class HybridModel(GemmShapes):
         self._buffers.clear()
         self._moe.clear()
         self._scratch.clear()
+        self._rows.clear()

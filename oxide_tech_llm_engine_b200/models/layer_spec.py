@@ -60,7 +60,10 @@ class AttentionSpec:
     else the last `window` positions and the first `keep_first` ones of the sequence (which keep their
     true positions). `chunk` (instead of a window): only positions of the same chunk, counted from position
     0. `sink`: score of one more term of the softmax denominator that has no value. `qk_norm` "projection": RMS norm over all heads of q (of k) at once, before the
-    rotation."""
+    rotation. `bias`: q, k and v have biases. `temp_coef`: q is multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1)
+    at position p. `diff`: differential attention, every head has two maps over the same values (q and k hold
+    [map 1, map 2] head by head); with lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff the result is a1 - lambda a2 divided
+    by its root mean square, times 1 - diff."""
     heads: int
     kv_heads: int
     dim: int
@@ -72,8 +75,111 @@ class AttentionSpec:
     qk_norm: str = "none"      # none | projection
     chunk: int = 0
     sink: Optional[float] = None
+    bias: bool = False
+    temp_coef: float = 0.0
+    temp_every: float = 1.0
+    diff: Optional[float] = None
 
     kind = "attention"
+
+    @property
+    def parts(self) -> tuple:
+        return (self,)
+
+    @property
+    def maps(self) -> int:
+        return 1 if self.diff is None else 2
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def in_width(self) -> int:
+        return self.maps * self.heads * self.dim + self.cache_values
+
+    @property
+    def cache_values(self) -> int:
+        """Values that a token keeps in the cache."""
+        return self.kv_heads * (self.maps * self.dim + self.vdim)
+
+    def tensors(self, d: int) -> list[tuple[str, tuple[int, ...]]]:
+        rows = {"q": self.heads * self.maps * self.dim, "k": self.kv_heads * self.maps * self.dim, "v": self.kv_heads * self.vdim}
+        out = []
+        for n, r in rows.items():
+            out += [(n, (r, d))] + ([(n + ".b", (r,))] if self.bias else [])
+        if self.qk_norm == "projection":
+            out += [("q.norm", (self.heads * self.dim,)), ("k.norm", (self.kv_heads * self.dim,))]
+        if self.diff is not None:
+            out += [(n, (self.dim,)) for n in ("lq1", "lk1", "lq2", "lk2")]
+        return out + [("o", (d, self.out_dim))]
+
+
+@dataclass(frozen=True)
+class LatentSpec:
+    """Latent attention. Queries: W_uq of the normed W_dq h, per head `dim` values and, rotated, rot.dims more. A token
+    keeps the normed first `kv_rank` values of W_dkv h (the latent) and the rotated rest, one key part for all heads;
+    keys and values of a head are W_uk and W_uv of the latent. `kv_from`: the layer has no W_dkv and reads what that
+    layer keeps."""
+    heads: int
+    dim: int
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float
+    rot: Optional[RotarySpec] = None
+    kv_from: Optional[int] = None
+
+    kind = "latent_attention"
+
+    @property
+    def parts(self) -> tuple:
+        return (self,)
+
+    @property
+    def rot_dim(self) -> int:
+        return self.rot.dims if self.rot is not None else 0
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def kv_col(self) -> int:
+        """Column of the latent in the projection, behind the query latent."""
+        return (self.q_rank + 7) // 8 * 8
+
+    @property
+    def in_width(self) -> int:
+        return self.kv_col + (self.kv_rank + self.rot_dim if self.kv_from is None else 0)
+
+    @property
+    def cache_row(self) -> int:
+        return _pad16(self.kv_rank + self.rot_dim)
+
+    @property
+    def cache_values(self) -> int:
+        return self.kv_rank + self.rot_dim if self.kv_from is None else 0
+
+    def tensors(self, d: int) -> list[tuple[str, tuple[int, ...]]]:
+        h, r = self.heads, self.kv_rank
+        out = [("dq", (self.q_rank, d)), ("dq.norm", (self.q_rank,)), ("uq", (h * (self.dim + self.rot_dim), self.q_rank))]
+        if self.kv_from is None:
+            out += [("dkv", (r + self.rot_dim, d)), ("dkv.norm", (r,))]
+        return out + [("uk", (h * self.dim, r)), ("uv", (h * self.vdim, r)), ("o", (d, self.out_dim))]
+
+
+@dataclass(frozen=True)
+class MemorySpec:
+    """Matrix memory with exponential gates under a running maximum (mLSTM of xLSTM): see memory.cu for the recurrence. Gate
+    pre-activations are capped by cap tanh(z / cap); every head's output is divided by its root mean square, times `norm`,
+    times sigmoid(W_g h)."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+    kind = "mlstm"
 
     @property
     def parts(self) -> tuple:
@@ -83,12 +189,19 @@ class AttentionSpec:
     def out_dim(self) -> int:
         return self.heads * self.vdim
 
+    @property
+    def in_width(self) -> int:
+        return 2 * self.heads * (self.dim + self.vdim)
+
+    @property
+    def state_elems(self) -> int:
+        """fp32 values of one sequence's state: the memory, its normaliser and the running maximum."""
+        return self.heads * (self.dim * self.vdim + self.dim + 1)
+
     def tensors(self, d: int) -> list[tuple[str, tuple[int, ...]]]:
-        out = [("q", (self.heads * self.dim, d)), ("k", (self.kv_heads * self.dim, d)),
-               ("v", (self.kv_heads * self.vdim, d)), ("o", (d, self.out_dim))]
-        if self.qk_norm == "projection":
-            out += [("q.norm", (self.heads * self.dim,)), ("k.norm", (self.kv_heads * self.dim,))]
-        return out
+        h, hd, hv = self.heads, self.heads * self.dim, self.heads * self.vdim
+        return [("q", (hd, d)), ("k", (hd, d)), ("v", (hv, d)), ("g", (hv, d)), ("o", (d, hv)), ("norm", (hv,)), ("i", (h, d)),
+                ("i.b", (h,)), ("f", (h, d)), ("f.b", (h,))]
 
 
 @dataclass(frozen=True)
@@ -110,6 +223,10 @@ class RetentionSpec:
     @property
     def out_dim(self) -> int:
         return self.heads * self.vdim
+
+    @property
+    def in_width(self) -> int:
+        return 2 * self.heads * (self.dim + self.vdim)
 
     @property
     def state_elems(self) -> int:
@@ -217,18 +334,29 @@ class DenseMlpSpec:
 
 @dataclass(frozen=True)
 class MoeSpec:
-    """Mixture of `experts` feed-forwards W_down act(W_up h); a token uses the `top` ones with the largest scores
-    of a softmax over all experts, weighted by their scores divided by the scores' sum."""
+    """Mixture of `experts` feed-forwards W_down act(W_up h), or with `act` "silu_glu" W_down (silu(W_gate h) * (W_up h)).
+    A token uses the `top` ones with the largest scores. `scores` "softmax": over all experts, the weights are the chosen
+    scores divided by their sum; "sigmoid": the weights are the chosen scores. `groups` > 0: the experts form that many
+    equal groups of neighbours, and only those of the `keep` groups with the largest sum of two largest scores can be
+    chosen."""
     ff: int
     experts: int
     top: int
-    act: str = "relu2"         # square of relu
+    act: str = "relu2"         # relu2 (square of relu) | silu_glu
+    scores: str = "softmax"    # softmax | sigmoid
+    groups: int = 0
+    keep: int = 0
 
     kind = "moe"
+
+    @property
+    def glu(self) -> bool:
+        return self.act == "silu_glu"
 
     def tensors(self, d: int) -> list[tuple[str, tuple[int, ...]]]:
         out = []
         for e in range(self.experts):
+            out += [(f"e{e}.gate", (self.ff, d))] if self.glu else []
             out += [(f"e{e}.up", (self.ff, d)), (f"e{e}.down", (d, self.ff))]
         return out + [("router", (self.experts, d))]
 
@@ -236,10 +364,12 @@ class MoeSpec:
 @dataclass(frozen=True)
 class LayerSpec:
     """`parallel`: mixer and feed-forward read the same residual stream, each through its own norm, and both are
-    added to it; else the feed-forward follows the mixer."""
-    mixer: Union[AttentionSpec, RetentionSpec, SsdSpec, ParallelSpec]
+    added to it; else the feed-forward follows the mixer. `post_norm`: a sublayer's result passes a norm of its own
+    and an element-wise scale before it is added."""
+    mixer: Union[AttentionSpec, RetentionSpec, SsdSpec, ParallelSpec, LatentSpec, MemorySpec]
     mlp: Union[DenseMlpSpec, MoeSpec, None]
     parallel: bool = False
+    post_norm: bool = False
 
     @property
     def sublayers(self) -> int:
@@ -434,6 +564,105 @@ def povatar_json(cfg) -> dict[str, Any]:
             "embedding": {"scale": cfg.emb_scale}, "layers": layers}
 
 
+def gated_moe_from_json(c: dict) -> MoeSpec:
+    """Gated experts behind sigmoid scores, in groups where the router has them."""
+    r = c["router"]
+    g = r.get("groups") or {}
+    m = MoeSpec(int(c["expert"]["ff"]), int(r["experts"]), int(r["top"]), act="silu_glu", scores="sigmoid",
+                groups=int(g.get("count", 0)), keep=int(g.get("keep", 0)))
+    if m.groups and (m.experts % m.groups or not 1 <= m.keep <= m.groups):
+        raise ConfigError(f"{m.keep} of {m.groups} groups of {m.experts} experts")
+    if not 1 <= m.top <= (m.experts // m.groups * m.keep if m.groups else m.experts):
+        raise ConfigError(f"{m.top} of {m.experts} experts")
+    return m
+
+
+def zagolix_mixer(c: dict, kind: str):
+    n = lambda k: int(c[k])
+    if kind == "attention":
+        t = c.get("q_temp") or {}
+        a = AttentionSpec(n("heads"), n("kv_heads"), n("dim"), n("vdim"), float(c["scale"]), bias=True, diff=float(c["diff"]),
+                          temp_coef=float(t.get("coef", 0.0)), temp_every=float(t.get("every", 1.0)))
+        if a.heads % a.kv_heads:
+            raise ConfigError(f"{a.heads} query heads do not divide over {a.kv_heads} key/value heads")
+        return a
+    if kind == "latent_attention":
+        rot = rotary_from_json(c.get("rot"), True, n("rot_dim"))
+        if (rot.dims if rot else 0) != n("rot_dim"):
+            raise ConfigError(f"{c.get('rot')} does not rotate all of {n('rot_dim')} dimensions")
+        src = c.get("kv_from")
+        return LatentSpec(n("heads"), n("dim"), n("vdim"), n("q_rank"), n("kv_rank"), float(c["scale"]), rot,
+                          None if src is None else int(src))
+    if kind == "mlstm":
+        return MemorySpec(n("heads"), n("dim"), n("vdim"), float(c["gate_cap"]))
+    raise ConfigError(f"layer type {kind!r} is not part of this design")
+
+
+def zagolix_mlp(c: Optional[dict]):
+    if c is None:
+        return None
+    if c.get("kind") == "dense":
+        return DenseMlpSpec(int(c["ff"]), act="gelu_tanh")
+    if c.get("kind") == "moe":
+        return gated_moe_from_json(c)
+    raise ConfigError(f"feed-forward kind {c.get('kind')!r} is not part of this design")
+
+
+def zagolix_model(layers: tuple, *, width: int, vocab: int, eps: float, emb_scale: float, name: str = "zagolix"):
+    """ModelConfig of Zagolix layers. No tokenizer comes with the design, so there is no end-of-text id."""
+    from .config import ModelConfig
+
+    for i, L in enumerate(layers):
+        m, j = L.mixer, getattr(L.mixer, "kv_from", None)
+        if j is None:
+            continue
+        o = layers[j].mixer if 0 <= j < i else None
+        if not isinstance(o, LatentSpec) or o.kv_from is not None or (o.kv_rank, o.rot) != (m.kv_rank, m.rot):
+            raise ConfigError(f"layer {i} cannot read what layer {j} keeps")
+    any_m = layers[0].mixer
+    return ModelConfig(name=name, arch="zagolix", n_layers=len(layers), d_model=width, n_heads=any_m.heads,
+                       n_kv_heads=getattr(any_m, "kv_heads", any_m.heads), head_dim=any_m.dim,
+                       ffn_dim=max((L.mlp.ff for L in layers if L.mlp), default=0), vocab_size=vocab, max_ctx=1 << 20, rms_eps=eps,
+                       emb_scale=emb_scale, tie_embeddings=True, bos_id=-1, eos_id=-1, layers=layers)
+
+
+def zagolix_config(c: dict[str, Any]):
+    """ModelConfig of a Zagolix checkpoint from its config.json."""
+    layers = tuple(LayerSpec(zagolix_mixer(x["mixer"], x["type"]), zagolix_mlp(x.get("mlp")), post_norm=True) for x in c["layers"])
+    return zagolix_model(layers, width=int(c["width"]), vocab=int(c["vocab"]), eps=float(c["norm"]["eps"]),
+                         emb_scale=float((c.get("embedding") or {}).get("scale", 1.0)))
+
+
+def zagolix_json(cfg) -> dict[str, Any]:
+    """config.json of a Zagolix ModelConfig (inverse of zagolix_config)."""
+    layers = []
+    for L in cfg.layers:
+        m, f = L.mixer, L.mlp
+        c: dict[str, Any] = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim}
+        if m.kind == "attention":
+            c.update(kv_heads=m.kv_heads, scale=m.scale, diff=m.diff)
+            if m.temp_coef:
+                c["q_temp"] = {"coef": m.temp_coef, "every": m.temp_every}
+        elif m.kind == "latent_attention":
+            c.update(q_rank=m.q_rank, kv_rank=m.kv_rank, scale=m.scale, rot_dim=m.rot_dim)
+            if m.rot is not None:
+                c["rot"] = {"base": m.rot.base, "dims": m.rot.dims}
+            if m.kv_from is not None:
+                c["kv_from"] = m.kv_from
+        else:
+            c["gate_cap"] = m.gate_cap
+        mlp = None
+        if f is not None and f.kind == "dense":
+            mlp = {"kind": "dense", "ff": f.ff}
+        elif f is not None:
+            mlp = {"kind": "moe", "expert": {"ff": f.ff}, "router": {"experts": f.experts, "top": f.top}}
+            if f.groups:
+                mlp["router"]["groups"] = {"count": f.groups, "keep": f.keep}
+        layers.append({"type": m.kind, "mixer": c, "mlp": mlp})
+    return {"architecture": "Zagolix", "vocab": cfg.vocab_size, "width": cfg.d_model, "norm": {"eps": cfg.rms_eps},
+            "embedding": {"scale": cfg.emb_scale}, "layers": layers}
+
+
 def initial_vector(cfg, name: str, shape: tuple):
     """Starting values of a vector (synthetic weights): unit norms (stored as the distance from one where the design
     does so), step sizes of 0.001 to 0.1, decay rates of 1 to 16."""
@@ -445,7 +674,9 @@ def initial_vector(cfg, name: str, shape: tuple):
         v = np.log(np.expm1(10.0 ** (-3.0 + 2.0 * ramp)))
     elif name.endswith(".A_log"):
         v = np.log(1.0 + 15.0 * ramp)
-    elif name.endswith(".conv.b"):
+    elif name.endswith(".f.b"):
+        v = 3.0 + 3.0 * ramp      # forget gates that keep 20 to 400 tokens
+    elif name.endswith((".b", ".lq1", ".lk1", ".lq2", ".lk2")):
         v = np.zeros(n)
     elif name.endswith((".q.norm", ".k.norm", ".D")):
         v = np.ones(n)
@@ -464,10 +695,12 @@ def layer_list_tensors(cfg) -> list[tuple[str, tuple[int, ...]]]:
         p = f"l{i}."
         for q in range(1, L.sublayers + 1):
             out.append((p + f"norm{q}", (d,)))
+            if L.post_norm:
+                out += [(p + f"norm{q}b", (d,)), (p + f"ls{q}", (d,))]
             if s:
                 out += [(p + f"hc{q}.in", (s,)), (p + f"hc{q}.out", (s,)), (p + f"hc{q}.mix", (s, s))]
         out += [(p + "mix." + n, sh) for n, sh in L.mixer.tensors(d)]
         if L.mlp is not None:
             out += [(p + "mlp." + n, sh) for n, sh in L.mlp.tensors(d)]
-    out += [("final.norm", (d,)), ("head", (cfg.vocab_size, d))]
-    return out
+    out.append(("final.norm", (d,)))
+    return out if cfg.tie_embeddings else out + [("head", (cfg.vocab_size, d))]

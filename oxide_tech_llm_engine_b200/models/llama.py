@@ -73,6 +73,10 @@ class StepInputs:
     prev_ids: Optional[torch.Tensor] = None      # [M] int32: the token before it in its sequence or -1
     decode_slots: Optional[torch.Tensor] = None  # [n_decode] int32: recurrent-state slot of each decode row (-1 = padding)
     prefill_slots: Optional[torch.Tensor] = None  # [n_prefill] int32
+    # prompts whose whole context is laid out in plain rows: first row of every sequence, and the passes over them, each
+    # (first sequence, end, first tile, end, rows, pages of the longest sequence)
+    kv_start: Optional[torch.Tensor] = None       # [n_prefill] int32
+    kv_passes: tuple = ()
 
 
 class QuantLinear:

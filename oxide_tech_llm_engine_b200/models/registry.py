@@ -58,6 +58,12 @@ def _povatar_json(c: dict):
     return povatar_config(c)
 
 
+def _zagolix_json(c: dict):
+    from .layer_spec import zagolix_config
+
+    return zagolix_config(c)
+
+
 ARCHITECTURES: dict[str, Architecture] = {}
 
 
@@ -69,6 +75,7 @@ register(Architecture("llama", _llama, _llama_cpu))
 register(Architecture("mixtral", _llama, _llama_cpu))
 register(Architecture("kipolix", _hybrid, _hybrid_cpu, from_json=_kipolix_json, hf_names=False))
 register(Architecture("povatar", _hybrid, _hybrid_cpu, from_json=_povatar_json, hf_names=False))
+register(Architecture("zagolix", _hybrid, _hybrid_cpu, from_json=_zagolix_json, hf_names=False))
 
 
 def architecture(cfg) -> Architecture:

@@ -222,6 +222,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, *, out: Optional[torch.Tensor] = None
     """tcgen05 GEMM  out = a @ w^T  (bf16 in, fp32 accumulate). See csrc/kernels/gemm_bf16.cu.
     `mt` = 2 keeps 256 rows with one CTA per weight tile; `splits` > 1 with a store / SwiGLU / slab
     epilogue combines the split partial tiles inside the kernel (`fixup`, default on for those).
+    3-D operands without `group_counts` are groups of equally many rows.
     With `sfa` / `sfb` the operands are NVFP4: `a` and `w` hold e2m1 values packed two per byte
     ([.., K / 2] uint8, see quant_act_nvfp4 / Nvfp4Weight) and the product runs on the block-scaled
     fp4 tensor-core path (128 x 128 tiles); `a_gscale` [rows] and `w_gscale` [groups] multiply the rows."""
@@ -439,7 +440,7 @@ def paged_decode(q, k_cache, v_cache, block_tables, seq_lens, pages_per_split, p
                  *, batch: int, max_splits: int, window: int = 0, scale: float,
                  page_ml: Optional[torch.Tensor] = None, block_mass: Optional[torch.Tensor] = None,
                  q8=None, keep_first: int = 0, out_d: int = 0, exact_p: bool = False, chunk: int = 0,
-                 sink: float = float("-inf")) -> None:
+                 sink: float = float("-inf"), diff: Sequence[float] = ()) -> None:
     """Paged split-KV decode attention + merge. With `page_ml` [B, max_blocks, Hq, 2] and `block_mass`
     [B, max_blocks] (fp32) the kernels also produce the softmax probability mass per KV block, summed
     over heads: the heavy-hitter score of H2O pruning (the reference accumulates it in its decode
@@ -448,11 +449,12 @@ def paged_decode(q, k_cache, v_cache, block_tables, seq_lens, pages_per_split, p
     window, the first positions of the sequence stay visible. `out_d`: values stored per head when the
     heads are padded to D. `exact_p`: softmax weights enter the value product with 16 instead of 8 bits.
     `chunk`: instead of a window, only positions of the query's own chunk (counted from position 0) are
-    visible. `sink`: score of one more term of the softmax denominator, which has no value."""
+    visible. `sink`: score of one more term of the softmax denominator, which has no value. `diff` = (lambda, gain, eps):
+    query heads 2i and 2i + 1 are the two maps of differential attention, the merge writes their normed difference."""
     q8t, q8d, q8s = q8 if q8 is not None else (None, None, None)
     _ext().paged_decode(q, k_cache, v_cache, block_tables, seq_lens, pages_per_split, part_o, part_ml,
                         out, batch, max_splits, window, scale, status_word(q.device) if CHECK_BOUNDS else None,
-                        page_ml, block_mass, q8t, q8d, q8s, keep_first, out_d, exact_p, chunk, sink)
+                        page_ml, block_mass, q8t, q8d, q8s, keep_first, out_d, exact_p, chunk, sink, list(diff))
     _bump(3 if page_ml is not None else 2)
 
 

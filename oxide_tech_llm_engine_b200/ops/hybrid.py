@@ -1,4 +1,4 @@
-"""Python front-ends of the layer-list kernels (``csrc/kernels/{stream_ops,mixer_ops,attn_rows,retention,ssd,moe_ops}.cu``).
+"""Python front-ends of the layer-list kernels (``csrc/kernels/{stream_ops,mixer_ops,attn_rows,retention,ssd,moe_ops,latent,memory,attn_prefill_wide}.cu``).
 
 Activations, weights and caches are bf16, or fp32 throughout; residual streams, states, norms, scores
 and angles are fp32 in both cases. As in `ops`, nothing here falls back to PyTorch.
@@ -65,20 +65,108 @@ def stream_norm(x: torch.Tensor, rows: int, *, norm_w: torch.Tensor, eps: float,
 
 def heads(proj: torch.Tensor, m: int, *, h: int, g: int, d: int, e: int, rot: Rotary, positions, q_out, q_hd: int,
           q_norm=None, k_norm=None, eps: float = 1e-5, k_scale: float = 1.0, k_out=None, k_cache=None, v_cache=None,
-          slots=None) -> None:
+          slots=None, q_pd: int = 0, maps: int = 1, bias=None, temp_coef: float = 0.0, temp_every: float = 1.0) -> None:
     """Projection rows q | k | v -> normed and rotated heads; k and v into the paged cache with q [M, h * q_hd], or
-    q and k to dense fp32 buffers [heads, M, d] (HeadsParams)."""
+    q and k to dense fp32 buffers [heads, M, d]; g = 0: queries only, q_pd columns apart (HeadsParams)."""
     hybrid_ext().heads(proj, m, h, g, d, e, q_norm, k_norm, eps, rot.hi, rot.lo, rot.interleaved, rot.gain, positions,
-                       k_scale, q_out, q_hd, k_out, k_cache, v_cache, slots, ops.status_word(proj.device))
+                       k_scale, q_out, q_hd, k_out, k_cache, v_cache, slots, q_pd, maps, bias, temp_coef, temp_every,
+                       ops.status_word(proj.device))
     ops._bump()
+
+
+def diff_norm(a, m: int, *, h: int, e: int, lam: float, gain: float, eps: float, out) -> None:
+    """The two maps of every head (fp32, side by side) -> a1 - lam a2, divided by its root mean square, times gain."""
+    hybrid_ext().diff_norm(a, m, h, e, lam, gain, eps, out)
+    ops._bump()
+
+
+def latent_rows(proj, m: int, *, q_rank: int, q_norm, q_out, positions, eps: float, kv_col: int = 0, kv_rank: int = 0, kv_norm=None,
+                cache=None, slots=None, rot: Optional[Rotary] = None) -> None:
+    """Normed query latent of every row; with kv_rank > 0 also the normed latent and the rotated key part into the
+    paged cache [blocks, 1, 16, values] (LatentRowsParams)."""
+    r = rot if rot is not None else Rotary(None, proj.device)
+    hybrid_ext().latent_rows(proj, m, q_rank, q_norm, q_out, kv_col, kv_rank, kv_norm, cache, slots, r.hi, r.lo, r.interleaved,
+                             r.gain, positions, eps, ops.status_word(proj.device))
+    ops._bump()
+
+
+def latent_gather(cache, block_tables, ctx_lens, row0, *, seq0: int, n_seqs: int, max_pages: int, out) -> None:
+    """Cache rows of sequences seq0 .. in order of position, from row0[sequence] on."""
+    hybrid_ext().latent_gather(cache, block_tables, ctx_lens, row0, seq0, n_seqs, max_pages, out, ops.status_word(cache.device))
+    ops._bump()
+
+
+def latent_decode_ok(kv_rank: int, row: int) -> bool:
+    return bool(hybrid_ext().latent_decode_ok(kv_rank, row))
+
+
+def latent_decode(q, cache, block_tables, seq_lens, pages_per_split, part_o, part_ml, out, *, rows: int, kv_rank: int,
+                  max_splits: int, scale: float, o_hd: int) -> None:
+    """Decode rows of latent attention against the cached latents (split-KV and merge)."""
+    hybrid_ext().latent_decode(q, cache, block_tables, seq_lens, pages_per_split, rows, kv_rank, max_splits, scale, part_o, part_ml,
+                               out, o_hd, ops.status_word(q.device))
+    ops._bump(2)
+
+
+PREFILL_SIZES = ((64, 64), (128, 128), (192, 128), (256, 256))   # (keys, values) of prefill_rows and prefill_pages
+
+
+def prefill_size(dk: int, dv: int) -> Optional[tuple]:
+    """Smallest built head sizes that hold keys of dk and values of dv."""
+    return next((z for z in PREFILL_SIZES if z[0] >= dk and z[1] >= dv), None)
+
+
+def prefill_rows(q, kv, tile_seq, tile_q0, q_start, q_lens, ctx_lens, row0, out, *, dk: int, dv: int, g: int, n_tiles: int,
+                 scale: float, out_d: int) -> None:
+    """Causal attention of prompt tiles over plain rows of keys (g heads of dk columns) and values (behind them)."""
+    hybrid_ext().prefill_rows(q, kv, dk, dv, g * dk, g, row0, tile_seq, tile_q0, q_start, q_lens, ctx_lens, out, n_tiles, scale, out_d,
+                              ops.status_word(q.device))
+    ops._bump()
+
+
+def prefill_pages(q, k_cache, v_cache, block_tables, tile_seq, tile_q0, q_start, q_lens, ctx_lens, out, *, n_tiles: int, scale: float,
+                  out_d: int) -> None:
+    """Causal attention of prompt tiles over the paged cache, heads of up to 256 values."""
+    hybrid_ext().prefill_pages(q, k_cache, v_cache, block_tables, tile_seq, tile_q0, q_start, q_lens, ctx_lens, out, n_tiles, scale, out_d,
+                               ops.status_word(q.device))
+    ops._bump()
+
+
+def memory_chunk() -> int:
+    return int(hybrid_ext().MEMORY_CHUNK)
+
+
+def memory_chunks_ok(d: int, e: int) -> bool:
+    return bool(hybrid_ext().memory_chunks_ok(d, e))
+
+
+def memory_ws_elems(h: int, d: int, e: int, n_tiles: int) -> int:
+    return 2 * n_tiles * h * (d * e + d + 3)
+
+
+def memory_decode(proj, rows: int, *, h: int, d: int, e: int, z_bias, cap: float, eps: float, norm_w, state, state_m, row_slots,
+                  positions, out, z=None, hidden=None, z_w=None) -> None:
+    """Matrix memory, one token per row: gates (from pre-activations `z`, or from the rows and the gate weights), state
+    update, read-out, head norm and gate in one launch."""
+    hybrid_ext().memory_decode(proj, rows, h, d, e, z, hidden, z_w, z_bias, cap, eps, norm_w, state, state_m, row_slots, positions,
+                               out, ops.status_word(proj.device))
+    ops._bump()
+
+
+def memory_prefill(proj, m: int, *, h: int, d: int, e: int, z, z_bias, cap: float, eps: float, norm_w, state, state_m, seq_slots,
+                   tile_seq, tile_q0, q_start, q_lens, ctx_lens, n_tiles: int, n_seqs: int, ws, chunks: bool, out) -> None:
+    """Prompt chunks: the chunked tensor-core form, or token by token."""
+    hybrid_ext().memory_prefill(proj, m, h, d, e, z, z_bias, cap, eps, norm_w, state, state_m, seq_slots, tile_seq, tile_q0, q_start,
+                                q_lens, ctx_lens, n_tiles, n_seqs, ws, chunks, out, ops.status_word(proj.device))
+    ops._bump(3 if chunks else 2)
 
 
 def row_attention(q, q_hd: int, k_cache, v_cache, block_tables, *, n: int, h: int, d: int, e: int, window: int,
                   keep_first: int, scale: float, out, chunk: int = 0, sink: float = float("-inf"), seq_lens=None,
-                  tile_seq=None, tile_q0=None, q_start=None, q_lens=None, ctx_lens=None) -> None:
+                  tile_seq=None, tile_q0=None, q_start=None, q_lens=None, ctx_lens=None, o_hd: int = 0) -> None:
     """Softmax attention of any head size in fp32 FMAs: decode rows (seq_lens) or prompt tiles."""
     hybrid_ext().row_attention(q, q_hd, k_cache, v_cache, block_tables, seq_lens, tile_seq, tile_q0, q_start, q_lens,
-                               ctx_lens, n, h, d, e, window, keep_first, chunk, scale, sink, out, ops.status_word(q.device))
+                               ctx_lens, n, h, d, e, window, keep_first, chunk, scale, sink, out, o_hd, ops.status_word(q.device))
     ops._bump()
 
 
@@ -117,11 +205,15 @@ def max_experts() -> tuple[int, int]:
     return int(ext.MAX_EXPERTS), int(ext.MAX_TOP)
 
 
+def max_groups() -> int:
+    return int(hybrid_ext().MAX_GROUPS)
+
+
 def branch_norm(x: torch.Tensor, rows: int, *, norm_w, h, eps: float, w_offset: float = 0.0, tokens=None, embed=None,
                 embed_scale: float = 1.0, branches=(), experts=None, store_x: bool = True, row_map=None, clear=None) -> None:
     """Embedding or the sum of a layer's branches into the residual stream x [M, N], and its RMS norm with one weight per
     output (BranchNormParams in csrc/kernels/hybrid.cuh). `branches`: (fp32 rows, norm weight or None, gain, clear);
-    `experts`: (rows, slots, weights, chosen per row)."""
+    `experts`: (rows, slots, weights, chosen per row); a branch whose rows are None is their weighted sum."""
     rows_e, slot, weight, top = experts if experts is not None else (None, None, None, 0)
     hybrid_ext().branch_norm(x, rows, tokens, embed, embed_scale, [b[0] for b in branches], [b[1] for b in branches],
                              [b[2] for b in branches], [bool(b[3]) for b in branches], rows_e, slot, weight, top, store_x,
@@ -151,9 +243,11 @@ def gated_norm(y, z, m: int, *, h: int, e: int, ep: int, groups: int, w, eps: fl
     ops._bump()
 
 
-def moe_route(h, router, m: int, *, e: int, top: int, weight, expert, slot, mode: int = 0, logits=None, counts=None, xs=None) -> None:
+def moe_route(h, router, m: int, *, e: int, top: int, weight, expert, slot, mode: int = 0, logits=None, counts=None, xs=None,
+              softmax: bool = True, groups: int = 0, keep: int = 0) -> None:
     """Chosen experts, their weights and row slots (MoeRouteParams); logits from h and router unless given."""
-    hybrid_ext().moe_route(h, router, logits, m, e, top, weight, expert, slot, mode, counts, xs, ops.status_word(h.device))
+    hybrid_ext().moe_route(h, router, logits, m, e, top, weight, expert, slot, mode, counts, xs, softmax, groups, keep,
+                           ops.status_word(h.device))
     ops._bump()
 
 
