@@ -125,6 +125,10 @@ def main() -> None:
                     help="instead of the headline workload: layers with attention and a state-space mixer side by side and a mixture "
                          "of experts, beside the Mixtral-shaped model of equal size")
     ap.add_argument("--povatar-size", default="", help="only this size of --povatar")
+    ap.add_argument("--zagolix", action="store_true",
+                    help="instead of the headline workload: differential and latent attention, matrix memory and gated experts beside "
+                         "the Mixtral-shaped model of equal size")
+    ap.add_argument("--zagolix-size", default="", help="only this size of --zagolix")
     args = ap.parse_args()
     if args.kipolix and args.impl != "reference":
         from oxide_tech_llm_engine_b200.bench_hybrid import run
@@ -133,6 +137,11 @@ def main() -> None:
         return
     if args.povatar and args.impl != "reference":
         from oxide_tech_llm_engine_b200.bench_povatar import run
+
+        run(args, ClockSampler(0))
+        return
+    if args.zagolix and args.impl != "reference":
+        from oxide_tech_llm_engine_b200.bench_zagolix import run
 
         run(args, ClockSampler(0))
         return

@@ -687,7 +687,7 @@ void latent_gather(const Tensor& cache, const Tensor& block_tables, const Tensor
   check_launch(oxb::launch_latent_gather(p, cur_stream()), "latent_gather");
 }
 
-void latent_decode(const Tensor& q, const Tensor& cache, const Tensor& block_tables, const Tensor& seq_lens, const Tensor& pages_per_split,
+void latent_decode(const Tensor& q, const Tensor& cache, const Tensor& block_tables, const Tensor& seq_lens,
                    int64_t rows, int64_t R, int64_t max_splits, double scale, const Tensor& part_o, const Tensor& part_ml, const Tensor& out,
                    int64_t o_hd, const Tensor& status) {
   oxb::LatentDecodeParams p{};
@@ -699,16 +699,13 @@ void latent_decode(const Tensor& q, const Tensor& cache, const Tensor& block_tab
   p.H = static_cast<int>(q.size(1));
   p.R = static_cast<int>(R);
   p.rows = static_cast<int>(rows);
-  TORCH_CHECK(R >= 1 && R <= p.CP && oxb::latent_decode_ok(p.R, p.CP) && max_splits >= 1 && max_splits <= 64, "latent_decode: sizes");
-  TORCH_CHECK(reinterpret_cast<uintptr_t>(q.data_ptr()) % 16 == 0 && reinterpret_cast<uintptr_t>(cache.data_ptr()) % 16 == 0, "latent_decode: alignment");
-  p.q = reinterpret_cast<const __nv_bfloat16*>(q.data_ptr());
-  p.cache = reinterpret_cast<const __nv_bfloat16*>(cache.data_ptr());
+  const int hn = oxb::latent_decode_heads(p.H, p.R, p.CP);
+  TORCH_CHECK(R >= 1 && R <= p.CP && hn > 0 && max_splits >= 1 && max_splits <= 64, "latent_decode: sizes");
   p.num_blocks = static_cast<int>(cache.size(0));
   TORCH_CHECK(block_tables.dim() == 2 && block_tables.is_contiguous() && block_tables.size(0) >= rows, "latent_decode: block_tables");
   p.block_tables = i32(block_tables, 1, "latent_decode block_tables");
   p.max_blocks = static_cast<int>(block_tables.size(1));
   p.seq_lens = i32(seq_lens, rows, "latent_decode seq_lens");
-  p.pages_per_split = i32(pages_per_split, 1, "latent_decode pages_per_split");
   p.max_splits = static_cast<int>(max_splits);
   p.scale_log2 = static_cast<float>(scale * 1.4426950408889634);
   p.part_o = const_cast<float*>(f32(part_o, rows * p.H * max_splits * R, "latent_decode part_o"));
@@ -718,7 +715,12 @@ void latent_decode(const Tensor& q, const Tensor& cache, const Tensor& block_tab
   p.ldo = pitch(out, rows, (p.H - 1) * o_hd + R, "latent_decode out");
   p.out = reinterpret_cast<__nv_bfloat16*>(out.data_ptr());
   p.status = status_ptr(status);
-  check_launch(oxb::launch_latent_decode(p, cur_stream()), "latent_decode");
+  const auto bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+  const auto sw = CU_TENSOR_MAP_SWIZZLE_128B;
+  const uint64_t row = static_cast<uint64_t>(p.CP) * 2;
+  CUtensorMap tmQ = oxb::make_tma_map(q.data_ptr(), bf, 2, 3, p.CP, p.H, rows, row, row * p.H, 64, hn, 1, sw);
+  CUtensorMap tmC = oxb::make_tma_map(cache.data_ptr(), bf, 2, 2, p.CP, static_cast<uint64_t>(p.num_blocks) * 16, 1, row, 0, 64, 16, 1, sw);
+  check_launch(oxb::launch_latent_decode(tmQ, tmC, p, cur_stream()), "latent_decode");
 }
 
 // Causal attention of prompt tiles over plain rows of keys and values: kv [rows, columns], head g's keys from column
@@ -945,7 +947,9 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("latent_rows", &latent_rows);
   m.def("latent_gather", &latent_gather);
   m.def("latent_decode", &latent_decode);
-  m.def("latent_decode_ok", [](int64_t R, int64_t CP) { return oxb::latent_decode_ok(static_cast<int>(R), static_cast<int>(CP)); });
+  m.def("latent_decode_heads", [](int64_t H, int64_t R, int64_t CP) {
+    return oxb::latent_decode_heads(static_cast<int>(H), static_cast<int>(R), static_cast<int>(CP));
+  });
   m.def("prefill_rows", &prefill_rows);
   m.def("prefill_pages", &prefill_pages);
   m.def("prefill_wide_tile", [](int64_t dk, int64_t dv) { return oxb::prefill_wide_tile(static_cast<int>(dk), static_cast<int>(dv)); });

@@ -3,6 +3,7 @@
 // size, retention, and the 32-bit matrix product. `dtype` 0: activations, weights and caches are bf16;
 // 1: fp32 throughout. Scores, norms, states, residual streams and angles are fp32 in both.
 #pragma once
+#include <cuda.h>
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -319,12 +320,10 @@ cudaError_t launch_latent_gather(const LatentGatherParams& p, cudaStream_t strea
 // Decoding: all heads of a row against the latents themselves. q rows [H, CP]: the query's product with the key
 // expansion (R values), then its rotated part; the output is the weighted sum of latents, per head R values.
 struct LatentDecodeParams {
-  const __nv_bfloat16* q;   // [rows, H, CP]
-  const __nv_bfloat16* cache;
   const int* block_tables;  // [rows, max_blocks]
   const int* seq_lens;
-  const int* pages_per_split;
   int rows, H, R, CP, max_blocks, max_splits, num_blocks;
+  int n_splits;             // set by the launch: splits in use
   float scale_log2;
   float* part_o;            // [rows, H, max_splits, R]
   float* part_ml;           // [rows, H, max_splits, 2]
@@ -333,8 +332,10 @@ struct LatentDecodeParams {
   int o_hd;
   int* status;
 };
-cudaError_t launch_latent_decode(const LatentDecodeParams& p, cudaStream_t stream);
-bool latent_decode_ok(int R, int CP);
+// tmQ: [rows, H, CP] in boxes of latent_decode_heads(H, R, CP) x 64 (0: sizes that do not fit); tmC: cache rows in boxes of
+// 16 x 64.
+cudaError_t launch_latent_decode(const CUtensorMap& tmQ, const CUtensorMap& tmC, const LatentDecodeParams& p, cudaStream_t stream);
+int latent_decode_heads(int H, int R, int CP);
 
 // Matrix memory with a running maximum (mLSTM). Log gates per head: i = cap tanh(zi / cap), f = logsigmoid(cap tanh(zf / cap));
 //   m' = max(f + m, i), S' = exp(f + m - m') S + exp(i - m') k v^T, n' likewise with k alone, m starts at 0

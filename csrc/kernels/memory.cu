@@ -551,30 +551,33 @@ __global__ void __launch_bounds__(kChThreads, 2) memory_chunk_out_kernel(const M
         v[1][x] = d < D && c1 ? __ldcg(sp + 8) : 0.f;
       }
     };
-    float cur[2][4], nxt[2][4];
-    fetch(0, cur);
+    constexpr int kAhead = 4;   // steps whose values are on their way
+    float v[kAhead][2][4];
     const int steps = Dp / 16;
-    for (int k = 0; k < steps; ++k) {
-      if (k + 1 < steps) fetch(k + 1, nxt);
-      uint32_t b[2][2][3];
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        split3(cur[h][0], cur[h][1], b[h][0]);
-        split3(cur[h][2], cur[h][3], b[h][1]);
+    for (int j = 0; j < kAhead; ++j) fetch(j, v[j]);
+    for (int k0 = 0; k0 < steps; k0 += kAhead) {
+#pragma unroll
+      for (int j = 0; j < kAhead; ++j) {
+        const int k = k0 + j;
+        if (k >= steps) break;
+        uint32_t b[2][2][3];
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          split3(v[j][h][0], v[j][h][1], b[h][0]);
+          split3(v[j][h][2], v[j][h][3], b[h][1]);
+        }
+        fetch(k + kAhead, v[j]);
+        uint32_t a[4][4];
+#pragma unroll
+        for (int mi = 0; mi < 4; ++mi) ldsm4(aQ + (mi * 16 + row_a) * L.pitch + k * 32 + col_a, a[mi]);
+#pragma unroll
+        for (int x = 2; x >= 0; --x)
+#pragma unroll
+          for (int mi = 0; mi < 4; ++mi)
+#pragma unroll
+            for (int h = 0; h < 2; ++h) mma_bf16(Y[mi][h], a[mi], b[h][0][x], b[h][1][x]);
       }
-      uint32_t a[4][4];
-#pragma unroll
-      for (int mi = 0; mi < 4; ++mi) ldsm4(aQ + (mi * 16 + row_a) * L.pitch + k * 32 + col_a, a[mi]);
-#pragma unroll
-      for (int x = 2; x >= 0; --x)
-#pragma unroll
-        for (int mi = 0; mi < 4; ++mi)
-#pragma unroll
-          for (int h = 0; h < 2; ++h) mma_bf16(Y[mi][h], a[mi], b[h][0][x], b[h][1][x]);
-#pragma unroll
-      for (int h = 0; h < 2; ++h)
-#pragma unroll
-        for (int x = 0; x < 4; ++x) cur[h][x] = nxt[h][x];
     }
 #pragma unroll
     for (int mi = 0; mi < 4; ++mi) {

@@ -188,7 +188,7 @@ class LatentRun:
         self.acc_k = round_up(a.heads * self.ep, 64)
         bf16 = m.dtype == torch.bfloat16
         self.expand = bf16 and self.dv > 0                                    # prompts over expanded keys and values
-        self.tc = bf16 and hops.latent_decode_ok(a.kv_rank, self.cp)
+        self.tc = bf16 and hops.latent_decode_heads(a.heads, a.kv_rank, self.cp) > 0
         if a.kv_from is None:
             self.cache = torch.zeros(m.num_blocks, 1, 16, self.cp, dtype=m.dtype, device=m.device)
             m.k_cache.append(self.cache)
@@ -223,7 +223,7 @@ class LatentRun:
         heads = lambda t, width, lo, hi: t[:n, :H * width].view(n, H, width)[:, :, lo:hi].transpose(0, 1)
         m.per_head(heads(q, self.dk, self.at, self.at + self.d8), w["w_uk"], heads(qa, self.cp, 0, a.kv_rank))
         if self.tc:
-            hops.latent_decode(qa[:n].view(n, H, self.cp), self.cache, s.block_tables, s.seq_lens, s.pages_per_split, m.part_o,
+            hops.latent_decode(qa[:n].view(n, H, self.cp), self.cache, s.block_tables, s.seq_lens, m.part_o,
                                m.part_ml, ctx, rows=n, kv_rank=a.kv_rank, max_splits=m.max_splits, scale=a.scale, o_hd=self.r8)
         else:
             kw = dict(h=H, d=a.kv_rank + a.rot_dim, e=a.kv_rank, window=0, keep_first=0, scale=a.scale, out=ctx, o_hd=self.r8)
@@ -533,7 +533,7 @@ class HybridModel(GemmShapes):
         att = [p for L in cfg.layers for p in L.mixer.parts if p.kind == "attention"]
         lat = [p for L in cfg.layers for p in L.mixer.parts if p.kind == "latent_attention"]
         # CTAs per sequence and split of the decode attention
-        self.hkv = min([a.kv_heads for a in att] + [(a.heads + 31) // 32 for a in lat], default=1)
+        self.hkv = min([a.kv_heads for a in att] + [1 for _ in lat], default=1)
         self.x = torch.zeros(max_tokens, self.streams, d, dtype=torch.float32, device=dev)
         self.h = torch.zeros(max_tokens, self.dp, dtype=self.dtype, device=dev)
         n_acc = 2 if self.parallel else 1

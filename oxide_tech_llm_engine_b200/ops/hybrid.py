@@ -1,4 +1,4 @@
-"""Python front-ends of the layer-list kernels (``csrc/kernels/{stream_ops,mixer_ops,attn_rows,retention,ssd,moe_ops,latent,memory,attn_prefill_wide}.cu``).
+"""Python front-ends of the layer-list kernels (``csrc/kernels/{stream_ops,mixer_ops,attn_rows,retention,ssd,moe_ops,latent,latent_decode,memory,attn_prefill_wide}.cu``).
 
 Activations, weights and caches are bf16, or fp32 throughout; residual streams, states, norms, scores
 and angles are fp32 in both cases. As in `ops`, nothing here falls back to PyTorch.
@@ -96,14 +96,15 @@ def latent_gather(cache, block_tables, ctx_lens, row0, *, seq0: int, n_seqs: int
     ops._bump()
 
 
-def latent_decode_ok(kv_rank: int, row: int) -> bool:
-    return bool(hybrid_ext().latent_decode_ok(kv_rank, row))
+def latent_decode_heads(heads: int, kv_rank: int, row: int) -> int:
+    """Heads that one CTA of the decode kernel takes; 0: latents that it has no room for."""
+    return int(hybrid_ext().latent_decode_heads(heads, kv_rank, row))
 
 
-def latent_decode(q, cache, block_tables, seq_lens, pages_per_split, part_o, part_ml, out, *, rows: int, kv_rank: int,
+def latent_decode(q, cache, block_tables, seq_lens, part_o, part_ml, out, *, rows: int, kv_rank: int,
                   max_splits: int, scale: float, o_hd: int) -> None:
     """Decode rows of latent attention against the cached latents (split-KV and merge)."""
-    hybrid_ext().latent_decode(q, cache, block_tables, seq_lens, pages_per_split, rows, kv_rank, max_splits, scale, part_o, part_ml,
+    hybrid_ext().latent_decode(q, cache, block_tables, seq_lens, rows, kv_rank, max_splits, scale, part_o, part_ml,
                                out, o_hd, ops.status_word(q.device))
     ops._bump(2)
 
