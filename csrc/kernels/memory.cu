@@ -206,19 +206,47 @@ __device__ __forceinline__ ChunkPos chunk_pos(const MemoryParams& p, int chunk) 
   return {p.q_start[seq] + q0, left < C ? left : C, seq, q0};
 }
 
-// [C x W] values of the projection rows, as bf16, into shared memory; rows >= n and columns >= w_ok become zero.
+// [C x w] values of the projection rows, as bf16, into shared memory; rows >= n and columns >= w_ok become zero. w is a
+// multiple of 16. bf16 rows of whole 16-byte pieces go asynchronously (wait with cp_wait<0>); otherwise eight or four
+// pieces per thread are on their way together.
 template <typename P>
-__device__ __forceinline__ void tile_bf16(uint8_t* dst, int pitch, const P* src, long long ld, int n, int w, int w_ok, bool vec) {
-  if (vec) {
-    const int per = w >> 2;
-    for (int i = threadIdx.x; i < C * per; i += kChThreads) {
-      const int r = i / per, c = (i - r * per) * 4;
-      float v[4] = {0.f, 0.f, 0.f, 0.f};
-      if (r < n && c < w_ok) load4<P>(src + r * ld + c, v);
-      uint2 x;
-      x.x = pack_bf16x2(v[0], v[1]);
-      x.y = pack_bf16x2(v[2], v[3]);
-      *reinterpret_cast<uint2*>(dst + r * pitch + c * 2) = x;
+__device__ __forceinline__ void tile_bf16(uint8_t* dst, int pitch, const P* src, long long ld, int n, int w, int w_ok) {
+  const bool row16 = ((reinterpret_cast<uintptr_t>(src) | (ld * sizeof(P))) & 15) == 0;
+  if (sizeof(P) == 2 && row16 && w_ok % 8 == 0) {
+    const int per = w >> 3;
+    int r = threadIdx.x / per, c = threadIdx.x - r * per;
+    const int dr = kChThreads / per, dc = kChThreads - dr * per;
+    while (r < C) {
+      const bool in = r < n && c * 8 < w_ok;
+      cp_async16(smem_u32(dst) + r * pitch + c * 16, in ? src + r * ld + c * 8 : src, in);
+      r += dr;
+      c += dc;
+      if (c >= per) {
+        c -= per;
+        ++r;
+      }
+    }
+    cp_commit();
+  } else if (sizeof(P) == 4 && row16 && w_ok % 4 == 0) {
+    const int per = w >> 2, total = C * per;
+    for (int i0 = threadIdx.x; i0 < total; i0 += kChThreads * 8) {
+      float v[8][4];
+#pragma unroll
+      for (int k = 0; k < 8; ++k) {
+        const int i = i0 + k * kChThreads, r = i / per, c = (i - r * per) * 4;
+#pragma unroll
+        for (int x = 0; x < 4; ++x) v[k][x] = 0.f;
+        if (i < total && r < n && c < w_ok) load4<P>(src + r * ld + c, v[k]);
+      }
+#pragma unroll
+      for (int k = 0; k < 8; ++k) {
+        const int i = i0 + k * kChThreads, r = i / per, c = (i - r * per) * 4;
+        if (i >= total) break;
+        uint2 x;
+        x.x = pack_bf16x2(v[k][0], v[k][1]);
+        x.y = pack_bf16x2(v[k][2], v[k][3]);
+        *reinterpret_cast<uint2*>(dst + r * pitch + c * 2) = x;
+      }
     }
   } else {
     for (int i = threadIdx.x; i < C * w; i += kChThreads) {
@@ -279,9 +307,8 @@ __global__ void __launch_bounds__(kChThreads) memory_chunk_sum_kernel(const Memo
   uint8_t* sV = s_raw + C * pitch;
   const P* prow = static_cast<const P*>(p.proj) + cp.row0 * p.ld;
   const int k_col = (p.H + head) * D, v_col = 2 * p.H * D + head * E + e0;
-  const bool al = p.ld % 4 == 0 && (reinterpret_cast<uintptr_t>(p.proj) & 15) == 0;
-  tile_bf16<P>(sK, pitch, prow + k_col, p.ld, cp.n, Dp, D, al && D % 4 == 0 && k_col % 4 == 0);
-  tile_bf16<P>(sV, kPitchV, prow + v_col, p.ld, cp.n, ET, E - e0, al && E % 4 == 0 && v_col % 4 == 0);
+  tile_bf16<P>(sK, pitch, prow + k_col, p.ld, cp.n, Dp, D);
+  tile_bf16<P>(sV, kPitchV, prow + v_col, p.ld, cp.n, ET, min(ET, E - e0));
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   if (warp == 0) {
     float mx[2];
@@ -299,6 +326,7 @@ __global__ void __launch_bounds__(kChThreads) memory_chunk_sum_kernel(const Memo
       w[2] = a;
     }
   }
+  cp_wait<0>();
   __syncthreads();
   float* U = p.ws + (static_cast<long long>(chunk) * p.H + head) * state_size(p);
   if (blockIdx.z == 0)
@@ -434,13 +462,14 @@ __global__ void __launch_bounds__(256) memory_scan_chunks_kernel(const MemoryPar
 
 // 3. grid (chunks, H, column slices), cluster (1, 1, slices). Warp w owns columns 16 w .. of the slice, all 64 rows.
 struct OutSmem {
-  int pitch, k, v, w, total;
+  int pitch, k, v, w, n, total;
   __host__ __device__ explicit OutSmem(int D) {
     pitch = ((D + 15) & ~15) * 2 + 16;
     k = C * pitch;
     v = 2 * C * pitch;
     w = v + C * kPitchV;
-    total = w + 3 * C * kPitchW;
+    n = w + 3 * C * kPitchW;
+    total = n + ((D + 31) & ~31) * 4;
   }
 };
 template <typename P>
@@ -457,10 +486,12 @@ __global__ void __launch_bounds__(kChThreads, 2) memory_chunk_out_kernel(const M
   const OutSmem L(D);
   const P* prow = static_cast<const P*>(p.proj) + cp.row0 * p.ld;
   const int q_col = head * D, k_col = (p.H + head) * D, v_col = 2 * p.H * D + head * E + e0;
-  const bool al = p.ld % 4 == 0 && (reinterpret_cast<uintptr_t>(p.proj) & 15) == 0;
-  tile_bf16<P>(s_raw, L.pitch, prow + q_col, p.ld, cp.n, Dp, D, al && D % 4 == 0);
-  tile_bf16<P>(s_raw + L.k, L.pitch, prow + k_col, p.ld, cp.n, Dp, D, al && D % 4 == 0);
-  tile_bf16<P>(s_raw + L.v, kPitchV, prow + v_col, p.ld, cp.n, ET, E - e0, al && E % 4 == 0 && v_col % 4 == 0);
+  const float* S0 = p.ws + (static_cast<long long>(chunk) * p.H + head) * state_size(p);
+  float* s_n = reinterpret_cast<float*>(s_raw + L.n);
+  tile_bf16<P>(s_raw, L.pitch, prow + q_col, p.ld, cp.n, Dp, D);
+  tile_bf16<P>(s_raw + L.k, L.pitch, prow + k_col, p.ld, cp.n, Dp, D);
+  tile_bf16<P>(s_raw + L.v, kPitchV, prow + v_col, p.ld, cp.n, ET, min(ET, E - e0));
+  for (int d = threadIdx.x; d < ((D + 31) & ~31); d += kChThreads) s_n[d] = d < D ? S0[static_cast<long long>(D) * E + d] : 0.f;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   const float* wm = p.ws_m + (static_cast<long long>(chunk) * p.H + head) * 3;
   if (warp == 0) {
@@ -482,12 +513,12 @@ __global__ void __launch_bounds__(kChThreads, 2) memory_chunk_out_kernel(const M
     }
   }
   for (int i = threadIdx.x; i < C / 16 * C; i += kChThreads) (&s_sum[0][0])[i] = 0.f;
+  cp_wait<0>();
   __syncthreads();
   const uint32_t aQ = smem_u32(s_raw), aK = aQ + L.k, aV = aQ + L.v, aW = aQ + L.w;
   const int lr = lane & 7, lm = lane >> 3;
   const int row_a = (lm & 1) * 8 + lr, col_a = (lm >> 1) * 16;
   const int row_b = (lm >> 1) * 8 + lr, col_b = (lm & 1) * 16;
-  const float* S0 = p.ws + (static_cast<long long>(chunk) * p.H + head) * state_size(p);
   // ---- weighted scores: 16 x 16 blocks on and below the diagonal ----
   for (int it = warp; it < 10; it += kChWarps) {
     int mi = 0, nj = it;
@@ -496,6 +527,7 @@ __global__ void __launch_bounds__(kChThreads, 2) memory_chunk_out_kernel(const M
       ++mi;
     }
     float sc[2][4] = {};
+#pragma unroll 4
     for (int k = 0; k < Dp / 16; ++k) {
       uint32_t a[4], b[4];
       ldsm4(aQ + (mi * 16 + row_a) * L.pitch + k * 32 + col_a, a);
@@ -528,9 +560,18 @@ __global__ void __launch_bounds__(kChThreads, 2) memory_chunk_out_kernel(const M
   // ---- q n: four threads per row ----
   {
     const int r = threadIdx.x >> 2, part = threadIdx.x & 3;
-    const float* n0 = S0 + static_cast<long long>(D) * E;
     float a = 0.f;
-    for (int d = part; d < D; d += 4) a = fmaf(__bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(s_raw + r * L.pitch + d * 2)), n0[d], a);
+    for (int d = part * 8; d < Dp; d += 32) {
+      float x[8], y[4];
+      load4<__nv_bfloat16>(reinterpret_cast<const __nv_bfloat16*>(s_raw + r * L.pitch) + d, *reinterpret_cast<float(*)[4]>(x));
+      load4<__nv_bfloat16>(reinterpret_cast<const __nv_bfloat16*>(s_raw + r * L.pitch) + d + 4, *reinterpret_cast<float(*)[4]>(x + 4));
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        load4<float>(s_n + d + 4 * h, y);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) a = fmaf(x[4 * h + k], y[k], a);
+      }
+    }
     a += __shfl_xor_sync(0xffffffffu, a, 1);
     a += __shfl_xor_sync(0xffffffffu, a, 2);
     if (part == 0) s_qn[r] = a * p.scale;
@@ -608,7 +649,11 @@ __global__ void __launch_bounds__(kChThreads, 2) memory_chunk_out_kernel(const M
         }
     }
   }
-  // ---- normaliser, head norm over the value dimensions ----
+  // ---- normaliser; the rows wait in shared memory (where values and weights were) for their norm over all columns ----
+  __syncthreads();
+  constexpr int kPitchO = ET + 4;
+  float* s_o = reinterpret_cast<float*>(s_raw + L.v);
+  static_assert(C * kPitchO * 4 <= C * kPitchV + 3 * C * kPitchW, "rows fit where values and weights were");
 #pragma unroll
   for (int mi = 0; mi < 4; ++mi)
 #pragma unroll
@@ -618,12 +663,11 @@ __global__ void __launch_bounds__(kChThreads, 2) memory_chunk_out_kernel(const M
       const float inv = 1.f / (fmaxf(fabsf(nq), expf(-s_m[i])) + 1e-6f);
       float ss = 0.f;
 #pragma unroll
-      for (int h = 0; h < 2; ++h)
-#pragma unroll
-        for (int x = 0; x < 2; ++x) {
-          Y[mi][h][2 * r + x] *= inv;
-          ss = fmaf(Y[mi][h][2 * r + x], Y[mi][h][2 * r + x], ss);
-        }
+      for (int h = 0; h < 2; ++h) {
+        float2 o = make_float2(Y[mi][h][2 * r] * inv, Y[mi][h][2 * r + 1] * inv);
+        ss = fmaf(o.x, o.x, fmaf(o.y, o.y, ss));
+        *reinterpret_cast<float2*>(s_o + i * kPitchO + warp * 16 + h * 8 + 2 * t) = o;
+      }
       ss += __shfl_xor_sync(0xffffffffu, ss, 1);
       ss += __shfl_xor_sync(0xffffffffu, ss, 2);
       if (t == 0) s_ssq[warp][i] = ss;
@@ -641,33 +685,49 @@ __global__ void __launch_bounds__(kChThreads, 2) memory_chunk_out_kernel(const M
     if (threadIdx.x < C) {
       float a = 0.f;
       for (unsigned x = 0; x < gridDim.z; ++x) a += cl.map_shared_rank(s_part, x)[threadIdx.x];
-      s_sum[0][threadIdx.x] = a;
+      s_qn[threadIdx.x] = 1.f / sqrtf(a / static_cast<float>(E) + p.eps);
     }
     cl.sync();  // nobody leaves while a neighbour still reads its part
   } else {
     __syncthreads();
-    if (threadIdx.x < C) s_sum[0][threadIdx.x] = s_part[threadIdx.x];
+    if (threadIdx.x < C) s_qn[threadIdx.x] = 1.f / sqrtf(s_part[threadIdx.x] / static_cast<float>(E) + p.eps);
     __syncthreads();
   }
-  if (!active) return;
-  const P* grow = prow + 2 * p.H * D + p.H * E + head * E;
-  const float* nw = p.norm_w + head * E;
-  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + cp.row0 * p.ldo + head * E;
+  const P* grow = prow + 2 * p.H * D + p.H * E + head * E + e0;
+  const float* nw = p.norm_w + head * E + e0;
+  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + cp.row0 * p.ldo + head * E + e0;
+  const int cols = min(ET, E - e0);
+  if (cols % 4 == 0 && E % 4 == 0 && D % 2 == 0 && p.ld % 4 == 0 && p.ldo % 4 == 0 && (reinterpret_cast<uintptr_t>(p.proj) & 15) == 0) {
+    // four columns per thread, a warp per row: gate, weight and output in whole runs
+    const int e = lane * 4;
+    if (e < cols) {
+      float w4[4];
+      load4<float>(nw + e, w4);
 #pragma unroll
-  for (int mi = 0; mi < 4; ++mi)
+      for (int i0 = 0; i0 < C; i0 += kChWarps * 4) {
+        float gt[4][4];
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      const int i = mi * 16 + g + r * 8;
-      if (i >= cp.n) continue;
-      const float rr = 1.f / sqrtf(s_sum[0][i] / static_cast<float>(E) + p.eps);
-#pragma unroll
-      for (int h = 0; h < 2; ++h)
-#pragma unroll
-        for (int x = 0; x < 2; ++x) {
-          const int e = ec + h * 8 + 2 * t + x;
-          if (e < E) out[i * p.ldo + e] = __float2bfloat16(Y[mi][h][2 * r + x] * rr * nw[e] * sigmoid_f(to_f(grow[i * p.ld + e])));
+        for (int k = 0; k < 4; ++k) {
+          const int i = i0 + k * kChWarps + warp;
+          if (i < cp.n) load4<P>(grow + i * p.ld + e, gt[k]);
         }
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const int i = i0 + k * kChWarps + warp;
+          if (i >= cp.n) continue;
+          float o[4];
+          load4<float>(s_o + i * kPitchO + e, o);
+#pragma unroll
+          for (int x = 0; x < 4; ++x) o[x] *= s_qn[i] * w4[x] * sigmoid_f(gt[k][x]);
+          store4<__nv_bfloat16>(out + i * p.ldo + e, o);
+        }
+      }
     }
+  } else {
+    for (int i = warp; i < cp.n; i += kChWarps)
+      for (int e = lane; e < cols; e += 32)
+        out[i * p.ldo + e] = __float2bfloat16(s_o[i * kPitchO + e] * s_qn[i] * nw[e] * sigmoid_f(to_f(grow[i * p.ld + e])));
+  }
 }
 
 // ------------------------------------------------------------------------------------------------

@@ -222,16 +222,15 @@ class LatentRun:
                        q_pd=self.dk)
         heads = lambda t, width, lo, hi: t[:n, :H * width].view(n, H, width)[:, :, lo:hi].transpose(0, 1)
         m.per_head(heads(q, self.dk, self.at, self.at + self.d8), w["w_uk"], heads(qa, self.cp, 0, a.kv_rank))
-        if self.tc:
-            hops.latent_decode(qa[:n].view(n, H, self.cp), self.cache, s.block_tables, s.seq_lens, m.part_o,
-                               m.part_ml, ctx, rows=n, kv_rank=a.kv_rank, max_splits=m.max_splits, scale=a.scale, o_hd=self.r8)
-        else:
-            kw = dict(h=H, d=a.kv_rank + a.rot_dim, e=a.kv_rank, window=0, keep_first=0, scale=a.scale, out=ctx, o_hd=self.r8)
-            if nd > 0:
-                hops.row_attention(qa, self.cp, self.cache, self.cache, s.block_tables, n=nd, seq_lens=s.seq_lens, **kw)
-            if s.n_prefill > 0:
-                hops.row_attention(qa, self.cp, self.cache, self.cache, s.prefill_block_tables, n=s.n_tiles, tile_seq=s.tile_seq,
-                                   tile_q0=s.tile_q0, q_start=s.q_start, q_lens=s.q_lens, ctx_lens=s.ctx_lens, **kw)
+        kw = dict(h=H, d=a.kv_rank + a.rot_dim, e=a.kv_rank, window=0, keep_first=0, scale=a.scale, out=ctx, o_hd=self.r8)
+        if nd > 0 and self.tc:
+            hops.latent_decode(qa[:nd].view(nd, H, self.cp), self.cache, s.block_tables, s.seq_lens, m.part_o, m.part_ml, ctx, rows=nd,
+                               kv_rank=a.kv_rank, max_splits=m.max_splits, scale=a.scale, o_hd=self.r8)
+        elif nd > 0:
+            hops.row_attention(qa, self.cp, self.cache, self.cache, s.block_tables, n=nd, seq_lens=s.seq_lens, **kw)
+        if n > nd:       # prompts that are not expanded
+            hops.row_attention(qa, self.cp, self.cache, self.cache, s.prefill_block_tables, n=s.n_tiles, tile_seq=s.tile_seq,
+                               tile_q0=s.tile_q0, q_start=s.q_start, q_lens=s.q_lens, ctx_lens=s.ctx_lens, **kw)
         m.per_head(heads(ctx, self.r8, 0, self.r8), w["w_uv"], heads(o, self.ep, 0, self.ep))
 
     def _expanded(self, s: StepInputs, q: torch.Tensor, o: torch.Tensor) -> None:
