@@ -182,8 +182,8 @@ cudaError_t launch_t(const StreamNormParams& p, cudaStream_t stream) {
   return launch_s<T, kMaxStreams>(p, stream);
 }
 
-// Layers whose mixer and feed-forward run side by side: four values per piece, CH pieces per thread, which stay
-// in registers.
+// Layers whose mixer and feed-forward run side by side, or one after the other with a norm on either side: four values
+// per piece, CH pieces per thread, which stay in registers; NB: branches that it can add.
 // The chosen experts' rows of a token wait in shared memory as (row, weight): a row outside the buffer weighs nothing.
 struct ChosenRow {
   int row;
@@ -231,8 +231,8 @@ __device__ __forceinline__ float2 block_sum2(float2 v, float2* scratch) {
   return make_float2(warp_sum(s.x), warp_sum(s.y));
 }
 
-template <typename T, int CH>
-__global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchNormParams p) {
+template <typename T, int CH, int NB, int THREADS, int CTAS>
+__global__ void __launch_bounds__(THREADS, CTAS) branch_norm_kernel(const BranchNormParams p) {
   __shared__ float s_red[32];
   __shared__ float2 s_red2[32];
   __shared__ ChosenRow s_chosen[2][kMaxTop];   // of this row and of the CTA's next one
@@ -271,13 +271,13 @@ __global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchNormParam
           for (int j = 0; j < 4; ++j) x[k][j] *= p.embed_scale;
         }
       }
-      for (int b = 0; b < kMaxBranches; ++b)
+      for (int b = 0; b < NB; ++b)
         if (b < p.n_branches && p.clear_y[b])
           for (int c = threadIdx.x * 4; c < N; c += blockDim.x * 4)
             *reinterpret_cast<float4*>(p.y[b] + static_cast<long long>(row) * p.ldy + c) = make_float4(0.f, 0.f, 0.f, 0.f);
     } else {
-      float y[kMaxBranches][CH][4];
-      float ss[kMaxBranches] = {};
+      float y[NB][CH][4];
+      float ss[NB] = {};
 #pragma unroll
       for (int k = 0; k < CH; ++k) {
         const int c = (k * blockDim.x + threadIdx.x) * 4;
@@ -288,7 +288,7 @@ __global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchNormParam
           if (e_plain) expert_sum4<T>(p, s_chosen[parity], c, x[k]);
         }
 #pragma unroll
-        for (int b = 0; b < kMaxBranches; ++b) {
+        for (int b = 0; b < NB; ++b) {
 #pragma unroll
           for (int j = 0; j < 4; ++j) y[b][k][j] = 0.f;
           if (b < p.n_branches && c < N) {
@@ -301,15 +301,15 @@ __global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchNormParam
       }
       // (the barriers of the sums and of the norm below publish the next row's table)
       if (p.e_rows != nullptr && row + gridDim.x < p.rows) chosen_rows(p, row + gridDim.x, s_chosen[parity ^ 1]);
-      const float2 tot = block_sum2(make_float2(ss[0], ss[1]), s_red2);
-      const float r[kMaxBranches] = {1.f / sqrtf(tot.x * inv_n + p.eps), 1.f / sqrtf(tot.y * inv_n + p.eps)};
+      const float2 tot = block_sum2(make_float2(ss[0], NB > 1 ? ss[NB - 1] : 0.f), s_red2);
+      const float r[2] = {1.f / sqrtf(tot.x * inv_n + p.eps), 1.f / sqrtf(tot.y * inv_n + p.eps)};
 #pragma unroll
       for (int k = 0; k < CH; ++k) {
         const int c = (k * blockDim.x + threadIdx.x) * 4;
         if (c >= N) continue;
         float a[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-        for (int b = 0; b < kMaxBranches; ++b)
+        for (int b = 0; b < NB; ++b)
           if (b < p.n_branches) {
             float w[4] = {1.f, 1.f, 1.f, 1.f};
             if (p.w[b] != nullptr) load4<float>(p.w[b] + c, w);
@@ -435,9 +435,15 @@ cudaError_t launch_branch(const BranchNormParams& p, cudaStream_t stream) {
   const bool vec = p.N % 4 == 0 && p.ldy % 4 == 0 && p.ldh % 4 == 0 && p.lde % 4 == 0;
   const int quads = (p.N + 3) / 4;
   auto threads = [&](int ch) { return dim3(((quads + ch - 1) / ch + 31) / 32 * 32); };
-  // one piece per thread: whole rows in flight, as many warps as the row has (measured against two and four pieces)
-  if (vec && quads <= 1024) return launch_kernel(branch_norm_kernel<T, 1>, grid, threads(1), 0, stream, true, false, p);
-  if (vec && quads <= 2048) return launch_kernel(branch_norm_kernel<T, 2>, grid, threads(2), 0, stream, true, false, p);
+  if (vec && p.n_branches <= 1 && quads <= 1024) {
+    // many rows: four CTAs of an SM in different phases of their rows
+    if (p.rows > 2 * sm_count())
+      return launch_kernel(branch_norm_kernel<T, 2, 1, 512, 4>, grid, threads(2), 0, stream, true, false, p);
+    return launch_kernel(branch_norm_kernel<T, 1, 1, 1024, 1>, grid, threads(1), 0, stream, true, false, p);
+  }
+  // two branches: one piece per thread, as many warps as the row has (measured against two and four pieces)
+  if (vec && quads <= 1024) return launch_kernel(branch_norm_kernel<T, 1, 2, 1024, 1>, grid, threads(1), 0, stream, true, false, p);
+  if (vec && quads <= 2048) return launch_kernel(branch_norm_kernel<T, 2, 2, 1024, 1>, grid, threads(2), 0, stream, true, false, p);
   const size_t smem = static_cast<size_t>(p.N) * sizeof(float);
   ensure_dynamic_smem(branch_norm_any_kernel<T>, smem);
   return launch_kernel(branch_norm_any_kernel<T>, grid, dim3(256), smem, stream, true, false, p);

@@ -108,11 +108,12 @@ class AttentionSpec:
         out = []
         for n, r in rows.items():
             out += [(n, (r, d))] + ([(n + ".b", (r,))] if self.bias else [])
-        if self.qk_norm == "projection":
-            out += [("q.norm", (self.heads * self.dim,)), ("k.norm", (self.kv_heads * self.dim,))]
         if self.diff is not None:
             out += [(n, (self.dim,)) for n in ("lq1", "lk1", "lq2", "lk2")]
-        return out + [("o", (d, self.out_dim))]
+        out.append(("o", (d, self.out_dim)))
+        if self.qk_norm == "projection":
+            out += [("q.norm", (self.heads * self.dim,)), ("k.norm", (self.kv_heads * self.dim,))]
+        return out
 
 
 @dataclass(frozen=True)

@@ -47,7 +47,7 @@ def chunk(n, ctx):
 
 # ---------------------------------------------------------------- norms on either side
 @pytest.mark.parametrize("dtype,tol", [(torch.float32, 3e-6), (torch.bfloat16, 6e-3)])
-@pytest.mark.parametrize("N,rows,top", [(64, 3, 2), (200, 700, 3), (76, 5, 1), (2048, 330, 6), (4096, 4, 2), (9000, 2, 3)])
+@pytest.mark.parametrize("N,rows,top", [(64, 3, 2), (200, 700, 3), (76, 5, 1), (2048, 330, 6), (4096, 300, 2), (4096, 4, 2), (9000, 2, 3)])
 def test_the_norm_of_the_weighted_expert_rows(H, N, rows, top, dtype, tol):
     g = gen(N + rows)
     ld, eps = (N + 63) // 64 * 64, 1e-3
@@ -258,14 +258,15 @@ def test_decoding_against_latents_in_batches_of_unequal_lengths(H, heads, R, T_)
                 assert rel(got[i], latent_want(q[i, :, :R + T_], rows[i], R, scale)) < 6e-3, (splits, n)
 
 
-def test_standing_out_latents_and_growing_scores(H):
+@pytest.mark.parametrize("heads,R,T_", [(5, 96, 16), (20, 512, 64), (33, 256, 32)])
+def test_standing_out_latents_and_growing_scores(H, heads, R, T_):
     """One position that takes nearly everything, at page, tile and split borders; then scores that rise tile after tile by far
     more than the reference's slack, and fall again."""
-    heads, R, T_, n = 5, 96, 16, 400
+    n = 400
     cache, bt, rows, CP = latent_cache([n], R, T_, 5, 0.1)
     q = torch.zeros(1, heads, CP)
     q[0, :, :R + T_] = b16(torch.randn(heads, R + T_, generator=gen(1)))
-    for j in (0, 1, 15, 16, 63, 64, 65, 127, 128, 191, 192, 255, 256, 398, 399):
+    for j in (0, 1, 15, 16, 63, 64, 65, 127, 128, 129, 191, 192, 255, 256, 383, 384, 398, 399):
         c, z = cache.clone(), rows[0].clone()
         z[j] = b16(q[0, 2, :R + T_])
         c[int(bt[0, j // 16]), 0, j % 16, :R + T_] = z[j]
