@@ -319,6 +319,13 @@ void gemm_packed(const Tensor& a, const Tensor& qw, int64_t qtype, int64_t N, co
 // ---------------------------------------------------------------------------------------------
 // attention
 // ---------------------------------------------------------------------------------------------
+// one fp32 score per query head, or nullptr
+const float* sinks_ptr(const c10::optional<Tensor>& t, int heads) {
+  if (!t.has_value() || !t->defined()) return nullptr;
+  TORCH_CHECK(t->is_cuda() && t->scalar_type() == torch::kFloat32 && t->is_contiguous() && t->numel() >= heads, "sinks: fp32, one per query head");
+  return t->data_ptr<float>();
+}
+
 void paged_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
                   const Tensor& block_tables, const Tensor& seq_lens, const Tensor& pages_per_split,
                   const Tensor& part_o, const Tensor& part_ml, const Tensor& out, int64_t batch,
@@ -326,7 +333,8 @@ void paged_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
                   const c10::optional<Tensor>& status, const c10::optional<Tensor>& page_ml,
                   const c10::optional<Tensor>& block_mass, const c10::optional<Tensor>& q8,
                   const c10::optional<Tensor>& q8_d, const c10::optional<Tensor>& q8_s, int64_t keep_first, int64_t out_d,
-                  bool exact_p, int64_t chunk, double sink, const std::vector<double>& diff) {
+                  bool exact_p, int64_t chunk, double sink, const std::vector<double>& diff, const c10::optional<Tensor>& sinks,
+                  double out_gain) {
   TORCH_CHECK(q.dim() == 3 && k_cache.dim() == 4, "paged_decode: q [B,Hq,D], cache [blk,Hkv,16,D]");
   TORCH_CHECK(k_cache.size(2) == 16, "paged_decode: 16-token pages");
   oxb::DecodeAttnParams p{};
@@ -360,6 +368,9 @@ void paged_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache,
   TORCH_CHECK(chunk >= 0 && (chunk == 0 || (window == 0 && keep_first == 0)), "paged_decode: a window or a chunk");
   p.chunk = static_cast<int>(chunk);
   p.sink_log2 = static_cast<float>(sink * 1.4426950408889634);
+  p.sinks = sinks_ptr(sinks, p.Hq);
+  p.out_gain = static_cast<float>(out_gain);
+  TORCH_CHECK(p.sinks == nullptr || (diff.empty() && !page_ml.has_value()), "paged_decode: sinks go with the plain maps");
   if (!diff.empty()) {
     TORCH_CHECK(diff.size() == 3 && p.Hq % 2 == 0 && !page_ml.has_value() && !q8.has_value() && !std::isfinite(sink),
                 "paged_decode: diff is (lambda, gain, eps) over pairs of query heads");
@@ -402,7 +413,8 @@ void paged_prefill_tc(const Tensor& q, const Tensor& k_cache, const Tensor& v_ca
                       const Tensor& block_tables, const Tensor& tile_seq, const Tensor& tile_q0,
                       const Tensor& q_start, const Tensor& q_lens, const Tensor& ctx_lens,
                       const Tensor& out, int64_t n_tiles, int64_t window, double scale,
-                      const Tensor& status, int64_t keep_first, int64_t out_d, bool exact_p, int64_t chunk, double sink) {
+                      const Tensor& status, int64_t keep_first, int64_t out_d, bool exact_p, int64_t chunk, double sink,
+                      const c10::optional<Tensor>& sinks, double out_gain) {
   TORCH_CHECK(q.dim() == 3 && k_cache.dim() == 4, "paged_prefill_tc: q [T,Hq,D], cache [blk,Hkv,16,D]");
   TORCH_CHECK(k_cache.is_contiguous() && v_cache.is_contiguous(), "paged_prefill_tc: contiguous caches");
   oxb::PrefillAttnParams p{};
@@ -433,6 +445,8 @@ void paged_prefill_tc(const Tensor& q, const Tensor& k_cache, const Tensor& v_ca
   TORCH_CHECK(chunk >= 0 && (chunk == 0 || (window == 0 && keep_first == 0)), "paged_prefill_tc: a window or a chunk");
   p.chunk = static_cast<int>(chunk);
   p.sink_log2 = static_cast<float>(sink * 1.4426950408889634);
+  p.sinks = sinks_ptr(sinks, p.Hq);
+  p.out_gain = static_cast<float>(out_gain);
   p.scale_log2 = static_cast<float>(scale * 1.4426950408889634);
   const uint64_t T = q.size(0);
   const uint64_t kv_rows = static_cast<uint64_t>(k_cache.size(0)) * p.Hkv * 16;

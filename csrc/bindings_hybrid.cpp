@@ -131,7 +131,7 @@ void heads(const Tensor& proj, int64_t M, int64_t H, int64_t G, int64_t D, int64
            const OptTensor& k_norm, double eps, const OptTensor& freq_hi, const OptTensor& freq_lo, bool interleaved,
            double gain, const Tensor& positions, double k_scale, const Tensor& q_out, int64_t q_hd, const OptTensor& k_out,
            const OptTensor& k_cache, const OptTensor& v_cache, const OptTensor& slots, int64_t q_pd, int64_t maps, const OptTensor& bias,
-           double t_coef, double t_every, const Tensor& status) {
+           double t_coef, double t_every, const OptTensor& k_rms, const Tensor& status) {
   oxb::HeadsParams p{};
   // storage type: that of the caches; dense q and k are fp32 whatever the projection is
   const int proj_dt = dtype_code(proj, "heads proj");
@@ -150,7 +150,7 @@ void heads(const Tensor& proj, int64_t M, int64_t H, int64_t G, int64_t D, int64
   p.E = static_cast<int>(E);
   p.q_norm = f32(q_norm, H * D, "heads q_norm");
   p.k_norm = f32(k_norm, G * D, "heads k_norm");
-  TORCH_CHECK((p.q_norm == nullptr) == (p.k_norm == nullptr), "heads: q and k norm go together");
+  TORCH_CHECK((p.q_norm == nullptr) == (p.k_norm == nullptr) || (given(k_rms) && p.k_norm == nullptr), "heads: q and k norm go together");
   p.eps = static_cast<float>(eps);
   TORCH_CHECK(p.q_norm == nullptr || (q_pd == D && !given(bias)), "heads: the norm spans packed heads without bias");
   p.bias = f32(bias, H * q_pd + G * D + G / maps * E, "heads bias");
@@ -185,18 +185,25 @@ void heads(const Tensor& proj, int64_t M, int64_t H, int64_t G, int64_t D, int64
       check_launch(oxb::launch_heads(p, dt, cur_stream()), "heads");
       return;
     }
-    TORCH_CHECK(given(k_cache) && given(v_cache) && given(slots), "heads: caches and slots, or k_out");
-    TORCH_CHECK(q_out.scalar_type() == k_cache->scalar_type() && v_cache->scalar_type() == k_cache->scalar_type(),
-                "heads: one storage type");
-    TORCH_CHECK(k_cache->dim() == 4 && v_cache->dim() == 4 && k_cache->is_contiguous() && v_cache->is_contiguous() &&
-                    k_cache->size(1) == G / maps && v_cache->size(1) == G / maps && k_cache->size(2) == 16 && v_cache->size(2) == 16 &&
-                    k_cache->size(0) == v_cache->size(0) && k_cache->size(3) >= maps * D && v_cache->size(3) >= E,
+    TORCH_CHECK(given(k_cache) && given(v_cache) != given(k_rms) && given(slots), "heads: caches and slots, or k_out");
+    TORCH_CHECK(q_out.scalar_type() == k_cache->scalar_type(), "heads: one storage type");
+    TORCH_CHECK(k_cache->dim() == 4 && k_cache->is_contiguous() && k_cache->size(1) == G / maps && k_cache->size(2) == 16 &&
+                    k_cache->size(3) >= maps * D,
                 "heads: caches [blocks, G, 16, >= head size]");
-    p.ld = pitch(proj, M, H * q_pd + G * D + G / maps * E, "heads proj");
     p.k_cache = k_cache->data_ptr();
-    p.v_cache = v_cache->data_ptr();
     p.DP = static_cast<int>(k_cache->size(3));
-    p.EP = static_cast<int>(v_cache->size(3));
+    if (given(k_rms)) {   // keys that are values: no value columns, no value cache
+      TORCH_CHECK(p.q_norm != nullptr && p.k_norm == nullptr && maps == 1 && k_scale == 1.0, "heads: keys that are values, with a norm");
+      p.k_rms = const_cast<float*>(f32(*k_rms, k_cache->size(0) * 16, "heads k_rms"));
+      p.ld = pitch(proj, M, H * q_pd + G * D, "heads proj");
+    } else {
+      TORCH_CHECK(v_cache->scalar_type() == k_cache->scalar_type() && v_cache->dim() == 4 && v_cache->is_contiguous() &&
+                      v_cache->size(1) == G / maps && v_cache->size(2) == 16 && k_cache->size(0) == v_cache->size(0) && v_cache->size(3) >= E,
+                  "heads: caches [blocks, G, 16, >= head size]");
+      p.ld = pitch(proj, M, H * q_pd + G * D + G / maps * E, "heads proj");
+      p.v_cache = v_cache->data_ptr();
+      p.EP = static_cast<int>(v_cache->size(3));
+    }
     TORCH_CHECK(slots->is_cuda() && slots->scalar_type() == torch::kInt64 && slots->numel() >= M, "heads: slots int64");
     p.slots = reinterpret_cast<const long long*>(slots->data_ptr<int64_t>());
     p.num_slots = k_cache->size(0) * 16;
@@ -208,7 +215,8 @@ void heads(const Tensor& proj, int64_t M, int64_t H, int64_t G, int64_t D, int64
 void row_attention(const Tensor& q, int64_t q_hd, const Tensor& k_cache, const Tensor& v_cache, const Tensor& block_tables,
                    const OptTensor& seq_lens, const OptTensor& tile_seq, const OptTensor& tile_q0, const OptTensor& q_start,
                    const OptTensor& q_lens, const OptTensor& ctx_lens, int64_t n, int64_t H, int64_t D, int64_t E, int64_t window,
-                   int64_t keep_first, int64_t chunk, double scale, double sink, const Tensor& out, int64_t o_hd, const Tensor& status) {
+                   int64_t keep_first, int64_t chunk, double scale, double sink, const OptTensor& sinks, double out_gain, const Tensor& out, int64_t o_hd,
+                   const Tensor& status) {
   oxb::RowAttnParams p{};
   const int dt = dtype_code(q, "row_attention q");
   TORCH_CHECK(k_cache.dim() == 4 && v_cache.dim() == 4 && k_cache.is_contiguous() && v_cache.is_contiguous() &&
@@ -252,6 +260,8 @@ void row_attention(const Tensor& q, int64_t q_hd, const Tensor& k_cache, const T
   p.chunk = static_cast<int>(chunk);
   p.scale = static_cast<float>(scale);
   p.sink = static_cast<float>(sink);
+  p.sinks = f32(sinks, H, "row_attention sinks");
+  p.out_gain = static_cast<float>(out_gain);
   if (o_hd == 0) o_hd = E;
   TORCH_CHECK(o_hd >= E, "row_attention: o_hd");
   p.o_hd = static_cast<int>(o_hd);
@@ -333,15 +343,17 @@ void branch_norm(const Tensor& x, int64_t rows, const OptTensor& tokens, const O
                  const std::vector<OptTensor>& ys, const std::vector<OptTensor>& ws, const std::vector<double>& gains,
                  const std::vector<bool>& clears, const OptTensor& e_rows, const OptTensor& e_slot, const OptTensor& e_weight,
                  int64_t top, bool store_x, const std::vector<Tensor>& norm_ws, const std::vector<Tensor>& hs, double eps,
-                 double w_offset, const OptTensor& row_map, const OptTensor& clear, const Tensor& status) {
+                 double w_offset, const OptTensor& row_map, const OptTensor& clear, const OptTensor& base, const OptTensor& split,
+                 int64_t split_off, const OptTensor& x0_tokens, const Tensor& status) {
   TORCH_CHECK(x.dim() == 2, "branch_norm: x [rows, N]");
   oxb::BranchNormParams p{};
   p.rows = static_cast<int>(rows);
   p.N = static_cast<int>(x.size(1));
   TORCH_CHECK(x.size(0) >= rows && p.N <= 32768, "branch_norm: rows of at most 32768 values");
   p.x = const_cast<float*>(f32(x, rows * p.N, "branch_norm x"));
-  TORCH_CHECK(!hs.empty() && hs.size() <= 2 && hs.size() == norm_ws.size(), "branch_norm: one or two outputs");
-  const int dt = dtype_code(hs[0], "branch_norm h");
+  TORCH_CHECK(hs.size() <= 2 && hs.size() == norm_ws.size() && hs.empty() == given(split), "branch_norm: one or two outputs, or split rows");
+  const Tensor& like = hs.empty() ? *split : hs[0];   // of the storage type
+  const int dt = dtype_code(like, "branch_norm h");
   p.n_out = static_cast<int>(hs.size());
   for (size_t o = 0; o < hs.size(); ++o) {
     TORCH_CHECK(hs[o].scalar_type() == hs[0].scalar_type(), "branch_norm: one storage type");
@@ -370,8 +382,8 @@ void branch_norm(const Tensor& x, int64_t rows, const OptTensor& tokens, const O
     p.clear_y[b] = clears[b] ? 1 : 0;
   }
   if (given(tokens)) {
-    TORCH_CHECK(given(embed) && embed->scalar_type() == hs[0].scalar_type() && embed->is_contiguous() && embed->dim() == 2 &&
-                    embed->size(1) == p.N && !given(e_rows),
+    TORCH_CHECK(given(embed) && embed->scalar_type() == like.scalar_type() && embed->is_contiguous() && embed->dim() == 2 &&
+                    embed->size(1) == p.N && !given(e_rows) && !given(base),
                 "branch_norm: embed [vocab, N] of h's type");
     p.tokens = i32(*tokens, rows, "branch_norm tokens");
     p.embed = embed->data_ptr();
@@ -381,7 +393,7 @@ void branch_norm(const Tensor& x, int64_t rows, const OptTensor& tokens, const O
     TORCH_CHECK(!ys.empty(), "branch_norm: tokens or branches");
   }
   if (given(e_rows)) {
-    TORCH_CHECK(given(e_slot) && given(e_weight) && top >= 1 && top <= oxb::kMaxTop && e_rows->scalar_type() == hs[0].scalar_type() && e_rows->is_cuda(),
+    TORCH_CHECK(given(e_slot) && given(e_weight) && top >= 1 && top <= oxb::kMaxTop && e_rows->scalar_type() == like.scalar_type() && e_rows->is_cuda(),
                 "branch_norm: expert rows of h's type, with slots and weights");
     p.lde = pitch(*e_rows, 1, p.N, "branch_norm expert rows");
     p.n_e_rows = e_rows->size(0);
@@ -389,6 +401,19 @@ void branch_norm(const Tensor& x, int64_t rows, const OptTensor& tokens, const O
     p.e_slot = i32(*e_slot, rows * top, "branch_norm slots");
     p.e_weight = f32(*e_weight, rows * top, "branch_norm weights");
     p.top = static_cast<int>(top);
+  }
+  p.base = f32(base, p.N, "branch_norm base");
+  if (given(split)) {
+    TORCH_CHECK(given(x0_tokens) && given(embed) && embed->scalar_type() == like.scalar_type() && embed->is_contiguous() && embed->dim() == 2 &&
+                    embed->size(1) == p.N && !given(row_map) && split_off >= p.N,
+                "branch_norm: split rows take the embedding and its tokens");
+    p.ld_split = pitch(*split, rows, (dt == 0 ? 2 : 1) * split_off + p.N, "branch_norm split");
+    p.split = split->data_ptr();
+    p.split_off = static_cast<int>(split_off);
+    p.x0_tokens = i32(*x0_tokens, rows, "branch_norm x0_tokens");
+    p.embed = embed->data_ptr();
+    p.vocab = static_cast<int>(embed->size(0));
+    p.embed_scale = static_cast<float>(embed_scale);
   }
   p.store_x = store_x ? 1 : 0;
   p.eps = static_cast<float>(eps);
@@ -897,6 +922,132 @@ void memory_prefill(const Tensor& proj, int64_t M, int64_t H, int64_t D, int64_t
   }
 }
 
+// Talking heads: decode rows (seq_lens) or prompt tiles; rows: the kernel for any sizes
+oxb::TalkParams talk_common(const Tensor& q, const Tensor& cache, const Tensor& k_rms, const Tensor& block_tables, int64_t n, int64_t H,
+                            int64_t D, int64_t window, double scale, double cap, const Tensor& talk, const Tensor& bias, const Tensor& gate,
+                            const Tensor& out, const Tensor& status) {
+  oxb::TalkParams p{};
+  const int dt = dtype_code(q, "talk q");
+  TORCH_CHECK(cache.dim() == 4 && cache.is_contiguous() && cache.size(2) == 16 && cache.scalar_type() == q.scalar_type() &&
+                  out.scalar_type() == q.scalar_type(),
+              "talk: cache [blocks, G, 16, head size], one storage type");
+  p.H = static_cast<int>(H);
+  p.G = static_cast<int>(cache.size(1));
+  p.D = static_cast<int>(D);
+  p.DP = static_cast<int>(cache.size(3));
+  TORCH_CHECK(H >= 1 && H % p.G == 0 && D >= 1 && D <= p.DP && window >= 0, "talk: head sizes");
+  p.q = q.data_ptr();
+  p.q_ld = pitch(q, 1, H * p.DP, "talk q");
+  TORCH_CHECK(dt == 1 || p.q_ld % 8 == 0, "talk: q rows in whole 16-byte pieces");
+  p.cache = cache.data_ptr();
+  p.k_rms = f32(k_rms, cache.size(0) * 16, "talk k_rms");
+  p.num_blocks = static_cast<int>(cache.size(0));
+  TORCH_CHECK(block_tables.dim() == 2, "talk: block_tables");
+  p.block_tables = i32(block_tables, 1, "talk block_tables");
+  p.max_blocks = static_cast<int>(block_tables.size(1));
+  p.n_rows = static_cast<int>(n);
+  p.window = static_cast<int>(window);
+  p.scale = static_cast<float>(scale);
+  p.cap = static_cast<float>(cap);
+  p.talk = f32(talk, H * H, "talk matrix");
+  TORCH_CHECK(bias.dim() == 2 && bias.size(0) == H && bias.size(1) >= 1, "talk: bias [H, distances]");
+  p.bias = f32(bias, H, "talk bias");
+  p.n_bias = static_cast<int>(bias.size(1));
+  TORCH_CHECK(window == 0 ? bias.size(1) >= 16 * block_tables.size(1) : bias.size(1) >= window, "talk: a bias for every visible distance");
+  p.gate_f32 = dtype_code(gate, "talk gate");
+  p.gate = gate.data_ptr();
+  p.gate_ld = pitch(gate, 1, H * D, "talk gate");
+  p.ldo = pitch(out, 1, H * D, "talk out");
+  p.out = out.data_ptr();
+  p.status = status_ptr(status);
+  return p;
+}
+
+void talk_decode(const Tensor& q, const Tensor& cache, const Tensor& k_rms, const Tensor& block_tables, const Tensor& seq_lens,
+                 const OptTensor& pages_per_split, int64_t rows, int64_t H, int64_t D, int64_t window, double scale, double cap,
+                 const Tensor& talk, const Tensor& bias, const Tensor& gate, const OptTensor& part_o, const OptTensor& part_ml,
+                 int64_t max_splits, const Tensor& out, const Tensor& status) {
+  oxb::TalkParams p = talk_common(q, cache, k_rms, block_tables, rows, H, D, window, scale, cap, talk, bias, gate, out, status);
+  TORCH_CHECK(block_tables.size(0) >= rows && q.size(0) >= rows && out.size(0) >= rows && gate.size(0) >= rows, "talk_decode: rows");
+  p.seq_lens = i32(seq_lens, rows, "talk_decode seq_lens");
+  if (!given(part_o)) {
+    check_launch(oxb::launch_talk_rows(p, dtype_code(q, "talk q"), cur_stream()), "talk_rows");
+    return;
+  }
+  TORCH_CHECK(dtype_code(q, "talk q") == 0 && oxb::talk_decode_ok(p.H, p.G, p.DP) && given(pages_per_split) && given(part_ml) && max_splits >= 1,
+              "talk_decode: sizes");
+  p.pages_per_split = i32(*pages_per_split, 1, "talk_decode pages_per_split");
+  p.part_o = const_cast<float*>(f32(*part_o, rows * H * max_splits * p.DP, "talk_decode part_o"));
+  p.part_ml = const_cast<float*>(f32(*part_ml, rows * H * max_splits * 2, "talk_decode part_ml"));
+  p.max_splits = static_cast<int>(max_splits);
+  check_launch(oxb::launch_talk_decode(p, cur_stream()), "talk_decode");
+}
+
+void talk_prefill(const Tensor& q, const Tensor& cache, const Tensor& k_rms, const Tensor& block_tables, const Tensor& tile_seq,
+                  const Tensor& tile_q0, const Tensor& q_start, const Tensor& q_lens, const Tensor& ctx_lens, int64_t n_tiles, int64_t H,
+                  int64_t D, int64_t window, double scale, double cap, const Tensor& talk, const Tensor& bias, const Tensor& gate,
+                  const OptTensor& scores, int64_t span, const Tensor& out, const Tensor& status) {
+  oxb::TalkParams p = talk_common(q, cache, k_rms, block_tables, n_tiles, H, D, window, scale, cap, talk, bias, gate, out, status);
+  p.tile_seq = i32(tile_seq, n_tiles, "talk_prefill tile_seq");
+  p.tile_q0 = i32(tile_q0, n_tiles, "talk_prefill tile_q0");
+  p.q_start = i32(q_start, 1, "talk_prefill q_start");
+  p.q_lens = i32(q_lens, 1, "talk_prefill q_lens");
+  p.ctx_lens = i32(ctx_lens, 1, "talk_prefill ctx_lens");
+  if (!given(scores)) {
+    check_launch(oxb::launch_talk_rows(p, dtype_code(q, "talk q"), cur_stream()), "talk_rows");
+    return;
+  }
+  TORCH_CHECK(dtype_code(q, "talk q") == 0 && oxb::talk_prefill_ok(p.H, p.DP) && span > 0 && span % 32 == 0, "talk_prefill: sizes");
+  p.scores = const_cast<float*>(f32(*scores, n_tiles * H * 128 * span, "talk_prefill scores"));
+  p.span = static_cast<int>(span);
+  check_launch(oxb::launch_talk_prefill(p, cur_stream()), "talk_prefill");
+}
+
+oxb::GruParams gru_common(const Tensor& proj, int64_t M, const Tensor& bias, double out_gain, const Tensor& state, const Tensor& out,
+                          const Tensor& status) {
+  oxb::GruParams p{};
+  TORCH_CHECK(state.dim() == 2 && state.size(1) % 4 == 0, "gru: state [slots, N], N a multiple of 4");
+  p.N = static_cast<int>(state.size(1));
+  p.state = const_cast<float*>(f32(state, 1, "gru state"));
+  p.num_slots = static_cast<int>(state.size(0));
+  p.ld = pitch(proj, M, 3 * p.N, "gru proj");
+  p.proj = proj.data_ptr();
+  p.proj_f32 = dtype_code(proj, "gru proj");
+  TORCH_CHECK(dtype_code(out, "gru out") == 0 || p.proj_f32 == 1, "gru: fp32 rows take fp32 projections");
+  p.bias = f32(bias, 2 * p.N, "gru bias");
+  p.out_gain = static_cast<float>(out_gain);
+  p.ldo = pitch(out, M, p.N, "gru out");
+  p.out = out.data_ptr();
+  TORCH_CHECK(p.ld % 4 == 0 && p.ldo % 4 == 0 && reinterpret_cast<uintptr_t>(p.proj) % 16 == 0 && reinterpret_cast<uintptr_t>(p.out) % 8 == 0,
+              "gru: rows in whole pieces of four values");
+  p.status = status_ptr(status);
+  return p;
+}
+
+void gru_decode(const Tensor& proj, int64_t rows, const Tensor& bias, double out_gain, const Tensor& state, const Tensor& row_slots,
+                const Tensor& positions, const Tensor& out, const Tensor& status) {
+  oxb::GruParams p = gru_common(proj, rows, bias, out_gain, state, out, status);
+  p.row_slots = i32(row_slots, rows, "gru_decode row_slots");
+  p.positions = i32(positions, rows, "gru_decode positions");
+  p.rows = static_cast<int>(rows);
+  check_launch(oxb::launch_gru_decode(p, dtype_code(out, "gru out"), cur_stream()), "gru_decode");
+}
+
+void gru_prefill(const Tensor& proj, int64_t M, const Tensor& bias, double out_gain, const Tensor& state, const Tensor& seq_slots,
+                 const Tensor& tile_seq, const Tensor& tile_q0, const Tensor& q_start, const Tensor& q_lens, const Tensor& ctx_lens,
+                 int64_t n_tiles, const Tensor& ws, const Tensor& out, const Tensor& status) {
+  oxb::GruParams p = gru_common(proj, M, bias, out_gain, state, out, status);
+  p.seq_slots = i32(seq_slots, 1, "gru_prefill seq_slots");
+  p.tile_seq = i32(tile_seq, n_tiles, "gru_prefill tile_seq");
+  p.tile_q0 = i32(tile_q0, n_tiles, "gru_prefill tile_q0");
+  p.q_start = i32(q_start, 1, "gru_prefill q_start");
+  p.q_lens = i32(q_lens, 1, "gru_prefill q_lens");
+  p.ctx_lens = i32(ctx_lens, 1, "gru_prefill ctx_lens");
+  p.n_tiles = static_cast<int>(n_tiles);
+  p.ws = const_cast<float*>(f32(ws, n_tiles * (1 + oxb::kGruParts) * 2 * p.N, "gru_prefill ws"));
+  check_launch(oxb::launch_gru_prefill(p, dtype_code(out, "gru out"), cur_stream()), "gru_prefill");
+}
+
 void gemm_f32(const Tensor& a, const Tensor& w, const Tensor& out) {
   TORCH_CHECK(a.is_cuda() && w.is_cuda() && out.is_cuda() && a.scalar_type() == torch::kFloat32 &&
                   w.scalar_type() == torch::kFloat32 && out.scalar_type() == torch::kFloat32 && a.dim() == 2 && w.dim() == 2 &&
@@ -911,7 +1062,7 @@ void gemm_f32(const Tensor& a, const Tensor& w, const Tensor& out) {
 
 void glu_f32(const Tensor& gu, const Tensor& out, int64_t M, int64_t I, int64_t act) {
   TORCH_CHECK(gu.is_cuda() && gu.scalar_type() == torch::kFloat32 && out.scalar_type() == torch::kFloat32, "glu_f32: fp32");
-  const int64_t ldg = pitch(gu, M, 2 * I, "glu_f32 gu"), ldo = pitch(out, M, I, "glu_f32 out");
+  const int64_t ldg = pitch(gu, M, act == 2 ? I : 2 * I, "glu_f32 gu"), ldo = pitch(out, M, I, "glu_f32 out");
   check_launch(oxb::launch_glu_f32(gu.data_ptr<float>(), ldg, out.data_ptr<float>(), ldo, static_cast<int>(M),
                                    static_cast<int>(I), static_cast<int>(act), cur_stream()),
                "glu_f32");
@@ -958,6 +1109,14 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("memory_chunks_ok", [](int64_t D, int64_t E) { return oxb::memory_chunks_ok(static_cast<int>(D), static_cast<int>(E)); });
   m.attr("MEMORY_CHUNK") = oxb::kMemChunk;
   m.attr("MAX_GROUPS") = oxb::kMaxGroups;
+  m.def("talk_decode", &talk_decode);
+  m.def("talk_prefill", &talk_prefill);
+  m.def("talk_decode_ok", [](int64_t H, int64_t G, int64_t DP) { return oxb::talk_decode_ok(static_cast<int>(H), static_cast<int>(G), static_cast<int>(DP)); });
+  m.def("talk_prefill_ok", [](int64_t H, int64_t DP) { return oxb::talk_prefill_ok(static_cast<int>(H), static_cast<int>(DP)); });
+  m.def("talk_span", [](int64_t window, int64_t max_ctx) { return oxb::talk_span(static_cast<int>(window), static_cast<int>(max_ctx)); });
+  m.def("gru_decode", &gru_decode);
+  m.def("gru_prefill", &gru_prefill);
+  m.attr("GRU_PARTS") = oxb::kGruParts;
   m.def("gemm_f32", &gemm_f32);
   m.def("glu_f32", &glu_f32);
 }

@@ -29,6 +29,8 @@ struct DecodeAttnParams {
   float scale_log2;  // softmax scale * log2(e)
   // score (times log2(e)) of a sink: one more term of the softmax denominator, without a value
   float sink_log2 = -INFINITY;
+  const float* sinks;   // [Hq] the sinks' scores, one per head, or nullptr
+  float out_gain = 1.f; // factor on the result
   // Differential attention (diff != 0): query heads 2 h and 2 h + 1 are the two maps of head h. The merge writes
   // o = a1 - diff_lambda a2, o / sqrt(mean(o^2) + diff_eps) * diff_gain, one row of out_d values per pair.
   int diff;
@@ -74,6 +76,8 @@ struct PrefillAttnParams {
   int keep_first, out_d, exact_p, chunk;  // as in DecodeAttnParams
   float scale_log2;
   float sink_log2 = -INFINITY;
+  const float* sinks;   // as in DecodeAttnParams
+  float out_gain = 1.f;
   int num_blocks;  // bound for block-table entries (<= 0: unchecked), violations go to *status
   int* status;
   float* out_f32;  // fp32 rows instead of `out` (the same pitch), or nullptr

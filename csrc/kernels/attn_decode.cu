@@ -430,9 +430,10 @@ __global__ void __launch_bounds__(D) decode_merge_kernel(const DecodeAttnParams 
   const int head = blockIdx.y;
   const int d = threadIdx.x;
   const long long base = (static_cast<long long>(seq) * p.Hq + head) * p.max_splits;
-  float M = p.sink_log2;
+  const float sink = p.sinks != nullptr ? p.sinks[head] * 1.4426950408889634f : p.sink_log2;
+  float M = sink;
   for (int s = 0; s < p.max_splits; ++s) M = fmaxf(M, p.part_ml[(base + s) * 2]);
-  float acc = 0.f, L = p.sink_log2 == -INFINITY ? 0.f : ex2(p.sink_log2 - M);
+  float acc = 0.f, L = sink == -INFINITY ? 0.f : ex2(sink - M);
   for (int s = 0; s < p.max_splits; ++s) {
     const float ms = p.part_ml[(base + s) * 2];
     if (ms == -INFINITY) continue;
@@ -440,7 +441,7 @@ __global__ void __launch_bounds__(D) decode_merge_kernel(const DecodeAttnParams 
     acc += f * p.part_o[(base + s) * D + d];
     L += f * p.part_ml[(base + s) * 2 + 1];
   }
-  const float r = L > 0.f ? acc / L : 0.f;
+  const float r = L > 0.f ? acc / L * p.out_gain : 0.f;
   const __nv_bfloat16 rb = __float2bfloat16(r);
   const int od = p.out_d > 0 ? p.out_d : D;
   if (d < od) p.out[static_cast<long long>(seq) * p.out_stride + head * od + d] = rb;

@@ -363,8 +363,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     if (!ok && lane == 0) set_status_once(status, kStatusMbarTimeoutEpilogue);
     if (ok && n_tiles > 0) {
       tc_fence_after_sync();
-      if (p.sink_log2 != -INFINITY) l_sum += ex2a(p.sink_log2 - m_used);
-      const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
+      const float sink = p.sinks != nullptr ? p.sinks[head] * 1.4426950408889634f : p.sink_log2;
+      if (sink != -INFINITY) l_sum += ex2a(sink - m_used);
+      const float inv = l_sum > 0.f ? p.out_gain / l_sum : 0.f;
       const int od = p.out_d > 0 ? p.out_d : DV;  // values stored per head
       const bool out_vec = (od & 7) == 0 && (p.out_stride & 7) == 0;
       __nv_bfloat16* orow = p.out + static_cast<long long>(row_base + qi) * p.out_stride + head * od;

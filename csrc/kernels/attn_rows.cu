@@ -40,7 +40,8 @@ __global__ void __launch_bounds__(kKeys) row_attention_kernel(const RowAttnParam
   const int lo = p.chunk > 0 ? pos / p.chunk * p.chunk : ((p.window > 0 && pos + 1 > p.window) ? pos + 1 - p.window : 0);
   const int n_first = min(p.keep_first, lo);
   const int n_vis = n_first + (pos + 1 - lo);
-  float m_run = p.sink, l_run = p.sink == -INFINITY ? 0.f : 1.f, acc[kMaxV];
+  const float sink = p.sinks != nullptr ? p.sinks[head] : p.sink;
+  float m_run = sink, l_run = sink == -INFINITY ? 0.f : 1.f, acc[kMaxV];
 #pragma unroll
   for (int i = 0; i < kMaxV; ++i) acc[i] = 0.f;
   __syncthreads();
@@ -86,8 +87,8 @@ __global__ void __launch_bounds__(kKeys) row_attention_kernel(const RowAttnParam
   for (int i = 0; i < kMaxV; ++i) {
     const int c = threadIdx.x + i * kKeys;
     if (c >= p.E) continue;
-    if (p.out_f32) static_cast<float*>(p.out)[at + c] = acc[i] / l_run;
-    else static_cast<T*>(p.out)[at + c] = from_f<T>(acc[i] / l_run);
+    if (p.out_f32) static_cast<float*>(p.out)[at + c] = acc[i] / l_run * p.out_gain;
+    else static_cast<T*>(p.out)[at + c] = from_f<T>(acc[i] / l_run * p.out_gain);
   }
 }
 

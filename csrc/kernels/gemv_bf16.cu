@@ -92,6 +92,10 @@ __global__ void __launch_bounds__(kWarpsPerCta * 32) gemv_bf16_kernel(const Gemv
       if (p.out_f32 != nullptr) p.out_f32[o] = y;
       else p.out_bf16[o] = __float2bfloat16(y);
     } else {
+      if (p.act == 2) {   // squared ReLU
+        v0 = fmaxf(v0, 0.f) * fmaxf(v0, 0.f);
+        v1 = fmaxf(v1, 0.f) * fmaxf(v1, 0.f);
+      }
       const long long o = static_cast<long long>(m) * p.ldo + rows[0];
       if (p.out_f32 != nullptr) {
         p.out_f32[o] = v0;

@@ -18,7 +18,7 @@ struct GemvParams {
   int M, N, K;
   int tiled;
   int swiglu;  // 1: rows are gate|up interleaved in units of 32; output [M, N/2] = act(gate) * up
-  int act;     // 0 = SiLU, 1 = tanh-GELU
+  int act;     // swiglu: 0 = SiLU, 1 = tanh-GELU; else 2 = squared ReLU
 };
 
 void launch_gemv_bf16(const GemvParams& p, cudaStream_t stream);

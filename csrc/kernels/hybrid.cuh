@@ -49,10 +49,13 @@ cudaError_t launch_stream_norm(const StreamNormParams& p, int dtype, cudaStream_
 // What stands between two layers whose mixer and feed-forward run side by side on one residual stream x, or between
 // two sublayers with a norm on either side. With N values per row:
 //   tokens given : x = embed[token] * embed_scale
+//   base given   : x = base + sum_b ... (the branches replace the stream)
 //   else         : x += sum_b gain[b] * (w[b] ? y_b / sqrt(mean(y_b^2) + eps) * w[b] : y_b)   (dense branches)
 //                     + e,   e = sum_c weight[c] * expert_rows[slot[c]]                       (chosen experts)
 //                  where y_b of a branch without rows is e, which is then not added a second time
 //   then         : h_o = x / sqrt(mean(x^2) + eps) * (w_offset + norm_w[o])                   for every output o
+//   split given  : instead of the norms, the operand of a product over [x; embedding]: bf16 rows of three parts, x rounded |
+//                  what the rounding left | embed[x0_tokens], or fp32 rows of two, x | embed[x0_tokens]
 // x is written back when store_x is set. Where clear_y is set for a branch, its rows are zeroed on the way (the
 // split-K GEMM of the layer that follows adds into them).
 constexpr int kMaxBranches = 2;
@@ -76,6 +79,11 @@ struct BranchNormParams {
   const float* e_weight;    // [rows, top]
   int top;
   int store_x;
+  const float* base;        // [N] or nullptr
+  void* split;              // [rows, ld_split], parts split_off apart, or nullptr
+  long long ld_split;
+  int split_off;
+  const int* x0_tokens;     // [rows]
   int n_out;
   const float* norm_w[2];
   void* h[2];
@@ -88,6 +96,9 @@ struct BranchNormParams {
   int* status;
 };
 cudaError_t launch_branch_norm(const BranchNormParams& p, int dtype, cudaStream_t stream);
+
+// Heads of attention over one projection that is key and value (HeadsParams::k_rms): the key is the stored value times
+// one number per token and times k_norm, so the cache keeps the values and that number, and k_norm is part of q_norm.
 
 // Rotary positions: pair i turns by position * (freq_hi[i] + freq_lo[i]) (the frequency as an unevaluated
 // sum of two floats, so the angle is good to the last bits of a 32-bit float at any position).
@@ -129,6 +140,7 @@ struct HeadsParams {
   const long long* slots;   // [M] cache slot of each row, < 0: not stored
   long long num_slots;
   int DP, EP;
+  float* k_rms;             // [cache slots] or nullptr: k goes to the cache as it is, and 1 / sqrt(mean(k^2) + eps) here
   int* status;
 };
 cudaError_t launch_heads(const HeadsParams& p, int dtype, cudaStream_t stream);
@@ -155,12 +167,95 @@ struct RowAttnParams {
   int chunk;                // > 0: only positions of the query's own chunk (counted from position 0) are visible
   float scale;
   float sink;               // score of one more term of the softmax denominator, without a value (-inf: none)
+  const float* sinks;       // [H] the same per head, or nullptr
+  float out_gain;           // factor on the result
   void* out;                // [rows, ldo], heads o_hd apart; fp32 when out_f32 is set
   int out_f32, o_hd;
   long long ldo;
   int* status;
 };
 cudaError_t launch_row_attention(const RowAttnParams& p, int dtype, cudaStream_t stream);
+
+// Talking heads over keys that are values. The score of head g for key j of a query at position i is
+//   c_g = cap tanh(q_g . k_j k_rms_j scale / cap)            (cap 0: as it is)
+// head h goes on with sum_g talk[h, g] c_g - bias[h, i - j] (bias: the heads' distance biases, mixed the same way), takes the
+// softmax over the visible keys and sums k_j; the result times sigmoid(gate).
+struct TalkParams {
+  const void* q;            // [rows, q_ld], heads DP apart: normed, times the keys' norm weights
+  long long q_ld;
+  const void* cache;        // [blocks, G, 16, DP]
+  const float* k_rms;       // [blocks, 16]
+  const int* block_tables;  // [sequences, max_blocks]
+  const int* seq_lens;      // decode: [rows]
+  const int* pages_per_split;
+  const int* tile_seq;      // prompt chunks: 128-row tiles
+  const int* tile_q0;
+  const int* q_start;
+  const int* q_lens;
+  const int* ctx_lens;
+  int n_rows;               // decode: rows; chunks: tiles
+  int max_blocks, num_blocks;
+  int H, G, D, DP;
+  int window;               // 0: all earlier positions
+  float scale, cap;
+  const float* talk;        // [H, H]
+  const float* bias;        // [H, n_bias], distance 0 first
+  int n_bias;
+  const void* gate;         // [rows, gate_ld] pre-activations, heads D apart; fp32 when gate_f32 is set
+  int gate_f32;
+  long long gate_ld;
+  float* part_o;            // decode: [rows, H, max_splits, DP]
+  float* part_ml;           // [rows, H, max_splits, 2]
+  int max_splits;
+  float* scores;            // prompt chunks: [tiles, H, 128, span] mixed scores times log2(e), keys from the tile's first one on
+  int span;
+  void* out;                // [rows, ldo], heads of D
+  long long ldo;
+  int* status;
+};
+// Any sizes, fp32 FMAs, one CTA per row: the fp32 path and sizes that the other kernels do not take.
+cudaError_t launch_talk_rows(const TalkParams& p, int dtype, cudaStream_t stream);
+size_t talk_rows_smem(int H, int D);
+// bf16, D padded to 64 or 128. Decoding: split-KV and merge.
+cudaError_t launch_talk_decode(const TalkParams& p, cudaStream_t stream);
+bool talk_decode_ok(int H, int G, int DP);
+// Prompt chunks: mixed scores of a step's tiles, then softmax and sums.
+cudaError_t launch_talk_prefill(const TalkParams& p, cudaStream_t stream);
+bool talk_prefill_ok(int H, int DP);
+int talk_span(int window, int max_ctx);   // keys per row of `scores`
+
+// Gated recurrence whose gates read only the current token (minGRU), element by element over N channels:
+//   z = sigmoid(z_in + b_z), u = x_in + b_x, c = u + 1/2 where u >= 0 else sigmoid(u),  S <- (1 - z) S + z c
+//   out = S silu(g) * out_gain
+struct GruParams {
+  const void* proj;         // [M, ld]: z (N) | x (N) | g (N); type as in HeadsParams
+  int proj_f32;
+  long long ld;
+  int N;                    // a multiple of 4
+  const float* bias;        // [2 N]: b_z | b_x
+  float out_gain;
+  float* state;             // [slots, N]
+  int num_slots;
+  // decode rows
+  const int* row_slots;     // [rows], < 0: padding row
+  const int* positions;     // [rows]; a row at position 0 starts from the zero state
+  int rows;
+  // prompt chunks
+  const int* seq_slots;
+  const int* tile_seq;      // 128-row tiles, those of a sequence one after the other
+  const int* tile_q0;
+  const int* q_start;
+  const int* q_lens;
+  const int* ctx_lens;
+  int n_tiles;
+  float* ws;                // [n_tiles, 1 + kGruParts, 2, N]: what a tile and its parts make of a state, S -> a S + b
+  void* out;                // [M, ldo]
+  long long ldo;
+  int* status;
+};
+constexpr int kGruParts = 4;   // 32-row parts of a tile that are walked at once
+cudaError_t launch_gru_decode(const GruParams& p, int dtype, cudaStream_t stream);
+cudaError_t launch_gru_prefill(const GruParams& p, int dtype, cudaStream_t stream);
 
 constexpr int kRetChunk = 64;   // rows per chunk of the chunked form (two per 128-row tile of the scheduler)
 
@@ -444,7 +539,7 @@ cudaError_t launch_moe_rows(const MoeRowsParams& p, int dtype, cudaStream_t stre
 // out[M, N] = a[M, K] w[N, K]^T in fp32 FMAs.
 cudaError_t launch_gemm_f32(const float* a, long long lda, const float* w, long long ldw, float* out, long long ldo,
                             int M, int N, int K, cudaStream_t stream);
-// out[m, i] = act(gu[m, i]) * gu[m, I + i]
+// out[m, i] = act(gu[m, i]) * gu[m, I + i]; act 0: silu, 1: tanh form of gelu, 2: relu(gu[m, i])^2 alone
 cudaError_t launch_glu_f32(const float* gu, long long ldg, float* out, long long ldo, int M, int I, int act,
                            cudaStream_t stream);
 

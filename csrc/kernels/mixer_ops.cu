@@ -61,6 +61,7 @@ __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
     if (h_lo < H) rq = 1.f / sqrtf(block_sum_all(sq, s_red) / static_cast<float>(H * D) + p.eps);
     if (need_k) rk = 1.f / sqrtf(block_sum_all(sk, s_red) / static_cast<float>(G * D) + p.eps);
   }
+  const float rw = p.k_norm != nullptr ? rk : 1.f;   // what the stored keys are multiplied by
   const float qt = p.t_coef != 0.f ? 1.f + p.t_coef * logf(floorf(static_cast<float>(pos + 1) / p.t_every) + 1.f) : 1.f;
   const long long k_col = p.q_pd * H;   // k follows q in the projection row
   __syncthreads();
@@ -69,6 +70,7 @@ __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
   if (p.slots != nullptr && slot >= p.num_slots && threadIdx.x == 0) set_status_once(p.status, kStatusBadIndex);
   const long long blk = slot >> 4;
   const int off = static_cast<int>(slot & 15);
+  if (p.k_rms != nullptr && store_kv && h_lo <= H && H < h_hi && threadIdx.x == 0) p.k_rms[slot] = rk;
 
   if constexpr (VEC) {
     // four values (two pairs of the interleaved layout) or two times four (the other) per item, items of all
@@ -82,7 +84,7 @@ __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
       if (!is_q && p.k_out == nullptr && !store_kv) continue;
       const long long col = is_q ? h * p.q_pd : k_col + (h - H) * D;
       const P* src = pr + col;
-      const float r = is_q ? rq : rk, ks = is_q ? qt : p.k_scale;
+      const float r = is_q ? rq : rw, ks = is_q ? qt : p.k_scale;
       const float* w = is_q ? p.q_norm : p.k_norm;
       if (w != nullptr) w += (is_q ? h : h - H) * D;
       auto get = [&](int d, float (&v)[4]) {
@@ -163,7 +165,7 @@ __global__ void __launch_bounds__(256) heads_kernel(const HeadsParams p) {
     const long long col = is_q ? h * p.q_pd : k_col + (h - H) * D;
     const P* src = pr + col;
     const float* bias = p.bias != nullptr ? p.bias + col : nullptr;
-    const float r = is_q ? rq : rk;
+    const float r = is_q ? rq : rw;
     const float* w = is_q ? p.q_norm : p.k_norm;
     if (w != nullptr) w += (is_q ? h : h - H) * D;
     const float ks = is_q ? qt : p.k_scale;
@@ -323,7 +325,13 @@ __global__ void __launch_bounds__(256) glu_f32_kernel(const float* gu, long long
   for (long long i = blockIdx.x * 256ll + threadIdx.x; i < total; i += gridDim.x * 256ll) {
     const long long m = i / I;
     const int c = static_cast<int>(i - m * I);
-    const float g = gu[m * ldg + c], u = gu[m * ldg + I + c];
+    const float g = gu[m * ldg + c];
+    if (act == 2) {
+      const float r = fmaxf(g, 0.f);
+      out[m * ldo + c] = r * r;
+      continue;
+    }
+    const float u = gu[m * ldg + I + c];
     const float a = act == 0 ? silu_f(g)
                              : 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
     out[m * ldo + c] = a * u;

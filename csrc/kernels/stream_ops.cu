@@ -231,6 +231,32 @@ __device__ __forceinline__ float2 block_sum2(float2 v, float2* scratch) {
   return make_float2(warp_sum(s.x), warp_sum(s.y));
 }
 
+// Operand of the product over [x; embedding] (BranchNormParams::split)
+template <typename T>
+__device__ __forceinline__ const T* x0_row(const BranchNormParams& p, int row) {
+  const int tok = p.x0_tokens[row];
+  const bool ok = tok >= 0 && tok < p.vocab;
+  if (!ok && threadIdx.x == 0) set_status_once(p.status, kStatusBadIndex);
+  return static_cast<const T*>(p.embed) + static_cast<long long>(ok ? tok : 0) * p.N;
+}
+template <typename T>
+__device__ __forceinline__ void split_row4(const BranchNormParams& p, int row, int c, const float (&x)[4]) {
+  T* d = static_cast<T*>(p.split) + static_cast<long long>(row) * p.ld_split + c;
+  store4<T>(d, x);
+  if constexpr (sizeof(T) == 2) {
+    float rest[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) rest[j] = x[j] - to_f(from_f<T>(x[j]));
+    d += p.split_off;
+    store4<T>(d, rest);
+  }
+  float e[4];
+  load4<T>(x0_row<T>(p, row) + c, e);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) e[j] *= p.embed_scale;
+  store4<T>(d + p.split_off, e);
+}
+
 template <typename T, int CH, int NB, int THREADS, int CTAS>
 __global__ void __launch_bounds__(THREADS, CTAS) branch_norm_kernel(const BranchNormParams p) {
   __shared__ float s_red[32];
@@ -284,7 +310,8 @@ __global__ void __launch_bounds__(THREADS, CTAS) branch_norm_kernel(const Branch
 #pragma unroll
         for (int j = 0; j < 4; ++j) x[k][j] = 0.f;
         if (c < N) {
-          load4_stream(xr + c, x[k]);
+          if (p.base != nullptr) load4<float>(p.base + c, x[k]);
+          else load4_stream(xr + c, x[k]);
           if (e_plain) expert_sum4<T>(p, s_chosen[parity], c, x[k]);
         }
 #pragma unroll
@@ -331,6 +358,14 @@ __global__ void __launch_bounds__(THREADS, CTAS) branch_norm_kernel(const Branch
       if (p.store_x) store4<float>(xr + c, x[k]);
 #pragma unroll
       for (int j = 0; j < 4; ++j) ssq = fmaf(x[k][j], x[k][j], ssq);
+    }
+    if (p.split != nullptr) {
+#pragma unroll
+      for (int k = 0; k < CH; ++k) {
+        const int c = (k * blockDim.x + threadIdx.x) * 4;
+        if (c < N) split_row4<T>(p, row, c, x[k]);
+      }
+      continue;
     }
     if (dst < 0) continue;  // a row without outputs; the same for every thread of the CTA
     const float r = 1.f / sqrtf(block_sum_all(ssq, s_red) * inv_n + p.eps);
@@ -410,16 +445,25 @@ __global__ void __launch_bounds__(256) branch_norm_any_kernel(const BranchNormPa
             const float y = branch(b, c);
             x = fmaf(p.gain[b] * (p.w[b] != nullptr ? r[b] * p.w[b][c] : 1.f), y, x);
           }
-        x += xr[c];
+        x += p.base != nullptr ? p.base[c] : xr[c];
       }
 #pragma unroll
       for (int b = 0; b < kMaxBranches; ++b)
         if (b < p.n_branches && p.clear_y[b]) p.y[b][static_cast<long long>(row) * p.ldy + c] = 0.f;
       if (p.store_x) xr[c] = x;
+      if (p.split != nullptr) {
+        T* d = static_cast<T*>(p.split) + static_cast<long long>(row) * p.ld_split + c;
+        d[0] = from_f<T>(x);
+        if constexpr (sizeof(T) == 2) {
+          d += p.split_off;
+          d[0] = from_f<T>(x - to_f(from_f<T>(x)));
+        }
+        d[p.split_off] = from_f<T>(to_f(x0_row<T>(p, row)[c]) * p.embed_scale);
+      }
       s_u[c] = x;
       ssq = fmaf(x, x, ssq);
     }
-    if (dst < 0) continue;
+    if (dst < 0 || p.split != nullptr) continue;
     const float rr = 1.f / sqrtf(block_sum_all(ssq, s_red) * inv_n + p.eps);
     for (int o = 0; o < p.n_out; ++o) {
       T* hr = static_cast<T*>(p.h[o]) + static_cast<long long>(dst) * p.ldh;
@@ -432,7 +476,7 @@ template <typename T>
 cudaError_t launch_branch(const BranchNormParams& p, cudaStream_t stream) {
   const int cap = 8 * sm_count();
   const dim3 grid(p.rows < cap ? p.rows : cap);
-  const bool vec = p.N % 4 == 0 && p.ldy % 4 == 0 && p.ldh % 4 == 0 && p.lde % 4 == 0;
+  const bool vec = p.N % 4 == 0 && p.ldy % 4 == 0 && p.ldh % 4 == 0 && p.lde % 4 == 0 && p.ld_split % 4 == 0 && p.split_off % 4 == 0;
   const int quads = (p.N + 3) / 4;
   auto threads = [&](int ch) { return dim3(((quads + ch - 1) / ch + 31) / 32 * 32); };
   if (vec && p.n_branches <= 1 && quads <= 1024) {

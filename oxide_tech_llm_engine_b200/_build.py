@@ -46,7 +46,7 @@ CUDA_FLAGS = [
 
 # kernels of the extension that only layer-list decoders load
 HYBRID_KERNELS = ("stream_ops.cu", "mixer_ops.cu", "attn_rows.cu", "retention.cu", "ssd.cu", "moe_ops.cu", "latent.cu", "latent_decode.cu", "memory.cu",
-                  "attn_prefill_wide.cu")
+                  "attn_prefill_wide.cu", "talking.cu", "gru.cu")
 HYBRID_HEADERS = ("hybrid.cuh", "hybrid_dev.cuh", "hybrid_mma.cuh")
 SHARED_HEADERS = ("attn.cuh", "attn_prefill_tc.cuh")   # of both kernel extensions
 # kernels of the extension that only quantised weights load

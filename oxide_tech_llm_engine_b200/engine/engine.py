@@ -470,7 +470,7 @@ class LLMEngine:
                        q_start=d("q_start"), q_lens=d("q_lens"), ctx_lens=d("ctx_lens"),
                        prefill_block_tables=d("prefill_block_tables").view(-1, W), logit_map=d("logit_map"),
                        prev_ids=d("prev_ids"), decode_slots=d("decode_slots"), prefill_slots=d("prefill_slots"),
-                       kv_start=d("kv_start"), kv_passes=passes)
+                       kv_start=d("kv_start"), kv_passes=passes, max_ctx=int(max(plan.ctx_lens)) if npf else 0)
         if n_cow:
             self.model.copy_blocks(d("cow_src")[:n_cow], d("cow_dst")[:n_cow])
         return s, bucket

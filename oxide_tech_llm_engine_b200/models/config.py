@@ -53,6 +53,10 @@ class ModelConfig:
     loop: Any = None           # (start, stop, times)
     streams: int = 0
     bigram: Any = None         # layer_spec.BigramSpec
+    # one plain residual stream with a norm before every sublayer, whose result is added times this (None: the other kinds)
+    residual_mult: Any = None
+    loop_inject: bool = False  # every pass of the loop starts with x <- W_in [x; embedding] + a vector of the pass
+    logit_scale: float = 1.0   # before the softcap
 
     @property
     def q_dim(self) -> int:
@@ -72,6 +76,14 @@ class ModelConfig:
         from .layer_spec import layer_runs
 
         return layer_runs(self.n_layers, self.loop)
+
+    @property
+    def pass_starts(self) -> dict:
+        """Number of the pass by the index of the layer run that it begins with."""
+        if self.loop is None:
+            return {}
+        a, b, times = self.loop
+        return {a + t * (b - a): t for t in range(times)}
 
     @property
     def is_recurrent(self) -> bool:
@@ -188,6 +200,21 @@ def _zagolix_preset(name: str, *, width: int, vocab: int, pattern: str, ff: int,
     return zagolix_model(tuple(layers), width=width, vocab=vocab, eps=1e-5, emb_scale=width ** 0.5, name=name)
 
 
+def _vokepel_preset(name: str, *, width: int, vocab: int, pattern: str, ff: int, heads: int, kv_heads: int, dim: int, window: int,
+                    t_heads: int, t_kv: int, t_dim: int, t_window: int, gru: int, loop=None) -> ModelConfig:
+    """A Vokepel-shaped configuration: one letter per layer, 'p' attention with sinks beside a gated recurrence, 't' talking
+    heads."""
+    from .layer_spec import (AttentionSpec, DenseMlpSpec, GruSpec, LayerSpec, ParallelSpec, RotarySpec, TalkingSpec,
+                             vokepel_model)
+
+    left = AttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, RotarySpec(dim, 500000.0, True), window, sinks=True)
+    pair = ParallelSpec(left, GruSpec(gru), (0.5, 0.5))
+    talk = TalkingSpec(t_heads, t_kv, t_dim, t_dim ** -0.5, 30.0, t_window)
+    layers = tuple(LayerSpec(pair if ch == "p" else talk, DenseMlpSpec(ff, act="relu2")) for ch in pattern)
+    return vokepel_model(layers, width=width, vocab=vocab, eps=1e-5, residual_mult=0.5, loop=loop, logit_scale=0.5,
+                         logit_softcap=30.0, name=name)
+
+
 LAYER_LIST_PRESETS = {
     "kipolix-tiny": dict(width=128, vocab=1024, ff=256, pattern="arar", heads=4, kv_heads=2, dim=64, window=56,
                          keep_first=3, r_heads=2, r_dim=64, r_vdim=64, streams=2, loop=(1, 3, 2), buckets=1000),
@@ -216,8 +243,17 @@ ZAGOLIX_PRESETS = {
 }
 
 
+VOKEPEL_PRESETS = {
+    "vokepel-tiny": dict(width=128, vocab=1024, pattern="ptp", ff=320, heads=4, kv_heads=2, dim=32, window=72, t_heads=3, t_kv=1,
+                         t_dim=48, t_window=40, gru=144, loop=(1, 3, 2)),
+    # the shapes of llama3-8b's layers (width, heads), eight of 24 layers run twice
+    "vokepel-8b": dict(width=4096, vocab=128256, pattern="pt" * 12, ff=16384, heads=32, kv_heads=8, dim=128, window=4096, t_heads=32,
+                       t_kv=8, t_dim=128, t_window=1024, gru=4096, loop=(8, 16, 2)),
+}
+
+
 def preset_names() -> list:
-    return [*PRESETS, *LAYER_LIST_PRESETS, *POVATAR_PRESETS, *ZAGOLIX_PRESETS]
+    return [*PRESETS, *LAYER_LIST_PRESETS, *POVATAR_PRESETS, *ZAGOLIX_PRESETS, *VOKEPEL_PRESETS]
 
 
 def preset(name: str, **overrides) -> ModelConfig:
@@ -227,6 +263,8 @@ def preset(name: str, **overrides) -> ModelConfig:
         return replace(_povatar_preset(name, **POVATAR_PRESETS[name]), **overrides)
     if name in ZAGOLIX_PRESETS:
         return replace(_zagolix_preset(name, **ZAGOLIX_PRESETS[name]), **overrides)
+    if name in VOKEPEL_PRESETS:
+        return replace(_vokepel_preset(name, **VOKEPEL_PRESETS[name]), **overrides)
     if name not in PRESETS:
         raise KeyError(f"unknown model preset {name!r}; known: {sorted(preset_names())}")
     return replace(PRESETS[name], **overrides)

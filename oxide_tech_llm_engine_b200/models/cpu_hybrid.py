@@ -37,6 +37,13 @@ class CpuHybridModel:
                     at.append(len(self.pk))
                     self.pk.append(torch.zeros(num_blocks, 1, 16, mx.rot_dim))
                     self.pv.append(torch.zeros(num_blocks, 1, 16, mx.kv_rank))
+                elif mx.kind == "talking_attention":   # keys before their norm, which are the values, and the norm's factor
+                    at.append(len(self.pk))
+                    self.pk.append(torch.zeros(num_blocks, mx.kv_heads, 16, mx.dim))
+                    self.pv.append(torch.zeros(num_blocks, 1, 16, 1))
+                elif mx.kind == "min_gru":
+                    at.append(len(self.states))
+                    self.states.append(torch.zeros(state_slots, mx.width))
                 elif mx.kind == "mlstm":   # memory, normaliser, running maximum
                     at.append(len(self.states))
                     self.states.append((torch.zeros(state_slots, mx.heads, mx.dim, mx.vdim), torch.zeros(state_slots, mx.heads, mx.dim),
@@ -104,6 +111,8 @@ class CpuHybridModel:
             s = s.masked_fill(~see[None], float("-inf"))
             if a.sink is not None:
                 s = torch.cat([s, torch.full_like(s[..., :1], a.sink)], -1)
+            if a.sinks:
+                s = torch.cat([s, w[p + "sink"][:, None, None].expand(-1, n, 1)], -1)
             out[r0:r0 + n] = torch.einsum("hij,jhe->ihe", torch.softmax(s, -1)[..., :ctx], values.repeat_interleave(g * n2, 1))
         if a.diff is not None:
             lam = torch.exp((w[p + "lq1"] * w[p + "lk1"]).sum()) - torch.exp((w[p + "lq2"] * w[p + "lk2"]).sum()) + a.diff
@@ -171,6 +180,41 @@ class CpuHybridModel:
         gate = torch.nn.functional.silu(h @ w[p + "g"].T)
         return (self._unit(out).reshape(T, -1) * gate) @ w[p + "o"].T
 
+    def _talking(self, a, p: str, ci: int, h, pos, seqs, blk, off):
+        T, w, g = h.shape[0], self.w, a.heads // a.kv_heads
+        q, k = h @ w[p + "q"].T, h @ w[p + "k"].T
+        # the keys' norm weights act on the queries, the norm itself is a number per cached token
+        wk = w[p + "k.norm"].view(a.kv_heads, a.dim).repeat_interleave(g, 0)
+        q = (self._unit(q) * w[p + "q.norm"]).view(T, a.heads, a.dim) * wk
+        self.pk[ci][blk, :, off] = k.view(T, a.kv_heads, a.dim)
+        self.pv[ci][blk, 0, off] = torch.rsqrt(k.pow(2).mean(-1, keepdim=True) + self.cfg.rms_eps)
+        out = torch.zeros(T, a.heads, a.dim)
+        for r0, n, ctx, table, _ in seqs:
+            rows = self._pages(self.pk[ci], table, ctx).repeat_interleave(g, 1)
+            s = torch.einsum("ihd,jhd->hij", q[r0:r0 + n], rows) * (self._pages(self.pv[ci], table, ctx)[:, 0, 0] * a.scale)
+            if a.softcap:
+                s = a.softcap * torch.tanh(s / a.softcap)
+            i, j = torch.arange(ctx - n, ctx)[:, None], torch.arange(ctx)[None]
+            far = (i - j).clamp(min=0)
+            s = s - w[p + "r1"][:, None, None] * torch.log1p(w[p + "r2"][:, None, None] * far)
+            s = torch.einsum("hg,gij->hij", w[p + "talk"], s)
+            see = (j <= i) & ((i - j < a.window) if a.window else True)
+            out[r0:r0 + n] = torch.einsum("hij,jhe->ihe", torch.softmax(s.masked_fill(~see[None], float("-inf")), -1), rows)
+        return (out.reshape(T, -1) * torch.sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T
+
+    def _gru(self, r, p: str, ci: int, h, seqs):
+        w = self.w
+        z, u = torch.sigmoid(h @ w[p + "z"].T + w[p + "z.b"]), h @ w[p + "x"].T + w[p + "x.b"]
+        c = torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
+        out = torch.zeros_like(c)
+        for r0, n, ctx, _, slot in seqs:
+            S = torch.zeros_like(self.states[ci][slot]) if ctx == n else self.states[ci][slot]
+            for t in range(r0, r0 + n):
+                S = (1.0 - z[t]) * S + z[t] * c[t]
+                out[t] = S
+            self.states[ci][slot] = S
+        return (out * torch.nn.functional.silu(h @ w[p + "g"].T)) @ w[p + "o"].T
+
     def _ssd(self, r, p: str, ci: int, h, seqs):
         T, w, F = h.shape[0], self.w, torch.nn.functional
         gn = r.groups * r.state
@@ -221,10 +265,20 @@ class CpuHybridModel:
 
     def _dense(self, f, p: str, h):
         w, F = self.w, torch.nn.functional
+        if not f.glu:
+            return torch.relu(h @ w[p + "up"].T).square() @ w[p + "down"].T
         act = (lambda z: F.gelu(z, approximate="tanh")) if f.act == "gelu_tanh" else F.silu
         return (act(h @ w[p + "gate"].T) * (h @ w[p + "up"].T)) @ w[p + "down"].T
 
-    def _mix(self, mx, p: str, ci: int, h, pos, seqs, blk, off):
+    def _mix(self, mx, p: str, at: list, h, pos, seqs, blk, off):
+        if mx.kind == "parallel":      # (the weighted sum; the other form belongs to _parallel_layers)
+            return (mx.gains[0] * self._mix(mx.left, p + "left.", at[:1], h, pos, seqs, blk, off)
+                    + mx.gains[1] * self._mix(mx.right, p + "right.", at[1:], h, pos, seqs, blk, off))
+        ci = at[0]
+        if mx.kind == "talking_attention":
+            return self._talking(mx, p, ci, h, pos, seqs, blk, off)
+        if mx.kind == "min_gru":
+            return self._gru(mx, p, ci, h, seqs)
         if mx.kind == "attention":
             return self._attention(mx, p, ci, h, pos, seqs, blk, off)
         if mx.kind == "latent_attention":
@@ -239,13 +293,27 @@ class CpuHybridModel:
     def _sandwich_layers(self, x, pos, seqs, blk, off):
         """Layers with a norm on either side of every sublayer; returns the stream."""
         w, one = self.w, self.cfg.norm_weight_offset
-        for li, (ci,) in self.runs:
+        for li, at in self.runs:
             L, p = self.cfg.layers[li], f"l{li}."
-            y = self._mix(L.mixer, p + "mix.", ci, self._unit(x) * (w[p + "norm1"] + one), pos, seqs, blk, off)
+            y = self._mix(L.mixer, p + "mix.", at, self._unit(x) * (w[p + "norm1"] + one), pos, seqs, blk, off)
             x = x + self._unit(y) * w[p + "norm1b"] * w[p + "ls1"]
             if L.mlp is not None:
                 y = self._feed(L.mlp, p + "mlp.", self._unit(x) * (w[p + "norm2"] + one))
                 x = x + self._unit(y) * w[p + "norm2b"] * w[p + "ls2"]
+        return x
+
+    def _single_layers(self, x, pos, seqs, blk, off):
+        """One plain residual stream, a norm before every sublayer; returns the stream."""
+        cfg, w, one, x0 = self.cfg, self.w, self.cfg.norm_weight_offset, x
+        starts = cfg.pass_starts
+        for ri, (li, at) in enumerate(self.runs):
+            L, p = cfg.layers[li], f"l{li}."
+            if cfg.loop_inject and ri in starts:
+                x = torch.cat([x, x0], -1) @ w["loop.in"].T + w["loop.step"][starts[ri]]
+            h = self._unit(x) * (w[p + "norm1"] + one)
+            x = x + cfg.residual_mult * self._mix(L.mixer, p + "mix.", at, h, pos, seqs, blk, off)
+            if L.mlp is not None:
+                x = x + cfg.residual_mult * self._feed(L.mlp, p + "mlp.", self._unit(x) * (w[p + "norm2"] + one))
         return x
 
     def _parallel_layers(self, x, pos, seqs, blk, off):
@@ -282,6 +350,8 @@ class CpuHybridModel:
             prev = torch.as_tensor(plan.prev_ids.astype(np.int64))
             row = torch.where(prev < 0, torch.full_like(prev, b.buckets), (prev * b.mul_prev + tok * b.mul_cur) % b.buckets)
             x = x + w["bigram"][row]
+        if cfg.residual_mult is not None:
+            return self._head(self._single_layers(x * cfg.emb_scale, pos, seqs, blk, off), plan)
         if any(L.parallel for L in cfg.layers):
             return self._head(self._parallel_layers(x * cfg.emb_scale, pos, seqs, blk, off), plan)
         if any(L.post_norm for L in cfg.layers):
@@ -295,9 +365,9 @@ class CpuHybridModel:
             h = self._unit(torch.einsum("s,std->td", ci, xs)) * (w[f"{p}norm{q}"] + cfg.norm_weight_offset)
             xs = torch.einsum("sz,std->ztd", mix, xs) + co[:, None, None] * fn(h)[None]
 
-        for li, (ci,) in self.runs:
+        for li, at in self.runs:
             L, p = cfg.layers[li], f"l{li}."
-            sub(p, 1, lambda h: self._mix(L.mixer, p + "mix.", ci, h, pos, seqs, blk, off))
+            sub(p, 1, lambda h: self._mix(L.mixer, p + "mix.", at, h, pos, seqs, blk, off))
             if L.mlp is not None:
                 sub(p, 2, lambda h: self._feed(L.mlp, p + "mlp.", h))
         return self._head(xs.sum(0), plan)
@@ -305,5 +375,7 @@ class CpuHybridModel:
     def _head(self, x: torch.Tensor, plan) -> torch.Tensor:
         rows = torch.as_tensor(plan.logit_rows.astype(np.int64))
         hl = self._unit(x[rows]) * (self.w["final.norm"] + self.cfg.norm_weight_offset)
-        self.logits = hl @ self.head.T
+        self.logits = hl @ self.head.T * self.cfg.logit_scale
+        if self.cfg.logit_softcap:
+            self.logits = self.cfg.logit_softcap * torch.tanh(self.logits / self.cfg.logit_softcap)
         return self.logits

@@ -39,7 +39,19 @@ and with a norm on either side of every sublayer:
       branch_norm  norm of the sublayer's result (of the weighted expert rows), residual, norm of the next sublayer
     final branch_norm over the logit rows -> gemm(head)
 
-In a captured decode step the three lines between two branch_norms run on streams of their own: the
+and with one plain residual stream, x <- x + m f(norm(x)):
+
+    branch_norm   embedding -> residual, norm of the first sublayer
+    per sublayer:
+      pair:           gemm(q|k|v | z|x|g) -> heads, paged attention with sinks | gated recurrence -> gemm(O of both)
+      talking heads:  gemm(q|k|gate) -> heads (norms; keys that are values) -> talk_decode / scores and values of a tile
+      MLP:            gemm(up, squared ReLU) -> gemm(down)
+      branch_norm     the result times m into the residual, norm of the next sublayer
+    ahead of a pass of the loop:
+      branch_norm     the stream and the embedding as operand rows -> gemm -> branch_norm (plus the pass's vector) as the stream
+    final branch_norm over the logit rows -> gemm(head) -> softcap
+
+In a captured decode step of side-by-side layers the three lines between two branch_norms run on streams of their own: the
 experts beside the projection and the mixers, the state-space mixer beside the attention.
 
 KV blocks come from the scheduler's paged pool like any model's (one cache per attention run, so a
@@ -76,7 +88,7 @@ def tc_head(a) -> int:
     if a.heads * a.maps // a.kv_heads > 16 or big > 256:
         return 0
     if big > 128:      # plain causal attention only
-        return 256 if not (a.window or a.chunk or a.sink is not None) else 0
+        return 256 if not (a.window or a.chunk or a.sink is not None or a.sinks) else 0
     return 64 if big <= 64 else 128
 
 
@@ -87,6 +99,13 @@ def latent_layout(a) -> tuple:
     z = hops.prefill_size(at + round_up(a.dim, 8), round_up(a.vdim, 8))
     return (*z, at) if z is not None else (at + round_up(a.dim, 8), 0, at)
 
+
+def talk_head(a) -> int:
+    """Padded head size of the talking-heads kernels, 0 when they do not take it."""
+    return 0 if a.dim > 128 else (64 if a.dim <= 64 else 128)
+
+
+TALK_SCORE_BYTES = 256 << 20   # mixed scores of prompt tiles that are held at a time
 
 KV_PASS_ROWS = 65536      # positions whose keys and values are expanded at a time
 
@@ -100,10 +119,12 @@ class _Sublayer:
 
 
 class _NormedSublayer:
-    """Norm weights of a sublayer's input and result (the latter times the layer scale), and the function that runs it."""
+    """Norm weights of a sublayer's input and result (the latter times the layer scale, or none), the function that runs it,
+    and the factor on its result. `base`: the result takes the place of the stream, plus this vector (the entry of a pass, whose
+    input is not normed)."""
 
-    def __init__(self, norm, out, run, last_of: int):
-        self.norm, self.out, self.run, self.last_of = norm, out, run, last_of
+    def __init__(self, norm, out, run, last_of: int, gain: float = 1.0, base=None):
+        self.norm, self.out, self.run, self.last_of, self.gain, self.base = norm, out, run, last_of, gain, base
 
 
 class _ParallelLayer:
@@ -135,20 +156,21 @@ class AttentionRun:
     def __call__(self, s: StepInputs, h: torch.Tensor) -> None:
         self.m.into_acc(self.attend(s, self.m.project(h, self.w["w_in"], self.width)), self.w["w_o"])
 
-    def attend(self, s: StepInputs, proj: torch.Tensor) -> torch.Tensor:
+    def attend(self, s: StepInputs, proj: torch.Tensor, out: Optional[torch.Tensor] = None, gain: float = 1.0) -> torch.Tensor:
+        """Projection rows -> heads' results times `gain`, in `out` or a buffer of their own."""
         m, a, w, M = self.m, self.spec, self.w, s.m
         q = m.buffer(("q", self.nq * self.dp, a.dim, a.maps), self.nq * self.dp)
         hops.heads(proj, M, h=self.nq, g=a.kv_heads * a.maps, d=a.dim, e=a.vdim, rot=w["rot"], positions=s.positions, q_out=q,
                    q_hd=self.dp, q_norm=w["q_norm"], k_norm=w["k_norm"], eps=m.cfg.rms_eps, k_cache=self.k,
                    v_cache=self.v, slots=s.slot_mapping, maps=a.maps, bias=w.get("bias"), temp_coef=a.temp_coef,
                    temp_every=a.temp_every)
-        out = m.buffer(("o", a.out_dim), self.acc_k)
+        out = m.buffer(("o", a.out_dim), self.acc_k) if out is None else out
         # both maps' results in fp32, where the difference is not taken in the merge
         both = m.maps_buffer(self.nq * a.vdim) if a.diff is not None else out
         lam = (w["lam"], 1.0 - a.diff, m.cfg.rms_eps) if a.diff is not None else ()
         nd = s.n_decode
         kw = dict(window=a.window, keep_first=a.keep_first if a.window else 0, scale=a.scale, chunk=a.chunk,
-                  sink=-math.inf if a.sink is None else a.sink)
+                  sink=-math.inf if a.sink is None else a.sink, sinks=w.get("sinks"), out_gain=gain)
         done = 0       # rows whose difference has been taken
         if self.tc:
             if nd > 0:
@@ -173,6 +195,100 @@ class AttentionRun:
         if lam and done < M:
             hops.diff_norm(both[done:], M - done, h=a.heads, e=a.vdim, lam=lam[0], gain=lam[1], eps=lam[2], out=out[done:])
         return out[:M]
+
+
+class TalkingRun:
+    """One run of attention with talking heads: a cache of unnormed keys, which are the values, and their norms' factors."""
+
+    def __init__(self, m: "HybridModel", spec, w: dict):
+        self.m, self.spec, self.w = m, spec, w
+        a = spec
+        self.width, self.acc_k = a.in_width, round_up(a.out_dim, 64)
+        dp = talk_head(a) if m.dtype == torch.bfloat16 else 0
+        self.dp = dp or round_up(a.dim, 8)
+        self.decode_tc = dp > 0 and hops.talk_decode_ok(a.heads, a.kv_heads, dp)
+        self.prefill_tc = dp > 0 and hops.talk_prefill_ok(a.heads, dp)
+        self.cache = torch.zeros(m.num_blocks, a.kv_heads, 16, self.dp, dtype=m.dtype, device=m.device)
+        self.k_rms = torch.zeros(m.num_blocks, 16, dtype=torch.float32, device=m.device)
+        m.k_cache.append(self.cache)
+        m.v_cache.append(self.k_rms)
+
+    def __call__(self, s: StepInputs, h: torch.Tensor) -> None:
+        m, a, w, M, nd = self.m, self.spec, self.w, s.m, s.n_decode
+        proj = m.project(h, w["w_in"], self.width)
+        q = m.buffer(("q_talk", a.heads, a.dim), round_up(a.heads * self.dp, 8))
+        hops.heads(proj, M, h=a.heads, g=a.kv_heads, d=a.dim, e=a.dim, rot=w["rot"], positions=s.positions, q_out=q, q_hd=self.dp,
+                   q_norm=w["q_norm"], eps=m.cfg.rms_eps, k_cache=self.cache, slots=s.slot_mapping, k_rms=self.k_rms)
+        out = m.buffer(("o", a.out_dim), self.acc_k)
+        gate = proj[:, a.gate_col:]
+        kw = dict(h=a.heads, d=a.dim, window=a.window, scale=a.scale, cap=a.softcap, talk=w["talk"], bias=w["bias"], gate=gate, out=out)
+        if nd > 0:
+            parts = dict(pages_per_split=s.pages_per_split, part_o=m.part_o, part_ml=m.part_ml, max_splits=m.max_splits) if self.decode_tc else {}
+            hops.talk_decode(q, self.cache, self.k_rms, s.block_tables, s.seq_lens, rows=nd, **kw, **parts)
+        if s.n_prefill > 0:
+            seqs = (s.q_start, s.q_lens, s.ctx_lens)
+            span = hops.talk_span(a.window, s.max_ctx)
+            per = a.heads * 128 * span       # scores of a tile
+            step = max(1, TALK_SCORE_BYTES // (4 * per)) if self.prefill_tc else s.n_tiles
+            for t0 in range(0, s.n_tiles, step):
+                n = min(step, s.n_tiles - t0)
+                ws = dict(scores=m.scratch("talk_scores", n * per), span=span) if self.prefill_tc else {}
+                hops.talk_prefill(q, self.cache, self.k_rms, s.prefill_block_tables, s.tile_seq[t0:], s.tile_q0[t0:], *seqs, n_tiles=n,
+                                  **kw, **ws)
+        m.into_acc(out[:M], w["w_o"])
+
+
+class GruRun:
+    """One run of a gated recurrence: a state per slot."""
+
+    def __init__(self, m: "HybridModel", spec, w: dict):
+        self.m, self.spec, self.w = m, spec, w
+        self.state = torch.zeros(m.state_slots, spec.width_p, dtype=torch.float32, device=m.device)
+        m.states.append(self.state)
+
+    def mix(self, s: StepInputs, proj: torch.Tensor, out: torch.Tensor, gain: float) -> None:
+        """Projection rows z | x | g -> states times silu(g) times `gain`."""
+        m, w, nd = self.m, self.w, s.n_decode
+        kw = dict(bias=w["bias"], gain=gain, state=self.state, out=out)
+        if nd > 0:
+            hops.gru_decode(proj, nd, row_slots=s.decode_slots, positions=s.positions, **kw)
+        if s.n_prefill > 0:
+            hops.gru_prefill(proj, s.m, seq_slots=s.prefill_slots, tile_seq=s.tile_seq, tile_q0=s.tile_q0, q_start=s.q_start, q_lens=s.q_lens,
+                             ctx_lens=s.ctx_lens, n_tiles=s.n_tiles, ws=m.scratch("gru_ws", hops.gru_ws_elems(self.spec.width_p, s.n_tiles)), **kw)
+
+
+class PairRun:
+    """Attention and a gated recurrence on the same rows, their results weighted and side by side in one row, so one output
+    projection adds them up."""
+
+    def __init__(self, m: "HybridModel", spec, w: dict):
+        self.m, self.spec, self.w = m, spec, w
+        self.left, self.right = AttentionRun(m, spec.left, w["left"]), GruRun(m, spec.right, w["right"])
+        self.split, self.width = round_up(self.left.width, 64), m._in_width(spec)
+        self.lk = round_up(spec.left.out_dim, 64)
+        self.acc_k = self.lk + round_up(spec.right.out_dim, 64)
+
+    def __call__(self, s: StepInputs, h: torch.Tensor) -> None:
+        m, g = self.m, self.spec.gains
+        proj = m.project(h, self.w["w_in"], self.width)
+        out = m.buffer(("pair", self.lk, self.acc_k, self.spec.left.out_dim), self.acc_k)
+        self.left.attend(s, proj, out, g[0])
+        self.right.mix(s, proj[:, self.split:], out[:, self.lk:], g[1])
+        m.into_acc(out[:s.m], self.w["w_o"])
+
+
+class EntryRun:
+    """x <- W [x; embedding] ahead of a pass of the loop. Its input rows come from branch_norm; bf16 rows hold x in two terms."""
+
+    def __init__(self, m: "HybridModel", w: torch.Tensor):
+        self.m, self.w = m, w
+        self.acc_k = (3 if m.dtype == torch.bfloat16 else 2) * m.dp
+
+    def rows(self) -> torch.Tensor:
+        return self.m.buffer(("entry", self.acc_k), self.acc_k)
+
+    def __call__(self, s: StepInputs, h: torch.Tensor) -> None:
+        self.m.into_acc(self.rows()[:s.m], self.w)
 
 
 class LatentRun:
@@ -454,13 +570,22 @@ class MlpRun:
     def __init__(self, m: "HybridModel", spec, w: dict):
         self.m, self.spec, self.w = m, spec, w
         self.ip = self.acc_k = round_up(spec.ff, 64)
-        self.act = 1 if spec.act == "gelu_tanh" else 0
+        self.act = {"gelu_tanh": 1, "relu2": 2}.get(spec.act, 0)
 
     def __call__(self, s: StepInputs, h: torch.Tensor) -> None:
         m, M = self.m, s.m
         act = m.buffer(("act", self.ip), self.ip)
         w = self.w["w_gu"]
-        if m.dtype == torch.float32:
+        if not self.spec.glu:
+            if m.dtype == torch.float32:
+                u = m.scratch("gate_up", M * self.ip).view(M, self.ip)
+                hops.gemm_f32(h, w, u)
+                hops.glu_f32(u, act, M, self.ip, self.act)
+            elif m.few_rows(M):
+                ops.gemv(h, w, act[:M], act=self.act)
+            else:
+                ops.gemm(h, w, out=act[:M], act=self.act, **m._gemm_shape(M, self.ip, m.dp, store=True))
+        elif m.dtype == torch.float32:
             gu = m.scratch("gate_up", M * 2 * self.ip).view(M, 2 * self.ip)
             hops.gemm_f32(h, w, gu)
             hops.glu_f32(gu, act, M, self.ip, self.act)
@@ -472,7 +597,8 @@ class MlpRun:
         m.into_acc(act[:M], self.w["w_down"])
 
 
-RUNS = {"attention": AttentionRun, "retention": RetentionRun, "latent_attention": LatentRun, "mlstm": MemoryRun}
+RUNS = {"attention": AttentionRun, "retention": RetentionRun, "latent_attention": LatentRun, "mlstm": MemoryRun,
+        "talking_attention": TalkingRun, "parallel": PairRun}
 MLP_RUNS = {"dense": MlpRun, "moe": MoeRun}
 
 
@@ -524,6 +650,11 @@ class HybridModel(GemmShapes):
         if self.sandwich and (self.parallel or cfg.streams or cfg.loop or cfg.bigram or not all(L.post_norm for L in cfg.layers)):
             raise ConfigError(f"{cfg.name}: layers with a norm behind every sublayer come without hyper-connected streams, loops and "
                               "a bigram embedding, and without other layers")
+        # one residual stream that branch_norm carries from sublayer to sublayer
+        self.single = self.sandwich or cfg.residual_mult is not None
+        if cfg.residual_mult is not None and (self.parallel or self.sandwich or cfg.streams or cfg.bigram):
+            raise ConfigError(f"{cfg.name}: layers over one plain residual stream come without hyper-connected streams, a bigram embedding "
+                              "and other layers")
         moe = [L.mlp for L in cfg.layers if L.mlp is not None and L.mlp.kind == "moe"]
         if any(e.experts > hops.max_experts()[0] or e.top > hops.max_experts()[1] for e in moe):
             raise ConfigError(f"{cfg.name}: at most {hops.max_experts()[0]} experts, {hops.max_experts()[1]} of them chosen")
@@ -531,8 +662,9 @@ class HybridModel(GemmShapes):
             raise ConfigError(f"{cfg.name}: at most {hops.max_groups()} groups of experts")
         att = [p for L in cfg.layers for p in L.mixer.parts if p.kind == "attention"]
         lat = [p for L in cfg.layers for p in L.mixer.parts if p.kind == "latent_attention"]
+        talk = [p for L in cfg.layers for p in L.mixer.parts if p.kind == "talking_attention"]
         # CTAs per sequence and split of the decode attention
-        self.hkv = min([a.kv_heads for a in att] + [1 for _ in lat], default=1)
+        self.hkv = min([a.kv_heads for a in att] + [1 for _ in lat], default=1)   # (talking heads: one, their window is short)
         self.x = torch.zeros(max_tokens, self.streams, d, dtype=torch.float32, device=dev)
         self.h = torch.zeros(max_tokens, self.dp, dtype=self.dtype, device=dev)
         n_acc = 2 if self.parallel else 1
@@ -546,8 +678,9 @@ class HybridModel(GemmShapes):
         self.lm_h = torch.zeros(self.max_logits, self.dp, dtype=self.dtype, device=dev)
         self.logits_buf = torch.zeros(self.max_logits, self.vp, dtype=torch.float32, device=dev)
         self.logits = self.logits_buf[:, :cfg.vocab_size]
-        heads = max([a.heads * a.maps for a in att] + [a.heads for a in lat], default=1)
-        part = max([a.heads * a.maps * max(128, tc_head(a)) for a in att] + [a.heads * a.kv_rank for a in lat], default=128)
+        heads = max([a.heads * a.maps for a in att] + [a.heads for a in lat + talk], default=1)
+        part = max([a.heads * a.maps * max(128, tc_head(a)) for a in att] + [a.heads * a.kv_rank for a in lat] +
+                   [a.heads * talk_head(a) for a in talk], default=128)
         self.part_o = torch.zeros(max_seqs * max_splits * part, dtype=torch.float32, device=dev)
         self.part_ml = torch.zeros(max_seqs * heads * max_splits * 2, dtype=torch.float32, device=dev)
         widths = [self._in_width(L.mixer) for L in cfg.layers]
@@ -572,7 +705,7 @@ class HybridModel(GemmShapes):
     @staticmethod
     def _in_width(mix) -> int:
         if mix.kind == "parallel":
-            n = HybridModel._in_width(mix.left) + mix.right.width_p
+            n = HybridModel._in_width(mix.left) + (mix.right.width_p if mix.right.kind == "ssd" else mix.right.in_width)
             return round_up(n, 256 if n >= 2048 else 64)      # wide projections in whole tiles of the widest kind
         return round_up(mix.in_width, 64)
 
@@ -583,6 +716,9 @@ class HybridModel(GemmShapes):
         for a in (p for i in cfg.layer_runs for p in cfg.layers[i].mixer.parts):
             if a.kind == "latent_attention":
                 total += 16 * a.cache_row * size if a.kv_from is None else 0
+            elif a.kind == "talking_attention":
+                dp = (talk_head(a) if dtype == "bfloat16" else 0) or round_up(a.dim, 8)
+                total += 16 * (a.kv_heads * dp * size + 4)
             elif a.kind == "attention" and dtype == "bfloat16" and tc_head(a):
                 total += a.kv_heads * 16 * 2 * tc_head(a) * 2
             elif a.kind == "attention":
@@ -598,11 +734,12 @@ class HybridModel(GemmShapes):
         """Device bytes of a step's work space: streams, fp32 projections, rotated q / k, chunk states of
         retention, rows of the experts."""
         parts = [p for L in cfg.layers for p in L.mixer.parts]
-        wide = max(p.width_p if p.kind == "ssd" else p.heads * getattr(p, "maps", 1) * (p.dim + p.vdim) for p in parts)
+        wide = max(p.width_p if p.kind == "ssd" else p.in_width if p.kind in ("min_gru", "talking_attention") else p.heads * getattr(p, "maps", 1) * (p.dim + p.vdim) for p in parts)
         chunk = max((p.state_elems for p in parts if p.kind in ("retention", "mlstm")), default=0)
         # gathered latents, keys and values of all heads in the largest pass
         lat = max((p.cache_row + p.heads * sum(latent_layout(p)[:2]) for p in parts if p.kind == "latent_attention"), default=0)
-        n = 2 * lat * max(KV_PASS_ROWS, max_tokens) + max_tokens * 4 * (max(1, cfg.streams) * cfg.d_model + 6 * wide) + 8 * (max_tokens // 128 + max_seqs) * chunk
+        n = max((4 * p.heads * 128 * (p.window + 256) + TALK_SCORE_BYTES for p in parts if p.kind == "talking_attention"), default=0)
+        n += 2 * lat * max(KV_PASS_ROWS, max_tokens) + max_tokens * 4 * (max(1, cfg.streams) * cfg.d_model + 6 * wide) + 8 * (max_tokens // 128 + max_seqs) * chunk
         return n + max((HybridModel._moe_rows(L.mlp.experts, L.mlp.top, max_tokens) * 4 * (2 * cfg.d_model + L.mlp.ff)
                         for L in cfg.layers if L.mlp is not None and L.mlp.kind == "moe"), default=0)
 
@@ -726,6 +863,10 @@ class HybridModel(GemmShapes):
     def _mixer_weights(self, mx, p: str, mat, vec) -> dict:
         if mx.kind == "latent_attention":
             return self._latent_weights(mx, p, mat, vec)
+        if mx.kind == "talking_attention":
+            return self._talking_weights(mx, p, mat, vec)
+        if mx.kind == "parallel":
+            return self._pair_weights(mx, p, mat, vec)
         names = ("q", "k", "v") if mx.kind == "attention" else ("q", "k", "v", "g")
         w = {"w_in": self._pad(torch.cat([mat(p + n) for n in names])), "w_o": self._pad(mat(p + "o")),
              "rot": self._rotary(getattr(mx, "rot", None)), "q_norm": None, "k_norm": None}
@@ -745,6 +886,35 @@ class HybridModel(GemmShapes):
             wz[:z.shape[0], :z.shape[1]] = z
             w.update(w_z=wz, z_bias=torch.cat([vec(p + "i.b"), vec(p + "f.b")]), norm=vec(p + "norm"))
         return w
+
+    def _talking_weights(self, a, p: str, mat, vec) -> dict:
+        """The keys' norm weights are part of the queries' (fp32 products), the distance biases a table of the mixed heads."""
+        q, k, g = mat(p + "q"), mat(p + "k"), mat(p + "g")
+        w_in = q.new_zeros(a.in_width, q.shape[1])
+        w_in[:q.shape[0]], w_in[q.shape[0]:q.shape[0] + k.shape[0]], w_in[a.gate_col:] = q, k, g
+        wk = vec(p + "k.norm").view(a.kv_heads, 1, a.dim).expand(a.kv_heads, a.heads // a.kv_heads, a.dim).reshape(-1)
+        talk = vec(p + "talk").contiguous()
+        far = a.window or 16 * self.max_blocks_per_seq
+        return {"w_in": self._pad(w_in), "w_o": self._pad(mat(p + "o")), "rot": self._rotary(None), "q_norm": (vec(p + "q.norm") * wk).contiguous(),
+                "talk": talk, "bias": hops.talk_bias(talk, vec(p + "r1"), vec(p + "r2"), far)}
+
+    def _pair_weights(self, mx, p: str, mat, vec) -> dict:
+        """q | k | v of the attention, then z | x | g of the recurrence; the output matrices side by side."""
+        a, r = mx.left, mx.right
+        rows = [mat(f"{p}left.{n}") for n in ("q", "k", "v")]
+        w_in = rows[0].new_zeros(self._in_width(mx), rows[0].shape[1])
+        w_in[:a.in_width] = torch.cat(rows)
+        at, bias = round_up(a.in_width, 64), torch.zeros(2, r.width_p, dtype=torch.float32, device=self.device)
+        for i, n in enumerate(("z", "x", "g")):
+            w_in[at + i * r.width_p:at + i * r.width_p + r.width] = mat(f"{p}right.{n}")
+            if n != "g":
+                bias[i, :r.width] = vec(f"{p}right.{n}.b")
+        lo, ro = mat(p + "left.o"), mat(p + "right.o")
+        lk = round_up(a.out_dim, 64)
+        w_o = lo.new_zeros(lo.shape[0], lk + round_up(r.out_dim, 64))
+        w_o[:, :a.out_dim], w_o[:, lk:lk + r.out_dim] = lo, ro
+        return {"w_in": self._pad(w_in), "w_o": self._pad(w_o), "right": {"bias": bias.view(-1)},
+                "left": {"rot": self._rotary(a.rot), "q_norm": None, "k_norm": None, "sinks": vec(p + "left.sink")}}
 
     def _latent_weights(self, a, p: str, mat, vec) -> dict:
         """Tensors of latent attention in the head layouts of LatentRun. The expansion of a step's latents to keys takes the
@@ -779,6 +949,8 @@ class HybridModel(GemmShapes):
     def _mlp_weights(self, f, p: str, mat) -> dict:
         if f.kind == "moe":
             return self._moe_weights(f, p, mat)
+        if not f.glu:
+            return {"w_gu": self._pad(mat(p + "up")), "w_down": self._pad(mat(p + "down"))}
         ip = round_up(f.ff, 64)
         g, u = mat(p + "gate"), mat(p + "up")
         if ip != f.ff:   # whole units of the interleaved layout; act(0) * 0 adds nothing
@@ -798,6 +970,30 @@ class HybridModel(GemmShapes):
             self.sublayers.append(_NormedSublayer(*norms[0], mixer, i if L.mlp is None else -1))
             if L.mlp is not None:
                 self.sublayers.append(_NormedSublayer(*norms[1], MLP_RUNS[L.mlp.kind](self, L.mlp, self._mlp_weights(L.mlp, p + "mlp.", mat)), i))
+        torch.cuda.empty_cache()
+
+    def _build_single(self, mat, vec) -> None:
+        """Layers over one plain residual stream, with the entries of the loop's passes."""
+        cfg, m = self.cfg, self.cfg.residual_mult
+        self.k_cache, self.v_cache, self.states, self.sublayers = [], [], [], []
+        entry, starts = None, cfg.pass_starts if cfg.loop_inject else {}
+        if starts:
+            w, d = mat("loop.in"), cfg.d_model
+            x, x0 = w[:, :d], w[:, d:]
+            parts = [x, x, x0] if self.dtype == torch.bfloat16 else [x, x0]
+            wide = w.new_zeros(d, len(parts) * self.dp)
+            for i, t in enumerate(parts):
+                wide[:, i * self.dp:i * self.dp + d] = t
+            entry, step = EntryRun(self, self._pad(wide)), vec("loop.step")
+        ws = [(self._mixer_weights(L.mixer, f"l{i}.mix.", mat, vec), self._mlp_weights(L.mlp, f"l{i}.mlp.", mat) if L.mlp is not None else None,
+               [vec(f"l{i}.norm{q}") for q in range(1, L.sublayers + 1)]) for i, L in enumerate(cfg.layers)]
+        for ri, li in enumerate(cfg.layer_runs):
+            L, (w, mw, norms) = cfg.layers[li], ws[li]
+            if ri in starts:
+                self.sublayers.append(_NormedSublayer(None, None, entry, -1, base=step[starts[ri]].contiguous()))
+            self.sublayers.append(_NormedSublayer(norms[0], None, RUNS[L.mixer.kind](self, L.mixer, w), ri if mw is None else -1, gain=m))
+            if mw is not None:
+                self.sublayers.append(_NormedSublayer(norms[1], None, MLP_RUNS[L.mlp.kind](self, L.mlp, mw), ri, gain=m))
         torch.cuda.empty_cache()
 
     def _build_parallel(self, get) -> None:
@@ -834,7 +1030,9 @@ class HybridModel(GemmShapes):
         self.embed = mat("embed").contiguous()
         self.bigram = mat("bigram").contiguous() if cfg.bigram is not None else None
         self.head = self._pad(mat("embed" if cfg.tie_embeddings else "head"))
-        self.out_norm = vec("final.norm")
+        self.out_norm = vec("final.norm") * cfg.logit_scale - cfg.norm_weight_offset * (1.0 - cfg.logit_scale)
+        if cfg.residual_mult is not None:
+            return self._build_single(mat, vec)
         if self.sandwich:
             return self._build_sandwich(mat, vec)
         one = torch.ones(1, dtype=torch.float32, device=self.device)
@@ -872,7 +1070,7 @@ class HybridModel(GemmShapes):
     def init_random(self, seed: int = 0, std: float = 0.02) -> None:
         """Random weights generated on the device (benchmarks): N(0, std) matrices, unit norms, and
         hyper-connections that act as a plain residual."""
-        from .layer_spec import initial_vector, layer_list_tensors
+        from .layer_spec import initial_matrix, initial_vector, layer_list_tensors
 
         g = torch.Generator(device=self.device)
         g.manual_seed(seed)
@@ -887,7 +1085,9 @@ class HybridModel(GemmShapes):
             if len(shape) == 1:
                 return torch.from_numpy(initial_vector(self.cfg, name, shape)).to(self.device)
             t = torch.empty(*shape, dtype=torch.float32 if f32 else self.dtype, device=self.device)
-            return t.normal_(0.0, self.cfg.d_model ** -0.5 if name.endswith(".router") else std, generator=g)
+            t = t.normal_(0.0, self.cfg.d_model ** -0.5 if name.endswith(".router") else std, generator=g)
+            start = initial_matrix(name, shape)
+            return t if start is None else t + torch.from_numpy(start).to(t)
 
         self._build(get)
 
@@ -986,7 +1186,7 @@ class HybridModel(GemmShapes):
         """acc = x @ w^T (fp32). The accumulator is zero here: stream_norm clears what it has read, branch_norm where
         the next product adds its splits up."""
         M, k = x.shape
-        if acc is None and self.sandwich:
+        if acc is None and self.single:
             return self.into_branch(0, x, w)
         acc = (self.acc if acc is None else acc)[:M]
         if self.dtype == torch.float32:
@@ -1003,8 +1203,8 @@ class HybridModel(GemmShapes):
         logit rows than the buffer holds get one of their own)."""
         if self.parallel:
             return self._forward_parallel(s)
-        if self.sandwich:
-            return self._forward_sandwich(s)
+        if self.single:
+            return self._forward_single(s)
         cfg, M = self.cfg, s.m
         h = self.h[:M]
         subs = self.sublayers
@@ -1061,7 +1261,7 @@ class HybridModel(GemmShapes):
                 experts = layers[i].run(s, h, h2)
         return self._head(lm_h, logits, n_log)
 
-    def _forward_sandwich(self, s: StepInputs) -> torch.Tensor:
+    def _forward_single(self, s: StepInputs) -> torch.Tensor:
         cfg, M, subs = self.cfg, s.m, self.sublayers
         h = self.h[:M]
         x = self.x.view(self.max_tokens, -1)
@@ -1069,7 +1269,8 @@ class HybridModel(GemmShapes):
         lm_h, logits = self._logit_rows(n_log)
         experts = self.gathered = None
         for i in range(len(subs) + 1):
-            # what the sublayer before left, normed, into the residual; then the norm of this one (or of the head)
+            # what the sublayer before left into the residual (through its norm, where it has one); then the norm of this one (or
+            # of the head), or the operand rows of the entry of a pass
             last = i == len(subs)
             # the accumulator has to be zero when the next sublayer that adds its splits up in it starts
             user = next((t.run.acc_k for t in subs[i:] if t.run.acc_k), 0)
@@ -1078,10 +1279,13 @@ class HybridModel(GemmShapes):
             if i == 0:
                 kw.update(tokens=s.token_ids, embed=self.embed, embed_scale=cfg.emb_scale, branches=[(self.acc, None, 1.0, clear)])
             elif subs[i - 1].run.acc_k:
-                kw["branches"] = [(self.acc, subs[i - 1].out, 1.0, clear)]
+                kw.update(branches=[(self.acc, subs[i - 1].out, subs[i - 1].gain, clear)], base=subs[i - 1].base)
             else:
                 kw.update(branches=[(None, subs[i - 1].out, 1.0, False)], experts=experts)
-            if last:
+            if not last and subs[i].base is not None:
+                kw.update(norm_w=(), h=(), split=subs[i].run.rows(), split_off=self.dp, x0_tokens=s.token_ids, embed=self.embed,
+                          embed_scale=cfg.emb_scale)
+            elif last:
                 kw.update(norm_w=[self.out_norm], h=[lm_h], row_map=s.logit_map, store_x=self.layer_hook is not None)
             else:
                 kw.update(norm_w=[subs[i].norm], h=[h], clear=self._proj_splits(M, subs[i]))
@@ -1107,6 +1311,8 @@ class HybridModel(GemmShapes):
             ops.gemv(lm_h, self.head, logits)
         else:
             ops.gemm(lm_h, self.head, out=logits, epi=ops.EPI_STORE_F32, **self._gemm_shape(n_log, self.vp, self.dp, store=True))
+        if self.cfg.logit_softcap:
+            ops.softcap(logits, self.cfg.logit_softcap)
         return logits[:, :self.cfg.vocab_size]
 
     # ------------------------------------------------------------------ state

@@ -59,7 +59,7 @@ class AttentionSpec:
     """Softmax attention with grouped key/value heads. `window` 0: every earlier position is visible;
     else the last `window` positions and the first `keep_first` ones of the sequence (which keep their
     true positions). `chunk` (instead of a window): only positions of the same chunk, counted from position
-    0. `sink`: score of one more term of the softmax denominator that has no value. `qk_norm` "projection": RMS norm over all heads of q (of k) at once, before the
+    0. `sink`: score of one more term of the softmax denominator that has no value; `sinks`: a learned one per head. `qk_norm` "projection": RMS norm over all heads of q (of k) at once, before the
     rotation. `bias`: q, k and v have biases. `temp_coef`: q is multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1)
     at position p. `diff`: differential attention, every head has two maps over the same values (q and k hold
     [map 1, map 2] head by head); with lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff the result is a1 - lambda a2 divided
@@ -79,6 +79,7 @@ class AttentionSpec:
     temp_coef: float = 0.0
     temp_every: float = 1.0
     diff: Optional[float] = None
+    sinks: bool = False
 
     kind = "attention"
 
@@ -110,10 +111,59 @@ class AttentionSpec:
             out += [(n, (r, d))] + ([(n + ".b", (r,))] if self.bias else [])
         if self.diff is not None:
             out += [(n, (self.dim,)) for n in ("lq1", "lk1", "lq2", "lk2")]
+        if self.sinks:
+            out.append(("sink", (self.heads,)))
         out.append(("o", (d, self.out_dim)))
         if self.qk_norm == "projection":
             out += [("q.norm", (self.heads * self.dim,)), ("k.norm", (self.kv_heads * self.dim,))]
         return out
+
+
+@dataclass(frozen=True)
+class TalkingSpec:
+    """Attention whose heads mix their scores (talking heads) over one projection that is key and value: k = W_k h is the value as
+    it is and, by its RMS norm over all heads, the key; q is normed the same way. A head's score is softcap tanh(q . k scale / softcap)
+    (`softcap` 0: as it is) minus r1_h ln(1 + r2_h distance); head h goes on with sum_g talk[h, g] score_g, and a softmax over the
+    last `window` positions (0: all). The result is multiplied by sigmoid(W_g h). No rotation."""
+    heads: int
+    kv_heads: int
+    dim: int
+    scale: float
+    softcap: float = 0.0
+    window: int = 0
+
+    kind = "talking_attention"
+
+    @property
+    def parts(self) -> tuple:
+        return (self,)
+
+    @property
+    def vdim(self) -> int:
+        return self.dim
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.dim
+
+    @property
+    def gate_col(self) -> int:
+        """Column of the gate in the projection, behind q and k."""
+        return _pad16((self.heads + self.kv_heads) * self.dim)
+
+    @property
+    def in_width(self) -> int:
+        return self.gate_col + self.out_dim
+
+    @property
+    def cache_values(self) -> int:
+        """Values that a token keeps: its keys before the norm, which are its values (and one fp32 number, their norm)."""
+        return self.kv_heads * self.dim
+
+    def tensors(self, d: int) -> list[tuple[str, tuple[int, ...]]]:
+        hd, gd, h = self.out_dim, self.cache_values, self.heads
+        return [("q", (hd, d)), ("k", (gd, d)), ("q.norm", (hd,)), ("k.norm", (gd,)), ("r1", (h,)), ("r2", (h,)), ("talk", (h, h)),
+                ("g", (hd, d)), ("o", (d, hd))]
 
 
 @dataclass(frozen=True)
@@ -302,11 +352,46 @@ class SsdSpec:
 
 
 @dataclass(frozen=True)
+class GruSpec:
+    """Gated recurrence whose gates read only the current token (minGRU): z = sigmoid(W_z h + b_z), u = W_x h + b_x,
+    S <- (1 - z) S + z c(u) element by element with c(u) = u + 1/2 from 0 on and sigmoid(u) below, output S silu(W_g h)."""
+    width: int
+
+    kind = "min_gru"
+
+    @property
+    def parts(self) -> tuple:
+        return (self,)
+
+    @property
+    def out_dim(self) -> int:
+        return self.width
+
+    @property
+    def width_p(self) -> int:
+        """Columns of each of the three projections (zero channels as padding)."""
+        return _pad16(self.width)
+
+    @property
+    def in_width(self) -> int:
+        return 3 * self.width_p
+
+    @property
+    def state_elems(self) -> int:
+        return self.width_p
+
+    def tensors(self, d: int) -> list[tuple[str, tuple[int, ...]]]:
+        n = self.width
+        return [("z", (n, d)), ("z.b", (n,)), ("x", (n, d)), ("x.b", (n,)), ("g", (n, d)), ("o", (d, n))]
+
+
+@dataclass(frozen=True)
 class ParallelSpec:
-    """Two mixers side by side on the same input; the result is half the sum of the two outputs, each by its
-    own RMS norm over the model width."""
+    """Two mixers side by side on the same input. The result is half the sum of the two outputs, each by its own RMS norm
+    over the model width, or with `gains` the outputs as they are, weighted by these two numbers."""
     left: AttentionSpec
-    right: SsdSpec
+    right: Union[SsdSpec, GruSpec]
+    gains: Optional[tuple] = None
 
     kind = "parallel"
 
@@ -318,18 +403,24 @@ class ParallelSpec:
         out = []
         for side in ("left", "right"):
             out += [(f"{side}.{n}", s) for n, s in getattr(self, side).tensors(d)]
-        return out + [("left.out", (d,)), ("right.out", (d,))]
+        return out if self.gains is not None else out + [("left.out", (d,)), ("right.out", (d,))]
 
 
 @dataclass(frozen=True)
 class DenseMlpSpec:
-    """W_down (act(W_gate h) * (W_up h))."""
+    """W_down (act(W_gate h) * (W_up h)), or with `act` "relu2" W_down relu(W_up h)^2."""
     ff: int
-    act: str = "silu"          # silu | gelu_tanh
+    act: str = "silu"          # silu | gelu_tanh | relu2
 
     kind = "dense"
 
+    @property
+    def glu(self) -> bool:
+        return self.act != "relu2"
+
     def tensors(self, d: int) -> list[tuple[str, tuple[int, ...]]]:
+        if not self.glu:
+            return [("up", (self.ff, d)), ("down", (d, self.ff))]
         return [("gate", (self.ff, d)), ("up", (self.ff, d)), ("down", (d, self.ff))]
 
 
@@ -367,7 +458,7 @@ class LayerSpec:
     """`parallel`: mixer and feed-forward read the same residual stream, each through its own norm, and both are
     added to it; else the feed-forward follows the mixer. `post_norm`: a sublayer's result passes a norm of its own
     and an element-wise scale before it is added."""
-    mixer: Union[AttentionSpec, RetentionSpec, SsdSpec, ParallelSpec, LatentSpec, MemorySpec]
+    mixer: Union[AttentionSpec, RetentionSpec, SsdSpec, ParallelSpec, LatentSpec, MemorySpec, TalkingSpec]
     mlp: Union[DenseMlpSpec, MoeSpec, None]
     parallel: bool = False
     post_norm: bool = False
@@ -664,9 +755,88 @@ def zagolix_json(cfg) -> dict[str, Any]:
             "embedding": {"scale": cfg.emb_scale}, "layers": layers}
 
 
+def vokepel_attention(c: dict) -> AttentionSpec:
+    """Left mixer of a Vokepel pair: rotation of neighbouring pairs, a window, a learned sink per head."""
+    a = AttentionSpec(heads=int(c["heads"]), kv_heads=int(c["kv_heads"]), dim=int(c["dim"]), vdim=int(c["vdim"]),
+                      scale=float(c["scale"]), rot=rotary_from_json(c.get("rot"), True, int(c["dim"])),
+                      window=int((c.get("mask") or {}).get("size", 0)), sinks=True)
+    if a.heads % a.kv_heads:
+        raise ConfigError(f"{a.heads} query heads do not divide over {a.kv_heads} key/value heads")
+    return a
+
+
+def vokepel_mixer(c: dict, kind: str):
+    if kind == "attention":
+        t = TalkingSpec(int(c["heads"]), int(c["kv_heads"]), int(c["dim"]), float(c["scale"]), float(c.get("softcap") or 0.0),
+                        int((c.get("mask") or {}).get("size", 0)))
+        if t.heads % t.kv_heads:
+            raise ConfigError(f"{t.heads} query heads do not divide over {t.kv_heads} key/value heads")
+        if int(c.get("vdim", t.dim)) != t.dim:
+            raise ConfigError(f"values of {c['vdim']} cannot be keys of {t.dim}")
+        return t
+    if kind == "parallel":
+        return ParallelSpec(vokepel_attention(c["left"]), GruSpec(int(c["right"]["width"])),
+                            (float(c["left_scale"]), float(c["right_scale"])))
+    raise ConfigError(f"layer type {kind!r} is not part of this design")
+
+
+def vokepel_mlp(c: Optional[dict]) -> Optional[DenseMlpSpec]:
+    if c is None:
+        return None
+    if c.get("kind") != "dense":
+        raise ConfigError(f"feed-forward kind {c.get('kind')!r} is not part of this design")
+    return DenseMlpSpec(int(c["ff"]), act="relu2")
+
+
+def vokepel_model(layers: tuple, *, width: int, vocab: int, eps: float, residual_mult: float, loop: Optional[tuple] = None,
+                  logit_scale: float = 1.0, logit_softcap: float = 0.0, name: str = "vokepel"):
+    """ModelConfig of Vokepel layers. No tokenizer comes with the design, so there is no end-of-text id."""
+    from .config import ModelConfig
+
+    layer_runs(len(layers), loop)
+    a = layers[0].mixer.parts[0]
+    return ModelConfig(name=name, arch="vokepel", n_layers=len(layers), d_model=width, n_heads=a.heads, n_kv_heads=a.kv_heads,
+                       head_dim=a.dim, ffn_dim=max((L.mlp.ff for L in layers if L.mlp), default=0), vocab_size=vocab,
+                       max_ctx=1 << 20, rms_eps=eps, tie_embeddings=True, bos_id=-1, eos_id=-1, layers=layers, loop=loop,
+                       residual_mult=residual_mult, loop_inject=loop is not None, logit_scale=logit_scale, logit_softcap=logit_softcap)
+
+
+def vokepel_config(c: dict[str, Any]):
+    """ModelConfig of a Vokepel checkpoint from its config.json."""
+    layers = tuple(LayerSpec(vokepel_mixer(x["mixer"], x["type"]), vokepel_mlp(x.get("mlp"))) for x in c["layers"])
+    lp = c.get("loop")
+    return vokepel_model(layers, width=int(c["width"]), vocab=int(c["vocab"]), eps=float(c["norm"]["eps"]),
+                         residual_mult=float(c.get("residual_mult", 1.0)),
+                         loop=(int(lp["start"]), int(lp["stop"]), int(lp["times"])) if lp else None,
+                         logit_scale=float(c.get("logit_scale", 1.0)), logit_softcap=float(c.get("logit_softcap") or 0.0))
+
+
+def vokepel_json(cfg) -> dict[str, Any]:
+    """config.json of a Vokepel ModelConfig (inverse of vokepel_config)."""
+    layers = []
+    for L in cfg.layers:
+        m = L.mixer
+        a = m.left if m.kind == "parallel" else m
+        c: dict[str, Any] = {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim, "scale": a.scale,
+                             "mask": {"size": a.window}}
+        if m.kind == "parallel":
+            if a.rot is not None:
+                c["rot"] = {"base": a.rot.base, "dims": a.rot.dims}
+            c = {"left": c, "right": {"width": m.right.width}, "left_scale": m.gains[0], "right_scale": m.gains[1]}
+        else:
+            c["softcap"] = m.softcap
+        layers.append({"type": "parallel" if m.kind == "parallel" else "attention", "mixer": c,
+                       "mlp": None if L.mlp is None else {"kind": "dense", "ff": L.mlp.ff}})
+    out = {"architecture": "Vokepel", "vocab": cfg.vocab_size, "width": cfg.d_model, "norm": {"eps": cfg.rms_eps}, "layers": layers,
+           "residual_mult": cfg.residual_mult, "logit_scale": cfg.logit_scale, "logit_softcap": cfg.logit_softcap}
+    if cfg.loop is not None:
+        out["loop"] = dict(zip(("start", "stop", "times"), cfg.loop))
+    return out
+
+
 def initial_vector(cfg, name: str, shape: tuple):
     """Starting values of a vector (synthetic weights): unit norms (stored as the distance from one where the design
-    does so), step sizes of 0.001 to 0.1, decay rates of 1 to 16."""
+    does so), step sizes of 0.001 to 0.1, decay rates of 1 to 16, distance biases of a few slopes."""
     import numpy as np
 
     n = shape[0]
@@ -677,7 +847,13 @@ def initial_vector(cfg, name: str, shape: tuple):
         v = np.log(1.0 + 15.0 * ramp)
     elif name.endswith(".f.b"):
         v = 3.0 + 3.0 * ramp      # forget gates that keep 20 to 400 tokens
-    elif name.endswith((".b", ".lq1", ".lk1", ".lq2", ".lk2")):
+    elif name.endswith(".z.b"):
+        v = -1.0 - 5.0 * ramp     # update gates that keep 3 to 400 tokens
+    elif name.endswith(".r1"):
+        v = 2.0 ** (1.0 - 4.0 * ramp)
+    elif name.endswith(".r2"):
+        v = np.full(n, 0.25)
+    elif name.endswith((".b", ".sink", ".lq1", ".lk1", ".lq2", ".lk2")):
         v = np.zeros(n)
     elif name.endswith((".q.norm", ".k.norm", ".D")):
         v = np.ones(n)
@@ -686,12 +862,21 @@ def initial_vector(cfg, name: str, shape: tuple):
     return v.astype(np.float32)
 
 
+def initial_matrix(name: str, shape: tuple):
+    """What synthetic matrices are added to: heads that keep their scores, passes that start with the stream as it is; else None."""
+    import numpy as np
+
+    return np.eye(*shape, dtype=np.float32) if name.endswith(".talk") or name == "loop.in" else None
+
+
 def layer_list_tensors(cfg) -> list[tuple[str, tuple[int, ...]]]:
     """(name, row-major shape) of every tensor of a layer-list model."""
     d, s = cfg.d_model, cfg.streams
     out = [("embed", (cfg.vocab_size, d))]
     if cfg.bigram is not None:
         out.append(("bigram", (cfg.bigram.buckets + 1, d)))
+    if cfg.loop_inject:
+        out += [("loop.in", (d, 2 * d)), ("loop.step", (cfg.loop[2], d))]
     for i, L in enumerate(cfg.layers):
         p = f"l{i}."
         for q in range(1, L.sublayers + 1):

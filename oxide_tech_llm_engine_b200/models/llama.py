@@ -77,6 +77,7 @@ class StepInputs:
     # (first sequence, end, first tile, end, rows, pages of the longest sequence)
     kv_start: Optional[torch.Tensor] = None       # [n_prefill] int32
     kv_passes: tuple = ()
+    max_ctx: int = 0       # longest context of the step's prompts
 
 
 class QuantLinear:

@@ -64,6 +64,12 @@ def _zagolix_json(c: dict):
     return zagolix_config(c)
 
 
+def _vokepel_json(c: dict):
+    from .layer_spec import vokepel_config
+
+    return vokepel_config(c)
+
+
 ARCHITECTURES: dict[str, Architecture] = {}
 
 
@@ -76,6 +82,7 @@ register(Architecture("mixtral", _llama, _llama_cpu))
 register(Architecture("kipolix", _hybrid, _hybrid_cpu, from_json=_kipolix_json, hf_names=False))
 register(Architecture("povatar", _hybrid, _hybrid_cpu, from_json=_povatar_json, hf_names=False))
 register(Architecture("zagolix", _hybrid, _hybrid_cpu, from_json=_zagolix_json, hf_names=False))
+register(Architecture("vokepel", _hybrid, _hybrid_cpu, from_json=_vokepel_json, hf_names=False))
 
 
 def architecture(cfg) -> Architecture:

@@ -162,7 +162,13 @@ class SyntheticSource(WeightSource):
             std = 1.0 / np.sqrt(self.cfg.d_model)
         if name.endswith(".bias"):
             std = 0.01
-        return (rng.standard_normal(shape, dtype=np.float32) * std).astype(np.float32)
+        x = (rng.standard_normal(shape, dtype=np.float32) * std).astype(np.float32)
+        if self.cfg.layers:
+            from .layer_spec import initial_matrix
+
+            start = initial_matrix(name, shape)
+            x = x if start is None else x + start
+        return x
 
 
 class GgufSource(WeightSource):

@@ -440,7 +440,7 @@ def paged_decode(q, k_cache, v_cache, block_tables, seq_lens, pages_per_split, p
                  *, batch: int, max_splits: int, window: int = 0, scale: float,
                  page_ml: Optional[torch.Tensor] = None, block_mass: Optional[torch.Tensor] = None,
                  q8=None, keep_first: int = 0, out_d: int = 0, exact_p: bool = False, chunk: int = 0,
-                 sink: float = float("-inf"), diff: Sequence[float] = ()) -> None:
+                 sink: float = float("-inf"), diff: Sequence[float] = (), sinks=None, out_gain: float = 1.0) -> None:
     """Paged split-KV decode attention + merge. With `page_ml` [B, max_blocks, Hq, 2] and `block_mass`
     [B, max_blocks] (fp32) the kernels also produce the softmax probability mass per KV block, summed
     over heads: the heavy-hitter score of H2O pruning (the reference accumulates it in its decode
@@ -449,12 +449,13 @@ def paged_decode(q, k_cache, v_cache, block_tables, seq_lens, pages_per_split, p
     window, the first positions of the sequence stay visible. `out_d`: values stored per head when the
     heads are padded to D. `exact_p`: softmax weights enter the value product with 16 instead of 8 bits.
     `chunk`: instead of a window, only positions of the query's own chunk (counted from position 0) are
-    visible. `sink`: score of one more term of the softmax denominator, which has no value. `diff` = (lambda, gain, eps):
+    visible. `sink`: score of one more term of the softmax denominator, which has no value (`sinks`: fp32, one per query head).
+    `out_gain`: factor on the result. `diff` = (lambda, gain, eps):
     query heads 2i and 2i + 1 are the two maps of differential attention, the merge writes their normed difference."""
     q8t, q8d, q8s = q8 if q8 is not None else (None, None, None)
     _ext().paged_decode(q, k_cache, v_cache, block_tables, seq_lens, pages_per_split, part_o, part_ml,
                         out, batch, max_splits, window, scale, status_word(q.device) if CHECK_BOUNDS else None,
-                        page_ml, block_mass, q8t, q8d, q8s, keep_first, out_d, exact_p, chunk, sink, list(diff))
+                        page_ml, block_mass, q8t, q8d, q8s, keep_first, out_d, exact_p, chunk, sink, list(diff), sinks, out_gain)
     _bump(3 if page_ml is not None else 2)
 
 
@@ -465,12 +466,12 @@ CHECK_BOUNDS = os.environ.get("OXB_CHECKS", "0") != "0"
 
 def paged_prefill(q, k_cache, v_cache, block_tables, tile_seq, tile_q0, q_start, q_lens, ctx_lens, out,
                   *, n_tiles: int, window: int = 0, scale: float, keep_first: int = 0, out_d: int = 0,
-                  exact_p: bool = False, chunk: int = 0, sink: float = float("-inf")) -> None:
+                  exact_p: bool = False, chunk: int = 0, sink: float = float("-inf"), sinks=None, out_gain: float = 1.0) -> None:
     """Causal paged attention over ragged prefill chunks on 128-row query tiles (tcgen05 / TMEM,
     attn_prefill_tc.cu); `tile_q0` entries are multiples of 128. Options as in `paged_decode`."""
     _ext().paged_prefill_tc(q, k_cache, v_cache, block_tables, tile_seq, tile_q0, q_start, q_lens,
                             ctx_lens, out, n_tiles, window, scale, status_word(q.device), keep_first, out_d, exact_p,
-                            chunk, sink)
+                            chunk, sink, sinks, out_gain)
     _bump()
 
 
@@ -605,7 +606,8 @@ def mmvq_mixed(parts: Sequence, x, out, *, k: int, xq) -> None:
 
 def gemv(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias=None, swiglu: bool = False, act: int = 0) -> None:
     """out[:M] = x @ w^T for M <= 8 rows (single-GPU latency-mode decoding); `w` row-major or
-    tile-major. `swiglu`: w holds gate|up interleaved by 32 rows and out gets act(gate) * up."""
+    tile-major. `swiglu`: w holds gate|up interleaved by 32 rows and out gets act(gate) * up; without it `act` 2 is the
+    square of relu."""
     _ext().gemv_bf16(x, w, out, bias, swiglu, act)
     _bump()
 

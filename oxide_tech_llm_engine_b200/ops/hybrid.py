@@ -1,4 +1,5 @@
-"""Python front-ends of the layer-list kernels (``csrc/kernels/{stream_ops,mixer_ops,attn_rows,retention,ssd,moe_ops,latent,latent_decode,memory,attn_prefill_wide}.cu``).
+"""Python front-ends of the layer-list kernels (``csrc/kernels/{stream_ops,mixer_ops,attn_rows,retention,ssd,moe_ops,latent,latent_decode,memory,
+attn_prefill_wide,talking,gru}.cu``).
 
 Activations, weights and caches are bf16, or fp32 throughout; residual streams, states, norms, scores
 and angles are fp32 in both cases. As in `ops`, nothing here falls back to PyTorch.
@@ -65,11 +66,13 @@ def stream_norm(x: torch.Tensor, rows: int, *, norm_w: torch.Tensor, eps: float,
 
 def heads(proj: torch.Tensor, m: int, *, h: int, g: int, d: int, e: int, rot: Rotary, positions, q_out, q_hd: int,
           q_norm=None, k_norm=None, eps: float = 1e-5, k_scale: float = 1.0, k_out=None, k_cache=None, v_cache=None,
-          slots=None, q_pd: int = 0, maps: int = 1, bias=None, temp_coef: float = 0.0, temp_every: float = 1.0) -> None:
+          slots=None, q_pd: int = 0, maps: int = 1, bias=None, temp_coef: float = 0.0, temp_every: float = 1.0,
+          k_rms=None) -> None:
     """Projection rows q | k | v -> normed and rotated heads; k and v into the paged cache with q [M, h * q_hd], or
-    q and k to dense fp32 buffers [heads, M, d]; g = 0: queries only, q_pd columns apart (HeadsParams)."""
+    q and k to dense fp32 buffers [heads, M, d]; g = 0: queries only, q_pd columns apart (HeadsParams). `k_rms`: keys that are
+    values, the cache takes them as they are and k_rms [blocks, 16] their norm's factor."""
     hybrid_ext().heads(proj, m, h, g, d, e, q_norm, k_norm, eps, rot.hi, rot.lo, rot.interleaved, rot.gain, positions,
-                       k_scale, q_out, q_hd, k_out, k_cache, v_cache, slots, q_pd, maps, bias, temp_coef, temp_every,
+                       k_scale, q_out, q_hd, k_out, k_cache, v_cache, slots, q_pd, maps, bias, temp_coef, temp_every, k_rms,
                        ops.status_word(proj.device))
     ops._bump()
 
@@ -164,10 +167,12 @@ def memory_prefill(proj, m: int, *, h: int, d: int, e: int, z, z_bias, cap: floa
 
 def row_attention(q, q_hd: int, k_cache, v_cache, block_tables, *, n: int, h: int, d: int, e: int, window: int,
                   keep_first: int, scale: float, out, chunk: int = 0, sink: float = float("-inf"), seq_lens=None,
-                  tile_seq=None, tile_q0=None, q_start=None, q_lens=None, ctx_lens=None, o_hd: int = 0) -> None:
+                  tile_seq=None, tile_q0=None, q_start=None, q_lens=None, ctx_lens=None, o_hd: int = 0, sinks=None,
+                  out_gain: float = 1.0) -> None:
     """Softmax attention of any head size in fp32 FMAs: decode rows (seq_lens) or prompt tiles."""
     hybrid_ext().row_attention(q, q_hd, k_cache, v_cache, block_tables, seq_lens, tile_seq, tile_q0, q_start, q_lens,
-                               ctx_lens, n, h, d, e, window, keep_first, chunk, scale, sink, out, o_hd, ops.status_word(q.device))
+                               ctx_lens, n, h, d, e, window, keep_first, chunk, scale, sink, sinks, out_gain, out, o_hd,
+                               ops.status_word(q.device))
     ops._bump()
 
 
@@ -211,14 +216,17 @@ def max_groups() -> int:
 
 
 def branch_norm(x: torch.Tensor, rows: int, *, norm_w, h, eps: float, w_offset: float = 0.0, tokens=None, embed=None,
-                embed_scale: float = 1.0, branches=(), experts=None, store_x: bool = True, row_map=None, clear=None) -> None:
+                embed_scale: float = 1.0, branches=(), experts=None, store_x: bool = True, row_map=None, clear=None, base=None,
+                split=None, split_off: int = 0, x0_tokens=None) -> None:
     """Embedding or the sum of a layer's branches into the residual stream x [M, N], and its RMS norm with one weight per
     output (BranchNormParams in csrc/kernels/hybrid.cuh). `branches`: (fp32 rows, norm weight or None, gain, clear);
-    `experts`: (rows, slots, weights, chosen per row); a branch whose rows are None is their weighted sum."""
+    `experts`: (rows, slots, weights, chosen per row); a branch whose rows are None is their weighted sum. `base`: the branches
+    are added to this vector instead of the stream. `split` (instead of h): operand rows of a product over [x; embedding]."""
     rows_e, slot, weight, top = experts if experts is not None else (None, None, None, 0)
     hybrid_ext().branch_norm(x, rows, tokens, embed, embed_scale, [b[0] for b in branches], [b[1] for b in branches],
                              [b[2] for b in branches], [bool(b[3]) for b in branches], rows_e, slot, weight, top, store_x,
-                             list(norm_w), list(h), eps, w_offset, row_map, clear, ops.status_word(x.device))
+                             list(norm_w), list(h), eps, w_offset, row_map, clear, base, split, split_off, x0_tokens,
+                             ops.status_word(x.device))
     ops._bump()
 
 
@@ -264,6 +272,61 @@ def moe_rows(x, w, expert, pairs: int, *, top: int, per_pair: bool, y, act: int 
     ops._bump()
 
 
+def talk_decode_ok(h: int, g: int, dp: int) -> bool:
+    return bool(hybrid_ext().talk_decode_ok(h, g, dp))
+
+
+def talk_prefill_ok(h: int, dp: int) -> bool:
+    return bool(hybrid_ext().talk_prefill_ok(h, dp))
+
+
+def talk_span(window: int, max_ctx: int) -> int:
+    """Keys per row of a tile's scores."""
+    return int(hybrid_ext().talk_span(window, max_ctx))
+
+
+def talk_bias(talk: torch.Tensor, r1: torch.Tensor, r2: torch.Tensor, n: int) -> torch.Tensor:
+    """[heads, n] fp32: the heads' distance biases r1 ln(1 + r2 distance), mixed like their scores."""
+    t, a, b = (x.double() for x in (talk, r1, r2))
+    far = torch.arange(n, dtype=torch.float64, device=talk.device)
+    return (t @ (a[:, None] * torch.log1p(b[:, None] * far))).float().contiguous()
+
+
+def talk_decode(q, cache, k_rms, block_tables, seq_lens, *, rows: int, h: int, d: int, window: int, scale: float, cap: float, talk, bias,
+                gate, out, pages_per_split=None, part_o=None, part_ml=None, max_splits: int = 0) -> None:
+    """Decode rows of talking heads (TalkParams): split-KV and merge, or without `part_o` the kernel for any sizes."""
+    hybrid_ext().talk_decode(q, cache, k_rms, block_tables, seq_lens, pages_per_split, rows, h, d, window, scale, cap, talk, bias, gate,
+                             part_o, part_ml, max_splits, out, ops.status_word(q.device))
+    ops._bump(1 if part_o is None else 2)
+
+
+def talk_prefill(q, cache, k_rms, block_tables, tile_seq, tile_q0, q_start, q_lens, ctx_lens, *, n_tiles: int, h: int, d: int, window: int,
+                 scale: float, cap: float, talk, bias, gate, out, scores=None, span: int = 0) -> None:
+    """Prompt tiles of talking heads: mixed scores into `scores` [n_tiles, h, 128, span] fp32, then softmax and sums; without
+    `scores` the kernel for any sizes."""
+    hybrid_ext().talk_prefill(q, cache, k_rms, block_tables, tile_seq, tile_q0, q_start, q_lens, ctx_lens, n_tiles, h, d, window, scale, cap,
+                              talk, bias, gate, scores, span, out, ops.status_word(q.device))
+    ops._bump(1 if scores is None else 2)
+
+
+def gru_ws_elems(n: int, n_tiles: int) -> int:
+    return n_tiles * (1 + int(hybrid_ext().GRU_PARTS)) * 2 * n
+
+
+def gru_decode(proj, rows: int, *, bias, gain: float, state, row_slots, positions, out) -> None:
+    """Gated recurrence (GruParams), one token per row."""
+    hybrid_ext().gru_decode(proj, rows, bias, gain, state, row_slots, positions, out, ops.status_word(proj.device))
+    ops._bump()
+
+
+def gru_prefill(proj, m: int, *, bias, gain: float, state, seq_slots, tile_seq, tile_q0, q_start, q_lens, ctx_lens, n_tiles: int, ws,
+                out) -> None:
+    """Prompt tiles: what every part of a tile makes of a state, then the outputs."""
+    hybrid_ext().gru_prefill(proj, m, bias, gain, state, seq_slots, tile_seq, tile_q0, q_start, q_lens, ctx_lens, n_tiles, ws, out,
+                             ops.status_word(proj.device))
+    ops._bump(2)
+
+
 def gemm_f32(a, w, out) -> None:
     """out = a @ w^T in fp32 FMAs."""
     hybrid_ext().gemm_f32(a, w, out)
@@ -271,5 +334,6 @@ def gemm_f32(a, w, out) -> None:
 
 
 def glu_f32(gu, out, m: int, i: int, act: int) -> None:
+    """act(gate) * up, or with act 2 the square of relu of rows without a gate."""
     hybrid_ext().glu_f32(gu, out, m, i, act)
     ops._bump()
