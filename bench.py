@@ -129,6 +129,10 @@ def main() -> None:
                     help="instead of the headline workload: differential and latent attention, matrix memory and gated experts beside "
                          "the Mixtral-shaped model of equal size")
     ap.add_argument("--zagolix-size", default="", help="only this size of --zagolix")
+    ap.add_argument("--vokepel", action="store_true",
+                    help="instead of the headline workload: attention with sinks beside a gated recurrence, and talking heads, beside the "
+                         "Kipolix-shaped model of equal size")
+    ap.add_argument("--vokepel-size", default="", help="only this size of --vokepel")
     args = ap.parse_args()
     if args.kipolix and args.impl != "reference":
         from oxide_tech_llm_engine_b200.bench_hybrid import run
@@ -142,6 +146,11 @@ def main() -> None:
         return
     if args.zagolix and args.impl != "reference":
         from oxide_tech_llm_engine_b200.bench_zagolix import run
+
+        run(args, ClockSampler(0))
+        return
+    if args.vokepel and args.impl != "reference":
+        from oxide_tech_llm_engine_b200.bench_vokepel import run
 
         run(args, ClockSampler(0))
         return

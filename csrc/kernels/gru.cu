@@ -1,5 +1,7 @@
-// Gated recurrence whose gates read only the current token (minGRU, sm_100a): S <- (1 - z) S + z c, element by element, so a
-// run of tokens makes S -> a S + b of a state. Prompts: every 32-row part of a tile is walked by itself for its (a, b), then,
+// Gated recurrence whose gates read only the current token (minGRU, sm_100a): S <- (1 - z) S + z c, element by element. It is
+// computed as S + z (c - S): with 1 - z as a factor its rounding would add up over the thousands of tokens that a small z keeps.
+// A run of tokens makes S -> S + (b - d S) of a state (d = 1 - the product of all 1 - z, b: what the run makes of 0).
+// Prompts: every 32-row part of a tile is walked by itself for its (d, b), then,
 // knowing what the rows before it make of the sequence's state, walked again for the outputs; both passes are streams of the
 // projection rows. Decoding: one launch, a thread per four channels of a row. Gates, candidates and states are fp32.
 #include "../common/device_info.h"
@@ -13,7 +15,7 @@ constexpr int kTileRows = 128;
 constexpr int kPartRows = kTileRows / kGruParts;
 constexpr int kQuads = 64;   // four-channel columns per CTA
 
-// 1 - z, z and z c of one channel. FAST: hardware exponential and reciprocal (both good to about 2^-22), for rows that come
+// z and c of one channel. FAST: hardware exponential and reciprocal (both good to about 2^-22), for rows that come
 // as bf16 products.
 template <bool FAST>
 __device__ __forceinline__ float sigmoid_of(float e) {   // 1 / (1 + e)
@@ -22,13 +24,13 @@ __device__ __forceinline__ float sigmoid_of(float e) {   // 1 / (1 + e)
 template <bool FAST>
 __device__ __forceinline__ float exp_of(float x) { return FAST ? __expf(x) : expf(x); }
 template <bool FAST>
-__device__ __forceinline__ void gates(float zin, float u, float* keep, float* add) {
-  const float e = exp_of<FAST>(-fmaxf(zin, -80.f));
-  const float z = sigmoid_of<FAST>(e);
-  *keep = e * z;
-  const float c = u >= 0.f ? u + 0.5f : sigmoid_of<FAST>(exp_of<FAST>(fminf(-u, 80.f)));
-  *add = z * c;
+__device__ __forceinline__ void gates(float zin, float u, float* z, float* c) {
+  *z = sigmoid_of<FAST>(exp_of<FAST>(-fmaxf(zin, -80.f)));
+  *c = u >= 0.f ? u + 0.5f : sigmoid_of<FAST>(exp_of<FAST>(fminf(-u, 80.f)));
 }
+// a state (or a run's b) one token on; a state after a run
+__device__ __forceinline__ float step_of(float s, float z, float c) { return fmaf(z, c - s, s); }
+__device__ __forceinline__ float after(float s, float d, float b) { return s + fmaf(-d, s, b); }
 template <bool FAST>
 __device__ __forceinline__ float silu_of(float g) {
   return g * sigmoid_of<FAST>(exp_of<FAST>(fminf(-g, 80.f)));
@@ -59,9 +61,9 @@ __global__ void __launch_bounds__(128) gru_decode_kernel(const GruParams p) {
   float o[4];
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
-    float keep, add;
-    gates<FAST>(z[j] + bz[j], u[j] + bx[j], &keep, &add);
-    s[j] = fmaf(keep, s[j], add);
+    float zj, cj;
+    gates<FAST>(z[j] + bz[j], u[j] + bx[j], &zj, &cj);
+    s[j] = step_of(s[j], zj, cj);
     o[j] = s[j] * silu_of<FAST>(g[j]) * p.out_gain;
   }
   store4<float>(st, s);
@@ -86,24 +88,24 @@ __device__ __forceinline__ TileRows tile_rows(const GruParams& p, int tile) {
   t.last = q0 + kTileRows >= len;
   return t;
 }
-// (a, b) of a tile (part 0) or of one of its parts (1 ..)
+// (d, b) of a tile (part 0) or of one of its parts (1 ..)
 __device__ __forceinline__ float* ws_of(const GruParams& p, int tile, int part) {
   return p.ws + (static_cast<long long>(tile) * (1 + kGruParts) + part) * 2 * p.N;
 }
 
 // What every part and every tile makes of a state. The first tile of a sequence takes the state itself: b is the state after
-// it, a the state before it.
+// it, d the state before it.
 template <typename T, typename P>
 __global__ void __launch_bounds__(kQuads * kGruParts) gru_sums_kernel(const GruParams p) {
   constexpr bool FAST = sizeof(T) == 2;
-  __shared__ float4 s_a[kGruParts][kQuads], s_b[kGruParts][kQuads];
+  __shared__ float4 s_d[kGruParts][kQuads], s_b[kGruParts][kQuads];
   pdl_launch_dependents();
   pdl_wait();
   const int part = threadIdx.y, N = p.N, c = (blockIdx.x * kQuads + threadIdx.x) * 4, tile = blockIdx.y;
   const TileRows t = tile_rows(p, tile);
   const bool in = c < N;
   if (in) {
-    float bz[4], bx[4], a[4] = {1.f, 1.f, 1.f, 1.f}, b[4] = {};
+    float bz[4], bx[4], d[4] = {}, b[4] = {};
     load4<float>(p.bias + c, bz);
     load4<float>(p.bias + N + c, bx);
     const int r0 = part * kPartRows, r1 = min(r0 + kPartRows, t.n);
@@ -115,22 +117,22 @@ __global__ void __launch_bounds__(kQuads * kGruParts) gru_sums_kernel(const GruP
       load4_stream(pr + r * p.ld + N, u);
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        float keep, add;
-        gates<FAST>(z[j] + bz[j], u[j] + bx[j], &keep, &add);
-        a[j] *= keep;
-        b[j] = fmaf(keep, b[j], add);
+        float zj, cj;
+        gates<FAST>(z[j] + bz[j], u[j] + bx[j], &zj, &cj);
+        d[j] = step_of(d[j], zj, 1.f);
+        b[j] = step_of(b[j], zj, cj);
       }
     }
     float* w = ws_of(p, tile, 1 + part);
-    store4<float>(w + c, a);
+    store4<float>(w + c, d);
     store4<float>(w + N + c, b);
-    s_a[part][threadIdx.x] = make_float4(a[0], a[1], a[2], a[3]);
+    s_d[part][threadIdx.x] = make_float4(d[0], d[1], d[2], d[3]);
     s_b[part][threadIdx.x] = make_float4(b[0], b[1], b[2], b[3]);
   }
   __syncthreads();
   if (!in || part != 0) return;
   const bool first = tile == t.first;
-  float a[4] = {1.f, 1.f, 1.f, 1.f}, b[4] = {}, start[4] = {};
+  float d[4] = {}, b[4] = {}, start[4] = {};
   if (first && !t.fresh) {
     if (t.slot >= 0 && t.slot < p.num_slots) load4_stream(p.state + static_cast<long long>(t.slot) * N + c, start);
     else set_status_once(p.status, kStatusBadIndex);
@@ -139,16 +141,16 @@ __global__ void __launch_bounds__(kQuads * kGruParts) gru_sums_kernel(const GruP
   }
 #pragma unroll
   for (int k = 0; k < kGruParts; ++k) {
-    const float4 x = s_a[k][threadIdx.x], y = s_b[k][threadIdx.x];
-    const float xa[4] = {x.x, x.y, x.z, x.w}, ya[4] = {y.x, y.y, y.z, y.w};
+    const float4 x = s_d[k][threadIdx.x], y = s_b[k][threadIdx.x];
+    const float xd[4] = {x.x, x.y, x.z, x.w}, yb[4] = {y.x, y.y, y.z, y.w};
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      b[j] = fmaf(xa[j], b[j], ya[j]);
-      a[j] *= xa[j];
+      b[j] = after(b[j], xd[j], yb[j]);
+      d[j] = after(d[j], xd[j], xd[j]);
     }
   }
   float* w = ws_of(p, tile, 0);
-  store4<float>(w + c, first ? start : a);
+  store4<float>(w + c, first ? start : d);
   store4<float>(w + N + c, b);
 }
 
@@ -157,7 +159,7 @@ __global__ void __launch_bounds__(kQuads * kGruParts) gru_sums_kernel(const GruP
 template <typename T, typename P>
 __global__ void __launch_bounds__(kQuads * kGruParts) gru_outputs_kernel(const GruParams p) {
   constexpr bool FAST = sizeof(T) == 2;
-  __shared__ float4 s_a[kGruParts][kQuads], s_b[kGruParts][kQuads];
+  __shared__ float4 s_d[kGruParts][kQuads], s_b[kGruParts][kQuads];
   pdl_launch_dependents();
   pdl_wait();
   const int part = threadIdx.y, N = p.N, c = (blockIdx.x * kQuads + threadIdx.x) * 4, tile = blockIdx.y;
@@ -167,7 +169,7 @@ __global__ void __launch_bounds__(kQuads * kGruParts) gru_outputs_kernel(const G
   if (in) {
     const int per = (before + kGruParts - 1) / kGruParts;
     const int k0 = t.first + part * per, k1 = min(k0 + per, tile);
-    float a[4] = {1.f, 1.f, 1.f, 1.f}, b[4] = {};
+    float d[4] = {}, b[4] = {};
 #pragma unroll 4
     for (int k = k0; k < k1; ++k) {
       const float* w = ws_of(p, k, 0);
@@ -176,12 +178,12 @@ __global__ void __launch_bounds__(kQuads * kGruParts) gru_outputs_kernel(const G
       load4_stream(w + N + c, y);
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        const float xa = k == t.first ? 0.f : x[j];   // nothing comes before the first tile: b is the state after it
-        b[j] = fmaf(xa, b[j], y[j]);
-        a[j] *= xa;
+        const float xd = k == t.first ? 1.f : x[j];   // nothing comes before the first tile: b is the state after it
+        b[j] = after(b[j], xd, y[j]);
+        d[j] = after(d[j], xd, xd);
       }
     }
-    s_a[part][threadIdx.x] = make_float4(a[0], a[1], a[2], a[3]);
+    s_d[part][threadIdx.x] = make_float4(d[0], d[1], d[2], d[3]);
     s_b[part][threadIdx.x] = make_float4(b[0], b[1], b[2], b[3]);
   }
   __syncthreads();
@@ -192,10 +194,10 @@ __global__ void __launch_bounds__(kQuads * kGruParts) gru_outputs_kernel(const G
   } else {
 #pragma unroll
     for (int k = 0; k < kGruParts; ++k) {
-      const float4 x = s_a[k][threadIdx.x], y = s_b[k][threadIdx.x];
-      const float xa[4] = {x.x, x.y, x.z, x.w}, ya[4] = {y.x, y.y, y.z, y.w};
+      const float4 x = s_d[k][threadIdx.x], y = s_b[k][threadIdx.x];
+      const float xd[4] = {x.x, x.y, x.z, x.w}, yb[4] = {y.x, y.y, y.z, y.w};
 #pragma unroll
-      for (int j = 0; j < 4; ++j) s[j] = fmaf(xa[j], s[j], ya[j]);
+      for (int j = 0; j < 4; ++j) s[j] = after(s[j], xd[j], yb[j]);
     }
   }
   for (int k = 0; k < part; ++k) {
@@ -204,7 +206,7 @@ __global__ void __launch_bounds__(kQuads * kGruParts) gru_outputs_kernel(const G
     load4_stream(w + c, x);
     load4_stream(w + N + c, y);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) s[j] = fmaf(x[j], s[j], y[j]);
+    for (int j = 0; j < 4; ++j) s[j] = after(s[j], x[j], y[j]);
   }
   float bz[4], bx[4];
   load4<float>(p.bias + c, bz);
@@ -220,9 +222,9 @@ __global__ void __launch_bounds__(kQuads * kGruParts) gru_outputs_kernel(const G
     load4_stream(pr + r * p.ld + 2 * N, g);
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      float keep, add;
-      gates<FAST>(z[j] + bz[j], u[j] + bx[j], &keep, &add);
-      s[j] = fmaf(keep, s[j], add);
+      float zj, cj;
+      gates<FAST>(z[j] + bz[j], u[j] + bx[j], &zj, &cj);
+      s[j] = step_of(s[j], zj, cj);
       o[j] = s[j] * silu_of<FAST>(g[j]) * p.out_gain;
     }
     store4<T>(out + r * p.ldo, o);

@@ -248,7 +248,7 @@ struct GruParams {
   const int* q_lens;
   const int* ctx_lens;
   int n_tiles;
-  float* ws;                // [n_tiles, 1 + kGruParts, 2, N]: what a tile and its parts make of a state, S -> a S + b
+  float* ws;                // [n_tiles, 1 + kGruParts, 2, N]: what a tile and its parts make of a state, S -> S + (b - d S)
   void* out;                // [M, ldo]
   long long ldo;
   int* status;

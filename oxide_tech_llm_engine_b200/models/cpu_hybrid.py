@@ -210,7 +210,7 @@ class CpuHybridModel:
         for r0, n, ctx, _, slot in seqs:
             S = torch.zeros_like(self.states[ci][slot]) if ctx == n else self.states[ci][slot]
             for t in range(r0, r0 + n):
-                S = (1.0 - z[t]) * S + z[t] * c[t]
+                S = S + z[t] * (c[t] - S)
                 out[t] = S
             self.states[ci][slot] = S
         return (out * torch.nn.functional.silu(h @ w[p + "g"].T)) @ w[p + "o"].T
