@@ -964,7 +964,7 @@ oxb::TalkParams talk_common(const Tensor& q, const Tensor& cache, const Tensor& 
 }
 
 void talk_decode(const Tensor& q, const Tensor& cache, const Tensor& k_rms, const Tensor& block_tables, const Tensor& seq_lens,
-                 const OptTensor& pages_per_split, int64_t rows, int64_t H, int64_t D, int64_t window, double scale, double cap,
+                 int64_t rows, int64_t H, int64_t D, int64_t window, double scale, double cap,
                  const Tensor& talk, const Tensor& bias, const Tensor& gate, const OptTensor& part_o, const OptTensor& part_ml,
                  int64_t max_splits, const Tensor& out, const Tensor& status) {
   oxb::TalkParams p = talk_common(q, cache, k_rms, block_tables, rows, H, D, window, scale, cap, talk, bias, gate, out, status);
@@ -974,9 +974,8 @@ void talk_decode(const Tensor& q, const Tensor& cache, const Tensor& k_rms, cons
     check_launch(oxb::launch_talk_rows(p, dtype_code(q, "talk q"), cur_stream()), "talk_rows");
     return;
   }
-  TORCH_CHECK(dtype_code(q, "talk q") == 0 && oxb::talk_decode_ok(p.H, p.G, p.DP) && given(pages_per_split) && given(part_ml) && max_splits >= 1,
+  TORCH_CHECK(dtype_code(q, "talk q") == 0 && oxb::talk_decode_ok(p.H, p.G, p.DP) && given(part_ml) && max_splits >= 1,
               "talk_decode: sizes");
-  p.pages_per_split = i32(*pages_per_split, 1, "talk_decode pages_per_split");
   p.part_o = const_cast<float*>(f32(*part_o, rows * H * max_splits * p.DP, "talk_decode part_o"));
   p.part_ml = const_cast<float*>(f32(*part_ml, rows * H * max_splits * 2, "talk_decode part_ml"));
   p.max_splits = static_cast<int>(max_splits);

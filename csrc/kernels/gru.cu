@@ -18,22 +18,23 @@ constexpr int kQuads = 64;   // four-channel columns per CTA
 // z and c of one channel. FAST: hardware exponential and reciprocal (both good to about 2^-22), for rows that come
 // as bf16 products.
 template <bool FAST>
-__device__ __forceinline__ float sigmoid_of(float e) {   // 1 / (1 + e)
-  return FAST ? __fdividef(1.f, 1.f + e) : 1.f / (1.f + e);
-}
-template <bool FAST>
-__device__ __forceinline__ float exp_of(float x) { return FAST ? __expf(x) : expf(x); }
-template <bool FAST>
 __device__ __forceinline__ void gates(float zin, float u, float* z, float* c) {
-  *z = sigmoid_of<FAST>(exp_of<FAST>(-fmaxf(zin, -80.f)));
-  *c = u >= 0.f ? u + 0.5f : sigmoid_of<FAST>(exp_of<FAST>(fminf(-u, 80.f)));
+  if constexpr (FAST) {   // one reciprocal for both
+    const float a = 1.f + __expf(-fmaxf(zin, -40.f)), b = 1.f + __expf(fminf(-u, 40.f));
+    const float r = __fdividef(1.f, a * b);
+    *z = r * b;
+    *c = u >= 0.f ? u + 0.5f : r * a;
+  } else {
+    *z = 1.f / (1.f + expf(-fmaxf(zin, -80.f)));
+    *c = u >= 0.f ? u + 0.5f : 1.f / (1.f + expf(fminf(-u, 80.f)));
+  }
 }
 // a state (or a run's b) one token on; a state after a run
 __device__ __forceinline__ float step_of(float s, float z, float c) { return fmaf(z, c - s, s); }
 __device__ __forceinline__ float after(float s, float d, float b) { return s + fmaf(-d, s, b); }
 template <bool FAST>
 __device__ __forceinline__ float silu_of(float g) {
-  return g * sigmoid_of<FAST>(exp_of<FAST>(fminf(-g, 80.f)));
+  return FAST ? __fdividef(g, 1.f + __expf(fminf(-g, 80.f))) : g / (1.f + expf(fminf(-g, 80.f)));
 }
 
 template <typename T, typename P>

@@ -187,7 +187,6 @@ struct TalkParams {
   const float* k_rms;       // [blocks, 16]
   const int* block_tables;  // [sequences, max_blocks]
   const int* seq_lens;      // decode: [rows]
-  const int* pages_per_split;
   const int* tile_seq;      // prompt chunks: 128-row tiles
   const int* tile_q0;
   const int* q_start;

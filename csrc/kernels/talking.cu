@@ -6,9 +6,9 @@
 // first the key operand (warps take page x key head), the capped scores meet in shared memory and are mixed there in fp32
 // (lanes are positions), and then the same block is the value operand (warps own pieces of the output, [16 dims x 8 heads]).
 //
-// Prompts: the sums of all heads of a query tile do not fit an SM, the scores of a tile do. talk_scores: one CTA = 32 queries x 32
-// keys; a warp keeps the scores of 8 queries x 16 keys for all heads in registers (mma.sync; the tile of one head is too small
-// for a 128-row tcgen05 tile), mixes them with fp32 FMAs and writes them out. talk_values: softmax and sums per head from there.
+// Prompts: the sums of all heads of a query tile do not fit an SM, the scores of a tile do. talk_scores: one CTA = 16 queries, 32 keys
+// at a time; the scores of all heads (mma.sync: a head's 16 x 32 tile is too small for a 128-row tcgen05 tile) meet in shared memory,
+// are mixed as a product with the heads' matrix and written out. talk_values: softmax and sums per head from there.
 //
 // talk_rows takes any sizes in fp32 FMAs, one row per CTA.
 #include "../common/device_info.h"
@@ -139,8 +139,11 @@ __global__ void __launch_bounds__(256) talk_rows_kernel(const TalkParams p) {
 }
 
 // ---------------------------------------------------------------- decoding
-constexpr int kMaxTiles = 16;    // 16 x 8 pieces of the output per warp
+constexpr int kDecWarps = 16, kDecThreads = kDecWarps * 32;
+constexpr int kMaxTiles = 8;     // 16 x 8 pieces of the output per warp
 constexpr int kMaxHeads = 64;
+constexpr int kHeadsPerWarp = kMaxHeads / kDecWarps;
+constexpr int kMaxPages = 8;     // pages per block
 
 struct DecodeLayout {
   int pages, stages, nt, cld, tld, pld;   // pages per block, ring stages, 8-head columns per key head, row pitches
@@ -152,7 +155,7 @@ __host__ __device__ inline DecodeLayout decode_layout(int H, int G, int D) {
   l.nt = (R + 7) / 8;
   l.page_bytes = G * 16 * D * 2;
   l.pages = 32768 / l.page_bytes;
-  l.pages = l.pages < 2 ? 2 : (l.pages > 8 ? 8 : l.pages);
+  l.pages = l.pages < 2 ? 2 : (l.pages < 4 ? l.pages : (l.pages < kMaxPages ? 4 : kMaxPages));
   l.stage_bytes = l.pages * (l.page_bytes + 64);      // a page and its 16 norm factors
   const int toks = l.pages * 16;
   l.cld = H | 1;                                      // odd: lanes are positions
@@ -162,8 +165,7 @@ __host__ __device__ inline DecodeLayout decode_layout(int H, int G, int D) {
   for (;; --l.stages) {
     l.q = l.stages * l.stage_bytes;
     l.c = l.q + H * (D * 2 + 16);
-    l.t = l.c + toks * l.cld * 4;
-    l.t = (l.t + 15) / 16 * 16;
+    l.t = (l.c + toks * l.cld * 4 + 15) / 16 * 16;
     l.phi = l.t + H * l.tld * 4;
     l.plo = l.phi + H * l.pld * 2;
     l.total = l.plo + H * l.pld * 2;
@@ -173,19 +175,19 @@ __host__ __device__ inline DecodeLayout decode_layout(int H, int G, int D) {
 }
 
 template <int D>
-__global__ void __launch_bounds__(256) talk_decode_kernel(const TalkParams p) {
-  constexpr int CH = D / 8;   // 16-byte chunks per row
+__global__ void __launch_bounds__(kDecThreads) talk_decode_kernel(const TalkParams p, const DecodeLayout L, int want_splits) {
+  constexpr int CH = D / 8, MT = D / 16;   // 16-byte chunks per row, pieces of 16 dims
   extern __shared__ __align__(128) uint8_t s_raw[];
   __shared__ float s_alpha[kMaxHeads];
-  __shared__ int s_ids[2][8];
+  __shared__ int s_ids[2][kMaxPages];
   const int H = p.H, G = p.G, R = H / G, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const DecodeLayout L = decode_layout(H, G, D);
   const uint32_t s_base = smem_u32(s_raw);
   float* s_c = reinterpret_cast<float*>(s_raw + L.c);
   float* s_t = reinterpret_cast<float*>(s_raw + L.t);
   __nv_bfloat16* s_hi = reinterpret_cast<__nv_bfloat16*>(s_raw + L.phi);
   __nv_bfloat16* s_lo = reinterpret_cast<__nv_bfloat16*>(s_raw + L.plo);
-  for (int i = tid; i < H * L.tld; i += 256) s_t[i] = i % L.tld < H ? p.talk[i / L.tld * H + i % L.tld] * kLog2e : 0.f;
+  for (int h = warp; h < H; h += kDecWarps)
+    for (int g = lane; g < L.tld; g += 32) s_t[h * L.tld + g] = g < H ? p.talk[h * H + g] * kLog2e : 0.f;
   pdl_wait();  // q and the newest cache rows come from the kernel before this one
   const int seq = blockIdx.x, split = blockIdx.y, seq_len = p.seq_lens[seq];
   const int win_start = p.window > 0 && seq_len > p.window ? seq_len - p.window : 0;
@@ -194,15 +196,12 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkParams p) {
     if (tid == 0) set_status_once(p.status, kStatusBadIndex);
     n_pages = p.max_blocks;
   }
-  int pps = *p.pages_per_split;
+  // the visible pages over `want_splits` CTAs, in whole blocks
   const int first_page = win_start / 16, n_list = n_pages - first_page;
-  if (first_page > 0) {   // the host sized the splits for the whole context: spread the visible pages over as many
-    const int used = (n_pages + pps - 1) / pps;
-    pps = ((n_list + used - 1) / used + L.pages - 1) / L.pages * L.pages;
-  }
+  const int pps = ((n_list + want_splits - 1) / want_splits + L.pages - 1) / L.pages * L.pages;
   const int pg_lo = first_page + split * pps, pg_hi = min(pg_lo + pps, n_pages);
   if (pg_lo >= pg_hi || seq_len <= 0) {
-    for (int h = tid; h < H; h += 256) {
+    for (int h = tid; h < H; h += kDecThreads) {
       float* ml = p.part_ml + ((static_cast<long long>(seq) * H + h) * p.max_splits + split) * 2;
       ml[0] = -INFINITY;
       ml[1] = 0.f;
@@ -216,14 +215,15 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkParams p) {
     const int pg = pg_lo + b * L.pages + tid;
     if (tid < L.pages) s_ids[b & 1][tid] = pg < pg_hi ? block_of(p, bt, pg) : -1;
   };
-  auto issue = [&](int b) {
-    const uint32_t stage = s_base + (b % L.stages) * L.stage_bytes;
+  auto issue = [&](int b, int slot) {
+    const uint32_t stage = s_base + slot * L.stage_bytes;
     for (int pg = 0; pg < L.pages; ++pg) {
       const int id = s_ids[b & 1][pg];
       const bool in = id >= 0;
       const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(p.cache) + static_cast<long long>(in ? id : 0) * G * 16 * D;
       const uint32_t dst = stage + pg * L.page_bytes;
-      for (int c = tid; c < page_chunks; c += 256) {
+#pragma unroll 4
+      for (int c = tid; c < page_chunks; c += kDecThreads) {
         const int r = c / CH, ch = c % CH;
         cp_async16(dst + r * (D * 2) + ((ch ^ (r & 7)) << 4), src + c * 8, in);
       }
@@ -232,148 +232,166 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkParams p) {
   };
   // queries of all heads, rows D * 2 + 16 bytes apart
   const __nv_bfloat16* qp = static_cast<const __nv_bfloat16*>(p.q) + static_cast<long long>(seq) * p.q_ld;
-  for (int c = tid; c < H * CH; c += 256)
+  for (int c = tid; c < H * CH; c += kDecThreads)
     *reinterpret_cast<uint4*>(s_raw + L.q + (c / CH) * (D * 2 + 16) + (c % CH) * 16) = *reinterpret_cast<const uint4*>(qp + c * 8);
   fetch_ids(0);
   fetch_ids(1);
   __syncthreads();
   for (int b = 0; b < L.stages - 1; ++b) {
-    if (b < n_blocks) issue(b);
+    if (b < n_blocks) issue(b, b);
     cp_commit();
     __syncthreads();
     fetch_ids(b + 2);
     __syncthreads();
   }
-  float acc[kMaxTiles][4], m_run[8], l_run[8];
+  float acc[kMaxTiles][4], m_run[kHeadsPerWarp], l_run[kHeadsPerWarp];
 #pragma unroll
   for (int j = 0; j < kMaxTiles; ++j)
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
+  for (int i = 0; i < kHeadsPerWarp; ++i) {
     m_run[i] = -INFINITY;
     l_run[i] = 0.f;
   }
   const int g8 = lane >> 2, t4 = lane & 3;
-  const int n_tiles = G * L.nt * (D / 16), toks = L.pages * 16;
+  const int n_tiles = G * L.nt * MT, per_warp = (n_tiles + kDecWarps - 1) / kDecWarps, ti0 = warp * per_warp;
+  const int toks = L.pages * 16;
   const float k2 = p.cap > 0.f ? 2.f * kLog2e / p.cap : 0.f;
+  // lanes' offsets in a page: rows of the key operand, rows (positions) of the transposed value operand
+  const int kr = lane & 15, kc = lane >> 4, vr = ((lane >> 4) << 3) + (lane & 7), vc = (lane >> 3) & 1;
+  int slot = 0;
   for (int b = 0; b < n_blocks; ++b) {
     if (L.stages == 3) cp_wait<1>();
     else cp_wait<0>();
     __syncthreads();   // block b has landed; every warp is done with the block before it
-    const int nb = b + L.stages - 1;
-    if (nb < n_blocks) issue(nb);
+    const int nb = b + L.stages - 1, slot_new = slot == 0 ? L.stages - 1 : slot - 1;
+    if (nb < n_blocks) issue(nb, slot_new);
     cp_commit();
-    const uint32_t stage = s_base + (b % L.stages) * L.stage_bytes;
-    const float* s_rms = reinterpret_cast<const float*>(s_raw + (b % L.stages) * L.stage_bytes + L.pages * L.page_bytes);
+    const uint32_t stage = s_base + slot * L.stage_bytes;
+    const float* s_rms = reinterpret_cast<const float*>(s_raw + slot * L.stage_bytes + L.pages * L.page_bytes);
     // ---- scores: [16 positions x 8 heads] per page, key head and column ----
-    for (int u = warp; u < L.pages * G; u += 8) {
-      const int pg = u / G, kv = u - pg * G;
-      const uint32_t rows = stage + pg * L.page_bytes + kv * (16 * D * 2);
+    for (int pg = 0, kv = warp; pg < L.pages;) {
+      if (kv >= G) {
+        kv -= G;
+        ++pg;
+        continue;
+      }
+      const uint32_t rows = stage + pg * L.page_bytes + (kv * 16 + kr) * (D * 2);
       const float r0 = s_rms[pg * 16 + g8] * p.scale, r1 = s_rms[pg * 16 + g8 + 8] * p.scale;
       for (int nt = 0; nt < L.nt; ++nt) {
         const int hq = min(kv * R + nt * 8 + g8, H - 1);
         const uint8_t* qr = s_raw + L.q + hq * (D * 2 + 16) + t4 * 4;
-        float s[4] = {};
+        float s[2][4] = {};
 #pragma unroll
-        for (int ks = 0; ks < D / 16; ++ks) {
+        for (int ks = 0; ks < MT; ++ks) {
           uint32_t a[4];
-          const int r = lane & 15, ch = ks * 2 + (lane >> 4);
-          ldsm4(rows + r * (D * 2) + ((ch ^ (r & 7)) << 4), a);
-          mma_bf16(s, a, *reinterpret_cast<const uint32_t*>(qr + ks * 32), *reinterpret_cast<const uint32_t*>(qr + ks * 32 + 16));
+          ldsm4(rows + (((ks * 2 + kc) ^ (kr & 7)) << 4), a);
+          mma_bf16(s[ks & 1], a, *reinterpret_cast<const uint32_t*>(qr + ks * 32), *reinterpret_cast<const uint32_t*>(qr + ks * 32 + 16));
         }
-        const int lh = nt * 8 + 2 * t4, h = kv * R + lh;
-        float* c0 = s_c + (pg * 16 + g8) * L.cld + h;
+        const int lh = nt * 8 + 2 * t4;
+        float* c0 = s_c + (pg * 16 + g8) * L.cld + kv * R + lh;
         float* c1 = c0 + 8 * L.cld;
         if (lh < R) {
-          c0[0] = capped(s[0] * r0, p.cap, k2);
-          c1[0] = capped(s[2] * r1, p.cap, k2);
+          c0[0] = capped((s[0][0] + s[1][0]) * r0, p.cap, k2);
+          c1[0] = capped((s[0][2] + s[1][2]) * r1, p.cap, k2);
         }
         if (lh + 1 < R) {
-          c0[1] = capped(s[1] * r0, p.cap, k2);
-          c1[1] = capped(s[3] * r1, p.cap, k2);
+          c0[1] = capped((s[0][1] + s[1][1]) * r0, p.cap, k2);
+          c1[1] = capped((s[0][3] + s[1][3]) * r1, p.cap, k2);
         }
       }
+      kv += kDecWarps;
     }
     __syncthreads();
-    // ---- mixed scores (times log2 e) and softmax: warps take heads warp + 8 i, lanes positions ----
+    // ---- mixed scores (times log2 e) and softmax: warps take heads warp + 16 i, lanes positions ----
     const int pos0 = (pg_lo + b * L.pages) * 16;
 #pragma unroll
-    for (int rep = 0; rep < 2; ++rep) {
-      const int hb = warp + 32 * rep;
-      if (hb < H) {
-        float x[4][4];   // [positions / 32][heads]
-        float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+    for (int rep = 0; rep < kHeadsPerWarp / 2; ++rep) {   // two heads at a time
+      const int h0 = warp + 2 * kDecWarps * rep;
+      if (h0 < H) {
+        const int hs[2] = {h0, min(h0 + kDecWarps, H - 1)};
+        float x[4][2], mx[2] = {-INFINITY, -INFINITY};   // [positions / 32][heads]
 #pragma unroll
         for (int tc = 0; tc < 4; ++tc) {
-          const int tok = tc * 32 + lane, dist = seq_len - 1 - pos0 - tok;
-          const bool see = tok < toks && dist >= 0 && (p.window == 0 || dist < p.window);
-#pragma unroll
-          for (int i = 0; i < 4; ++i) x[tc][i] = 0.f;
+          x[tc][0] = x[tc][1] = -INFINITY;
           if (tc * 32 < toks) {
+            const int tok = tc * 32 + lane, dist = seq_len - 1 - pos0 - tok;
+            const bool see = tok < toks && dist >= 0 && (p.window == 0 || dist < p.window);
             const float* c = s_c + min(tok, toks - 1) * L.cld;
+            float bias[2], a[2][2] = {};
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+              bias[i] = see ? __ldg(p.bias + static_cast<long long>(hs[i]) * p.n_bias + min(dist, p.n_bias - 1)) : 0.f;
+#pragma unroll 4
             for (int g = 0; g < L.tld; g += 4) {
               float cv[4];
 #pragma unroll
               for (int e = 0; e < 4; ++e) cv[e] = g + e < H ? c[g + e] : 0.f;
 #pragma unroll
-              for (int i = 0; i < 4; ++i) {
-                const float4 t = *reinterpret_cast<const float4*>(s_t + min(hb + 8 * i, H - 1) * L.tld + g);
-                x[tc][i] = fmaf(t.x, cv[0], fmaf(t.y, cv[1], fmaf(t.z, cv[2], fmaf(t.w, cv[3], x[tc][i]))));
+              for (int i = 0; i < 2; ++i) {
+                const float4 t = *reinterpret_cast<const float4*>(s_t + hs[i] * L.tld + g);
+                a[i][0] = fmaf(t.x, cv[0], fmaf(t.y, cv[1], a[i][0]));
+                a[i][1] = fmaf(t.z, cv[2], fmaf(t.w, cv[3], a[i][1]));
               }
             }
-          }
 #pragma unroll
-          for (int i = 0; i < 4; ++i) {
-            const int h = min(hb + 8 * i, H - 1);
-            x[tc][i] = see ? x[tc][i] - kLog2e * __ldg(p.bias + static_cast<long long>(h) * p.n_bias + min(dist, p.n_bias - 1)) : -INFINITY;
-            mx[i] = fmaxf(mx[i], x[tc][i]);
+            for (int i = 0; i < 2; ++i) {
+              if (see) x[tc][i] = a[i][0] + a[i][1] - kLog2e * bias[i];
+              mx[i] = fmaxf(mx[i], x[tc][i]);
+            }
           }
         }
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const int h = hb + 8 * i;
-          if (h >= H) break;
-          const float m = fmaxf(m_run[rep * 4 + i], warp_max(mx[i])), ms = m == -INFINITY ? 0.f : m;
-          const float alpha = ex2t(m_run[rep * 4 + i] - ms);
-          float sum = 0.f;
+        for (int o = 16; o > 0; o >>= 1) {
+          mx[0] = fmaxf(mx[0], __shfl_xor_sync(0xffffffffu, mx[0], o));
+          mx[1] = fmaxf(mx[1], __shfl_xor_sync(0xffffffffu, mx[1], o));
+        }
 #pragma unroll
-          for (int tc = 0; tc < 4; ++tc) {
-            const int tok = tc * 32 + lane;
-            if (tok < toks) {
-              const float e = ex2t(x[tc][i] - ms);
-              const __nv_bfloat16 hi = __float2bfloat16(e);
-              s_hi[h * L.pld + tok] = hi;
-              s_lo[h * L.pld + tok] = __float2bfloat16(e - __bfloat162float(hi));
-              sum += e;
+        for (int i = 0; i < 2; ++i) {
+          const int h = h0 + kDecWarps * i;
+          if (h < H) {
+            const float m = fmaxf(m_run[rep * 2 + i], mx[i]), ms = m == -INFINITY ? 0.f : m;
+            const float alpha = ex2t(m_run[rep * 2 + i] - ms);
+            float sum = 0.f;
+#pragma unroll
+            for (int tc = 0; tc < 4; ++tc) {
+              const int tok = tc * 32 + lane;
+              if (tok < toks) {
+                const float e = ex2t(x[tc][i] - ms);
+                const __nv_bfloat16 hi = __float2bfloat16(e);
+                s_hi[h * L.pld + tok] = hi;
+                s_lo[h * L.pld + tok] = __float2bfloat16(e - __bfloat162float(hi));
+                sum += e;
+              }
             }
+            m_run[rep * 2 + i] = m;
+            l_run[rep * 2 + i] = l_run[rep * 2 + i] * alpha + sum;   // of this lane's positions
+            if (lane == 0) s_alpha[h] = alpha;
           }
-          m_run[rep * 4 + i] = m;
-          l_run[rep * 4 + i] = l_run[rep * 4 + i] * alpha + sum;   // of this lane's positions
-          if (lane == 0) s_alpha[h] = alpha;
         }
       }
     }
     fetch_ids(nb + 1);   // (the ids of block nb have been read)
     __syncthreads();
-    // ---- sums: warps own tiles of [16 dims x 8 heads] ----
+    // ---- sums: warps own tiles of [16 dims x 8 heads], one after the other ----
 #pragma unroll
     for (int j = 0; j < kMaxTiles; ++j) {
-      const int ti = warp + 8 * j;
-      if (ti < n_tiles) {
-        const int mt = ti % (D / 16), gn = ti / (D / 16), kv = gn / L.nt, nt = gn - kv * L.nt;
-        const int h0 = kv * R + nt * 8, left = R - nt * 8;
-        const float a0 = s_alpha[min(h0 + 2 * t4, H - 1)], a1 = s_alpha[min(h0 + 2 * t4 + 1, H - 1)];
+      const int ti = ti0 + j;
+      if (j < per_warp && ti < n_tiles) {
+        const int mt = ti % MT, gn = ti / MT, kv = L.nt == 1 ? gn : gn / L.nt, nt = gn - kv * L.nt;
+        const int hb = kv * R + nt * 8, left = R - nt * 8;
+        const float a0 = s_alpha[min(hb + 2 * t4, H - 1)], a1 = s_alpha[min(hb + 2 * t4 + 1, H - 1)];
         acc[j][0] *= a0;
         acc[j][1] *= a1;
         acc[j][2] *= a0;
         acc[j][3] *= a1;
         const bool on = g8 < left;
-        const int pr = (h0 + (on ? g8 : 0)) * L.pld + 2 * t4;
+        const int pr = (hb + (on ? g8 : 0)) * L.pld + 2 * t4;
+        const uint32_t rows = stage + (kv * 16 + vr) * (D * 2) + (((mt * 2 + vc) ^ (vr & 7)) << 4);
         for (int pg = 0; pg < L.pages; ++pg) {
           uint32_t a[4];
-          const int r = ((lane >> 4) << 3) + (lane & 7), ch = mt * 2 + ((lane >> 3) & 1);
-          ldsm4t(stage + pg * L.page_bytes + kv * (16 * D * 2) + r * (D * 2) + ((ch ^ (r & 7)) << 4), a);
+          ldsm4t(rows + pg * L.page_bytes, a);
           const uint32_t* hi = reinterpret_cast<const uint32_t*>(s_hi + pr + pg * 16);
           const uint32_t* lo = reinterpret_cast<const uint32_t*>(s_lo + pr + pg * 16);
           mma_bf16(acc[j], a, on ? hi[0] : 0u, on ? hi[4] : 0u);
@@ -381,15 +399,16 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkParams p) {
         }
       }
     }
+    slot = slot + 1 == L.stages ? 0 : slot + 1;
   }
   cp_wait<0>();
   pdl_launch_dependents();
   const long long part0 = static_cast<long long>(seq) * H;
 #pragma unroll
   for (int j = 0; j < kMaxTiles; ++j) {
-    const int ti = warp + 8 * j;
-    if (ti < n_tiles) {
-      const int mt = ti % (D / 16), gn = ti / (D / 16), kv = gn / L.nt, nt = gn - kv * L.nt;
+    const int ti = ti0 + j;
+    if (j < per_warp && ti < n_tiles) {
+      const int mt = ti % MT, gn = ti / MT, kv = gn / L.nt, nt = gn - kv * L.nt;
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int lh = nt * 8 + 2 * t4 + (e & 1), d = mt * 16 + g8 + (e >> 1) * 8;
@@ -398,8 +417,8 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkParams p) {
     }
   }
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
-    const int h = warp + 8 * (i & 3) + 32 * (i >> 2);
+  for (int i = 0; i < kHeadsPerWarp; ++i) {
+    const int h = warp + kDecWarps * i;
     const float l = warp_sum(l_run[i]);
     if (h < H && lane == 0) {
       float* ml = p.part_ml + ((part0 + h) * p.max_splits + split) * 2;
@@ -433,9 +452,11 @@ __global__ void __launch_bounds__(D) talk_merge_kernel(const TalkParams p) {
 
 // ---------------------------------------------------------------- prompts
 constexpr int kTile = 128;   // query rows of the scheduler's tiles
-constexpr int kSub = 32;     // queries and keys of a scores CTA
+constexpr int kKeys = 32;    // keys of a block
+constexpr int kQ = 16;       // queries of a scores CTA
+constexpr int kBlocks = 4;   // blocks of keys that a scores CTA walks
 
-// What a 32-query piece of a tile sees: positions of its first and last row, first visible key.
+// What a piece of a tile's rows sees: positions of its first and last row, first visible key.
 struct Piece {
   int seq, len, pos0, pos1, row0, lo;
 };
@@ -451,188 +472,185 @@ __device__ __forceinline__ Piece piece_of(const TalkParams& p, int tile, int q, 
   return x;
 }
 // first key of a tile's row of scores
-__device__ __forceinline__ int first_key(const TalkParams& p, int tile) { return piece_of(p, tile, 0, kTile).lo / kSub * kSub; }
+__device__ __forceinline__ int first_key(const TalkParams& p, int tile) { return piece_of(p, tile, 0, kTile).lo / kKeys * kKeys; }
 
-__device__ __forceinline__ void fma2(float2& d, float2 a, float2 b) {
-  asm("fma.rn.f32x2 %0, %1, %2, %0;"
-      : "+l"(reinterpret_cast<unsigned long long&>(d))
-      : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)));
-}
+// Row pitch of a head's scores in shared memory, and of a query's keys inside: a warp's stores (8 keys x 4 queries) and its
+// reads (4 heads, two apart, x 8 keys) both touch 32 banks.
+constexpr int kQPitch = kKeys + 4, kHPitch = kQ * kQPitch + 4;
+static_assert(kHPitch % 16 == 4, "banks");
+constexpr int kBiasPitch = 72;
 
-// HM: heads of this instantiation (H <= HM)
+// HM: heads of this instantiation, 16 or 32 (H <= HM). 8 warps = 4 sets of heads x 2 halves of the keys: a warp multiplies 16 keys
+// x 16 queries for the heads of its set, operands straight from memory (16-byte pieces, the same permutation of the dimensions in q
+// and k). Then the scores of all heads are mixed as a product with the matrix T: 8 keys of a query are the columns, T is bf16 and
+// exact, and the fp32 scores enter as three bf16 terms that carry all their bits.
 template <int D, int HM>
-__global__ void __launch_bounds__(256, HM <= 16 ? 2 : 1) talk_scores_kernel(const TalkParams p) {
-  constexpr int CH = D / 8, kBlk = kSub * D * 2;
-  constexpr int kRing = 4;
+__global__ void __launch_bounds__(256, 2) talk_scores_kernel(const TalkParams p) {
+  constexpr int CPL = D / 32;   // 16-byte pieces of a row per lane
+  constexpr int HT = HM / 16;
   extern __shared__ __align__(128) uint8_t s_raw[];
-  uint8_t* s_q = s_raw;                    // ring of heads: [32 queries x D]
-  uint8_t* s_k = s_raw + kRing * kBlk;     // ring of key heads: [32 keys x D]
-  float2* s_t = reinterpret_cast<float2*>(s_raw + 2 * kRing * kBlk);   // [H][HM], every factor twice, times log2 e
-  float* s_b = reinterpret_cast<float*>(s_t + p.H * HM);               // [H][64]: bias by distance; +inf hides a key
-  __shared__ float s_r[kSub];
-  const int H = p.H, R = H / p.G, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  for (int i = tid; i < H * HM; i += 256) {
-    const float t = i % HM < H ? p.talk[i / HM * H + i % HM] * kLog2e : 0.f;
-    s_t[i] = make_float2(t, t);
-  }
+  float* s_c = reinterpret_cast<float*>(s_raw);   // [HM][kQ][keys]
+  float* s_b = s_c + HM * kHPitch;                // [H][distances]: bias times log2 e; +inf hides a key
+  float* s_r = s_b + p.H * kBiasPitch;            // [keys] norm factors times the scale
+  const int H = p.H, R = H / p.G, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
+  uint32_t ta[HT][HT][4];   // T as the left operand
+#pragma unroll
+  for (int m = 0; m < HT; ++m)
+#pragma unroll
+    for (int k = 0; k < HT; ++k)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int h = m * 16 + g8 + (i & 1) * 8, g = k * 16 + 2 * t4 + (i >> 1) * 8;
+        ta[m][k][i] = pack_bf16x2(h < H && g < H ? p.talk[h * H + g] : 0.f, h < H && g + 1 < H ? p.talk[h * H + g + 1] : 0.f);
+      }
+  for (int i = tid; i < (HM - H) * kHPitch; i += 256) s_c[H * kHPitch + i] = 0.f;
   pdl_wait();
-  const int tile = blockIdx.z, q_in = blockIdx.y * kSub;
-  const Piece x = piece_of(p, tile, q_in, kSub);
+  const int tile = blockIdx.z, q_in = blockIdx.y * kQ;
+  const Piece x = piece_of(p, tile, q_in, kQ);
   if (p.tile_q0[tile] + q_in >= x.len) return;
-  const int k_start = first_key(p, tile), k0 = k_start + blockIdx.x * kSub;
-  if (k0 > x.pos1 || k0 + kSub <= x.lo) return;
+  const int k_start = first_key(p, tile);
   const int* bt = p.block_tables + static_cast<long long>(x.seq) * p.max_blocks;
-  const int ctx = p.ctx_lens[x.seq], pg0 = k0 >> 4, n_pg = (ctx + 15) >> 4;
-  const int id0 = block_of(p, bt, pg0), id1 = pg0 + 1 < n_pg ? block_of(p, bt, pg0 + 1) : -1;
-  const __nv_bfloat16* qp = static_cast<const __nv_bfloat16*>(p.q) + static_cast<long long>(x.row0) * p.q_ld;
+  const int n_pg = (p.ctx_lens[x.seq] + 15) >> 4;
   const int n_q = x.pos1 - x.pos0 + 1;
-  auto issue = [&](int h) {
-    if (h < H) {
-      const uint32_t dq = smem_u32(s_q) + (h & (kRing - 1)) * kBlk;
-#pragma unroll
-      for (int i = 0; i < kSub * CH / 256; ++i) {
-        const int c = tid + i * 256, r = c / CH, ch = c % CH;
-        const bool in = r < n_q;
-        cp_async16(dq + r * (D * 2) + ((ch ^ (r & 7)) << 4), qp + (in ? r : 0) * p.q_ld + h * D + ch * 8, in);
-      }
-      if (h % R == 0) {
-        const int kv = h / R;
-        const uint32_t dk = smem_u32(s_k) + (kv & (kRing - 1)) * kBlk;
-#pragma unroll
-        for (int i = 0; i < kSub * CH / 256; ++i) {
-          const int c = tid + i * 256, r = c / CH, ch = c % CH, id = r < 16 ? id0 : id1;
-          const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(p.cache) + (static_cast<long long>(max(id, 0)) * p.G + kv) * 16 * D;
-          cp_async16(dk + r * (D * 2) + ((ch ^ (r & 7)) << 4), src + (r & 15) * D + ch * 8, id >= 0);
-        }
-      }
-    }
-    cp_commit();
-  };
-#pragma unroll
-  for (int h = 0; h < kRing - 1; ++h) issue(h);
-  if (tid < kSub) {
-    const int id = tid < 16 ? id0 : id1;
-    s_r[tid] = id >= 0 ? p.k_rms[id * 16ll + (tid & 15)] * p.scale : 0.f;
-  }
-  const int far0 = x.pos0 - k0 - 31;   // distance of bias entry 0
-  for (int i = tid; i < H * 64; i += 256) {
-    const int dist = far0 + (i & 63);
-    const bool see = dist >= 0 && (p.window == 0 || dist < p.window);
-    s_b[i] = see ? kLog2e * __ldg(p.bias + static_cast<long long>(i >> 6) * p.n_bias + min(dist, p.n_bias - 1)) : INFINITY;
-  }
-  const int kh = warp & 1, qo = warp >> 1, g8 = lane >> 2, t4 = lane & 3;   // 16 keys, 8 queries of this warp
+  const int half = warp & 1, hc = (H + 3) / 4, h_lo = (warp >> 1) * hc, h_hi = min(h_lo + hc, H);
   const float k2 = p.cap > 0.f ? 2.f * kLog2e / p.cap : 0.f;
-  float2 c[HM][2];   // scores: (key g8 | key g8 + 8) x (queries 2 t4, 2 t4 + 1)
-  uint32_t kf[D / 16][4];
-  float r0 = 0.f, r1 = 0.f;
-#pragma unroll
-  for (int h = 0; h < HM; ++h) {
-    c[h][0] = c[h][1] = make_float2(0.f, 0.f);
-    if (h < H) {
-      cp_wait<kRing - 2>();
-      __syncthreads();   // head h has landed; every warp is done with head h - 1
-      issue(h + kRing - 1);
-      if (h == 0) {
-        r0 = s_r[kh * 16 + g8];
-        r1 = s_r[kh * 16 + g8 + 8];
+  const __nv_bfloat16* q0 = static_cast<const __nv_bfloat16*>(p.q) + (static_cast<long long>(x.row0) + min(g8, n_q - 1)) * p.q_ld + t4 * 8;
+  const __nv_bfloat16* q1 = static_cast<const __nv_bfloat16*>(p.q) + (static_cast<long long>(x.row0) + min(g8 + 8, n_q - 1)) * p.q_ld + t4 * 8;
+  bool first = true;
+  for (int blk = 0; blk < kBlocks; ++blk) {
+    const int kb = blockIdx.x * kBlocks + blk, k0 = k_start + kb * kKeys;
+    if (k0 > x.pos1) break;
+    if (k0 + kKeys <= x.lo) continue;
+    if (!first) __syncthreads();   // every warp is done with the block before
+    first = false;
+    const int pg = (k0 >> 4) + half;
+    const int id = pg < n_pg ? block_of(p, bt, pg) : -1;
+    if (lane < 16 && (warp >> 1) == 0) s_r[half * 16 + lane] = id >= 0 ? p.k_rms[id * 16ll + lane] * p.scale : 0.f;
+    const int far0 = x.pos0 - k0 - (kKeys - 1);   // distance of bias entry 0
+    for (int h = warp; h < H; h += 8)
+      for (int i = lane; i < kKeys + kQ - 1; i += 32) {
+        const int dist = far0 + i;
+        const bool see = dist >= 0 && (p.window == 0 || dist < p.window);
+        s_b[h * kBiasPitch + i] = see ? kLog2e * __ldg(p.bias + static_cast<long long>(h) * p.n_bias + min(dist, p.n_bias - 1)) : INFINITY;
       }
-      if (h % R == 0) {
-        const uint32_t kb = smem_u32(s_k) + ((h / R) & (kRing - 1)) * kBlk;
+    __syncthreads();
+    // ---- scores of this warp's heads: [16 keys x 16 queries] ----
+    const float r0 = s_r[half * 16 + g8], r1 = s_r[half * 16 + g8 + 8];
+    uint4 ka[2][CPL];
+    int kv_have = -1;
+    for (int h = h_lo; h < h_hi; ++h) {
+      const int kv = h / R;
+      if (kv != kv_have) {
+        kv_have = kv;
+        const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(p.cache) + (static_cast<long long>(max(id, 0)) * p.G + kv) * 16 * D + t4 * 8;
 #pragma unroll
-        for (int ks = 0; ks < D / 16; ++ks) {
-          const int r = kh * 16 + (lane & 15), ch = ks * 2 + (lane >> 4);
-          ldsm4(kb + r * (D * 2) + ((ch ^ (r & 7)) << 4), kf[ks]);
-        }
+        for (int r = 0; r < 2; ++r)
+#pragma unroll
+          for (int c = 0; c < CPL; ++c) ka[r][c] = *reinterpret_cast<const uint4*>(kp + (g8 + 8 * r) * D + c * 32);
       }
-      const uint32_t qb = smem_u32(s_q) + (h & (kRing - 1)) * kBlk;
+      uint4 qb[2][CPL];
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) {
+        qb[0][c] = *reinterpret_cast<const uint4*>(q0 + h * D + c * 32);
+        qb[1][c] = *reinterpret_cast<const uint4*>(q1 + h * D + c * 32);
+      }
       float s[2][4] = {};
 #pragma unroll
-      for (int k2s = 0; k2s < D / 32; ++k2s) {
-        uint32_t b[4];
-        const int r = qo * 8 + (lane & 7), ch = k2s * 4 + (lane >> 3);
-        ldsm4(qb + r * (D * 2) + ((ch ^ (r & 7)) << 4), b);
-        mma_bf16(s[0], kf[2 * k2s], b[0], b[1]);
-        mma_bf16(s[1], kf[2 * k2s + 1], b[2], b[3]);
+      for (int c = 0; c < CPL; ++c)
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          mma_bf16(s[n], ka[0][c].x, ka[1][c].x, ka[0][c].y, ka[1][c].y, qb[n][c].x, qb[n][c].y);
+          mma_bf16(s[n], ka[0][c].z, ka[1][c].z, ka[0][c].w, ka[1][c].w, qb[n][c].z, qb[n][c].w);
+        }
+      float* d = s_c + h * kHPitch + 2 * t4 * kQPitch + half * 16 + g8;
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          d[(n * 8 + (e & 1)) * kQPitch + (e >> 1) * 8] = capped(s[n][e] * (e < 2 ? r0 : r1), p.cap, k2);
+    }
+    __syncthreads();
+    // ---- mixed scores: a warp takes two queries, 8 keys at a time ----
+#pragma unroll
+    for (int it = 0; it < 2 * kKeys / 8; ++it) {
+      const int q = warp * 2 + it / (kKeys / 8), k8 = it % (kKeys / 8) * 8;
+      const float* src = s_c + 2 * t4 * kHPitch + q * kQPitch + k8 + g8;
+      float o[HT][4] = {};
+#pragma unroll
+      for (int k = 0; k < HT; ++k) {
+        const float* f = src + k * 16 * kHPitch;
+        uint32_t b0[3], b1[3];
+        split3(f[0], f[kHPitch], b0);
+        split3(f[8 * kHPitch], f[9 * kHPitch], b1);
+#pragma unroll
+        for (int t = 2; t >= 0; --t)   // small terms first
+#pragma unroll
+          for (int m = 0; m < HT; ++m) mma_bf16(o[m], ta[m][k], b0[t], b1[t]);
       }
+      const int bi = kKeys - 1 + q - k8 - 2 * t4;   // bias entry of the lane's first key; the second one is one nearer
+      float* dst = p.scores + ((static_cast<long long>(tile) * H) * kTile + q_in + q) * p.span + kb * kKeys + k8 + 2 * t4;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) s[0][e] = capped((s[0][e] + s[1][e]) * (e < 2 ? r0 : r1), p.cap, k2);
-      c[h][0] = make_float2(s[0][0], s[0][1]);
-      c[h][1] = make_float2(s[0][2], s[0][3]);
-    }
-  }
-  cp_wait<0>();
-  const int key = kh * 16 + g8, q = qo * 8 + 2 * t4;
-  float* dst = p.scores + (static_cast<long long>(tile) * H * kTile + q_in + q) * p.span + (k0 - k_start) + key;
-  const int bi = 31 + q - key;
-  for (int h = 0; h < H; ++h) {
-    const float4* t = reinterpret_cast<const float4*>(s_t + h * HM);
-    float2 a[2][2] = {};
+      for (int m = 0; m < HT; ++m)
 #pragma unroll
-    for (int g = 0; g < HM; g += 2) {
-      const float4 f = t[g >> 1];
-      const float2 f0 = make_float2(f.x, f.y), f1 = make_float2(f.z, f.w);
-      fma2(a[0][0], c[g][0], f0);
-      fma2(a[0][1], c[g][1], f0);
-      fma2(a[1][0], c[g + 1][0], f1);
-      fma2(a[1][1], c[g + 1][1], f1);
+        for (int r = 0; r < 2; ++r) {
+          const int h = m * 16 + g8 + 8 * r;
+          if (h < H) {
+            const float* bb = s_b + h * kBiasPitch + bi;
+            *reinterpret_cast<float2*>(dst + static_cast<long long>(h) * kTile * p.span) =
+                make_float2(fmaf(o[m][2 * r], kLog2e, -bb[0]), fmaf(o[m][2 * r + 1], kLog2e, -bb[-1]));
+          }
+        }
     }
-    const float* bb = s_b + h * 64 + bi;
-    float* d = dst + static_cast<long long>(h) * kTile * p.span;
-    d[0] = a[0][0].x + a[1][0].x - bb[0];
-    d[p.span] = a[0][0].y + a[1][0].y - bb[1];
-    d[8] = a[0][1].x + a[1][1].x - bb[-8];
-    d[p.span + 8] = a[0][1].y + a[1][1].y - bb[-7];
   }
 }
 
 constexpr int kValueRows = 64;   // query rows of a values CTA: 4 warps of 16
+constexpr int kValueRing = 4;
 
 template <int D>
-__global__ void __launch_bounds__(128) talk_values_kernel(const TalkParams p) {
-  constexpr int CH = D / 8, kBlk = kSub * D * 2, kRing = 4;
+__global__ void __launch_bounds__(128, D == 64 ? 4 : 3) talk_values_kernel(const TalkParams p) {
+  constexpr int CH = D / 8, kBlk = kKeys * D * 2, kScr = 16 * kKeys * 4, kRing = kValueRing;
   extern __shared__ __align__(128) uint8_t s_raw[];
   pdl_wait();
   const int head = blockIdx.x, tile = blockIdx.z, q_in = blockIdx.y * kValueRows, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const Piece x = piece_of(p, tile, q_in, kValueRows);
   if (p.tile_q0[tile] + q_in >= x.len) return;
   const int k_start = first_key(p, tile), H = p.H, kv = head / (H / p.G);
-  const int b0 = (x.lo - k_start) / kSub, n_blk = (x.pos1 - k_start) / kSub + 1 - b0;   // 32-key blocks that some row sees
+  const int b0 = (x.lo - k_start) / kKeys, n_blk = (x.pos1 - k_start) / kKeys + 1 - b0;   // blocks that some row sees
   const int* bt = p.block_tables + static_cast<long long>(x.seq) * p.max_blocks;
   const int n_pg = (p.ctx_lens[x.seq] + 15) >> 4;
+  // blocks whose scores exist for this warp's rows
+  const int qw = q_in + warp * 16;
+  const Piece y = piece_of(p, tile, qw, 16);
+  const bool rows = p.tile_q0[tile] + qw < x.len;
+  const int w0 = rows ? (y.lo - k_start) / kKeys - b0 : 1 << 30, w1 = rows ? (y.pos1 - k_start) / kKeys - b0 : -1;
+  const uint32_t sv = smem_u32(s_raw), ss = sv + kRing * kBlk + warp * kRing * kScr;   // values of the CTA, scores of the warp
+  const float* sp = p.scores + ((static_cast<long long>(tile) * H + head) * kTile + qw) * p.span + b0 * kKeys;
   auto issue = [&](int i) {
     if (i < n_blk) {
       const int pg0 = (k_start >> 4) + (b0 + i) * 2;
-      const uint32_t dst = smem_u32(s_raw) + (i & (kRing - 1)) * kBlk;
+      const uint32_t dst = sv + (i & (kRing - 1)) * kBlk;
+      const int ids[2] = {pg0 < n_pg ? block_of(p, bt, pg0) : -1, pg0 + 1 < n_pg ? block_of(p, bt, pg0 + 1) : -1};
 #pragma unroll
-      for (int k = 0; k < kSub * CH / 128; ++k) {
-        const int c = tid + k * 128, r = c / CH, ch = c % CH, pg = pg0 + (r >> 4);
-        const bool in = pg < n_pg;
-        const int id = in ? block_of(p, bt, pg) : 0;
+      for (int k = 0; k < kKeys * CH / 128; ++k) {
+        const int c = tid + k * 128, r = c / CH, ch = c % CH, id = ids[k * 128 / CH >= 16 ? 1 : 0];
         cp_async16(dst + r * (D * 2) + ((ch ^ (r & 7)) << 4),
-                   static_cast<const __nv_bfloat16*>(p.cache) + ((static_cast<long long>(id) * p.G + kv) * 16 + (r & 15)) * D + ch * 8, in);
+                   static_cast<const __nv_bfloat16*>(p.cache) + ((static_cast<long long>(max(id, 0)) * p.G + kv) * 16 + (r & 15)) * D + ch * 8, id >= 0);
+      }
+      if (i >= w0 && i <= w1) {   // 16 rows of 32 scores, 16-byte pieces
+        const uint32_t d = ss + (i & (kRing - 1)) * kScr;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const int r = k * 4 + (lane >> 3), ch = lane & 7;
+          cp_async16(d + r * 128 + ((ch ^ (r & 7)) << 4), sp + static_cast<long long>(r) * p.span + i * kKeys + ch * 4, true);
+        }
       }
     }
     cp_commit();
   };
 #pragma unroll
   for (int i = 0; i < kRing - 1; ++i) issue(i);
-  // blocks whose scores exist for this warp's rows
-  const int qw = q_in + warp * 16;
-  const Piece y = piece_of(p, tile, qw / kSub * kSub, kSub);
-  const bool rows = p.tile_q0[tile] + qw < x.len;
-  const int w0 = rows ? (y.lo - k_start) / kSub - b0 : 1 << 30, w1 = rows ? (y.pos1 - k_start) / kSub - b0 : -1;
   const int g8 = lane >> 2, t4 = lane & 3;
-  const float* sp = p.scores + ((static_cast<long long>(tile) * H + head) * kTile + qw + g8) * p.span + b0 * kSub + 2 * t4;
-  float2 nxt[2][4];
-  auto load = [&](int i) {
-    if (i >= w0 && i <= w1) {
-#pragma unroll
-      for (int r = 0; r < 2; ++r)
-#pragma unroll
-        for (int j = 0; j < 4; ++j) nxt[r][j] = __ldcs(reinterpret_cast<const float2*>(sp + r * 8ll * p.span + i * kSub + j * 8));
-    }
-  };
-  load(0);
   float o[D / 8][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
 #pragma unroll
   for (int i = 0; i < D / 8; ++i)
@@ -642,32 +660,31 @@ __global__ void __launch_bounds__(128) talk_values_kernel(const TalkParams p) {
     cp_wait<kRing - 2>();
     __syncthreads();
     issue(i + kRing - 1);
-    if (i < w0 || i > w1) {
-      load(i + 1);
-      continue;
-    }
-    float2 s[2][4];
-#pragma unroll
-    for (int r = 0; r < 2; ++r)
-#pragma unroll
-      for (int j = 0; j < 4; ++j) s[r][j] = nxt[r][j];
-    load(i + 1);
+    if (i < w0 || i > w1) continue;
+    const uint8_t* sc = s_raw + (ss - sv) + (i & (kRing - 1)) * kScr + (t4 & 1) * 8;
     uint32_t hi[2][4], lo[2][4];   // [row half][8-key group]
     float alpha[2];
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
-      float mx = -INFINITY;
+      float2 s[4];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) mx = fmaxf(mx, fmaxf(s[r][j].x, s[r][j].y));
+      for (int j = 0; j < 4; ++j)
+        s[j] = *reinterpret_cast<const float2*>(sc + (g8 + 8 * r) * 128 + (((2 * j + (t4 >> 1)) ^ g8) << 4));
+      float mx = fmaxf(fmaxf(fmaxf(s[0].x, s[0].y), fmaxf(s[1].x, s[1].y)), fmaxf(fmaxf(s[2].x, s[2].y), fmaxf(s[3].x, s[3].y)));
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-      const float mn = fmaxf(m[r], mx), ms = mn == -INFINITY ? 0.f : mn;
-      alpha[r] = ex2t(m[r] - ms);
-      m[r] = mn;
+      // the reference moves only when a maximum grows by more than 2^8 (or there was none)
+      alpha[r] = 1.f;
+      if (mx > m[r] + 8.f || m[r] == -INFINITY) {
+        const float mn = fmaxf(m[r], mx);
+        alpha[r] = m[r] == -INFINITY ? 1.f : ex2t(m[r] - mn);   // (nothing has been added yet: any factor will do)
+        m[r] = mn;
+      }
+      const float ms = m[r] == -INFINITY ? 0.f : m[r];
       float sum = 0.f;
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        const float a = ex2t(s[r][j].x - ms), b = ex2t(s[r][j].y - ms);
+        const float a = ex2t(s[j].x - ms), b = ex2t(s[j].y - ms);
         sum += a + b;
         hi[r][j] = pack_bf16x2(a, b);
         lo[r][j] = pack_bf16x2(a - __uint_as_float(hi[r][j] << 16), b - __uint_as_float(hi[r][j] & 0xffff0000u));
@@ -683,7 +700,7 @@ __global__ void __launch_bounds__(128) talk_values_kernel(const TalkParams p) {
         o[n][3] *= alpha[1];
       }
     }
-    const uint32_t vb = smem_u32(s_raw) + (i & (kRing - 1)) * kBlk;
+    const uint32_t vb = sv + (i & (kRing - 1)) * kBlk;
 #pragma unroll
     for (int ks = 0; ks < 2; ++ks)
 #pragma unroll
@@ -692,13 +709,15 @@ __global__ void __launch_bounds__(128) talk_values_kernel(const TalkParams p) {
         const int r = ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), ch = n * 2 + (lane >> 4);
         ldsm4t(vb + r * (D * 2) + ((ch ^ (r & 7)) << 4), v);
 #pragma unroll
-        for (int w = 0; w < 2; ++w) {
+        for (int w = 0; w < 2; ++w)
           mma_bf16(o[2 * n + w], hi[0][2 * ks], hi[1][2 * ks], hi[0][2 * ks + 1], hi[1][2 * ks + 1], v[2 * w], v[2 * w + 1]);
+#pragma unroll
+        for (int w = 0; w < 2; ++w)
           mma_bf16(o[2 * n + w], lo[0][2 * ks], lo[1][2 * ks], lo[0][2 * ks + 1], lo[1][2 * ks + 1], v[2 * w], v[2 * w + 1]);
-        }
       }
   }
   cp_wait<0>();
+  const bool even = (p.D & 1) == 0 && (p.ldo & 1) == 0 && (p.gate_ld & 1) == 0;   // pairs of values stay aligned
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     float sum = l[r];
@@ -710,37 +729,49 @@ __global__ void __launch_bounds__(128) talk_values_kernel(const TalkParams p) {
     const long long row = x.row0 + qr;
     __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + row * p.ldo;
 #pragma unroll
-    for (int n = 0; n < D / 8; ++n)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int d = n * 8 + 2 * t4 + e, col = head * p.D + d;
-        if (d < p.D) out[col] = __float2bfloat16(o[n][2 * r + e] * inv * gate_at(p, row, col));
+    for (int n = 0; n < D / 8; ++n) {
+      const int d = n * 8 + 2 * t4, col = head * p.D + d;
+      const float a = o[n][2 * r] * inv, b = o[n][2 * r + 1] * inv;
+      if (even) {
+        if (d < p.D) {
+          const float2 z = p.gate_f32 ? *reinterpret_cast<const float2*>(static_cast<const float*>(p.gate) + row * p.gate_ld + col)
+                                      : __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(static_cast<const __nv_bfloat16*>(p.gate) + row * p.gate_ld + col));
+          *reinterpret_cast<uint32_t*>(out + col) = pack_bf16x2(__fdividef(a, 1.f + __expf(-z.x)), __fdividef(b, 1.f + __expf(-z.y)));
+        }
+      } else {
+        if (d < p.D) out[col] = __float2bfloat16(a * gate_at(p, row, col));
+        if (d + 1 < p.D) out[col + 1] = __float2bfloat16(b * gate_at(p, row, col + 1));
       }
+    }
   }
 }
 
 template <int D, int HM>
 cudaError_t launch_scores(const TalkParams& p, cudaStream_t stream) {
   auto kern = talk_scores_kernel<D, HM>;
-  const size_t smem = 8ull * kSub * D * 2 + p.H * HM * 8ull + p.H * 64 * 4ull;
+  const size_t smem = 4ull * (HM * kHPitch + p.H * kBiasPitch + kKeys);
   ensure_dynamic_smem(kern, smem);
-  return launch_kernel(kern, dim3(p.span / kSub, kTile / kSub, p.n_rows), dim3(256), smem, stream, true, false, p);
+  const int groups = (p.span / kKeys + kBlocks - 1) / kBlocks;
+  return launch_kernel(kern, dim3(groups, kTile / kQ, p.n_rows), dim3(256), smem, stream, true, false, p);
 }
 template <int D>
 cudaError_t launch_prefill(const TalkParams& p, cudaStream_t stream) {
-  const cudaError_t e = p.H <= 8 ? launch_scores<D, 8>(p, stream) : (p.H <= 16 ? launch_scores<D, 16>(p, stream) : launch_scores<D, 32>(p, stream));
+  const cudaError_t e = p.H <= 16 ? launch_scores<D, 16>(p, stream) : launch_scores<D, 32>(p, stream);
   if (e != cudaSuccess) return e;
   auto kern = talk_values_kernel<D>;
-  const size_t smem = 4ull * kSub * D * 2;
+  const size_t smem = static_cast<size_t>(kValueRing) * (kKeys * D * 2 + 4 * 16 * kKeys * 4);
   ensure_dynamic_smem(kern, smem);
   return launch_kernel(kern, dim3(p.H, kTile / kValueRows, p.n_rows), dim3(128), smem, stream, true, false, p);
 }
 template <int D>
 cudaError_t launch_decode(const TalkParams& p, cudaStream_t stream) {
   auto kern = talk_decode_kernel<D>;
-  const size_t smem = decode_layout(p.H, p.G, D).total;
-  ensure_dynamic_smem(kern, smem);
-  const cudaError_t e = launch_kernel(kern, dim3(p.n_rows, p.max_splits), dim3(256), smem, stream, true, false, p);
+  const DecodeLayout l = decode_layout(p.H, p.G, D);
+  ensure_dynamic_smem(kern, l.total + 1024);
+  // about as many CTAs as fit the SMs at once
+  const int fit = (l.total > 100 * 1024 ? 1 : 2) * sm_count() / p.n_rows;
+  const int splits = fit < 1 ? 1 : (fit < p.max_splits ? fit : p.max_splits);
+  const cudaError_t e = launch_kernel(kern, dim3(p.n_rows, p.max_splits), dim3(kDecThreads), static_cast<size_t>(l.total), stream, true, false, p, l, splits);
   if (e != cudaSuccess) return e;
   return launch_kernel(talk_merge_kernel<D>, dim3(p.n_rows, p.H), dim3(D), 0, stream, true, false, p);
 }
@@ -764,7 +795,7 @@ cudaError_t launch_talk_rows(const TalkParams& p, int dtype, cudaStream_t stream
 bool talk_decode_ok(int H, int G, int DP) {
   if ((DP != 64 && DP != 128) || H > kMaxHeads || H % G != 0) return false;
   const DecodeLayout l = decode_layout(H, G, DP);
-  return G * l.nt * (DP / 16) <= 8 * kMaxTiles && l.total <= 220 * 1024;
+  return G * l.nt * (DP / 16) <= kDecWarps * kMaxTiles && l.total <= 220 * 1024;
 }
 
 cudaError_t launch_talk_decode(const TalkParams& p, cudaStream_t stream) {
@@ -777,7 +808,7 @@ bool talk_prefill_ok(int H, int DP) { return (DP == 64 || DP == 128) && H <= 32;
 
 int talk_span(int window, int max_ctx) {
   const int n = window > 0 && window + kTile - 1 < max_ctx ? window + kTile - 1 : max_ctx;
-  return (n + 2 * kSub - 2) / kSub * kSub;
+  return (n + 2 * kKeys - 2) / kKeys * kKeys;
 }
 
 cudaError_t launch_talk_prefill(const TalkParams& p, cudaStream_t stream) {

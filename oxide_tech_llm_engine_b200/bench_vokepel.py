@@ -137,9 +137,8 @@ def kernel_numbers(vok, kip, peaks: dict, timer: Timer, batch: int, ctx: int, m:
         bt = torch.randperm(batch * nb_seq, device=dev).to(torch.int32).view(batch, nb_seq)
         q, out, gate = torch.randn(batch, H * P, **bf), torch.empty(batch, H * D, **bf), torch.randn(batch, H * D, **bf)
         po, pm = torch.empty(batch * H * splits * P, device=dev), torch.empty(batch * H * splits * 2, device=dev)
-        pps = plan(att.kv_heads)
         return lambda: hops.talk_decode(q, c, r, bt, lens, rows=batch, h=H, d=D, window=talk.window, scale=0.1, cap=30.0, gate=gate, out=out,
-                                        pages_per_split=pps, part_o=po, part_ml=pm, max_splits=splits, **mats)
+                                        part_o=po, part_ml=pm, max_splits=splits, **mats)
     vis = lambda w: min(ctx, w + 16) if w else ctx
     add(f"paged_decode, window and sinks [{batch} x {vis(att.window)} keys]", lambda i: dec(att, i, True),
         batch * vis(att.window) * att.kv_heads * att.dim * 4)

@@ -223,7 +223,7 @@ class TalkingRun:
         gate = proj[:, a.gate_col:]
         kw = dict(h=a.heads, d=a.dim, window=a.window, scale=a.scale, cap=a.softcap, talk=w["talk"], bias=w["bias"], gate=gate, out=out)
         if nd > 0:
-            parts = dict(pages_per_split=s.pages_per_split, part_o=m.part_o, part_ml=m.part_ml, max_splits=m.max_splits) if self.decode_tc else {}
+            parts = dict(part_o=m.part_o, part_ml=m.part_ml, max_splits=m.max_splits) if self.decode_tc else {}
             hops.talk_decode(q, self.cache, self.k_rms, s.block_tables, s.seq_lens, rows=nd, **kw, **parts)
         if s.n_prefill > 0:
             seqs = (s.q_start, s.q_lens, s.ctx_lens)
@@ -893,7 +893,7 @@ class HybridModel(GemmShapes):
         w_in = q.new_zeros(a.in_width, q.shape[1])
         w_in[:q.shape[0]], w_in[q.shape[0]:q.shape[0] + k.shape[0]], w_in[a.gate_col:] = q, k, g
         wk = vec(p + "k.norm").view(a.kv_heads, 1, a.dim).expand(a.kv_heads, a.heads // a.kv_heads, a.dim).reshape(-1)
-        talk = vec(p + "talk").contiguous()
+        talk = mat(p + "talk").float().contiguous()      # a matrix: of the model's dtype, like the others
         far = a.window or 16 * self.max_blocks_per_seq
         return {"w_in": self._pad(w_in), "w_o": self._pad(mat(p + "o")), "rot": self._rotary(None), "q_norm": (vec(p + "q.norm") * wk).contiguous(),
                 "talk": talk, "bias": hops.talk_bias(talk, vec(p + "r1"), vec(p + "r2"), far)}

@@ -293,9 +293,9 @@ def talk_bias(talk: torch.Tensor, r1: torch.Tensor, r2: torch.Tensor, n: int) ->
 
 
 def talk_decode(q, cache, k_rms, block_tables, seq_lens, *, rows: int, h: int, d: int, window: int, scale: float, cap: float, talk, bias,
-                gate, out, pages_per_split=None, part_o=None, part_ml=None, max_splits: int = 0) -> None:
+                gate, out, part_o=None, part_ml=None, max_splits: int = 0) -> None:
     """Decode rows of talking heads (TalkParams): split-KV and merge, or without `part_o` the kernel for any sizes."""
-    hybrid_ext().talk_decode(q, cache, k_rms, block_tables, seq_lens, pages_per_split, rows, h, d, window, scale, cap, talk, bias, gate,
+    hybrid_ext().talk_decode(q, cache, k_rms, block_tables, seq_lens, rows, h, d, window, scale, cap, talk, bias, gate,
                              part_o, part_ml, max_splits, out, ops.status_word(q.device))
     ops._bump(1 if part_o is None else 2)
 
