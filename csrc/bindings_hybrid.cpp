@@ -963,6 +963,12 @@ oxb::TalkParams talk_common(const Tensor& q, const Tensor& cache, const Tensor& 
   return p;
 }
 
+// cache rows (one position of one key head) in boxes of `rows` x 64
+CUtensorMap talk_cache_map(const Tensor& cache, const oxb::TalkParams& p, int rows) {
+  return oxb::make_tma_map(cache.data_ptr(), CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, 2, p.DP, static_cast<uint64_t>(p.num_blocks) * p.G * 16, 1,
+                           static_cast<uint64_t>(p.DP) * 2, 0, 64, rows, 1, CU_TENSOR_MAP_SWIZZLE_128B);
+}
+
 void talk_decode(const Tensor& q, const Tensor& cache, const Tensor& k_rms, const Tensor& block_tables, const Tensor& seq_lens,
                  int64_t rows, int64_t H, int64_t D, int64_t window, double scale, double cap,
                  const Tensor& talk, const Tensor& bias, const Tensor& gate, const OptTensor& part_o, const OptTensor& part_ml,
@@ -979,7 +985,8 @@ void talk_decode(const Tensor& q, const Tensor& cache, const Tensor& k_rms, cons
   p.part_o = const_cast<float*>(f32(*part_o, rows * H * max_splits * p.DP, "talk_decode part_o"));
   p.part_ml = const_cast<float*>(f32(*part_ml, rows * H * max_splits * 2, "talk_decode part_ml"));
   p.max_splits = static_cast<int>(max_splits);
-  check_launch(oxb::launch_talk_decode(p, cur_stream()), "talk_decode");
+  CUtensorMap tmC = talk_cache_map(cache, p, oxb::talk_decode_box(p.H, p.G, p.DP));
+  check_launch(oxb::launch_talk_decode(tmC, p, cur_stream()), "talk_decode");
 }
 
 void talk_prefill(const Tensor& q, const Tensor& cache, const Tensor& k_rms, const Tensor& block_tables, const Tensor& tile_seq,
@@ -999,7 +1006,8 @@ void talk_prefill(const Tensor& q, const Tensor& cache, const Tensor& k_rms, con
   TORCH_CHECK(dtype_code(q, "talk q") == 0 && oxb::talk_prefill_ok(p.H, p.DP) && span > 0 && span % 32 == 0, "talk_prefill: sizes");
   p.scores = const_cast<float*>(f32(*scores, n_tiles * H * 128 * span, "talk_prefill scores"));
   p.span = static_cast<int>(span);
-  check_launch(oxb::launch_talk_prefill(p, cur_stream()), "talk_prefill");
+  CUtensorMap tmV = talk_cache_map(cache, p, 16);
+  check_launch(oxb::launch_talk_prefill(tmV, p, cur_stream()), "talk_prefill");
 }
 
 oxb::GruParams gru_common(const Tensor& proj, int64_t M, const Tensor& bias, double out_gain, const Tensor& state, const Tensor& out,

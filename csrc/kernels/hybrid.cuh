@@ -207,7 +207,7 @@ struct TalkParams {
   float* part_ml;           // [rows, H, max_splits, 2]
   int max_splits;
   float* scores;            // prompt chunks: [tiles, H, 128, span] mixed scores times log2(e), keys from the tile's first one on
-  int span;
+  int span;                 // a multiple of 32
   void* out;                // [rows, ldo], heads of D
   long long ldo;
   int* status;
@@ -215,11 +215,12 @@ struct TalkParams {
 // Any sizes, fp32 FMAs, one CTA per row: the fp32 path and sizes that the other kernels do not take.
 cudaError_t launch_talk_rows(const TalkParams& p, int dtype, cudaStream_t stream);
 size_t talk_rows_smem(int H, int D);
-// bf16, D padded to 64 or 128. Decoding: split-KV and merge.
-cudaError_t launch_talk_decode(const TalkParams& p, cudaStream_t stream);
+// bf16, D padded to 64 or 128. Decoding: split-KV and merge. tmC: cache rows in boxes of talk_decode_box x 64.
+cudaError_t launch_talk_decode(const CUtensorMap& tmC, const TalkParams& p, cudaStream_t stream);
+int talk_decode_box(int H, int G, int DP);
 bool talk_decode_ok(int H, int G, int DP);
-// Prompt chunks: mixed scores of a step's tiles, then softmax and sums.
-cudaError_t launch_talk_prefill(const TalkParams& p, cudaStream_t stream);
+// Prompt chunks: mixed scores of a step's tiles, then softmax and sums. tmV: cache rows in boxes of 16 x 64.
+cudaError_t launch_talk_prefill(const CUtensorMap& tmV, const TalkParams& p, cudaStream_t stream);
 bool talk_prefill_ok(int H, int DP);
 int talk_span(int window, int max_ctx);   // keys per row of `scores`
 

@@ -105,7 +105,7 @@ def talk_head(a) -> int:
     return 0 if a.dim > 128 else (64 if a.dim <= 64 else 128)
 
 
-TALK_SCORE_BYTES = 256 << 20   # mixed scores of prompt tiles that are held at a time
+TALK_SCORE_BYTES = 1 << 30   # mixed scores of prompt tiles that are held at a time
 
 KV_PASS_ROWS = 65536      # positions whose keys and values are expanded at a time
 
