@@ -48,13 +48,15 @@ __device__ __forceinline__ float gate_at(const TalkParams& p, long long row, int
                              : to_f(static_cast<const __nv_bfloat16*>(p.gate)[row * p.gate_ld + col]);
   return 1.f / (1.f + expf(-z));
 }
-// block id of page pg of a sequence; ids outside the pool are recorded and replaced by 0
-__device__ __forceinline__ int block_of(const TalkParams& p, const int* bt, int pg) {
-  const int b = pg < p.max_blocks ? bt[pg] : -1;
+// Block id of page pg of a sequence, as it stands in the table (loaded ahead of its use), and checked: ids outside the pool are
+// recorded and replaced by 0.
+__device__ __forceinline__ int raw_block(const TalkParams& p, const int* bt, int pg) { return pg < p.max_blocks ? bt[pg] : -1; }
+__device__ __forceinline__ int checked_block(const TalkParams& p, int b) {
   if (static_cast<unsigned>(b) < static_cast<unsigned>(p.num_blocks)) return b;
   set_status_once(p.status, kStatusBadIndex);
   return 0;
 }
+__device__ __forceinline__ int block_of(const TalkParams& p, const int* bt, int pg) { return checked_block(p, raw_block(p, bt, pg)); }
 
 // Mixing the heads' scores is a product with the heads' matrix: the scores (fp32) enter as two fp16 terms, which carry 22 bits of
 // them (scores without a cap are kept inside fp16's range); the matrix holds bf16 values, exact in fp16 but for tiny ones.
@@ -279,16 +281,19 @@ __global__ void __launch_bounds__(kDecThreads) talk_decode_kernel(const __grid_c
     return;
   }
   const int n_blocks = (pg_hi - pg_lo + L.pages - 1) / L.pages;
-  // copies (warp 0): per page the boxes of its key heads and 64 dims, and its norm factors; lane pg holds the block id of page pg
+  // copies (by the last warp, which is the likeliest to have no scores to mix): per page the boxes of its key heads and 64 dims, and
+  // its norm factors; lane pg holds the block id of page pg
+  constexpr int kCopyWarp = kDecWarps - 1;
   const int per_page = G / L.box * HF + 1;
   const int* bt = p.block_tables + static_cast<long long>(seq) * p.max_blocks;
   auto id_of = [&](int b) {
     const int pg = pg_lo + b * L.pages + lane;
-    return lane < L.pages && pg < pg_hi ? block_of(p, bt, pg) : 0;
+    return lane < L.pages && pg < pg_hi ? raw_block(p, bt, pg) : 0;
   };
   auto issue = [&](int b, int slot, int id) {
     const int n = min(L.pages, pg_hi - pg_lo - b * L.pages);
     if (lane == 0) mbar_arrive_expect_tx(&full[slot], n * (L.page_bytes + 64));
+    id = checked_block(p, id);
     __syncwarp();
     for (int c0 = 0; c0 < n * per_page; c0 += 32) {
       const int c = c0 + lane, pg = c / per_page, k = c - pg * per_page;
@@ -307,7 +312,7 @@ __global__ void __launch_bounds__(kDecThreads) talk_decode_kernel(const __grid_c
   };
   __syncthreads();   // (the barriers are set up)
   int id = 0;
-  if (warp == 0) {
+  if (warp == kCopyWarp) {
     id = id_of(0);
     for (int b = 0; b < L.stages - 1; ++b) {
       if (b < n_blocks) issue(b, b, id);
@@ -373,8 +378,8 @@ __global__ void __launch_bounds__(kDecThreads) talk_decode_kernel(const __grid_c
       for (int e = 0; e < 2; ++e) {
         const int d = dist - 8 * e, at = min(d, p.n_bias - 1);
         if (d >= 0 && (p.window == 0 || d < p.window)) {
-          if (mh < H) x[2 * e] = kLog2e * __ldg(m_bias0 + at);
-          if (mh + 1 < H) x[2 * e + 1] = kLog2e * __ldg(m_bias1 + at);
+          if (mh < H) x[2 * e] = __ldg(m_bias0 + at);
+          if (mh + 1 < H) x[2 * e + 1] = __ldg(m_bias1 + at);
         }
       }
     }
@@ -416,7 +421,7 @@ __global__ void __launch_bounds__(kDecThreads) talk_decode_kernel(const __grid_c
       }
     }
     __syncthreads();   // (and every warp is done with the sums of the block before)
-    if (warp == 0) {
+    if (warp == kCopyWarp) {
       const int nb = b + L.stages - 1;
       if (nb < n_blocks) issue(nb, slot == 0 ? L.stages - 1 : slot - 1, id);
       id = id_of(nb + 1);
@@ -452,7 +457,7 @@ __global__ void __launch_bounds__(kDecThreads) talk_decode_kernel(const __grid_c
         mma_f16(mixed, hi, b0, b1);
       }
 #pragma unroll
-      for (int e = 0; e < 4; ++e) x[e] = mixed[e] - x[e];
+      for (int e = 0; e < 4; ++e) x[e] = fmaf(-kLog2e, x[e], mixed[e]);
       float m0 = fmaxf(x[0], x[2]), m1 = fmaxf(x[1], x[3]);
 #pragma unroll
       for (int w = 4; w < 32; w <<= 1) {
@@ -603,11 +608,15 @@ __device__ __forceinline__ Piece piece_of(const TalkParams& p, int tile, int q, 
 // first key of a tile's row of scores
 __device__ __forceinline__ int first_key(const TalkParams& p, int tile) { return piece_of(p, tile, 0, kTile).lo / kKeys * kKeys; }
 
-// Row pitch of a head's scores in shared memory, and of a query's keys inside: a warp's stores (8 keys x 4 queries) and its
-// reads (4 heads, two apart, x 8 keys) both touch 32 banks.
-constexpr int kQPitch = kKeys + 4, kHPitch = kQ * kQPitch + 4;
-static_assert(kHPitch % 16 == 4, "banks");
-constexpr int kBiasPitch = 72;
+// Places in shared memory, so that no access of a warp meets a bank twice. Scores [head][query][key]: of 16 keys, key 4 t + 2 a + b
+// lies at 8 a + 2 t + b, so a lane that mixes the places 2 t and 2 t + 1 of both eights has four neighbouring keys. Biases
+// [head][distance].
+constexpr int kHPitch = 580;
+__device__ __forceinline__ int query_at(int q) { return q * 34 + (q >> 2) * 8; }
+__device__ __forceinline__ int key_at(int k) { return (k & 16) + ((k >> 1) & 1) * 8 + ((k >> 2) & 3) * 2 + (k & 1); }
+static_assert(kHPitch >= 15 * 34 + 3 * 8 + kKeys && kHPitch % 16 == 4, "banks");
+constexpr int kBiasPitch = 80;
+__device__ __forceinline__ int bias_at(int h) { return h * kBiasPitch + ((h >> 1) & 3); }
 
 // HM: heads of this instantiation, 16 or 32 (H <= HM). The queries of all heads stay in shared memory while the CTA walks its
 // blocks of keys. 16 warps = 8 sets of heads x 2 halves of a block: a warp multiplies 16 keys x 16 queries for the heads of its set,
@@ -657,21 +666,19 @@ __global__ void __launch_bounds__(kScoreThreads, 1) talk_scores_kernel(const Tal
   const float unit = p.scale * cap.k;
   uint4 ka[2][CPL];
   float r0 = 0.f, r1 = 0.f;   // factors of the lane's keys
+  const int c_at = query_at(2 * t4) + key_at(half * 16 + g8);
   int id = 0;
-  auto page = [&](int b) {    // block id of this warp's half of key block b, -1 beyond the context
-    const int pg = (k_start >> 4) + 2 * b + half;
-    return b < b_hi && pg < n_pg ? block_of(p, bt, pg) : -1;
-  };
+  auto page = [&](int b) { return raw_block(p, bt, min((k_start >> 4) + 2 * b + half, n_pg - 1)); };   // of this warp's half of key block b
   auto load_keys = [&](int kv) {
-    const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(p.cache) + (static_cast<long long>(max(id, 0)) * p.G + kv) * 16 * D + t4 * 8;
+    const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(p.cache) + (static_cast<long long>(id) * p.G + kv) * 16 * D + t4 * 8;
 #pragma unroll
     for (int r = 0; r < 2; ++r)
 #pragma unroll
       for (int c = 0; c < CPL; ++c) ka[r][c] = *reinterpret_cast<const uint4*>(kp + (g8 + 8 * r) * D + c * 32);
   };
   auto load_norms = [&]() {
-    r0 = id >= 0 ? p.k_rms[id * 16ll + g8] * unit : 0.f;
-    r1 = id >= 0 ? p.k_rms[id * 16ll + g8 + 8] * unit : 0.f;
+    r0 = p.k_rms[id * 16ll + g8];
+    r1 = p.k_rms[id * 16ll + g8 + 8];
   };
   // biases of key block b, two heads per warp (HM <= 32): lanes are distances
   float bias_next[2][2];
@@ -686,7 +693,7 @@ __global__ void __launch_bounds__(kScoreThreads, 1) talk_scores_kernel(const Tal
         bias_next[u][v] = see ? __ldg(p.bias + static_cast<long long>(h) * p.n_bias + min(dist, p.n_bias - 1)) : INFINITY;
       }
   };
-  id = page(b_lo);
+  id = checked_block(p, page(b_lo));
   if (h_lo < h_hi) load_keys(kv_lo);
   load_norms();
   load_bias(b_lo);
@@ -697,11 +704,13 @@ __global__ void __launch_bounds__(kScoreThreads, 1) talk_scores_kernel(const Tal
 #pragma unroll
     for (int u = 0; u < 2; ++u)
       if (warp + 16 * u < H) {
-        float* d = s_b + (warp + 16 * u) * kBiasPitch + lane;
+        float* d = s_b + bias_at(warp + 16 * u) + lane;
         d[0] = kLog2e * bias_next[u][0];
         if (lane < kQ - 1) d[32] = kLog2e * bias_next[u][1];
       }
-    // ---- scores of this warp's heads: [16 keys x 16 queries] ----
+    // ---- scores of this warp's heads: [16 keys x 16 queries]; positions behind the context are hidden by their bias ----
+    r0 *= unit;
+    r1 *= unit;
     int kv = kv_lo, left = R - (h_lo - kv_lo * R);   // heads of this key head that are still to come
     for (int h = h_lo; h < h_hi; ++h, --left) {
       if (left == 0) {
@@ -720,14 +729,13 @@ __global__ void __launch_bounds__(kScoreThreads, 1) talk_scores_kernel(const Tal
           mma_bf16(s[n], ka[0][c].z, ka[1][c].z, ka[0][c].w, ka[1][c].w, f.z, f.w);
         }
       }
-      float* d = s_c + h * kHPitch + 2 * t4 * kQPitch + half * 16 + g8;
+      float* d = s_c + h * kHPitch + c_at;   // (queries 8 and 1, and keys 8 further on are a fixed way off)
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-          d[(n * 8 + (e & 1)) * kQPitch + (e >> 1) * 8] = capped(s[n][e], e < 2 ? r0 : r1, cap);
+        for (int e = 0; e < 4; ++e) d[n * 288 + (e & 1) * 34 + (e >> 1) * 4] = capped(s[n][e], e < 2 ? r0 : r1, cap);
     }
-    id = id_next;      // the next block's keys while this one's scores are mixed
+    id = checked_block(p, id_next);   // the next block's keys while this one's scores are mixed
     if (h_lo < h_hi) load_keys(kv_lo);
     load_norms();
     load_bias(b + 1);
@@ -735,36 +743,41 @@ __global__ void __launch_bounds__(kScoreThreads, 1) talk_scores_kernel(const Tal
     __syncthreads();
     // ---- mixed scores: a warp takes a query, 8 keys at a time ----
     const int q = warp;
+    const float* src = s_c + 2 * t4 * kHPitch + query_at(q) + g8;
+    const float* bb = s_b + bias_at(g8) + kKeys - 1 + q - 4 * t4;   // bias of the lane's first key; the next ones are one nearer each
+    float* dst = p.scores + ((static_cast<long long>(tile) * H + g8) * kTile + q_in + q) * p.span + b * kKeys + 4 * t4;
 #pragma unroll
-    for (int k8 = 0; k8 < kKeys; k8 += 8) {
-      const float* src = s_c + 2 * t4 * kHPitch + q * kQPitch + k8 + g8;
-      const float* bb = s_b + g8 * kBiasPitch + kKeys - 1 + q - k8 - 2 * t4;   // bias of the lane's first key; the second is one nearer
-      float o[HT][4];
+    for (int k16 = 0; k16 < kKeys; k16 += 16) {
+      float o[2][HT][4];   // places of the lower and of the upper eight
 #pragma unroll
-      for (int m = 0; m < HT; ++m)
+      for (int a = 0; a < 2; ++a)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int h = m * 16 + 8 * (e >> 1);
-          o[m][e] = h + g8 < H ? -bb[h * kBiasPitch - (e & 1)] : 0.f;
+        for (int m = 0; m < HT; ++m)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int h = m * 16 + 8 * (e >> 1);   // (bias_at(g8 + h) = bias_at(g8) + h * pitch)
+            o[a][m][e] = h + g8 < H ? -bb[h * kBiasPitch - k16 - 2 * a - (e & 1)] : 0.f;
+          }
+#pragma unroll
+      for (int a = 0; a < 2; ++a)
+#pragma unroll
+        for (int k = 0; k < HT; ++k) {
+          const float* f = src + k * 16 * kHPitch + k16 + 8 * a;
+          uint32_t h0, h1, l0, l1;
+          split_f16(f[0], f[kHPitch], h0, l0);
+          split_f16(f[8 * kHPitch], f[9 * kHPitch], h1, l1);
+#pragma unroll
+          for (int m = 0; m < HT; ++m) mma_f16(o[a][m], ta[m][k], l0, l1);
+#pragma unroll
+          for (int m = 0; m < HT; ++m) mma_f16(o[a][m], ta[m][k], h0, h1);
         }
-#pragma unroll
-      for (int k = 0; k < HT; ++k) {
-        const float* f = src + k * 16 * kHPitch;
-        uint32_t h0, h1, l0, l1;
-        split_f16(f[0], f[kHPitch], h0, l0);
-        split_f16(f[8 * kHPitch], f[9 * kHPitch], h1, l1);
-#pragma unroll
-        for (int m = 0; m < HT; ++m) mma_f16(o[m], ta[m][k], l0, l1);
-#pragma unroll
-        for (int m = 0; m < HT; ++m) mma_f16(o[m], ta[m][k], h0, h1);
-      }
-      float* dst = p.scores + ((static_cast<long long>(tile) * H + g8) * kTile + q_in + q) * p.span + b * kKeys + k8 + 2 * t4;
 #pragma unroll
       for (int m = 0; m < HT; ++m)
 #pragma unroll
         for (int r = 0; r < 2; ++r)
           if (m * 16 + 8 * r + g8 < H)
-            *reinterpret_cast<float2*>(dst + static_cast<long long>(m * 16 + 8 * r) * kTile * p.span) = make_float2(o[m][2 * r], o[m][2 * r + 1]);
+            *reinterpret_cast<float4*>(dst + static_cast<long long>(m * 16 + 8 * r) * kTile * p.span + k16) =
+                make_float4(o[0][m][2 * r], o[0][m][2 * r + 1], o[1][m][2 * r], o[1][m][2 * r + 1]);
     }
     __syncthreads();
   }
@@ -837,6 +850,8 @@ __global__ void __launch_bounds__(kValueThreads, 2) talk_values_kernel(const __g
   if (warp == 0) {
     const int* bt = p.block_tables + static_cast<long long>(x.seq) * p.max_blocks;
     const int n_pg = (p.ctx_lens[x.seq] + 15) >> 4;
+    const int my_pg = (k_start >> 4) + lane / VH;   // lane = (page of the step, 64 dims); pages beyond the context weigh nothing
+    int id = lane < 4 * VH ? raw_block(p, bt, min(my_pg, n_pg - 1)) : 0;
     for (int j = 0; j < n_steps; ++j) {
       const int s = j & 1;
       bool ok = j < 2 || mbar_wait(&v_empty[s], ((j >> 1) - 1) & 1);
@@ -847,10 +862,10 @@ __global__ void __launch_bounds__(kValueThreads, 2) talk_values_kernel(const __g
       }
       if (lane == 0) mbar_arrive_expect_tx(&v_full[s], VH * L::kSub);
       __syncwarp();
-      if (lane < 4 * VH) {   // one box of 16 rows per page and 64 dims; pages beyond the context weigh nothing
-        const int pg = lane / VH, hf = lane % VH, pi = (k_start >> 4) + j * 4 + pg;
-        const int blk = pi < n_pg ? block_of(p, bt, pi) : 0;
-        tma_load_2d(s_v + (s * VH + hf) * L::kSub + pg * 2048, &tmV, &v_full[s], hf * 64, (blk * p.G + kv) * 16);
+      if (lane < 4 * VH) {
+        const int hf = lane % VH;
+        tma_load_2d(s_v + (s * VH + hf) * L::kSub + lane / VH * 2048, &tmV, &v_full[s], hf * 64, (checked_block(p, id) * p.G + kv) * 16);
+        id = raw_block(p, bt, min(my_pg + 4 * (j + 1), n_pg - 1));
       }
     }
   } else if (warp == 1) {
@@ -888,11 +903,8 @@ __global__ void __launch_bounds__(kValueThreads, 2) talk_values_kernel(const __g
     float4 buf[kRows][2];
     auto load = [&](int j, int i) {
 #pragma unroll
-      for (int u = 0; u < 2; ++u) {
-        const int blk = 2 * j + u;
-        buf[i][u] = blk >= w0 && blk <= w1 ? *reinterpret_cast<const float4*>(sp + (i * p.span + j * kStep + u * kKeys))   // (128 spans fit an int)
-                                           : make_float4(-INFINITY, -INFINITY, -INFINITY, -INFINITY);
-      }
+      for (int u = 0; u < 2; ++u)   // (blocks without scores are hidden when they are used; 128 spans fit an int)
+        buf[i][u] = __ldcg(reinterpret_cast<const float4*>(sp + (i * p.span + min(j * kStep + u * kKeys, p.span - kKeys))));
     };
 #pragma unroll
     for (int i = 0; i < kRows; ++i) load(0, i);
@@ -909,18 +921,28 @@ __global__ void __launch_bounds__(kValueThreads, 2) talk_values_kernel(const __g
       if (j >= 2 && !mbar_wait(&pv_done[b], ((j >> 1) - 1) & 1)) ok = false;   // this buffer's last products
       ok = __all_sync(0xffffffffu, ok);
       uint8_t* pb = s_p + b * 2 * L::kWeights;
+      const bool in[2] = {2 * j >= w0 && 2 * j <= w1, 2 * j + 1 >= w0 && 2 * j + 1 <= w1};   // blocks with scores
       bool grow = false;
+      float mx[kRows];
 #pragma unroll
       for (int i = 0; i < kRows; ++i) {
-        float s[8] = {buf[i][0].x, buf[i][0].y, buf[i][0].z, buf[i][0].w, buf[i][1].x, buf[i][1].y, buf[i][1].z, buf[i][1].w};
-        load(j + 1, i);   // (no block behind the last one exists)
-        float mx = fmaxf(fmaxf(fmaxf(s[0], s[1]), fmaxf(s[2], s[3])), fmaxf(fmaxf(s[4], s[5]), fmaxf(s[6], s[7])));
+        if (!in[0]) buf[i][0] = make_float4(-INFINITY, -INFINITY, -INFINITY, -INFINITY);
+        if (!in[1]) buf[i][1] = make_float4(-INFINITY, -INFINITY, -INFINITY, -INFINITY);
+        mx[i] = fmaxf(fmaxf(fmaxf(buf[i][0].x, buf[i][0].y), fmaxf(buf[i][0].z, buf[i][0].w)),
+                      fmaxf(fmaxf(buf[i][1].x, buf[i][1].y), fmaxf(buf[i][1].z, buf[i][1].w)));
+      }
 #pragma unroll
-        for (int o = 1; o < 8; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      for (int o = 1; o < 8; o <<= 1)
+#pragma unroll
+        for (int i = 0; i < kRows; ++i) mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], o));
+#pragma unroll
+      for (int i = 0; i < kRows; ++i) {
+        const float s[8] = {buf[i][0].x, buf[i][0].y, buf[i][0].z, buf[i][0].w, buf[i][1].x, buf[i][1].y, buf[i][1].z, buf[i][1].w};
+        load(j + 1, i);
         float alpha = 1.f;
-        if (mx > m[i] + 8.f || (m[i] == -INFINITY && mx > -INFINITY)) {
-          alpha = m[i] == -INFINITY ? 0.f : ex2t(m[i] - mx);
-          m[i] = mx;
+        if (mx[i] > m[i] + 8.f) {   // (of a reference of -inf: any score)
+          alpha = m[i] == -INFINITY ? 0.f : ex2t(m[i] - mx[i]);
+          m[i] = mx[i];
           grow = true;
         }
         const float ms = m[i] == -INFINITY ? 0.f : m[i];
@@ -1054,11 +1076,18 @@ cudaError_t launch_scores(const TalkParams& p, cudaStream_t stream) {
   auto kern = talk_scores_kernel<D, HM>;
   const size_t smem = scores_smem(p.H, D);
   ensure_dynamic_smem(kern, smem);
-  // at least eight blocks of keys per CTA (its queries are loaded once), more CTAs than SMs where there are that many
-  const int blocks = p.span / kKeys, pieces = p.n_rows * (kTile / kQ);
-  int parts = (4 * sm_count() + pieces - 1) / pieces;
-  parts = parts > (blocks + 7) / 8 ? (blocks + 7) / 8 : parts;
-  const int per = (blocks + parts - 1) / parts;
+  // parts of a piece's keys, so that the CTAs' rounds are shortest (loading the queries costs about one and a half blocks)
+  const int blocks = p.span / kKeys, pieces = p.n_rows * (kTile / kQ), sms = sm_count();
+  int per = blocks;
+  float best = 0.f;
+  for (int parts = 1; parts <= 16 && parts <= blocks; ++parts) {
+    const int n = (blocks + parts - 1) / parts;
+    const float cost = static_cast<float>((static_cast<long long>(pieces) * parts + sms - 1) / sms) * (n + 1.5f);
+    if (parts == 1 || cost < best) {
+      best = cost;
+      per = n;
+    }
+  }
   return launch_kernel(kern, dim3((blocks + per - 1) / per, kTile / kQ, p.n_rows), dim3(kScoreThreads), smem, stream, true, false, p, per);
 }
 template <int D>

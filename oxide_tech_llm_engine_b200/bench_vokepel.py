@@ -43,7 +43,7 @@ def _configs(name: str):
 def kernel_numbers(vok, kip, peaks: dict, timer: Timer, batch: int, ctx: int, m: int, only: str = "") -> list:
     """One row per kernel: name, microseconds, roofline microseconds, fraction of the roofline. `only`: names that contain it."""
     from . import ops
-    from .models.hybrid import TALK_SCORE_BYTES, talk_head, tc_head
+    from .models.hybrid import talk_head, talk_pass, tc_head
     from .ops import hybrid as hops
 
     dev = torch.device("cuda", 0)
@@ -170,8 +170,8 @@ def kernel_numbers(vok, kip, peaks: dict, timer: Timer, batch: int, ctx: int, m:
         c, r = torch.randn(m // 16, G, 16, P, **bf), torch.ones(m // 16, 16, device=dev)
         q, out, gate = torch.randn(m, H * P, **bf), torch.empty(m, H * D, **bf), torch.randn(m, H * D, **bf)
         span = hops.talk_span(talk.window, L)
-        step = max(1, TALK_SCORE_BYTES // (4 * H * 128 * span))
-        ws = torch.empty(min(step, len(tiles)) * H * 128 * span, device=dev)
+        step = talk_pass(len(tiles), H * 128 * span)
+        ws = torch.empty(step * H * 128 * span, device=dev)
 
         def call():
             for t0 in range(0, len(tiles), step):

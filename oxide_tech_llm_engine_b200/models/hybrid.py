@@ -105,7 +105,13 @@ def talk_head(a) -> int:
     return 0 if a.dim > 128 else (64 if a.dim <= 64 else 128)
 
 
-TALK_SCORE_BYTES = 1 << 30   # mixed scores of prompt tiles that are held at a time
+TALK_SCORE_BYTES = 2 << 30   # mixed scores of prompt tiles that are held at a time
+
+def talk_pass(n_tiles: int, scores: int) -> int:
+    """Prompt tiles per pass: about equal passes whose scores (so many per tile) fit."""
+    most = max(1, TALK_SCORE_BYTES // (4 * scores))
+    return -(-n_tiles // -(-n_tiles // most))
+
 
 KV_PASS_ROWS = 65536      # positions whose keys and values are expanded at a time
 
@@ -229,7 +235,7 @@ class TalkingRun:
             seqs = (s.q_start, s.q_lens, s.ctx_lens)
             span = hops.talk_span(a.window, s.max_ctx)
             per = a.heads * 128 * span       # scores of a tile
-            step = max(1, TALK_SCORE_BYTES // (4 * per)) if self.prefill_tc else s.n_tiles
+            step = talk_pass(s.n_tiles, per) if self.prefill_tc else s.n_tiles
             for t0 in range(0, s.n_tiles, step):
                 n = min(step, s.n_tiles - t0)
                 ws = dict(scores=m.scratch("talk_scores", n * per), span=span) if self.prefill_tc else {}
