@@ -953,7 +953,7 @@ oxb::TalkParams talk_common(const Tensor& q, const Tensor& cache, const Tensor& 
   TORCH_CHECK(bias.dim() == 2 && bias.size(0) == H && bias.size(1) >= 1, "talk: bias [H, distances]");
   p.bias = f32(bias, H, "talk bias");
   p.n_bias = static_cast<int>(bias.size(1));
-  TORCH_CHECK(window == 0 ? bias.size(1) >= 16 * block_tables.size(1) : bias.size(1) >= window, "talk: a bias for every visible distance");
+  TORCH_CHECK(bias.size(1) >= 16 * block_tables.size(1) || (window > 0 && bias.size(1) >= window), "talk: a bias for every visible distance");
   p.gate_f32 = dtype_code(gate, "talk gate");
   p.gate = gate.data_ptr();
   p.gate_ld = pitch(gate, 1, H * D, "talk gate");

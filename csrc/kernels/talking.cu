@@ -588,7 +588,6 @@ __global__ void __launch_bounds__(D) talk_merge_kernel(const TalkParams p, int n
 constexpr int kTile = 128;   // query rows of the scheduler's tiles
 constexpr int kKeys = 32;    // keys of a block
 constexpr int kQ = 16;       // queries of a scores CTA
-constexpr int kScoreThreads = 512;
 
 // What a piece of a tile's rows sees: positions of its first and last row, first visible key.
 struct Piece {
@@ -619,11 +618,12 @@ constexpr int kBiasPitch = 80;
 __device__ __forceinline__ int bias_at(int h) { return h * kBiasPitch + ((h >> 1) & 3); }
 
 // HM: heads of this instantiation, 16 or 32 (H <= HM). The queries of all heads stay in shared memory while the CTA walks its
-// blocks of keys. 16 warps = 8 sets of heads x 2 halves of a block: a warp multiplies 16 keys x 16 queries for the heads of its set,
+// blocks of keys. HM / 2 warps = HM / 4 sets of heads x 2 halves of a block: a warp multiplies 16 keys x 16 queries for the heads of its set,
 // keys straight from memory a block ahead (16-byte pieces, the same permutation of the dimensions in q and k). Then the scores of
 // all heads are mixed as a product with the heads' matrix T, 8 keys of a query as its columns.
 template <int D, int HM>
-__global__ void __launch_bounds__(kScoreThreads, 1) talk_scores_kernel(const TalkParams p, int blocks_per_cta) {
+__global__ void __launch_bounds__(HM * 16, HM == 16 ? 2 : 1) talk_scores_kernel(const TalkParams p, int blocks_per_cta) {
+  constexpr int kThreads = HM * 16, W = HM / 2;
   constexpr int CPL = D / 32, CH = D / 8;   // 16-byte pieces of a row per lane, and in all
   constexpr int HT = HM / 16;
   extern __shared__ __align__(128) uint8_t s_raw[];
@@ -641,7 +641,7 @@ __global__ void __launch_bounds__(kScoreThreads, 1) talk_scores_kernel(const Tal
         const int h = m * 16 + g8 + (i & 1) * 8, g = k * 16 + 2 * t4 + (i >> 1) * 8;
         ta[m][k][i] = pack_f16x2(h < H && g < H ? p.talk[h * H + g] : 0.f, h < H && g + 1 < H ? p.talk[h * H + g + 1] : 0.f);
       }
-  for (int i = tid; i < (HM - H) * kHPitch; i += kScoreThreads) s_c[H * kHPitch + i] = 0.f;
+  for (int i = tid; i < (HM - H) * kHPitch; i += kThreads) s_c[H * kHPitch + i] = 0.f;
   pdl_wait();
   const int tile = blockIdx.z, q_in = blockIdx.y * kQ;
   const Piece x = piece_of(p, tile, q_in, kQ);
@@ -654,14 +654,14 @@ __global__ void __launch_bounds__(kScoreThreads, 1) talk_scores_kernel(const Tal
   // a row's 16-byte piece c lies at c ^ swz(row): a lane's reads (row g8, piece t4 + 4 c) touch all banks
   auto swz = [](int row) { return (((row >> 1) & 3) << 1) ^ ((row & 1) << 2); };
   const __nv_bfloat16* qp = static_cast<const __nv_bfloat16*>(p.q) + static_cast<long long>(x.row0) * p.q_ld;
-  for (int c = tid; c < H * kQ * CH; c += kScoreThreads) {
+  for (int c = tid; c < H * kQ * CH; c += kThreads) {
     const int row = c / CH, ch = c % CH, h = row / kQ, q = row % kQ;
     cp_async16(smem_u32(s_q) + row * (D * 2) + ((ch ^ swz(q)) << 4), qp + (q < n_q ? q : 0) * p.q_ld + h * D + ch * 8, q < n_q);
   }
   cp_commit();
   const int* bt = p.block_tables + static_cast<long long>(x.seq) * p.max_blocks;
   const int n_pg = (p.ctx_lens[x.seq] + 15) >> 4;
-  const int half = warp & 1, hc = (H + 7) / 8, h_lo = min((warp >> 1) * hc, H), h_hi = min(h_lo + hc, H), kv_lo = h_lo / R;
+  const int half = warp & 1, hc = (H + W / 2 - 1) / (W / 2), h_lo = min((warp >> 1) * hc, H), h_hi = min(h_lo + hc, H), kv_lo = h_lo / R;
   const Cap cap = cap_of(p.cap, kLog2e);   // scores times log2 e
   const float unit = p.scale * cap.k;
   uint4 ka[2][CPL];
@@ -680,7 +680,7 @@ __global__ void __launch_bounds__(kScoreThreads, 1) talk_scores_kernel(const Tal
     r0 = p.k_rms[id * 16ll + g8];
     r1 = p.k_rms[id * 16ll + g8 + 8];
   };
-  // biases of key block b, two heads per warp (HM <= 32): lanes are distances
+  // biases of key block b, two heads per warp: lanes are distances
   float bias_next[2][2];
   auto load_bias = [&](int b) {
     const int far0 = x.pos0 - (k_start + b * kKeys) - (kKeys - 1);   // distance of entry 0
@@ -688,7 +688,7 @@ __global__ void __launch_bounds__(kScoreThreads, 1) talk_scores_kernel(const Tal
     for (int u = 0; u < 2; ++u)
 #pragma unroll
       for (int v = 0; v < 2; ++v) {
-        const int h = warp + 16 * u, dist = far0 + lane + 32 * v;
+        const int h = warp + W * u, dist = far0 + lane + 32 * v;
         const bool see = h < H && dist >= 0 && (p.window == 0 || dist < p.window);
         bias_next[u][v] = see ? __ldg(p.bias + static_cast<long long>(h) * p.n_bias + min(dist, p.n_bias - 1)) : INFINITY;
       }
@@ -703,8 +703,8 @@ __global__ void __launch_bounds__(kScoreThreads, 1) talk_scores_kernel(const Tal
   for (int b = b_lo; b < b_hi; ++b) {
 #pragma unroll
     for (int u = 0; u < 2; ++u)
-      if (warp + 16 * u < H) {
-        float* d = s_b + bias_at(warp + 16 * u) + lane;
+      if (warp + W * u < H) {
+        float* d = s_b + bias_at(warp + W * u) + lane;
         d[0] = kLog2e * bias_next[u][0];
         if (lane < kQ - 1) d[32] = kLog2e * bias_next[u][1];
       }
@@ -741,43 +741,45 @@ __global__ void __launch_bounds__(kScoreThreads, 1) talk_scores_kernel(const Tal
     load_bias(b + 1);
     id_next = page(b + 2);
     __syncthreads();
-    // ---- mixed scores: a warp takes a query, 8 keys at a time ----
-    const int q = warp;
-    const float* src = s_c + 2 * t4 * kHPitch + query_at(q) + g8;
-    const float* bb = s_b + bias_at(g8) + kKeys - 1 + q - 4 * t4;   // bias of the lane's first key; the next ones are one nearer each
-    float* dst = p.scores + ((static_cast<long long>(tile) * H + g8) * kTile + q_in + q) * p.span + b * kKeys + 4 * t4;
+    // ---- mixed scores: a warp takes a query, 16 keys at a time ----
 #pragma unroll
-    for (int k16 = 0; k16 < kKeys; k16 += 16) {
-      float o[2][HT][4];   // places of the lower and of the upper eight
+    for (int q = warp; q < kQ; q += W) {
+      const float* src = s_c + 2 * t4 * kHPitch + query_at(q) + g8;
+      const float* bb = s_b + bias_at(g8) + kKeys - 1 + q - 4 * t4;   // bias of the lane's first key; the next ones are one nearer each
+      float* dst = p.scores + ((static_cast<long long>(tile) * H + g8) * kTile + q_in + q) * p.span + b * kKeys + 4 * t4;
 #pragma unroll
-      for (int a = 0; a < 2; ++a)
+      for (int k16 = 0; k16 < kKeys; k16 += 16) {
+        float o[2][HT][4];   // places of the lower and of the upper eight
+#pragma unroll
+        for (int a = 0; a < 2; ++a)
+#pragma unroll
+          for (int m = 0; m < HT; ++m)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const int h = m * 16 + 8 * (e >> 1);   // (bias_at(g8 + h) = bias_at(g8) + h * pitch)
+              o[a][m][e] = h + g8 < H ? -bb[h * kBiasPitch - k16 - 2 * a - (e & 1)] : 0.f;
+            }
+#pragma unroll
+        for (int a = 0; a < 2; ++a)
+#pragma unroll
+          for (int k = 0; k < HT; ++k) {
+            const float* f = src + k * 16 * kHPitch + k16 + 8 * a;
+            uint32_t h0, h1, l0, l1;
+            split_f16(f[0], f[kHPitch], h0, l0);
+            split_f16(f[8 * kHPitch], f[9 * kHPitch], h1, l1);
+#pragma unroll
+            for (int m = 0; m < HT; ++m) mma_f16(o[a][m], ta[m][k], l0, l1);
+#pragma unroll
+            for (int m = 0; m < HT; ++m) mma_f16(o[a][m], ta[m][k], h0, h1);
+          }
 #pragma unroll
         for (int m = 0; m < HT; ++m)
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int h = m * 16 + 8 * (e >> 1);   // (bias_at(g8 + h) = bias_at(g8) + h * pitch)
-            o[a][m][e] = h + g8 < H ? -bb[h * kBiasPitch - k16 - 2 * a - (e & 1)] : 0.f;
-          }
-#pragma unroll
-      for (int a = 0; a < 2; ++a)
-#pragma unroll
-        for (int k = 0; k < HT; ++k) {
-          const float* f = src + k * 16 * kHPitch + k16 + 8 * a;
-          uint32_t h0, h1, l0, l1;
-          split_f16(f[0], f[kHPitch], h0, l0);
-          split_f16(f[8 * kHPitch], f[9 * kHPitch], h1, l1);
-#pragma unroll
-          for (int m = 0; m < HT; ++m) mma_f16(o[a][m], ta[m][k], l0, l1);
-#pragma unroll
-          for (int m = 0; m < HT; ++m) mma_f16(o[a][m], ta[m][k], h0, h1);
-        }
-#pragma unroll
-      for (int m = 0; m < HT; ++m)
-#pragma unroll
-        for (int r = 0; r < 2; ++r)
-          if (m * 16 + 8 * r + g8 < H)
-            *reinterpret_cast<float4*>(dst + static_cast<long long>(m * 16 + 8 * r) * kTile * p.span + k16) =
-                make_float4(o[0][m][2 * r], o[0][m][2 * r + 1], o[1][m][2 * r], o[1][m][2 * r + 1]);
+          for (int r = 0; r < 2; ++r)
+            if (m * 16 + 8 * r + g8 < H)
+              *reinterpret_cast<float4*>(dst + static_cast<long long>(m * 16 + 8 * r) * kTile * p.span + k16) =
+                  make_float4(o[0][m][2 * r], o[0][m][2 * r + 1], o[1][m][2 * r], o[1][m][2 * r + 1]);
+      }
     }
     __syncthreads();
   }
@@ -1077,18 +1079,18 @@ cudaError_t launch_scores(const TalkParams& p, cudaStream_t stream) {
   const size_t smem = scores_smem(p.H, D);
   ensure_dynamic_smem(kern, smem);
   // parts of a piece's keys, so that the CTAs' rounds are shortest (loading the queries costs about one and a half blocks)
-  const int blocks = p.span / kKeys, pieces = p.n_rows * (kTile / kQ), sms = sm_count();
+  const int blocks = p.span / kKeys, pieces = p.n_rows * (kTile / kQ), room = (HM == 16 ? 2 : 1) * sm_count();
   int per = blocks;
   float best = 0.f;
   for (int parts = 1; parts <= 16 && parts <= blocks; ++parts) {
     const int n = (blocks + parts - 1) / parts;
-    const float cost = static_cast<float>((static_cast<long long>(pieces) * parts + sms - 1) / sms) * (n + 1.5f);
+    const float cost = static_cast<float>((static_cast<long long>(pieces) * parts + room - 1) / room) * (n + 1.5f);
     if (parts == 1 || cost < best) {
       best = cost;
       per = n;
     }
   }
-  return launch_kernel(kern, dim3((blocks + per - 1) / per, kTile / kQ, p.n_rows), dim3(kScoreThreads), smem, stream, true, false, p, per);
+  return launch_kernel(kern, dim3((blocks + per - 1) / per, kTile / kQ, p.n_rows), dim3(HM * 16), smem, stream, true, false, p, per);
 }
 template <int D>
 cudaError_t launch_prefill(const CUtensorMap& tmV, const TalkParams& p, cudaStream_t stream) {

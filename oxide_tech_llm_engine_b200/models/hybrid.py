@@ -900,7 +900,8 @@ class HybridModel(GemmShapes):
         w_in[:q.shape[0]], w_in[q.shape[0]:q.shape[0] + k.shape[0]], w_in[a.gate_col:] = q, k, g
         wk = vec(p + "k.norm").view(a.kv_heads, 1, a.dim).expand(a.kv_heads, a.heads // a.kv_heads, a.dim).reshape(-1)
         talk = mat(p + "talk").float().contiguous()      # a matrix: of the model's dtype, like the others
-        far = a.window or 16 * self.max_blocks_per_seq
+        far = 16 * self.max_blocks_per_seq      # no distance is larger
+        far = min(a.window, far) if a.window else far
         return {"w_in": self._pad(w_in), "w_o": self._pad(mat(p + "o")), "rot": self._rotary(None), "q_norm": (vec(p + "q.norm") * wk).contiguous(),
                 "talk": talk, "bias": hops.talk_bias(talk, vec(p + "r1"), vec(p + "r2"), far)}
 

@@ -70,7 +70,8 @@ def mix_sink(c, w, p, h, pos, eps):
     """Rotated grouped attention with a learned sink per head."""
     T, (H, G, D, E) = h.shape[0], (c["heads"], c["kv_heads"], c["dim"], c["vdim"])
     q, k, v = (h @ w[p + "q"].T).view(T, H, D), (h @ w[p + "k"].T).view(T, G, D), (h @ w[p + "v"].T).view(T, G, E)
-    q, k = (rotate(x, pos, c["rot"]["base"], c["rot"]["dims"], True) for x in (q, k))
+    if c.get("rot"):
+        q, k = (rotate(x, pos, c["rot"]["base"], c["rot"]["dims"], True) for x in (q, k))
     a = values_of(masked_softmax(raw_scores(q, k, c["scale"]), c["mask"]["size"], w[p + "sink"]), v)
     return a.reshape(T, H * E) @ w[p + "o"].T
 
